@@ -127,6 +127,12 @@ constexpr int EPI_ROPE = 3;       // fused qkv projection: RoPE on q/k heads, q 
 constexpr int EPI_SWIGLU = 2;     // weight rows interleaved per tile (64 gate rows, then their 64 up rows):
                                   // Y[t, n0/2 + c] = silu(acc[c]) * acc[64 + c], Y has N/2 columns
 constexpr int EPI_GEGLU = 4;      // the same with the tanh form of GELU on the gate (Gemma)
+constexpr int EPI_RELU2 = 5;      // Y = relu(acc + bias)^2 (feed-forward blocks without a gate)
+__device__ __forceinline__ float epi_act(float v, int epi_mode) {
+  if (epi_mode != EPI_RELU2) return v;
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
 
 // RMSNorm folded into the GEMMs around it.  The norm weight is multiplied into the consuming projection's
 // columns when the model is loaded; what remains of the norm is one scalar per token, 1/rms(x_t), which
@@ -379,7 +385,8 @@ struct GroupArgs {
   int l2_prefetch_kb;  // weight k-blocks to request into the L2 before the grid dependency (any launch)
   // Token-gathered groups (mixture-of-experts dispatch): group z multiplies activation rows
   // [row_offsets[z], row_offsets[z + 1]) (device array, written by the upstream kernel) and writes the same rows
-  // of Y; blockIdx.z = z * t_tiles + token tile, and a CTA whose tile lies past the group's rows leaves at once.
+  // of Y; blockIdx.z = z * t_tiles + token tile (in every grouped launch), and a CTA whose tile lies past a gathered
+  // group's rows leaves at once.
   const int* row_offsets;
   int t_tiles;
 };
@@ -418,7 +425,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
                  const QwArgs qw, const GroupArgs gr, const RopeArgs ro, const NormArgs nm) {
   constexpr bool MMQ = QT != QT_BF16;
   const bool gathered = gr.enabled && gr.row_offsets != nullptr;
-  const int zg = gr.enabled ? (gathered ? (int)blockIdx.z / gr.t_tiles : (int)blockIdx.z) : 0;
+  const int zg = gr.enabled ? (int)blockIdx.z / gr.t_tiles : 0;
   int g_row0 = 0;  // first activation / output row of this group (gathered groups)
   if (gathered) {
     pdl_wait();  // the row lists come from the upstream kernel
@@ -480,7 +487,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
   }
   const int n0 = tile_n * GEMM_BM;
   const int split = blockIdx.y;
-  const int t0 = gathered ? ((int)blockIdx.z % gr.t_tiles) * TN : (gr.enabled ? 0 : tile_t * TN);
+  const int t0 = (gr.enabled ? (int)blockIdx.z % gr.t_tiles : tile_t) * TN;
   const int w_row0 = n0 + zg * gr.w_rows;  // first weight row of this tile in the (stacked) matrix
   const int x_row0 = gathered ? g_row0 + t0 : t0 + zg * gr.x_rows;
   const int kb_total = (K + GEMM_BK - 1) / GEMM_BK;
@@ -831,7 +838,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             const float sc = use_nm ? tok_scale[c * 16 + j] : 1.f;
-            stage[(c * 16 + j) * GEMM_BM + row] = __float2bfloat16(__uint_as_float(r[j]) * sc + badd);
+            stage[(c * 16 + j) * GEMM_BM + row] = __float2bfloat16(epi_act(__uint_as_float(r[j]) * sc + badd, epi_mode));
           }
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -854,7 +861,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
             for (int j = 0; j < 16; ++j) {
               const int t = t0 + c * 16 + j;
               if (t < T) {
-                float v = __uint_as_float(r[j]) * (use_nm ? tok_scale[c * 16 + j] : 1.f) + b;
+                float v = epi_act(__uint_as_float(r[j]) * (use_nm ? tok_scale[c * 16 + j] : 1.f) + b, epi_mode);
                 __nv_bfloat16* dst = Y + (size_t)t * ldY + n;
                 if (epi_mode == EPI_ADD_INTO) v += __bfloat162float(*dst);
                 *dst = __float2bfloat16(v);
@@ -887,7 +894,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
         const float badd = use_ar ? 0.f : b;
         const uint32_t a0 = smem_u32(part + row);
         auto emit = [&](int j, float acc) {
-          stage[(j - jb) * GEMM_BM + row] = __float2bfloat16(acc * (use_nm ? tok_scale[j] : 1.f) + badd);
+          stage[(j - jb) * GEMM_BM + row] = __float2bfloat16(epi_act(acc * (use_nm ? tok_scale[j] : 1.f) + badd, epi_mode));
         };
         if (splits <= 2) {
           splitk_reduce_dsmem<8, 2>(a0, splits, jb, je, emit);
@@ -965,7 +972,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant_
           if (use_ar) {
             stage[(j - jb) * GEMM_BM + row] = __float2bfloat16(acc);
           } else if (n < N) {
-            acc += b;
+            acc = epi_act(acc + b, epi_mode);
             __nv_bfloat16* dst = Y + (size_t)(t0 + j) * ldY + n;
             if (epi_mode == EPI_ADD_INTO) acc += __bfloat162float(*dst);
             *dst = __float2bfloat16(acc);
@@ -1152,7 +1159,7 @@ int gemm_launch(const CUtensorMap& tmW, const CUtensorMap& tmX, __nv_bfloat16* Y
     const int mc = gemm_max_cluster<TN, QT>();
     if (splits > mc) splits = mc;
   }
-  dim3 grid(p.n_tiles, splits, gr.enabled ? (gr.row_offsets != nullptr ? groups * gr.t_tiles : groups) : p.t_tiles);
+  dim3 grid(p.n_tiles, splits, gr.enabled ? groups * gr.t_tiles : p.t_tiles);
   const dim3 block(QT == QT_BF16 ? GEMM_THREADS : GEMM_THREADS_MMQ);
   cudaError_t le;
   GroupArgs grl = gr;

@@ -372,6 +372,33 @@ OXB_API int oxb_gemm_grouped(const void* X, int x_rows, const void* W, int qtype
 }
 
 
+// Batched GEMM, any number of tokens: for every group g
+//   Y + g*y_stride [T, N] (row stride ldY) = X[g*T .. (g+1)*T) [T, K] . W[g*N .. (g+1)*N) [N, K]^T   (bf16)
+// (the per-head products around latent attention: X head-major, the heads' results side by side in each row of Y).
+OXB_API int oxb_gemm_batched(const void* X, const void* W, void* Y, long long y_stride, int groups, int T, int N, int K, int ldY,
+                             cudaStream_t stream) {
+  if (T <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
+  if (K % 8 != 0) return (int)cudaErrorInvalidValue;
+  GemmPlan p = gemm_plan(T, N, K, 1, sm_count(), 0, 0, false, groups);
+  CUtensorMap tmW, tmX;
+  int e = oxb_make_tmap_2d(&tmX, X, (uint64_t)groups * T, K, (uint64_t)K * 2, p.tn, GEMM_BK, 2);
+  if (e) return e;
+  e = oxb_make_tmap_2d(&tmW, W, (uint64_t)groups * N, K, (uint64_t)K * 2, GEMM_BM, GEMM_BK, 2);
+  if (e) return e;
+  __nv_bfloat16* y = reinterpret_cast<__nv_bfloat16*>(Y);
+  ArArgs ar;
+  memset(&ar, 0, sizeof(ar));
+  const GroupArgs gr{1, N, T, y_stride, nullptr, 0, 0, nullptr, p.t_tiles};
+  const QwArgs qw{nullptr, 0, nullptr, 0, 0};
+  switch (p.tn) {
+    case 16: return gemm_launch<16>(tmW, tmX, y, nullptr, N, T, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
+    case 32: return gemm_launch<32>(tmW, tmX, y, nullptr, N, T, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
+    case 64: return gemm_launch<64>(tmW, tmX, y, nullptr, N, T, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
+    case 128: return gemm_launch<128>(tmW, tmX, y, nullptr, N, T, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
+    default: return gemm_launch<256>(tmW, tmX, y, nullptr, N, T, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
+  }
+}
+
 // Grouped GEMM over token-gathered groups (mixture-of-experts dispatch): group g multiplies the activation rows
 // [row_offsets[g], row_offsets[g+1]) of X ([rows_cap, K], gathered expert by expert) with its own weights
 // W_g ([N, K] at rows g*N of the stacked matrix) and writes the same rows of Y ([rows_cap, ldY]).  row_offsets is a

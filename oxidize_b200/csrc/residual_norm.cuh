@@ -1,0 +1,134 @@
+// Norm after the sum: x <- norm(alpha * x + y) with the residual stream x in float32, and the same rows in the
+// activation type for the matrix products that follow, in one kernel.  Layer norm (mean removed, weight and bias) or RMS
+// norm; the variance is the mean of the squared deviations, taken in a second pass over the row held in registers.
+#pragma once
+#include "common.cuh"
+
+namespace oxb {
+
+struct ResidualNormArgs {
+  const float* res;  // [T, H] or null
+  const void* y;     // [T, H] in the activation type, or null
+  float alpha;
+  const float *w, *b;  // [H]; b may be null
+  float* x_out;        // [T, H] or null (may be res: the rows are read before they are written)
+  void* a_out;         // [T, H] in the activation type, or null
+  int H;
+  float eps;
+  int layer_norm;  // 1: layer norm, 0: RMS norm
+};
+
+__device__ __forceinline__ float4 rn_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 rn_load4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void rn_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void rn_store4(__nv_bfloat16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+__device__ __forceinline__ float rn_load(const float* p) { return *p; }
+__device__ __forceinline__ float rn_load(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void rn_store(float* p, float v) { *p = v; }
+__device__ __forceinline__ void rn_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+// One CTA per row; every thread owns CH groups of four neighbouring values (H % 4 == 0, H <= 4 * CH * threads).
+template <typename A, int CH>
+__global__ void __launch_bounds__(1024) residual_norm_kernel(const ResidualNormArgs a) {
+  __shared__ float red[32];
+  const int H4 = a.H >> 2;
+  const size_t base = (size_t)blockIdx.x * a.H;
+  float4 v[CH], w[CH], b[CH];
+  pdl_launch_dependents();
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {  // weights are static: fetched ahead of the dependency
+    const int i = threadIdx.x + c * blockDim.x;
+    w[c] = b[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H4) {
+      w[c] = rn_load4(a.w + 4 * i);
+      if (a.b != nullptr) b[c] = rn_load4(a.b + 4 * i);
+    }
+  }
+  pdl_wait();
+  float sum = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H4) {
+      float4 r = v[c], y = v[c];
+      if (a.y != nullptr) y = rn_load4(reinterpret_cast<const A*>(a.y) + base + 4 * i);
+      if (a.res != nullptr) r = rn_load4(a.res + base + 4 * i);
+      v[c] = make_float4(a.alpha * r.x + y.x, a.alpha * r.y + y.y, a.alpha * r.z + y.z, a.alpha * r.w + y.w);
+    }
+    sum += (v[c].x + v[c].y) + (v[c].z + v[c].w);
+  }
+  const float mean = a.layer_norm ? block_sum(sum, red) / (float)a.H : 0.f;
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    if (threadIdx.x + c * blockDim.x < H4) {
+      v[c] = make_float4(v[c].x - mean, v[c].y - mean, v[c].z - mean, v[c].w - mean);
+      ss += (v[c].x * v[c].x + v[c].y * v[c].y) + (v[c].z * v[c].z + v[c].w * v[c].w);
+    }
+  }
+  const float inv = rsqrtf(block_sum(ss, red) / (float)a.H + a.eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    if (i < H4) {
+      const float4 o = make_float4(v[c].x * inv * w[c].x + b[c].x, v[c].y * inv * w[c].y + b[c].y,
+                                   v[c].z * inv * w[c].z + b[c].z, v[c].w * inv * w[c].w + b[c].w);
+      if (a.x_out != nullptr) rn_store4(a.x_out + base + 4 * i, o);
+      if (a.a_out != nullptr) rn_store4(reinterpret_cast<A*>(a.a_out) + base + 4 * i, o);
+    }
+  }
+}
+
+// Any width: the row is staged in shared memory (dynamic, H floats).
+template <typename A>
+__global__ void __launch_bounds__(256) residual_norm_any_kernel(const ResidualNormArgs a) {
+  extern __shared__ float rn_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t base = (size_t)blockIdx.x * a.H;
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    float v = a.res != nullptr ? a.alpha * a.res[base + i] : 0.f;
+    if (a.y != nullptr) v += rn_load(reinterpret_cast<const A*>(a.y) + base + i);
+    rn_row[i] = v;
+    sum += v;
+  }
+  const float mean = a.layer_norm ? block_sum(sum, red) / (float)a.H : 0.f;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    const float v = rn_row[i] - mean;
+    ss += v * v;
+  }
+  const float inv = rsqrtf(block_sum(ss, red) / (float)a.H + a.eps);
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    const float o = (rn_row[i] - mean) * inv * a.w[i] + (a.b != nullptr ? a.b[i] : 0.f);
+    if (a.x_out != nullptr) a.x_out[base + i] = o;
+    if (a.a_out != nullptr) rn_store(reinterpret_cast<A*>(a.a_out) + base + i, o);
+  }
+}
+
+template <typename A>
+int residual_norm_launch(const ResidualNormArgs& a, int T, cudaStream_t stream) {
+  if (a.H % 4 == 0 && a.H <= 16384) {
+    const int H4 = a.H / 4, ch = H4 <= 1024 ? 1 : (H4 <= 2048 ? 2 : 4);
+    const int threads = ((H4 + ch - 1) / ch + 31) / 32 * 32;
+    if (ch == 1) oxb_launch(residual_norm_kernel<A, 1>, dim3(T), dim3(threads), 0, stream, a);
+    else if (ch == 2) oxb_launch(residual_norm_kernel<A, 2>, dim3(T), dim3(threads), 0, stream, a);
+    else oxb_launch(residual_norm_kernel<A, 4>, dim3(T), dim3(threads), 0, stream, a);
+  } else {
+    if (a.H > 12 * 1024) return (int)cudaErrorInvalidValue;  // 48 KB of shared memory
+    oxb_launch(residual_norm_any_kernel<A>, dim3(T), dim3(256), (size_t)a.H * sizeof(float), stream, a);
+  }
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+}  // namespace oxb

@@ -11,6 +11,9 @@ block id here addresses device memory:
                     uint8 codes (q8: head_dim bytes, q4: head_dim/2 bytes)
     scales[layer] : [num_blocks, n_kv_heads, 2, page, head_dim/32] f32   (q8/q4 only)
 
+(latent attention keeps one plane of rows instead of the K / V pair, and the rows of different layers may differ in
+width: ``KVCacheSpec.planes`` / ``row_dims``),
+
 so one (block, head, K) tile of a 16-token page with head_dim 128 is 4 KB contiguous — one
 TMA box / one fully coalesced burst in the attention kernels.
 """
@@ -164,16 +167,24 @@ class KVCacheSpec:
     head_dim: int
     page_size: int = 16
     dtype_name: str = "bf16"
+    planes: int = 2  # rows per token and head: K and V, or one shared (latent) row
+    row_dims: Optional[Tuple[int, ...]] = None  # row width of each layer where they differ (else head_dim everywhere)
+
+    def row_dim(self, layer: int) -> int:
+        return self.head_dim if self.row_dims is None else self.row_dims[layer]
 
     def bytes_per_block(self) -> int:
-        e = self.n_kv_heads * 2 * self.page_size
-        if self.dtype_name == "q8":
-            per = e * (self.head_dim + self.head_dim // 32 * 4)
-        elif self.dtype_name == "q4":
-            per = e * (self.head_dim // 2 + self.head_dim // 32 * 4)
-        else:
-            per = e * self.head_dim * torch.empty(0, dtype=KV_DTYPES[self.dtype_name]).element_size()
-        return per * self.n_layers
+        e = self.n_kv_heads * self.planes * self.page_size
+        total = 0
+        for l in range(self.n_layers):
+            d = self.row_dim(l)
+            if self.dtype_name == "q8":
+                total += e * (d + d // 32 * 4)
+            elif self.dtype_name == "q4":
+                total += e * (d // 2 + d // 32 * 4)
+            else:
+                total += e * d * torch.empty(0, dtype=KV_DTYPES[self.dtype_name]).element_size()
+        return total
 
 
 class KVCache:
@@ -182,21 +193,20 @@ class KVCache:
     def __init__(self, spec: KVCacheSpec, num_blocks: int, device="cpu"):
         if spec.dtype_name not in KV_DTYPES:
             raise ValueError(f"kv dtype must be one of {sorted(KV_DTYPES)}")
-        if spec.dtype_name in ("q8", "q4") and spec.head_dim % 32:
+        dims = [spec.row_dim(l) for l in range(spec.n_layers)]
+        if spec.dtype_name in ("q8", "q4") and any(d % 32 for d in dims):
             raise ValueError("quantized KV needs head_dim % 32 == 0")
         self.spec = spec
         self.num_blocks = num_blocks
         self.page_size = spec.page_size
         self.dtype_name = spec.dtype_name
         self.device = torch.device(device)
-        hd = spec.head_dim
-        inner = hd if spec.dtype_name != "q4" else hd // 2
-        shape = (num_blocks, spec.n_kv_heads, 2, spec.page_size, inner)
-        self.data = [torch.zeros(shape, dtype=KV_DTYPES[spec.dtype_name], device=self.device) for _ in range(spec.n_layers)]
+        lead = (num_blocks, spec.n_kv_heads, spec.planes, spec.page_size)
+        self.data = [torch.zeros(lead + (d if spec.dtype_name != "q4" else d // 2,), dtype=KV_DTYPES[spec.dtype_name],
+                                 device=self.device) for d in dims]
         self.scales: List[Optional[torch.Tensor]] = [None] * spec.n_layers
         if spec.dtype_name in ("q8", "q4"):
-            sshape = (num_blocks, spec.n_kv_heads, 2, spec.page_size, hd // 32)
-            self.scales = [torch.zeros(sshape, dtype=torch.float32, device=self.device) for _ in range(spec.n_layers)]
+            self.scales = [torch.zeros(lead + (d // 32,), dtype=torch.float32, device=self.device) for d in dims]
 
     def copy_block(self, src: int, dst: int) -> None:
         """Copy-on-write support: duplicate one page in every layer."""

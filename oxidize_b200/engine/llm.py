@@ -16,12 +16,13 @@ from typing import Callable, Dict, Iterable, List, Optional, Sequence as Seq, Un
 
 import torch
 
-from ..formats.gguf import GGUFFile, load_gguf
-from ..models.config import ModelConfig, config_from_gguf
+from ..formats.layered import Checkpoint, open_checkpoint
+from ..models.config import ModelConfig
+from ..models.registry import act_dtype_for, config_from_checkpoint, load_checkpoint_weights
 from ..models.transformer import Transformer
-from ..models.weights import ModelWeights, load_weights
+from ..models.weights import ModelWeights
 from ..utils import profiler as _profiler
-from .kv_pool import BlockPool, KVCache, KVCacheSpec, make_block_pool
+from .kv_pool import BlockPool, KVCacheSpec, make_block_pool
 from .runner import ModelRunner, StepResult
 from .sampler import SamplingParams
 from .scheduler import ScheduledSeq, Scheduler, SchedulerConfig, SchedulerOutput, Sequence
@@ -56,6 +57,9 @@ class EngineConfig:
     fuse_swiglu: bool = True  # SiLU(gate) * up as the gate_up GEMM's epilogue for dense bf16 FFNs
     kernel_options: Optional[object] = None  # ops.cuda.KernelOptions; None = the library's defaults
     eos_token_id: Optional[int] = None
+    # auto: bfloat16 activations and matrix products on the GPU, float32 on the CPU.  f32: float32 on the GPU as well (no
+    # reduced-precision products); available for the models whose device kernels all exist in that type.
+    compute_dtype: str = "auto"  # auto | bf16 | f32
     # > 0: keep only this many decoder layers loaded, streaming the others from the file mapping as the forward pass
     # reaches them (for checkpoints larger than the memory left beside the KV cache)
     resident_layers: int = 0
@@ -95,13 +99,14 @@ class LLM:
 
             _opcuda.configure(c.kernel_options)
         self.model = Transformer(weights, comm, fold_norms=c.fold_norms, fuse_qkv_rope=c.fuse_qkv_rope,
-                                 fuse_swiglu=c.fuse_swiglu, pipe=pipe, max_context=c.max_model_len)
+                                 fuse_swiglu=c.fuse_swiglu, pipe=pipe, max_context=c.max_model_len,
+                                 act_dtype=torch.float32 if c.compute_dtype == "f32" else None)
         self.device = self.model.device
         self.tokenizer = tokenizer
         kv_dtype = c.kv_cache_dtype
         if kv_dtype == "auto":
-            kv_dtype = "bf16" if self.device.type == "cuda" else "f32"
-        spec = KVCacheSpec(max(1, self.model.n_kv_layers), self.model.n_kv_local, self.model.kv_head_dim, c.kv_page_size, kv_dtype)
+            kv_dtype = "bf16" if self.model.act_dtype == torch.bfloat16 else "f32"
+        spec = self.model.cache_spec(c.kv_page_size, kv_dtype)
         # (a hybrid model's convolution layers keep one hidden-sized row per token as well)
         conv_bytes = self.model.n_conv_layers * c.kv_page_size * self.cfg.hidden_size * (2 if self.device.type == "cuda" else 4)
         nblocks = c.num_kv_blocks or self._auto_blocks(spec, conv_bytes)
@@ -110,9 +115,8 @@ class LLM:
         prefix_cache = c.enable_prefix_cache and not self.cfg.is_ssm
         self.pool = make_block_pool(nblocks, c.kv_page_size, prefix_cache)
         # a window that applies to every layer lets the scheduler hand pages back as they fall out of it
-        uniform_window = self.cfg.sliding_window if (self.cfg.sliding_window > 0 and self.cfg.sliding_window_pattern == 0) else 0
         self.scheduler = Scheduler(SchedulerConfig(c.max_num_batched_tokens, c.prefill_chunk_size, c.max_num_seqs,
-                                                   c.policy, prefix_cache, c.max_model_len, uniform_window), self.pool)
+                                                   c.policy, prefix_cache, c.max_model_len, self.cfg.uniform_window), self.pool)
         self.runner = ModelRunner(self.model, self.kv, max(c.max_num_batched_tokens, c.max_num_seqs), c.max_num_seqs,
                                   c.max_model_len, c.cuda_graphs and not _profiler.PROFILE and not _profiler.TRACE_FWD
                                   and isinstance(weights.layers, list)  # a captured graph would pin evicted layers' addresses
@@ -127,14 +131,15 @@ class LLM:
 
     # ------------------------------------------------------------------ construction helpers
     @classmethod
-    def from_gguf(cls, path: Union[str, GGUFFile], config: Optional[EngineConfig] = None, device=None, comm=None,
+    def from_gguf(cls, path: Union[str, Checkpoint], config: Optional[EngineConfig] = None, device=None, comm=None,
                   tp_rank: int = 0, ep_rank: int = 0, rope_pairing: Optional[str] = None, pipe=None,
                   experts_per_token: int = 0) -> "LLM":
+        """An engine over a checkpoint: a GGUF file, or a directory that lists its layers (``formats.layered``)."""
         from ..formats.tokenizer import TokenizerError, load_tokenizer_from_metadata
 
         config = config or EngineConfig()
-        g = path if isinstance(path, GGUFFile) else load_gguf(path)
-        cfg = config_from_gguf(g)
+        g = open_checkpoint(path) if isinstance(path, str) else path
+        cfg = config_from_checkpoint(g)
         if rope_pairing:
             cfg.rope_pairing = rope_pairing
         if experts_per_token:
@@ -143,7 +148,7 @@ class LLM:
                 raise ValueError(f"experts_per_token must be between 1 and the model's {cfg.n_experts} experts")
             cfg.n_experts_used = experts_per_token
         device = torch.device(device if device is not None else ("cuda" if torch.cuda.is_available() else "cpu"))
-        act = torch.bfloat16 if device.type == "cuda" else torch.float32
+        act = act_dtype_for(cfg, device, config.compute_dtype)
         ep_size = config.ep_size or config.tp_size
         if ep_size == config.tp_size and ep_rank == 0:
             ep_rank = tp_rank  # the expert partition follows the tensor-parallel rank
@@ -156,8 +161,8 @@ class LLM:
             if pipe is None:
                 raise ValueError("pp_size > 1 needs the stage's StageIO")
             layer_range = split_layers(cfg.n_layers, config.pp_size)[pipe.rank]
-        w = load_weights(g, cfg, device, act, tp_rank, config.tp_size, ep_rank, ep_size, layer_range=layer_range,
-                         resident_layers=config.resident_layers, transcode=config.weight_transcode)
+        w = load_checkpoint_weights(g, cfg, device, act, tp_rank, config.tp_size, ep_rank, ep_size, layer_range=layer_range,
+                                    resident_layers=config.resident_layers, transcode=config.weight_transcode)
         try:
             tok = load_tokenizer_from_metadata(g.metadata)
         except TokenizerError:
@@ -167,6 +172,8 @@ class LLM:
 
         llm.chat_template = chat_template_from_metadata(g.metadata)  # None when the file carries none
         return llm
+
+    from_checkpoint = from_gguf
 
     def _auto_blocks(self, spec: KVCacheSpec, extra_bytes_per_block: int = 0) -> int:
         c = self.config
@@ -450,10 +457,8 @@ class LLM:
             meta = BatchMeta(torch.tensor(ids, **i32), pos, pos.clone(), torch.tensor([0, n], **i32), torch.tensor([n], **i32),
                              torch.arange(nblk, **i32)[None, :], torch.arange(n, **i32), n, n, 1, logits_all=True)
             h, residual = m.run_layers(m.embed(meta.token_ids), None, meta, kv)
-            from .. import ops
-
             m.release_state(kv)
-            x = ops.add_rmsnorm(h, residual, m.w.out_norm, m.cfg.rms_eps)[0].float()
+            x = m.final_norm(h, residual)[0].float()
             v = x.mean(dim=0) if pooling == "mean" else x[-1]
             if normalize:
                 v = v / v.norm().clamp_min(1e-12)

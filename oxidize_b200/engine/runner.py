@@ -168,7 +168,10 @@ class ModelRunner:
                 slot[t] = blist[start // ps] * ps + start % ps
                 sl[i] = start + 1
                 qs[i + 1] = t + 1
-                if ss.sample:
+                if ss.want is not None:
+                    li[nl : nl + len(ss.want)] = t
+                    nl += len(ss.want)
+                elif ss.sample:
                     li[nl] = t
                     rows.append((ss, nl, 1))
                     nl += 1
@@ -189,7 +192,10 @@ class ModelRunner:
             slot[t : t + n] = cache[2][p // ps] * ps + p % ps
             sl[i] = start + n
             qs[i + 1] = t + n
-            if ss.sample:
+            if ss.want is not None:
+                li[nl : nl + len(ss.want)] = [t + r for r in ss.want]
+                nl += len(ss.want)
+            elif ss.sample:
                 k = n if (not ss.is_prefill and n > 1) else 1
                 li[nl : nl + k] = np.arange(t + n - k, t + n, dtype=np.int32)
                 rows.append((ss, nl, k))
@@ -322,6 +328,17 @@ class ModelRunner:
                                              torch.stack(vecs).to(self.device))
 
     # ------------------------------------------------------------------ execution
+    def score(self, out: SchedulerOutput) -> torch.Tensor:
+        """One step that samples nothing: logits [n, vocab] of the rows its entries want (``ScheduledSeq.want``), in order."""
+        for src, dst in out.cow_copies:
+            self.kv.copy_block(src, dst)
+        self.buf.flip()
+        T, B, nl, max_q, max_len, _ = self.build(out.scheduled)
+        self.buf.upload()
+        meta = self._meta(T, B, nl, max_q, max_len)
+        meta.host_lens = [(ss.num_tokens, ss.start + ss.num_tokens) for ss in out.scheduled]
+        return self.model.forward(meta, self.kv)
+
     def _forward_sample(self, meta: BatchMeta, all_greedy: bool, tie: str, feed: Optional[torch.Tensor] = None):
         if all_greedy and not self.keep_logits:
             return self.model.greedy_tokens(meta, self.kv, tie, feed=feed), None
@@ -409,6 +426,7 @@ class ModelRunner:
             meta = self._meta(T, B, nl, max_q, max_len, logits_all=decode_only and nl == T)
             if not decode_only:
                 self._embed_overrides(scheduled, meta)
+                meta.host_lens = [(ss.num_tokens, ss.start + ss.num_tokens) for ss in scheduled]
             toks, logits = self._forward_sample(meta, all_greedy and not needs_host_logits, tie,
                                                 feed=feed if not needs_host_logits else None)
         if toks is None:  # not the last pipeline stage

@@ -20,7 +20,7 @@ import enum
 import itertools
 from collections import deque
 from dataclasses import dataclass, field
-from typing import Deque, Dict, List, Optional, Sequence, Tuple
+from typing import Deque, Dict, Iterable, List, Optional, Sequence, Tuple
 
 from .kv_pool import FNV_OFFSET, BlockPool, OutOfBlocks, block_hash
 from .sampler import RequestRng, SamplingParams
@@ -104,6 +104,7 @@ class ScheduledSeq:
     num_tokens: int  # rows fed this step
     is_prefill: bool
     sample: bool  # whether the last row's logits are sampled
+    want: Optional[List[int]] = None  # rows (of num_tokens) whose logits the caller reads; None = what sampling needs
 
 
 @dataclass
@@ -315,6 +316,39 @@ class Scheduler:
             out.num_prefill_tokens += chunk
         self.waiting = still
         return out
+
+    def schedule_portions(self, portions: Iterable[Tuple[Sequence, int, List[int]]]) -> SchedulerOutput:
+        """A step whose content the caller decides: ``portions`` are (sequence, number of its tokens to feed, rows whose
+        logits are wanted), the tokens being the next ones of the sequence's prompt.  Unknown sequences are admitted,
+        blocks come from the pool as in :meth:`schedule`; nothing is sampled and nobody is preempted."""
+        out = SchedulerOutput([])
+        for seq, n, want in portions:
+            if seq.status is SeqStatus.WAITING:
+                if len(self.running) >= self.config.max_num_running_seqs:
+                    raise RuntimeError(f"more than {self.config.max_num_running_seqs} sequences at a time")
+                seq.status = SeqStatus.RUNNING
+                self.running.append(seq)
+            start = seq.num_computed
+            if n < 1 or start + n > len(seq.prompt):
+                raise ValueError(f"sequence {seq.request_id} has {len(seq.prompt) - start} tokens left, {n} were asked for")
+            if not self._ensure_blocks(seq, start + n, out):
+                raise OutOfBlocks(f"no KV blocks left for sequence {seq.request_id}")
+            decode = n == 1 and start > 0
+            out.scheduled.append(ScheduledSeq(seq, start, n, not decode, False, list(want)))
+            if decode:
+                out.num_decode_tokens += 1
+            else:
+                out.num_prefill_tokens += n
+        if out.total_tokens > self.config.max_num_batched_tokens:
+            raise RuntimeError(f"{out.total_tokens} tokens in one step, the limit is {self.config.max_num_batched_tokens}")
+        return out
+
+    def finish_portions(self, out: SchedulerOutput) -> None:
+        """Advance the sequences of a :meth:`schedule_portions` step (after its forward pass)."""
+        for ss in out.scheduled:
+            ss.seq.num_computed = ss.start + ss.num_tokens
+            if self.config.attention_window > 0:
+                self._release_outside_window(ss.seq)
 
     def _pick_victim(self, exclude: Sequence) -> Optional[Sequence]:
         for s in reversed(self.running):

@@ -61,6 +61,69 @@ class RopeScaling:
     original_context_length: int = 0
     beta_fast: float = 32.0
     beta_slow: float = 1.0
+    # YaRN: the largest pair index at which the ramp between kept and interpolated frequencies may end; 0 = the last pair
+    ramp_limit: int = 0
+    magnitude: float = 0.0  # factor on cos and sin; 0 = the rule of the scaling type
+
+
+@dataclass
+class RotarySpec:
+    """Rotation of one layer's positional dimensions: ``dims`` of them, frequencies ``base ** (-2 i / dims)``."""
+
+    dims: int
+    base: float
+    scaling: Optional[RopeScaling] = None
+    pairing: str = "split_half"
+
+
+@dataclass
+class LatentAttentionSpec:
+    """Attention over one shared latent row per token, with the geometry of a single layer.
+
+    A cached row is [latent (kv_rank), rotated key (rope_dim)]; per head the key is (W_uk latent, rotated key) and the
+    value W_uv latent.  ``window`` > 0 limits a query to that many latest positions (itself included); ``sink`` adds a
+    learned per-head logit to the softmax denominator only; ``kv_from`` names an earlier layer whose cached rows this
+    layer attends over instead of writing its own."""
+
+    heads: int
+    nope_dim: int
+    rope_dim: int
+    v_dim: int
+    kv_rank: int
+    scale: float
+    rotary: RotarySpec
+    window: int = 0
+    sink: bool = False
+    kv_from: Optional[int] = None
+
+    # The two parts of a row start on multiples of 16 values (one tensor-core k-step, a 16-byte copy); the padding is zero.
+    @property
+    def latent_pad(self) -> int:
+        return (self.kv_rank + 15) // 16 * 16
+
+    @property
+    def row_dim(self) -> int:
+        return self.latent_pad + (self.rope_dim + 15) // 16 * 16
+
+    @property
+    def qk_dim(self) -> int:
+        return self.nope_dim + self.rope_dim
+
+
+@dataclass
+class FeedForwardSpec:
+    """W_down act(W_up x): a feed-forward block without a gate projection."""
+
+    size: int
+    act: str = "relu2"  # the square of relu
+
+
+@dataclass
+class LayerSpec:
+    """One decoder layer of a model whose layers are listed one by one."""
+
+    mixer: LatentAttentionSpec
+    ffn: Optional[FeedForwardSpec] = None  # None: the layer has no feed-forward block
 
 
 @dataclass
@@ -143,6 +206,14 @@ class ModelConfig:
     router_bias: bool = False
     # multi-token prediction (in-GGUF nextn layers appended after the decoder stack)
     nextn_layers: int = 0
+    # Models that describe every layer on its own (each with its own geometry, window and rotation): one entry per layer,
+    # in place of the uniform attention / feed-forward fields above.
+    layer_specs: List[LayerSpec] = field(default_factory=list)
+    norm_kind: str = "rms"  # rms | layer (mean removed, weight and bias)
+    # > 0: norm after the sum, x <- norm(residual_alpha * x + branch(x)), with the residual stream in float32;
+    # 0: norm in front of the branch, x <- x + branch(norm(x))
+    residual_alpha: float = 0.0
+    embed_norm: bool = False  # the embedding passes a norm of its own
 
     @property
     def is_moe(self) -> bool:
@@ -151,6 +222,23 @@ class ModelConfig:
     @property
     def is_mla(self) -> bool:
         return self.kv_lora_rank > 0
+
+    @property
+    def is_layered(self) -> bool:
+        return bool(self.layer_specs)
+
+    @property
+    def cache_rows(self) -> List[int]:
+        """Widths of the cached rows of a layered model, one per layer that owns cache rows (in layer order)."""
+        return [l.mixer.row_dim for l in self.layer_specs if l.mixer.kv_from is None]
+
+    @property
+    def uniform_window(self) -> int:
+        """> 0 when every layer is windowed: no query of any layer looks back further than this."""
+        if self.layer_specs:
+            ws = [l.mixer.window for l in self.layer_specs]
+            return max(ws) if min(ws) > 0 else 0
+        return self.sliding_window if (self.sliding_window > 0 and self.sliding_window_pattern == 0) else 0
 
     @property
     def is_ssm(self) -> bool:
@@ -181,6 +269,14 @@ class ModelConfig:
 
     def param_count(self) -> int:
         h = self.hidden_size
+        if self.layer_specs:
+            n = 2 * self.vocab_size * h + (4 if self.norm_kind == "layer" else 2) * h
+            for l in self.layer_specs:
+                m, f = l.mixer, l.ffn
+                n += m.heads * (h * (m.qk_dim + m.v_dim) + m.kv_rank * (m.nope_dim + m.v_dim) + int(m.sink)) + 2 * h
+                n += 0 if m.kv_from is not None else h * (m.kv_rank + m.rope_dim) + m.kv_rank
+                n += 0 if f is None else 2 * h * f.size + 2 * h
+            return n
         attn = h * self.q_size * 2 + h * self.kv_size * 2
         dense = 3 * h * self.ffn_size
         n = 0

@@ -36,6 +36,7 @@ class RopeState:
     n_heads: int  # local (this rank's) head counts
     n_kv_heads: int
     head_dim: int
+    max_pos: int = 0  # positions the device's cos / sin table must reach (0 = its default)
 
 
 @dataclass
@@ -55,6 +56,9 @@ class BatchMeta:
     logits_all: bool = False  # logits_indices is the identity (every row is a logits row): no row gather needed
     # host copies for CPU-side loops (reference path); optional on the GPU path
     extra: dict = field(default_factory=dict)
+    # (rows fed, context length) of every sequence, known on the host for steps that are built eagerly; kernels that prepare
+    # whole contexts (latent attention over long portions) size their work from it
+    host_lens: Optional[List[Tuple[int, int]]] = None
 
 
 class SingleRankComm:
@@ -141,6 +145,8 @@ class Transformer:
         self._ssm_clock = 0
         if cfg.ssm_d_inner > 0:
             self.n_kv_layers = 0
+        if cfg.is_layered:
+            self._init_layered(max_context or cfg.context_length)
         if cfg.is_mla:
             # One cached row per token, shared by all heads: the normalised latent followed by the rotary key.
             self.n_kv_local = 1
@@ -162,6 +168,37 @@ class Transformer:
             self._interleave_gate_up()
         if dev.type == "cuda" and fold_norms and not streamed:
             self._fold_norm_weights()
+
+    def _init_layered(self, max_context: int) -> None:
+        """Per-layer state of a model that lists its layers: rotations (one per distinct setting) and which cache layer a
+        decoder layer reads (its own, or the one of the layer it takes its rows from)."""
+        cfg = self.cfg
+        if self.pipe is not None:
+            raise ValueError("a model with per-layer geometry runs as one pipeline stage (layers may share cached rows)")
+        ropes: dict = {}
+        self.layer_ropes: List[RopeState] = []
+        owners = [i for i, l in enumerate(cfg.layer_specs) if l.mixer.kv_from is None]
+        self.kv_index = []
+        for i, l in enumerate(cfg.layer_specs):
+            r = l.mixer.rotary
+            key = repr(r)
+            if key not in ropes:
+                ropes[key] = RopeState(
+                    inv_freq=opref.rope_inv_freq(r.dims, r.base, r.scaling, device=self.device, dtype=torch.float64),
+                    pairing=r.pairing, mscale=opref.rope_mscale(r.scaling), n_heads=0, n_kv_heads=1, head_dim=r.dims,
+                    max_pos=min(max_context, 1 << 20))
+            self.layer_ropes.append(ropes[key])
+            self.kv_index.append(owners.index(i if l.mixer.kv_from is None else l.mixer.kv_from))
+        self.n_kv_layers, self.n_kv_local, self.kv_head_dim = len(owners), 1, cfg.head_dim
+
+    def cache_spec(self, page_size: int, dtype_name: str):
+        """Shape of this model's paged cache: K / V rows of the attention layers, or latent rows (one plane; of each
+        layer's own width where the layers are listed one by one)."""
+        from ..engine.kv_pool import KVCacheSpec
+
+        layered = self.cfg.is_layered
+        return KVCacheSpec(max(1, self.n_kv_layers), self.n_kv_local, self.kv_head_dim, page_size, dtype_name,
+                           planes=1 if layered else 2, row_dims=tuple(self.cfg.cache_rows) if layered else None)
 
     def _fold_norm_weights(self) -> None:
         """Fold the two RMSNorm weight vectors of a dense bf16 layer into the columns of the projections that
@@ -257,8 +294,7 @@ class Transformer:
         (same pages, same block ids) whose rows are the convolution layers' gated inputs, split over its K and V halves."""
         from ..engine.kv_pool import KVCache, KVCacheSpec
 
-        kv = KVCache(KVCacheSpec(max(1, self.n_kv_layers), self.n_kv_local, self.kv_head_dim, page_size, dtype_name),
-                     num_blocks, self.device)
+        kv = KVCache(self.cache_spec(page_size, dtype_name), num_blocks, self.device)
         if self.n_conv_layers:
             if self.cfg.hidden_size % 2:
                 raise ValueError("convolution layers need an even hidden size")
@@ -426,6 +462,38 @@ class Transformer:
             acc = acc + w[:, L - 1 - j] * prev * ok[:, None]
         return ops.linear((gate_c * acc).to(x.dtype), lw.conv_out)
 
+    def _layers_norm_after(self, h: torch.Tensor, meta: BatchMeta, kv, lo: int, hi: int, capture: Optional[dict]):
+        """Layers whose norm acts after the sum, x <- norm(alpha x + branch(x)): the stream ``x`` stays in float32, the
+        branches read it in the activation type (written by the same norm kernel)."""
+        cfg = self.cfg
+        alpha, eps, kind = cfg.residual_alpha, cfg.rms_eps, cfg.norm_kind
+        if lo == 0 and cfg.embed_norm:
+            x, xa = ops.residual_norm(None, h, 1.0, self.w.embed_norm, self.w.embed_norm_bias, eps, kind, self.act_dtype)
+        else:
+            x, xa = h.float(), h.to(self.act_dtype)
+        for li in range(lo, hi):
+            lw, spec = self.w.layers[li], cfg.layer_specs[self.w.first_layer + li]
+            o = ops.latent_mixer(xa, lw.mla, spec.mixer, self.layer_ropes[li], meta, kv, self.kv_index[li], eps)
+            x, xa = ops.residual_norm(x, self.comm.linear_allreduce(o, lw.wo), alpha, lw.attn_norm, lw.attn_norm_bias, eps, kind,
+                                      self.act_dtype)
+            if spec.ffn is not None:
+                a = ops.linear_act(xa, lw.w_up, spec.ffn.act)
+                x, xa = ops.residual_norm(x, self.comm.linear_allreduce(a, lw.w_down), alpha, lw.ffn_norm, lw.ffn_norm_bias, eps,
+                                          kind, self.act_dtype)
+            if capture is not None and self.w.first_layer + li in capture.get("layers", ()):
+                capture.setdefault("hidden", {})[self.w.first_layer + li] = x.clone()
+            if _profiler.TRACE_FWD:
+                _profiler.trace_hidden(self.w.first_layer + li, x, None)
+        return x, None
+
+    def final_norm(self, h: torch.Tensor, residual: Optional[torch.Tensor]):
+        """(normed rows for the output head, the hidden state in front of that norm)."""
+        cfg = self.cfg
+        if cfg.is_layered:
+            return ops.residual_norm(h, None, 1.0, self.w.out_norm, self.w.out_norm_bias, cfg.rms_eps, cfg.norm_kind,
+                                     self.act_dtype, keep_stream=False)[1], h
+        return ops.add_rmsnorm(h, residual, self.w.out_norm, cfg.rms_eps)
+
     def _layer_rope(self, window: int) -> RopeState:
         """Rotary state of a layer: windowed layers use their own base when the model has one."""
         return self.rope_swa if (window > 0 and self.rope_swa is not None) else self.rope
@@ -554,6 +622,8 @@ class Transformer:
         """Run local layers; returns (h, residual) where the true hidden is h + residual."""
         cfg = self.cfg
         lo, hi = layers if layers is not None else (0, len(self.w.layers))
+        if cfg.is_layered:
+            return self._layers_norm_after(h, meta, kv, lo, hi, capture)
         acc, cur = None, 0  # per-token sum-of-squares accumulators of the residual stream while it is in folded form
         for li in range(lo, hi):
             lw = self.w.layers[li]
@@ -642,7 +712,7 @@ class Transformer:
             idx = logits_indices.long()
             h = h.index_select(0, idx)
             residual = residual.index_select(0, idx) if residual is not None else None
-        x, hidden = ops.add_rmsnorm(h, residual, self.w.out_norm, self.cfg.rms_eps)
+        x, hidden = self.final_norm(h, residual)
         logits = ops.linear(x, self.w.lm_head).float()
         if self.w.tp_size > 1 and self.w.lm_head.out_features != self.cfg.vocab_size:
             logits = self.comm.all_gather_cat(logits, dim=-1)
@@ -667,7 +737,7 @@ class Transformer:
             h = h.index_select(0, idx)
             residual = residual.index_select(0, idx) if residual is not None else None
         self._keep_features(cap, idx)
-        x, hid = ops.add_rmsnorm(h, residual, self.w.out_norm, self.cfg.rms_eps)
+        x, hid = self.final_norm(h, residual)
         self.last_hidden = hid  # pre-norm hidden of the logits rows (input of an MTP head)
         logits = ops.linear(x, self.w.lm_head)
         sharded = self.w.tp_size > 1 and self.w.lm_head.out_features != self.cfg.vocab_size

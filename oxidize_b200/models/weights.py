@@ -168,14 +168,17 @@ class MLAWeights:
     per head and dense, split into its key part ``w_uk`` and value part ``w_uv``: the forward pass multiplies the queries
     by ``w_uk`` and the attention output by ``w_uv`` instead of rebuilding per-head keys and values."""
 
-    kv_a: QTensor  # [kv_lora + rope, hidden]: latent and the shared rotary key
-    kv_a_norm: torch.Tensor
+    # [kv_lora + rope, hidden]: latent and the shared rotary key; None where its rows follow the query rows in ``q``, or
+    # where the layer reads another layer's cached rows
+    kv_a: Optional[QTensor]
+    kv_a_norm: Optional[torch.Tensor]
     w_uk: torch.Tensor  # [heads, nope, kv_lora]
     w_uv: torch.Tensor  # [heads, v, kv_lora]
     q: Optional[LinearWeight] = None  # full query projection, or
     q_a: Optional[QTensor] = None  # down-projection,
     q_a_norm: Optional[torch.Tensor] = None
     q_b: Optional[LinearWeight] = None  # up-projection [heads * (nope + rope), q_lora]
+    sink: Optional[torch.Tensor] = None  # [heads] logits that join the softmax denominator only
 
 
 @dataclass
@@ -233,6 +236,10 @@ class LayerWeights:
     # dense FFN
     w_gate_up: Optional[LinearWeight] = None
     w_down: Optional[LinearWeight] = None
+    w_up: Optional[LinearWeight] = None  # feed-forward block without a gate (w_gate_up is None)
+    # layer norms with a bias (``attn_norm`` / ``ffn_norm`` then act after the mixer's / the block's sum)
+    attn_norm_bias: Optional[torch.Tensor] = None
+    ffn_norm_bias: Optional[torch.Tensor] = None
     # MoE
     router: Optional[QTensor] = None
     router_bias: Optional[torch.Tensor] = None
@@ -320,11 +327,14 @@ class ModelWeights:
     # Phi-3 LongRoPE ``rope_factors_short / _long.weight``), or None
     rope_freq_factors: Optional[torch.Tensor] = None
     rope_freq_factors_long: Optional[torch.Tensor] = None  # LongRoPE: used instead once the context exceeds the original one
+    out_norm_bias: Optional[torch.Tensor] = None
+    embed_norm: Optional[torch.Tensor] = None  # norm on the embedding rows (ModelConfig.embed_norm)
+    embed_norm_bias: Optional[torch.Tensor] = None
 
     def nbytes(self) -> int:
         n = self.embed.nbytes() + self.lm_head.nbytes()
         for l in (self.layers.resident() if isinstance(self.layers, StreamedLayers) else self.layers):
-            for lw in (l.wqkv, l.wo, l.w_gate_up, l.w_down, l.shared_gate_up, l.shared_down):
+            for lw in (l.wqkv, l.wo, l.w_gate_up, l.w_up, l.w_down, l.shared_gate_up, l.shared_down):
                 if lw is not None:
                     n += lw.nbytes()
             if l.experts is not None:

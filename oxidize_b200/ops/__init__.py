@@ -21,6 +21,12 @@ def _cuda():
     return _c
 
 
+def _cuda_latent():
+    from . import cuda_latent as _c
+
+    return _c
+
+
 @instrument("linear")
 def linear(x: torch.Tensor, w, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y = x @ W^T (+bias) for a :class:`LinearWeight` (row segments concatenated) or a QTensor."""
@@ -30,6 +36,8 @@ def linear(x: torch.Tensor, w, bias: Optional[torch.Tensor] = None, out: Optiona
     else:
         bias = w.bias if bias is None else bias
     if x.is_cuda:
+        if x.dtype == torch.float32 and all(p.qtype == "F32" for p in parts):
+            return _cuda_latent().linear_f32(x, parts, bias, out)
         return _cuda().linear(x, parts, bias, out)
     ys = [ref.linear(x, p) for p in parts]
     y = ys[0] if len(ys) == 1 else torch.cat(ys, dim=-1)
@@ -104,6 +112,36 @@ def paged_attention(q, kv, layer, meta, scale, sliding_window=0, softcap=0.0):
     if q.is_cuda:
         return _cuda().paged_attention(q, kv, layer, meta, scale, sliding_window, softcap=softcap)
     return ref.paged_attention(q, kv, layer, meta, scale, sliding_window, softcap)
+
+
+@instrument("residual_norm")
+def residual_norm(res, y, alpha, w, b, eps, kind="layer", act_dtype=torch.float32, keep_stream=True):
+    """norm(alpha * res + y) computed in float32: (the new float32 stream, the same in ``act_dtype``).  ``res`` (float32) or
+    ``y`` may be None; without ``keep_stream`` the caller wants the second result only."""
+    if w.is_cuda:
+        return _cuda_latent().residual_norm(res, y, alpha, w, b, eps, kind, act_dtype, keep_stream)
+    return ref.residual_norm(res, y, alpha, w, b, eps, kind, act_dtype)
+
+
+@instrument("linear_act")
+def linear_act(x, w, act):
+    """act(x @ W^T): the up projection of a feed-forward block without a gate."""
+    if x.is_cuda:
+        return _cuda_latent().linear_act(x, w, act)
+    return ref.activation(linear(x, w), act)
+
+
+@instrument("latent_mixer")
+def latent_mixer(x, m, spec, rope, meta, kv, layer, eps):
+    """Latent attention of one layer up to (not including) its output projection: [T, heads * v_dim].  ``m`` holds the
+    projections (``models.weights.MLAWeights``), ``spec`` the geometry (``models.config.LatentAttentionSpec``); the cache
+    layer receives this step's rows unless the layer reads another layer's."""
+    if x.is_cuda:
+        return _cuda_latent().latent_mixer(x, m, spec, rope, meta, kv, layer, eps)
+    qkv = linear(x, m.q)
+    q = ref.latent_rows(qkv, m, spec, rope, meta, kv, layer, eps)
+    o = ref.latent_attention(q, kv, layer, meta, spec.scale, spec.kv_rank, spec.window, m.sink)
+    return torch.einsum("thc,hvc->thv", o.float(), m.w_uv.float()).to(x.dtype).reshape(x.shape[0], -1)
 
 
 @instrument("moe_route")

@@ -246,7 +246,7 @@ def gemm_plan(T: int, N: int, K: int, splits_hint: int = 0):
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
               ld_out: Optional[int] = None, add_into: bool = False, splits: int = 0, swiglu: bool = False,
               sumsq_in: Optional[torch.Tensor] = None, eps: float = 0.0, clear: Optional[torch.Tensor] = None,
-              sumsq_out: Optional[torch.Tensor] = None, gelu: bool = False) -> torch.Tensor:
+              sumsq_out: Optional[torch.Tensor] = None, gelu: bool = False, epi: Optional[int] = None) -> torch.Tensor:
     """out[T, N] = x[T, K] @ w[N, K]^T on the tcgen05 kernel; ``out`` may be a column slice of a
     wider row-major buffer (pass its row stride as ``ld_out``).
 
@@ -265,7 +265,8 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = No
     elif ld_out is None:
         ld_out = out.stride(0)
     s = scratch(x.device)
-    epi = (4 if gelu else 2) if swiglu else (1 if add_into else 0)  # EPI_GEGLU / EPI_SWIGLU / EPI_ADD_INTO / EPI_STORE
+    if epi is None:  # EPI_GEGLU / EPI_SWIGLU / EPI_ADD_INTO / EPI_STORE
+        epi = (4 if gelu else 2) if swiglu else (1 if add_into else 0)
     if sumsq_in is None and sumsq_out is None:
         _check(lib().oxb_gemm_bf16(x.data_ptr(), w.data_ptr(), out.data_ptr(), _p(bias), T, N, K, ld_out, epi, splits,
                                    s.gemm_ws.data_ptr(), s.gemm_ws.numel() * 4, s.gemm_counters.data_ptr(),
@@ -315,6 +316,17 @@ def dequant_rows(w, out: Optional[torch.Tensor] = None, fast: bool = False) -> t
     return out
 
 
+def pad_k(x: torch.Tensor, p):
+    """(x, bf16 weight) with the inner size padded to a multiple of 8: the tensor copies move rows of 16-byte multiples."""
+    k = p.shape[1]
+    if k % 8 == 0:
+        return x, p.data
+    pad = (0, 8 - k % 8)
+    if getattr(p, "_pad8", None) is None:
+        p._pad8 = torch.nn.functional.pad(p.data, pad).contiguous()
+    return torch.nn.functional.pad(x, pad), p._pad8
+
+
 def linear(x: torch.Tensor, parts: Sequence, bias: Optional[torch.Tensor] = None,
            out: Optional[torch.Tensor] = None) -> torch.Tensor:
     if x.dtype != torch.bfloat16:
@@ -330,7 +342,8 @@ def linear(x: torch.Tensor, parts: Sequence, bias: Optional[torch.Tensor] = None
         b = None if bias is None else bias[off : off + n]
         view = out[:, off : off + n]
         if p.qtype == "BF16":
-            gemm_bf16(x, p.data, view, b, ld_out=out.stride(0))
+            xp, data = pad_k(x, p)
+            gemm_bf16(xp, data, view, b, ld_out=out.stride(0))
         elif p.qtype in ("F32", "F16"):
             if getattr(p, "_bf16", None) is None:
                 p._bf16 = p.data.to(torch.bfloat16).contiguous()
@@ -406,6 +419,7 @@ def gelu_mul(gate_up: torch.Tensor) -> torch.Tensor:
 
 def rope_table(rope, max_pos: int) -> torch.Tensor:
     """[max_pos, rot] fp32: cos at [:, :rot/2], sin at [:, rot/2:], computed in float64."""
+    max_pos = max(max_pos, getattr(rope, "max_pos", 0))
     tab = getattr(rope, "_table", None)
     if tab is None or tab.shape[0] < max_pos:
         n = max(max_pos, 32768)

@@ -1,0 +1,155 @@
+"""Bindings of the kernels behind models with latent attention and norms after the sum (``csrc/oxb_latent.cu``), and of the
+float32 compute path.  CUDA tensors only; see :mod:`oxidize_b200.ops` for the operators' meaning."""
+from __future__ import annotations
+
+import ctypes
+from typing import Optional, Sequence
+
+import torch
+
+from . import cuda as opcuda
+from .cuda import _check, _p, _stream
+
+_declared = False
+
+DT = {torch.float32: 0, torch.bfloat16: 2}
+ACTS = {"relu2": 1}
+EPI_RELU2 = 5
+
+
+def lib():
+    global _declared
+    L = opcuda.lib()
+    if not _declared:
+        vp, i32, f32, i64 = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
+        L.oxb_residual_norm.argtypes = [vp, vp, f32, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp]
+        L.oxb_gemm_f32.argtypes = [vp, vp, vp, vp] + [i32] * 7 + [i64, i64, i64, i32, vp]
+        L.oxb_latent_prep.argtypes = ([vp, i32, i32, vp, vp, vp, i32, i32, i32, vp, f32] + [i32] * 6 + [vp, i32, vp, vp, i32, vp,
+                                      i32, i32, vp])
+        L.oxb_latent_attention_simt.argtypes = [vp, vp, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp]
+        L.oxb_gemm_batched.argtypes = [vp, vp, vp, i64] + [i32] * 5 + [vp]
+        _declared = True
+    return L
+
+
+# --------------------------------------------------------------------------- norms and products
+def residual_norm(res: Optional[torch.Tensor], y: Optional[torch.Tensor], alpha: float, w: torch.Tensor,
+                  b: Optional[torch.Tensor], eps: float, kind: str, act_dtype: torch.dtype, keep_stream: bool = True):
+    like = y if res is None else res
+    T, H = like.shape
+    if y is not None and (y.dtype != act_dtype or not y.is_contiguous()):
+        y = y.to(act_dtype).contiguous()
+    x = torch.empty(T, H, dtype=torch.float32, device=like.device) if keep_stream or act_dtype == torch.float32 else None
+    a = x if act_dtype == torch.float32 else torch.empty(T, H, dtype=act_dtype, device=like.device)
+    _check(lib().oxb_residual_norm(_p(res), _p(y), alpha, w.data_ptr(), _p(b), _p(x), None if a is x else a.data_ptr(),
+                                   DT[act_dtype], T, H, eps, 1 if kind == "layer" else 0, _stream()), "oxb_residual_norm")
+    return x, a
+
+
+def gemm_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None, act: int = 0,
+             groups: int = 1, dims=None, strides=(0, 0, 0)) -> torch.Tensor:
+    """out = act(x @ w^T + bias) in float32; grouped calls give (T, N, K, ldx, ldw, ldy) and the group strides."""
+    if dims is None:
+        T, K = x.shape
+        dims = (T, w.shape[0], K, x.stride(0), w.stride(0), out.stride(0))
+    _check(lib().oxb_gemm_f32(x.data_ptr(), w.data_ptr(), out.data_ptr(), _p(bias), *dims, groups, *strides, act, _stream()),
+           "oxb_gemm_f32")
+    return out
+
+
+def linear_f32(x: torch.Tensor, parts: Sequence, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
+               act: int = 0) -> torch.Tensor:
+    x = x.contiguous()
+    if out is None:
+        out = torch.empty(x.shape[0], sum(p.shape[0] for p in parts), dtype=torch.float32, device=x.device)
+    off = 0
+    for p in parts:
+        n = p.shape[0]
+        gemm_f32(x, p.data, out[:, off : off + n], None if bias is None else bias[off : off + n], act)
+        off += n
+    return out
+
+
+def linear_act(x: torch.Tensor, w, act: str) -> torch.Tensor:
+    """act(x W^T): the activation is the product's epilogue."""
+    p = w.parts[0]
+    if x.dtype == torch.float32:
+        return linear_f32(x, w.parts, w.bias, act=ACTS[act])
+    if act != "relu2" or len(w.parts) != 1 or w.bias is not None or p.qtype != "BF16":
+        raise ValueError("linear_act covers one bfloat16 matrix and the relu2 activation")
+    x, data = opcuda.pad_k(x.contiguous(), p)
+    return opcuda.gemm_bf16(x, data, epi=EPI_RELU2)
+
+
+# --------------------------------------------------------------------------- latent attention
+class LatentOperands:
+    """A layer's per-head up-projections in the shapes the products read: ``k`` [H * rank, nope (padded)] multiplies the
+    queries (W_uk transposed per head), ``v`` [H * v_dim, latent_pad] the attended latents."""
+
+    def __init__(self, m, spec, dtype: torch.dtype):
+        H = m.w_uk.shape[0]
+        ld = (spec.nope_dim + 7) // 8 * 8
+        dev = m.w_uk.device
+        k = torch.zeros(H, spec.kv_rank, ld, dtype=dtype, device=dev)
+        k[:, :, : spec.nope_dim] = m.w_uk.transpose(1, 2)
+        v = torch.zeros(H, spec.v_dim, spec.latent_pad, dtype=dtype, device=dev)
+        v[:, :, : spec.kv_rank] = m.w_uv
+        self.heads, self.nope_ld, self.k, self.v = H, ld, k, v
+
+
+def operands(m, spec, dtype: torch.dtype) -> LatentOperands:
+    op = getattr(m, "_operands", None)
+    if op is None:
+        op = m._operands = LatentOperands(m, spec, dtype)
+    return op
+
+
+def batched(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, y_stride: int, ldy: int) -> None:
+    """For every head g: y[:, g * y_stride : g * y_stride + N] = x[g] @ w[g]^T, x [H, T, K], w [H, N, K], rows of y ``ldy``
+    apart."""
+    H, T, K = x.shape
+    N = w.shape[1]
+    if x.dtype == torch.float32:
+        gemm_f32(x, w, y, groups=H, dims=(T, N, K, K, K, ldy), strides=(T * K, N * K, y_stride))
+        return
+    _check(lib().oxb_gemm_batched(x.data_ptr(), w.data_ptr(), y.data_ptr(), y_stride, H, T, N, K, ldy, _stream()),
+           "oxb_gemm_batched")
+
+
+def latent_prep(qkv, m, spec, rope, meta, kv, layer: int, eps: float, op: LatentOperands, q_nope=None, q_rows=None, q_full=None):
+    tab = opcuda.rope_table(rope, rope.max_pos)
+    own = spec.kv_from is None
+    _check(lib().oxb_latent_prep(qkv.data_ptr(), qkv.stride(0), DT[qkv.dtype], meta.positions.data_ptr(),
+                                 meta.slot_mapping.data_ptr() if own else None, tab.data_ptr(), tab.shape[0], spec.rope_dim,
+                                 0 if rope.pairing == "split_half" else 1, _p(m.kv_a_norm), eps, qkv.shape[0], op.heads,
+                                 spec.nope_dim, spec.kv_rank, spec.latent_pad, spec.row_dim, _p(q_nope), op.nope_ld, _p(q_rows),
+                                 _p(q_full), 0 if q_full is None else q_full.shape[-1], kv.data[layer].data_ptr(), kv.page_size,
+                                 kv.num_blocks, _stream()), "oxb_latent_prep")
+
+
+def attention_simt(q, kv, layer: int, meta, spec, sink, out):
+    T, H, width = q.shape
+    B = meta.seq_lens.shape[0]
+    _check(lib().oxb_latent_attention_simt(q.data_ptr(), out.data_ptr(), kv.data[layer].data_ptr(), DT[q.dtype],
+                                           meta.block_tables.data_ptr(), meta.seq_lens.data_ptr(), meta.query_start.data_ptr(),
+                                           _p(sink), B, meta.block_tables.stride(0), T, H, spec.latent_pad, width, kv.page_size,
+                                           kv.num_blocks, spec.window, spec.scale, _stream()), "oxb_latent_attention_simt")
+
+
+def latent_mixer(x, m, spec, rope, meta, kv, layer: int, eps: float) -> torch.Tensor:
+    from . import linear
+
+    if kv.data[layer].dtype != x.dtype:
+        raise ValueError(f"latent cache rows are kept in the compute type on the GPU ({x.dtype}), not {kv.dtype_name}")
+    op = operands(m, spec, x.dtype)
+    T, H = x.shape[0], op.heads
+    qkv = linear(x, m.q)
+    q_nope = torch.empty(H, T, op.nope_ld, dtype=x.dtype, device=x.device)
+    q = torch.empty(T, H, spec.row_dim, dtype=x.dtype, device=x.device)
+    latent_prep(qkv, m, spec, rope, meta, kv, layer, eps, op, q_nope=q_nope, q_rows=q)
+    batched(q_nope, op.k, q, spec.row_dim, H * spec.row_dim)
+    o = torch.empty(H, T, spec.latent_pad, dtype=x.dtype, device=x.device)
+    attention_simt(q, kv, layer, meta, spec, m.sink, o)
+    out = torch.empty(T, H * spec.v_dim, dtype=x.dtype, device=x.device)
+    batched(o, op.v, out, spec.v_dim, H * spec.v_dim)
+    return out

@@ -76,10 +76,31 @@ def gelu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return (torch.nn.functional.gelu(g, approximate="tanh") * u).to(gate_up.dtype)
 
 
+def residual_norm(res: Optional[torch.Tensor], y: Optional[torch.Tensor], alpha: float, w: torch.Tensor,
+                  b: Optional[torch.Tensor], eps: float, kind: str = "layer", act_dtype: torch.dtype = torch.float32):
+    """Norm after the sum: norm(alpha * res + y) in float32, as (float32 stream, the same in ``act_dtype``).  ``layer``
+    subtracts the mean and divides by the root of the mean squared deviation; ``rms`` divides by the root mean square."""
+    z = y.float() if res is None else (alpha * res.float() if y is None else alpha * res.float() + y.float())
+    if kind == "layer":
+        z = z - z.mean(-1, keepdim=True)
+    z = z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    if b is not None:
+        z = z + b.float()
+    return z, z.to(act_dtype)
+
+
+def activation(x: torch.Tensor, act: str) -> torch.Tensor:
+    """Elementwise activation of a feed-forward block without a gate: ``relu2`` is the square of relu."""
+    if act == "relu2":
+        return torch.relu(x.float()).square().to(x.dtype)
+    raise ValueError(f"unknown activation {act!r}")
+
+
 # --------------------------------------------------------------------------- rope
 
 
-def rope_inv_freq(rotary_dim: int, theta: float, scaling=None, device=None, freq_factors=None) -> torch.Tensor:
+def rope_inv_freq(rotary_dim: int, theta: float, scaling=None, device=None, freq_factors=None,
+                  dtype: torch.dtype = torch.float32) -> torch.Tensor:
     """Per-pair inverse frequencies [rotary_dim/2] with optional linear / YaRN scaling.  ``freq_factors``
     ([rotary_dim/2], from a ``rope_freqs.weight`` / ``rope_factors_*.weight`` tensor of the checkpoint) divides each
     frequency: that is how Llama-3.1-style and LongRoPE context extensions are stored in GGUF files."""
@@ -88,14 +109,15 @@ def rope_inv_freq(rotary_dim: int, theta: float, scaling=None, device=None, freq
     inv = theta ** (-2.0 * idx / rotary_dim)
     if scaling is not None and scaling.type == "linear" and scaling.factor > 0:
         inv = inv / scaling.factor
-    elif scaling is not None and scaling.type == "yarn" and scaling.factor > 1 and scaling.original_context_length > 0:
+    elif (scaling is not None and scaling.type == "yarn" and scaling.original_context_length > 0
+          and (scaling.factor > 1 or scaling.magnitude > 0)):
         orig = scaling.original_context_length
 
         def corr_dim(n_rot):
             return rotary_dim * math.log(orig / (n_rot * 2 * math.pi)) / (2 * math.log(theta))
 
         lo = max(math.floor(corr_dim(scaling.beta_fast)), 0)
-        hi = min(math.ceil(corr_dim(scaling.beta_slow)), half - 1)
+        hi = min(math.ceil(corr_dim(scaling.beta_slow)), scaling.ramp_limit or half - 1)
         ramp = ((idx - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
         mix = 1.0 - ramp  # 1 => extrapolate (keep), 0 => interpolate
         inv = inv / scaling.factor * (1 - mix) + inv * mix
@@ -104,10 +126,12 @@ def rope_inv_freq(rotary_dim: int, theta: float, scaling=None, device=None, freq
         if ff.numel() < half:
             raise ValueError(f"rope frequency factors have {ff.numel()} entries, the rotary half dimension is {half}")
         inv = inv / ff[:half]
-    return inv.float()
+    return inv.to(dtype)
 
 
 def rope_mscale(scaling) -> float:
+    if scaling is not None and scaling.magnitude > 0:
+        return scaling.magnitude
     if scaling is not None and scaling.type == "yarn" and scaling.factor > 1:
         return 0.1 * math.log(scaling.factor) + 1.0
     return 1.0
@@ -163,26 +187,28 @@ def kv_dequantize(codes: torch.Tensor, scales: torch.Tensor, bits: int) -> torch
     return q.flatten(-2)
 
 
-def kv_write(kv, layer: int, k: torch.Tensor, v: torch.Tensor, slot_mapping: torch.Tensor) -> None:
-    """Scatter post-RoPE K/V rows [T, n_kv, hd] into the paged cache at flat slots."""
+def kv_write(kv, layer: int, k: torch.Tensor, v: Optional[torch.Tensor], slot_mapping: torch.Tensor) -> None:
+    """Scatter post-RoPE K/V rows [T, n_kv, hd] into the paged cache at flat slots (``v`` None: a cache of single rows)."""
     page = kv.page_size
     slots = slot_mapping.long()
     valid = slots >= 0
     if not bool(valid.all()):
-        k, v, slots = k[valid], v[valid], slots[valid]
+        k, v, slots = k[valid], None if v is None else v[valid], slots[valid]
     blk, off = slots // page, slots % page
     data = kv.data[layer]
     if kv.dtype_name in ("f16", "bf16", "f32"):
         data[blk, :, 0, off] = k.to(data.dtype)
-        data[blk, :, 1, off] = v.to(data.dtype)
+        if v is not None:
+            data[blk, :, 1, off] = v.to(data.dtype)
     else:
         bits = 8 if kv.dtype_name == "q8" else 4
         kc, ks = kv_quantize(k, bits)
-        vc, vs = kv_quantize(v, bits)
         data[blk, :, 0, off] = kc
-        data[blk, :, 1, off] = vc
         kv.scales[layer][blk, :, 0, off] = ks
-        kv.scales[layer][blk, :, 1, off] = vs
+        if v is not None:
+            vc, vs = kv_quantize(v, bits)
+            data[blk, :, 1, off] = vc
+            kv.scales[layer][blk, :, 1, off] = vs
 
 
 def kv_gather(kv, layer: int, block_table: torch.Tensor, seq_len: int) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -235,11 +261,40 @@ def paged_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, sliding
     return out.to(q.dtype)
 
 
-def latent_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, latent_dim: int) -> torch.Tensor:
+def latent_rows(qkv: torch.Tensor, m, spec, rope, meta, kv, layer: int, eps: float) -> torch.Tensor:
+    """From the projections of a latent-attention layer ([queries | latent | rotary key], the last two only where the
+    layer owns cache rows) write this step's cache rows and return the queries in absorbed form [T, H, row_dim]: the
+    position-free part multiplied by W_uk, the rotated part behind it, zeros in the padding."""
+    H, nope, rot, c = m.w_uk.shape[0], spec.nope_dim, spec.rope_dim, spec.kv_rank
+    T, pad, width = qkv.shape[0], spec.latent_pad, spec.row_dim
+    q = qkv[:, : H * spec.qk_dim].reshape(T, H, spec.qk_dim)
+    if spec.kv_from is None:
+        ckv = qkv[:, H * spec.qk_dim :]
+        row = torch.zeros(T, 1, width, dtype=qkv.dtype, device=qkv.device)
+        row[:, 0, :c] = rmsnorm(ckv[:, :c], m.kv_a_norm, eps)
+        row[:, :, pad : pad + rot] = apply_rope(ckv[:, None, c:], meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
+        kv_write(kv, layer, row, None, meta.slot_mapping)
+    out = torch.zeros(T, H, width, dtype=qkv.dtype, device=qkv.device)
+    out[:, :, :c] = torch.einsum("thn,hnc->thc", q[:, :, :nope].float(), m.w_uk.float())
+    out[:, :, pad : pad + rot] = apply_rope(q[:, :, nope:], meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
+    return out
+
+
+def softmax_sink(s: torch.Tensor, sink: Optional[torch.Tensor]) -> torch.Tensor:
+    """Softmax over the last axis; ``sink`` (a logit per row, broadcast against ``s[..., :1]``) joins the denominator only."""
+    if sink is None:
+        return torch.softmax(s, dim=-1)
+    sk = sink.float().expand(*s.shape[:-1], 1)
+    return torch.softmax(torch.cat([s, sk], dim=-1), dim=-1)[..., :-1]
+
+
+def latent_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, latent_dim: int, window: int = 0,
+                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Multi-query attention over latent cache rows (DeepSeek latent attention in absorbed form).
 
     q: [T, H, latent_dim + rope]; the cache holds one row of that width per token, shared by all heads, and the value of
-    a row is its first ``latent_dim`` entries.  Returns [T, H, latent_dim].  A decode step (one row per sequence) is one
+    a row is its first ``latent_dim`` entries.  ``window`` > 0 keeps the latest ``window`` positions of each query (itself
+    included); ``sink`` [H] is a logit that joins the softmax denominator only.  Returns [T, H, latent_dim].  A decode step (one row per sequence) is one
     batched gather + two batched matrix products over all sequences; other steps go sequence by sequence.  Device-agnostic
     torch: this is what runs on a GPU too, where the attention kernel has no 576-wide head."""
     T, H, D = q.shape
@@ -259,9 +314,13 @@ def latent_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, latent
         nb = (max_len + page - 1) // page
         K = rows_of(meta.block_tables[:, :nb].long())[:, :max_len]  # [B, L, D]
         s = torch.einsum("bhd,bld->bhl", q.float(), K) * scale
-        live = torch.arange(max_len, device=q.device)[None, :] < meta.seq_lens.long()[:, None]
+        kpos = torch.arange(max_len, device=q.device)[None, :]
+        live = kpos < meta.seq_lens.long()[:, None]
+        if window > 0:
+            live &= kpos >= meta.seq_lens.long()[:, None] - window
         s = s.masked_fill(~live[:, None, :], float("-inf"))
-        return torch.einsum("bhl,blc->bhc", torch.softmax(s, dim=-1), K[..., :latent_dim]).to(q.dtype)
+        p = softmax_sink(s, None if sink is None else sink[None, :, None])
+        return torch.einsum("bhl,blc->bhc", p, K[..., :latent_dim]).to(q.dtype)
     out = torch.zeros(T, H, latent_dim, dtype=torch.float32, device=q.device)
     qs, sl = meta.query_start.tolist(), meta.seq_lens.tolist()
     for b in range(B):
@@ -271,9 +330,13 @@ def latent_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, latent
             continue
         K = rows_of(meta.block_tables[b, : (L + page - 1) // page].long())[:L]  # [L, D]
         s = torch.einsum("qhd,ld->hql", q[t0:t1].float(), K) * scale
-        causal = torch.arange(L, device=q.device)[None, :] <= torch.arange(L - n, L, device=q.device)[:, None]
-        s = s.masked_fill(~causal[None], float("-inf"))
-        out[t0:t1] = torch.einsum("hql,lc->qhc", torch.softmax(s, dim=-1), K[:, :latent_dim])
+        kpos, qpos = torch.arange(L, device=q.device)[None, :], torch.arange(L - n, L, device=q.device)[:, None]
+        seen = kpos <= qpos
+        if window > 0:
+            seen &= kpos > qpos - window
+        s = s.masked_fill(~seen[None], float("-inf"))
+        p = softmax_sink(s, None if sink is None else sink[:, None, None])
+        out[t0:t1] = torch.einsum("hql,lc->qhc", p, K[:, :latent_dim])
     return out.to(q.dtype)
 
 
