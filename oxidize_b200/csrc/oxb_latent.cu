@@ -3,6 +3,7 @@
 #include "common.cuh"
 #include "gemm_f32.cuh"
 #include "latent.cuh"
+#include "latent_mma.cuh"
 #include "residual_norm.cuh"
 using namespace oxb;
 
@@ -58,4 +59,70 @@ OXB_API int oxb_latent_attention_simt(const void* q, void* out, const void* cach
   const LatentAttnArgs a{q, out, cache, block_tables, seq_lens, query_start, sink, B, max_blocks, T, H, pad, width, page,
                          num_blocks, window, scale};
   return dtype == 0 ? latent_simt_launch<float>(a, stream) : latent_simt_launch<__nv_bfloat16>(a, stream);
+}
+
+// 1 when latent_attention_mma_kernel covers rows of this shape (else: the plain kernel)
+OXB_API int oxb_latent_mma_supported(int nr, int pad, int width, int page) {
+  return (nr == 16 || nr == 32) && latent_mma_plan(nr, pad, width, page).ok;
+}
+
+template <int NR>
+static int latent_mma_launch(const CUtensorMap& tk, const CUtensorMap& tq, const LatentMmaArgs& a, int B, int smem,
+                             cudaStream_t stream) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
+  if (!configured[dev]) {
+    cudaError_t e = cudaFuncSetAttribute(latent_attention_mma_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);
+    if (e != cudaSuccess) return (int)e;
+    configured[dev] = true;
+  }
+  const cudaError_t le = oxb_launch(latent_attention_mma_kernel<NR>, dim3(a.row_blocks * a.n_splits, B), dim3(LM_THREADS),
+                                    (size_t)smem, stream, tk, tq, a);
+  if (le != cudaSuccess) return (int)le;
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+// Latent attention, absorbed form, bf16: q [T, H, width] and the cache rows [num_blocks * page, width]; the B sequences
+// have at most max_query_len rows each.  n_splits > 1 needs ws_o [B * row_blocks * n_splits * nr * pad] and ws_ml
+// [.. * nr * 2] floats and one zeroed ticket per (sequence, row block), row_blocks = ceil(max_query_len * H / nr).
+OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache, const int* block_tables, const int* seq_lens,
+                                     const int* query_start, const float* sink, int B, int max_blocks, int T, int H, int pad,
+                                     int width, int page, int num_blocks, int window, float scale, int nr, int max_query_len,
+                                     int n_splits, float* ws_o, float* ws_ml, int* counters, cudaStream_t stream) {
+  if (T <= 0 || B <= 0 || max_query_len <= 0) return 0;
+  const LatentMmaPlan pl = latent_mma_plan(nr, pad, width, page);
+  if ((nr != 16 && nr != 32) || !pl.ok || B > 65535) return (int)cudaErrorInvalidValue;
+  if (n_splits > 1 && (ws_o == nullptr || ws_ml == nullptr || counters == nullptr)) return (int)cudaErrorInvalidValue;
+  CUtensorMap tk, tq;
+  int e = oxb_make_tmap_2d(&tk, cache, (uint64_t)num_blocks * page, width, (uint64_t)width * 2, page, 64, 2);
+  if (e) return e;
+  e = oxb_make_tmap_2d(&tq, q, (uint64_t)T * H, width, (uint64_t)width * 2, nr, 64, 2);
+  if (e) return e;
+  LatentMmaArgs a;
+  a.block_tables = block_tables;
+  a.seq_lens = seq_lens;
+  a.query_start = query_start;
+  a.sink = sink;
+  a.out = reinterpret_cast<__nv_bfloat16*>(out);
+  a.ws_o = ws_o;
+  a.ws_ml = ws_ml;
+  a.counters = counters;
+  a.max_blocks = max_blocks;
+  a.T = T;
+  a.H = H;
+  a.pad = pad;
+  a.width = width;
+  a.page = page;
+  a.num_blocks = num_blocks;
+  a.window = window;
+  a.n_splits = n_splits < 1 ? 1 : n_splits;
+  a.row_blocks = (max_query_len * H + nr - 1) / nr;
+  a.pairs = pl.pairs;
+  a.rest = pl.rest;
+  a.slots = pl.slots;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  return nr == 16 ? latent_mma_launch<16>(tk, tq, a, B, pl.smem, stream) : latent_mma_launch<32>(tk, tq, a, B, pl.smem, stream);
 }
