@@ -222,6 +222,26 @@ __device__ __forceinline__ void umma_bf16(uint32_t tmem_d, uint64_t adesc, uint6
       ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
+// The same with the issuing lane chosen by a predicate instead of a branch (called by the whole warp) and the descriptors
+// given as their low words, which hold the address; the high words (layout) are constants: short, warp-uniform operands.
+template <uint32_t AHI, uint32_t BHI, uint32_t IDESC>
+__device__ __forceinline__ void umma_bf16_if(bool issue, uint32_t tmem_d, uint32_t alo, uint32_t blo, bool accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\t.reg .b64 da, db;\n\t"
+      "setp.ne.b32 p, %3, 0;\n\t"
+      "setp.ne.b32 q, %4, 0;\n\t"
+      "mov.b64 da, {%1, %5};\n\t"
+      "mov.b64 db, {%2, %6};\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], da, db, %7, p;\n\t}"
+      ::"r"(tmem_d), "r"(alo), "r"(blo), "r"((uint32_t)accumulate), "r"((uint32_t)issue), "n"(AHI), "n"(BHI), "n"(IDESC)
+      : "memory");
+}
+// low word of a shared-memory descriptor: address and leading byte offset, both in 16-byte units
+__device__ __forceinline__ uint32_t umma_desc_lo(uint32_t smem_addr, uint32_t leading_bytes = 16) {
+  return ((smem_addr & 0x3FFFF) >> 4) | ((leading_bytes >> 4) << 16);
+}
+// high word: stride byte offset 1024 (8 rows of 128 bytes), version 1, 128-byte swizzle
+constexpr uint32_t UMMA_DESC_HI_SW128 = (1024u >> 4) | (1u << 14) | (2u << 29);
 // A operand in tensor memory (row = lane, two bf16 per 32-bit column), B through a shared-memory descriptor
 __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
   asm volatile(
@@ -239,6 +259,15 @@ __device__ __forceinline__ void tmem_st4(uint32_t taddr, uint32_t a, uint32_t b,
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void umma_commit(uint64_t* bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
+}
+
+__device__ __forceinline__ void umma_commit_if(bool issue, uint64_t* bar) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\t"
+      "setp.ne.b32 q, %1, 0;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}"
+      ::"r"(smem_u32(bar)), "r"((uint32_t)issue)
+      : "memory");
 }
 
 // 32 lanes x 16 consecutive 32-bit columns: thread i of the warp reads lane (base_lane + i)
@@ -352,5 +381,11 @@ __device__ __forceinline__ uint32_t dsmem_map(uint32_t local_smem_addr, uint32_t
 __device__ __forceinline__ float dsmem_ld_f32(uint32_t cluster_addr) {
   float v;
   asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(cluster_addr) : "memory");
+  return v;
+}
+__device__ __forceinline__ float4 dsmem_ld_f32x4(uint32_t cluster_addr) {
+  float4 v;
+  asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];"
+               : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(cluster_addr) : "memory");
   return v;
 }

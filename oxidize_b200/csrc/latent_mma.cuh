@@ -1,27 +1,34 @@
 // Latent attention in absorbed form on the tensor cores: all heads of a query attend over the same cached rows.
 //
-// The work is turned around so that the cached rows are the wide operand: a tile of 128 rows (keys) is the M dimension of
-// S^T[keys, rows] = K Q^T, and the latent values are the M dimension of O^T[values, rows] = V^T P^T, where K and V are ONE
-// tile in shared memory: V^T is the same 128-byte-swizzled tile read as an MN-major operand.  N is a block of NR query rows
-// ((token, head) pairs, token-major), so a decode step of 32 heads is one instruction shape and the kernel is a stream of
-// cache rows: every CTA owns (sequence, block of query rows, split of the keys), one warp brings the pages in with TMA
-// (column chunks of 64 values, in pairs of chunks so that a pair is one 128-value block of the second product), one warp
-// issues tcgen05.mma, four warps do the softmax on S^T read from tensor memory.  A slot of the ring is given back as soon
-// as the second product has read its block, so the copies of the next tile run while this one is finished.
+// The work is turned around so that the cached rows are the wide operand: a tile of 64 rows (keys) is the M dimension of
+// S^T[keys, rows] = K Q^T, and the latent values are the M dimension (128 at a time) of O^T[values, rows] = V^T P^T, where K
+// and V are ONE tile in shared memory: V^T is the same 128-byte-swizzled tile read as an MN-major operand.  N is a block of
+// 32 query rows ((token, head) pairs, token-major), so a decode step of 32 heads is one instruction shape and the kernel is a
+// stream of cache rows: every CTA owns (sequence, block of query rows, split of the keys), two warps bring the pages in with
+// TMA (column chunks of 64 values, in pairs of chunks so that a pair is one 128-value block of the second product), one warp
+// issues tcgen05.mma, four warps do the softmax on S^T read from tensor memory.  The ring holds two tiles and a bit: the
+// first product of the next tile and the copies of the one after run while this tile is in its softmax.
 //
-// Softmax: a thread holds one key of every row; row maxima are found with a transposing butterfly (31 shuffles for 32
-// rows).  The running maximum is only moved when a tile exceeds it by more than 2^8, so O^T is rarely rescaled; the
-// result is exact either way.  Partial (max, sum, O) of key splits are merged by whichever CTA finishes last.
+// Softmax: a thread holds one key of 16 rows (a half-warp split of tcgen05.ld: 64 rows of S^T sit in 16 lanes per warp).
+// Running maxima are moved by the first tile and then only when a score exceeds one by more than 2^8, which one vote
+// settles; row maxima are found with a transposing butterfly, and O^T is then rescaled in tensor memory.  The result is
+// exact either way.  The key splits of a row block are one thread-block cluster: each leaves its partial O^T in its own
+// shared memory (the ring is idle by then), and every CTA merges a share of the rows out of its peers' memory.
 #pragma once
 #include "common.cuh"
 
 namespace oxb {
 
-constexpr int LM_KEYS = 128;                 // keys per tile
-constexpr int LM_CHUNK = LM_KEYS * 128;      // bytes of one 64-value column chunk of a tile
+constexpr int LM_KEYS = 64;              // keys per tile
+constexpr int LM_NR = 32;                // query rows per CTA
+constexpr int LM_CN = 16;                // of them per softmax thread
+constexpr int LM_CHUNK = LM_KEYS * 128;  // bytes of one 64-value column chunk of a tile
 constexpr int LM_PAIR = 2 * LM_CHUNK;
-constexpr int LM_THREADS = 192;              // warps 0-3 softmax and output, 4 TMA, 5 MMA
-constexpr int LM_MAX_SLOTS = 8;
+constexpr int LM_TMA_WARPS = 2;          // each brings every second page of a tile
+// warps: 0-3 softmax and output, then TMA, then MMA
+constexpr int LM_WARP_MMA = 4 + LM_TMA_WARPS, LM_WARPS = LM_WARP_MMA + 1, LM_THREADS = 32 * LM_WARPS;
+constexpr int LM_MAX_SLOTS = 16;
+constexpr int LM_DYN_SMEM = 224 * 1024;
 constexpr float LM_LAZY = 8.f;               // log2 of the factor by which scores may exceed the running maximum
 
 struct LatentMmaArgs {
@@ -30,28 +37,16 @@ struct LatentMmaArgs {
   const int* query_start;   // [B + 1]
   const float* sink;        // [H] or null
   __nv_bfloat16* out;       // [H, T, pad]
-  float* ws_o;              // [tasks, NR, pad] (key splits only)
-  float* ws_ml;             // [tasks, NR, 2]
-  int* counters;            // [B * row blocks] zero-initialised tickets
   int max_blocks, T, H, pad, width, page, num_blocks, window;
-  int n_splits, row_blocks;
+  int n_splits;             // CTAs of a cluster
   int pairs, rest, slots;   // 128-value blocks of the latent part, further 64-value chunks, ring slots (pairs)
+  int rest_slots;           // buffers of the further chunks
   float scale_log2;
 };
 
-// MN-major operand (64 contiguous values per 128-byte row, rows = the K dimension) with the 128-byte swizzle: 64-value
-// chunks `chunk_bytes` apart (leading offset), groups of 8 rows 1024 bytes apart (stride offset)
-__device__ __forceinline__ uint64_t umma_desc_mn_sw128(uint32_t smem_addr, uint32_t chunk_bytes) {
-  uint64_t d = 0;
-  d |= (uint64_t)((smem_addr & 0x3FFFF) >> 4);
-  d |= (uint64_t)((chunk_bytes >> 4) & 0x3FFF) << 16;
-  d |= (uint64_t)(1024 >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
-}
+// An MN-major operand (64 contiguous values per 128-byte row, rows = the K dimension) with the 128-byte swizzle: 64-value
+// chunks lie the descriptor's leading offset apart, groups of 8 rows its stride offset (1024 bytes).
 constexpr uint32_t UMMA_A_MN_MAJOR = 1u << 15;
-constexpr uint32_t UMMA_B_MN_MAJOR = 1u << 16;
 
 __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
   asm volatile(
@@ -60,16 +55,21 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
       "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
       : "memory");
 }
+// 16 tensor-memory lanes x 32 columns spread over the warp: thread i < 16 gets columns 0-15 of lane i, thread 16 + i
+// columns 16-31 of the same lane
+__device__ __forceinline__ void tmem_ld16_halves(uint32_t taddr, uint32_t* r) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.16x32bx2.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16], 16;"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
+        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr));
+}
 
-// Reduce v[n] over the 32 lanes for every n < NR; lane L returns the result of n = L % NR.  v is used up.
-template <int NR, class Op>
+// Reduce v[j] (j < 16) over the 16 lanes of each half-warp; lane L returns the result of j = L % 16 of its half.
+template <class Op>
 __device__ __forceinline__ float butterfly_rows(float* v, int lane, Op op) {
-  if constexpr (NR == 16) {
 #pragma unroll
-    for (int j = 0; j < 16; ++j) v[j] = op(v[j], __shfl_xor_sync(0xffffffffu, v[j], 16));
-  }
-#pragma unroll
-  for (int o = NR / 2; o > 0; o >>= 1) {
+  for (int o = 8; o > 0; o >>= 1) {
 #pragma unroll
     for (int j = 0; j < o; ++j) {
       const bool up = (lane & o) != 0;
@@ -80,23 +80,68 @@ __device__ __forceinline__ float butterfly_rows(float* v, int lane, Op op) {
   return v[0];
 }
 
-template <int NR>
-__global__ void __launch_bounds__(LM_THREADS, 1)
+// Merge of a cluster's key splits with the log-sum-exp weights exp2(m_s - M) / sum: this CTA takes rows rank, rank + n, ...
+constexpr int LM_MAX_SPLITS = 8;
+__device__ __forceinline__ void merge_splits(const LatentMmaArgs& a, const uint8_t* part, const float2* part_ml,
+                                             const long long* row_out, int rank, int tiles, int per) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const uint32_t part_addr = smem_u32(part), ml_addr = smem_u32(part_ml);
+  for (int row = rank + warp * a.n_splits; row < LM_NR; row += LM_WARPS * a.n_splits) {
+    const long long o = row_out[row];
+    if (o < 0) continue;
+    // lane s holds split s
+    float ms = -INFINITY, ls = 0.f;
+    if (lane < a.n_splits && lane * per < tiles) {
+      const uint32_t src = dsmem_map(ml_addr + row * 8, lane);
+      ms = dsmem_ld_f32(src);
+      ls = dsmem_ld_f32(src + 4);
+    }
+    const float M = warp_max(ms);
+    float w = ms == -INFINITY ? 0.f : exp2f(ms - M);  // 0: that split saw no key of this row
+    const float den = warp_sum(w * ls);
+    w *= den > 0.f ? 1.f / den : 0.f;
+    float wv[LM_MAX_SPLITS];
+#pragma unroll
+    for (int s = 0; s < LM_MAX_SPLITS; ++s) wv[s] = __shfl_sync(0xffffffffu, w, s);
+    for (int d = lane * 4; d < a.pad; d += 128) {
+      float4 v[LM_MAX_SPLITS];
+#pragma unroll
+      for (int s = 0; s < LM_MAX_SPLITS; ++s) {
+        v[s] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (s < a.n_splits && s * per < tiles) v[s] = dsmem_ld_f32x4(dsmem_map(part_addr + (row * a.pad + d) * 4, s));
+      }
+      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int s = 0; s < LM_MAX_SPLITS; ++s) {
+        acc.x += wv[s] * v[s].x;
+        acc.y += wv[s] * v[s].y;
+        acc.z += wv[s] * v[s].z;
+        acc.w += wv[s] * v[s].w;
+      }
+      *reinterpret_cast<uint2*>(a.out + o + d) = make_uint2(pack_bf16x2(acc.x, acc.y), pack_bf16x2(acc.z, acc.w));
+    }
+  }
+}
+
+static __global__ void __launch_bounds__(LM_THREADS, 1)
 latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmQ,
                             const LatentMmaArgs a) {
-  static_assert(NR == 16 || NR == 32, "rows per block");
+  constexpr int NR = LM_NR;
   extern __shared__ uint8_t lm_raw[];
-  __shared__ uint64_t full[LM_MAX_SLOTS], empty[LM_MAX_SLOTS], rest_full, rest_empty, q_full, s_full, p_full, pv_done;
+  // s_full / p_full / pv_done: one per parity of the tile (S^T and P are double-buffered)
+  __shared__ uint64_t full[LM_MAX_SLOTS], empty[LM_MAX_SLOTS], rest_full[2], rest_empty[2], q_full, s_full[2], p_full[2], pv_done[2];
   __shared__ uint32_t tmem_slot;
   __shared__ volatile int abort_flag;
-  __shared__ int ticket;
-  __shared__ int2 row_keys[NR];        // first and last key that a row sees
-  __shared__ float wmax[4][NR];        // per-warp maxima of a tile, then per-warp sums
-  __shared__ __align__(16) float mrow[4][NR];  // running maxima (a copy per warp)
-  __shared__ __align__(16) float frow[4][NR];  // factors of a rescale / normalisation
+  __shared__ int2 row_keys[NR];                 // first and last key that a row sees
+  __shared__ __align__(8) float2 part_ml[NR];   // maximum and sum of this split
+  __shared__ long long row_out[NR];             // offset of a row's output, < 0: no such row
+  __shared__ float wmax[4][NR];                 // per-warp maxima of a tile, then per-warp sums
+  __shared__ __align__(16) float mrow[4][NR];   // running maxima (a copy per warp)
+  __shared__ __align__(16) float frow[4][NR];   // factors of a rescale / normalisation
   pdl_launch_dependents();
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  // (broadcast from lane 0: the role branches and what is computed inside them are then known to be warp-uniform)
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
   const int b = blockIdx.y;
   const int rb = blockIdx.x / a.n_splits, split = blockIdx.x % a.n_splits;
   const int q0 = a.query_start[b], qlen = a.query_start[b + 1] - q0;
@@ -118,311 +163,324 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
 
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lm_raw) + 1023) & ~uintptr_t(1023));
   const int nch = (a.width + 63) / 64;
-  uint8_t* s_rest = smem + a.slots * LM_PAIR;
-  uint8_t* s_q = s_rest + a.rest * LM_CHUNK;       // [nch][NR][128 bytes]
-  uint8_t* s_p = s_q + nch * NR * 128;             // [2][NR][128 bytes]: 64 keys per 128-byte row
-  uint32_t tmem_cols = 32;
-  while ((int)tmem_cols < NR * (1 + a.pairs)) tmem_cols <<= 1;
+  uint8_t* s_rest = smem + a.slots * LM_PAIR;                     // [rest_slots][rest chunks]
+  uint8_t* s_q = s_rest + a.rest_slots * a.rest * LM_CHUNK;       // [nch][NR][128 bytes]
+  uint8_t* s_p = s_q + nch * NR * 128;                            // [2][NR][128 bytes]: the tile's 64 keys
+  uint32_t tmem_cols = 64;
+  while ((int)tmem_cols < NR * (2 + a.pairs)) tmem_cols <<= 1;
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < a.slots; ++i) {
-      mbar_init(&full[i], 1);
+      mbar_init(&full[i], LM_TMA_WARPS);
       mbar_init(&empty[i], 1);
     }
-    mbar_init(&rest_full, 1);
-    mbar_init(&rest_empty, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&rest_full[i], LM_TMA_WARPS);
+      mbar_init(&rest_empty[i], 1);
+      mbar_init(&s_full[i], 1);
+      mbar_init(&p_full[i], 128);
+      mbar_init(&pv_done[i], 1);
+    }
     mbar_init(&q_full, 1);
-    mbar_init(&s_full, 1);
-    mbar_init(&p_full, 128);
-    mbar_init(&pv_done, 1);
     abort_flag = 0;
-    ticket = 0;
     mbar_fence_init();
   }
   if (threadIdx.x < NR) {
-    const int r = min(row_base + (int)threadIdx.x, R - 1);  // rows past the end see what the last row sees; never stored
+    const int r0 = row_base + (int)threadIdx.x, r = min(r0, R - 1);  // rows past the end see what the last row sees
     const int p = pos0 + r / a.H;
     row_keys[threadIdx.x] = make_int2(a.window > 0 ? max(0, p - a.window + 1) : 0, p);
+    row_out[threadIdx.x] = r0 < R ? ((long long)(r % a.H) * a.T + q0 + r / a.H) * a.pad : -1;
   }
-  if (warp == 5) {
+  if (warp == LM_WARP_MMA) {
     tmem_alloc(&tmem_slot, tmem_cols);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = tmem_slot;
+  const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_slot, 0);  // columns: S^T (two buffers of NR), then the blocks of O^T
   pdl_wait();  // queries and this step's cache rows come from the upstream kernels
 
-  if (warp == 4) {
-    // ---------------- TMA: lane p brings page p of the tile
-    if (lane == 0) {
+  if (warp >= 4 && warp < LM_WARP_MMA) {
+    // ---------------- TMA: warp-uniform loops, one elected lane issues
+    const int w = warp - 4;
+    const bool leader = elect_one();
+    if (leader && w == 0) {
       tma_prefetch_desc(&tmK);
       tma_prefetch_desc(&tmQ);
       mbar_expect_tx(&q_full, nch * NR * 128);
       for (int c = 0; c < nch; ++c) tma_load_2d(s_q + c * NR * 128, &tmQ, &q_full, c * 64, q0 * a.H + row_base);
     }
     const int* bt = a.block_tables + (size_t)b * a.max_blocks;
-    int cnt = 0;  // pairs issued
+    const int mine = (ppt + LM_TMA_WARPS - 1 - w) / LM_TMA_WARPS;  // pages of this warp: w, w + LM_TMA_WARPS, ...
+    int slot = 0, use = 0;  // ring position and how often it has been round
     bool ok = true;
     for (int t = t_begin; t < t_end && ok; ++t) {
-      int blk = 0;
-      if (lane < ppt) {
-        blk = bt[min(page_lo + t * ppt + lane, page_hi)];  // pages past the last one: any valid page, its keys are masked
+      const int i = t - t_begin;
+      int blk = a.num_blocks;  // pages past the last one: a row outside the pool, which the copy fills with zeros
+      if (lane < ppt && page_lo + t * ppt + lane <= page_hi) {
+        blk = bt[page_lo + t * ppt + lane];
         if ((unsigned)blk >= (unsigned)a.num_blocks) {
           oxb_report(OXB_BAD_BLOCK_ID, blk);
           blk = 0;
         }
       }
-      const int row = blk * a.page;
-      for (int p = 0; p < a.pairs + (a.rest > 0 ? 1 : 0) && ok; ++p) {
-        const bool is_rest = p == a.pairs;
-        const int slot = cnt % a.slots;
-        uint64_t* fb = is_rest ? &rest_full : &full[slot];
-        if (is_rest) {
-          const int i = t - t_begin;
-          if (i > 0) ok = mbar_wait_bounded(&rest_empty, (i - 1) & 1, &abort_flag, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
-        } else {
-          if (cnt >= a.slots) ok = mbar_wait_bounded(&empty[slot], (cnt / a.slots - 1) & 1, &abort_flag, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
-          ++cnt;
-        }
-        ok = __all_sync(0xffffffffu, ok);
-        if (!ok) break;
-        uint8_t* dst = is_rest ? s_rest : smem + slot * LM_PAIR;
-        const int c0 = 2 * p, c1 = is_rest ? nch : min(nch, c0 + 2);
-        if (lane == 0) mbar_expect_tx(fb, (c1 - c0) * LM_CHUNK);
-        __syncwarp();
-        if (lane < ppt)
-          for (int c = c0; c < c1; ++c) tma_load_2d(dst + (c - c0) * LM_CHUNK + lane * a.page * 128, &tmK, fb, c * 64, row);
-        __syncwarp();
-      }
-    }
-  } else if (warp == 5) {
-    // ---------------- MMA
-    const bool leader = elect_one();
-    constexpr uint32_t idesc_s = umma_idesc_bf16(128, NR);
-    constexpr uint32_t idesc_o = umma_idesc_bf16(128, NR) | UMMA_A_MN_MAJOR;
-    const uint32_t base = smem_u32(smem), q_addr = smem_u32(s_q), p_addr = smem_u32(s_p), r_addr = smem_u32(s_rest);
-    const int ksteps = a.width / 16;
-    int cnt = 0;
-    bool ok = t_begin < t_end && mbar_wait_bounded(&q_full, 0, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
-    ok = __all_sync(0xffffffffu, ok);
-    for (int t = t_begin; t < t_end && ok; ++t) {
-      const int i = t - t_begin;
       for (int p = 0; p < a.pairs + (a.rest > 0 ? 1 : 0); ++p) {
         const bool is_rest = p == a.pairs;
-        const int slot = (cnt + p) % a.slots;
-        ok = is_rest ? mbar_wait_bounded(&rest_full, i & 1, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x)
-                     : mbar_wait_bounded(&full[slot], ((cnt + p) / a.slots) & 1, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+        const int rs = a.rest_slots == 2 ? i & 1 : 0, ru = a.rest_slots == 2 ? i >> 1 : i;
+        uint64_t* fb = is_rest ? &rest_full[rs] : &full[slot];
+        const int round = is_rest ? ru : use;
+        if (round > 0)
+          ok = mbar_wait_bounded(is_rest ? &rest_empty[rs] : &empty[slot], (round - 1) & 1, &abort_flag, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
-        tc_fence_after();
-        if (leader) {
-          const uint32_t src = is_rest ? r_addr : base + slot * LM_PAIR;
-          const int k0 = p * 8, k1 = is_rest ? ksteps : min(ksteps, k0 + 8);
-          for (int k = k0; k < k1; ++k)
-            umma_bf16(tmem, umma_desc_k_sw128(src + ((k - k0) >> 2) * LM_CHUNK) + 2 * (k & 3),
-                      umma_desc_k_sw128(q_addr + (k >> 2) * (NR * 128)) + 2 * (k & 3), idesc_s, k > 0 ? 1u : 0u);
-          if (is_rest) umma_commit(&rest_empty);
+        uint8_t* dst = is_rest ? s_rest + rs * a.rest * LM_CHUNK : smem + slot * LM_PAIR;
+        const int c0 = 2 * p, nc = (is_rest ? nch : min(nch, c0 + 2)) - c0;
+        if (leader) mbar_expect_tx(fb, nc * mine * a.page * 128);
+        for (int g = w; g < ppt; g += LM_TMA_WARPS) {
+          const int row = __shfl_sync(0xffffffffu, blk, g) * a.page;
+          uint8_t* d = dst + g * a.page * 128;
+          if (leader) {
+            tma_load_2d(d, &tmK, fb, c0 * 64, row);
+            for (int c = 1; c < nc; ++c) tma_load_2d(d + c * LM_CHUNK, &tmK, fb, (c0 + c) * 64, row);
+          }
         }
         __syncwarp();
-      }
-      if (!ok) break;
-      if (leader) umma_commit(&s_full);
-      ok = __all_sync(0xffffffffu, mbar_wait_bounded(&p_full, i & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x));
-      if (!ok) break;
-      tc_fence_after();
-      for (int p = 0; p < a.pairs; ++p) {
-        const int slot = (cnt + p) % a.slots;
-        if (leader) {
-          const uint64_t vdesc = umma_desc_mn_sw128(base + slot * LM_PAIR, LM_CHUNK);
-#pragma unroll
-          for (int k = 0; k < LM_KEYS / 16; ++k)
-            umma_bf16(tmem + NR * (1 + p), vdesc + (uint64_t)(k * (2048 >> 4)),
-                      umma_desc_k_sw128(p_addr + (k >> 2) * (NR * 128)) + 2 * (k & 3), idesc_o, (i > 0 || k > 0) ? 1u : 0u);
-          umma_commit(&empty[slot]);
+        if (!is_rest && ++slot == a.slots) {
+          slot = 0;
+          ++use;
         }
       }
-      if (leader) umma_commit(&pv_done);
-      __syncwarp();
-      cnt += a.pairs;
     }
+  } else if (warp == LM_WARP_MMA) {
+    // ---------------- MMA
+    const bool leader = elect_one();
+    constexpr uint32_t idesc_s = umma_idesc_bf16(LM_KEYS, NR);
+    constexpr uint32_t idesc_o = umma_idesc_bf16(128, NR) | UMMA_A_MN_MAJOR;
+    const uint32_t base = smem_u32(smem), q_addr = smem_u32(s_q), p_addr = smem_u32(s_p), r_addr = smem_u32(s_rest);
+    const int ksteps = a.width / 16, n = t_end - t_begin;
+    int slot = 0, use = 0;  // of the first product; the second follows in the same order
+    // S^T of tile i
+    auto first = [&](int i) -> bool {
+      for (int p = 0; p < a.pairs + (a.rest > 0 ? 1 : 0); ++p) {
+        const bool is_rest = p == a.pairs;
+        const int rs = a.rest_slots == 2 ? i & 1 : 0, ru = a.rest_slots == 2 ? i >> 1 : i;
+        const bool ok = mbar_wait_bounded(is_rest ? &rest_full[rs] : &full[slot], (is_rest ? ru : use) & 1, &abort_flag,
+                                          OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+        if (!__all_sync(0xffffffffu, ok)) return false;
+        tc_fence_after();
+        const uint32_t kd = umma_desc_lo(is_rest ? r_addr + rs * a.rest * LM_CHUNK : base + slot * LM_PAIR);
+        const uint32_t qd = umma_desc_lo(q_addr + 2 * p * (NR * 128)), d = tmem + NR * (i & 1);
+        const int left = ksteps - 8 * p;
+        if (left >= 8 && !is_rest) {
+#pragma unroll
+          for (int k = 0; k < 8; ++k)  // a 64-value chunk is four k-steps of 32 bytes
+            umma_bf16_if<UMMA_DESC_HI_SW128, UMMA_DESC_HI_SW128, idesc_s>(
+                leader, d, kd + (k >> 2) * (LM_CHUNK >> 4) + 2 * (k & 3), qd + (k >> 2) * (NR * 128 >> 4) + 2 * (k & 3), k > 0 || p > 0);
+        } else {
+          for (int k = 0; k < left; ++k)
+            umma_bf16_if<UMMA_DESC_HI_SW128, UMMA_DESC_HI_SW128, idesc_s>(
+                leader, d, kd + (k >> 2) * (LM_CHUNK >> 4) + 2 * (k & 3), qd + (k >> 2) * (NR * 128 >> 4) + 2 * (k & 3), k > 0 || p > 0);
+        }
+        if (is_rest) umma_commit_if(leader, &rest_empty[rs]);
+        if (!is_rest && ++slot == a.slots) {
+          slot = 0;
+          ++use;
+        }
+      }
+      umma_commit_if(leader, &s_full[i & 1]);
+      return true;
+    };
+    // O^T += V^T P^T of tile i
+    int vslot = 0;
+    auto second = [&](int i) -> bool {
+      const bool ok = mbar_wait_bounded(&p_full[i & 1], (i >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+      if (!__all_sync(0xffffffffu, ok)) return false;
+      tc_fence_after();
+      const uint32_t pd = umma_desc_lo(p_addr + (i & 1) * (NR * 128));
+      for (int p = 0; p < a.pairs; ++p) {
+        const uint32_t vd = umma_desc_lo(base + vslot * LM_PAIR, LM_CHUNK);
+#pragma unroll
+        for (int k = 0; k < LM_KEYS / 16; ++k)  // 16 keys: 2 KB of the value tile, 32 bytes of a P row
+          umma_bf16_if<UMMA_DESC_HI_SW128, UMMA_DESC_HI_SW128, idesc_o>(leader, tmem + NR * (2 + p), vd + k * (2048 >> 4), pd + 2 * k,
+                                                                      i > 0 || k > 0);
+        umma_commit_if(leader, &empty[vslot]);
+        if (++vslot == a.slots) vslot = 0;
+      }
+      umma_commit_if(leader, &pv_done[i & 1]);
+      return true;
+    };
+    bool ok = n > 0 && mbar_wait_bounded(&q_full, 0, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+    ok = __all_sync(0xffffffffu, ok);
+    // the next tile's first product goes ahead of this tile's second one where the ring holds two tiles
+    const bool ahead = a.slots >= 2 * a.pairs;
+    if (ok) ok = first(0);
+    for (int i = 0; i < n && ok; ++i) {
+      if (ahead && i + 1 < n) ok = first(i + 1);
+      if (ok) ok = second(i);
+      if (ok && !ahead && i + 1 < n) ok = first(i + 1);
+    }
+    __syncwarp();
   } else {
-    // ---------------- softmax: thread = key of the tile (its tensor-memory lane)
+    // ---------------- softmax: thread = key of the tile x 16 query rows
     const uint32_t lanes = (uint32_t)(warp * 32) << 16;
-    const int tid = threadIdx.x;
+    const int key_in = warp * 16 + (lane & 15), n0 = lane & 16;  // key of the tile, first of this thread's rows
+    auto group_sync = [&]() { asm volatile("bar.sync 1, 128;" ::: "memory"); };
     // widest key range that every row of the block sees: tiles inside it need no mask
     const int all_lo = row_keys[NR - 1].x, all_hi = row_keys[0].y;
-    const int my_h = (row_base + lane % NR) % a.H;
-    const float sink = (a.sink != nullptr && split == 0) ? a.sink[my_h] * 1.4426950408889634f : -INFINITY;
-    float m = sink;  // running maximum of row lane % NR (log2 units), the same in every warp
-    float l[NR];
+    const float sink = (a.sink != nullptr && split == 0) ? a.sink[(row_base + lane) % a.H] * 1.4426950408889634f : -INFINITY;
+    float m = sink;  // running maximum of row `lane` (log2 units), the same in every warp
+    float l[LM_CN];
 #pragma unroll
-    for (int n = 0; n < NR; ++n) l[n] = 0.f;
-    for (int t = t_begin; t < t_end; ++t) {
-      const int i = t - t_begin;
+    for (int j = 0; j < LM_CN; ++j) l[j] = 0.f;
+    const int n = t_end - t_begin;
+    for (int i = 0; i < n; ++i) {
       // (no early exit on a failed wait: every thread passes every barrier, later waits return at once)
-      mbar_wait_bounded(&s_full, i & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+      mbar_wait_bounded(&s_full[i & 1], (i >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
       __syncwarp();
       tc_fence_after();
-      float s[NR];
-#pragma unroll
-      for (int c = 0; c < NR / 16; ++c) tmem_ld16(tmem + lanes + 16 * c, reinterpret_cast<uint32_t*>(s) + 16 * c);
+      float s[LM_CN];
+      tmem_ld16_halves(tmem + lanes + NR * (i & 1), reinterpret_cast<uint32_t*>(s));
       tmem_ld_wait();
-      const int key0 = (page_lo + t * ppt) * a.page, key = key0 + tid;
-      const bool inside = key0 >= all_lo && key0 + LM_KEYS - 1 <= all_hi;
+      const int key0 = (page_lo + (t_begin + i) * ppt) * a.page;
 #pragma unroll
-      for (int n = 0; n < NR; ++n) {
-        s[n] *= a.scale_log2;
-        if (!inside) {
-          const int2 rk = row_keys[n];
-          if (key < rk.x || key > rk.y) s[n] = -INFINITY;
+      for (int j = 0; j < LM_CN; ++j) s[j] *= a.scale_log2;
+      if (!(key0 >= all_lo && key0 + LM_KEYS - 1 <= all_hi)) {
+        const int key = key0 + key_in;
+#pragma unroll
+        for (int j = 0; j < LM_CN; ++j) {
+          const int2 rk = row_keys[n0 + j];
+          if (key < rk.x || key > rk.y) s[j] = -INFINITY;
         }
       }
-      {
-        float v[NR];
+      // running maxima of this thread's rows; usually no score exceeds them by the lazy margin, which one vote settles
+      float mm[LM_CN];
+      auto load_max = [&]() {
 #pragma unroll
-        for (int n = 0; n < NR; ++n) v[n] = s[n];
-        const float wm = butterfly_rows<NR>(v, lane, [](float x, float y) { return fmaxf(x, y); });
-        if (lane < NR) wmax[warp][lane] = wm;
-      }
-      asm volatile("bar.sync 1, 128;" ::: "memory");
-      const int n_ = lane % NR;
-      const float tm = fmaxf(fmaxf(wmax[0][n_], wmax[1][n_]), fmaxf(wmax[2][n_], wmax[3][n_]));
-      const bool move = tm > m + LM_LAZY || (m == -INFINITY && tm > -INFINITY);
-      const float m_new = move ? tm : m;
-      const float f = move ? exp2f(m - m_new) : 1.f;  // 0 when nothing was accumulated
-      m = m_new;
-      if (lane < NR) mrow[warp][lane] = m == -INFINITY ? 0.f : m;
-      const bool any_move = __any_sync(0xffffffffu, move);
-      if (any_move && lane < NR) frow[warp][lane] = f;
-      __syncwarp();
+        for (int j = 0; j < LM_CN; j += 4) {
+          const float4 v = *reinterpret_cast<const float4*>(&mrow[warp][n0 + j]);
+          mm[j] = v.x;
+          mm[j + 1] = v.y;
+          mm[j + 2] = v.z;
+          mm[j + 3] = v.w;
+        }
+      };
+      bool over = i == 0 || m == -INFINITY;
       if (i > 0) {
-        mbar_wait_bounded(&pv_done, (i - 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);  // P is free, O^T is complete
+        load_max();
+#pragma unroll
+        for (int j = 0; j < LM_CN; ++j) over |= s[j] > mm[j] + LM_LAZY;
+      }
+      int any_over;
+      asm volatile(
+          "{\n\t.reg .pred p, q;\n\tsetp.ne.s32 p, %1, 0;\n\tbarrier.cta.red.or.pred q, 1, 128, p;\n\tselp.s32 %0, 1, 0, q;\n\t}"
+          : "=r"(any_over)
+          : "r"((int)over)
+          : "memory");
+      bool any_move = false;
+      if (any_over) {
+        float v[LM_CN];
+#pragma unroll
+        for (int j = 0; j < LM_CN; ++j) v[j] = s[j];
+        wmax[warp][lane] = butterfly_rows(v, lane, [](float x, float y) { return fmaxf(x, y); });
+        group_sync();
+        const float tm = fmaxf(fmaxf(wmax[0][lane], wmax[1][lane]), fmaxf(wmax[2][lane], wmax[3][lane]));
+        // the first tile sets the maximum, later ones move it past the margin only
+        const bool move = tm > m + (i == 0 ? 0.f : LM_LAZY) || (m == -INFINITY && tm > -INFINITY);
+        const float m_new = move ? tm : m;
+        frow[warp][lane] = move ? exp2f(m - m_new) : 1.f;  // 0 when nothing was accumulated
+        m = m_new;
+        mrow[warp][lane] = m == -INFINITY ? 0.f : m;
+        any_move = __any_sync(0xffffffffu, move) && i > 0;
+        __syncwarp();
+        load_max();
+      }
+#pragma unroll
+      for (int j = 0; j < LM_CN; ++j) s[j] = exp2f(s[j] - mm[j]);
+      if (any_move) {  // every earlier tile's second product is complete: rescale the sums and O^T
+        mbar_wait_bounded(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+        __syncwarp();
+        tc_fence_after();
+#pragma unroll
+        for (int j = 0; j < LM_CN; ++j) l[j] *= frow[warp][n0 + j];
+        for (int p = 0; p < 2 * a.pairs; ++p) {
+          uint32_t r[16];
+          const uint32_t addr = tmem + lanes + NR * 2 + 16 * p;
+          tmem_ld16(addr, r);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * frow[warp][(p & 1) * 16 + j]);
+          tmem_st16(addr, r);
+        }
+        tmem_st_wait();
+      } else if (i > 1) {  // this P buffer was read by the second product two tiles ago
+        mbar_wait_bounded(&pv_done[i & 1], ((i >> 1) - 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
         __syncwarp();
       }
-      if (any_move) {
+      // P^T as the second product's B operand: row = 128 bytes of 64 keys, 16-byte pieces swizzled by the row
+      uint8_t* pb = s_p + (i & 1) * (NR * 128) + n0 * 128;
+      const int piece = key_in >> 3, in = (key_in & 7) * 2;
 #pragma unroll
-        for (int n = 0; n < NR; ++n) l[n] *= frow[warp][n];
-        if (i > 0) {
-          tc_fence_after();
-          for (int p = 0; p < a.pairs; ++p) {
-#pragma unroll
-            for (int c = 0; c < NR / 16; ++c) {
-              uint32_t r[16];
-              const uint32_t addr = tmem + lanes + NR * (1 + p) + 16 * c;
-              tmem_ld16(addr, r);
-              tmem_ld_wait();
-#pragma unroll
-              for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * frow[warp][16 * c + j]);
-              tmem_st16(addr, r);
-            }
-          }
-          tmem_st_wait();
-        }
-      }
-      // P^T as the second product's B operand: row n = 128 bytes of 64 keys, 16-byte pieces swizzled by the row
-      uint8_t* pb = s_p + (tid >> 6) * (NR * 128);
-      const int piece = (tid & 63) >> 3, in = (tid & 7) * 2;
-#pragma unroll
-      for (int n = 0; n < NR; ++n) {
-        const float p = exp2f(s[n] - mrow[warp][n]);
-        l[n] += p;
-        *reinterpret_cast<__nv_bfloat16*>(pb + n * 128 + ((piece ^ (n & 7)) << 4) + in) = __float2bfloat16(p);
+      for (int j = 0; j < LM_CN; ++j) {
+        l[j] += s[j];
+        *reinterpret_cast<__nv_bfloat16*>(pb + j * 128 + ((piece ^ (j & 7)) << 4) + in) = __float2bfloat16(s[j]);
       }
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       tc_fence_before();
-      mbar_arrive(&p_full);
+      mbar_arrive(&p_full[i & 1]);
     }
     // ---------------- sums over the keys, then the output
-    const float ws = butterfly_rows<NR>(l, lane, [](float x, float y) { return x + y; });
-    if (t_end > t_begin) mbar_wait_bounded(&pv_done, (t_end - t_begin - 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+    const float ws = butterfly_rows(l, lane, [](float x, float y) { return x + y; });
+    if (n > 0) mbar_wait_bounded(&pv_done[(n - 1) & 1], ((n - 1) >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
     __syncwarp();
     tc_fence_after();
-    asm volatile("bar.sync 1, 128;" ::: "memory");
-    if (lane < NR) wmax[warp][lane] = ws;
-    asm volatile("bar.sync 1, 128;" ::: "memory");
-    const int n_ = lane % NR;
-    float L = (wmax[0][n_] + wmax[1][n_]) + (wmax[2][n_] + wmax[3][n_]);
+    group_sync();
+    wmax[warp][lane] = ws;
+    group_sync();
+    float L = (wmax[0][lane] + wmax[1][lane]) + (wmax[2][lane] + wmax[3][lane]);
     if (sink > -INFINITY) L += exp2f(sink - m);  // the sink's share of the denominator, once
-    const int rows = min(NR, R - row_base);
-    if (a.n_splits == 1) {
-      if (lane < NR) frow[warp][lane] = L > 0.f ? 1.f / L : 0.f;
-      __syncwarp();
-      for (int p = 0; p < a.pairs; ++p) {
-        const int d = p * 128 + tid;
+    if (a.n_splits > 1) {
+      // O^T of this split into shared memory as [row][pad], next to its maxima and sums
+      if (warp == 0) part_ml[lane] = make_float2(m, L);
+      float* part = reinterpret_cast<float*>(smem);
+      for (int p = 0; n > 0 && p < 2 * a.pairs; ++p) {
+        uint32_t r[16];
+        tmem_ld16(tmem + lanes + NR * 2 + 16 * p, r);
+        tmem_ld_wait();
+        const int d = (p >> 1) * 128 + threadIdx.x;
+        if (d < a.pad) {
 #pragma unroll
-        for (int c = 0; c < NR / 16; ++c) {
-          uint32_t r[16];
-          tmem_ld16(tmem + lanes + NR * (1 + p) + 16 * c, r);
-          tmem_ld_wait();
-#pragma unroll
-          for (int j = 0; j < 16; ++j) {
-            const int n = 16 * c + j;
-            if (n < rows && d < a.pad) {
-              const int g = row_base + n;
-              a.out[((size_t)(g % a.H) * a.T + q0 + g / a.H) * a.pad + d] = __float2bfloat16(__uint_as_float(r[j]) * frow[warp][n]);
-            }
-          }
+          for (int j = 0; j < 16; ++j) part[((p & 1) * 16 + j) * a.pad + d] = __uint_as_float(r[j]);
         }
       }
     } else {
-      const size_t task0 = ((size_t)b * a.row_blocks + rb) * a.n_splits;
-      float* po = a.ws_o + (task0 + split) * NR * a.pad;
-      if (warp == 0 && lane < NR) {
-        a.ws_ml[((task0 + split) * NR + lane) * 2] = m;
-        a.ws_ml[((task0 + split) * NR + lane) * 2 + 1] = L;
-      }
-      if (t_end > t_begin) {
-        for (int p = 0; p < a.pairs; ++p) {
-          const int d = p * 128 + tid;
+      frow[warp][lane] = L > 0.f ? 1.f / L : 0.f;
+      __syncwarp();
+      // neighbouring lanes (values d, d + 1) swap one row of each pair of rows, so that a lane stores two values of one row
+      const bool odd = lane & 1;
+      for (int p = 0; p < 2 * a.pairs; ++p) {
+        uint32_t r[16];
+        tmem_ld16(tmem + lanes + NR * 2 + 16 * p, r);
+        tmem_ld_wait();
+        const int d = (p >> 1) * 128 + (threadIdx.x & ~1), c0 = (p & 1) * 16;
 #pragma unroll
-          for (int c = 0; c < NR / 16; ++c) {
-            uint32_t r[16];
-            tmem_ld16(tmem + lanes + NR * (1 + p) + 16 * c, r);
-            tmem_ld_wait();
-#pragma unroll
-            for (int j = 0; j < 16; ++j)
-              if (16 * c + j < rows && d < a.pad) po[(size_t)(16 * c + j) * a.pad + d] = __uint_as_float(r[j]);
-          }
+        for (int j = 0; j < 16; j += 2) {
+          const float lo_v = __uint_as_float(r[j]) * frow[warp][c0 + j], hi_v = __uint_as_float(r[j + 1]) * frow[warp][c0 + j + 1];
+          const float got = __shfl_xor_sync(0xffffffffu, odd ? lo_v : hi_v, 1);
+          const int row = c0 + j + (odd ? 1 : 0);
+          const float v0 = odd ? got : lo_v, v1 = odd ? hi_v : got;
+          const long long o = row_out[row];
+          if (o >= 0 && d < a.pad) *reinterpret_cast<uint32_t*>(a.out + o + d) = pack_bf16x2(v0, v1);
         }
-      }
-      __threadfence();
-      asm volatile("bar.sync 1, 128;" ::: "memory");
-      int* cnt = a.counters + (size_t)b * a.row_blocks + rb;
-      if (tid == 0) ticket = atomicAdd(cnt, 1);
-      asm volatile("bar.sync 1, 128;" ::: "memory");
-      if (ticket == a.n_splits - 1) {
-        __threadfence();
-        for (int n = warp; n < rows; n += 4) {  // a warp per row
-          float M = -INFINITY;
-          for (int s = 0; s < a.n_splits; ++s) M = fmaxf(M, __ldcg(a.ws_ml + ((task0 + s) * NR + n) * 2));
-          float den = 0.f;
-          for (int s = 0; s < a.n_splits; ++s) {
-            const float ms = __ldcg(a.ws_ml + ((task0 + s) * NR + n) * 2);
-            if (ms > -INFINITY) den += exp2f(ms - M) * __ldcg(a.ws_ml + ((task0 + s) * NR + n) * 2 + 1);
-          }
-          const float inv = den > 0.f ? 1.f / den : 0.f;
-          const int g = row_base + n;
-          __nv_bfloat16* o = a.out + ((size_t)(g % a.H) * a.T + q0 + g / a.H) * a.pad;
-          for (int d = lane * 4; d < a.pad; d += 128) {
-            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-            for (int s = 0; s < a.n_splits; ++s) {
-              const float ms = __ldcg(a.ws_ml + ((task0 + s) * NR + n) * 2);
-              if (ms == -INFINITY || (s * per >= tiles)) continue;  // that split saw no key of this row (or had no tile)
-              const float w = exp2f(ms - M) * inv;
-              const float4 v = __ldcg(reinterpret_cast<const float4*>(a.ws_o + ((task0 + s) * NR + n) * (size_t)a.pad + d));
-              acc.x += w * v.x;
-              acc.y += w * v.y;
-              acc.z += w * v.z;
-              acc.w += w * v.w;
-            }
-            *reinterpret_cast<uint2*>(o + d) = make_uint2(pack_bf16x2(acc.x, acc.y), pack_bf16x2(acc.z, acc.w));
-          }
-        }
-        if (tid == 0) *cnt = 0;  // re-armed for the next launch / graph replay
       }
     }
+  }
+  if (a.n_splits > 1) {
+    __syncwarp();
+    cluster_sync_all();
+    merge_splits(a, smem, part_ml, row_out, split, tiles, per);
+    __syncwarp();
+    cluster_sync_all();  // every peer has finished reading this CTA's partial
   }
   if (abort_flag) {
     // a wait gave up: give copies that may still be in flight time to land before the CTA exits
@@ -430,25 +488,29 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 5) tmem_dealloc(tmem, tmem_cols);
+  if (warp == LM_WARP_MMA) tmem_dealloc(tmem, tmem_cols);
 }
-
 struct LatentMmaPlan {
-  int ok, pairs, rest, slots, smem;
+  int ok, pairs, rest, slots, rest_slots, smem;
 };
 
 // Shared-memory plan for rows of `width` values of which the first `pad` are the latent part.
-inline LatentMmaPlan latent_mma_plan(int nr, int pad, int width, int page) {
-  LatentMmaPlan p{0, (pad + 127) / 128, 0, 0, 0};
+inline LatentMmaPlan latent_mma_plan(int pad, int width, int page) {
+  LatentMmaPlan p{0, (pad + 127) / 128, 0, 0, 0, 0};
   const int nch = (width + 63) / 64;
   p.rest = nch > 2 * p.pairs ? nch - 2 * p.pairs : 0;
-  const int fixed = p.rest * LM_CHUNK + nch * nr * 128 + 2 * nr * 128 + 1024;
-  const int budget = 225 * 1024;  // the static variables of the kernel share the 227 KB
-  p.slots = (budget - fixed) / LM_PAIR;
-  if (p.slots > 2 * p.pairs) p.slots = 2 * p.pairs;
+  const int budget = LM_DYN_SMEM;  // the static variables of the kernel share the 227 KB
+  const int fixed = nch * LM_NR * 128 + 2 * LM_NR * 128 + 1024;
+  p.rest_slots = 2;
+  p.slots = (budget - fixed - 2 * p.rest * LM_CHUNK) / LM_PAIR;
+  if (p.slots < 2 * p.pairs && p.rest > 0) {
+    p.rest_slots = 1;
+    p.slots = (budget - fixed - p.rest * LM_CHUNK) / LM_PAIR;
+  }
+  if (p.slots > 4 * p.pairs) p.slots = 4 * p.pairs;
   if (p.slots > LM_MAX_SLOTS) p.slots = LM_MAX_SLOTS;
-  p.smem = p.slots * LM_PAIR + fixed;
-  p.ok = p.slots >= p.pairs && page % 8 == 0 && LM_KEYS % page == 0 && width % 16 == 0 && nr * (1 + p.pairs) <= 512;
+  p.smem = p.slots * LM_PAIR + p.rest_slots * p.rest * LM_CHUNK + fixed;
+  p.ok = p.slots >= p.pairs && page % 8 == 0 && LM_KEYS % page == 0 && width % 16 == 0 && LM_NR * (2 + p.pairs) <= 512;
   return p;
 }
 

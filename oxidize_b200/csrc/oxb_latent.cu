@@ -62,44 +62,31 @@ OXB_API int oxb_latent_attention_simt(const void* q, void* out, const void* cach
 }
 
 // 1 when latent_attention_mma_kernel covers rows of this shape (else: the plain kernel)
-OXB_API int oxb_latent_mma_supported(int nr, int pad, int width, int page) {
-  return (nr == 16 || nr == 32) && latent_mma_plan(nr, pad, width, page).ok;
-}
+OXB_API int oxb_latent_mma_supported(int pad, int width, int page) { return latent_mma_plan(pad, width, page).ok; }
 
-template <int NR>
-static int latent_mma_launch(const CUtensorMap& tk, const CUtensorMap& tq, const LatentMmaArgs& a, int B, int smem,
-                             cudaStream_t stream) {
+// Latent attention, absorbed form, bf16: q [T, H, width] and the cache rows [num_blocks * page, width]; the B sequences
+// have at most max_query_len rows each.  n_splits (at most 8) CTAs share the keys of a block of 32 rows.
+OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache, const int* block_tables, const int* seq_lens,
+                                     const int* query_start, const float* sink, int B, int max_blocks, int T, int H, int pad,
+                                     int width, int page, int num_blocks, int window, float scale, int max_query_len,
+                                     int n_splits, cudaStream_t stream) {
+  if (T <= 0 || B <= 0 || max_query_len <= 0) return 0;
+  const LatentMmaPlan pl = latent_mma_plan(pad, width, page);
+  if (!pl.ok || B > 65535) return (int)cudaErrorInvalidValue;
+  if (n_splits > LM_MAX_SPLITS) return (int)cudaErrorInvalidValue;
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
   if (!configured[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(latent_attention_mma_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);
-    if (e != cudaSuccess) return (int)e;
+    const cudaError_t ce = cudaFuncSetAttribute(latent_attention_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LM_DYN_SMEM);
+    if (ce != cudaSuccess) return (int)ce;
     configured[dev] = true;
   }
-  const cudaError_t le = oxb_launch(latent_attention_mma_kernel<NR>, dim3(a.row_blocks * a.n_splits, B), dim3(LM_THREADS),
-                                    (size_t)smem, stream, tk, tq, a);
-  if (le != cudaSuccess) return (int)le;
-  OXB_CHECK_LAUNCH();
-  return 0;
-}
-
-// Latent attention, absorbed form, bf16: q [T, H, width] and the cache rows [num_blocks * page, width]; the B sequences
-// have at most max_query_len rows each.  n_splits > 1 needs ws_o [B * row_blocks * n_splits * nr * pad] and ws_ml
-// [.. * nr * 2] floats and one zeroed ticket per (sequence, row block), row_blocks = ceil(max_query_len * H / nr).
-OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache, const int* block_tables, const int* seq_lens,
-                                     const int* query_start, const float* sink, int B, int max_blocks, int T, int H, int pad,
-                                     int width, int page, int num_blocks, int window, float scale, int nr, int max_query_len,
-                                     int n_splits, float* ws_o, float* ws_ml, int* counters, cudaStream_t stream) {
-  if (T <= 0 || B <= 0 || max_query_len <= 0) return 0;
-  const LatentMmaPlan pl = latent_mma_plan(nr, pad, width, page);
-  if ((nr != 16 && nr != 32) || !pl.ok || B > 65535) return (int)cudaErrorInvalidValue;
-  if (n_splits > 1 && (ws_o == nullptr || ws_ml == nullptr || counters == nullptr)) return (int)cudaErrorInvalidValue;
   CUtensorMap tk, tq;
   int e = oxb_make_tmap_2d(&tk, cache, (uint64_t)num_blocks * page, width, (uint64_t)width * 2, page, 64, 2);
   if (e) return e;
-  e = oxb_make_tmap_2d(&tq, q, (uint64_t)T * H, width, (uint64_t)width * 2, nr, 64, 2);
+  e = oxb_make_tmap_2d(&tq, q, (uint64_t)T * H, width, (uint64_t)width * 2, LM_NR, 64, 2);
   if (e) return e;
   LatentMmaArgs a;
   a.block_tables = block_tables;
@@ -107,9 +94,6 @@ OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache
   a.query_start = query_start;
   a.sink = sink;
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
-  a.ws_o = ws_o;
-  a.ws_ml = ws_ml;
-  a.counters = counters;
   a.max_blocks = max_blocks;
   a.T = T;
   a.H = H;
@@ -119,10 +103,17 @@ OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache
   a.num_blocks = num_blocks;
   a.window = window;
   a.n_splits = n_splits < 1 ? 1 : n_splits;
-  a.row_blocks = (max_query_len * H + nr - 1) / nr;
   a.pairs = pl.pairs;
   a.rest = pl.rest;
   a.slots = pl.slots;
+  a.rest_slots = pl.rest_slots;
   a.scale_log2 = scale * 1.4426950408889634f;
-  return nr == 16 ? latent_mma_launch<16>(tk, tq, a, B, pl.smem, stream) : latent_mma_launch<32>(tk, tq, a, B, pl.smem, stream);
+  const dim3 grid((max_query_len * H + LM_NR - 1) / LM_NR * a.n_splits, B);
+  const cudaError_t le =
+      a.n_splits > 1 ? oxb_launch_cluster(latent_attention_mma_kernel, grid, dim3(LM_THREADS), dim3(a.n_splits, 1, 1),
+                                          (size_t)pl.smem, stream, tk, tq, a)
+                     : oxb_launch(latent_attention_mma_kernel, grid, dim3(LM_THREADS), (size_t)pl.smem, stream, tk, tq, a);
+  if (le != cudaSuccess) return (int)le;
+  OXB_CHECK_LAUNCH();
+  return 0;
 }

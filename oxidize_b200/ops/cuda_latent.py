@@ -27,8 +27,8 @@ def lib():
         L.oxb_latent_prep.argtypes = ([vp, i32, i32, vp, vp, vp, i32, i32, i32, vp, f32] + [i32] * 6 + [vp, i32, vp, vp, i32, vp,
                                       i32, i32, vp])
         L.oxb_latent_attention_simt.argtypes = [vp, vp, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp]
-        L.oxb_latent_mma_supported.argtypes = [i32] * 4
-        L.oxb_latent_attention_mma.argtypes = [vp] * 7 + [i32] * 9 + [f32] + [i32] * 3 + [vp] * 4
+        L.oxb_latent_mma_supported.argtypes = [i32] * 3
+        L.oxb_latent_attention_mma.argtypes = [vp] * 7 + [i32] * 9 + [f32] + [i32] * 2 + [vp]
         L.oxb_gemm_batched.argtypes = [vp, vp, vp, i64] + [i32] * 5 + [vp]
         _declared = True
     return L
@@ -139,10 +139,10 @@ def attention_simt(q, kv, layer: int, meta, spec, sink, out):
 
 
 def mma_splits(B: int, row_blocks: int, window: int, max_len: int, sms: int) -> int:
-    """Key splits of the tensor-core kernel: as many as fit one wave of CTAs (one per SM), at least one 128-key tile each."""
+    """Key splits of the tensor-core kernel: as many as fit one wave of CTAs (one per SM), at least two 64-key tiles each."""
     span = min(window, max_len) if window > 0 else max_len
     tiles = span // 128 + 1
-    return max(1, min(sms // max(1, B * row_blocks), tiles, 16))
+    return max(1, min(sms // max(1, B * row_blocks), tiles, 8))
 
 
 def attention_mma(q, kv, layer: int, meta, spec, sink, out, splits: Optional[int] = None):
@@ -150,24 +150,15 @@ def attention_mma(q, kv, layer: int, meta, spec, sink, out, splits: Optional[int
     T, H, width = q.shape
     B = meta.seq_lens.shape[0]
     mq = max(1, meta.max_query_len)
-    nr = 16 if mq * H <= 16 else 32
-    if not lib().oxb_latent_mma_supported(nr, spec.latent_pad, width, kv.page_size):
+    if not lib().oxb_latent_mma_supported(spec.latent_pad, width, kv.page_size):
         return False
-    row_blocks = (mq * H + nr - 1) // nr
-    sc = opcuda.scratch(q.device)
+    row_blocks = (mq * H + 31) // 32
     if splits is None:
         splits = mma_splits(B, row_blocks, spec.window, meta.max_seq_len or kv.page_size, opcuda.sm_count(q.device))
-    if B * row_blocks > sc.attn_counters.numel():
-        splits = 1
-    ws_o = ws_ml = cnt = None
-    if splits > 1:
-        tasks = B * row_blocks * splits
-        ws_o, ws_ml = sc.attn(tasks * nr * spec.latent_pad, tasks * nr * 2)
-        cnt = sc.attn_counters
     _check(lib().oxb_latent_attention_mma(q.data_ptr(), out.data_ptr(), kv.data[layer].data_ptr(), meta.block_tables.data_ptr(),
                                           meta.seq_lens.data_ptr(), meta.query_start.data_ptr(), _p(sink), B,
                                           meta.block_tables.stride(0), T, H, spec.latent_pad, width, kv.page_size, kv.num_blocks,
-                                          spec.window, spec.scale, nr, mq, splits, _p(ws_o), _p(ws_ml), _p(cnt), _stream()),
+                                          spec.window, spec.scale, mq, splits, _stream()),
            "oxb_latent_attention_mma")
     return True
 
