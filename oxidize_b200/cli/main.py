@@ -15,6 +15,8 @@ import sys
 import time
 from typing import List, Optional
 
+from ..formats.layered import LayeredCheckpoint, is_layered_checkpoint, open_checkpoint
+
 VERBS = ("run", "chat", "serve", "pull", "show", "list", "inspect", "bench", "gpu-cluster")
 DEAD_BACKENDS = ("metal", "mlx", "rocm", "vulkan", "intel-arc")
 MODEL_DIR = os.path.expanduser(os.environ.get("OXIDIZE_MODEL_DIR", "~/.cache/oxidize/models"))
@@ -98,6 +100,8 @@ def build_parser() -> argparse.ArgumentParser:
     a("--max-batched-tokens", type=int, default=0, help="tokens per engine step; 0 = chosen from the model's shapes")
     a("--fused-comm", default="on", choices=["on", "off"])
     a("--weights-dtype", default="auto", choices=["auto", "bf16", "fp8", "nvfp4"])
+    a("--compute-dtype", default="auto", choices=["auto", "bf16", "f32"],
+      help="activations and matrix products on the GPU; f32 = true 32-bit, for models whose kernels all have it")
     a("--rope-pairing", default=None, choices=["split_half", "adjacent"])
     a("--cuda-graphs", action="store_true", default=True)
     a("--no-cuda-graphs", action="store_true")
@@ -224,6 +228,9 @@ def resolve_model(name: Optional[str]) -> str:
     for cand in (name, os.path.join(MODEL_DIR, name), os.path.join(MODEL_DIR, name + ".gguf")):
         if os.path.isfile(cand):
             return cand
+    for cand in (name, os.path.join(MODEL_DIR, name)):
+        if os.path.isdir(cand) and is_layered_checkpoint(cand):
+            return cand  # served as it is (formats.layered)
     if os.path.isdir(name) and os.path.isfile(os.path.join(name, "config.json")):
         return convert_on_the_fly(name)
     if name.startswith("hf://") or "/" in name and not os.path.exists(name):
@@ -236,13 +243,12 @@ def make_engine(args, passed: set, device_index: Optional[int] = None):
     import torch
 
     from ..engine.llm import LLM, EngineConfig
-    from ..formats.gguf import load_gguf
     from ..utils import autotune
 
     if args.backend in DEAD_BACKENDS:
         raise SystemExit(f"error: backend {args.backend!r} is not available in this build; use cpu or cuda")
     path = resolve_model(args.model)
-    g = load_gguf(path)
+    g = open_checkpoint(path)
     if args.cpu_optimized and args.backend != "cuda":
         # the CPU path is torch's: use every core for the matrix products, flush denormals (the reference pins its own
         # thread pool instead, oxidize-cli/src/main.rs:306)
@@ -267,12 +273,13 @@ def make_engine(args, passed: set, device_index: Optional[int] = None):
     if args.turboquant_kv and "kv_cache_dtype" not in passed:
         kvd = "q8"
     if kvd == "auto":
-        kvd = plan.kv_cache_dtype if (use_plan and backend == plan.backend) else "auto"
+        # (latent cache rows of a layer-list model are kept in the compute type: the engine's own choice)
+        kvd = plan.kv_cache_dtype if (use_plan and backend == plan.backend and not isinstance(g, LayeredCheckpoint)) else "auto"
     tp = args.tp or (args.gpus if args.parallelism == "tensor" and args.gpus > 1 else 0) or 1
     ec = EngineConfig(kv_cache_dtype=kvd, kv_page_size=args.kv_page_size,
                       max_model_len=args.ctx_size or plan.ctx_size, max_num_seqs=args.max_running or plan.max_num_seqs,
                       max_num_batched_tokens=args.max_batched_tokens, prefill_chunk_size=args.prefill_batch_size,
-                      cuda_graphs=not args.no_cuda_graphs, tp_size=tp, ep_size=args.ep or tp, pp_size=max(1, args.pp),
+                      compute_dtype=args.compute_dtype, cuda_graphs=not args.no_cuda_graphs, tp_size=tp, ep_size=args.ep or tp, pp_size=max(1, args.pp),
                       fused_comm=args.fused_comm == "on",
                       resident_layers=max(1, args.layer_cache) if args.layer_wise else 0,
                       weight_transcode=("Q4_0" if args.turboquant_bits == 4 else "Q8_0")
@@ -282,8 +289,11 @@ def make_engine(args, passed: set, device_index: Optional[int] = None):
         import psutil
 
         n = max(1, fp.n_layers)
-        layer_bytes = sum(t.nbytes for name, t in g.tensors.items() if name.startswith("blk.")) // n
-        fixed = sum(t.nbytes for name, t in g.tensors.items() if not name.startswith("blk."))
+        def in_layer(name: str) -> bool:
+            return name.startswith("blk.") or (name[0] == "l" and name[1 : name.find(".")].isdigit())
+
+        layer_bytes = sum(t.nbytes for name, t in g.tensors.items() if in_layer(name)) // n
+        fixed = sum(t.nbytes for name, t in g.tensors.items() if not in_layer(name))
         kv = autotune.kv_bytes_per_token(fp, "bf16" if backend == "cuda" else "f32", tp) * ec.max_model_len * min(ec.max_num_seqs, 8)
         if backend == "cuda":
             free, _total = torch.cuda.mem_get_info()
@@ -486,9 +496,7 @@ def cmd_serve(args, passed) -> int:
 
 
 def cmd_show(args, passed, verbose: bool) -> int:
-    from ..formats.gguf import load_gguf
-
-    g = load_gguf(resolve_model(args.model))
+    g = open_checkpoint(resolve_model(args.model))
     info = {"path": g.path, "version": g.version, "architecture": g.architecture, "alignment": g.alignment,
             "tensor_count": len(g.tensors), "metadata": {k: (v if not isinstance(v, list) or len(v) <= 8 else
                                                              f"[{len(v)} items]") for k, v in g.metadata.items()}}
@@ -508,7 +516,10 @@ def cmd_list(args) -> int:
         print(f"(no models under {MODEL_DIR})")
         return 0
     for f in sorted(os.listdir(MODEL_DIR)):
-        if f.endswith(".gguf"):
+        if is_layered_checkpoint(os.path.join(MODEL_DIR, f)):
+            size = sum(os.path.getsize(os.path.join(MODEL_DIR, f, x)) for x in os.listdir(os.path.join(MODEL_DIR, f)))
+            print(f"{f}\t{size / 1e9:.2f} GB")
+        elif f.endswith(".gguf"):
             print(f"{f}\t{os.path.getsize(os.path.join(MODEL_DIR, f)) / 1e9:.2f} GB")
     return 0
 

@@ -417,7 +417,7 @@ def attach_speculation(llm, draft_model_path: Optional[str], k: int = 4, use_mtp
     long-context decode step is bound by, and the target's verification keeps the output exact."""
     c = llm.config
     if quantspec and not draft_model_path:
-        if llm.cfg.is_ssm or llm.cfg.is_mla:
+        if llm.cfg.is_ssm or llm.cfg.is_mla or llm.cfg.is_layered:
             raise ValueError("self-speculation over a 4-bit cache needs ordinary attention layers")
         if llm.model.kv_head_dim % 32:
             raise ValueError("a 4-bit cache needs a head width that is a multiple of 32")
