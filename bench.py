@@ -63,6 +63,9 @@ def parse_args():
     ap.add_argument("--expert-quant", default=None, help="encoding of the MoE expert matrices when it differs from --quant")
     ap.add_argument("--draft-model", default=None, help="preset of a draft model: measure speculative decoding as well")
     ap.add_argument("--draft-tokens", type=int, default=4)
+    ap.add_argument("--layered", default=None, metavar="WIDTHxHEADS",
+                    help="instead of the headline workload: a model that lists its layers (Vefilix) beside the closest uniform "
+                         "models of that size (see bench/layered_bench.py), e.g. 4096x32")
     return ap.parse_args()
 
 
@@ -132,6 +135,11 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.layered:
+        sys.path.insert(0, os.path.join(ROOT, "bench"))
+        import layered_bench
+
+        return layered_bench.main(args)
     # last-resort guard: never sit on a GPU box forever if something blocks
     guard = threading.Timer(1500.0, lambda: os._exit(3))
     guard.daemon = True

@@ -168,16 +168,19 @@ def latent_mixer(x, m, spec, rope, meta, kv, layer: int, eps: float) -> torch.Te
 
     if kv.data[layer].dtype != x.dtype:
         raise ValueError(f"latent cache rows are kept in the compute type on the GPU ({x.dtype}), not {kv.dtype_name}")
-    op = operands(m, spec, x.dtype)
-    T, H = x.shape[0], op.heads
-    qkv = linear(x, m.q)
-    q_nope = torch.empty(H, T, op.nope_ld, dtype=x.dtype, device=x.device)
-    q = torch.empty(T, H, spec.row_dim, dtype=x.dtype, device=x.device)
+    return latent_core(linear(x, m.q), m, spec, rope, meta, kv, layer, eps, operands(m, spec, x.dtype))
+
+
+def latent_core(qkv, m, spec, rope, meta, kv, layer: int, eps: float, op: LatentOperands) -> torch.Tensor:
+    """From the layer's projections to its heads' outputs [T, heads * v_dim]."""
+    T, H, dt, dev = qkv.shape[0], op.heads, qkv.dtype, qkv.device
+    q_nope = torch.empty(H, T, op.nope_ld, dtype=dt, device=dev)
+    q = torch.empty(T, H, spec.row_dim, dtype=dt, device=dev)
     latent_prep(qkv, m, spec, rope, meta, kv, layer, eps, op, q_nope=q_nope, q_rows=q)
     batched(q_nope, op.k, q, spec.row_dim, H * spec.row_dim)
-    o = torch.empty(H, T, spec.latent_pad, dtype=x.dtype, device=x.device)
-    if x.dtype != torch.bfloat16 or not attention_mma(q, kv, layer, meta, spec, m.sink, o):
+    o = torch.empty(H, T, spec.latent_pad, dtype=dt, device=dev)
+    if dt != torch.bfloat16 or not attention_mma(q, kv, layer, meta, spec, m.sink, o):
         attention_simt(q, kv, layer, meta, spec, m.sink, o)
-    out = torch.empty(T, H * spec.v_dim, dtype=x.dtype, device=x.device)
+    out = torch.empty(T, H * spec.v_dim, dtype=dt, device=dev)
     batched(o, op.v, out, spec.v_dim, H * spec.v_dim)
     return out

@@ -294,6 +294,8 @@ def synth_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: int = 0, 
     Every rank draws its own shard from a rank-specific stream; replicated tensors (norms,
     embedding, router) use a shared stream so that all ranks hold identical copies."""
     device = torch.device(device)
+    if cfg.is_layered:
+        return synth_layered_weights(cfg, device, quant, seed, tp_rank, tp_size)
     shared = torch.Generator(device=device)
     shared.manual_seed(seed)
     own = torch.Generator(device=device)
@@ -340,6 +342,49 @@ def synth_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: int = 0, 
     else:
         head = _rand_matrix(v1 - v0, h, pick_type(quant, "output", 0, L, h), device, own)
     return ModelWeights(cfg, embed, layers, ones(h), LinearWeight([head]), [], tp_rank, tp_size, ep_rank, ep_size, l0, v0)
+
+
+def synth_layered_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: int = 0, tp_rank: int = 0,
+                          tp_size: int = 1) -> ModelWeights:
+    """``synth_weights`` for a model that lists its layers (bfloat16 or float32 weights)."""
+    from ..models.layered import dense_qtensor, latent_weights
+
+    if quant.upper() not in ("BF16", "F32"):
+        raise ValueError("models with listed layers are drawn in BF16 or F32")
+    dt = torch.bfloat16 if quant.upper() == "BF16" else torch.float32
+    gens = [torch.Generator(device=device), torch.Generator(device=device)]
+    gens[0].manual_seed(seed)
+    gens[1].manual_seed(seed * 1000003 + 7919 * (tp_rank + 1))
+
+    def mat(out_f: int, in_f: int, own: bool = True) -> torch.Tensor:
+        return (torch.randn(out_f, in_f, generator=gens[1 if own else 0], device=device) * WEIGHT_STD).to(dt)
+
+    def ones(n: int) -> torch.Tensor:
+        return torch.ones(n, dtype=torch.float32, device=device)
+
+    h, bias = cfg.hidden_size, cfg.norm_kind == "layer"
+    zeros = (lambda n: torch.zeros(n, dtype=torch.float32, device=device)) if bias else (lambda n: None)
+    layers = []
+    for spec in cfg.layer_specs:
+        m, f = spec.mixer, spec.ffn
+        H, own = m.heads // tp_size, m.kv_from is None
+        mla = latent_weights(m, mat(H * m.qk_dim, h), mat(m.kv_rank + m.rope_dim, h, own=False) if own else None,
+                             ones(m.kv_rank) if own else None, mat(H * m.nope_dim, m.kv_rank), mat(H * m.v_dim, m.kv_rank),
+                             torch.zeros(H, device=device) if m.sink else None)
+        lw = LayerWeights(attn_norm=ones(h), attn_norm_bias=zeros(h), wqkv=None, wo=LinearWeight([dense_qtensor(mat(h, H * m.v_dim))]),
+                          ffn_norm=None, mla=mla)
+        if f is not None:
+            lw.ffn_norm, lw.ffn_norm_bias = ones(h), zeros(h)
+            lw.w_up = LinearWeight([dense_qtensor(mat(f.size // tp_size, h))])
+            lw.w_down = LinearWeight([dense_qtensor(mat(h, f.size // tp_size))])
+        layers.append(lw)
+    v = cfg.vocab_size // tp_size
+    mw = ModelWeights(cfg, dense_qtensor(mat(cfg.vocab_size, h, own=False)), layers, ones(h), LinearWeight([dense_qtensor(mat(v, h))]),
+                      [], tp_rank, tp_size, 0, 1, 0, v * tp_rank)
+    mw.out_norm_bias = zeros(h)
+    if cfg.embed_norm:
+        mw.embed_norm, mw.embed_norm_bias = ones(h), zeros(h)
+    return mw
 
 
 def _main(argv=None) -> int:

@@ -37,7 +37,7 @@ CONFIGS = {
 gpu = pytest.mark.gpu
 PATHS = [pytest.param("cpu", "float32", id="cpu"), pytest.param("cuda:0", "float32", id="gpu32", marks=gpu),
          pytest.param("cuda:0", "bfloat16", id="gpu16", marks=gpu)]
-TOL = {("cpu", "float32"): 3e-5, ("cuda:0", "float32"): 3e-5, ("cuda:0", "bfloat16"): 4e-2}
+TOL = {("cpu", "float32"): 3e-5, ("cuda:0", "float32"): 3e-5, ("cuda:0", "bfloat16"): 0.12}
 
 
 @functools.lru_cache(None)
@@ -70,6 +70,7 @@ def check(got, want, tol, what=""):
     d -= d.mean(-1, keepdims=True)
     err = np.sqrt((d * d).mean(-1)) / want.std()
     assert err.max() < tol, f"{what}: worst {err.max():.3g} at row {int(err.argmax())}"
+    assert err.mean() < tol / 5, f"{what}: mean {err.mean():.3g}"  # (a few rows amplify rounding, most do not)
 
 
 def feed(rep, name, tokens, cuts, rid="a", end=True):
