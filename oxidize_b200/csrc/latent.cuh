@@ -32,8 +32,8 @@ struct LatentPrepArgs {
   void* q_nope;         // absorbed form: [H, T, nope_ld], the operand of the per-head products with W_uk
   int nope_ld;
   void* q_rows;         // absorbed form: [T, H, width], of which the rotated part is written here
-  void* q_full;         // expanded form (instead of the two above): [T, H, full_ld] = nope | rotated part | zeros
-  int full_ld;
+  void* q_full;         // expanded form (instead of the two above): [T, H, full_ld], the rotated part at full_rot, zeros elsewhere
+  int full_ld, full_rot;
   void* cache;          // layer base [blocks, page, width]
   int page, num_blocks;
 };
@@ -99,7 +99,10 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepArgs a
     if (a.q_full != nullptr) {
       T* dst = reinterpret_cast<T*>(a.q_full) + ((size_t)t * a.H + h) * a.full_ld;
       for (int i = tid; i < a.full_ld; i += blockDim.x)
-        dst[i] = i < a.nope ? q[i] : lat_from<T>(i < qk ? lat_rotated(q + a.nope, i - a.nope, cs, a.rot, a.pairing) : 0.f);
+        dst[i] = i < a.nope ? q[i]
+                            : lat_from<T>((i >= a.full_rot && i < a.full_rot + a.rot)
+                                              ? lat_rotated(q + a.nope, i - a.full_rot, cs, a.rot, a.pairing)
+                                              : 0.f);
       continue;
     }
     T* qn = reinterpret_cast<T*>(a.q_nope) + ((size_t)h * a.T + t) * a.nope_ld;

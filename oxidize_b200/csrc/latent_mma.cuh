@@ -46,7 +46,7 @@ struct LatentMmaArgs {
 
 // An MN-major operand (64 contiguous values per 128-byte row, rows = the K dimension) with the 128-byte swizzle: 64-value
 // chunks lie the descriptor's leading offset apart, groups of 8 rows its stride offset (1024 bytes).
-constexpr uint32_t UMMA_A_MN_MAJOR = 1u << 15;
+constexpr uint32_t UMMA_A_MN_MAJOR = 1u << 15, UMMA_B_MN_MAJOR = 1u << 16;  // instruction descriptor bits
 
 __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
   asm volatile(

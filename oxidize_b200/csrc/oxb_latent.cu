@@ -4,6 +4,7 @@
 #include "gemm_f32.cuh"
 #include "latent.cuh"
 #include "latent_mma.cuh"
+#include "latent_prefill.cuh"
 #include "residual_norm.cuh"
 using namespace oxb;
 
@@ -26,12 +27,12 @@ OXB_API int oxb_gemm_f32(const float* x, const float* w, float* y, const float* 
 
 OXB_API int oxb_latent_prep(const void* qkv, int ld, int dtype, const int* positions, const int* slots, const float* cos_sin,
                             int max_pos, int rot, int pairing, const float* norm_w, float eps, int T, int H, int nope, int rank,
-                            int pad, int width, void* q_nope, int nope_ld, void* q_rows, void* q_full, int full_ld, void* cache,
+                            int pad, int width, void* q_nope, int nope_ld, void* q_rows, void* q_full, int full_ld, int full_rot, void* cache,
                             int page, int num_blocks, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (rot <= 0 || rot % 2 != 0 || rank > pad || pad + rot > width || page <= 0) return (int)cudaErrorInvalidValue;
   const LatentPrepArgs a{qkv, ld, positions, slots, cos_sin, max_pos, rot, pairing, norm_w, eps, T, H, nope, rank, pad, width,
-                         q_nope, nope_ld, q_rows, q_full, full_ld, cache, page, num_blocks};
+                         q_nope, nope_ld, q_rows, q_full, full_ld, full_rot, cache, page, num_blocks};
   const dim3 grid(T, 1 + (H + LAT_PREP_HEADS - 1) / LAT_PREP_HEADS);
   if (dtype == 0) oxb_launch(latent_prep_kernel<float>, grid, dim3(128), 0, stream, a);
   else oxb_launch(latent_prep_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, a);
@@ -113,6 +114,73 @@ OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache
       a.n_splits > 1 ? oxb_launch_cluster(latent_attention_mma_kernel, grid, dim3(LM_THREADS), dim3(a.n_splits, 1, 1),
                                           (size_t)pl.smem, stream, tk, tq, a)
                      : oxb_launch(latent_attention_mma_kernel, grid, dim3(LM_THREADS), (size_t)pl.smem, stream, tk, tq, a);
+  if (le != cudaSuccess) return (int)le;
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+// Dense copies of the cache rows that the sequences of a step see (latent_gather_kernel); `rows` = span_off[B].
+OXB_API int oxb_latent_gather(const void* cache, const int* block_tables, const int* span_lo, const int* span_off, int B, int rows,
+                              int max_blocks, int pad, int width, int page, int num_blocks, void* lat, void* rot,
+                              cudaStream_t stream) {
+  if (rows <= 0 || B <= 0) return 0;
+  if (pad % 8 != 0 || width % 8 != 0 || page <= 0) return (int)cudaErrorInvalidValue;
+  oxb_launch(latent_gather_kernel, dim3((rows + 3) / 4), dim3(128), 0, stream, reinterpret_cast<const __nv_bfloat16*>(cache),
+             block_tables, span_lo, span_off, B, max_blocks, pad, width, page, num_blocks, reinterpret_cast<__nv_bfloat16*>(lat),
+             reinterpret_cast<__nv_bfloat16*>(rot));
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+// 1 when latent_prefill_kernel covers heads of these sizes
+OXB_API int oxb_latent_prefill_supported(int nope, int rot, int v) { return latent_prefill_plan(nope, rot, v).smem > 0; }
+
+// Attention of long portions over expanded keys and values: q [T, H, full_ld] (nope | rotated part, each padded with zeros
+// to a multiple of 16), kv [rows, kv_ld] (head h's key at h * nope_ld, its value at v_off + h * v_ld, all multiples of 8),
+// rot [rows, rot padded to 16]; out [T, H * v].
+OXB_API int oxb_latent_prefill(const void* q, const void* kv, const void* rot_rows, void* out, const int* query_start,
+                               const int* seq_lens, const int* span_lo, const int* span_off, const float* sink, int B, int T, int H,
+                               int rows, int nope, int rot, int v, int kv_ld, int nope_ld, int v_off, int v_ld, int window,
+                               float scale, int max_query_len, cudaStream_t stream) {
+  if (T <= 0 || B <= 0 || max_query_len <= 0 || rows <= 0) return 0;
+  const LatentPrefillPlan pl = latent_prefill_plan(nope, rot, v);
+  if (pl.smem == 0 || kv_ld % 8 != 0 || nope_ld % 8 != 0 || v_off % 8 != 0 || v_ld % 8 != 0 || H > 65535 || B > 65535)
+    return (int)cudaErrorInvalidValue;
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
+  if (!configured[dev]) {
+    const cudaError_t ce = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LM_DYN_SMEM);
+    if (ce != cudaSuccess) return (int)ce;
+    configured[dev] = true;
+  }
+  LatentPrefillArgs a;
+  a.query_start = query_start;
+  a.seq_lens = seq_lens;
+  a.span_lo = span_lo;
+  a.span_off = span_off;
+  a.sink = sink;
+  a.out = reinterpret_cast<__nv_bfloat16*>(out);
+  a.H = H;
+  a.window = window;
+  a.nope16 = (nope + 15) / 16;
+  a.rot16 = (rot + 15) / 16;
+  a.full_ld = 16 * (a.nope16 + a.rot16);
+  a.nope_ld = nope_ld;
+  a.v_off = v_off;
+  a.v_ld = v_ld;
+  a.v = v;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  CUtensorMap tq, tkv, tr;
+  int e = oxb_make_tmap_2d(&tq, q, T, (uint64_t)H * a.full_ld, (uint64_t)H * a.full_ld * 2, LP_M, 64, 2);
+  if (e) return e;
+  e = oxb_make_tmap_2d(&tkv, kv, rows, kv_ld, (uint64_t)kv_ld * 2, LP_KEYS, 64, 2);
+  if (e) return e;
+  e = oxb_make_tmap_2d(&tr, rot_rows, rows, 16 * a.rot16, (uint64_t)a.rot16 * 32, LP_KEYS, 64, 2);
+  if (e) return e;
+  const dim3 grid((max_query_len + 2 * LP_M - 1) / (2 * LP_M), H, B);
+  const cudaError_t le = oxb_launch(latent_prefill_kernel, grid, dim3(LP_THREADS), (size_t)pl.smem, stream, tq, tkv, tr, a);
   if (le != cudaSuccess) return (int)le;
   OXB_CHECK_LAUNCH();
   return 0;

@@ -24,11 +24,14 @@ def lib():
         vp, i32, f32, i64 = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
         L.oxb_residual_norm.argtypes = [vp, vp, f32, vp, vp, vp, vp, i32, i32, i32, f32, i32, vp]
         L.oxb_gemm_f32.argtypes = [vp, vp, vp, vp] + [i32] * 7 + [i64, i64, i64, i32, vp]
-        L.oxb_latent_prep.argtypes = ([vp, i32, i32, vp, vp, vp, i32, i32, i32, vp, f32] + [i32] * 6 + [vp, i32, vp, vp, i32, vp,
-                                      i32, i32, vp])
+        L.oxb_latent_prep.argtypes = ([vp, i32, i32, vp, vp, vp, i32, i32, i32, vp, f32] + [i32] * 6 + [vp, i32, vp, vp, i32, i32,
+                                      vp, i32, i32, vp])
         L.oxb_latent_attention_simt.argtypes = [vp, vp, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp]
         L.oxb_latent_mma_supported.argtypes = [i32] * 3
         L.oxb_latent_attention_mma.argtypes = [vp] * 7 + [i32] * 9 + [f32] + [i32] * 2 + [vp]
+        L.oxb_latent_gather.argtypes = [vp] * 4 + [i32] * 7 + [vp] * 3
+        L.oxb_latent_prefill_supported.argtypes = [i32] * 3
+        L.oxb_latent_prefill.argtypes = [vp] * 9 + [i32] * 12 + [f32, i32, vp]
         L.oxb_gemm_batched.argtypes = [vp, vp, vp, i64] + [i32] * 5 + [vp]
         _declared = True
     return L
@@ -97,6 +100,15 @@ class LatentOperands:
         v = torch.zeros(H, spec.v_dim, spec.latent_pad, dtype=dtype, device=dev)
         v[:, :, : spec.kv_rank] = m.w_uv
         self.heads, self.nope_ld, self.k, self.v = H, ld, k, v
+        # expanded form: one matrix that turns a latent into every head's key part and value
+        self.v_ld, self.v_off = (spec.v_dim + 7) // 8 * 8, H * ld
+        self.kv_ld = H * (ld + self.v_ld)
+        self.expand = None
+        if dtype == torch.bfloat16:
+            e = torch.zeros(self.kv_ld, spec.latent_pad, dtype=dtype, device=dev)
+            e[: self.v_off].view(H, ld, -1)[:, : spec.nope_dim, : spec.kv_rank] = m.w_uk
+            e[self.v_off :].view(H, self.v_ld, -1)[:, : spec.v_dim, : spec.kv_rank] = m.w_uv
+            self.expand = e
 
 
 def operands(m, spec, dtype: torch.dtype) -> LatentOperands:
@@ -125,7 +137,7 @@ def latent_prep(qkv, m, spec, rope, meta, kv, layer: int, eps: float, op: Latent
                                  meta.slot_mapping.data_ptr() if own else None, tab.data_ptr(), tab.shape[0], spec.rope_dim,
                                  0 if rope.pairing == "split_half" else 1, _p(m.kv_a_norm), eps, qkv.shape[0], op.heads,
                                  spec.nope_dim, spec.kv_rank, spec.latent_pad, spec.row_dim, _p(q_nope), op.nope_ld, _p(q_rows),
-                                 _p(q_full), 0 if q_full is None else q_full.shape[-1], kv.data[layer].data_ptr(), kv.page_size,
+                                 _p(q_full), 0 if q_full is None else q_full.shape[-1], (spec.nope_dim + 15) // 16 * 16, kv.data[layer].data_ptr(), kv.page_size,
                                  kv.num_blocks, _stream()), "oxb_latent_prep")
 
 
@@ -171,8 +183,93 @@ def latent_mixer(x, m, spec, rope, meta, kv, layer: int, eps: float) -> torch.Te
     return latent_core(linear(x, m.q), m, spec, rope, meta, kv, layer, eps, operands(m, spec, x.dtype))
 
 
+# Sequences that feed at least this many rows in a step take the expanded form; MAX_SPAN bounds the rows expanded at once.
+EXPAND_ROWS, MAX_SPAN = 64, 1 << 16
+
+
+def _spans(meta, window: int):
+    """(first visible position of every sequence, its first dense row, total rows) of a step for one window, kept for the
+    other layers of the step."""
+    key = ("latent_spans", window)
+    got = meta.extra.get(key)
+    if got is None:
+        lo = [max(0, ctx - n - window + 1) if window > 0 else 0 for n, ctx in meta.host_lens]
+        off = [0]
+        for l, (_, ctx) in zip(lo, meta.host_lens):
+            off.append(off[-1] + ctx - l)
+        t = torch.tensor(lo + off, dtype=torch.int32, device=meta.seq_lens.device)
+        got = meta.extra[key] = (t[: len(lo)], t[len(lo) :], off[-1])
+    return got
+
+
+def latent_expanded(qkv, m, spec, rope, meta, kv, layer: int, eps: float, op: LatentOperands, out: torch.Tensor) -> None:
+    """Long portions: keys and values of the visible rows are expanded per head, then flash attention."""
+    T, H, dt, dev = qkv.shape[0], op.heads, qkv.dtype, qkv.device
+    B = meta.seq_lens.shape[0]
+    full = (spec.nope_dim + 15) // 16 * 16 + (spec.row_dim - spec.latent_pad)
+    q = torch.empty(T, H, full, dtype=dt, device=dev)
+    latent_prep(qkv, m, spec, rope, meta, kv, layer, eps, op, q_full=q)
+    lo, off, rows = _spans(meta, spec.window)
+    lat = torch.empty(rows, spec.latent_pad, dtype=dt, device=dev)
+    rot = torch.empty(rows, spec.row_dim - spec.latent_pad, dtype=dt, device=dev)
+    _check(lib().oxb_latent_gather(kv.data[layer].data_ptr(), meta.block_tables.data_ptr(), lo.data_ptr(), off.data_ptr(), B, rows,
+                                   meta.block_tables.stride(0), spec.latent_pad, spec.row_dim, kv.page_size, kv.num_blocks,
+                                   lat.data_ptr(), rot.data_ptr(), _stream()), "oxb_latent_gather")
+    full_kv = opcuda.gemm_bf16(lat, op.expand)
+    _check(lib().oxb_latent_prefill(q.data_ptr(), full_kv.data_ptr(), rot.data_ptr(), out.data_ptr(), meta.query_start.data_ptr(),
+                                    meta.seq_lens.data_ptr(), lo.data_ptr(), off.data_ptr(), _p(m.sink), B, T, H, rows, spec.nope_dim,
+                                    spec.rope_dim, spec.v_dim, op.kv_ld, op.nope_ld, op.v_off, op.v_ld, spec.window, spec.scale,
+                                    max(n for n, _ in meta.host_lens), _stream()), "oxb_latent_prefill")
+
+
+def _runs(lens):
+    """Maximal runs [(first, end, long)] of neighbouring sequences that are all long or all short portions."""
+    runs = []
+    for b, (n, _) in enumerate(lens):
+        big = n >= EXPAND_ROWS
+        if runs and runs[-1][2] == big:
+            runs[-1][1] = b + 1
+        else:
+            runs.append([b, b + 1, big])
+    return runs
+
+
+def _sub_batch(meta, b0: int, b1: int, t0: int, t1: int):
+    """Sequences [b0, b1) (rows [t0, t1)) of a step as a step of their own, kept for the other layers."""
+    key = ("latent_sub", b0, b1)
+    sub = meta.extra.get(key)
+    if sub is None:
+        lens = meta.host_lens[b0:b1]
+        sub = meta.extra[key] = type(meta)(
+            None, meta.positions[t0:t1], meta.slot_mapping[t0:t1], (meta.query_start[b0 : b1 + 1] - t0).contiguous(),
+            meta.seq_lens[b0:b1], meta.block_tables[b0:b1], None, max(n for n, _ in lens), max(c for _, c in lens), b1 - b0,
+            host_lens=lens)
+    return sub
+
+
 def latent_core(qkv, m, spec, rope, meta, kv, layer: int, eps: float, op: LatentOperands) -> torch.Tensor:
     """From the layer's projections to its heads' outputs [T, heads * v_dim]."""
+    T, H, dt, dev = qkv.shape[0], op.heads, qkv.dtype, qkv.device
+    out = torch.empty(T, H * spec.v_dim, dtype=dt, device=dev)
+    if (dt == torch.bfloat16 and meta.host_lens and any(n >= EXPAND_ROWS for n, _ in meta.host_lens)
+            and lib().oxb_latent_prefill_supported(spec.nope_dim, spec.rope_dim, spec.v_dim)
+            and _spans(meta, spec.window)[2] <= MAX_SPAN):
+        starts = [0]
+        for n, _ in meta.host_lens:
+            starts.append(starts[-1] + n)
+        runs = _runs(meta.host_lens)
+        for b0, b1, big in runs:
+            t0, t1 = starts[b0], starts[b1]
+            sub = meta if len(runs) == 1 else _sub_batch(meta, b0, b1, t0, t1)
+            (latent_expanded if big else latent_absorbed)(qkv[t0:t1], m, spec, rope, sub, kv, layer, eps, op, out[t0:t1])
+    else:
+        latent_absorbed(qkv, m, spec, rope, meta, kv, layer, eps, op, out)
+    return out
+
+
+def latent_absorbed(qkv, m, spec, rope, meta, kv, layer: int, eps: float, op: LatentOperands, out: torch.Tensor) -> None:
+    """Decode rows and short portions: attention over the cached rows themselves, W_uk and W_uv applied to the queries and
+    to the attended latents."""
     T, H, dt, dev = qkv.shape[0], op.heads, qkv.dtype, qkv.device
     q_nope = torch.empty(H, T, op.nope_ld, dtype=dt, device=dev)
     q = torch.empty(T, H, spec.row_dim, dtype=dt, device=dev)
@@ -181,6 +278,4 @@ def latent_core(qkv, m, spec, rope, meta, kv, layer: int, eps: float, op: Latent
     o = torch.empty(H, T, spec.latent_pad, dtype=dt, device=dev)
     if dt != torch.bfloat16 or not attention_mma(q, kv, layer, meta, spec, m.sink, o):
         attention_simt(q, kv, layer, meta, spec, m.sink, o)
-    out = torch.empty(T, H * spec.v_dim, dtype=dt, device=dev)
     batched(o, op.v, out, spec.v_dim, H * spec.v_dim)
-    return out

@@ -308,3 +308,64 @@ def test_heads_and_feed_forward_are_sharded_over_ranks(tmp_path):
     whole, parts = branch(0, 1), [branch(r, 2) for r in range(2)]
     for i in range(2):
         assert rel(parts[0][i] + parts[1][i], whole[i]) < 1e-6
+
+
+# --------------------------------------------------------------------------- the whole mixer on the device, both forms
+MIXERS = [  # heads, nope, rot, v, rank, window, (rows, context) per sequence, page
+    (3, 24, 8, 20, 40, 19, [(100, 100)], 16), (4, 128, 64, 128, 512, 130, [(300, 700), (64, 64), (257, 300)], 16),
+    (2, 16, 16, 16, 48, 1, [(65, 65)], 8), (5, 40, 6, 36, 72, 64, [(1, 200), (1, 3), (128, 128), (70, 400), (2, 90)], 16),
+    (2, 64, 32, 96, 128, 0, [(200, 513)], 32), (1, 192, 16, 8, 32, 77, [(90, 150), (64, 65)], 64), (2, 8, 2, 1, 16, 500, [(64, 64)], 16)]
+
+
+@gpu
+@pytest.mark.parametrize("case", MIXERS, ids=str)
+def test_expanded_and_absorbed_forms_agree_with_the_32_bit_path(case, monkeypatch):
+    """Long portions attend over expanded keys and values, short ones over the cached rows; in one step beside each other.
+    Every row against the float32 path on the same (16-bit representable) inputs, with attention peaked on single keys."""
+    from oxidize_b200.models.layered import latent_weights
+    from oxidize_b200.models.transformer import RopeState
+    from oxidize_b200.ops import cuda_latent as CL
+
+    H, nope, rot, v, rank, window, lens, page = case
+    g = torch.Generator().manual_seed(H * 100 + v)
+    rnd = lambda *s: torch.randn(*s, generator=g).bfloat16().float()
+    spec = LatentAttentionSpec(H, nope, rot, v, rank, 3.0 / (nope + rot) ** 0.5, RotarySpec(rot, 1e4), window, True)
+    T, W = sum(n for n, _ in lens), H * (nope + rot) + rank + rot
+    qkv = rnd(T, W)
+    uk, uv = rnd(H * nope, rank) / rank ** 0.5, rnd(H * v, rank) / rank ** 0.5
+    norm, sink = torch.rand(rank, generator=g) + 0.5, torch.randn(H, generator=g)
+    nb = [(c + page - 1) // page for _, c in lens]
+    perm = torch.randperm(sum(nb), generator=g).int()
+    bt = torch.zeros(len(lens), max(nb), dtype=torch.int32)
+    o = 0
+    for b, k in enumerate(nb):
+        bt[b, :k] = perm[o : o + k]
+        o += k
+    past = rnd(sum(nb), 1, 1, page, spec.row_dim)
+    past[..., rank : spec.latent_pad] = 0
+    past[..., spec.latent_pad + rot :] = 0
+    pos = torch.cat([torch.arange(c - n, c) for n, c in lens]).int()
+    seq = torch.repeat_interleave(torch.arange(len(lens)), torch.tensor([n for n, _ in lens]))
+    slots = (bt[seq, (pos // page).long()] * page + pos % page).int()
+    qs = torch.tensor([0] + list(itertools.accumulate(n for n, _ in lens)), dtype=torch.int32)
+
+    def run(dtype, expand):
+        monkeypatch.setattr(CL, "EXPAND_ROWS", expand)
+        c = lambda t: t.cuda()
+        m = latent_weights(spec, torch.zeros(H * (nope + rot), 8), torch.zeros(rank + rot, 8), c(norm), c(uk.to(dtype)), c(uv.to(dtype)),
+                           c(sink))
+        kv = KVCache(KVCacheSpec(1, 1, spec.row_dim, page, "bf16" if dtype == torch.bfloat16 else "f32", planes=1), sum(nb), "cuda")
+        kv.data[0].copy_(past)
+        meta = BatchMeta(None, c(pos), c(slots), c(qs), c(torch.tensor([x for _, x in lens], dtype=torch.int32)), c(bt), None,
+                         max(n for n, _ in lens), max(x for _, x in lens), len(lens), host_lens=list(lens))
+        rope = RopeState(opref.rope_inv_freq(rot, 1e4, None, device="cuda", dtype=torch.float64), "split_half", 1.0, 0, 1, rot, 1024)
+        out = CL.latent_core(c(qkv).to(dtype), m, spec, rope, meta, kv, 0, 1e-5, CL.operands(m, spec, dtype))
+        return out.double().cpu(), kv.data[0].double().cpu()
+
+    want, rows = run(torch.float32, 1 << 30)
+    scale = float(want.pow(2).mean().sqrt())
+    for expand in (64, 1 << 30):  # the second: everything in absorbed form
+        got, r16 = run(torch.bfloat16, expand)
+        assert rel(r16, rows) < 4e-3
+        err = (got - want).pow(2).mean(-1).sqrt() / scale
+        assert float(err.max()) < 0.08 and float(err.mean()) < 0.02, (expand, float(err.max()), int(err.argmax()), float(err.mean()))
