@@ -1,32 +1,32 @@
 // Latent attention in absorbed form on the tensor cores: all heads of a query attend over the same cached rows.
 //
-// The work is turned around so that the cached rows are the wide operand: a tile of 64 rows (keys) is the M dimension of
+// The work is turned around so that the cached rows are the wide operand: a tile of 128 rows (keys) is the M dimension of
 // S^T[keys, rows] = K Q^T, and the latent values are the M dimension (128 at a time) of O^T[values, rows] = V^T P^T, where K
 // and V are ONE tile in shared memory: V^T is the same 128-byte-swizzled tile read as an MN-major operand.  N is a block of
 // 32 query rows ((token, head) pairs, token-major), so a decode step of 32 heads is one instruction shape and the kernel is a
-// stream of cache rows: every CTA owns (sequence, block of query rows, split of the keys), two warps bring the pages in with
-// TMA (column chunks of 64 values, in pairs of chunks so that a pair is one 128-value block of the second product), one warp
-// issues tcgen05.mma, four warps do the softmax on S^T read from tensor memory.  The ring holds two tiles and a bit: the
-// first product of the next tile and the copies of the one after run while this tile is in its softmax.
+// stream of cache rows: every CTA owns (sequence, block of query rows, split of the keys), TMA warps bring the pages in
+// (column chunks of 64 values, in pairs of chunks so that a pair is one 128-value block of the second product), one warp
+// issues tcgen05.mma, two warpgroups do the softmax on S^T read from tensor memory (16 rows each).  A slot of the ring is
+// given back as soon as the second product has read its block, so the copies of the next tile run under this one's end.
 //
-// Softmax: a thread holds one key of 16 rows (a half-warp split of tcgen05.ld: 64 rows of S^T sit in 16 lanes per warp).
-// Running maxima are moved by the first tile and then only when a score exceeds one by more than 2^8, which one vote
-// settles; row maxima are found with a transposing butterfly, and O^T is then rescaled in tensor memory.  The result is
-// exact either way.  The key splits of a row block are one thread-block cluster: each leaves its partial O^T in its own
-// shared memory (the ring is idle by then), and every CTA merges a share of the rows out of its peers' memory.
+// Softmax: a thread holds one key of 16 rows.  Running maxima are moved by the first tile and then only when a score exceeds
+// one by more than 2^8, which one vote settles; row maxima are found with a transposing butterfly, and O^T is then rescaled
+// in tensor memory.  The result is exact either way.  The key splits of a row block are one thread-block cluster: each leaves
+// its partial O^T in its own shared memory (the ring is idle by then), and every CTA merges a share of the rows out of its
+// peers' memory.
 #pragma once
 #include "common.cuh"
 
 namespace oxb {
 
-constexpr int LM_KEYS = 64;              // keys per tile
+constexpr int LM_KEYS = 128;             // keys per tile
 constexpr int LM_NR = 32;                // query rows per CTA
-constexpr int LM_CN = 16;                // of them per softmax thread
+constexpr int LM_CN = 16;                // of them per softmax warpgroup
 constexpr int LM_CHUNK = LM_KEYS * 128;  // bytes of one 64-value column chunk of a tile
 constexpr int LM_PAIR = 2 * LM_CHUNK;
-constexpr int LM_TMA_WARPS = 2;          // each brings every second page of a tile
-// warps: 0-3 softmax and output, then TMA, then MMA
-constexpr int LM_WARP_MMA = 4 + LM_TMA_WARPS, LM_WARPS = LM_WARP_MMA + 1, LM_THREADS = 32 * LM_WARPS;
+constexpr int LM_TMA_WARPS = 4;          // each brings every fourth page of a tile
+// warps: softmax and output, then TMA, then MMA
+constexpr int LM_SOFT_WARPS = 4 * (LM_NR / LM_CN), LM_WARP_MMA = LM_SOFT_WARPS + LM_TMA_WARPS, LM_WARPS = LM_WARP_MMA + 1, LM_THREADS = 32 * LM_WARPS;
 constexpr int LM_MAX_SLOTS = 16;
 constexpr int LM_DYN_SMEM = 224 * 1024;
 constexpr float LM_LAZY = 8.f;               // log2 of the factor by which scores may exceed the running maximum
@@ -40,7 +40,7 @@ struct LatentMmaArgs {
   int max_blocks, T, H, pad, width, page, num_blocks, window;
   int n_splits;             // CTAs of a cluster
   int pairs, rest, slots;   // 128-value blocks of the latent part, further 64-value chunks, ring slots (pairs)
-  int rest_slots;           // buffers of the further chunks
+  int rest_slots, p_bufs;   // buffers of the further chunks and of P
   float scale_log2;
 };
 
@@ -55,19 +55,11 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
       "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
       : "memory");
 }
-// 16 tensor-memory lanes x 32 columns spread over the warp: thread i < 16 gets columns 0-15 of lane i, thread 16 + i
-// columns 16-31 of the same lane
-__device__ __forceinline__ void tmem_ld16_halves(uint32_t taddr, uint32_t* r) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.16x32bx2.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16], 16;"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-      : "r"(taddr));
-}
-
-// Reduce v[j] (j < 16) over the 16 lanes of each half-warp; lane L returns the result of j = L % 16 of its half.
+// Reduce v[j] (j < 16) over the 32 lanes; lane L returns the result of j = L % 16.  v is used up.
 template <class Op>
 __device__ __forceinline__ float butterfly_rows(float* v, int lane, Op op) {
+#pragma unroll
+  for (int j = 0; j < 16; ++j) v[j] = op(v[j], __shfl_xor_sync(0xffffffffu, v[j], 16));
 #pragma unroll
   for (int o = 8; o > 0; o >>= 1) {
 #pragma unroll
@@ -128,16 +120,16 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
                             const LatentMmaArgs a) {
   constexpr int NR = LM_NR;
   extern __shared__ uint8_t lm_raw[];
-  // s_full / p_full / pv_done: one per parity of the tile (S^T and P are double-buffered)
+  // s_full / p_full / pv_done: one per parity of the tile (S^T is double-buffered)
   __shared__ uint64_t full[LM_MAX_SLOTS], empty[LM_MAX_SLOTS], rest_full[2], rest_empty[2], q_full, s_full[2], p_full[2], pv_done[2];
   __shared__ uint32_t tmem_slot;
   __shared__ volatile int abort_flag;
   __shared__ int2 row_keys[NR];                 // first and last key that a row sees
   __shared__ __align__(8) float2 part_ml[NR];   // maximum and sum of this split
   __shared__ long long row_out[NR];             // offset of a row's output, < 0: no such row
-  __shared__ float wmax[4][NR];                 // per-warp maxima of a tile, then per-warp sums
-  __shared__ __align__(16) float mrow[4][NR];   // running maxima (a copy per warp)
-  __shared__ __align__(16) float frow[4][NR];   // factors of a rescale / normalisation
+  __shared__ float wmax[LM_SOFT_WARPS][LM_CN];                // per-warp maxima of a tile, then per-warp sums
+  __shared__ __align__(16) float mrow[LM_SOFT_WARPS][LM_CN];  // running maxima (a copy per warp)
+  __shared__ __align__(16) float frow[LM_SOFT_WARPS][LM_CN];  // factors of a rescale / normalisation
   pdl_launch_dependents();
 
   // (broadcast from lane 0: the role branches and what is computed inside them are then known to be warp-uniform)
@@ -165,7 +157,7 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
   const int nch = (a.width + 63) / 64;
   uint8_t* s_rest = smem + a.slots * LM_PAIR;                     // [rest_slots][rest chunks]
   uint8_t* s_q = s_rest + a.rest_slots * a.rest * LM_CHUNK;       // [nch][NR][128 bytes]
-  uint8_t* s_p = s_q + nch * NR * 128;                            // [2][NR][128 bytes]: the tile's 64 keys
+  uint8_t* s_p = s_q + nch * NR * 128;                            // [p_bufs][2][NR][128 bytes]: 64 keys per row
   uint32_t tmem_cols = 64;
   while ((int)tmem_cols < NR * (2 + a.pairs)) tmem_cols <<= 1;
 
@@ -178,7 +170,7 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
       mbar_init(&rest_full[i], LM_TMA_WARPS);
       mbar_init(&rest_empty[i], 1);
       mbar_init(&s_full[i], 1);
-      mbar_init(&p_full[i], 128);
+      mbar_init(&p_full[i], 32 * LM_SOFT_WARPS);
       mbar_init(&pv_done[i], 1);
     }
     mbar_init(&q_full, 1);
@@ -201,9 +193,9 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
   const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_slot, 0);  // columns: S^T (two buffers of NR), then the blocks of O^T
   pdl_wait();  // queries and this step's cache rows come from the upstream kernels
 
-  if (warp >= 4 && warp < LM_WARP_MMA) {
+  if (warp >= LM_SOFT_WARPS && warp < LM_WARP_MMA) {
     // ---------------- TMA: warp-uniform loops, one elected lane issues
-    const int w = warp - 4;
+    const int w = warp - LM_SOFT_WARPS;
     const bool leader = elect_one();
     if (leader && w == 0) {
       tma_prefetch_desc(&tmK);
@@ -297,13 +289,13 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
       const bool ok = mbar_wait_bounded(&p_full[i & 1], (i >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
       if (!__all_sync(0xffffffffu, ok)) return false;
       tc_fence_after();
-      const uint32_t pd = umma_desc_lo(p_addr + (i & 1) * (NR * 128));
+      const uint32_t pd = umma_desc_lo(p_addr + (a.p_bufs == 2 ? i & 1 : 0) * (2 * NR * 128));
       for (int p = 0; p < a.pairs; ++p) {
         const uint32_t vd = umma_desc_lo(base + vslot * LM_PAIR, LM_CHUNK);
 #pragma unroll
-        for (int k = 0; k < LM_KEYS / 16; ++k)  // 16 keys: 2 KB of the value tile, 32 bytes of a P row
-          umma_bf16_if<UMMA_DESC_HI_SW128, UMMA_DESC_HI_SW128, idesc_o>(leader, tmem + NR * (2 + p), vd + k * (2048 >> 4), pd + 2 * k,
-                                                                      i > 0 || k > 0);
+        for (int k = 0; k < LM_KEYS / 16; ++k)  // 16 keys: 2 KB of the value tile, 32 bytes of a P row (64 keys per row)
+          umma_bf16_if<UMMA_DESC_HI_SW128, UMMA_DESC_HI_SW128, idesc_o>(
+              leader, tmem + NR * (2 + p), vd + k * (2048 >> 4), pd + (k >> 2) * (NR * 128 >> 4) + 2 * (k & 3), i > 0 || k > 0);
         umma_commit_if(leader, &empty[vslot]);
         if (++vslot == a.slots) vslot = 0;
       }
@@ -322,14 +314,15 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
     }
     __syncwarp();
   } else {
-    // ---------------- softmax: thread = key of the tile x 16 query rows
-    const uint32_t lanes = (uint32_t)(warp * 32) << 16;
-    const int key_in = warp * 16 + (lane & 15), n0 = lane & 16;  // key of the tile, first of this thread's rows
-    auto group_sync = [&]() { asm volatile("bar.sync 1, 128;" ::: "memory"); };
-    // widest key range that every row of the block sees: tiles inside it need no mask
-    const int all_lo = row_keys[NR - 1].x, all_hi = row_keys[0].y;
-    const float sink = (a.sink != nullptr && split == 0) ? a.sink[(row_base + lane) % a.H] * 1.4426950408889634f : -INFINITY;
-    float m = sink;  // running maximum of row `lane` (log2 units), the same in every warp
+    // ---------------- softmax: thread = key of the tile (its tensor-memory lane); warpgroup g has query rows n0 .. n0 + 15
+    const int g = warp >> 2, n0 = g * LM_CN, w0 = g * 4;
+    const uint32_t lanes = ((uint32_t)((warp & 3) * 32) << 16) + n0;
+    const int key_in = threadIdx.x & 127, my = lane & 15;  // my: the row whose maximum this lane keeps
+    auto group_sync = [&]() { asm volatile("bar.sync %0, 128;" ::"r"(1 + g) : "memory"); };
+    // widest key range that every row of the group sees: tiles inside it need no mask
+    const int all_lo = row_keys[n0 + LM_CN - 1].x, all_hi = row_keys[n0].y;
+    const float sink = (a.sink != nullptr && split == 0) ? a.sink[(row_base + n0 + my) % a.H] * 1.4426950408889634f : -INFINITY;
+    float m = sink;  // running maximum of row n0 + my (log2 units), the same in every warp of the group
     float l[LM_CN];
 #pragma unroll
     for (int j = 0; j < LM_CN; ++j) l[j] = 0.f;
@@ -340,7 +333,7 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
       __syncwarp();
       tc_fence_after();
       float s[LM_CN];
-      tmem_ld16_halves(tmem + lanes + NR * (i & 1), reinterpret_cast<uint32_t*>(s));
+      tmem_ld16(tmem + lanes + NR * (i & 1), reinterpret_cast<uint32_t*>(s));
       tmem_ld_wait();
       const int key0 = (page_lo + (t_begin + i) * ppt) * a.page;
 #pragma unroll
@@ -353,12 +346,12 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
           if (key < rk.x || key > rk.y) s[j] = -INFINITY;
         }
       }
-      // running maxima of this thread's rows; usually no score exceeds them by the lazy margin, which one vote settles
+      // running maxima of the group's rows; usually no score exceeds them by the lazy margin, which one vote settles
       float mm[LM_CN];
       auto load_max = [&]() {
 #pragma unroll
         for (int j = 0; j < LM_CN; j += 4) {
-          const float4 v = *reinterpret_cast<const float4*>(&mrow[warp][n0 + j]);
+          const float4 v = *reinterpret_cast<const float4*>(&mrow[warp][j]);
           mm[j] = v.x;
           mm[j + 1] = v.y;
           mm[j + 2] = v.z;
@@ -373,53 +366,55 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
       }
       int any_over;
       asm volatile(
-          "{\n\t.reg .pred p, q;\n\tsetp.ne.s32 p, %1, 0;\n\tbarrier.cta.red.or.pred q, 1, 128, p;\n\tselp.s32 %0, 1, 0, q;\n\t}"
+          "{\n\t.reg .pred p, q;\n\tsetp.ne.s32 p, %1, 0;\n\tbarrier.cta.red.or.pred q, %2, 128, p;\n\tselp.s32 %0, 1, 0, q;\n\t}"
           : "=r"(any_over)
-          : "r"((int)over)
+          : "r"((int)over), "r"(1 + g)
           : "memory");
       bool any_move = false;
       if (any_over) {
         float v[LM_CN];
 #pragma unroll
         for (int j = 0; j < LM_CN; ++j) v[j] = s[j];
-        wmax[warp][lane] = butterfly_rows(v, lane, [](float x, float y) { return fmaxf(x, y); });
+        const float wm = butterfly_rows(v, lane, [](float x, float y) { return fmaxf(x, y); });
+        if (lane < LM_CN) wmax[warp][lane] = wm;
         group_sync();
-        const float tm = fmaxf(fmaxf(wmax[0][lane], wmax[1][lane]), fmaxf(wmax[2][lane], wmax[3][lane]));
+        const float tm = fmaxf(fmaxf(wmax[w0][my], wmax[w0 + 1][my]), fmaxf(wmax[w0 + 2][my], wmax[w0 + 3][my]));
         // the first tile sets the maximum, later ones move it past the margin only
         const bool move = tm > m + (i == 0 ? 0.f : LM_LAZY) || (m == -INFINITY && tm > -INFINITY);
         const float m_new = move ? tm : m;
-        frow[warp][lane] = move ? exp2f(m - m_new) : 1.f;  // 0 when nothing was accumulated
+        if (lane < LM_CN) {
+          frow[warp][lane] = move ? exp2f(m - m_new) : 1.f;  // 0 when nothing was accumulated
+          mrow[warp][lane] = m_new == -INFINITY ? 0.f : m_new;
+        }
         m = m_new;
-        mrow[warp][lane] = m == -INFINITY ? 0.f : m;
         any_move = __any_sync(0xffffffffu, move) && i > 0;
         __syncwarp();
         load_max();
       }
 #pragma unroll
       for (int j = 0; j < LM_CN; ++j) s[j] = exp2f(s[j] - mm[j]);
-      if (any_move) {  // every earlier tile's second product is complete: rescale the sums and O^T
-        mbar_wait_bounded(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
-        __syncwarp();
+      // O^T is rescaled once every earlier second product is complete; a P buffer is free once its last reader is
+      const int done = (any_move || a.p_bufs == 1) ? i - 1 : i - 2;
+      if (done >= 0) mbar_wait_bounded(&pv_done[done & 1], (done >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+      __syncwarp();
+      if (any_move) {
         tc_fence_after();
 #pragma unroll
-        for (int j = 0; j < LM_CN; ++j) l[j] *= frow[warp][n0 + j];
-        for (int p = 0; p < 2 * a.pairs; ++p) {
+        for (int j = 0; j < LM_CN; ++j) l[j] *= frow[warp][j];
+        for (int p = 0; p < a.pairs; ++p) {
           uint32_t r[16];
-          const uint32_t addr = tmem + lanes + NR * 2 + 16 * p;
+          const uint32_t addr = tmem + lanes + NR * (2 + p);
           tmem_ld16(addr, r);
           tmem_ld_wait();
 #pragma unroll
-          for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * frow[warp][(p & 1) * 16 + j]);
+          for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * frow[warp][j]);
           tmem_st16(addr, r);
         }
         tmem_st_wait();
-      } else if (i > 1) {  // this P buffer was read by the second product two tiles ago
-        mbar_wait_bounded(&pv_done[i & 1], ((i >> 1) - 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
-        __syncwarp();
       }
       // P^T as the second product's B operand: row = 128 bytes of 64 keys, 16-byte pieces swizzled by the row
-      uint8_t* pb = s_p + (i & 1) * (NR * 128) + n0 * 128;
-      const int piece = key_in >> 3, in = (key_in & 7) * 2;
+      uint8_t* pb = s_p + (a.p_bufs == 2 ? i & 1 : 0) * (2 * NR * 128) + (key_in >> 6) * (NR * 128) + n0 * 128;
+      const int piece = (key_in & 63) >> 3, in = (key_in & 7) * 2;
 #pragma unroll
       for (int j = 0; j < LM_CN; ++j) {
         l[j] += s[j];
@@ -435,41 +430,41 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
     __syncwarp();
     tc_fence_after();
     group_sync();
-    wmax[warp][lane] = ws;
+    if (lane < LM_CN) wmax[warp][lane] = ws;
     group_sync();
-    float L = (wmax[0][lane] + wmax[1][lane]) + (wmax[2][lane] + wmax[3][lane]);
+    float L = (wmax[w0][my] + wmax[w0 + 1][my]) + (wmax[w0 + 2][my] + wmax[w0 + 3][my]);
     if (sink > -INFINITY) L += exp2f(sink - m);  // the sink's share of the denominator, once
     if (a.n_splits > 1) {
       // O^T of this split into shared memory as [row][pad], next to its maxima and sums
-      if (warp == 0) part_ml[lane] = make_float2(m, L);
+      if (warp == w0 && lane < LM_CN) part_ml[n0 + lane] = make_float2(m, L);
       float* part = reinterpret_cast<float*>(smem);
-      for (int p = 0; n > 0 && p < 2 * a.pairs; ++p) {
+      asm volatile("bar.sync 3, 256;" ::: "memory");  // both groups are past their last product: the ring is idle
+      for (int p = 0; n > 0 && p < a.pairs; ++p) {
         uint32_t r[16];
-        tmem_ld16(tmem + lanes + NR * 2 + 16 * p, r);
+        tmem_ld16(tmem + lanes + NR * (2 + p), r);
         tmem_ld_wait();
-        const int d = (p >> 1) * 128 + threadIdx.x;
+        const int d = p * 128 + key_in;
         if (d < a.pad) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) part[((p & 1) * 16 + j) * a.pad + d] = __uint_as_float(r[j]);
+          for (int j = 0; j < 16; ++j) part[(n0 + j) * a.pad + d] = __uint_as_float(r[j]);
         }
       }
     } else {
-      frow[warp][lane] = L > 0.f ? 1.f / L : 0.f;
+      if (lane < LM_CN) frow[warp][lane] = L > 0.f ? 1.f / L : 0.f;
       __syncwarp();
       // neighbouring lanes (values d, d + 1) swap one row of each pair of rows, so that a lane stores two values of one row
       const bool odd = lane & 1;
-      for (int p = 0; p < 2 * a.pairs; ++p) {
+      for (int p = 0; p < a.pairs; ++p) {
         uint32_t r[16];
-        tmem_ld16(tmem + lanes + NR * 2 + 16 * p, r);
+        tmem_ld16(tmem + lanes + NR * (2 + p), r);
         tmem_ld_wait();
-        const int d = (p >> 1) * 128 + (threadIdx.x & ~1), c0 = (p & 1) * 16;
+        const int d = p * 128 + (key_in & ~1);
 #pragma unroll
         for (int j = 0; j < 16; j += 2) {
-          const float lo_v = __uint_as_float(r[j]) * frow[warp][c0 + j], hi_v = __uint_as_float(r[j + 1]) * frow[warp][c0 + j + 1];
+          const float lo_v = __uint_as_float(r[j]) * frow[warp][j], hi_v = __uint_as_float(r[j + 1]) * frow[warp][j + 1];
           const float got = __shfl_xor_sync(0xffffffffu, odd ? lo_v : hi_v, 1);
-          const int row = c0 + j + (odd ? 1 : 0);
           const float v0 = odd ? got : lo_v, v1 = odd ? hi_v : got;
-          const long long o = row_out[row];
+          const long long o = row_out[n0 + j + (odd ? 1 : 0)];
           if (o >= 0 && d < a.pad) *reinterpret_cast<uint32_t*>(a.out + o + d) = pack_bf16x2(v0, v1);
         }
       }
@@ -491,25 +486,24 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
   if (warp == LM_WARP_MMA) tmem_dealloc(tmem, tmem_cols);
 }
 struct LatentMmaPlan {
-  int ok, pairs, rest, slots, rest_slots, smem;
+  int ok, pairs, rest, slots, rest_slots, p_bufs, smem;
 };
 
-// Shared-memory plan for rows of `width` values of which the first `pad` are the latent part.
+// Shared-memory plan for rows of `width` values of which the first `pad` are the latent part: the ring gets what queries, P
+// and the chunks past the latent blocks leave; these are double-buffered where the ring then holds two tiles.
 inline LatentMmaPlan latent_mma_plan(int pad, int width, int page) {
-  LatentMmaPlan p{0, (pad + 127) / 128, 0, 0, 0, 0};
-  const int nch = (width + 63) / 64;
+  LatentMmaPlan p{0, (pad + 127) / 128, 0, 0, 2, 2, 0};
+  const int nch = (width + 63) / 64, pbuf = 2 * LM_NR * 128;
   p.rest = nch > 2 * p.pairs ? nch - 2 * p.pairs : 0;
-  const int budget = LM_DYN_SMEM;  // the static variables of the kernel share the 227 KB
-  const int fixed = nch * LM_NR * 128 + 2 * LM_NR * 128 + 1024;
-  p.rest_slots = 2;
-  p.slots = (budget - fixed - 2 * p.rest * LM_CHUNK) / LM_PAIR;
-  if (p.slots < 2 * p.pairs && p.rest > 0) {
-    p.rest_slots = 1;
-    p.slots = (budget - fixed - p.rest * LM_CHUNK) / LM_PAIR;
+  const int fixed = nch * LM_NR * 128 + 1024;
+  p.slots = (LM_DYN_SMEM - fixed - 2 * p.rest * LM_CHUNK - 2 * pbuf) / LM_PAIR;
+  if (p.slots < 2 * p.pairs) {
+    p.rest_slots = p.p_bufs = 1;
+    p.slots = (LM_DYN_SMEM - fixed - p.rest * LM_CHUNK - pbuf) / LM_PAIR;
   }
   if (p.slots > 4 * p.pairs) p.slots = 4 * p.pairs;
   if (p.slots > LM_MAX_SLOTS) p.slots = LM_MAX_SLOTS;
-  p.smem = p.slots * LM_PAIR + p.rest_slots * p.rest * LM_CHUNK + fixed;
+  p.smem = p.slots * LM_PAIR + p.rest_slots * p.rest * LM_CHUNK + p.p_bufs * pbuf + fixed;
   p.ok = p.slots >= p.pairs && page % 8 == 0 && LM_KEYS % page == 0 && width % 16 == 0 && LM_NR * (2 + p.pairs) <= 512;
   return p;
 }

@@ -108,6 +108,7 @@ OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache
   a.rest = pl.rest;
   a.slots = pl.slots;
   a.rest_slots = pl.rest_slots;
+  a.p_bufs = pl.p_bufs;
   a.scale_log2 = scale * 1.4426950408889634f;
   const dim3 grid((max_query_len * H + LM_NR - 1) / LM_NR * a.n_splits, B);
   const cudaError_t le =
