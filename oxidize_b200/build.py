@@ -30,9 +30,16 @@ def _sources(exts):
     return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(exts))
 
 
-def build_kernels(force: bool = False, verbose: bool = False) -> str:
-    out = os.path.join(CSRC, "liboxb.so")
-    srcs = _sources((".cu", ".cuh", ".h"))
+PACKED_UNITS = ("oxb_mmq_", "oxb_gemv")  # packed-weight kernels: most of the compile time
+NO_PACKED = "oxb_no_packed.cu"
+
+
+def build_kernels(force: bool = False, verbose: bool = False, core: bool = False) -> str:
+    """The kernel library; ``core`` leaves the packed-weight kernels out (``liboxb_core.so``: all that a model with bf16 or
+    f32 weights runs, built in a fraction of the time)."""
+    out = os.path.join(CSRC, "liboxb_core.so" if core else "liboxb.so")
+    srcs = [s for s in _sources((".cu", ".cuh", ".h"))
+            if (not os.path.basename(s).startswith(PACKED_UNITS) if core else os.path.basename(s) != NO_PACKED) or not s.endswith(".cu")]
     if not force and _newer(out, srcs):
         return out
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"

@@ -92,7 +92,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   __shared__ uint32_t tmem_slot;
   __shared__ volatile int abort_flag;
   pdl_launch_dependents();
-  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0);
   const int h = blockIdx.y, b = blockIdx.z;
   const int q0 = a.query_start[b], qlen = a.query_start[b + 1] - q0;
   const int m0 = blockIdx.x * 2 * LP_M;  // first token (of the sequence's rows) of this CTA

@@ -379,7 +379,13 @@ OXB_API int oxb_gemm_batched(const void* X, const void* W, void* Y, long long y_
                              cudaStream_t stream) {
   if (T <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
   if (K % 8 != 0) return (int)cudaErrorInvalidValue;
+  // split K inside clusters where the groups' tiles alone leave SMs idle (at least two k-blocks per CTA)
   GemmPlan p = gemm_plan(T, N, K, 1, sm_count(), 0, 0, false, groups);
+  const int kb = (K + GEMM_BK - 1) / GEMM_BK;
+  int splits = sm_count() / (p.n_tiles * p.t_tiles * groups);
+  if (splits > 4) splits = 4;
+  if (splits > kb / 2) splits = kb / 2;
+  if (splits > 1 && p.tn <= 64 && g_oxb_cluster_splitk) p = gemm_plan(T, N, K, splits, sm_count(), 1, 0, false, groups);
   CUtensorMap tmW, tmX;
   int e = oxb_make_tmap_2d(&tmX, X, (uint64_t)groups * T, K, (uint64_t)K * 2, p.tn, GEMM_BK, 2);
   if (e) return e;

@@ -16,7 +16,7 @@ from typing import Callable, Dict, Iterable, List, Optional, Sequence as Seq, Un
 
 import torch
 
-from ..formats.layered import Checkpoint, open_checkpoint
+from ..formats.layered import Checkpoint, LayeredCheckpoint, open_checkpoint
 from ..models.config import ModelConfig
 from ..models.registry import act_dtype_for, config_from_checkpoint, load_checkpoint_weights
 from ..models.transformer import Transformer
@@ -148,6 +148,10 @@ class LLM:
                 raise ValueError(f"experts_per_token must be between 1 and the model's {cfg.n_experts} experts")
             cfg.n_experts_used = experts_per_token
         device = torch.device(device if device is not None else ("cuda" if torch.cuda.is_available() else "cpu"))
+        if device.type == "cuda" and isinstance(g, LayeredCheckpoint):
+            from ..ops import cuda as _opcuda
+
+            _opcuda.core_will_do()  # its weights are bf16 or f32
         act = act_dtype_for(cfg, device, config.compute_dtype)
         ep_size = config.ep_size or config.tp_size
         if ep_size == config.tp_size and ep_rank == 0:

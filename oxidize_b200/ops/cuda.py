@@ -16,6 +16,7 @@ import torch
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _CSRC = os.path.join(os.path.dirname(_HERE), "csrc")
 LIB_PATH = os.path.join(_CSRC, "liboxb.so")
+_core_will_do = False
 
 _lib = None
 _lock = threading.Lock()
@@ -32,16 +33,23 @@ class OxbError(RuntimeError):
     pass
 
 
+def core_will_do() -> None:
+    """The model about to run needs no packed-weight kernels: if the library has to be built first, its core is enough."""
+    global _core_will_do
+    _core_will_do = True
+
+
 def lib():
     global _lib
     if _lib is None:
         with _lock:
             if _lib is None:
-                if not os.path.exists(LIB_PATH):
+                path = LIB_PATH
+                if not os.path.exists(path):
                     from ..build import build_kernels
 
-                    build_kernels()
-                _lib = ctypes.CDLL(LIB_PATH)
+                    path = build_kernels(core=_core_will_do)
+                _lib = ctypes.CDLL(path)
                 _declare(_lib)
     return _lib
 
