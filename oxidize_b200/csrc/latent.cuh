@@ -36,9 +36,10 @@ struct LatentPrepArgs {
   int full_ld, full_rot;
   void* cache;          // layer base [blocks, page, width]
   int page, num_blocks;
+  int vec8;             // sizes and strides allow pieces of eight values (bf16)
 };
 
-constexpr int LAT_PREP_HEADS = 4;  // query heads per CTA
+constexpr int LAT_PREP_HEADS = 8;  // query heads per CTA
 
 // element i of the rotation of v[0..rot)
 template <typename T>
@@ -54,6 +55,57 @@ __device__ __forceinline__ float lat_rotated(const T* v, int i, const float* cs,
   const float c = cs[p], s = cs[half + p];
   const float x = lat_f32(v[i]), o = lat_f32(v[i ^ 1]);
   return (i & 1) ? x * c + o * s : x * c - o * s;
+}
+
+// Eight neighbouring values of the rotation at once (split-half pairing, rot a multiple of 16, 16-byte aligned).
+__device__ __forceinline__ uint4 lat_rotated8(const __nv_bfloat16* v, int i, const float* cs, int rot) {
+  const int half = rot >> 1;
+  const bool lo = i < half;
+  const int p = lo ? i : i - half;
+  const uint4 xv = *reinterpret_cast<const uint4*>(v + i), ov = *reinterpret_cast<const uint4*>(v + (lo ? i + half : p));
+  const uint32_t xs[4] = {xv.x, xv.y, xv.z, xv.w}, os[4] = {ov.x, ov.y, ov.z, ov.w};
+  float c[8], sn[8];
+#pragma unroll
+  for (int j = 0; j < 8; j += 4) {
+    *reinterpret_cast<float4*>(c + j) = *reinterpret_cast<const float4*>(cs + p + j);
+    *reinterpret_cast<float4*>(sn + j) = *reinterpret_cast<const float4*>(cs + half + p + j);
+  }
+  uint32_t r[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float2 x = unpack_bf16x2(xs[j]), o = unpack_bf16x2(os[j]);
+    const float sgn = lo ? -1.f : 1.f;
+    r[j] = pack_bf16x2(x.x * c[2 * j] + sgn * o.x * sn[2 * j], x.y * c[2 * j + 1] + sgn * o.y * sn[2 * j + 1]);
+  }
+  return make_uint4(r[0], r[1], r[2], r[3]);
+}
+
+// The query heads of one CTA in pieces of eight values; every size and stride involved is a multiple of eight.
+__device__ __forceinline__ void latent_prep_queries8(const LatentPrepArgs& a, const __nv_bfloat16* row, const float* cs, int t, int h0,
+                                                     int h1) {
+  const int qk = a.nope + a.rot;
+  const bool full = a.q_full != nullptr;
+  const int n1 = (full ? a.full_ld : a.nope_ld) / 8, n2 = full ? 0 : (a.width - a.rank) / 8, per = n1 + n2;
+  for (int i = threadIdx.x; i < (h1 - h0) * per; i += blockDim.x) {
+    const int h = h0 + i / per, c = i % per;
+    const __nv_bfloat16* q = row + (size_t)h * qk;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    uint4* dst;
+    int e;  // value of the rotated part, < 0 or >= rot: none
+    if (c < n1) {
+      const int d = 8 * c;
+      dst = full ? reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(a.q_full) + ((size_t)t * a.H + h) * a.full_ld + d)
+                 : reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(a.q_nope) + ((size_t)h * a.T + t) * a.nope_ld + d);
+      if (d < a.nope) v = *reinterpret_cast<const uint4*>(q + d);
+      e = full ? d - a.full_rot : -1;
+    } else {
+      const int d = a.rank + 8 * (c - n1);
+      dst = reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(a.q_rows) + ((size_t)t * a.H + h) * a.width + d);
+      e = d - a.pad;
+    }
+    if (e >= 0 && e < a.rot) v = lat_rotated8(q + a.nope, e, cs, a.rot);
+    *dst = v;
+  }
 }
 
 // grid (T, 1 + ceil(H / LAT_PREP_HEADS)): CTA (t, 0) makes token t's cache row, the others its query heads
@@ -94,6 +146,12 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepArgs a
     return;
   }
   const int h0 = (blockIdx.y - 1) * LAT_PREP_HEADS, h1 = min(a.H, h0 + LAT_PREP_HEADS);
+  if constexpr (sizeof(T) == 2) {
+    if (a.vec8) {
+      latent_prep_queries8(a, row, cs, t, h0, h1);
+      return;
+    }
+  }
   for (int h = h0; h < h1; ++h) {
     const T* q = row + (size_t)h * qk;
     if (a.q_full != nullptr) {

@@ -32,7 +32,9 @@ OXB_API int oxb_latent_prep(const void* qkv, int ld, int dtype, const int* posit
   if (T <= 0) return 0;
   if (rot <= 0 || rot % 2 != 0 || rank > pad || pad + rot > width || page <= 0) return (int)cudaErrorInvalidValue;
   const LatentPrepArgs a{qkv, ld, positions, slots, cos_sin, max_pos, rot, pairing, norm_w, eps, T, H, nope, rank, pad, width,
-                         q_nope, nope_ld, q_rows, q_full, full_ld, full_rot, cache, page, num_blocks};
+                         q_nope, nope_ld, q_rows, q_full, full_ld, full_rot, cache, page, num_blocks,
+                         (ld | nope | rank | pad | width | nope_ld | full_ld | full_rot) % 8 == 0 && rot % 16 == 0 && pairing == 0 &&
+                             (reinterpret_cast<uintptr_t>(qkv) & 15) == 0};
   const dim3 grid(T, 1 + (H + LAT_PREP_HEADS - 1) / LAT_PREP_HEADS);
   if (dtype == 0) oxb_launch(latent_prep_kernel<float>, grid, dim3(128), 0, stream, a);
   else oxb_launch(latent_prep_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, a);

@@ -118,8 +118,9 @@ __global__ void __launch_bounds__(256) residual_norm_any_kernel(const ResidualNo
 template <typename A>
 int residual_norm_launch(const ResidualNormArgs& a, int T, cudaStream_t stream) {
   if (a.H % 4 == 0 && a.H <= 16384) {
-    // few threads with several groups each: short reductions, and several rows resident per SM
-    const int H4 = a.H / 4, ch = H4 <= 256 ? 1 : (H4 <= 512 ? 2 : 4);
+    // many rows: few threads with several groups each, so that several rows are resident per SM; few rows: the row is spread
+    // over as many threads as there are groups
+    const int H4 = a.H / 4, lim = T >= 512 ? 256 : 1024, ch = H4 <= lim ? 1 : (H4 <= 2 * lim ? 2 : 4);
     const int threads = ((H4 + ch - 1) / ch + 31) / 32 * 32;
     if (ch == 1) oxb_launch(residual_norm_kernel<A, 1>, dim3(T), dim3(threads), 0, stream, a);
     else if (ch == 2) oxb_launch(residual_norm_kernel<A, 2>, dim3(T), dim3(threads), 0, stream, a);

@@ -132,6 +132,7 @@ class ModelRunner:
         self._out_which = 0
         self.keep_logits = False
         self._bt_owners = [[None] * max_seqs for _ in self.buf.hosts]
+        self._scored: list = [None] * len(self.buf.hosts)  # events behind the staging copies of scored steps
 
     # ------------------------------------------------------------------ batch building
     def build(self, scheduled: Sequence[ScheduledSeq], pad_to: Optional[int] = None):
@@ -332,9 +333,14 @@ class ModelRunner:
         """One step that samples nothing: logits [n, vocab] of the rows its entries want (``ScheduledSeq.want``), in order."""
         for src, dst in out.cow_copies:
             self.kv.copy_block(src, dst)
-        self.buf.flip()
+        which = self.buf.flip()
+        if self._scored[which] is not None:  # nobody waits for a scored step's result: its staging copy may still be pending
+            self._scored[which].synchronize()
         T, B, nl, max_q, max_len, _ = self.build(out.scheduled)
         self.buf.upload()
+        if self.device.type == "cuda":
+            self._scored[which] = torch.cuda.Event()
+            self._scored[which].record()
         meta = self._meta(T, B, nl, max_q, max_len)
         meta.host_lens = [(ss.num_tokens, ss.start + ss.num_tokens) for ss in out.scheduled]
         return self.model.forward(meta, self.kv)
