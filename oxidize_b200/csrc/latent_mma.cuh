@@ -73,7 +73,7 @@ __device__ __forceinline__ float butterfly_rows(float* v, int lane, Op op) {
 }
 
 // Merge of a cluster's key splits with the log-sum-exp weights exp2(m_s - M) / sum: this CTA takes rows rank, rank + n, ...
-constexpr int LM_MAX_SPLITS = 8;
+constexpr int LM_MAX_SPLITS = 16;  // clusters of more than 8 CTAs where the device takes them
 __device__ __forceinline__ void merge_splits(const LatentMmaArgs& a, const uint8_t* part, const float2* part_ml,
                                              const long long* row_out, int rank, int tiles, int per) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;

@@ -67,8 +67,39 @@ OXB_API int oxb_latent_attention_simt(const void* q, void* out, const void* cach
 // 1 when latent_attention_mma_kernel covers rows of this shape (else: the plain kernel)
 OXB_API int oxb_latent_mma_supported(int pad, int width, int page) { return latent_mma_plan(pad, width, page).ok; }
 
+// Shared memory and cluster sizes of latent_attention_mma_kernel, set up once per device; returns the largest cluster it
+// can be launched with (its key splits), or 0 on an error.
+static int latent_mma_max_splits() {
+  static int cached[64] = {0};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return 0;
+  if (cached[dev]) return cached[dev];
+  if (cudaFuncSetAttribute(latent_attention_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LM_DYN_SMEM) != cudaSuccess)
+    return 0;
+  cached[dev] = 8;
+  if (cudaFuncSetAttribute(latent_attention_mma_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(LM_MAX_SPLITS, 1, 1);
+    cfg.blockDim = dim3(LM_THREADS);
+    cfg.dynamicSmemBytes = LM_DYN_SMEM;
+    cudaLaunchAttribute at;
+    at.id = cudaLaunchAttributeClusterDimension;
+    at.val.clusterDim.x = LM_MAX_SPLITS;
+    at.val.clusterDim.y = 1;
+    at.val.clusterDim.z = 1;
+    cfg.attrs = &at;
+    cfg.numAttrs = 1;
+    int n = 0;
+    if (cudaOccupancyMaxActiveClusters(&n, latent_attention_mma_kernel, &cfg) == cudaSuccess && n > 0) cached[dev] = LM_MAX_SPLITS;
+  }
+  cudaGetLastError();
+  return cached[dev];
+}
+OXB_API int oxb_latent_max_splits() { return latent_mma_max_splits(); }
+
 // Latent attention, absorbed form, bf16: q [T, H, width] and the cache rows [num_blocks * page, width]; the B sequences
-// have at most max_query_len rows each.  n_splits (at most 8) CTAs share the keys of a block of 32 rows.
+// have at most max_query_len rows each.  n_splits CTAs (at most oxb_latent_max_splits()) share the keys of a block of 32 rows.
 OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache, const int* block_tables, const int* seq_lens,
                                      const int* query_start, const float* sink, int B, int max_blocks, int T, int H, int pad,
                                      int width, int page, int num_blocks, int window, float scale, int max_query_len,
@@ -76,16 +107,9 @@ OXB_API int oxb_latent_attention_mma(const void* q, void* out, const void* cache
   if (T <= 0 || B <= 0 || max_query_len <= 0) return 0;
   const LatentMmaPlan pl = latent_mma_plan(pad, width, page);
   if (!pl.ok || B > 65535) return (int)cudaErrorInvalidValue;
-  if (n_splits > LM_MAX_SPLITS) return (int)cudaErrorInvalidValue;
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
-  if (!configured[dev]) {
-    const cudaError_t ce = cudaFuncSetAttribute(latent_attention_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LM_DYN_SMEM);
-    if (ce != cudaSuccess) return (int)ce;
-    configured[dev] = true;
-  }
+  const int max_splits = latent_mma_max_splits();
+  if (max_splits == 0) return (int)cudaErrorInvalidDevice;
+  if (n_splits > max_splits) n_splits = max_splits;
   CUtensorMap tk, tq;
   int e = oxb_make_tmap_2d(&tk, cache, (uint64_t)num_blocks * page, width, (uint64_t)width * 2, page, 64, 2);
   if (e) return e;

@@ -150,11 +150,14 @@ def attention_simt(q, kv, layer: int, meta, spec, sink, out):
                                            kv.num_blocks, spec.window, spec.scale, _stream()), "oxb_latent_attention_simt")
 
 
-def mma_splits(B: int, row_blocks: int, window: int, max_len: int, sms: int) -> int:
-    """Key splits of the tensor-core kernel: as many as fit one wave of CTAs (one per SM), at least two 64-key tiles each."""
+def mma_splits(B: int, row_blocks: int, window: int, max_len: int, sms: int, most: int) -> int:
+    """Key splits of the tensor-core kernel: as many as fit one wave of CTAs (one per SM), a 128-key tile or more each; the
+    splits of a row block are one cluster of at most ``most`` CTAs (more than eight only where they fill few clusters)."""
     span = min(window, max_len) if window > 0 else max_len
     tiles = span // 128 + 1
-    return max(1, min(sms // max(1, B * row_blocks), tiles, 8))
+    if B * row_blocks > 2:
+        most = min(most, 8)
+    return max(1, min(sms // max(1, B * row_blocks), tiles, most))
 
 
 def attention_mma(q, kv, layer: int, meta, spec, sink, out, splits: Optional[int] = None):
@@ -166,7 +169,8 @@ def attention_mma(q, kv, layer: int, meta, spec, sink, out, splits: Optional[int
         return False
     row_blocks = (mq * H + 31) // 32
     if splits is None:
-        splits = mma_splits(B, row_blocks, spec.window, meta.max_seq_len or kv.page_size, opcuda.sm_count(q.device))
+        splits = mma_splits(B, row_blocks, spec.window, meta.max_seq_len or kv.page_size, opcuda.sm_count(q.device),
+                            lib().oxb_latent_max_splits())
     _check(lib().oxb_latent_attention_mma(q.data_ptr(), out.data_ptr(), kv.data[layer].data_ptr(), meta.block_tables.data_ptr(),
                                           meta.seq_lens.data_ptr(), meta.query_start.data_ptr(), _p(sink), B,
                                           meta.block_tables.stride(0), T, H, spec.latent_pad, width, kv.page_size, kv.num_blocks,

@@ -169,7 +169,8 @@ def attend_plain(q, rows, qlens, ctx, spec, sink):
 CASES = [  # heads, rank, rotated, window, rows per sequence, context lengths, page, key splits
     (5, 40, 6, 19, [1, 1, 1], [100, 5, 19], 16, None), (5, 40, 6, 19, [37, 1, 2], [100, 5, 64], 16, 1),
     (3, 96, 8, 0, [1, 4], [300, 130], 16, 3), (12, 136, 24, 130, [1, 1], [400, 131], 32, 2), (2, 24, 2, 1, [9, 1], [20, 64], 8, None),
-    (40, 200, 16, 65, [3, 2], [128, 65], 64, None), (7, 512, 64, 100, [2, 1], [260, 33], 16, 2), (33, 64, 64, 64, [70], [70], 16, None)]
+    (40, 200, 16, 65, [3, 2], [128, 65], 64, None), (7, 512, 64, 100, [2, 1], [260, 33], 16, 2), (33, 64, 64, 64, [70], [70], 16, None),
+    (4, 48, 8, 0, [1], [1500], 16, 12), (4, 48, 8, 0, [1], [300], 16, 16)]
 
 
 @pytest.mark.parametrize("device,dtype", [CPU, F32, B16])
