@@ -390,6 +390,8 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, sumsq_in: Option
 def embed(tokens: torch.Tensor, table, dtype: torch.dtype, scale: float = 1.0) -> torch.Tensor:
     T = tokens.shape[0]
     V, H = table.shape
+    if dtype == torch.float32 and table.qtype == "F32":  # float32 compute: the kernel's output is bf16
+        return table.data.index_select(0, tokens.long()) * scale
     out = torch.empty(T, H, dtype=torch.bfloat16, device=tokens.device)
     row_bytes = table.data.stride(0) * table.data.element_size()
     _check(lib().oxb_embed(tokens.data_ptr(), table.data.data_ptr(), QTYPE_CODE[table.qtype], row_bytes, H, V, scale,
