@@ -154,7 +154,7 @@ def kernel_numbers(width: int, heads: int, window: int, dev, steps: int) -> list
     model = Transformer(weights(cfg, dev), max_context=1 << 15)
     m = model.w.layers[0].mla
     op = CL.operands(m, spec, torch.bfloat16)
-    rope = model.layer_ropes[0]
+    rope = model.layer_ropes[0][0]
     nkv = max(1, heads // 4)
     grope = RopeState(ref.rope_inv_freq(128, 1e6, None, device=dev), "split_half", 1.0, heads, nkv, 128)
 

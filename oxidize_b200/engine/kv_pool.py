@@ -11,8 +11,9 @@ block id here addresses device memory:
                     uint8 codes (q8: head_dim bytes, q4: head_dim/2 bytes)
     scales[layer] : [num_blocks, n_kv_heads, 2, page, head_dim/32] f32   (q8/q4 only)
 
-(latent attention keeps one plane of rows instead of the K / V pair, and the rows of different layers may differ in
-width: ``KVCacheSpec.planes`` / ``row_dims``),
+(latent attention keeps one plane of rows instead of the K / V pair, and different layers may differ in heads, planes and
+row width: ``KVCacheSpec.planes`` / ``shapes``; recurrent layers keep one state per sequence instead of rows, see
+``StateStore``),
 
 so one (block, head, K) tile of a 16-token page with head_dim 128 is 4 KB contiguous — one
 TMA box / one fully coalesced burst in the attention kernels.
@@ -168,16 +169,23 @@ class KVCacheSpec:
     page_size: int = 16
     dtype_name: str = "bf16"
     planes: int = 2  # rows per token and head: K and V, or one shared (latent) row
-    row_dims: Optional[Tuple[int, ...]] = None  # row width of each layer where they differ (else head_dim everywhere)
+    # (heads, planes, row width) of each layer where they differ (else n_kv_heads, planes, head_dim everywhere)
+    shapes: Optional[Tuple[Tuple[int, int, int], ...]] = None
+
+    def shape(self, layer: int) -> Tuple[int, int, int]:
+        return (self.n_kv_heads, self.planes, self.head_dim) if self.shapes is None else tuple(self.shapes[layer])
 
     def row_dim(self, layer: int) -> int:
-        return self.head_dim if self.row_dims is None else self.row_dims[layer]
+        return self.shape(layer)[2]
+
+    def heads(self, layer: int) -> int:
+        return self.shape(layer)[0]
 
     def bytes_per_block(self) -> int:
-        e = self.n_kv_heads * self.planes * self.page_size
         total = 0
         for l in range(self.n_layers):
-            d = self.row_dim(l)
+            heads, planes, d = self.shape(l)
+            e = heads * planes * self.page_size
             if self.dtype_name == "q8":
                 total += e * (d + d // 32 * 4)
             elif self.dtype_name == "q4":
@@ -193,20 +201,21 @@ class KVCache:
     def __init__(self, spec: KVCacheSpec, num_blocks: int, device="cpu"):
         if spec.dtype_name not in KV_DTYPES:
             raise ValueError(f"kv dtype must be one of {sorted(KV_DTYPES)}")
-        dims = [spec.row_dim(l) for l in range(spec.n_layers)]
-        if spec.dtype_name in ("q8", "q4") and any(d % 32 for d in dims):
+        shapes = [spec.shape(l) for l in range(spec.n_layers)]
+        if spec.dtype_name in ("q8", "q4") and any(d % 32 for _, _, d in shapes):
             raise ValueError("quantized KV needs head_dim % 32 == 0")
         self.spec = spec
         self.num_blocks = num_blocks
         self.page_size = spec.page_size
         self.dtype_name = spec.dtype_name
         self.device = torch.device(device)
-        lead = (num_blocks, spec.n_kv_heads, spec.planes, spec.page_size)
-        self.data = [torch.zeros(lead + (d if spec.dtype_name != "q4" else d // 2,), dtype=KV_DTYPES[spec.dtype_name],
-                                 device=self.device) for d in dims]
+        self.data = [torch.zeros((num_blocks, h, n, spec.page_size, d if spec.dtype_name != "q4" else d // 2),
+                                 dtype=KV_DTYPES[spec.dtype_name], device=self.device) for h, n, d in shapes]
         self.scales: List[Optional[torch.Tensor]] = [None] * spec.n_layers
         if spec.dtype_name in ("q8", "q4"):
-            self.scales = [torch.zeros(lead + (d // 32,), dtype=torch.float32, device=self.device) for d in dims]
+            self.scales = [torch.zeros((num_blocks, h, n, spec.page_size, d // 32), dtype=torch.float32, device=self.device)
+                           for h, n, d in shapes]
+        self.states: Optional["StateStore"] = None  # recurrent state beside the rows (models that carry one)
 
     def copy_block(self, src: int, dst: int) -> None:
         """Copy-on-write support: duplicate one page in every layer."""
@@ -240,3 +249,33 @@ class KVCache:
         if "scales" in state:
             for l, s in enumerate(state["scales"]):
                 self.scales[l][idx] = s.to(self.device)
+
+
+class StateSlots:
+    """Host-side allocator of recurrent-state slots: one per running sequence, handed out at admission and given back when
+    the sequence ends or is preempted.  A slot carries nothing over: the kernels start a sequence's first token from zero."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self.free: List[int] = list(range(num_slots - 1, -1, -1))
+
+    def allocate(self) -> int:
+        if not self.free:
+            raise OutOfBlocks("no recurrent-state slot is free")
+        return self.free.pop()
+
+    def release(self, slot: int) -> None:
+        if not 0 <= slot < self.num_slots or slot in self.free:
+            raise RuntimeError(f"double free of state slot {slot}")
+        self.free.append(slot)
+
+
+class StateStore:
+    """Device storage of the recurrent states: data[layer] [num_slots, heads, keys, values] float32."""
+
+    def __init__(self, shapes: Sequence[Tuple[int, int, int]], num_slots: int, device="cpu"):
+        self.num_slots = num_slots
+        self.data = [torch.zeros((num_slots,) + tuple(s), dtype=torch.float32, device=device) for s in shapes]
+
+    def nbytes(self) -> int:
+        return sum(d.numel() * 4 for d in self.data)

@@ -22,7 +22,7 @@ from ..models.registry import act_dtype_for, config_from_checkpoint, load_checkp
 from ..models.transformer import Transformer
 from ..models.weights import ModelWeights
 from ..utils import profiler as _profiler
-from .kv_pool import BlockPool, KVCacheSpec, make_block_pool
+from .kv_pool import BlockPool, KVCacheSpec, StateSlots, make_block_pool
 from .runner import ModelRunner, StepResult
 from .sampler import SamplingParams
 from .scheduler import ScheduledSeq, Scheduler, SchedulerConfig, SchedulerOutput, Sequence
@@ -110,13 +110,14 @@ class LLM:
         # (a hybrid model's convolution layers keep one hidden-sized row per token as well)
         conv_bytes = self.model.n_conv_layers * c.kv_page_size * self.cfg.hidden_size * (2 if self.device.type == "cuda" else 4)
         nblocks = c.num_kv_blocks or self._auto_blocks(spec, conv_bytes)
-        self.kv = self.model.new_cache(nblocks, c.kv_page_size, kv_dtype)
-        # a recurrent state cannot be rebuilt from shared pages: state-space models run without the prefix cache
-        prefix_cache = c.enable_prefix_cache and not self.cfg.is_ssm
+        self.kv = self.model.new_cache(nblocks, c.kv_page_size, kv_dtype, c.max_num_seqs)
+        # a recurrent state cannot be rebuilt from shared pages: models that carry one run without the prefix cache
+        prefix_cache = c.enable_prefix_cache and not self.cfg.has_state
         self.pool = make_block_pool(nblocks, c.kv_page_size, prefix_cache)
         # a window that applies to every layer lets the scheduler hand pages back as they fall out of it
         self.scheduler = Scheduler(SchedulerConfig(c.max_num_batched_tokens, c.prefill_chunk_size, c.max_num_seqs,
-                                                   c.policy, prefix_cache, c.max_model_len, self.cfg.uniform_window), self.pool)
+                                                   c.policy, prefix_cache, c.max_model_len, self.cfg.uniform_window), self.pool,
+                                   StateSlots(c.max_num_seqs) if self.kv.states is not None else None)
         self.runner = ModelRunner(self.model, self.kv, max(c.max_num_batched_tokens, c.max_num_seqs), c.max_num_seqs,
                                   c.max_model_len, c.cuda_graphs and not _profiler.PROFILE and not _profiler.TRACE_FWD
                                   and isinstance(weights.layers, list)  # a captured graph would pin evicted layers' addresses
@@ -186,6 +187,7 @@ class LLM:
             return max(16, min(want, 4096))
         free, total = torch.cuda.mem_get_info(self.device)
         budget = int(free - (1.0 - c.gpu_memory_utilization) * total)
+        budget -= 4 * c.max_num_seqs * sum(h * k * v for h, k, v in self.cfg.state_shapes)
         fit = max(16, budget // max(spec.bytes_per_block() + extra_bytes_per_block, 1))
         return int(min(want, fit))
 

@@ -2,8 +2,8 @@
 (CUDA-graph replay for decode-only steps), samples, and hands tokens back to the host.
 
 Per step the host writes ONE pinned int32 staging buffer laid out as
-``[token_ids | positions | slot_mapping | query_start | seq_lens | logits_indices |
-block_tables]`` plus a small float section with per-sequence sampling knobs and this step's
+``[token_ids | positions | slot_mapping | query_start | seq_lens | state_slots |
+logits_indices | block_tables]`` plus a small float section with per-sequence sampling knobs and this step's
 uniform draws; one async copy moves it to a device buffer of identical layout whose
 sub-views have fixed addresses, so captured graphs stay valid (the role of the reference's
 3-word ``{pos, context, token}`` device state, ``backends/cuda/cuda_decode_graph.rs:45-52``,
@@ -40,7 +40,7 @@ class StagingBuffers:
         self.max_tokens, self.max_seqs, self.max_blocks = max_tokens, max_seqs, max_blocks_per_seq
         T, B, M = max_tokens, max_seqs, max_blocks_per_seq
         sizes = [("token_ids", T), ("positions", T), ("slot_mapping", T), ("query_start", B + 1), ("seq_lens", B),
-                 ("logits_indices", T), ("top_k", T), ("block_tables", B * M)]
+                 ("state_slots", B), ("logits_indices", T), ("top_k", T), ("block_tables", B * M)]
         fsizes = [("temperature", T), ("top_p", T), ("min_p", T), ("random", T)]
         self.offsets: Dict[str, Tuple[int, int]] = {}
         off = 0
@@ -140,6 +140,7 @@ class ModelRunner:
         b = self.buf
         tok, pos, slot = b.h("token_ids"), b.h("positions"), b.h("slot_mapping")
         qs, sl, li, bt = b.h("query_start"), b.h("seq_lens"), b.h("logits_indices"), b.h("block_tables")
+        ss_slot = b.h("state_slots")
         M, ps = self.max_blocks, self.page
         t = 0
         nl = 0
@@ -162,6 +163,7 @@ class ModelRunner:
                 cache = (nb, blist[-1] if nb else -1, np.asarray(blist, dtype=np.int32))
                 seq._blocks_np = cache
             bt[i * M : i * M + nb] = cache[2]
+            ss_slot[i] = seq.state_slot
             if n == 1 and not ss.is_prefill:
                 # decode row: plain integer arithmetic, no temporaries
                 tok[t] = seq.token_at(start)
@@ -212,6 +214,7 @@ class ModelRunner:
                 pos[t] = 0
                 slot[t] = -1
                 sl[i] = 0
+                ss_slot[i] = -1
                 qs[i + 1] = t + 1
                 li[nl] = t
                 nl += 1
@@ -248,6 +251,8 @@ class ModelRunner:
         pos[:n] = starts
         slot[:n] = [seq.blocks[st // ps] * ps + st % ps for seq, st in zip(seqs, starts)]
         np.add(pos[:n], 1, out=sl[:n])
+        st_slot = b.h("state_slots")
+        st_slot[:n] = [seq.state_slot for seq in seqs]
         qs[: n + 1] = ar[: n + 1]
         if all(ss.sample for ss in scheduled):
             rows = [(ss, i, 1) for i, ss in enumerate(scheduled)]
@@ -270,6 +275,7 @@ class ModelRunner:
             pos[t : t + k] = 0
             slot[t : t + k] = -1
             sl[B:pad_to] = 0
+            st_slot[B:pad_to] = -1
             qs[B + 1 : pad_to + 1] = ar[t + 1 : t + k + 1]
             li[nl : nl + k] = ar[t : t + k]
             nl += k
@@ -305,7 +311,7 @@ class ModelRunner:
         return BatchMeta(
             logits_all=logits_all,
             token_ids=b.d("token_ids", T), positions=b.d("positions", T), slot_mapping=b.d("slot_mapping", T),
-            query_start=b.d("query_start", B + 1), seq_lens=b.d("seq_lens", B),
+            query_start=b.d("query_start", B + 1), seq_lens=b.d("seq_lens", B), state_slots=b.d("state_slots", B),
             block_tables=b.d("block_tables").view(b.max_seqs, self.max_blocks)[:B],
             logits_indices=b.d("logits_indices", nl), max_query_len=max_q, max_seq_len=max_len, num_seqs=B)
 
@@ -494,6 +500,9 @@ class ModelRunner:
     def _capture(self, B: int, tie: str):
         """Capture one decode step for bucket ``B`` (every sequence feeds exactly one row)."""
         meta = self._meta(B, B, B, 1, self.max_blocks * self.page, logits_all=True)
+        # (the warm-up runs execute for real: without state slots they leave every recurrent state alone)
+        slots = meta.state_slots.clone()
+        meta.state_slots.fill_(-1)
         feed = self.buf.d("token_ids", B)  # every row's next input id, left on the device for a step that runs ahead
         # warm up on a side stream so lazy initialisation does not land inside the capture
         s = torch.cuda.Stream()
@@ -503,6 +512,7 @@ class ModelRunner:
                 # (no token feed here: these runs execute for real and must leave the step's input ids alone)
                 self.model.greedy_tokens(meta, self.kv, tie)
         torch.cuda.current_stream().wait_stream(s)
+        meta.state_slots.copy_(slots)
         torch.cuda.synchronize()
         from ..ops import cuda as opcuda
 

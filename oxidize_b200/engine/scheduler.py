@@ -22,7 +22,7 @@ from collections import deque
 from dataclasses import dataclass, field
 from typing import Deque, Dict, Iterable, List, Optional, Sequence, Tuple
 
-from .kv_pool import FNV_OFFSET, BlockPool, OutOfBlocks, block_hash
+from .kv_pool import FNV_OFFSET, BlockPool, OutOfBlocks, StateSlots, block_hash
 from .sampler import RequestRng, SamplingParams
 
 
@@ -58,6 +58,7 @@ class Sequence:
         self.params = params
         self.status = SeqStatus.WAITING
         self.blocks: List[int] = []
+        self.state_slot = -1  # slot of the recurrent state while the sequence runs (models that carry one)
         self.num_computed = 0  # tokens whose KV is in the cache
         self.finish_reason: Optional[str] = None
         self.rng = RequestRng(params.seed)
@@ -125,9 +126,10 @@ class SchedulerOutput:
 
 
 class Scheduler:
-    def __init__(self, config: SchedulerConfig, pool: BlockPool):
+    def __init__(self, config: SchedulerConfig, pool: BlockPool, slots: Optional[StateSlots] = None):
         self.config = config
         self.pool = pool
+        self.slots = slots  # recurrent-state slots; None: the model carries no state
         self.waiting: Deque[Sequence] = deque()
         self.running: List[Sequence] = []
         self.finished: List[Sequence] = []
@@ -155,13 +157,26 @@ class Scheduler:
     def has_work(self) -> bool:
         return bool(self.waiting or self.running)
 
+    def _start(self, seq: Sequence) -> None:
+        seq.status = SeqStatus.RUNNING
+        if self.slots is not None:
+            seq.state_slot = self.slots.allocate()
+        self.running.append(seq)
+
+    def _give_back(self, seq: Sequence) -> None:
+        """What a sequence holds in the cache and the state store."""
+        self.pool.release_all(seq.blocks[seq._released:])
+        seq.blocks, seq._released = [], 0
+        if seq.state_slot >= 0:
+            self.slots.release(seq.state_slot)
+            seq.state_slot = -1
+
     def _finish(self, seq: Sequence, reason: str) -> None:
         if seq.is_finished:
             return
         seq.status = SeqStatus.FINISHED
         seq.finish_reason = reason
-        self.pool.release_all(seq.blocks[seq._released:])
-        seq.blocks, seq._released = [], 0
+        self._give_back(seq)
         if seq in self.running:
             self.running.remove(seq)
         try:
@@ -171,8 +186,7 @@ class Scheduler:
         self.finished.append(seq)
 
     def _preempt(self, seq: Sequence) -> None:
-        self.pool.release_all(seq.blocks[seq._released:])
-        seq.blocks, seq._released = [], 0
+        self._give_back(seq)
         seq.num_computed = 0
         seq._hash_state = FNV_OFFSET
         seq._published = 0
@@ -308,8 +322,7 @@ class Scheduler:
                 still.append(seq)
                 blocked = True
                 continue
-            seq.status = SeqStatus.RUNNING
-            self.running.append(seq)
+            self._start(seq)
             last = seq.num_computed + chunk == len(seq.prompt)
             out.scheduled.append(ScheduledSeq(seq, seq.num_computed, chunk, True, last))
             budget -= chunk
@@ -326,8 +339,7 @@ class Scheduler:
             if seq.status is SeqStatus.WAITING:
                 if len(self.running) >= self.config.max_num_running_seqs:
                     raise RuntimeError(f"more than {self.config.max_num_running_seqs} sequences at a time")
-                seq.status = SeqStatus.RUNNING
-                self.running.append(seq)
+                self._start(seq)
             start = seq.num_computed
             if n < 1 or start + n > len(seq.prompt):
                 raise ValueError(f"sequence {seq.request_id} has {len(seq.prompt) - start} tokens left, {n} were asked for")

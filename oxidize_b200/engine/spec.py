@@ -424,8 +424,8 @@ def attach_speculation(llm, draft_model_path: Optional[str], k: int = 4, use_mtp
         prop = DraftModelProposer(llm.weights, k, c.max_num_seqs, c.max_model_len, comm=llm.model.comm, kv_dtype="q4")
         llm.spec = SpecDecoder(prop, k)
         return llm.spec
-    if llm.cfg.is_ssm:
-        raise ValueError("speculative decoding needs a cache that can be rolled back: not available for state-space models")
+    if llm.cfg.has_state:
+        raise ValueError("speculative decoding needs a cache that can be rolled back: not available for models with a recurrent state")
     if draft_model_path:
         from ..formats.gguf import load_gguf
         from ..models.config import config_from_gguf

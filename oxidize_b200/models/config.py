@@ -10,7 +10,7 @@ from __future__ import annotations
 
 import dataclasses
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Tuple, Union
 
 from ..formats.gguf import GGUFFile
 
@@ -109,21 +109,174 @@ class LatentAttentionSpec:
     def qk_dim(self) -> int:
         return self.nope_dim + self.rope_dim
 
+    @property
+    def kv_heads(self) -> int:
+        return 1
+
+    @property
+    def cache_shape(self) -> Tuple[int, int, int]:
+        """(heads, planes, row width) of a cached token."""
+        return 1, 1, self.row_dim
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.v_dim
+
+
+# Head widths of the attention kernels (query, key and value rows of a head share one).
+HEAD_WIDTHS = (32, 64, 96, 128, 192, 256)
+
+
+@dataclass
+class AttentionSpec:
+    """Grouped-query attention with the geometry of a single layer.
+
+    ``window`` > 0 limits a query to that many latest positions (itself included); ``sink`` adds a learned per-head logit
+    to the softmax denominator only; ``qk_norm`` is an RMS norm of the queries and keys ahead of the rotation, per ``head``
+    (one weight for all heads) or over the ``full`` projection."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    v_dim: int
+    scale: float
+    rotary: RotarySpec
+    window: int = 0
+    sink: bool = False
+    qk_norm: str = ""  # "" | head | full
+
+    kv_from = None  # (every layer of this kind owns cache rows)
+
+    @property
+    def width(self) -> int:
+        """Values per head in queries, cached rows and outputs: the next kernel width (the padding is zero)."""
+        d = max(self.dim, self.v_dim)
+        return next((w for w in HEAD_WIDTHS if w >= d), (d + 31) // 32 * 32)
+
+    @property
+    def cache_shape(self) -> Tuple[int, int, int]:
+        return self.kv_heads, 2, self.width
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.width
+
+    @property
+    def proj_dim(self) -> int:
+        return (self.heads + 2 * self.kv_heads) * self.width
+
+
+@dataclass
+class RetentionSpec:
+    """Linear attention with a fixed decay per head: S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, with rotated queries
+    and keys and k scaled by dim ** -0.5; each head's o is divided by its root mean square and multiplied by silu of a gate
+    projection.  Every sequence carries one [dim, v_dim] float32 state per head."""
+
+    heads: int
+    dim: int
+    v_dim: int
+    decay: List[float]
+    rotary: RotarySpec
+
+    # head widths in projections, state and outputs (the padding is zero)
+    @property
+    def k_width(self) -> int:
+        return (self.dim + 31) // 32 * 32
+
+    @property
+    def v_width(self) -> int:
+        return (self.v_dim + 15) // 16 * 16
+
+    @property
+    def state_shape(self) -> Tuple[int, int, int]:
+        return self.heads, self.k_width, self.v_width
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.v_width
+
+    @property
+    def proj_dim(self) -> int:
+        return 2 * self.heads * (self.k_width + self.v_width)
+
+
+@dataclass
+class ParallelSpec:
+    """Attention and retention side by side on the same input: left_scale * left + right_scale * right."""
+
+    left: AttentionSpec
+    right: RetentionSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
 
 @dataclass
 class FeedForwardSpec:
-    """W_down act(W_up x): a feed-forward block without a gate projection."""
+    """W_down act(W_up x), or with a gate projection W_down (act(W_gate x) * (W_up x))."""
 
     size: int
-    act: str = "relu2"  # the square of relu
+    act: str = "relu2"  # the square of relu | silu
+    gated: bool = False
+
+    @property
+    def pad_size(self) -> int:
+        """Rows of a gated block's two projections: the tile of the fused kernel (the padding is zero)."""
+        return (self.size + 63) // 64 * 64 if self.gated else self.size
+
+
+@dataclass
+class MoESpec:
+    """Routed experts: the ``n_experts_used`` largest router logits choose, their softmax weighs; ``shared`` runs for every
+    token and is added.  (The routing fields carry the names that the routing operators read from ``ModelConfig``.)"""
+
+    n_experts: int
+    n_experts_used: int
+    expert: FeedForwardSpec
+    shared: Optional[FeedForwardSpec] = None
+    expert_gating: str = "softmax"
+    expert_weights_norm: bool = True
+    expert_weights_scale: float = 1.0
+    expert_group_count: int = 0
+    expert_group_used_count: int = 0
+
+    @property
+    def size(self) -> int:
+        """Feed-forward columns a token passes through."""
+        return self.n_experts_used * self.expert.size + (self.shared.size if self.shared else 0)
 
 
 @dataclass
 class LayerSpec:
     """One decoder layer of a model whose layers are listed one by one."""
 
-    mixer: LatentAttentionSpec
-    ffn: Optional[FeedForwardSpec] = None  # None: the layer has no feed-forward block
+    mixer: Union[LatentAttentionSpec, AttentionSpec, RetentionSpec, ParallelSpec]
+    ffn: Union[FeedForwardSpec, MoESpec, None] = None  # None: the layer has no feed-forward block
+    weights_of: Optional[int] = None  # an earlier layer whose weights this one uses (with cache rows and state of its own)
+
+    @property
+    def attention(self) -> Union[LatentAttentionSpec, AttentionSpec, None]:
+        """The part of the mixer that attends over cached rows."""
+        m = self.mixer
+        return m.left if isinstance(m, ParallelSpec) else None if isinstance(m, RetentionSpec) else m
+
+    @property
+    def retention(self) -> Optional[RetentionSpec]:
+        """The part of the mixer that carries a recurrent state."""
+        m = self.mixer
+        return m.right if isinstance(m, ParallelSpec) else m if isinstance(m, RetentionSpec) else None
+
+    @property
+    def owns_rows(self) -> bool:
+        return self.attention is not None and self.attention.kv_from is None
+
+    @property
+    def branch_scales(self) -> Tuple[float, float]:
+        m = self.mixer
+        return (m.left_scale, m.right_scale) if isinstance(m, ParallelSpec) else (1.0, 1.0)
+
+    @property
+    def out_dim(self) -> int:
+        return sum(p.out_dim for p in (self.attention, self.retention) if p is not None)
 
 
 @dataclass
@@ -213,6 +366,9 @@ class ModelConfig:
     # > 0: norm after the sum, x <- norm(residual_alpha * x + branch(x)), with the residual stream in float32;
     # 0: norm in front of the branch, x <- x + branch(norm(x))
     residual_alpha: float = 0.0
+    # Listed layers only: "after_sum" (the rule above), or "sandwich": norms on both sides of the branch,
+    # x <- x + norm_b(branch(norm_a(x))), with the residual stream in float32
+    norm_placement: str = "after_sum"
     embed_norm: bool = False  # the embedding passes a norm of its own
 
     @property
@@ -228,16 +384,26 @@ class ModelConfig:
         return bool(self.layer_specs)
 
     @property
-    def cache_rows(self) -> List[int]:
-        """Widths of the cached rows of a layered model, one per layer that owns cache rows (in layer order)."""
-        return [l.mixer.row_dim for l in self.layer_specs if l.mixer.kv_from is None]
+    def cache_shapes(self) -> List[Tuple[int, int, int]]:
+        """(heads, planes, row width) of a listed model's cached tokens, one per layer that owns cache rows (in layer order)."""
+        return [l.attention.cache_shape for l in self.layer_specs if l.owns_rows]
+
+    @property
+    def state_shapes(self) -> List[Tuple[int, int, int]]:
+        """Recurrent state of a sequence, one [heads, keys, values] per layer that carries one."""
+        return [l.retention.state_shape for l in self.layer_specs if l.retention is not None]
+
+    @property
+    def has_state(self) -> bool:
+        """Sequences carry a recurrent state, which cannot be rebuilt from shared pages or rolled back."""
+        return self.is_ssm or any(l.retention is not None for l in self.layer_specs)
 
     @property
     def uniform_window(self) -> int:
         """> 0 when every layer is windowed: no query of any layer looks back further than this."""
         if self.layer_specs:
-            ws = [l.mixer.window for l in self.layer_specs]
-            return max(ws) if min(ws) > 0 else 0
+            ws = [l.attention.window for l in self.layer_specs if l.attention is not None]
+            return max(ws) if ws and min(ws) > 0 else 0
         return self.sliding_window if (self.sliding_window > 0 and self.sliding_window_pattern == 0) else 0
 
     @property
@@ -270,13 +436,7 @@ class ModelConfig:
     def param_count(self) -> int:
         h = self.hidden_size
         if self.layer_specs:
-            n = 2 * self.vocab_size * h + (4 if self.norm_kind == "layer" else 2) * h
-            for l in self.layer_specs:
-                m, f = l.mixer, l.ffn
-                n += m.heads * (h * (m.qk_dim + m.v_dim) + m.kv_rank * (m.nope_dim + m.v_dim) + int(m.sink)) + 2 * h
-                n += 0 if m.kv_from is not None else h * (m.kv_rank + m.rope_dim) + m.kv_rank
-                n += 0 if f is None else 2 * h * f.size + 2 * h
-            return n
+            return self._listed_param_count()
         attn = h * self.q_size * 2 + h * self.kv_size * 2
         dense = 3 * h * self.ffn_size
         n = 0
@@ -288,6 +448,32 @@ class ModelConfig:
             else:
                 n += dense
         n += self.vocab_size * h * (1 if self.tie_embeddings else 2) + h
+        return n
+
+    def _listed_param_count(self) -> int:
+        h = self.hidden_size
+        norm = 2 * h if self.norm_kind == "layer" else h
+
+        def ffn(f) -> int:
+            if isinstance(f, MoESpec):
+                return f.n_experts * (ffn(f.expert) + h) + (ffn(f.shared) if f.shared else 0)
+            return (3 if f.gated else 2) * h * f.size
+
+        n = 2 * self.vocab_size * h + (2 if self.embed_norm else 1) * norm
+        for l in self.layer_specs:
+            if l.weights_of is not None:
+                continue
+            a, r = l.attention, l.retention
+            per_branch = 2 * norm if self.norm_placement == "sandwich" else norm
+            n += per_branch * (1 if l.ffn is None else 2) + (0 if l.ffn is None else ffn(l.ffn))
+            if isinstance(a, LatentAttentionSpec):
+                n += a.heads * (h * (a.qk_dim + a.v_dim) + a.kv_rank * (a.nope_dim + a.v_dim))
+                n += 0 if a.kv_from is not None else h * (a.kv_rank + a.rope_dim) + a.kv_rank
+            elif a is not None:
+                n += h * (a.heads + a.kv_heads) * (a.dim + a.v_dim)
+                n += {"": 0, "head": 2, "full": a.heads + a.kv_heads}[a.qk_norm] * a.dim
+            n += a.heads if a is not None and a.sink else 0
+            n += h * r.heads * (2 * r.dim + 3 * r.v_dim) if r is not None else 0
         return n
 
     def to_dict(self) -> Dict[str, Any]:

@@ -5,7 +5,12 @@
 
 Vefilix: layer norm (weight and bias) after each sum, ``x <- norm(alpha x + branch(x))``, with latent attention in a
 sliding window (a softmax sink per head, YaRN-scaled rotation, later layers reading an earlier layer's cached rows) and
-ungated squared-relu feed-forward blocks; the embedding and the output pass norms of their own."""
+ungated squared-relu feed-forward blocks; the embedding and the output pass norms of their own.
+
+Sokirax: RMS norms on both sides of every branch, x <- x + norm_b(branch(norm_a(x))); grouped-query attention in a window
+(per-head q / k norm, partial YaRN rotation), or such attention (norm over the whole projection, a softmax sink per head)
+beside retention on the same input; gated feed-forward blocks, dense or routed experts with a shared one; a layer may use an
+earlier layer's weights."""
 from __future__ import annotations
 
 import math
@@ -15,9 +20,10 @@ import numpy as np
 import torch
 
 from ..formats.layered import LayeredCheckpoint
-from .config import (FeedForwardSpec, LatentAttentionSpec, LayerSpec, ModelConfig, RopeScaling, RotarySpec,
-                     UnsupportedArchitecture)
-from .weights import LayerWeights, LinearWeight, MLAWeights, ModelWeights, QTensor, StreamedLayers, shard_range
+from .config import (AttentionSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, ModelConfig, MoESpec, ParallelSpec,
+                     RetentionSpec, RopeScaling, RotarySpec, UnsupportedArchitecture)
+from .weights import (ExpertWeights, LayerWeights, LinearWeight, MLAWeights, ModelWeights, QTensor, StreamedLayers,
+                      shard_range)
 
 
 # --------------------------------------------------------------------------- configuration
@@ -30,6 +36,11 @@ def _yarn(s: Optional[Dict[str, Any]], dims: int) -> Optional[RopeScaling]:
                        magnitude=0.1 * math.log(factor) + 1.0)
 
 
+def _rotary(rot: Dict[str, Any]) -> RotarySpec:
+    dims = int(rot["dims"])
+    return RotarySpec(dims, float(rot["base"]), _yarn(rot.get("scaling"), dims))
+
+
 def _latent_mixer(m: Dict[str, Any], layer: int) -> LatentAttentionSpec:
     rot = m["rot"]
     dims = int(rot["dims"])
@@ -39,7 +50,7 @@ def _latent_mixer(m: Dict[str, Any], layer: int) -> LatentAttentionSpec:
     src = m.get("kv_from")
     return LatentAttentionSpec(heads=int(m["heads"]), nope_dim=int(m["dim"]), rope_dim=int(m["rot_dim"]), v_dim=int(m["vdim"]),
                                kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
-                               rotary=RotarySpec(dims, float(rot["base"]), _yarn(rot.get("scaling"), dims)),
+                               rotary=_rotary(rot),
                                window=int(mask.get("size") or 0), sink=True, kv_from=None if src is None else int(src))
 
 
@@ -76,17 +87,90 @@ def _vefilix_config(ck: LayeredCheckpoint) -> ModelConfig:
                           residual_alpha=float(c["postln_alpha"]), embed_norm=True, name=str(ck.get("general.name", "")))
 
 
+def _attention(m: Dict[str, Any], qk_norm: str, sink: bool, layer: int) -> AttentionSpec:
+    mask = m.get("mask") or {}
+    a = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), v_dim=int(m["vdim"]),
+                      scale=float(m["scale"]), rotary=_rotary(m["rot"]), window=int(mask.get("size") or 0), sink=sink,
+                      qk_norm=qk_norm)
+    if a.heads % a.kv_heads:
+        raise UnsupportedArchitecture(f"layer {layer}: {a.heads} query heads over {a.kv_heads} key / value heads")
+    if a.rotary.dims % 2 or a.rotary.dims > a.dim:
+        raise UnsupportedArchitecture(f"layer {layer}: rotation of {a.rotary.dims} of {a.dim} values per head")
+    return a
+
+
+def _retention(m: Dict[str, Any], layer: int) -> RetentionSpec:
+    r = RetentionSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), [float(d) for d in m["decay"]], _rotary(m["rot"]))
+    if len(r.decay) != r.heads:
+        raise ValueError(f"layer {layer}: {len(r.decay)} decays for {r.heads} heads")
+    if any(not 0.0 < d <= 1.0 for d in r.decay):
+        raise UnsupportedArchitecture(f"layer {layer}: decays must lie in (0, 1]")
+    if r.rotary.dims % 2 or r.rotary.dims > r.dim:
+        raise UnsupportedArchitecture(f"layer {layer}: rotation of {r.rotary.dims} of {r.dim} values per head")
+    return r
+
+
+def _gated_ffn(f: Optional[Dict[str, Any]], layer: int):
+    if f is None:
+        return None
+    if f.get("kind") == "dense":
+        return FeedForwardSpec(int(f["ff"]), "silu", gated=True)
+    if f.get("kind") != "moe":
+        raise UnsupportedArchitecture(f"layer {layer}: feed-forward kind {f.get('kind')!r}")
+    shared = f.get("shared")
+    m = MoESpec(int(f["router"]["experts"]), int(f["router"]["top"]), FeedForwardSpec(int(f["expert"]["ff"]), "silu", True),
+                FeedForwardSpec(int(shared["ff"]), "silu", True) if shared else None)
+    if not 1 <= m.n_experts_used <= m.n_experts:
+        raise ValueError(f"layer {layer}: {m.n_experts_used} of {m.n_experts} experts per token")
+    return m
+
+
+def check_shared_weights(specs: List[LayerSpec]) -> None:
+    """A layer that uses another layer's weights names one that has weights of its own and the same geometry."""
+    for i, l in enumerate(specs):
+        j = l.weights_of
+        if j is None:
+            continue
+        if not 0 <= j < len(specs) or specs[j].weights_of is not None:
+            raise ValueError(f"layer {i}: weights_of {j} is not a layer with weights of its own")
+        if (l.mixer, l.ffn) != (specs[j].mixer, specs[j].ffn):
+            raise ValueError(f"layer {i} uses the weights of layer {j} but differs from it")
+
+
+def _sokirax_config(ck: LayeredCheckpoint) -> ModelConfig:
+    c = ck.config
+    specs = []
+    for i, l in enumerate(c["layers"]):
+        m = l["mixer"]
+        if l.get("type") == "attention":
+            mixer = _attention(m, "head", False, i)
+        elif l.get("type") == "parallel":
+            mixer = ParallelSpec(_attention(m["left"], "full", True, i), _retention(m["right"], i), float(m["left_scale"]),
+                                 float(m["right_scale"]))
+        else:
+            raise UnsupportedArchitecture(f"layer {i}: mixer type {l.get('type')!r}")
+        src = l.get("weights_of")
+        specs.append(LayerSpec(mixer, _gated_ffn(l.get("mlp"), i), None if src is None else int(src)))
+    check_shared_weights(specs)
+    return layered_config("sokirax", int(c["vocab"]), int(c["width"]), specs, eps=float(c["norm"]["eps"]), norm_kind="rms",
+                          norm_placement="sandwich", name=str(ck.get("general.name", "")))
+
+
 def layered_config(arch: str, vocab: int, width: int, specs: List[LayerSpec], eps: float, norm_kind: str,
-                   residual_alpha: float, embed_norm: bool, name: str = "") -> ModelConfig:
-    m0 = specs[0].mixer
+                   residual_alpha: float = 1.0, embed_norm: bool = False, name: str = "",
+                   norm_placement: str = "after_sum") -> ModelConfig:
+    atts = [l.attention for l in specs if l.attention is not None]
+    m0 = atts[0] if atts else specs[0].retention
     ffn = max([l.ffn.size for l in specs if l.ffn is not None], default=0)
     return ModelConfig(arch=arch, name=name, vocab_size=vocab, hidden_size=width, n_layers=len(specs), n_heads=m0.heads,
-                       n_kv_heads=1, head_dim=max(l.mixer.row_dim for l in specs), ffn_size=ffn, rms_eps=eps,
-                       rope_theta=m0.rotary.base, rope_dim=m0.rotary.dims, attn_scale=m0.scale, context_length=1 << 20,
-                       layer_specs=specs, norm_kind=norm_kind, residual_alpha=residual_alpha, embed_norm=embed_norm)
+                       n_kv_heads=max([a.kv_heads for a in atts], default=1),
+                       head_dim=max([a.cache_shape[2] for a in atts], default=16), ffn_size=ffn, rms_eps=eps,
+                       rope_theta=m0.rotary.base, rope_dim=m0.rotary.dims, attn_scale=getattr(m0, "scale", 0.0),
+                       context_length=1 << 20, layer_specs=specs, norm_kind=norm_kind, residual_alpha=residual_alpha,
+                       embed_norm=embed_norm, norm_placement=norm_placement)
 
 
-READERS: Dict[str, Callable[[LayeredCheckpoint], ModelConfig]] = {"vefilix": _vefilix_config}
+READERS: Dict[str, Callable[[LayeredCheckpoint], ModelConfig]] = {"vefilix": _vefilix_config, "sokirax": _sokirax_config}
 
 
 def config_from_layered(ck: LayeredCheckpoint) -> ModelConfig:
@@ -138,6 +222,101 @@ def latent_weights(spec: LatentAttentionSpec, q: torch.Tensor, dkv: Optional[tor
                       q=LinearWeight([dense_qtensor(rows.contiguous())]), sink=sink)
 
 
+def pad_heads(t: torch.Tensor, heads: int, width: int, dim: int = 0) -> torch.Tensor:
+    """Every head's values along axis ``dim`` followed by zeros up to ``width`` of them."""
+    n = t.shape[dim] // heads
+    if n == width:
+        return t
+    shape = list(t.shape)
+    parts = t.reshape(shape[:dim] + [heads, n] + shape[dim + 1 :])
+    pad = torch.zeros(shape[:dim] + [heads, width - n] + shape[dim + 1 :], dtype=t.dtype, device=t.device)
+    return torch.cat([parts, pad], dim=dim + 1).reshape(shape[:dim] + [heads * width] + shape[dim + 1 :])
+
+
+def listed_mixer(spec: LayerSpec, att: Dict[str, torch.Tensor], ret: Dict[str, torch.Tensor]) -> Dict[str, Any]:
+    """Attention and / or retention tensors (as stored) of one layer in the layout the forward pass uses: one matrix over
+    the layer's input, attention q | k | v then retention q | k | v | gate, and one output matrix over both mixers' heads,
+    every head padded with zeros to its kernel width."""
+    ins, outs, kw = [], [], {}
+    a, r = spec.attention, spec.retention
+    if a is not None:
+        for n, heads in (("q", a.heads), ("k", a.kv_heads), ("v", a.kv_heads)):
+            ins.append(pad_heads(att[n], heads, a.width))
+        outs.append(pad_heads(att["o"], a.heads, a.width, dim=1))
+        if a.qk_norm:
+            full = a.qk_norm == "full"
+            kw["q_norm"] = pad_heads(att["q.norm"], a.heads if full else 1, a.width).contiguous()
+            kw["k_norm"] = pad_heads(att["k.norm"], a.kv_heads if full else 1, a.width).contiguous()
+        kw["sink"] = att["sink"] if a.sink else None
+    if r is not None:
+        for n, width in (("q", r.k_width), ("k", r.k_width), ("v", r.v_width), ("g", r.v_width)):
+            ins.append(pad_heads(ret[n], r.heads, width))
+        outs.append(pad_heads(ret["o"], r.heads, r.v_width, dim=1))
+    kw["wqkv"] = LinearWeight([dense_qtensor(torch.cat(ins, dim=0).contiguous())])
+    kw["wo"] = LinearWeight([dense_qtensor(torch.cat(outs, dim=1).contiguous())])
+    return kw
+
+
+def gated_pair(gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor, size: int, rows: int = 0,
+               cols: int = 0) -> Tuple[QTensor, QTensor]:
+    """([gate | up], down) with ``size`` feed-forward columns, the input padded to ``cols`` values and the output to
+    ``rows``."""
+    def grow(t, n, k):
+        return torch.nn.functional.pad(t, (0, max(k - t.shape[1], 0), 0, max(n - t.shape[0], 0)))
+
+    gu = torch.cat([grow(gate, size, cols), grow(up, size, cols)], dim=0).contiguous()
+    return dense_qtensor(gu), dense_qtensor(grow(down, rows, size).contiguous())
+
+
+def listed_experts(spec: MoESpec, triples, hidden: int) -> ExpertWeights:
+    """The experts' (gate, up, down), stacked; inner sizes are multiples of the grouped product's k-block."""
+    h64 = (hidden + 63) // 64 * 64
+    pairs = [gated_pair(g, u, d, spec.expert.pad_size, h64, h64) for g, u, d in triples]
+    ex = ExpertWeights([p[0] for p in pairs], [p[1] for p in pairs])
+    for name in ("gate_up", "down"):
+        lst = getattr(ex, name)
+        n, k = lst[0].shape
+        stack = dense_qtensor(torch.cat([q.data for q in lst], dim=0).contiguous())
+        setattr(ex, name + "_stack", stack)
+        for i, q in enumerate(lst):
+            q.data = stack.data[i * n : (i + 1) * n]
+    return ex
+
+
+def _load_listed(src: LayeredWeightSource, cfg: ModelConfig, i: int) -> LayerWeights:
+    """A layer with norms on both sides of its branches."""
+    spec, p = cfg.layer_specs[i], f"l{i}"
+
+    def mixer(prefix: str, names, part) -> Dict[str, torch.Tensor]:
+        return {n: src.dense(f"{p}.mix.{prefix}{n}") for n in names} if part is not None else {}
+
+    both = isinstance(spec.mixer, ParallelSpec)
+    a, r = spec.attention, spec.retention
+    att, ret = mixer("left." if both else "", ("q", "k", "v", "o"), a), mixer("right." if both else "", ("q", "k", "v", "g", "o"), r)
+    for n in (("q.norm", "k.norm") if a is not None and a.qk_norm else ()) + (("sink",) if a is not None and a.sink else ()):
+        att[n] = src.vector(f"{p}.mix.{'left.' if both else ''}{n}")
+    lw = LayerWeights(attn_norm=src.vector(f"{p}.norm1"), post_attn_norm=src.vector(f"{p}.norm1b"), ffn_norm=None,
+                      **listed_mixer(spec, att, ret))
+    f = spec.ffn
+    if f is None:
+        return lw
+    lw.ffn_norm, lw.post_ffn_norm = src.vector(f"{p}.norm2"), src.vector(f"{p}.norm2b")
+
+    def triple(prefix: str):
+        return tuple(src.dense(f"{p}.mlp.{prefix}{n}") for n in ("gate", "up", "down"))
+
+    if isinstance(f, MoESpec):
+        lw.router = src.matrix(f"{p}.mlp.router")
+        lw.experts = listed_experts(f, [triple(f"e{e}.") for e in range(f.n_experts)], cfg.hidden_size)
+        if f.shared is not None:
+            gu, down = gated_pair(*triple("shared."), f.shared.pad_size)
+            lw.shared_gate_up, lw.shared_down = LinearWeight([gu]), LinearWeight([down])
+    else:
+        gu, down = gated_pair(*triple(""), f.pad_size)
+        lw.w_gate_up, lw.w_down = LinearWeight([gu]), LinearWeight([down])
+    return lw
+
+
 def _load_layer(src: LayeredWeightSource, spec: LayerSpec, i: int, tp_rank: int, tp_size: int) -> LayerWeights:
     p, m = f"l{i}", spec.mixer
     h0, h1 = shard_range(m.heads, tp_rank, tp_size)
@@ -163,13 +342,24 @@ def load_layered_weights(ck: LayeredCheckpoint, cfg: ModelConfig, device="cpu", 
     replicated (every rank caches the whole latent row)."""
     src = LayeredWeightSource(ck, device, act_dtype)
     n = cfg.n_layers
+    sandwich = cfg.norm_placement == "sandwich"
+    if sandwich and tp_size > 1:
+        raise ValueError("a norm over all heads and per-sequence states are not sharded: run this model with tp_size = 1")
+
+    def load(i: int) -> LayerWeights:
+        return _load_listed(src, cfg, i) if sandwich else _load_layer(src, cfg.layer_specs[i], i, tp_rank, tp_size)
+
+    source = [i if l.weights_of is None else l.weights_of for i, l in enumerate(cfg.layer_specs)]
     if 0 < resident_layers < n:
-        layers = StreamedLayers(lambda i: _load_layer(src, cfg.layer_specs[i], i, tp_rank, tp_size), n, resident_layers)
+        layers = StreamedLayers(lambda i: load(source[i]), n, resident_layers)
     else:
-        layers = [_load_layer(src, cfg.layer_specs[i], i, tp_rank, tp_size) for i in range(n)]
+        own = {i: load(i) for i in sorted(set(source))}
+        layers = [own[i] for i in source]
     v0, v1 = shard_range(cfg.vocab_size, tp_rank, tp_size) if cfg.vocab_size % tp_size == 0 else (0, cfg.vocab_size)
     mw = ModelWeights(cfg, src.matrix("embed"), layers, src.vector("final.norm"), LinearWeight([src.matrix("head", rows=(v0, v1))]),
                       [], tp_rank, tp_size, 0, 1, 0, v0)
-    mw.out_norm_bias = src.vector("final.norm.b")
-    mw.embed_norm, mw.embed_norm_bias = src.vector("embed.norm"), src.vector("embed.norm.b")
+    if cfg.norm_kind == "layer":
+        mw.out_norm_bias = src.vector("final.norm.b")
+    if cfg.embed_norm:
+        mw.embed_norm, mw.embed_norm_bias = src.vector("embed.norm"), src.vector("embed.norm.b")
     return mw

@@ -24,7 +24,7 @@ import torch
 from .. import ops
 from ..utils import profiler as _profiler
 from ..ops import ref as opref
-from .config import ModelConfig
+from .config import ModelConfig, MoESpec
 from .weights import LayerWeights, ModelWeights
 
 
@@ -59,6 +59,7 @@ class BatchMeta:
     # (rows fed, context length) of every sequence, known on the host for steps that are built eagerly; kernels that prepare
     # whole contexts (latent attention over long portions) size their work from it
     host_lens: Optional[List[Tuple[int, int]]] = None
+    state_slots: Optional[torch.Tensor] = None  # [B] slot of each sequence's recurrent state, -1 = none (padding rows)
 
 
 class SingleRankComm:
@@ -176,29 +177,33 @@ class Transformer:
         if self.pipe is not None:
             raise ValueError("a model with per-layer geometry runs as one pipeline stage (layers may share cached rows)")
         ropes: dict = {}
-        self.layer_ropes: List[RopeState] = []
-        owners = [i for i, l in enumerate(cfg.layer_specs) if l.mixer.kv_from is None]
-        self.kv_index = []
-        for i, l in enumerate(cfg.layer_specs):
-            r = l.mixer.rotary
+
+        def rope(r):
             key = repr(r)
             if key not in ropes:
                 ropes[key] = RopeState(
                     inv_freq=opref.rope_inv_freq(r.dims, r.base, r.scaling, device=self.device, dtype=torch.float64),
                     pairing=r.pairing, mscale=opref.rope_mscale(r.scaling), n_heads=0, n_kv_heads=1, head_dim=r.dims,
                     max_pos=min(max_context, 1 << 20))
-            self.layer_ropes.append(ropes[key])
-            self.kv_index.append(owners.index(i if l.mixer.kv_from is None else l.mixer.kv_from))
+            return ropes[key]
+
+        # (attention's, retention's) rotation of every layer
+        self.layer_ropes = [tuple(None if p is None else rope(p.rotary) for p in (l.attention, l.retention)) for l in cfg.layer_specs]
+        owners = [i for i, l in enumerate(cfg.layer_specs) if l.owns_rows]
+        self.kv_index = [-1 if l.attention is None else owners.index(i if l.attention.kv_from is None else l.attention.kv_from)
+                         for i, l in enumerate(cfg.layer_specs)]
+        stateful = [i for i, l in enumerate(cfg.layer_specs) if l.retention is not None]
+        self.state_index = {i: n for n, i in enumerate(stateful)}
         self.n_kv_layers, self.n_kv_local, self.kv_head_dim = len(owners), 1, cfg.head_dim
 
     def cache_spec(self, page_size: int, dtype_name: str):
-        """Shape of this model's paged cache: K / V rows of the attention layers, or latent rows (one plane; of each
-        layer's own width where the layers are listed one by one)."""
+        """Shape of this model's paged cache: K / V rows of the attention layers, or latent rows (one plane); of each
+        layer's own geometry where the layers are listed one by one."""
         from ..engine.kv_pool import KVCacheSpec
 
         layered = self.cfg.is_layered
         return KVCacheSpec(max(1, self.n_kv_layers), self.n_kv_local, self.kv_head_dim, page_size, dtype_name,
-                           planes=1 if layered else 2, row_dims=tuple(self.cfg.cache_rows) if layered else None)
+                           shapes=(tuple(self.cfg.cache_shapes) or ((1, 1, 16),)) if layered else None)
 
     def _fold_norm_weights(self) -> None:
         """Fold the two RMSNorm weight vectors of a dense bf16 layer into the columns of the projections that
@@ -289,10 +294,11 @@ class Transformer:
             w.swiglu_interleaved = True
 
     # ------------------------------------------------------------------ blocks
-    def new_cache(self, num_blocks: int, page_size: int, dtype_name: str):
+    def new_cache(self, num_blocks: int, page_size: int, dtype_name: str, state_slots: int = 0):
         """A paged cache shaped for this model: KV rows for the attention layers and, for a hybrid model, a second cache
-        (same pages, same block ids) whose rows are the convolution layers' gated inputs, split over its K and V halves."""
-        from ..engine.kv_pool import KVCache, KVCacheSpec
+        (same pages, same block ids) whose rows are the convolution layers' gated inputs, split over its K and V halves.
+        Listed layers with a recurrent state get ``state_slots`` slots beside it."""
+        from ..engine.kv_pool import KVCache, KVCacheSpec, StateStore
 
         kv = KVCache(self.cache_spec(page_size, dtype_name), num_blocks, self.device)
         if self.n_conv_layers:
@@ -301,6 +307,8 @@ class Transformer:
             plain = "bf16" if self.device.type == "cuda" else "f32"  # never quantized: the rows are convolved, not attended
             kv.conv = KVCache(KVCacheSpec(self.n_conv_layers, 1, self.cfg.hidden_size // 2, page_size, plain), num_blocks,
                               self.device)
+        if self.cfg.state_shapes:
+            kv.states = StateStore(self.cfg.state_shapes, state_slots, self.device)
         return kv
 
     def _ssm_slot(self, kv, first_block: int, position: int) -> int:
@@ -473,18 +481,56 @@ class Transformer:
             x, xa = h.float(), h.to(self.act_dtype)
         for li in range(lo, hi):
             lw, spec = self.w.layers[li], cfg.layer_specs[self.w.first_layer + li]
-            o = ops.latent_mixer(xa, lw.mla, spec.mixer, self.layer_ropes[li], meta, kv, self.kv_index[li], eps)
-            x, xa = ops.residual_norm(x, self.comm.linear_allreduce(o, lw.wo), alpha, lw.attn_norm, lw.attn_norm_bias, eps, kind,
-                                      self.act_dtype)
+            x, xa = ops.residual_norm(x, self._listed_mixer(li, lw, spec, xa, meta, kv), alpha, lw.attn_norm, lw.attn_norm_bias,
+                                      eps, kind, self.act_dtype)
             if spec.ffn is not None:
-                a = ops.linear_act(xa, lw.w_up, spec.ffn.act)
-                x, xa = ops.residual_norm(x, self.comm.linear_allreduce(a, lw.w_down), alpha, lw.ffn_norm, lw.ffn_norm_bias, eps,
-                                          kind, self.act_dtype)
-            if capture is not None and self.w.first_layer + li in capture.get("layers", ()):
-                capture.setdefault("hidden", {})[self.w.first_layer + li] = x.clone()
-            if _profiler.TRACE_FWD:
-                _profiler.trace_hidden(self.w.first_layer + li, x, None)
+                x, xa = ops.residual_norm(x, self._listed_ffn(lw, spec.ffn, xa), alpha, lw.ffn_norm, lw.ffn_norm_bias, eps, kind,
+                                          self.act_dtype)
+            self._layer_done(li, x, capture)
         return x, None
+
+    def _layers_sandwich(self, h: torch.Tensor, meta: BatchMeta, kv, lo: int, hi: int, capture: Optional[dict]):
+        """Layers with norms on both sides of every branch, x <- x + norm_b(branch(norm_a(x))), the stream ``x`` in float32.
+        One kernel ends a branch and starts the next: it norms the branch's output ``y`` (norm ``post``), adds it to the
+        stream and norms the sum for the branch that follows."""
+        cfg = self.cfg
+        eps = cfg.rms_eps
+        x, y, post = h.float(), None, None
+        want = set(capture.get("layers", ())) if capture is not None else set()
+        for li in range(lo, hi):
+            lw, spec = self.w.layers[li], cfg.layer_specs[self.w.first_layer + li]
+            x, xa = ops.branch_norm(x, y, post, lw.attn_norm, eps, self.act_dtype)
+            y, post = self._listed_mixer(li, lw, spec, xa, meta, kv), lw.post_attn_norm
+            if spec.ffn is not None:
+                x, xa = ops.branch_norm(x, y, post, lw.ffn_norm, eps, self.act_dtype)
+                y, post = self._listed_ffn(lw, spec.ffn, xa), lw.post_ffn_norm
+            if self.w.first_layer + li in want or _profiler.TRACE_FWD:
+                x, y = ops.branch_norm(x, y, post, None, eps, self.act_dtype)[0], None
+                self._layer_done(li, x, capture)
+        return (x if y is None else ops.branch_norm(x, y, post, None, eps, self.act_dtype)[0]), None
+
+    def _layer_done(self, li: int, x: torch.Tensor, capture: Optional[dict]) -> None:
+        gl = self.w.first_layer + li
+        if capture is not None and gl in capture.get("layers", ()):
+            capture.setdefault("hidden", {})[gl] = x.clone()
+        if _profiler.TRACE_FWD:
+            _profiler.trace_hidden(gl, x, None)
+
+    def _listed_mixer(self, li: int, lw: LayerWeights, spec, xa: torch.Tensor, meta: BatchMeta, kv) -> torch.Tensor:
+        """The mixer branch of a listed layer: from its normed input to its output projection."""
+        eps = self.cfg.rms_eps
+        if lw.mla is not None:
+            o = ops.latent_mixer(xa, lw.mla, spec.mixer, self.layer_ropes[li][0], meta, kv, self.kv_index[li], eps)
+        else:
+            o = ops.listed_mixer(xa, lw, spec, self.layer_ropes[li], meta, kv, self.kv_index[li], self.state_index.get(li, -1), eps)
+        return self.comm.linear_allreduce(o, lw.wo)
+
+    def _listed_ffn(self, lw: LayerWeights, f, xa: torch.Tensor) -> torch.Tensor:
+        if isinstance(f, MoESpec):
+            return ops.moe_ffn(xa, lw, f)
+        if f.gated:
+            return ops.gated_ffn(xa, lw.w_gate_up, lw.w_down)
+        return self.comm.linear_allreduce(ops.linear_act(xa, lw.w_up, f.act), lw.w_down)
 
     def final_norm(self, h: torch.Tensor, residual: Optional[torch.Tensor]):
         """(normed rows for the output head, the hidden state in front of that norm)."""
@@ -623,7 +669,8 @@ class Transformer:
         cfg = self.cfg
         lo, hi = layers if layers is not None else (0, len(self.w.layers))
         if cfg.is_layered:
-            return self._layers_norm_after(h, meta, kv, lo, hi, capture)
+            layers_fn = self._layers_sandwich if cfg.norm_placement == "sandwich" else self._layers_norm_after
+            return layers_fn(h, meta, kv, lo, hi, capture)
         acc, cur = None, 0  # per-token sum-of-squares accumulators of the residual stream while it is in folded form
         for li in range(lo, hi):
             lw = self.w.layers[li]

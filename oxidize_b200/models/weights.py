@@ -223,6 +223,9 @@ class LayerWeights:
     q_norm: Optional[torch.Tensor] = None
     k_norm: Optional[torch.Tensor] = None
     mla: Optional[MLAWeights] = None
+    # listed layers: per-head logits of the attention's softmax denominator.  ``wqkv`` then holds every projection of the
+    # layer's input (attention q | k | v, retention q | k | v | gate) and ``wo`` the output projections side by side
+    sink: Optional[torch.Tensor] = None
     # short-convolution mixer (LFM2) instead of attention: in_proj [3 hidden, hidden] (rows: B, C, x), depthwise kernel
     # [hidden, l_cache] (oldest tap first), out_proj [hidden, hidden]
     conv_in: Optional[QTensor] = None

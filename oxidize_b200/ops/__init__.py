@@ -27,6 +27,12 @@ def _cuda_latent():
     return _c
 
 
+def _cuda_listed():
+    from . import cuda_listed as _c
+
+    return _c
+
+
 @instrument("linear")
 def linear(x: torch.Tensor, w, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y = x @ W^T (+bias) for a :class:`LinearWeight` (row segments concatenated) or a QTensor."""
@@ -80,6 +86,63 @@ def gelu_mul(gate_up):
     if gate_up.is_cuda:
         return _cuda().gelu_mul(gate_up)
     return ref.gelu_mul(gate_up)
+
+
+@instrument("branch_norm")
+def branch_norm(res, y, w_post, w_next, eps, act_dtype=torch.float32):
+    """Norms on both sides of a branch: x = res + rmsnorm(y) * w_post (float32; ``y`` None: x = res) and the next branch's
+    input rmsnorm(x) * w_next in ``act_dtype`` (None without ``w_next``)."""
+    if res.is_cuda:
+        return _cuda_listed().branch_norm(res, y, w_post, w_next, eps, act_dtype)
+    return ref.branch_norm(res, y, w_post, w_next, eps, act_dtype)
+
+
+@instrument("listed_mixer")
+def listed_mixer(x, lw, spec, ropes, meta, kv, kv_layer, state_layer, eps):
+    """Attention and / or retention of one listed layer on its normed input, up to (not including) the output projection:
+    [T, spec.out_dim], attention heads first.  ``ropes``: rotations of the two; in a layer with both, each side's output
+    carries its scale."""
+    if x.is_cuda:
+        return _cuda_listed().listed_mixer(x, lw, spec, ropes, meta, kv, kv_layer, state_layer, eps)
+    z = linear(x, lw.wqkv)
+    a, r, outs = spec.attention, spec.retention, []
+    sl, sr = spec.branch_scales
+    if a is not None:
+        q = ref.head_prep(z[:, : a.proj_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps)
+        o = ref.paged_attention(q, kv, kv_layer, meta, a.scale, a.window, sink=lw.sink)
+        outs.append(o.reshape(x.shape[0], -1) * sl)
+    if r is not None:
+        zr = z[:, 0 if a is None else a.proj_dim :]
+        outs.append((ref.retention(zr, r, ropes[1], meta, kv.states.data[state_layer], eps) * sr).to(x.dtype))
+    return torch.cat(outs, dim=-1)
+
+
+@instrument("gated_ffn")
+def gated_ffn(x, gate_up, down):
+    """W_down (silu(W_gate x) * (W_up x)) with gate | up as one matrix."""
+    if x.is_cuda:
+        return _cuda_listed().gated_ffn(x, gate_up, down)
+    return linear(silu_mul(linear(x, gate_up)), down)
+
+
+@instrument("moe_ffn")
+def moe_ffn(x, lw, spec):
+    """Routed experts (``spec``: ``models.config.MoESpec``) with float32 router logits, plus the shared expert."""
+    if x.is_cuda:
+        return _cuda_listed().moe_ffn(x, lw, spec)
+    ids, wts = ref.moe_route(linear(x.float(), lw.router), spec)
+    ex, H = lw.experts, x.shape[1]
+    xp = torch.nn.functional.pad(x, (0, ex.gate_up[0].shape[1] - H))
+    out = torch.zeros(x.shape[0], ex.down[0].shape[0], dtype=torch.float32)
+    for e in range(spec.n_experts):
+        rows, slot = (ids == e).nonzero(as_tuple=True)
+        if rows.numel():
+            y = gated_ffn(xp[rows], ex.gate_up[e], ex.down[e]).float()
+            out.index_add_(0, rows, y * wts[rows, slot][:, None])
+    out = out[:, :H]
+    if lw.shared_gate_up is not None:
+        out = out + gated_ffn(x, lw.shared_gate_up, lw.shared_down).float()
+    return out.to(x.dtype)
 
 
 @instrument("qk_rope_kv_write")

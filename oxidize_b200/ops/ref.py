@@ -89,6 +89,14 @@ def residual_norm(res: Optional[torch.Tensor], y: Optional[torch.Tensor], alpha:
     return z, z.to(act_dtype)
 
 
+def branch_norm(res: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torch.Tensor], w_next: Optional[torch.Tensor],
+                eps: float, act_dtype: torch.dtype = torch.float32):
+    """Norms on both sides of a branch: x = res + rmsnorm(y) * w_post in float32 and the next branch's input
+    rmsnorm(x) * w_next in ``act_dtype``; (x, None) without ``w_next``."""
+    x = res.float() if y is None else res.float() + rmsnorm(y.float(), w_post, eps)
+    return x, None if w_next is None else rmsnorm(x, w_next, eps).to(act_dtype)
+
+
 def activation(x: torch.Tensor, act: str) -> torch.Tensor:
     """Elementwise activation of a feed-forward block without a gate: ``relu2`` is the square of relu."""
     if act == "relu2":
@@ -225,13 +233,14 @@ def kv_gather(kv, layer: int, block_table: torch.Tensor, seq_len: int) -> Tuple[
 
 
 def paged_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, sliding_window: int = 0,
-                    softcap: float = 0.0) -> torch.Tensor:
+                    softcap: float = 0.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal GQA attention of packed query rows against the paged cache.
 
     q: [T, n_heads, hd].  For sequence b the rows ``query_start[b]:query_start[b+1]`` are its
     last ``qlen`` positions (context length ``seq_lens[b]`` already includes them), so one
     code path covers decode (qlen 1), chunked prefill and speculative verify (qlen K+1).
-    ``softcap`` > 0 replaces the scaled scores by ``softcap * tanh(scores / softcap)`` before masking (Gemma-2)."""
+    ``softcap`` > 0 replaces the scaled scores by ``softcap * tanh(scores / softcap)`` before masking (Gemma-2);
+    ``sink`` [heads] is a logit that joins the softmax denominator only."""
     T, nh, hd = q.shape
     out = torch.zeros(T, nh, hd, dtype=torch.float32, device=q.device)
     qs = meta.query_start.tolist()
@@ -255,7 +264,7 @@ def paged_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, sliding
         if sliding_window > 0:
             mask &= kpos > qpos - sliding_window
         s = s.masked_fill(~mask, float("-inf"))
-        p = torch.softmax(s, dim=-1)
+        p = softmax_sink(s, None if sink is None else sink.reshape(nkv, g, 1, 1))
         o = torch.einsum("kgql,lkd->qkgd", p, V)
         out[t0:t1] = o.reshape(qlen, nh, hd)
     return out.to(q.dtype)
@@ -338,6 +347,55 @@ def latent_attention(q: torch.Tensor, kv, layer: int, meta, scale: float, latent
         p = softmax_sink(s, None if sink is None else sink[:, None, None])
         out[t0:t1] = torch.einsum("hql,lc->qhc", p, K[:, :latent_dim])
     return out.to(q.dtype)
+
+
+# --------------------------------------------------------------------------- listed mixers
+
+
+def padded_norm(x: torch.Tensor, w: torch.Tensor, n: int, eps: float) -> torch.Tensor:
+    """RMS norm over the last axis of zero-padded rows that hold ``n`` values."""
+    return x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / n + eps) * w
+
+
+def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int, eps: float) -> torch.Tensor:
+    """From a layer's q | k | v projections (heads of ``spec.width`` values): norms, rotation, this step's cache rows; the
+    queries [T, heads, width]."""
+    T, H, G, W = z.shape[0], spec.heads, spec.kv_heads, spec.width
+    q, k, v = z[:, : H * W].float(), z[:, H * W : (H + G) * W].float(), z[:, (H + G) * W : (H + 2 * G) * W]
+    if spec.qk_norm == "full":
+        q, k = padded_norm(q, q_norm, H * spec.dim, eps), padded_norm(k, k_norm, G * spec.dim, eps)
+    q, k = q.reshape(T, H, W), k.reshape(T, G, W)
+    if spec.qk_norm == "head":
+        q, k = padded_norm(q, q_norm, spec.dim, eps), padded_norm(k, k_norm, spec.dim, eps)
+    q = apply_rope(q, meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
+    k = apply_rope(k, meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
+    kv_write(kv, layer, k, v.reshape(T, G, W), meta.slot_mapping)
+    return q.to(z.dtype)
+
+
+def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, eps: float) -> torch.Tensor:
+    """Retention of one layer, token by token: z [T, q | k | v | gate], state [slots, heads, k_width, v_width] (updated);
+    a sequence whose rows start at position 0 starts from a zero state.  Returns [T, heads * v_width]."""
+    T, H, K, V = z.shape[0], spec.heads, spec.k_width, spec.v_width
+    z = z.float()
+    q, k = z[:, : H * K].reshape(T, H, K), z[:, H * K : 2 * H * K].reshape(T, H, K)
+    v, g = z[:, 2 * H * K : 2 * H * K + H * V].reshape(T, H, V), z[:, 2 * H * K + H * V :].reshape(T, H, V)
+    q = apply_rope(q, meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
+    k = apply_rope(k, meta.positions, rope.inv_freq, rope.pairing, rope.mscale) * spec.dim ** -0.5
+    decay = torch.tensor(spec.decay, dtype=torch.float32, device=z.device)[:, None, None]
+    o = torch.zeros(T, H, V, dtype=torch.float32, device=z.device)
+    qs, lens, slots = meta.query_start.tolist(), meta.seq_lens.tolist(), meta.state_slots.tolist()
+    for b in range(len(lens)):
+        t0, t1 = qs[b], qs[b + 1]
+        if slots[b] < 0 or t1 == t0:
+            continue
+        S = torch.zeros_like(state[slots[b]]) if lens[b] == t1 - t0 else state[slots[b]]
+        for t in range(t0, t1):
+            S = decay * S + k[t][:, :, None] * v[t][:, None, :]
+            o[t] = (S * q[t][:, :, None]).sum(1)
+        state[slots[b]] = S
+    y = padded_norm(o, 1.0, spec.v_dim, eps) * torch.nn.functional.silu(g)
+    return y.reshape(T, H * V)
 
 
 # --------------------------------------------------------------------------- MoE routing

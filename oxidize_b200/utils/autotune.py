@@ -16,7 +16,7 @@ from dataclasses import asdict, dataclass, field
 from typing import Any, Dict, List, Optional
 
 from ..formats.layered import Checkpoint
-from ..models.config import ModelConfig
+from ..models.config import LatentAttentionSpec, ModelConfig
 from ..models.registry import config_from_checkpoint
 
 B200_HBM_GBS = 6555.0  # sustained copy bandwidth of a B200 (HBM3e), GB/s: the bound the decode estimates use
@@ -99,8 +99,8 @@ def fingerprint(g: Checkpoint, cfg: Optional[ModelConfig] = None) -> ModelFinger
     dom = max(by_type, key=by_type.get) if by_type else "F32"
     # what one token's cache row holds: KV heads x head_dim, or with latent attention one shared (latent + rotary key) row
     kv_heads, kv_dim = (1, cfg.kv_lora_rank + cfg.rotary_dim) if cfg.is_mla else (cfg.n_kv_heads, cfg.head_dim)
-    if cfg.is_layered:  # one latent row in each layer that owns rows: spread over the layers' notional key / value pairs
-        kv_heads, kv_dim = 1, max(1, -(-sum(cfg.cache_rows) // (2 * cfg.n_layers)))
+    if cfg.is_layered:  # rows of different widths in the layers that own some: spread over notional key / value pairs
+        kv_heads, kv_dim = 1, max(1, -(-sum(h * p * d for h, p, d in cfg.cache_shapes) // (2 * cfg.n_layers)))
     return ModelFingerprint(cfg.arch, cfg.n_layers, cfg.hidden_size, cfg.n_heads, kv_heads, kv_dim,
                             cfg.is_moe, cfg.n_experts, total, cfg.context_length, cfg.nextn_layers > 0, dom)
 
@@ -241,8 +241,12 @@ def prefill_token_budget(cfg: ModelConfig, tp: int = 1, sm_count: int = 148, lo:
         (h, max(ffn // tp, 1)),
     ]
     if cfg.is_layered:
-        m, f = cfg.layer_specs[0].mixer, cfg.ffn_size
-        shapes = [(m.heads * m.qk_dim // tp + m.kv_rank + m.rope_dim, h), (h, m.heads * m.v_dim // tp)]
+        l, f = cfg.layer_specs[0], cfg.ffn_size
+        m = l.mixer
+        if isinstance(m, LatentAttentionSpec):
+            shapes = [(m.heads * m.qk_dim // tp + m.kv_rank + m.rope_dim, h), (h, m.heads * m.v_dim // tp)]
+        else:
+            shapes = [(sum(p.proj_dim for p in (l.attention, l.retention) if p is not None) // tp, h), (h, l.out_dim // tp)]
         shapes += [(f // tp, h), (h, f // tp)] if f >= tp else []
     best, best_eff = lo, -1.0
     t = (lo + token_tile - 1) // token_tile * token_tile

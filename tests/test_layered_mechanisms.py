@@ -301,8 +301,8 @@ def test_heads_and_feed_forward_are_sharded_over_ranks(tmp_path):
     def branch(rank, size):
         w = load_checkpoint_weights(ck, mc, tp_rank=rank, tp_size=size)
         lw, spec = w.layers[0], mc.layer_specs[0]
-        kv = KVCache(KVCacheSpec(1, 1, 32, 16, "f32", planes=1, row_dims=(32,)), 2, "cpu")
-        rope = Transformer(load_checkpoint_weights(ck, mc), max_context=64).layer_ropes[0]
+        kv = KVCache(KVCacheSpec(1, 1, 32, 16, "f32", planes=1, shapes=((1, 1, 32),)), 2, "cpu")
+        rope = Transformer(load_checkpoint_weights(ck, mc), max_context=64).layer_ropes[0][0]
         a = ops.linear(ops.latent_mixer(x, lw.mla, spec.mixer, rope, meta, kv, 0, mc.rms_eps), lw.wo)
         return a, ops.linear(ops.linear_act(x, lw.w_up, "relu2"), lw.w_down)
 
