@@ -24,7 +24,7 @@ constexpr int ATT_STAGES = 3;
 
 struct AttnArgs {
   const __nv_bfloat16* q;   // [T, nq, hd]
-  __nv_bfloat16* out;       // [T, nq, hd]
+  __nv_bfloat16* out;       // [T, nq, hd], rows ld_out apart
   const void* kv_data;      // layer base
   const float* kv_scales;   // layer base (q8/q4) or null
   const int* block_tables;  // [B, max_blocks]
@@ -37,6 +37,9 @@ struct AttnArgs {
   // soft-capped scores (Gemma-2): score = cap * tanh(q.k * scale / cap).  cap_log2 = cap * log2(e) (0 = off),
   // cap_arg = scale / cap
   float cap_log2, cap_arg;
+  const float* sink;  // [nq] logits that join the softmax denominator only, or null
+  int ld_out;         // values between the output rows of neighbouring tokens
+  float out_scale;    // factor on the outputs
   float* ws_o;   // [B*nkv*max_mtiles*n_cta_splits, 16, hd]
   float* ws_ml;  // [.., 16, 2]
   int* counters; // [B*nkv*max_mtiles] zero-initialised tickets (CTA splits only)
@@ -154,7 +157,9 @@ __device__ __forceinline__ void attn_merge_rows(const AttnArgs& a, int G, int b,
   const size_t task0 = ((size_t)b * a.nkv + kvh) * gx + (size_t)mtile * a.n_cta_splits;
   float M = -INFINITY;
   for (int s = 0; s < a.n_cta_splits; ++s) M = fmaxf(M, __ldcg(a.ws_ml + ((task0 + s) * 16 + row) * 2));
-  float L = 0.f;
+  const float sink = a.sink != nullptr ? a.sink[kvh * G + r % G] * 1.4426950408889634f : -INFINITY;
+  M = fmaxf(M, sink);
+  float L = sink == -INFINITY ? 0.f : exp2f(sink - M);
   float acc[HD / 8];
 #pragma unroll
   for (int d = 0; d < HD / 8; ++d) acc[d] = 0.f;
@@ -172,8 +177,8 @@ __device__ __forceinline__ void attn_merge_rows(const AttnArgs& a, int G, int b,
       acc[4 * d + 3] += w * v.w;
     }
   }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
-  __nv_bfloat16* dst = a.out + ((size_t)(q0 + r / G) * a.nq + kvh * G + r % G) * HD + seg;
+  const float inv = L > 0.f ? a.out_scale / L : 0.f;
+  __nv_bfloat16* dst = a.out + (size_t)(q0 + r / G) * a.ld_out + (kvh * G + r % G) * HD + seg;
 #pragma unroll
   for (int d = 0; d < HD / 8; d += 2) *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(acc[d] * inv, acc[d + 1] * inv);
 }
@@ -413,6 +418,11 @@ paged_attention_kernel(const AttnArgs a, int G /*q heads per kv head*/) {
     if (valid) {
 #pragma unroll
       for (int w = 0; w < ATT_WARPS; ++w) M = fmaxf(M, mml[(w * 16 + row) * 2]);
+      if (a.sink != nullptr && a.n_cta_splits == 1) {  // (CTA splits: joined once, where they merge)
+        const float sink = a.sink[kvh * G + r % G] * 1.4426950408889634f;
+        M = fmaxf(M, sink);
+        L = exp2f(sink - M);
+      }
 #pragma unroll
       for (int w = 0; w < ATT_WARPS; ++w) {
         const float mw = mml[(w * 16 + row) * 2];
@@ -422,8 +432,8 @@ paged_attention_kernel(const AttnArgs a, int G /*q heads per kv head*/) {
     }
     if (a.n_cta_splits == 1) {
       if (valid) {
-        const float inv = L > 0.f ? 1.f / L : 0.f;
-        __nv_bfloat16* dst = a.out + ((size_t)(q0 + r / G) * a.nq + kvh * G + r % G) * HD + seg;
+        const float inv = L > 0.f ? a.out_scale / L : 0.f;
+        __nv_bfloat16* dst = a.out + (size_t)(q0 + r / G) * a.ld_out + (kvh * G + r % G) * HD + seg;
         for (int d = 0; d < HD / 8; d += 2) {
           float v0 = 0.f, v1 = 0.f;
 #pragma unroll

@@ -14,6 +14,8 @@ struct GemmF32Args {
   int T, N, K, ldx, ldw, ldy;
   long long xs, ws, ys;  // strides of a group
   int act;               // 0 none, 1 square of relu
+  // routed groups: group g multiplies rows [offsets[g], offsets[g + 1]) of Y; row r of Y reads row perm[r] of X (perm null: r)
+  const int *offsets, *perm;
 };
 
 static __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Args a) {
@@ -21,17 +23,26 @@ static __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Args 
   pdl_launch_dependents();
   pdl_wait();
   const int tid = threadIdx.x;
+  const int g0 = a.offsets != nullptr ? a.offsets[blockIdx.z] : 0;
+  const int T = a.offsets != nullptr ? a.offsets[blockIdx.z + 1] : a.T;  // rows end here
   const float* X = a.x + (size_t)blockIdx.z * a.xs;
   const float* W = a.w + (size_t)blockIdx.z * a.ws;
   float* Y = a.y + (size_t)blockIdx.z * a.ys;
-  const int t0 = blockIdx.y * F32_TILE, n0 = blockIdx.x * F32_TILE;
+  const int t0 = g0 + blockIdx.y * F32_TILE, n0 = blockIdx.x * F32_TILE;
+  if (t0 >= T) return;
   const int lr = tid >> 4, lk = tid & 15;  // loads: 16 rows x 16 k per pass, 4 passes
   float rx[4], rw[4];
+  size_t xrow[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = t0 + lr + 16 * i;
+    xrow[i] = t < T ? (a.perm != nullptr ? a.perm[t] : t) : 0;
+  }
   auto fetch = [&](int k0) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int r = lr + 16 * i, k = k0 + lk;
-      rx[i] = (t0 + r < a.T && k < a.K) ? X[(size_t)(t0 + r) * a.ldx + k] : 0.f;
+      rx[i] = (t0 + r < T && k < a.K) ? X[xrow[i] * a.ldx + k] : 0.f;
       rw[i] = (n0 + r < a.N && k < a.K) ? W[(size_t)(n0 + r) * a.ldw + k] : 0.f;
     }
   };
@@ -67,7 +78,7 @@ static __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Args 
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    if (t0 + tr + i >= a.T) break;
+    if (t0 + tr + i >= T) break;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tc + j;

@@ -1,8 +1,13 @@
-// Latent attention for long portions of a prompt: keys and values are expanded per head (one matrix product over the
-// sequence's visible rows), and ordinary flash attention runs on them with tcgen05.  Against the absorbed form
+// Attention for long portions of a prompt: flash attention with tcgen05 over dense rows of per-head keys and values.
+//
+// Latent attention: keys and values are expanded per head (one matrix product over the sequence's visible rows).  Against the absorbed form
 // (latent_mma.cuh) this trades (2 rank + rot) products per query, key and head for (nope + rot + v).
 //
-// latent_gather_kernel copies the visible rows out of the pages into dense [rows, latent] and [rows, rot] matrices; the
+// Grouped-query attention: the visible rows' keys and values are gathered as they are, `group` query heads share a key head,
+// and there is no separate rotated part.
+//
+// latent_gather_kernel / kv_gather_kernel copy the visible rows out of the pages into dense matrices ([rows, latent] and [rows, rot], or
+// [rows, keys of all heads | values of all heads]); the
 // expansion is the library's GEMM; latent_prefill_kernel attends.  A CTA owns one head and 256 query tokens of a sequence as
 // two tiles of 128 rows: S = Q K^T (M = 128 tokens, N = 64 keys) goes to tensor memory, a warpgroup per tile does the softmax
 // with one thread per row and writes P back to tensor memory as the A operand of O += P V (V read MN-major).  The two tiles
@@ -41,6 +46,36 @@ latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restr
   for (int i = lane; i < p8 + r8; i += 32) (i < p8 ? l[i] : r[i - p8]) = src[i];
 }
 
+// dense copies of the K / V pages' rows [span_lo[b], ...) of every sequence: out [rows, K of all heads | V of all heads]
+static __global__ void __launch_bounds__(128)
+kv_gather_kernel(const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_tables, const int* __restrict__ span_lo,
+                 const int* __restrict__ span_off, int B, int max_blocks, int heads, int width, int page, int num_blocks,
+                 __nv_bfloat16* __restrict__ out) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= span_off[B]) return;
+  int b = 0, hi = B - 1;
+  while (b < hi) {
+    const int mid = (b + hi + 1) >> 1;
+    if (span_off[mid] <= row) b = mid;
+    else hi = mid - 1;
+  }
+  const int pos = span_lo[b] + row - span_off[b];
+  int blk = block_tables[(size_t)b * max_blocks + pos / page];
+  if ((unsigned)blk >= (unsigned)num_blocks) {
+    if (lane == 0) oxb_report(OXB_BAD_BLOCK_ID, blk);
+    blk = 0;
+  }
+  const int w8 = width / 8, n = 2 * heads * w8;
+  const uint4* src = reinterpret_cast<const uint4*>(cache) + ((size_t)blk * 2 * heads * page + pos % page) * w8;
+  uint4* dst = reinterpret_cast<uint4*>(out) + (size_t)row * n;
+  for (int i = lane; i < n; i += 32) {
+    const int head = i / w8, plane = head >= heads;  // (pages are [heads][K, V][page][width])
+    dst[i] = src[(size_t)((head - plane * heads) * 2 + plane) * page * w8 + i % w8];
+  }
+}
+
 constexpr int LP_KEYS = 64;       // keys per tile
 constexpr int LP_M = 128;         // query tokens per tile, two tiles per CTA
 constexpr int LP_QCHUNK = LP_M * 128, LP_KCHUNK = LP_KEYS * 128;  // bytes of a 64-value column chunk
@@ -53,8 +88,10 @@ struct LatentPrefillArgs {
   const int* span_lo;       // [B] first position of the dense rows
   const int* span_off;      // [B + 1] first dense row of every sequence
   const float* sink;        // [H] or null
-  __nv_bfloat16* out;       // [T, H * v]
-  int H, window;
+  __nv_bfloat16* out;       // [T, H * v], rows ld_out apart
+  int H, window, group;     // group: query heads per key head
+  int ld_out;
+  float out_scale;
   int nope16, rot16, full_ld;  // k-steps of 16 values of the two key parts; values per head of a query row
   int nope_ld, v_off, v_ld, v; // expanded row: head h's key at h * nope_ld, its value at v_off + h * v_ld
   float scale_log2;
@@ -157,7 +194,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       if (leader) {
         mbar_expect_tx(&k_full[s], q_ch * LP_KCHUNK);
         uint8_t* d = s_k + s * q_ch * LP_KCHUNK;
-        for (int c = 0; c < nope_ch; ++c) tma_load_2d(d + c * LP_KCHUNK, &tmKV, &k_full[s], h * a.nope_ld + c * 64, row);
+        for (int c = 0; c < nope_ch; ++c) tma_load_2d(d + c * LP_KCHUNK, &tmKV, &k_full[s], (h / a.group) * a.nope_ld + c * 64, row);
         for (int c = 0; c < rot_ch; ++c) tma_load_2d(d + (nope_ch + c) * LP_KCHUNK, &tmR, &k_full[s], c * 64, row);
       }
       if (i > 1) ok = mbar_wait_bounded(&v_empty[s], ((i >> 1) - 1) & 1, &abort_flag, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
@@ -166,7 +203,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       if (leader) {
         mbar_expect_tx(&v_full[s], v_ch * LP_KCHUNK);
         for (int c = 0; c < v_ch; ++c)
-          tma_load_2d(s_v + (s * v_ch + c) * LP_KCHUNK, &tmKV, &v_full[s], a.v_off + h * a.v_ld + c * 64, row);
+          tma_load_2d(s_v + (s * v_ch + c) * LP_KCHUNK, &tmKV, &v_full[s], a.v_off + (h / a.group) * a.v_ld + c * 64, row);
       }
       __syncwarp();
     }
@@ -293,14 +330,14 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     __syncwarp();
     tc_fence_after();
     if (sink > -INFINITY) l += exp2f(sink - m);  // the sink's share of the denominator, once
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    __nv_bfloat16* o_row = a.out + ((size_t)(q0 + r) * a.H + h) * a.v;
+    const float inv = l > 0.f ? a.out_scale / l : 0.f;
+    __nv_bfloat16* o_row = a.out + (size_t)(q0 + r) * a.ld_out + h * a.v;
     for (int c = 0; c < v16; ++c) {
       uint32_t o[16];
       tmem_ld16(o_col + 16 * c, o);
       tmem_ld_wait();
       if (r < qlen) {
-        if (a.v % 8 == 0) {
+        if ((a.v | a.ld_out) % 8 == 0) {
 #pragma unroll
           for (int j = 0; j < 16; j += 8) {
             uint32_t w[4];

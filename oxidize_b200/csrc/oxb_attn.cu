@@ -16,7 +16,7 @@ OXB_API int oxb_attn_ws_floats(int B, int nkv, int max_mtiles, int n_cta_splits,
 template <int HD>
 static int attn_launch(const AttnArgs& a, int B, int G, cudaStream_t stream) {
   constexpr int STAGE = 32 * (HD * 2 + 16);
-  constexpr int SMEM_MAX = ATT_WARPS * (ATT_STAGES + 1) * STAGE;
+  constexpr int SMEM_MAX = ATT_WARPS * (ATT_STAGES + (HD <= 128 ? 1 : 0)) * STAGE;
   // quantized KV needs one extra decode buffer per warp
   const int smem = ATT_WARPS * (ATT_STAGES + (a.kv_mode >= 2 ? 1 : 0)) * STAGE;
   static bool configured = false;
@@ -37,8 +37,9 @@ static int attn_launch(const AttnArgs& a, int B, int G, cudaStream_t stream) {
 OXB_API int oxb_paged_attention(const void* q, void* out, const void* kv_data, const float* kv_scales,
                                 const int* block_tables, const int* seq_lens, const int* query_start, int B,
                                 int max_blocks, int nq, int nkv, int hd, int kv_mode, int max_query_len,
-                                int n_cta_splits, int window, float scale, float softcap, float* ws_o, float* ws_ml,
-                                int* counters, int num_blocks, cudaStream_t stream) {
+                                int n_cta_splits, int window, float scale, float softcap, const float* sink, int ld_out,
+                                float out_scale, float* ws_o, float* ws_ml, int* counters, int num_blocks,
+                                cudaStream_t stream) {
   if (B <= 0) return 0;
   if (nq % nkv != 0) return (int)cudaErrorInvalidValue;
   const int G = nq / nkv;
@@ -60,6 +61,9 @@ OXB_API int oxb_paged_attention(const void* q, void* out, const void* kv_data, c
   a.scale_log2 = scale * 1.4426950408889634f;
   a.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   a.cap_arg = softcap > 0.f ? scale / softcap : 0.f;
+  a.sink = sink;
+  a.ld_out = ld_out;
+  a.out_scale = out_scale;
   a.ws_o = ws_o;
   a.ws_ml = ws_ml;
   a.counters = counters;
@@ -67,6 +71,11 @@ OXB_API int oxb_paged_attention(const void* q, void* out, const void* kv_data, c
   a.trace = g_oxb_attn_trace;
   if (hd == 128) return attn_launch<128>(a, B, G, stream);
   if (hd == 64) return attn_launch<64>(a, B, G, stream);
+  if (kv_mode != 0) return (int)cudaErrorInvalidValue;
+  if (hd == 32) return attn_launch<32>(a, B, G, stream);
+  if (hd == 96) return attn_launch<96>(a, B, G, stream);
+  if (hd == 192) return attn_launch<192>(a, B, G, stream);
+  if (hd == 256) return attn_launch<256>(a, B, G, stream);
   return (int)cudaErrorInvalidValue;
 }
 

@@ -19,8 +19,20 @@ OXB_API int oxb_residual_norm(const float* res, const void* y, float alpha, cons
 OXB_API int oxb_gemm_f32(const float* x, const float* w, float* y, const float* bias, int T, int N, int K, int ldx, int ldw,
                          int ldy, int groups, long long xs, long long ws, long long ys, int act, cudaStream_t stream) {
   if (T <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
-  const GemmF32Args a{x, w, bias, y, T, N, K, ldx, ldw, ldy, xs, ws, ys, act};
+  const GemmF32Args a{x, w, bias, y, T, N, K, ldx, ldw, ldy, xs, ws, ys, act, nullptr, nullptr};
   oxb_launch(gemm_f32_kernel, dim3((N + F32_TILE - 1) / F32_TILE, (T + F32_TILE - 1) / F32_TILE, groups), dim3(256), 0, stream, a);
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+// Routed groups: y[r] = x[perm[r]] . W_g^T for the rows r of every group g (offsets [groups + 1], perm null: x[r]);
+// max_rows bounds the rows of one group.
+OXB_API int oxb_gemm_f32_rows(const float* x, const float* w, float* y, const int* offsets, const int* perm, int groups,
+                              int max_rows, int N, int K, int ldx, int ldy, cudaStream_t stream) {
+  if (max_rows <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
+  const GemmF32Args a{x, w, nullptr, y, 0, N, K, ldx, K, ldy, 0, (long long)N * K, 0, 0, offsets, perm};
+  oxb_launch(gemm_f32_kernel, dim3((N + F32_TILE - 1) / F32_TILE, (max_rows + F32_TILE - 1) / F32_TILE, groups), dim3(256), 0,
+             stream, a);
   OXB_CHECK_LAUNCH();
   return 0;
 }
@@ -162,6 +174,32 @@ OXB_API int oxb_latent_gather(const void* cache, const int* block_tables, const 
 // 1 when latent_prefill_kernel covers heads of these sizes
 OXB_API int oxb_latent_prefill_supported(int nope, int rot, int v) { return latent_prefill_plan(nope, rot, v).smem > 0; }
 
+static int prefill_launch(LatentPrefillArgs a, const void* q, const void* kv, const void* rot_rows, int B, int T, int rows, int kv_ld,
+                          int max_query_len, const LatentPrefillPlan& pl, cudaStream_t stream) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
+  if (!configured[dev]) {
+    const cudaError_t ce = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LM_DYN_SMEM);
+    if (ce != cudaSuccess) return (int)ce;
+    configured[dev] = true;
+  }
+  CUtensorMap tq, tkv, tr;
+  int e = oxb_make_tmap_2d(&tq, q, T, (uint64_t)a.H * a.full_ld, (uint64_t)a.H * a.full_ld * 2, LP_M, 64, 2);
+  if (e) return e;
+  e = oxb_make_tmap_2d(&tkv, kv, rows, kv_ld, (uint64_t)kv_ld * 2, LP_KEYS, 64, 2);
+  if (e) return e;
+  tr = tkv;  // (never read without a rotated part)
+  if (a.rot16 > 0) e = oxb_make_tmap_2d(&tr, rot_rows, rows, 16 * a.rot16, (uint64_t)a.rot16 * 32, LP_KEYS, 64, 2);
+  if (e) return e;
+  const dim3 grid((max_query_len + 2 * LP_M - 1) / (2 * LP_M), a.H, B);
+  const cudaError_t le = oxb_launch(latent_prefill_kernel, grid, dim3(LP_THREADS), (size_t)pl.smem, stream, tq, tkv, tr, a);
+  if (le != cudaSuccess) return (int)le;
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
 // Attention of long portions over expanded keys and values: q [T, H, full_ld] (nope | rotated part, each padded with zeros
 // to a multiple of 16), kv [rows, kv_ld] (head h's key at h * nope_ld, its value at v_off + h * v_ld, all multiples of 8),
 // rot [rows, rot padded to 16]; out [T, H * v].
@@ -173,15 +211,6 @@ OXB_API int oxb_latent_prefill(const void* q, const void* kv, const void* rot_ro
   const LatentPrefillPlan pl = latent_prefill_plan(nope, rot, v);
   if (pl.smem == 0 || kv_ld % 8 != 0 || nope_ld % 8 != 0 || v_off % 8 != 0 || v_ld % 8 != 0 || H > 65535 || B > 65535)
     return (int)cudaErrorInvalidValue;
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
-  if (!configured[dev]) {
-    const cudaError_t ce = cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LM_DYN_SMEM);
-    if (ce != cudaSuccess) return (int)ce;
-    configured[dev] = true;
-  }
   LatentPrefillArgs a;
   a.query_start = query_start;
   a.seq_lens = seq_lens;
@@ -191,6 +220,9 @@ OXB_API int oxb_latent_prefill(const void* q, const void* kv, const void* rot_ro
   a.out = reinterpret_cast<__nv_bfloat16*>(out);
   a.H = H;
   a.window = window;
+  a.group = 1;
+  a.ld_out = H * v;
+  a.out_scale = 1.f;
   a.nope16 = (nope + 15) / 16;
   a.rot16 = (rot + 15) / 16;
   a.full_ld = 16 * (a.nope16 + a.rot16);
@@ -199,16 +231,48 @@ OXB_API int oxb_latent_prefill(const void* q, const void* kv, const void* rot_ro
   a.v_ld = v_ld;
   a.v = v;
   a.scale_log2 = scale * 1.4426950408889634f;
-  CUtensorMap tq, tkv, tr;
-  int e = oxb_make_tmap_2d(&tq, q, T, (uint64_t)H * a.full_ld, (uint64_t)H * a.full_ld * 2, LP_M, 64, 2);
-  if (e) return e;
-  e = oxb_make_tmap_2d(&tkv, kv, rows, kv_ld, (uint64_t)kv_ld * 2, LP_KEYS, 64, 2);
-  if (e) return e;
-  e = oxb_make_tmap_2d(&tr, rot_rows, rows, 16 * a.rot16, (uint64_t)a.rot16 * 32, LP_KEYS, 64, 2);
-  if (e) return e;
-  const dim3 grid((max_query_len + 2 * LP_M - 1) / (2 * LP_M), H, B);
-  const cudaError_t le = oxb_launch(latent_prefill_kernel, grid, dim3(LP_THREADS), (size_t)pl.smem, stream, tq, tkv, tr, a);
-  if (le != cudaSuccess) return (int)le;
+  return prefill_launch(a, q, kv, rot_rows, B, T, rows, kv_ld, max_query_len, pl, stream);
+}
+
+// Dense rows [keys of all heads | values of all heads] of the K / V pages that the sequences of a step see
+// (kv_gather_kernel); `rows` = span_off[B].
+OXB_API int oxb_kv_gather(const void* cache, const int* block_tables, const int* span_lo, const int* span_off, int B, int rows,
+                          int max_blocks, int heads, int width, int page, int num_blocks, void* out, cudaStream_t stream) {
+  if (rows <= 0 || B <= 0) return 0;
+  if (width % 8 != 0 || page <= 0) return (int)cudaErrorInvalidValue;
+  oxb_launch(kv_gather_kernel, dim3((rows + 3) / 4), dim3(128), 0, stream, reinterpret_cast<const __nv_bfloat16*>(cache), block_tables,
+             span_lo, span_off, B, max_blocks, heads, width, page, num_blocks, reinterpret_cast<__nv_bfloat16*>(out));
   OXB_CHECK_LAUNCH();
   return 0;
+}
+
+// Grouped-query attention of long portions: q [T, H, width], kv as oxb_kv_gather leaves it, out [T, H * width] with rows
+// ld_out apart; width a multiple of 16.
+OXB_API int oxb_gqa_prefill(const void* q, const void* kv, void* out, int ld_out, float out_scale, const int* query_start,
+                            const int* seq_lens, const int* span_lo, const int* span_off, const float* sink, int B, int T, int H,
+                            int G, int rows, int width, int window, float scale, int max_query_len, cudaStream_t stream) {
+  if (T <= 0 || B <= 0 || max_query_len <= 0 || rows <= 0) return 0;
+  const LatentPrefillPlan pl = latent_prefill_plan(width, 0, width);
+  if (pl.smem == 0 || width % 16 != 0 || G <= 0 || H % G != 0 || H > 65535 || B > 65535) return (int)cudaErrorInvalidValue;
+  LatentPrefillArgs a;
+  a.query_start = query_start;
+  a.seq_lens = seq_lens;
+  a.span_lo = span_lo;
+  a.span_off = span_off;
+  a.sink = sink;
+  a.out = reinterpret_cast<__nv_bfloat16*>(out);
+  a.H = H;
+  a.window = window;
+  a.group = H / G;
+  a.ld_out = ld_out;
+  a.out_scale = out_scale;
+  a.nope16 = width / 16;
+  a.rot16 = 0;
+  a.full_ld = width;
+  a.nope_ld = width;
+  a.v_off = G * width;
+  a.v_ld = width;
+  a.v = width;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  return prefill_launch(a, q, kv, nullptr, B, T, rows, 2 * G * width, max_query_len, pl, stream);
 }

@@ -133,4 +133,114 @@ int residual_norm_launch(const ResidualNormArgs& a, int T, cudaStream_t stream) 
   return 0;
 }
 
+// Norms on both sides of a branch: x = res + rms(y) * w_post, then the next branch's input rms(x) * w_next in the activation
+// type, in one kernel (the stream x in float32; w_next null: the sum alone; y null: the norm alone).
+struct BranchNormArgs {
+  const float* res;              // [T, H]
+  const void* y;                 // [T, H] in the activation type, or null
+  const float *w_post, *w_next;  // [H]
+  float* x_out;                  // [T, H] or null
+  void* a_out;                   // [T, H] in the activation type, or null
+  int H;
+  float eps;
+};
+
+// One CTA per row; every thread owns CH groups of four neighbouring values (H % 4 == 0, H <= 4 * CH * threads).
+template <typename A, int CH>
+__global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchNormArgs a) {
+  __shared__ float red[32];
+  const int H4 = a.H >> 2;
+  const size_t base = (size_t)blockIdx.x * a.H;
+  float4 y[CH], v[CH], w[CH], n[CH];
+  pdl_launch_dependents();
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {  // weights are static: fetched ahead of the dependency
+    const int i = threadIdx.x + c * blockDim.x;
+    w[c] = n[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H4) {
+      if (a.w_post != nullptr) w[c] = rn_load4(a.w_post + 4 * i);
+      if (a.w_next != nullptr) n[c] = rn_load4(a.w_next + 4 * i);
+    }
+  }
+  pdl_wait();
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    y[c] = v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H4) {
+      v[c] = rn_load4(a.res + base + 4 * i);
+      if (a.y != nullptr) y[c] = rn_load4(reinterpret_cast<const A*>(a.y) + base + 4 * i);
+    }
+    ss += (y[c].x * y[c].x + y[c].y * y[c].y) + (y[c].z * y[c].z + y[c].w * y[c].w);
+  }
+  if (a.y != nullptr) {
+    const float inv = rsqrtf(block_sum(ss, red) / (float)a.H + a.eps);
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int i = threadIdx.x + c * blockDim.x;
+      v[c] = make_float4(v[c].x + y[c].x * inv * w[c].x, v[c].y + y[c].y * inv * w[c].y, v[c].z + y[c].z * inv * w[c].z,
+                         v[c].w + y[c].w * inv * w[c].w);
+      if (i < H4 && a.x_out != nullptr) rn_store4(a.x_out + base + 4 * i, v[c]);
+    }
+  }
+  if (a.a_out == nullptr) return;
+  ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) ss += (v[c].x * v[c].x + v[c].y * v[c].y) + (v[c].z * v[c].z + v[c].w * v[c].w);
+  const float inv = rsqrtf(block_sum(ss, red) / (float)a.H + a.eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    if (i < H4)
+      rn_store4(reinterpret_cast<A*>(a.a_out) + base + 4 * i,
+                make_float4(v[c].x * inv * n[c].x, v[c].y * inv * n[c].y, v[c].z * inv * n[c].z, v[c].w * inv * n[c].w));
+  }
+}
+
+// Any width: the row is staged in shared memory (dynamic, H floats).
+template <typename A>
+__global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormArgs a) {
+  extern __shared__ float rn_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t base = (size_t)blockIdx.x * a.H;
+  const A* y = reinterpret_cast<const A*>(a.y);
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    rn_row[i] = y != nullptr ? rn_load(y + base + i) : 0.f;
+    ss += rn_row[i] * rn_row[i];
+  }
+  const float inv_y = y != nullptr ? rsqrtf(block_sum(ss, red) / (float)a.H + a.eps) : 0.f;
+  ss = 0.f;
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    float v = a.res[base + i];
+    if (y != nullptr) v += rn_row[i] * inv_y * a.w_post[i];
+    rn_row[i] = v;
+    if (a.x_out != nullptr) a.x_out[base + i] = v;
+    ss += v * v;
+  }
+  if (a.a_out == nullptr) return;
+  const float inv = rsqrtf(block_sum(ss, red) / (float)a.H + a.eps);
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x)
+    rn_store(reinterpret_cast<A*>(a.a_out) + base + i, rn_row[i] * inv * a.w_next[i]);
+}
+
+template <typename A>
+int branch_norm_launch(const BranchNormArgs& a, int T, cudaStream_t stream) {
+  if (a.H % 4 == 0 && a.H <= 16384) {
+    const int H4 = a.H / 4, lim = T >= 512 ? 256 : 1024, ch = H4 <= lim ? 1 : (H4 <= 2 * lim ? 2 : 4);
+    const int threads = ((H4 + ch - 1) / ch + 31) / 32 * 32;
+    if (ch == 1) oxb_launch(branch_norm_kernel<A, 1>, dim3(T), dim3(threads), 0, stream, a);
+    else if (ch == 2) oxb_launch(branch_norm_kernel<A, 2>, dim3(T), dim3(threads), 0, stream, a);
+    else oxb_launch(branch_norm_kernel<A, 4>, dim3(T), dim3(threads), 0, stream, a);
+  } else {
+    if (a.H > 12 * 1024) return (int)cudaErrorInvalidValue;  // 48 KB of shared memory
+    oxb_launch(branch_norm_any_kernel<A>, dim3(T), dim3(256), (size_t)a.H * sizeof(float), stream, a);
+  }
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
 }  // namespace oxb

@@ -181,7 +181,7 @@ class RetentionSpec:
     # head widths in projections, state and outputs (the padding is zero)
     @property
     def k_width(self) -> int:
-        return (self.dim + 31) // 32 * 32
+        return next((w for w in HEAD_WIDTHS if w >= self.dim), (self.dim + 31) // 32 * 32)
 
     @property
     def v_width(self) -> int:

@@ -283,8 +283,9 @@ class Transformer:
         epilogue of the gate_up GEMM (one kernel and one activation round trip less per layer)."""
         from ..ops import cuda as opcuda
 
-        for lw in self.w.layers:
-            w = lw.w_gate_up
+        # (shared experts: listed layers only, whose feed-forward operator reads either layout)
+        pairs = [w for lw in self.w.layers for w in (lw.w_gate_up, lw.shared_gate_up if self.cfg.is_layered else None)]
+        for w in pairs:
             if w is None or w.swiglu_interleaved or len(w.parts) != 1 or w.bias is not None:
                 continue
             p = w.parts[0]

@@ -123,7 +123,7 @@ def _declare(L) -> None:
                                       i32, i32, vp]
     L.oxb_argmax.argtypes = [vp, i32, i32, i32, i32, vp, vp, i32, vp]
     L.oxb_paged_attention.argtypes = [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32,
-                                      vp, vp, vp, i32, vp]
+                                      vp, i32, f32, vp, vp, vp, i32, vp]
     L.oxb_sample.argtypes = [vp, i32, i32, i32, vp, vp, vp, vp, vp, i32, vp, vp]
     L.oxb_gemm_quant.argtypes =[vp, vp, i32, sz, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, sz, vp, i32, vp]
     u64p, ull = ctypes.POINTER(ctypes.c_uint64), ctypes.c_ulonglong
@@ -510,15 +510,21 @@ def attn_splits(B: int, nkv: int, mtiles: int, max_seq_len: int, sms: int) -> in
     return max(1, min(want, cap, 16))
 
 
-def paged_attention(q, kv, layer, meta, scale, sliding_window=0, splits: Optional[int] = None, softcap: float = 0.0):
+def paged_attention(q, kv, layer, meta, scale, sliding_window=0, splits: Optional[int] = None, softcap: float = 0.0,
+                    sink: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, out_scale: float = 1.0):
+    """``sink`` [nq]: logits of the softmax denominator; ``out`` [T, nq * hd] may be a column slice of a wider buffer."""
     T, nq, hd = q.shape
-    nkv = kv.spec.n_kv_heads
+    nkv = kv.spec.heads(layer)
     B = meta.seq_lens.shape[0]
     G = nq // nkv
     mtiles = (max(1, meta.max_query_len) * G + 15) // 16
     if splits is None:
-        splits = attn_splits(B, nkv, mtiles, meta.max_seq_len or kv.page_size, sm_count(q.device))
-    out = torch.empty_like(q)
+        span = meta.max_seq_len or kv.page_size
+        if sliding_window > 0:
+            span = min(span, sliding_window + max(1, meta.max_query_len))
+        splits = attn_splits(B, nkv, mtiles, span, sm_count(q.device))
+    if out is None:
+        out = torch.empty_like(q)
     ws_o = ws_ml = cnt = None
     if splits > 1 and B * nkv * mtiles > scratch(q.device).attn_counters.numel():
         splits = 1
@@ -529,9 +535,9 @@ def paged_attention(q, kv, layer, meta, scale, sliding_window=0, splits: Optiona
     _check(lib().oxb_paged_attention(q.data_ptr(), out.data_ptr(), kv.data[layer].data_ptr(), _p(kv.scales[layer]),
                                      meta.block_tables.data_ptr(), meta.seq_lens.data_ptr(), meta.query_start.data_ptr(),
                                      B, meta.block_tables.stride(0), nq, nkv, hd, KV_MODE[kv.dtype_name],
-                                     max(1, meta.max_query_len), splits, sliding_window, scale, float(softcap), _p(ws_o),
-                                     _p(ws_ml),
-                                     _p(cnt), kv.num_blocks, _stream()), "oxb_paged_attention")
+                                     max(1, meta.max_query_len), splits, sliding_window, scale, float(softcap), _p(sink),
+                                     out.stride(0), out_scale, _p(ws_o), _p(ws_ml), _p(cnt), kv.num_blocks, _stream()),
+           "oxb_paged_attention")
     return out
 
 

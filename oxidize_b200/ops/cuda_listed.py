@@ -1,0 +1,242 @@
+"""Bindings of the kernels behind listed layers with grouped-query attention, retention, norms on both sides of a branch and
+gated or routed feed-forward blocks (``csrc/oxb_listed.cu``), in bfloat16 and float32.  CUDA tensors only; see
+:mod:`oxidize_b200.ops` for the operators' meaning."""
+from __future__ import annotations
+
+import ctypes
+from typing import Optional
+
+import torch
+
+from ..models.config import HEAD_WIDTHS
+from . import cuda as opcuda
+from . import cuda_latent as latent
+from .cuda import _check, _p, _stream
+
+_declared = False
+
+DT = latent.DT
+
+
+def lib():
+    global _declared
+    L = latent.lib()
+    if not _declared:
+        vp, i32, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
+        L.oxb_branch_norm.argtypes = [vp] * 6 + [i32] * 3 + [f32, vp]
+        L.oxb_head_prep.argtypes = [vp, i32, i32, vp, vp, vp] + [i32] * 3 + [vp, vp, i32, f32] + [i32] * 5 + [vp, vp, i32, i32, vp]
+        L.oxb_gqa_attention_simt.argtypes = [vp, vp, i32, f32, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp]
+        L.oxb_kv_gather.argtypes = [vp] * 4 + [i32] * 7 + [vp, vp]
+        L.oxb_gqa_prefill.argtypes = [vp, vp, vp, i32, f32] + [vp] * 5 + [i32] * 7 + [f32, i32, vp]
+        L.oxb_retention_chunk_supported.argtypes = [i32, i32]
+        L.oxb_retention.argtypes = ([vp, i32, i32] + [vp] * 4 + [i32] * 3 + [vp, vp, i32, vp, i32, f32] + [i32] * 5 + [f32, f32]
+                                    + [i32] * 4 + [vp, vp])
+        L.oxb_silu_mul_f32.argtypes = [vp, vp, vp, i32, i32, vp]
+        L.oxb_moe_combine_f32.argtypes = [vp, i32, vp, vp, i32, vp, vp, i32, i32, vp]
+        L.oxb_router_logits.argtypes = [vp, vp, i32, vp] + [i32] * 3 + [vp]
+        L.oxb_gemm_f32_rows.argtypes = [vp] * 5 + [i32] * 6 + [vp]
+        _declared = True
+    return L
+
+
+# --------------------------------------------------------------------------- norms
+def branch_norm(res: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torch.Tensor], w_next: Optional[torch.Tensor],
+                eps: float, act_dtype: torch.dtype):
+    T, H = res.shape
+    if y is not None and (y.dtype != act_dtype or not y.is_contiguous()):
+        y = y.to(act_dtype).contiguous()
+    x = res if y is None else torch.empty_like(res)
+    a = None if w_next is None else torch.empty(T, H, dtype=act_dtype, device=res.device)
+    _check(lib().oxb_branch_norm(res.data_ptr(), _p(y), _p(w_post), _p(w_next), None if y is None else x.data_ptr(), _p(a),
+                                 DT[act_dtype], T, H, eps, _stream()), "oxb_branch_norm")
+    return x, a
+
+
+# --------------------------------------------------------------------------- attention
+def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int, eps: float) -> torch.Tensor:
+    """q | k | v projections [T, ...] to rotated queries [T, heads, width]; keys and values go into the cache pages."""
+    T = z.shape[0]
+    tab = opcuda.rope_table(rope, rope.max_pos)
+    q = torch.empty(T, spec.heads, spec.width, dtype=z.dtype, device=z.device)
+    _check(lib().oxb_head_prep(z.data_ptr(), z.stride(0), DT[z.dtype], meta.positions.data_ptr(), meta.slot_mapping.data_ptr(),
+                               tab.data_ptr(), tab.shape[0], tab.shape[1], 0 if rope.pairing == "split_half" else 1, _p(q_norm),
+                               _p(k_norm), 1 if spec.qk_norm == "full" else 0, eps, T, spec.heads, spec.kv_heads, spec.dim,
+                               spec.width, q.data_ptr(), kv.data[layer].data_ptr(), kv.page_size, kv.num_blocks, _stream()),
+           "oxb_head_prep")
+    return q
+
+
+def attention_simt(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> None:
+    T, H, W = q.shape
+    B = meta.seq_lens.shape[0]
+    _check(lib().oxb_gqa_attention_simt(q.data_ptr(), out.data_ptr(), out.stride(0), out_scale, kv.data[layer].data_ptr(), DT[q.dtype],
+                                        meta.block_tables.data_ptr(), meta.seq_lens.data_ptr(), meta.query_start.data_ptr(), _p(sink),
+                                        B, meta.block_tables.stride(0), T, H, spec.kv_heads, W, kv.page_size, kv.num_blocks,
+                                        spec.window, spec.scale, _stream()), "oxb_gqa_attention_simt")
+
+
+def attention_prefill(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> None:
+    """Long portions: the visible rows are gathered from their pages, then flash attention on tcgen05."""
+    T, H, W = q.shape
+    B, G = meta.seq_lens.shape[0], spec.kv_heads
+    lo, off, rows = latent._spans(meta, spec.window)
+    dense = torch.empty(rows, 2 * G * W, dtype=q.dtype, device=q.device)
+    _check(lib().oxb_kv_gather(kv.data[layer].data_ptr(), meta.block_tables.data_ptr(), lo.data_ptr(), off.data_ptr(), B, rows,
+                               meta.block_tables.stride(0), G, W, kv.page_size, kv.num_blocks, dense.data_ptr(), _stream()),
+           "oxb_kv_gather")
+    _check(lib().oxb_gqa_prefill(q.data_ptr(), dense.data_ptr(), out.data_ptr(), out.stride(0), out_scale, meta.query_start.data_ptr(),
+                                 meta.seq_lens.data_ptr(), lo.data_ptr(), off.data_ptr(), _p(sink), B, T, H, G, rows, W, spec.window,
+                                 spec.scale, max(n for n, _ in meta.host_lens), _stream()), "oxb_gqa_prefill")
+
+
+def attention(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> None:
+    """Attention of a step's queries over the cache into ``out`` [T, heads * width] (may be a column slice)."""
+    if q.dtype != torch.bfloat16 or kv.page_size != 16 or spec.width not in HEAD_WIDTHS:
+        attention_simt(q, kv, layer, meta, spec, sink, out, out_scale)
+        return
+    if (not meta.host_lens or max(n for n, _ in meta.host_lens) < latent.EXPAND_ROWS
+            or not lib().oxb_latent_prefill_supported(spec.width, 0, spec.width)
+            or latent._spans(meta, spec.window)[2] > latent.MAX_SPAN):
+        opcuda.paged_attention(q, kv, layer, meta, spec.scale, spec.window, sink=sink, out=out, out_scale=out_scale)
+        return
+    starts = [0]
+    for n, _ in meta.host_lens:
+        starts.append(starts[-1] + n)
+    runs = latent._runs(meta.host_lens)
+    for b0, b1, big in runs:
+        t0, t1 = starts[b0], starts[b1]
+        sub = meta if len(runs) == 1 else latent._sub_batch(meta, b0, b1, t0, t1)
+        if big:
+            attention_prefill(q[t0:t1], kv, layer, sub, spec, sink, out[t0:t1], out_scale)
+        else:
+            opcuda.paged_attention(q[t0:t1], kv, layer, sub, spec.scale, spec.window, sink=sink, out=out[t0:t1], out_scale=out_scale)
+
+
+# --------------------------------------------------------------------------- retention
+CHUNK_ROWS = 9  # sequences that feed at least this many rows in a step go through chunks on the tensor cores
+SEGMENT_ROWS = 128  # a segment of a long portion is at least this long
+_ALL = 1 << 30
+
+
+def segments(rows: int, seqs: int, heads: int, sms: int) -> int:
+    """Segments of the longest portion: as many as keep one CTA per SM busy."""
+    return max(1, min(rows // SEGMENT_ROWS, sms // max(1, seqs * heads), 32))
+
+
+def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, decay: torch.Tensor, eps: float, out: torch.Tensor,
+              out_scale: float, chunk_rows: Optional[int] = None, n_seg: Optional[int] = None) -> None:
+    """z [T, q | k | v | gate] to the normed, gated heads ``out`` [T, heads * v_width]; ``state`` [slots, H, K, V] is updated."""
+    L = lib()
+    H, K, V = spec.state_shape
+    B = meta.seq_lens.shape[0]
+    tab = opcuda.rope_table(rope, rope.max_pos)
+    if meta.state_slots is None:
+        raise ValueError("a layer with a recurrent state needs the sequences' state slots")
+
+    def run(lo: int, hi: int, chunk: int, seg: int, ws) -> None:
+        _check(L.oxb_retention(z.data_ptr(), z.stride(0), DT[z.dtype], meta.query_start.data_ptr(), meta.seq_lens.data_ptr(),
+                               meta.state_slots.data_ptr(), tab.data_ptr(), tab.shape[0], tab.shape[1],
+                               0 if rope.pairing == "split_half" else 1, decay.data_ptr(), state.data_ptr(), state.shape[0],
+                               out.data_ptr(), out.stride(0), out_scale, B, H, K, V, spec.v_dim, spec.dim ** -0.5, eps, lo, hi, chunk,
+                               seg, _p(ws), _stream()), "oxb_retention")
+
+    most = max(1, meta.max_query_len)
+    least = 1 if meta.host_lens is None else min(n for n, _ in meta.host_lens)
+    cut = CHUNK_ROWS if chunk_rows is None else chunk_rows
+    if z.dtype != torch.bfloat16 or most < cut or not L.oxb_retention_chunk_supported(K, V):
+        run(1, _ALL, 0, 1, None)
+        return
+    if least < cut:
+        run(1, cut - 1, 0, 1, None)
+    if n_seg is None:
+        seqs = B if meta.host_lens is None else sum(n >= cut for n, _ in meta.host_lens)
+        n_seg = segments(most, seqs, H, opcuda.sm_count(z.device))
+    ws = torch.empty(B * H * n_seg * K * V, dtype=torch.float32, device=z.device) if n_seg > 1 else None
+    run(cut, _ALL, 1, n_seg, ws)
+
+
+def listed_mixer(x: torch.Tensor, lw, spec, ropes, meta, kv, kv_layer: int, state_layer: int, eps: float) -> torch.Tensor:
+    from . import linear
+
+    z = linear(x, lw.wqkv)
+    a, r = spec.attention, spec.retention
+    sl, sr = spec.branch_scales
+    out = torch.empty(x.shape[0], spec.out_dim, dtype=x.dtype, device=x.device)
+    na = no = 0
+    if a is not None:
+        if kv.data[kv_layer].dtype != x.dtype:
+            raise ValueError(f"cache rows of listed layers are kept in the compute type on the GPU ({x.dtype}), not {kv.dtype_name}")
+        na, no = a.proj_dim, a.out_dim
+        q = head_prep(z[:, :na], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps)
+        attention(q, kv, kv_layer, meta, a, lw.sink, out[:, :no], sl)
+    if r is not None:
+        decay = getattr(lw, "_decay", None)
+        if decay is None:
+            decay = lw._decay = torch.tensor(r.decay, dtype=torch.float32, device=x.device)
+        retention(z[:, na:], r, ropes[1], meta, kv.states.data[state_layer], decay, eps, out[:, no:], sr)
+    return out
+
+
+# --------------------------------------------------------------------------- feed-forward blocks
+def silu_mul_f32(gu: torch.Tensor, n_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    T, F2 = gu.shape
+    out = torch.empty(T, F2 // 2, dtype=torch.float32, device=gu.device)
+    _check(lib().oxb_silu_mul_f32(gu.data_ptr(), out.data_ptr(), _p(n_rows), T, F2 // 2, _stream()), "oxb_silu_mul_f32")
+    return out
+
+
+def gated_ffn(x: torch.Tensor, gate_up, down) -> torch.Tensor:
+    from . import linear
+
+    if x.dtype == torch.float32:
+        return linear(silu_mul_f32(linear(x, gate_up)), down)
+    if gate_up.swiglu_interleaved:
+        xp, data = opcuda.pad_k(x.contiguous(), gate_up.parts[0])
+        return linear(opcuda.linear_swiglu(xp, data), down)
+    return linear(opcuda.silu_mul(linear(x, gate_up)), down)
+
+
+def router_logits(x: torch.Tensor, w) -> torch.Tensor:
+    """[T, experts] float32, never rounded to 16 bits."""
+    x = x.contiguous()
+    T, K = x.shape
+    out = torch.empty(T, w.shape[0], dtype=torch.float32, device=x.device)
+    if w.data.dtype != x.dtype:
+        raise ValueError(f"router weights are kept in the compute type ({x.dtype}), not {w.data.dtype}")
+    _check(lib().oxb_router_logits(x.data_ptr(), w.data.data_ptr(), DT[x.dtype], out.data_ptr(), T, w.shape[0], K, _stream()),
+           "oxb_router_logits")
+    return out
+
+
+def _gemm_rows(x, w, offsets, perm, groups: int, rows: int, max_rows: int) -> torch.Tensor:
+    N, K = w.shape[0] // groups, w.shape[1]
+    y = torch.empty(rows, N, dtype=torch.float32, device=x.device)
+    _check(lib().oxb_gemm_f32_rows(x.data_ptr(), w.data.data_ptr(), y.data_ptr(), offsets.data_ptr(), _p(perm), groups, max_rows, N, K,
+                                   x.stride(0), N, _stream()), "oxb_gemm_f32_rows")
+    return y
+
+
+def moe_ffn(x: torch.Tensor, lw, spec) -> torch.Tensor:
+    from . import cuda_moe
+
+    T, H = x.shape
+    ex = lw.experts
+    logits = router_logits(x, lw.router)
+    shared = gated_ffn(x, lw.shared_gate_up, lw.shared_down) if lw.shared_gate_up is not None else None
+    pad = ex.gate_up_stack.shape[1] - H
+    xp = torch.nn.functional.pad(x, (0, pad)) if pad else x.contiguous()
+    if x.dtype == torch.bfloat16:
+        sp = torch.nn.functional.pad(shared, (0, pad)) if pad and shared is not None else shared
+        out = cuda_moe.moe_layer(xp, logits, spec, None, ex, sp)[0]
+        return out[:, :H].contiguous() if pad else out
+    E, k = spec.n_experts, spec.n_experts_used
+    if E > 256 or T * k > cuda_moe.MAX_DISPATCH_ENTRIES:
+        raise ValueError("float32 expert dispatch covers up to 256 experts and 2^17 token x expert pairs in a step")
+    ids, wts = cuda_moe.moe_route(logits, spec)
+    offsets, perm, inv = cuda_moe.moe_dispatch(ids, 0, E)
+    h = _gemm_rows(xp, ex.gate_up_stack, offsets, perm, E, T * k, T)
+    y = _gemm_rows(silu_mul_f32(h, offsets[E:]), ex.down_stack, offsets, None, E, T * k, T)
+    out = torch.empty(T, H, dtype=torch.float32, device=x.device)
+    _check(lib().oxb_moe_combine_f32(y.data_ptr(), y.stride(0), inv.data_ptr(), wts.data_ptr(), k, _p(shared), out.data_ptr(), T, H,
+                                     _stream()), "oxb_moe_combine_f32")
+    return out
