@@ -230,7 +230,8 @@ __global__ void __launch_bounds__(256) retention_chunk_kernel(const RetentionArg
 #pragma unroll
   for (int i = 0; i < 2 * KT; ++i) S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.f;
   float* ws = a.ws + (((size_t)b * a.H + h) * nseg) * K * V + tid;  // (blocks are laid out thread by thread)
-  if (pos0 > 0 && (OUT ? nseg == 1 : seg == 0)) {  // (written by an earlier step: no need to wait for this step's kernels)
+  const bool single = n_all <= L;  // nobody else reads or writes this state
+  if (pos0 > 0 && (OUT ? single : seg == 0)) {  // (written by an earlier step: no need to wait for this step's kernels)
 #pragma unroll
     for (int i = 0; i < 2 * KT; ++i)
 #pragma unroll
@@ -246,7 +247,7 @@ __global__ void __launch_bounds__(256) retention_chunk_kernel(const RetentionArg
         S[i][e] = 0.f;
       }
   }
-  if (OUT && nseg > 1) {
+  if (OUT && !single) {
     for (int j = 0; j <= seg; ++j) {
       const float f = exp2f(l2 * (float)(j == 0 ? s0 : (seg - j) * L));
       const float* w = ws + (size_t)j * K * V;

@@ -366,6 +366,14 @@ def synth_layered_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: i
     zeros = (lambda n: torch.zeros(n, dtype=torch.float32, device=device)) if bias else (lambda n: None)
     layers = []
     for spec in cfg.layer_specs:
+        if spec.weights_of is not None:
+            layers.append(layers[spec.weights_of])
+            continue
+        if cfg.norm_placement == "sandwich":
+            if tp_size > 1:
+                raise ValueError("layers with per-sequence states and norms over all heads are not sharded")
+            layers.append(_synth_listed(spec, h, mat, ones))
+            continue
         m, f = spec.mixer, spec.ffn
         H, own = m.heads // tp_size, m.kv_from is None
         mla = latent_weights(m, mat(H * m.qk_dim, h), mat(m.kv_rank + m.rope_dim, h, own=False) if own else None,
@@ -385,6 +393,37 @@ def synth_layered_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: i
     if cfg.embed_norm:
         mw.embed_norm, mw.embed_norm_bias = ones(h), zeros(h)
     return mw
+
+
+def _synth_listed(spec, h: int, mat, ones) -> LayerWeights:
+    """One layer with norms on both sides of its branches (``mat(out, in)`` draws a matrix)."""
+    from ..models.config import MoESpec
+    from ..models.layered import dense_qtensor, gated_pair, listed_experts, listed_mixer
+
+    a, r, f = spec.attention, spec.retention, spec.ffn
+    att, ret = {}, {}
+    if a is not None:
+        att = {"q": mat(a.heads * a.dim, h), "k": mat(a.kv_heads * a.dim, h), "v": mat(a.kv_heads * a.v_dim, h),
+               "o": mat(h, a.heads * a.v_dim), "sink": ones(a.heads)}
+        full = a.qk_norm == "full"
+        att["q.norm"], att["k.norm"] = ones(a.dim * (a.heads if full else 1)), ones(a.dim * (a.kv_heads if full else 1))
+    if r is not None:
+        ret = {n: mat(r.heads * (r.dim if n in "qk" else r.v_dim), h) for n in "qkvg"}
+        ret["o"] = mat(h, r.heads * r.v_dim)
+    lw = LayerWeights(attn_norm=ones(h), post_attn_norm=ones(h), ffn_norm=None, **listed_mixer(spec, att, ret))
+    if f is None:
+        return lw
+    lw.ffn_norm, lw.post_ffn_norm = ones(h), ones(h)
+    pair = lambda s: [LinearWeight([q]) for q in gated_pair(mat(s.size, h), mat(s.size, h), mat(h, s.size), s.pad_size)]
+    if isinstance(f, MoESpec):
+        lw.router = dense_qtensor(mat(f.n_experts, h))
+        lw.experts = listed_experts(f, ((mat(f.expert.size, h), mat(f.expert.size, h), mat(h, f.expert.size))
+                                        for _ in range(f.n_experts)), h)
+        if f.shared is not None:
+            lw.shared_gate_up, lw.shared_down = pair(f.shared)
+    else:
+        lw.w_gate_up, lw.w_down = pair(f)
+    return lw
 
 
 def _main(argv=None) -> int:
