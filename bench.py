@@ -64,8 +64,9 @@ def parse_args():
     ap.add_argument("--draft-model", default=None, help="preset of a draft model: measure speculative decoding as well")
     ap.add_argument("--draft-tokens", type=int, default=4)
     ap.add_argument("--layered", default=None, metavar="WIDTHxHEADS",
-                    help="instead of the headline workload: a model that lists its layers (Vefilix) beside the closest uniform "
-                         "models of that size (see bench/layered_bench.py), e.g. 4096x32")
+                    help="instead of the headline workload: a model that lists its layers beside the closest uniform "
+                         "models of that size (see bench/layered_bench.py, bench/sokirax_bench.py), e.g. 4096x32")
+    ap.add_argument("--design", default="vefilix", choices=["vefilix", "sokirax"], help="the design that --layered measures")
     return ap.parse_args()
 
 

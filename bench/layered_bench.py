@@ -220,6 +220,10 @@ def kernel_numbers(width: int, heads: int, window: int, dev, steps: int) -> list
 def main(args) -> int:
     if args.gpus != 1:
         raise SystemExit("--layered runs on one GPU")
+    if args.design == "sokirax":
+        import sokirax_bench
+
+        return sokirax_bench.main(args)
     from oxidize_b200.ops import cuda as C
 
     dev = torch.device("cuda", 0)

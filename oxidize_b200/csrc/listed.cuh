@@ -22,6 +22,7 @@ struct HeadPrepArgs {
   void* q;              // [T, H, width]
   void* cache;          // layer base [blocks, G, 2, page, width]
   int page, num_blocks;
+  int per_cta;          // heads (of q, k and v together) per CTA
 };
 
 constexpr int HEAD_PREP_WARPS = 8;
@@ -93,8 +94,8 @@ __device__ __forceinline__ void head_rotate(const float* row, const float* cs, i
   }
 }
 
-// One CTA per token, one warp per head at a time, VPL neighbouring values per lane (32 * VPL >= width).  Dynamic shared
-// memory: one row of floats per warp.
+// grid (T, head groups), one warp per head at a time, VPL neighbouring values per lane (32 * VPL >= width).  A norm over all
+// heads is summed up by every CTA that needs it.  Dynamic shared memory: one row of floats per warp.
 template <typename T, int VPL>
 __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const HeadPrepArgs a) {
   extern __shared__ float hp_rows[];
@@ -105,10 +106,13 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
   const int W = a.width, d0 = lane * VPL;
   const T* z = reinterpret_cast<const T*>(a.z) + (size_t)t * a.ld;
   const bool norm = a.q_norm != nullptr, on = d0 < W;
+  const int h0 = blockIdx.y * a.per_cta, h1 = min(h0 + a.per_cta, a.H + 2 * a.G);
   float inv_q = 0.f, inv_k = 0.f;
-  if (norm && a.full) {
+  if (norm && a.full && h0 < a.H + a.G) {
     float sq = 0.f, sk = 0.f;
-    for (int h = warp; h < a.H + a.G; h += HEAD_PREP_WARPS) {
+    const int f0 = h0 < a.H ? 0 : a.H, f1 = h1 > a.H ? a.H + a.G : a.H;
+#pragma unroll 4
+    for (int h = f0 + warp; h < f1; h += HEAD_PREP_WARPS) {
       float v[VPL], s = 0.f;
       if (on) {
         head_load<VPL>(z + (size_t)h * W + d0, v);
@@ -126,9 +130,9 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
   const float* cs = a.cos_sin + (size_t)pos * a.rot;
   const int slot = a.slots[t], blk = slot < 0 ? -1 : slot / a.page, off = slot < 0 ? 0 : slot % a.page;
   const bool keep = blk >= 0 && blk < a.num_blocks;
-  if (blk >= a.num_blocks && threadIdx.x == 0) oxb_report(OXB_BAD_SLOT, slot);  // never write outside the pool
+  if (blk >= a.num_blocks && threadIdx.x == 0 && blockIdx.y == 0) oxb_report(OXB_BAD_SLOT, slot);  // never write outside the pool
   float* row = hp_rows + warp * W;
-  for (int h = warp; h < a.H + 2 * a.G; h += HEAD_PREP_WARPS) {
+  for (int h = h0 + warp; h < h1; h += HEAD_PREP_WARPS) {
     const bool is_q = h < a.H, is_v = h >= a.H + a.G;
     if (!is_q && !keep) continue;
     float v[VPL];

@@ -15,8 +15,12 @@ OXB_API int oxb_branch_norm(const float* res, const void* y, const float* w_post
 }
 
 template <typename T>
-static int head_prep_launch(const HeadPrepArgs& a, int rows, cudaStream_t stream) {
-  const dim3 grid(rows), block(HEAD_PREP_WARPS * 32);
+static int head_prep_launch(HeadPrepArgs a, int rows, cudaStream_t stream) {
+  // few tokens: their heads are spread over CTAs, a head per warp
+  const int heads = a.H + 2 * a.G, groups = (heads + HEAD_PREP_WARPS - 1) / HEAD_PREP_WARPS;
+  const int split = rows * groups <= 4 * oxb_sm_count() ? groups : 1;
+  a.per_cta = (heads + split - 1) / split;
+  const dim3 grid(rows, split), block(HEAD_PREP_WARPS * 32);
   const size_t smem = (size_t)HEAD_PREP_WARPS * a.width * sizeof(float);
   if (a.width <= 32) oxb_launch(head_prep_kernel<T, 1>, grid, block, smem, stream, a);
   else if (a.width <= 64) oxb_launch(head_prep_kernel<T, 2>, grid, block, smem, stream, a);
@@ -35,7 +39,7 @@ OXB_API int oxb_head_prep(const void* z, int ld, int dtype, const int* positions
   if (T <= 0) return 0;
   if (rot < 0 || rot % 2 != 0 || rot > width || width % 32 != 0 || page <= 0 || H <= 0 || G <= 0) return (int)cudaErrorInvalidValue;
   const HeadPrepArgs a{z, ld, positions, slots, cos_sin, max_pos, rot, pairing, q_norm, k_norm, full, eps, H, G, dim, width,
-                       q, cache, page, num_blocks};
+                       q, cache, page, num_blocks, 0};
   return dtype == 0 ? head_prep_launch<float>(a, T, stream) : head_prep_launch<__nv_bfloat16>(a, T, stream);
 }
 

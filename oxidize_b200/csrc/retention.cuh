@@ -104,6 +104,7 @@ __global__ void __launch_bounds__(THREADS) retention_step_kernel(const Retention
           o.y = fmaf(qq, s[i].y, o.y);
           o.z = fmaf(qq, s[i].z, o.z);
           o.w = fmaf(qq, s[i].w, o.w);
+          if (j == n - 1) S[(size_t)k * cols + c] = s[i];
         }
       }
       *reinterpret_cast<float4*>(part + r * V + 4 * c) = o;
@@ -114,11 +115,6 @@ __global__ void __launch_bounds__(THREADS) retention_step_kernel(const Retention
       for (int i = 0; i < R; ++i) o += part[i * V + tid];
     const float inv = rsqrtf(block_sum(o * o, red) / (float)a.v_dim + a.eps);
     if (tid < V) out[(size_t)j * a.ld_out + tid] = lat_from<T>(o * inv * (gate / (1.f + expf(-gate))) * a.out_scale);
-  }
-#pragma unroll
-  for (int i = 0; i < NK; ++i) {
-    const int k = i * R + r;
-    if (on && k < K) S[(size_t)k * cols + c] = s[i];
   }
 }
 
