@@ -130,7 +130,6 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
   __shared__ float wmax[LM_SOFT_WARPS][LM_CN];                // per-warp maxima of a tile, then per-warp sums
   __shared__ __align__(16) float mrow[LM_SOFT_WARPS][LM_CN];  // running maxima (a copy per warp)
   __shared__ __align__(16) float frow[LM_SOFT_WARPS][LM_CN];  // factors of a rescale / normalisation
-  pdl_launch_dependents();
 
   // (broadcast from lane 0: the role branches and what is computed inside them are then known to be warp-uniform)
   const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
@@ -190,6 +189,7 @@ latent_attention_mma_kernel(const __grid_constant__ CUtensorMap tmK, const __gri
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  pdl_launch_dependents();  // (only now: a CTA of the next kernel must not take the tensor memory that this one still waits for)
   const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_slot, 0);  // columns: S^T (two buffers of NR), then the blocks of O^T
   pdl_wait();  // queries and this step's cache rows come from the upstream kernels
 

@@ -128,7 +128,6 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   __shared__ uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], pv_done[2];
   __shared__ uint32_t tmem_slot;
   __shared__ volatile int abort_flag;
-  pdl_launch_dependents();
   const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0);
   const int h = blockIdx.y, b = blockIdx.z;
   const int q0 = a.query_start[b], qlen = a.query_start[b + 1] - q0;
@@ -171,6 +170,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
+  pdl_launch_dependents();  // (only now: a CTA of the next kernel must not take the tensor memory that this one still waits for)
   // tensor-memory columns of tile t: S at 64 t, P at 128 + 32 t, O at 256 + 128 t
   const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_slot, 0);
   pdl_wait();

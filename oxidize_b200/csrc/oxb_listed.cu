@@ -4,6 +4,7 @@
 #include "listed.cuh"
 #include "residual_norm.cuh"
 #include "retention.cuh"
+#include "retention_mma.cuh"
 using namespace oxb;
 
 // dtype codes of the activation type: 0 float32, 2 bfloat16
@@ -112,6 +113,30 @@ static int retention_chunk_go(const RetentionArgs& a, int B, int nseg, cudaStrea
   return 0;
 }
 
+static int retention_mma_go(const RetentionArgs& a, int B, int nseg, cudaStream_t stream) {
+  const int smem = retention_mma_plan(a.K, a.V).smem;
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
+  if (!configured[dev]) {
+    const int most = retention_mma_plan(128, 128).smem;
+    cudaError_t e = cudaFuncSetAttribute(retention_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(retention_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
+    if (e != cudaSuccess) return (int)e;
+    configured[dev] = true;
+  }
+  cudaError_t le = cudaSuccess;
+  if (nseg > 1) le = oxb_launch(retention_mma_kernel<false>, dim3(a.H, B, nseg - 1), dim3(RM_THREADS), (size_t)smem, stream, a);
+  if (le == cudaSuccess) le = oxb_launch(retention_mma_kernel<true>, dim3(a.H, B, nseg), dim3(RM_THREADS), (size_t)smem, stream, a);
+  if (le != cudaSuccess) return (int)le;
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+// 1 when retention_mma_kernel covers heads of these widths
+OXB_API int oxb_retention_mma_supported(int K, int V) { return retention_mma_plan(K, V).smem > 0; }
+
 // 1 when retention_chunk_kernel covers heads of these widths
 OXB_API int oxb_retention_chunk_supported(int K, int V) {
   return (K == 32 || K == 64 || K == 96 || K == 128 || K == 192) && V % 16 == 0 && V > 0 && V <= 128 &&
@@ -119,8 +144,8 @@ OXB_API int oxb_retention_chunk_supported(int K, int V) {
 }
 
 // Retention of a step: z [T, ld] holds q | k (H heads of K values) and v | gate (H heads of V values), the state
-// [num_slots, H, K, V] float32 is read and updated.  chunk 0: retention_step_kernel, 1: retention_chunk_kernel (bf16) in
-// n_seg segments with scratch ws [B * H * n_seg * K * V] floats (unused with one segment); only sequences that feed
+// [num_slots, H, K, V] float32 is read and updated.  chunk 0: retention_step_kernel, 1: retention_chunk_kernel, 2:
+// retention_mma_kernel (both bf16) in n_seg segments with scratch ws [B * H * n_seg * K * V] floats (unused with one segment); only sequences that feed
 // min_rows .. max_rows rows take part.
 OXB_API int oxb_retention(const void* z, int ld, int dtype, const int* query_start, const int* seq_lens, const int* slots,
                           const float* cos_sin, int max_pos, int rot, int pairing, const float* decay, float* state, int num_slots,
@@ -132,9 +157,11 @@ OXB_API int oxb_retention(const void* z, int ld, int dtype, const int* query_sta
   const RetentionArgs a{z, ld, query_start, seq_lens, slots, cos_sin, max_pos, rot, pairing, decay, state, num_slots,
                         out, ld_out, out_scale, H, K, V, v_dim, k_scale, eps, min_rows, max_rows, ws};
   if (!chunk) return dtype == 0 ? retention_step_launch<float>(a, B, stream) : retention_step_launch<__nv_bfloat16>(a, B, stream);
-  if (dtype != 2 || !oxb_retention_chunk_supported(K, V) || n_seg < 1 || n_seg > 64 || (n_seg > 1 && ws == nullptr) || ld % 8 != 0 ||
-      ld_out % 2 != 0 || (reinterpret_cast<uintptr_t>(z) & 15) != 0)
+  if (dtype != 2 || n_seg < 1 || n_seg > 64 || (n_seg > 1 && ws == nullptr) || ld % 8 != 0 || ld_out % 8 != 0 ||
+      ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15) != 0)
     return (int)cudaErrorInvalidValue;
+  if (chunk == 2) return oxb_retention_mma_supported(K, V) ? retention_mma_go(a, B, n_seg, stream) : (int)cudaErrorInvalidValue;
+  if (!oxb_retention_chunk_supported(K, V)) return (int)cudaErrorInvalidValue;
   switch (K) {
     case 32: return retention_chunk_go<2>(a, B, n_seg, stream);
     case 64: return retention_chunk_go<4>(a, B, n_seg, stream);

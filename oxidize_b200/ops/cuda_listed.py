@@ -28,7 +28,7 @@ def lib():
         L.oxb_gqa_attention_simt.argtypes = [vp, vp, i32, f32, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp]
         L.oxb_kv_gather.argtypes = [vp] * 4 + [i32] * 7 + [vp, vp]
         L.oxb_gqa_prefill.argtypes = [vp, vp, vp, i32, f32] + [vp] * 5 + [i32] * 7 + [f32, i32, vp]
-        L.oxb_retention_chunk_supported.argtypes = [i32, i32]
+        L.oxb_retention_chunk_supported.argtypes = L.oxb_retention_mma_supported.argtypes = [i32, i32]
         L.oxb_retention.argtypes = ([vp, i32, i32] + [vp] * 4 + [i32] * 3 + [vp, vp, i32, vp, i32, f32] + [i32] * 5 + [f32, f32]
                                     + [i32] * 4 + [vp, vp])
         L.oxb_silu_mul_f32.argtypes = [vp, vp, vp, i32, i32, vp]
@@ -114,7 +114,7 @@ def attention(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> Non
 
 # --------------------------------------------------------------------------- retention
 CHUNK_ROWS = 9  # sequences that feed at least this many rows in a step go through chunks on the tensor cores
-SEGMENT_ROWS = 128  # a segment of a long portion is at least this long
+SEGMENT_ROWS = 256  # a segment of a long portion is at least this long
 _ALL = 1 << 30
 
 
@@ -123,8 +123,14 @@ def segments(rows: int, seqs: int, heads: int, sms: int) -> int:
     return max(1, min(rows // SEGMENT_ROWS, sms // max(1, seqs * heads), 32))
 
 
+def chunk_form(K: int, V: int) -> int:
+    """Which kernel takes long portions: 2 tcgen05, 1 mma.sync (wider keys), 0 neither (the token-by-token kernel does)."""
+    L = lib()
+    return 2 if L.oxb_retention_mma_supported(K, V) else 1 if L.oxb_retention_chunk_supported(K, V) else 0
+
+
 def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, decay: torch.Tensor, eps: float, out: torch.Tensor,
-              out_scale: float, chunk_rows: Optional[int] = None, n_seg: Optional[int] = None) -> None:
+              out_scale: float, chunk_rows: Optional[int] = None, n_seg: Optional[int] = None, form: Optional[int] = None) -> None:
     """z [T, q | k | v | gate] to the normed, gated heads ``out`` [T, heads * v_width]; ``state`` [slots, H, K, V] is updated."""
     L = lib()
     H, K, V = spec.state_shape
@@ -143,7 +149,9 @@ def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, decay: tor
     most = max(1, meta.max_query_len)
     least = 1 if meta.host_lens is None else min(n for n, _ in meta.host_lens)
     cut = CHUNK_ROWS if chunk_rows is None else chunk_rows
-    if z.dtype != torch.bfloat16 or most < cut or not L.oxb_retention_chunk_supported(K, V):
+    if form is None:
+        form = chunk_form(K, V)
+    if z.dtype != torch.bfloat16 or most < cut or form == 0:
         run(1, _ALL, 0, 1, None)
         return
     if least < cut:
@@ -152,7 +160,7 @@ def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, decay: tor
         seqs = B if meta.host_lens is None else sum(n >= cut for n, _ in meta.host_lens)
         n_seg = segments(most, seqs, H, opcuda.sm_count(z.device))
     ws = torch.empty(B * H * n_seg * K * V, dtype=torch.float32, device=z.device) if n_seg > 1 else None
-    run(cut, _ALL, 1, n_seg, ws)
+    run(cut, _ALL, form, n_seg, ws)
 
 
 def listed_mixer(x: torch.Tensor, lw, spec, ropes, meta, kv, kv_layer: int, state_layer: int, eps: float) -> torch.Tensor:

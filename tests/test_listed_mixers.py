@@ -362,23 +362,27 @@ def test_retention_of_unequal_sequences_in_one_step(device, dtype):
 @gpu
 @pytest.mark.parametrize("K,V", [(128, 128), (64, 96), (32, 16), (192, 64)])
 @pytest.mark.parametrize("n_seg", [1, 2, 5])
-def test_retention_segments_and_their_state(K, V, n_seg):
+@pytest.mark.parametrize("form", [1, 2])
+def test_retention_segments_and_their_state(K, V, n_seg, form):
     """A long portion in segments leaves the same outputs and, to float32 rounding of split products, the same state as the
     float32 steps; with a decay of one nothing is forgotten over the whole length."""
+    if form == 2 and K > 128:
+        return
     lens = [(500, 700), (321, 321), (64, 128), (1, 7)]
     spec, zs = retention_case(2, K, V, 16, [1.0, 0.995], lens, seed=n_seg)
     z = torch.cat([x[c - n :] for x, (n, c) in zip(zs, lens)])
     first = torch.randn(4, *spec.state_shape, device="cuda")
     a, b = first.clone(), first.clone()
     want = run_retention(z, spec, lens, [3, 1, 0, 2], a, "cuda", torch.float32)
-    got = run_retention(z, spec, lens, [3, 1, 0, 2], b, "cuda", torch.bfloat16, n_seg=n_seg)
+    got = run_retention(z, spec, lens, [3, 1, 0, 2], b, "cuda", torch.bfloat16, n_seg=n_seg, form=form)
     assert worst_row(got, want.double().cpu()) < 0.02
     for s in range(4):
         assert rel(b[s], a[s]) < 3e-5, s
 
 
 @gpu
-def test_retention_keeps_32_bits_of_what_enters_the_recurrence():
+@pytest.mark.parametrize("form", [1, 2])
+def test_retention_keeps_32_bits_of_what_enters_the_recurrence(form):
     """One early key and value, and a query far behind that stands on it: with a decay of one the output before the norm is
     their product; factors rounded to 16 bits would show in the state."""
     spec = RetentionSpec(1, 64, 64, [1.0], RotarySpec(64, 1e4))
@@ -386,7 +390,7 @@ def test_retention_keeps_32_bits_of_what_enters_the_recurrence():
     z = torch.zeros(600, 256)
     z[3] = torch.randn(256, generator=g).bfloat16().float()
     state = torch.zeros(1, 1, 64, 64, device="cuda")
-    run_retention(z, spec, [(600, 600)], [0], state, "cuda", torch.bfloat16, n_seg=3)
+    run_retention(z, spec, [(600, 600)], [0], state, "cuda", torch.bfloat16, n_seg=3, form=form)
     k = plain.rotate_heads(np.pad(z[3:4, None, 64:128].double().numpy(), ((3, 0), (0, 0), (0, 0))), {"dims": 64, "base": 1e4})[3, 0] / 8
     want = np.outer(k, z[3, 128:192].double().numpy())
     assert rel(state[0, 0], want) < 2e-5
