@@ -145,7 +145,7 @@ OXB_API int oxb_retention_chunk_supported(int K, int V) {
 
 // Retention of a step: z [T, ld] holds q | k (H heads of K values) and v | gate (H heads of V values), the state
 // [num_slots, H, K, V] float32 is read and updated.  chunk 0: retention_step_kernel, 1: retention_chunk_kernel, 2:
-// retention_mma_kernel (both bf16) in n_seg segments with scratch ws [B * H * n_seg * K * V] floats (unused with one segment); only sequences that feed
+// retention_mma_kernel (both bf16) in n_seg segments with scratch ws [B * H * n_seg * (K * V; 16384 in form 2)] floats (unused with one segment); only sequences that feed
 // min_rows .. max_rows rows take part.
 OXB_API int oxb_retention(const void* z, int ld, int dtype, const int* query_start, const int* seq_lens, const int* slots,
                           const float* cos_sin, int max_pos, int rot, int pairing, const float* decay, float* state, int num_slots,

@@ -159,7 +159,8 @@ def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, decay: tor
     if n_seg is None:
         seqs = B if meta.host_lens is None else sum(n >= cut for n, _ in meta.host_lens)
         n_seg = segments(most, seqs, H, opcuda.sm_count(z.device))
-    ws = torch.empty(B * H * n_seg * K * V, dtype=torch.float32, device=z.device) if n_seg > 1 else None
+    block = 128 * 128 if form == 2 else K * V  # floats of a segment's block
+    ws = torch.empty(B * H * n_seg * block, dtype=torch.float32, device=z.device) if n_seg > 1 else None
     run(cut, _ALL, form, n_seg, ws)
 
 
