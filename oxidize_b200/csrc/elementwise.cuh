@@ -12,16 +12,19 @@ namespace oxb {
 
 // ----------------------------------------------------------------------------- embedding
 // one CTA per token; qtype as in quant_blocks.cuh
+__device__ __forceinline__ void embed_put(__nv_bfloat16* o, float v) { *o = __float2bfloat16(v); }
+__device__ __forceinline__ void embed_put(float* o, float v) { *o = v; }
+template <typename O>
 static __global__ void embed_kernel(const int* __restrict__ tokens, const uint8_t* __restrict__ table, int qtype,
-                             size_t row_bytes, int H, int vocab, float scale, __nv_bfloat16* __restrict__ out) {
+                             size_t row_bytes, int H, int vocab, float scale, O* __restrict__ out) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
   int tok = tokens[t];
   if (tok < 0 || tok >= vocab) tok = 0;
   const uint8_t* row = table + (size_t)tok * row_bytes;
-  __nv_bfloat16* o = out + (size_t)t * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = __float2bfloat16(dequant_elem(qtype, row, i) * scale);
+  O* o = out + (size_t)t * H;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) embed_put(o + i, dequant_elem(qtype, row, i) * scale);
 }
 
 // ----------------------------------------------------------------------------- add + RMSNorm

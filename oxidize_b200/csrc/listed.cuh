@@ -23,6 +23,10 @@ struct HeadPrepArgs {
   void* cache;          // layer base [blocks, G, 2, page, width]
   int page, num_blocks;
   int per_cta;          // heads (of q, k and v together) per CTA
+  float temp_coef, temp_every;  // queries times 1 + temp_coef ln(floor((pos + 1) / temp_every) + 1); 0: off
+  const void* v_first;  // values that are mixed into this layer's, rows ld_first apart, heads first_width apart; or null
+  int ld_first, first_width, v_dim;
+  const float* v_mix;   // [1]: their share
 };
 
 constexpr int HEAD_PREP_WARPS = 8;
@@ -129,6 +133,7 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
   pos = pos < 0 ? 0 : (pos >= a.max_pos ? a.max_pos - 1 : pos);
   const float* cs = a.cos_sin + (size_t)pos * a.rot;
   const int slot = a.slots[t], blk = slot < 0 ? -1 : slot / a.page, off = slot < 0 ? 0 : slot % a.page;
+  const float temp = a.temp_coef != 0.f ? 1.f + a.temp_coef * logf(floorf((float)(a.positions[t] + 1) / a.temp_every) + 1.f) : 1.f;
   const bool keep = blk >= 0 && blk < a.num_blocks;
   if (blk >= a.num_blocks && threadIdx.x == 0 && blockIdx.y == 0) oxb_report(OXB_BAD_SLOT, slot);  // never write outside the pool
   float* row = hp_rows + warp * W;
@@ -158,8 +163,19 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
       __syncwarp();
       if (on) head_rotate<VPL>(row, cs, d0, a.rot, a.pairing, v);
       __syncwarp();
+      if (is_q) {
+#pragma unroll
+        for (int j = 0; j < VPL; ++j) v[j] *= temp;
+      }
     }
     if (!on) continue;
+    if (is_v && a.v_first != nullptr) {
+      const float mix = *a.v_mix;
+      const T* f = reinterpret_cast<const T*>(a.v_first) + (size_t)t * a.ld_first + (size_t)(h - a.H - a.G) * a.first_width;
+#pragma unroll
+      for (int j = 0; j < VPL; ++j)
+        if (d0 + j < a.v_dim) v[j] = (1.f - mix) * v[j] + mix * lat_f32(f[d0 + j]);
+    }
     T* dst;
     if (is_q) {
       dst = reinterpret_cast<T*>(a.q) + ((size_t)t * a.H + h) * W;
@@ -168,6 +184,26 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
       dst = reinterpret_cast<T*>(a.cache) + ((((size_t)blk * a.G + g) * 2 + is_v) * a.page + off) * W;
     }
     head_store<VPL>(dst + d0, v);
+  }
+}
+
+// Heads' outputs times the sigmoid of their gates, in place: one gate per head (per_value 0: gate [T, H]) or per value.
+template <typename T>
+__global__ void __launch_bounds__(256) head_gate_kernel(T* __restrict__ o, int ld, const T* __restrict__ gate, int ld_gate,
+                                                        int per_value, int rows, int H, int W) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n = H * W >> 2;  // groups of four values
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < (size_t)rows * n; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / n;
+    const int c = (int)(i % n) * 4;
+    float v[4], g[4];
+    head_load<4>(o + t * ld + c, v);
+    if (per_value) head_load<4>(gate + t * ld_gate + c, g);
+    else g[0] = g[1] = g[2] = g[3] = lat_f32(gate[t * ld_gate + c / W]);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] /= 1.f + expf(-g[j]);
+    head_store<4>(o + t * ld + c, v);
   }
 }
 

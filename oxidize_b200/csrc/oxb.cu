@@ -249,10 +249,15 @@ OXB_API int oxb_dequant_rows(const void* src, int qtype, size_t row_bytes, int r
 }
 
 OXB_API int oxb_embed(const int* tokens, const void* table, int qtype, size_t row_bytes, int H, int vocab, float scale,
-                      void* out_bf16, int T, cudaStream_t stream) {
+                      void* out, int f32, int T, cudaStream_t stream) {
   if (T <= 0) return 0;
-  oxb_launch(embed_kernel, dim3(T), dim3(256), 0, stream, tokens, reinterpret_cast<const uint8_t*>(table), qtype, row_bytes,
-             H, vocab, scale, reinterpret_cast<__nv_bfloat16*>(out_bf16));
+  const uint8_t* tab = reinterpret_cast<const uint8_t*>(table);
+  if (f32)
+    oxb_launch(embed_kernel<float>, dim3(T), dim3(256), 0, stream, tokens, tab, qtype, row_bytes, H, vocab, scale,
+               reinterpret_cast<float*>(out));
+  else
+    oxb_launch(embed_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, tokens, tab, qtype, row_bytes, H, vocab, scale,
+               reinterpret_cast<__nv_bfloat16*>(out));
   OXB_CHECK_LAUNCH();
   return 0;
 }

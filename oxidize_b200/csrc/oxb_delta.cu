@@ -1,0 +1,61 @@
+// liboxb, entry points of the gated delta rule (delta.cuh).
+#include "common.cuh"
+#include "delta.cuh"
+using namespace oxb;
+
+template <typename T, int NK, int THREADS>
+static int delta_step_go(const DeltaArgs& a, int B, cudaStream_t stream) {
+  const int R = THREADS / (a.V / 4);
+  const size_t smem = (size_t)(3 * a.K + 3 * a.V + 2 * R * a.V) * sizeof(float);
+  if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
+  oxb_launch(delta_step_kernel<T, NK, THREADS>, dim3(a.H, B), dim3(THREADS), smem, stream, a);
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+template <typename T>
+static int delta_step_launch(const DeltaArgs& a, int B, cudaStream_t stream) {
+  const int cols = a.V / 4;
+  if (a.V <= 256) {
+    const int nk = (a.K + 256 / cols - 1) / (256 / cols);
+    if (nk <= 4) return delta_step_go<T, 4, 256>(a, B, stream);
+    if (nk <= 8) return delta_step_go<T, 8, 256>(a, B, stream);
+    if (nk <= 16) return delta_step_go<T, 16, 256>(a, B, stream);
+    if (nk <= 32) return delta_step_go<T, 32, 256>(a, B, stream);
+  }
+  if (a.V <= 1024 && (a.K + 1024 / cols - 1) / (1024 / cols) <= 32) return delta_step_go<T, 32, 1024>(a, B, stream);
+  return (int)cudaErrorInvalidValue;
+}
+
+// Gated delta rule of a step: z [T, ld] holds q | k (G heads of K values) | v (H heads of V values) and, at the given columns,
+// gate, decay and beta; the state [num_slots, H, K, V] float32 is read and updated, the ring of convolution inputs [num_slots,
+// taps, channels] read.  Only sequences that feed min_rows .. max_rows rows take part.  write_window (single-row steps): the
+// ring is updated too; elsewhere oxb_delta_window does that afterwards.
+OXB_API int oxb_delta(const void* z, int ld, int dtype, int gate_off, int decay_off, int beta_off, const int* query_start,
+                      const int* seq_lens, const int* slots, const float* conv, int taps, const float* a_log, const float* dt_bias,
+                      const void* decay_up, int decay_rank, const void* gate_up, int gate_rank, const float* norm, float* state,
+                      float* window, int num_slots, void* out, int ld_out, float out_scale, int B, int H, int G, int K, int V,
+                      int v_dim, float q_scale, float eps, int min_rows, int max_rows, int write_window, cudaStream_t stream) {
+  if (B <= 0 || H <= 0) return 0;
+  if (G <= 0 || H % G != 0 || V % 4 != 0 || V <= 0 || K <= 0 || taps <= 0 || B > 65535 || slots == nullptr ||
+      (decay_up != nullptr && (decay_rank % 8 != 0 || decay_off % 8 != 0)) || (gate_up != nullptr && (gate_rank % 8 != 0 || gate_off % 8 != 0)) ||
+      ld % 8 != 0 || (reinterpret_cast<uintptr_t>(z) & 15) != 0)
+    return (int)cudaErrorInvalidValue;
+  const DeltaArgs a{z, ld, gate_off, decay_off, beta_off, query_start, seq_lens, slots, conv, taps, a_log, dt_bias, decay_up, decay_rank,
+                    gate_up, gate_rank, norm, state, window, num_slots, out, ld_out, out_scale, H, G, K, V, v_dim, q_scale, eps,
+                    min_rows, max_rows, write_window};
+  return dtype == 0 ? delta_step_launch<float>(a, B, stream) : delta_step_launch<__nv_bfloat16>(a, B, stream);
+}
+
+OXB_API int oxb_delta_window(const void* z, int ld, int dtype, const int* query_start, const int* seq_lens, const int* slots, int taps,
+                             float* window, int num_slots, int B, int H, int G, int K, int V, cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (taps <= 0 || B > 65535 || slots == nullptr) return (int)cudaErrorInvalidValue;
+  DeltaArgs a{};
+  a.z = z, a.ld = ld, a.query_start = query_start, a.seq_lens = seq_lens, a.slots = slots, a.taps = taps, a.window = window;
+  a.num_slots = num_slots, a.H = H, a.G = G, a.K = K, a.V = V;
+  const dim3 grid((2 * G * K + H * V + 255) / 256, B);
+  if (dtype == 0) oxb_launch(delta_window_kernel<float>, grid, dim3(256), 0, stream, a);
+  else oxb_launch(delta_window_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, a);
+  OXB_CHECK_LAUNCH();
+  return 0;
+}

@@ -412,9 +412,9 @@ OXB_API int oxb_gemm_batched(const void* X, const void* W, void* Y, long long y_
 // the token tile and the grid; CTAs past a group's rows leave at once).
 OXB_API int oxb_gemm_grouped_rows(const void* X, int rows_cap, const void* W, int qtype, size_t row_bytes, void* Y,
                                   const int* row_offsets, int groups, int max_rows, int N, int K, int ldY,
-                                  cudaStream_t stream) {
+                                  int epi, cudaStream_t stream) {
   if (rows_cap <= 0 || max_rows <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
-  if (K % 64 != 0 || row_offsets == nullptr) return (int)cudaErrorInvalidValue;
+  if (K % 64 != 0 || row_offsets == nullptr || (epi != EPI_STORE && epi != EPI_RELU2)) return (int)cudaErrorInvalidValue;
   const bool packed = qtype != QT_BF16;
   GemmPlan p = gemm_plan(max_rows, N, K, 0, sm_count(), 1, 0, packed, groups);
   if (p.splits > 1 && !p.cluster) p = gemm_plan(max_rows, N, K, 1, sm_count(), 1, 0, packed, groups);
@@ -430,14 +430,14 @@ OXB_API int oxb_gemm_grouped_rows(const void* X, int rows_cap, const void* W, in
     e = oxb_make_tmap_2d(&tmW, W, (uint64_t)groups * N, K, (uint64_t)K * 2, GEMM_BM, GEMM_BK, 2);
     if (e) return e;
     switch (p.tn) {
-      case 16: return gemm_launch<16>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
-      case 32: return gemm_launch<32>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
-      case 64: return gemm_launch<64>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
-      case 128: return gemm_launch<128>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
-      default: return gemm_launch<256>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr, groups);
+      case 16: return gemm_launch<16>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, epi, ar, stream, qw, gr, groups);
+      case 32: return gemm_launch<32>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, epi, ar, stream, qw, gr, groups);
+      case 64: return gemm_launch<64>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, epi, ar, stream, qw, gr, groups);
+      case 128: return gemm_launch<128>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, epi, ar, stream, qw, gr, groups);
+      default: return gemm_launch<256>(tmW, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, epi, ar, stream, qw, gr, groups);
     }
   }
   if (qtype == QT_FP8B) return (int)cudaErrorInvalidValue;
-  return launch_mmq(qtype, W, (uint64_t)groups * N, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, 0, ar, stream, qw, gr,
+  return launch_mmq(qtype, W, (uint64_t)groups * N, tmX, y, nullptr, N, max_rows, K, ldY, p, nullptr, nullptr, epi, ar, stream, qw, gr,
                     groups);
 }

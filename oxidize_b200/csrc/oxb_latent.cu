@@ -28,9 +28,9 @@ OXB_API int oxb_gemm_f32(const float* x, const float* w, float* y, const float* 
 // Routed groups: y[r] = x[perm[r]] . W_g^T for the rows r of every group g (offsets [groups + 1], perm null: x[r]);
 // max_rows bounds the rows of one group.
 OXB_API int oxb_gemm_f32_rows(const float* x, const float* w, float* y, const int* offsets, const int* perm, int groups,
-                              int max_rows, int N, int K, int ldx, int ldy, cudaStream_t stream) {
+                              int max_rows, int N, int K, int ldx, int ldy, int act, cudaStream_t stream) {
   if (max_rows <= 0 || N <= 0 || K <= 0 || groups <= 0) return 0;
-  const GemmF32Args a{x, w, nullptr, y, 0, N, K, ldx, K, ldy, 0, (long long)N * K, 0, 0, offsets, perm};
+  const GemmF32Args a{x, w, nullptr, y, 0, N, K, ldx, K, ldy, 0, (long long)N * K, 0, act, offsets, perm};
   oxb_launch(gemm_f32_kernel, dim3((N + F32_TILE - 1) / F32_TILE, (max_rows + F32_TILE - 1) / F32_TILE, groups), dim3(256), 0,
              stream, a);
   OXB_CHECK_LAUNCH();

@@ -15,6 +15,32 @@ OXB_API int oxb_branch_norm(const float* res, const void* y, const float* w_post
   return dtype == 0 ? branch_norm_launch<float>(a, T, stream) : branch_norm_launch<__nv_bfloat16>(a, T, stream);
 }
 
+OXB_API int oxb_joint_norm(const float* res, const void* y0, const void* y1, const float* w0, const float* w1, float s0, float s1,
+                           const void* f, int ldf, const int* index, const float* weights, int k, const float* w_next, float* x_out,
+                           void* a_out, int dtype, int T, int H, float eps, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if ((w0 != nullptr) != (w1 != nullptr) || (w0 != nullptr && (y0 == nullptr || y1 == nullptr))) return (int)cudaErrorInvalidValue;
+  const JointNormArgs a{res, y0, y1, w0, w1, s0, s1, f, index, weights, k, ldf, w_next, x_out, a_out, H, eps};
+  return dtype == 0 ? joint_norm_launch<float>(a, T, stream) : joint_norm_launch<__nv_bfloat16>(a, T, stream);
+}
+
+// o [T, ld] (H heads of W values, W a multiple of 4) times the sigmoid of its gates, in place
+OXB_API int oxb_head_gate(void* o, int ld, const void* gate, int ld_gate, int per_value, int dtype, int T, int H, int W,
+                          cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (W % 4 != 0 || ld % 4 != 0 || (per_value && ld_gate % 4 != 0)) return (int)cudaErrorInvalidValue;
+  const size_t blocks = ((size_t)T * H * W / 4 + 255) / 256;
+  const dim3 grid((unsigned)(blocks < 8192 ? blocks : 8192));
+  if (dtype == 0)
+    oxb_launch(head_gate_kernel<float>, grid, dim3(256), 0, stream, reinterpret_cast<float*>(o), ld, reinterpret_cast<const float*>(gate),
+               ld_gate, per_value, T, H, W);
+  else
+    oxb_launch(head_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, reinterpret_cast<__nv_bfloat16*>(o), ld,
+               reinterpret_cast<const __nv_bfloat16*>(gate), ld_gate, per_value, T, H, W);
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
 template <typename T>
 static int head_prep_launch(HeadPrepArgs a, int rows, cudaStream_t stream) {
   // few tokens: their heads are spread over CTAs, a head per warp
@@ -36,11 +62,14 @@ static int head_prep_launch(HeadPrepArgs a, int rows, cudaStream_t stream) {
 // Norms, rotation, queries and cache rows of a step's q | k | v projections (head_prep_kernel); width a multiple of 32.
 OXB_API int oxb_head_prep(const void* z, int ld, int dtype, const int* positions, const int* slots, const float* cos_sin, int max_pos,
                           int rot, int pairing, const float* q_norm, const float* k_norm, int full, float eps, int T, int H, int G,
-                          int dim, int width, void* q, void* cache, int page, int num_blocks, cudaStream_t stream) {
+                          int dim, int width, void* q, void* cache, int page, int num_blocks, float temp_coef, float temp_every,
+                          const void* v_first, int ld_first, int first_width, int v_dim, const float* v_mix, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (rot < 0 || rot % 2 != 0 || rot > width || width % 32 != 0 || page <= 0 || H <= 0 || G <= 0) return (int)cudaErrorInvalidValue;
+  if (rot < 0 || rot % 2 != 0 || rot > width || width % 32 != 0 || page <= 0 || H <= 0 || G <= 0 || (temp_coef != 0.f && !(temp_every > 0.f)) ||
+      (v_first != nullptr && (v_mix == nullptr || v_dim > first_width)))
+    return (int)cudaErrorInvalidValue;
   const HeadPrepArgs a{z, ld, positions, slots, cos_sin, max_pos, rot, pairing, q_norm, k_norm, full, eps, H, G, dim, width,
-                       q, cache, page, num_blocks, 0};
+                       q, cache, page, num_blocks, 0, temp_coef, temp_every, v_first, ld_first, first_width, v_dim, v_mix};
   return dtype == 0 ? head_prep_launch<float>(a, T, stream) : head_prep_launch<__nv_bfloat16>(a, T, stream);
 }
 

@@ -227,6 +227,162 @@ __global__ void __launch_bounds__(256) branch_norm_any_kernel(const BranchNormAr
     rn_store(reinterpret_cast<A*>(a.a_out) + base + i, rn_row[i] * inv * a.w_next[i]);
 }
 
+// Both branches of a layer join the stream and the next layer's norm follows, in one kernel:
+//     x = res + mixer + ffn,   a = rms(x) * w_next  in the activation type.
+// The mixer's output is y0, or s0 rms(y0) w0 + s1 rms(y1) w1 where two mixers have norms of their own; the feed-forward
+// output is f, or the weighted sum of routed rows, sum_j weights[t, j] f[index[t, j]].
+struct JointNormArgs {
+  const float* res;     // [T, H]
+  const void *y0, *y1;  // [T, H] in the activation type, or null
+  const float *w0, *w1; // [H]; null: y0 as it is
+  float s0, s1;
+  const void* f;        // [T, H], or rows ldf apart with index; or null
+  const int* index;     // [T, k] or null; < 0: none
+  const float* weights; // [T, k]
+  int k, ldf;
+  const float* w_next;  // [H] or null: the sum alone
+  float* x_out;         // [T, H] or null
+  void* a_out;          // [T, H] in the activation type, or null
+  int H;
+  float eps;
+};
+
+// One CTA per row; every thread owns CH groups of four neighbouring values (H % 4 == 0, H <= 4 * CH * threads).
+template <typename A, int CH>
+__global__ void __launch_bounds__(1024) joint_norm_kernel(const JointNormArgs a) {
+  __shared__ float red[32];
+  const int H4 = a.H >> 2, t = blockIdx.x;
+  const size_t base = (size_t)t * a.H;
+  float4 v[CH], n[CH];
+  pdl_launch_dependents();
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {  // weights are static: fetched ahead of the dependency
+    const int i = threadIdx.x + c * blockDim.x;
+    n[c] = (i < H4 && a.w_next != nullptr) ? rn_load4(a.w_next + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H4) v[c] = rn_load4(a.res + base + 4 * i);
+  }
+  if (a.f != nullptr) {
+    const A* f = reinterpret_cast<const A*>(a.f);
+    const int k = a.index != nullptr ? a.k : 1;
+    for (int j = 0; j < k; ++j) {
+      const int r = a.index != nullptr ? a.index[(size_t)t * k + j] : t;
+      if (r < 0) continue;
+      const float w = a.index != nullptr ? a.weights[(size_t)t * k + j] : 1.f;
+#pragma unroll
+      for (int c = 0; c < CH; ++c) {
+        const int i = threadIdx.x + c * blockDim.x;
+        if (i < H4) {
+          const float4 y = rn_load4(f + (size_t)r * a.ldf + 4 * i);
+          v[c] = make_float4(fmaf(w, y.x, v[c].x), fmaf(w, y.y, v[c].y), fmaf(w, y.z, v[c].z), fmaf(w, y.w, v[c].w));
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int side = 0; side < 2; ++side) {
+    const A* yp = reinterpret_cast<const A*>(side == 0 ? a.y0 : a.y1);
+    const float* wp = side == 0 ? a.w0 : a.w1;
+    if (yp == nullptr) continue;
+    float4 y[CH];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int i = threadIdx.x + c * blockDim.x;
+      y[c] = i < H4 ? rn_load4(yp + base + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += (y[c].x * y[c].x + y[c].y * y[c].y) + (y[c].z * y[c].z + y[c].w * y[c].w);
+    }
+    const float inv = wp != nullptr ? rsqrtf(block_sum(ss, red) / (float)a.H + a.eps) * (side == 0 ? a.s0 : a.s1) : 1.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int i = threadIdx.x + c * blockDim.x;
+      if (i >= H4) continue;
+      const float4 w = wp != nullptr ? rn_load4(wp + 4 * i) : make_float4(1.f, 1.f, 1.f, 1.f);
+      v[c] = make_float4(v[c].x + y[c].x * inv * w.x, v[c].y + y[c].y * inv * w.y, v[c].z + y[c].z * inv * w.z,
+                         v[c].w + y[c].w * inv * w.w);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    if (i < H4 && a.x_out != nullptr) rn_store4(a.x_out + base + 4 * i, v[c]);
+    ss += (v[c].x * v[c].x + v[c].y * v[c].y) + (v[c].z * v[c].z + v[c].w * v[c].w);
+  }
+  if (a.a_out == nullptr) return;
+  const float inv = rsqrtf(block_sum(ss, red) / (float)a.H + a.eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    if (i < H4)
+      rn_store4(reinterpret_cast<A*>(a.a_out) + base + 4 * i,
+                make_float4(v[c].x * inv * n[c].x, v[c].y * inv * n[c].y, v[c].z * inv * n[c].z, v[c].w * inv * n[c].w));
+  }
+}
+
+// Any width: the row is staged in shared memory (dynamic, H floats).
+template <typename A>
+__global__ void __launch_bounds__(256) joint_norm_any_kernel(const JointNormArgs a) {
+  extern __shared__ float rn_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const size_t base = (size_t)t * a.H;
+  const A *y0 = reinterpret_cast<const A*>(a.y0), *y1 = reinterpret_cast<const A*>(a.y1), *f = reinterpret_cast<const A*>(a.f);
+  float i0 = 1.f, i1 = 1.f;
+  if (a.w0 != nullptr) {
+    float ss0 = 0.f, ss1 = 0.f;
+    for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+      const float u = rn_load(y0 + base + i), w = rn_load(y1 + base + i);
+      ss0 += u * u;
+      ss1 += w * w;
+    }
+    i0 = rsqrtf(block_sum(ss0, red) / (float)a.H + a.eps) * a.s0;
+    i1 = rsqrtf(block_sum(ss1, red) / (float)a.H + a.eps) * a.s1;
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    float v = a.res[base + i];
+    if (f != nullptr && a.index == nullptr) v += rn_load(f + (size_t)t * a.ldf + i);
+    if (f != nullptr && a.index != nullptr)
+      for (int j = 0; j < a.k; ++j) {
+        const int r = a.index[(size_t)t * a.k + j];
+        if (r >= 0) v = fmaf(a.weights[(size_t)t * a.k + j], rn_load(f + (size_t)r * a.ldf + i), v);
+      }
+    if (y0 != nullptr) v += rn_load(y0 + base + i) * i0 * (a.w0 != nullptr ? a.w0[i] : 1.f);
+    if (y1 != nullptr) v += rn_load(y1 + base + i) * i1 * (a.w1 != nullptr ? a.w1[i] : 1.f);
+    rn_row[i] = v;
+    if (a.x_out != nullptr) a.x_out[base + i] = v;
+    ss += v * v;
+  }
+  if (a.a_out == nullptr) return;
+  const float inv = rsqrtf(block_sum(ss, red) / (float)a.H + a.eps);
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x)
+    rn_store(reinterpret_cast<A*>(a.a_out) + base + i, rn_row[i] * inv * a.w_next[i]);
+}
+
+template <typename A>
+int joint_norm_launch(const JointNormArgs& a, int T, cudaStream_t stream) {
+  if (a.H % 4 == 0 && a.ldf % 4 == 0 && a.H <= 16384) {
+    const int H4 = a.H / 4, lim = T >= 512 ? 256 : 1024, ch = H4 <= lim ? 1 : (H4 <= 2 * lim ? 2 : 4);
+    const int threads = ((H4 + ch - 1) / ch + 31) / 32 * 32;
+    if (ch == 1) oxb_launch(joint_norm_kernel<A, 1>, dim3(T), dim3(threads), 0, stream, a);
+    else if (ch == 2) oxb_launch(joint_norm_kernel<A, 2>, dim3(T), dim3(threads), 0, stream, a);
+    else oxb_launch(joint_norm_kernel<A, 4>, dim3(T), dim3(threads), 0, stream, a);
+  } else {
+    if (a.H > 12 * 1024) return (int)cudaErrorInvalidValue;  // 48 KB of shared memory
+    oxb_launch(joint_norm_any_kernel<A>, dim3(T), dim3(256), (size_t)a.H * sizeof(float), stream, a);
+  }
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
 template <typename A>
 int branch_norm_launch(const BranchNormArgs& a, int T, cudaStream_t stream) {
   if (a.H % 4 == 0 && a.H <= 16384) {

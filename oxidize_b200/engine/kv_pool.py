@@ -271,11 +271,20 @@ class StateSlots:
 
 
 class StateStore:
-    """Device storage of the recurrent states: data[layer] [num_slots, heads, keys, values] float32."""
+    """Device storage of the recurrent states: data[layer] [num_slots, heads, keys, values] float32, and for layers with short
+    convolutions the last inputs of those, windows[layer] [num_slots, tokens, channels] float32 (None elsewhere)."""
 
-    def __init__(self, shapes: Sequence[Tuple[int, int, int]], num_slots: int, device="cpu"):
+    def __init__(self, shapes: Sequence[Tuple[int, int, int]], num_slots: int, device="cpu",
+                 windows: Optional[Sequence[Optional[Tuple[int, int]]]] = None):
         self.num_slots = num_slots
-        self.data = [torch.zeros((num_slots,) + tuple(s), dtype=torch.float32, device=device) for s in shapes]
+        new = lambda s: None if s is None else torch.zeros((num_slots,) + tuple(s), dtype=torch.float32, device=device)
+        self.data = [new(s) for s in shapes]
+        self.windows = [new(s) for s in (windows or [None] * len(self.data))]
+
+    @staticmethod
+    def slot_bytes(shapes, windows) -> int:
+        """Bytes of one sequence."""
+        return 4 * (sum(h * k * v for h, k, v in shapes) + sum(w[0] * w[1] for w in windows if w is not None))
 
     def nbytes(self) -> int:
-        return sum(d.numel() * 4 for d in self.data)
+        return sum(d.numel() * 4 for d in self.data + [w for w in self.windows if w is not None])

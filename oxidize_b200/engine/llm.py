@@ -22,7 +22,7 @@ from ..models.registry import act_dtype_for, config_from_checkpoint, load_checkp
 from ..models.transformer import Transformer
 from ..models.weights import ModelWeights
 from ..utils import profiler as _profiler
-from .kv_pool import BlockPool, KVCacheSpec, StateSlots, make_block_pool
+from .kv_pool import BlockPool, KVCacheSpec, StateSlots, StateStore, make_block_pool
 from .runner import ModelRunner, StepResult
 from .sampler import SamplingParams
 from .scheduler import ScheduledSeq, Scheduler, SchedulerConfig, SchedulerOutput, Sequence
@@ -187,7 +187,7 @@ class LLM:
             return max(16, min(want, 4096))
         free, total = torch.cuda.mem_get_info(self.device)
         budget = int(free - (1.0 - c.gpu_memory_utilization) * total)
-        budget -= 4 * c.max_num_seqs * sum(h * k * v for h, k, v in self.cfg.state_shapes)
+        budget -= c.max_num_seqs * StateStore.slot_bytes(self.cfg.state_shapes, self.cfg.state_windows)
         fit = max(16, budget // max(spec.bytes_per_block() + extra_bytes_per_block, 1))
         return int(min(want, fit))
 

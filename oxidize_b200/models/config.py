@@ -127,23 +127,37 @@ class LatentAttentionSpec:
 HEAD_WIDTHS = (32, 64, 96, 128, 192, 256)
 
 
+def pad_to(n: int, unit: int) -> int:
+    return (n + unit - 1) // unit * unit
+
+
 @dataclass
 class AttentionSpec:
     """Grouped-query attention with the geometry of a single layer.
 
     ``window`` > 0 limits a query to that many latest positions (itself included); ``sink`` adds a learned per-head logit
     to the softmax denominator only; ``qk_norm`` is an RMS norm of the queries and keys ahead of the rotation, per ``head``
-    (one weight for all heads) or over the ``full`` projection."""
+    (one weight for all heads) or over the ``full`` projection; ``rotary`` None: queries and keys are not rotated.
+    ``temp_coef`` != 0: a query at position p is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1).
+    ``v_mix``: the values are mixed, v <- (1 - lambda) v + lambda v_first, with those that the first such layer of the model
+    has for the same token (lambda is a weight of the layer; the first layer's values stay as they are).  ``gate``: the
+    outputs are multiplied by the sigmoid of a projection of the layer's input, one value per ``head`` or per output
+    ``value``.  ``bias``: the q, k and v projections have one."""
 
     heads: int
     kv_heads: int
     dim: int
     v_dim: int
     scale: float
-    rotary: RotarySpec
+    rotary: Optional[RotarySpec]
     window: int = 0
     sink: bool = False
     qk_norm: str = ""  # "" | head | full
+    bias: bool = False
+    temp_coef: float = 0.0
+    temp_every: float = 1.0
+    v_mix: bool = False
+    gate: str = ""  # "" | head | value
 
     kv_from = None  # (every layer of this kind owns cache rows)
 
@@ -162,8 +176,17 @@ class AttentionSpec:
         return self.heads * self.width
 
     @property
-    def proj_dim(self) -> int:
+    def qkv_dim(self) -> int:
         return (self.heads + 2 * self.kv_heads) * self.width
+
+    @property
+    def gate_dim(self) -> int:
+        return {"": 0, "head": pad_to(self.heads, 8), "value": self.heads * self.width}[self.gate]
+
+    @property
+    def proj_dim(self) -> int:
+        """Columns of the projections of the layer's input: q | k | v | gate."""
+        return self.qkv_dim + self.gate_dim
 
 
 @dataclass
@@ -201,13 +224,77 @@ class RetentionSpec:
 
 
 @dataclass
+class DeltaSpec:
+    """Linear attention with the gated delta rule: S <- g S; S <- S + k (beta (v - S^T k))^T; o = S^T q.
+
+    q, k and v pass a short causal convolution over ``conv`` tokens and silu, q and k are then unit vectors per head (q also
+    times dim ** -0.5); consecutive heads share a q / k head.  The decay is g = exp(-exp(A_log) softplus(a + dt_bias)): one per
+    head, or with ``decay_rank`` > 0 one per key channel from two projections through that many values.  Each head's o is
+    divided by its root mean square, weighted, and gated by the silu of a projection of the input, or with ``gate_rank`` > 0 by
+    the sigmoid of two projections through that many values.  Every sequence carries one [dim, v_dim] float32 state per head
+    and the last inputs of the convolutions."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    v_dim: int
+    conv: int
+    decay_rank: int = 0
+    gate_rank: int = 0
+
+    rotary = None  # (positions enter through the recurrence alone)
+
+    # head widths in projections, state and outputs (the padding is zero)
+    @property
+    def k_width(self) -> int:
+        return next((w for w in HEAD_WIDTHS if w >= self.dim), pad_to(self.dim, 32))
+
+    @property
+    def v_width(self) -> int:
+        return pad_to(self.v_dim, 16)
+
+    @property
+    def state_shape(self) -> Tuple[int, int, int]:
+        return self.heads, self.k_width, self.v_width
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.v_width
+
+    @property
+    def channels(self) -> int:
+        """Channels of the convolutions: q | k | v."""
+        return 2 * self.kv_heads * self.k_width + self.heads * self.v_width
+
+    @property
+    def window_shape(self) -> Tuple[int, int]:
+        """Convolution inputs kept per sequence: position p's row is row p % conv."""
+        return self.conv, self.channels
+
+    # columns of the projections of the layer's input: q | k | v | gate | decay | beta
+    @property
+    def gate_dim(self) -> int:
+        return pad_to(self.gate_rank, 16) if self.gate_rank else self.out_dim
+
+    @property
+    def decay_dim(self) -> int:
+        return pad_to(self.decay_rank, 16) if self.decay_rank else pad_to(self.heads, 8)
+
+    @property
+    def proj_dim(self) -> int:
+        return self.channels + self.gate_dim + self.decay_dim + pad_to(self.heads, 8)
+
+
+@dataclass
 class ParallelSpec:
-    """Attention and retention side by side on the same input: left_scale * left + right_scale * right."""
+    """Attention and a recurrent mixer side by side on the same input: left_scale * left + right_scale * right; with
+    ``norms`` each side's projected output first passes an RMS norm of its own."""
 
     left: AttentionSpec
-    right: RetentionSpec
+    right: Union[RetentionSpec, DeltaSpec]
     left_scale: float = 1.0
     right_scale: float = 1.0
+    norms: bool = False
 
 
 @dataclass
@@ -226,8 +313,10 @@ class FeedForwardSpec:
 
 @dataclass
 class MoESpec:
-    """Routed experts: the ``n_experts_used`` largest router logits choose, their softmax weighs; ``shared`` runs for every
-    token and is added.  (The routing fields carry the names that the routing operators read from ``ModelConfig``.)"""
+    """Routed experts: the ``n_experts_used`` largest scores choose, the chosen scores divided by their sum weigh (with
+    softmax scores: the softmax over the chosen logits); ``correction`` adds a learned offset per expert to the scores that
+    choose; ``shared`` runs for every token and is added.  (The routing fields carry the names that the routing operators read
+    from ``ModelConfig``.)"""
 
     n_experts: int
     n_experts_used: int
@@ -238,6 +327,7 @@ class MoESpec:
     expert_weights_scale: float = 1.0
     expert_group_count: int = 0
     expert_group_used_count: int = 0
+    correction: bool = False
 
     @property
     def size(self) -> int:
@@ -249,7 +339,7 @@ class MoESpec:
 class LayerSpec:
     """One decoder layer of a model whose layers are listed one by one."""
 
-    mixer: Union[LatentAttentionSpec, AttentionSpec, RetentionSpec, ParallelSpec]
+    mixer: Union[LatentAttentionSpec, AttentionSpec, RetentionSpec, DeltaSpec, ParallelSpec]
     ffn: Union[FeedForwardSpec, MoESpec, None] = None  # None: the layer has no feed-forward block
     weights_of: Optional[int] = None  # an earlier layer whose weights this one uses (with cache rows and state of its own)
 
@@ -257,13 +347,23 @@ class LayerSpec:
     def attention(self) -> Union[LatentAttentionSpec, AttentionSpec, None]:
         """The part of the mixer that attends over cached rows."""
         m = self.mixer
-        return m.left if isinstance(m, ParallelSpec) else None if isinstance(m, RetentionSpec) else m
+        return m.left if isinstance(m, ParallelSpec) else None if isinstance(m, (RetentionSpec, DeltaSpec)) else m
+
+    @property
+    def recurrent(self) -> Union[RetentionSpec, DeltaSpec, None]:
+        """The part of the mixer that carries a recurrent state."""
+        m = self.mixer
+        return m.right if isinstance(m, ParallelSpec) else m if isinstance(m, (RetentionSpec, DeltaSpec)) else None
 
     @property
     def retention(self) -> Optional[RetentionSpec]:
-        """The part of the mixer that carries a recurrent state."""
-        m = self.mixer
-        return m.right if isinstance(m, ParallelSpec) else m if isinstance(m, RetentionSpec) else None
+        r = self.recurrent
+        return r if isinstance(r, RetentionSpec) else None
+
+    @property
+    def delta(self) -> Optional[DeltaSpec]:
+        r = self.recurrent
+        return r if isinstance(r, DeltaSpec) else None
 
     @property
     def owns_rows(self) -> bool:
@@ -276,7 +376,12 @@ class LayerSpec:
 
     @property
     def out_dim(self) -> int:
-        return sum(p.out_dim for p in (self.attention, self.retention) if p is not None)
+        return sum(p.out_dim for p in (self.attention, self.recurrent) if p is not None)
+
+    @property
+    def in_dim(self) -> int:
+        """Columns of the projections of the layer's input (not of latent attention)."""
+        return sum(p.proj_dim for p in (self.attention, self.recurrent) if p is not None)
 
 
 @dataclass
@@ -366,8 +471,9 @@ class ModelConfig:
     # > 0: norm after the sum, x <- norm(residual_alpha * x + branch(x)), with the residual stream in float32;
     # 0: norm in front of the branch, x <- x + branch(norm(x))
     residual_alpha: float = 0.0
-    # Listed layers only: "after_sum" (the rule above), or "sandwich": norms on both sides of the branch,
-    # x <- x + norm_b(branch(norm_a(x))), with the residual stream in float32
+    # Listed layers only: "after_sum" (the rule above); "sandwich": norms on both sides of the branch,
+    # x <- x + norm_b(branch(norm_a(x))); "parallel": one norm that both branches read, x <- x + mixer(h) + ffn(h) with
+    # h = norm(x).  The residual stream is in float32 in all three
     norm_placement: str = "after_sum"
     embed_norm: bool = False  # the embedding passes a norm of its own
 
@@ -391,12 +497,17 @@ class ModelConfig:
     @property
     def state_shapes(self) -> List[Tuple[int, int, int]]:
         """Recurrent state of a sequence, one [heads, keys, values] per layer that carries one."""
-        return [l.retention.state_shape for l in self.layer_specs if l.retention is not None]
+        return [l.recurrent.state_shape for l in self.layer_specs if l.recurrent is not None]
+
+    @property
+    def state_windows(self) -> List[Optional[Tuple[int, int]]]:
+        """Convolution inputs of a sequence, one [tokens, channels] (or None) per layer with a recurrent state."""
+        return [getattr(l.recurrent, "window_shape", None) for l in self.layer_specs if l.recurrent is not None]
 
     @property
     def has_state(self) -> bool:
         """Sequences carry a recurrent state, which cannot be rebuilt from shared pages or rolled back."""
-        return self.is_ssm or any(l.retention is not None for l in self.layer_specs)
+        return self.is_ssm or any(l.recurrent is not None for l in self.layer_specs)
 
     @property
     def uniform_window(self) -> int:
@@ -456,24 +567,34 @@ class ModelConfig:
 
         def ffn(f) -> int:
             if isinstance(f, MoESpec):
-                return f.n_experts * (ffn(f.expert) + h) + (ffn(f.shared) if f.shared else 0)
+                return f.n_experts * (ffn(f.expert) + h + f.correction) + (ffn(f.shared) if f.shared else 0)
             return (3 if f.gated else 2) * h * f.size
 
-        n = 2 * self.vocab_size * h + (2 if self.embed_norm else 1) * norm
+        n = (1 if self.tie_embeddings else 2) * self.vocab_size * h + (2 if self.embed_norm else 1) * norm
         for l in self.layer_specs:
             if l.weights_of is not None:
                 continue
-            a, r = l.attention, l.retention
-            per_branch = 2 * norm if self.norm_placement == "sandwich" else norm
-            n += per_branch * (1 if l.ffn is None else 2) + (0 if l.ffn is None else ffn(l.ffn))
+            a, r, d = l.attention, l.retention, l.delta
+            if self.norm_placement == "parallel":
+                n += norm * (3 if isinstance(l.mixer, ParallelSpec) and l.mixer.norms else 1)
+            else:
+                n += (2 * norm if self.norm_placement == "sandwich" else norm) * (1 if l.ffn is None else 2)
+            n += 0 if l.ffn is None else ffn(l.ffn)
             if isinstance(a, LatentAttentionSpec):
                 n += a.heads * (h * (a.qk_dim + a.v_dim) + a.kv_rank * (a.nope_dim + a.v_dim))
                 n += 0 if a.kv_from is not None else h * (a.kv_rank + a.rope_dim) + a.kv_rank
             elif a is not None:
                 n += h * (a.heads + a.kv_heads) * (a.dim + a.v_dim)
                 n += {"": 0, "head": 2, "full": a.heads + a.kv_heads}[a.qk_norm] * a.dim
+                n += ((a.heads + a.kv_heads) * a.dim + a.kv_heads * a.v_dim if a.bias else 0) + a.v_mix
+                n += {"": 0, "head": a.heads, "value": a.heads * a.v_dim}[a.gate] * h
             n += a.heads if a is not None and a.sink else 0
             n += h * r.heads * (2 * r.dim + 3 * r.v_dim) if r is not None else 0
+            if d is not None:
+                qk, v = d.kv_heads * d.dim, d.heads * d.v_dim
+                n += (2 * qk + v) * (h + d.conv) + h * (v + d.heads) + d.heads + d.v_dim
+                n += d.decay_rank * (h + d.heads * d.dim) + d.heads * d.dim if d.decay_rank else (h + 1) * d.heads
+                n += d.gate_rank * (h + v) if d.gate_rank else h * v
         return n
 
     def to_dict(self) -> Dict[str, Any]:

@@ -10,7 +10,13 @@ ungated squared-relu feed-forward blocks; the embedding and the output pass norm
 Sokirax: RMS norms on both sides of every branch, x <- x + norm_b(branch(norm_a(x))); grouped-query attention in a window
 (per-head q / k norm, partial YaRN rotation), or such attention (norm over the whole projection, a softmax sink per head)
 beside retention on the same input; gated feed-forward blocks, dense or routed experts with a shared one; a layer may use an
-earlier layer's weights."""
+earlier layer's weights.
+
+Pavatar: one RMS norm that mixer and feed-forward block both read, x <- x + mixer(h) + ffn(h); unrotated attention (biases,
+a query factor that grows with the position, values mixed with an earlier layer's, a gate per head), the gated delta rule with
+a decay per head, or rotated attention (q / k norms, a gate per output value) beside the gated delta rule with a decay per key
+channel, each side with a norm of its own; routed squared-relu experts with a correction of the choice; a scaled embedding that
+is the output head as well, and soft-capped logits."""
 from __future__ import annotations
 
 import math
@@ -20,10 +26,10 @@ import numpy as np
 import torch
 
 from ..formats.layered import LayeredCheckpoint
-from .config import (AttentionSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, ModelConfig, MoESpec, ParallelSpec,
-                     RetentionSpec, RopeScaling, RotarySpec, UnsupportedArchitecture)
-from .weights import (ExpertWeights, LayerWeights, LinearWeight, MLAWeights, ModelWeights, QTensor, StreamedLayers,
-                      shard_range)
+from .config import (AttentionSpec, DeltaSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, ModelConfig, MoESpec,
+                     ParallelSpec, RetentionSpec, RopeScaling, RotarySpec, UnsupportedArchitecture, pad_to)
+from .weights import (DeltaWeights, ExpertWeights, LayerWeights, LinearWeight, MLAWeights, ModelWeights, QTensor,
+                      StreamedLayers, shard_range)
 
 
 # --------------------------------------------------------------------------- configuration
@@ -87,14 +93,14 @@ def _vefilix_config(ck: LayeredCheckpoint) -> ModelConfig:
                           residual_alpha=float(c["postln_alpha"]), embed_norm=True, name=str(ck.get("general.name", "")))
 
 
-def _attention(m: Dict[str, Any], qk_norm: str, sink: bool, layer: int) -> AttentionSpec:
+def _attention(m: Dict[str, Any], qk_norm: str, sink: bool, layer: int, **kw) -> AttentionSpec:
     mask = m.get("mask") or {}
     a = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), v_dim=int(m["vdim"]),
-                      scale=float(m["scale"]), rotary=_rotary(m["rot"]), window=int(mask.get("size") or 0), sink=sink,
-                      qk_norm=qk_norm)
+                      scale=float(m["scale"]), rotary=_rotary(m["rot"]) if m.get("rot") else None,
+                      window=int(mask.get("size") or 0), sink=sink, qk_norm=qk_norm, **kw)
     if a.heads % a.kv_heads:
         raise UnsupportedArchitecture(f"layer {layer}: {a.heads} query heads over {a.kv_heads} key / value heads")
-    if a.rotary.dims % 2 or a.rotary.dims > a.dim:
+    if a.rotary is not None and (a.rotary.dims % 2 or a.rotary.dims > a.dim):
         raise UnsupportedArchitecture(f"layer {layer}: rotation of {a.rotary.dims} of {a.dim} values per head")
     return a
 
@@ -156,21 +162,89 @@ def _sokirax_config(ck: LayeredCheckpoint) -> ModelConfig:
                           norm_placement="sandwich", name=str(ck.get("general.name", "")))
 
 
+def _unrotated(m: Dict[str, Any], layer: int) -> AttentionSpec:
+    t = m.get("q_temp") or {}
+    a = _attention(dict(m, rot=None), "", False, layer, bias=True, temp_coef=float(t.get("coef", 0.0)),
+                   temp_every=float(t.get("every", 1.0)), v_mix=bool(m.get("v_mix")), gate="head")
+    if not a.temp_every > 0:
+        raise ValueError(f"layer {layer}: query temperature every {a.temp_every} positions")
+    return a
+
+
+def _delta(ck: LayeredCheckpoint, m: Dict[str, Any], prefix: str, layer: int, low_rank: bool) -> DeltaSpec:
+    rank = (lambda n: int(ck.tensors[f"{prefix}{n}"].shape[0])) if low_rank else (lambda n: 0)
+    d = DeltaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]), rank("a1"), rank("g1"))
+    if d.heads % d.kv_heads:
+        raise UnsupportedArchitecture(f"layer {layer}: {d.heads} value heads over {d.kv_heads} query / key heads")
+    if d.conv < 1:
+        raise ValueError(f"layer {layer}: a convolution over {d.conv} tokens")
+    return d
+
+
+def _corrected_experts(f: Optional[Dict[str, Any]], layer: int) -> Optional[MoESpec]:
+    if f is None:
+        return None
+    if f.get("kind") != "moe":
+        raise UnsupportedArchitecture(f"layer {layer}: feed-forward kind {f.get('kind')!r}")
+    r = f["router"]
+    m = MoESpec(int(r["experts"]), int(r["top"]), FeedForwardSpec(int(f["expert"]["ff"]), "relu2"),
+                expert_weights_scale=float(r.get("scale", 1.0)), correction=True)
+    if not 1 <= m.n_experts_used <= m.n_experts:
+        raise ValueError(f"layer {layer}: {m.n_experts_used} of {m.n_experts} experts per token")
+    return m
+
+
+def check_value_mixing(specs: List[LayerSpec]) -> None:
+    """Layers that mix their values with the first such layer's have values of its geometry."""
+    mixed = [(i, l.attention) for i, l in enumerate(specs) if isinstance(l.attention, AttentionSpec) and l.attention.v_mix]
+    for i, a in mixed:
+        f = mixed[0][1]
+        if (a.kv_heads, a.v_dim) != (f.kv_heads, f.v_dim):
+            raise ValueError(f"layer {i} mixes values of {a.kv_heads} x {a.v_dim} with layer {mixed[0][0]}'s of "
+                             f"{f.kv_heads} x {f.v_dim}")
+
+
+def _pavatar_config(ck: LayeredCheckpoint) -> ModelConfig:
+    c = ck.config
+    specs = []
+    for i, l in enumerate(c["layers"]):
+        m, p = l["mixer"], f"l{i}.mix."
+        if l.get("type") == "attention":
+            mixer = _unrotated(m, i)
+        elif l.get("type") == "delta":
+            mixer = _delta(ck, m, p, i, False)
+        elif l.get("type") == "parallel":
+            mixer = ParallelSpec(_attention(m["left"], "head", False, i, gate="value"), _delta(ck, m["right"], p + "right.", i, True),
+                                 0.5, 0.5, norms=True)
+        else:
+            raise UnsupportedArchitecture(f"layer {i}: mixer type {l.get('type')!r}")
+        specs.append(LayerSpec(mixer, _corrected_experts(l.get("mlp"), i)))
+    check_value_mixing(specs)
+    cfg = layered_config("pavatar", int(c["vocab"]), int(c["width"]), specs, eps=float(c["norm"]["eps"]), norm_kind="rms",
+                         norm_placement="parallel", name=str(ck.get("general.name", "")))
+    cfg.embedding_scale = float((c.get("embedding") or {}).get("scale") or 1.0)
+    cfg.final_softcap = float(c.get("logit_softcap") or 0.0)
+    cfg.tie_embeddings = True
+    return cfg
+
+
 def layered_config(arch: str, vocab: int, width: int, specs: List[LayerSpec], eps: float, norm_kind: str,
                    residual_alpha: float = 1.0, embed_norm: bool = False, name: str = "",
                    norm_placement: str = "after_sum") -> ModelConfig:
     atts = [l.attention for l in specs if l.attention is not None]
-    m0 = atts[0] if atts else specs[0].retention
+    m0 = atts[0] if atts else specs[0].recurrent
+    rot = next((p.rotary for l in specs for p in (l.attention, l.recurrent) if p is not None and p.rotary is not None), None)
     ffn = max([l.ffn.size for l in specs if l.ffn is not None], default=0)
     return ModelConfig(arch=arch, name=name, vocab_size=vocab, hidden_size=width, n_layers=len(specs), n_heads=m0.heads,
                        n_kv_heads=max([a.kv_heads for a in atts], default=1),
                        head_dim=max([a.cache_shape[2] for a in atts], default=16), ffn_size=ffn, rms_eps=eps,
-                       rope_theta=m0.rotary.base, rope_dim=m0.rotary.dims, attn_scale=getattr(m0, "scale", 0.0),
+                       rope_theta=rot.base if rot else 10000.0, rope_dim=rot.dims if rot else 0, attn_scale=getattr(m0, "scale", 0.0),
                        context_length=1 << 20, layer_specs=specs, norm_kind=norm_kind, residual_alpha=residual_alpha,
                        embed_norm=embed_norm, norm_placement=norm_placement)
 
 
-READERS: Dict[str, Callable[[LayeredCheckpoint], ModelConfig]] = {"vefilix": _vefilix_config, "sokirax": _sokirax_config}
+READERS: Dict[str, Callable[[LayeredCheckpoint], ModelConfig]] = {"vefilix": _vefilix_config, "sokirax": _sokirax_config,
+                                                                      "pavatar": _pavatar_config}
 
 
 def config_from_layered(ck: LayeredCheckpoint) -> ModelConfig:
@@ -233,15 +307,55 @@ def pad_heads(t: torch.Tensor, heads: int, width: int, dim: int = 0) -> torch.Te
     return torch.cat([parts, pad], dim=dim + 1).reshape(shape[:dim] + [heads * width] + shape[dim + 1 :])
 
 
-def listed_mixer(spec: LayerSpec, att: Dict[str, torch.Tensor], ret: Dict[str, torch.Tensor]) -> Dict[str, Any]:
-    """Attention and / or retention tensors (as stored) of one layer in the layout the forward pass uses: one matrix over
-    the layer's input, attention q | k | v then retention q | k | v | gate, and one output matrix over both mixers' heads,
-    every head padded with zeros to its kernel width."""
+def pad_rows(t: torch.Tensor, rows: int) -> torch.Tensor:
+    """``t`` followed by zero rows up to ``rows``."""
+    return t if t.shape[0] == rows else torch.cat([t, t.new_zeros(rows - t.shape[0], *t.shape[1:])])
+
+
+def pad_cols(t: torch.Tensor, cols: int) -> torch.Tensor:
+    return torch.nn.functional.pad(t, (0, cols - t.shape[1])).contiguous()
+
+
+def delta_weights(d: DeltaSpec, t: Dict[str, torch.Tensor], act_dtype: torch.dtype) -> Tuple[List[torch.Tensor], DeltaWeights]:
+    """Delta-rule tensors (as stored) in the layout the forward pass uses: (rows over the layer's input q | k | v | gate |
+    decay | beta, what acts behind them)."""
+    K, V, H, G = d.k_width, d.v_width, d.heads, d.kv_heads
+    ins = [pad_heads(t["q"], G, K), pad_heads(t["k"], G, K), pad_heads(t["v"], H, V)]
+    taps = torch.cat([pad_heads(t["q.conv"].float(), G, K), pad_heads(t["k.conv"].float(), G, K), pad_heads(t["v.conv"].float(), H, V)])
+    w = DeltaWeights(conv=taps.t().contiguous(), a_log=t["A_log"].float().contiguous(),
+                     norm=torch.nn.functional.pad(t["norm"].float(), (0, V - d.v_dim)).contiguous(), dt_bias=t["dt_bias"].float().contiguous())
+    if d.gate_rank:
+        ins.append(pad_rows(t["g1"], d.gate_dim))
+        w.gate_up = pad_cols(pad_heads(t["g2"], H, V), d.gate_dim).to(act_dtype)
+    else:
+        ins.append(pad_heads(t["g"], H, V))
+    if d.decay_rank:
+        ins.append(pad_rows(t["a1"], d.decay_dim))
+        w.decay_up = pad_cols(pad_heads(t["a2"], H, K), d.decay_dim).to(act_dtype)
+        w.dt_bias = pad_heads(w.dt_bias, H, K).contiguous()
+    else:
+        ins.append(pad_rows(t["a"], d.decay_dim))
+    ins.append(pad_rows(t["b"], pad_to(H, 8)))
+    return ins, w
+
+
+def listed_mixer(spec: LayerSpec, att: Dict[str, torch.Tensor], rec: Dict[str, torch.Tensor]) -> Dict[str, Any]:
+    """Attention and / or recurrent tensors (as stored) of one layer in the layout the forward pass uses: one matrix over
+    the layer's input, attention q | k | v | gate then retention q | k | v | gate or the delta rule's rows, and one output
+    matrix over both mixers' heads (two where each side's output has a norm of its own), every head padded with zeros to its
+    kernel width."""
     ins, outs, kw = [], [], {}
-    a, r = spec.attention, spec.retention
+    a, r, d = spec.attention, spec.retention, spec.delta
+    ret, bias = rec, None
     if a is not None:
         for n, heads in (("q", a.heads), ("k", a.kv_heads), ("v", a.kv_heads)):
             ins.append(pad_heads(att[n], heads, a.width))
+        if a.gate:
+            ins.append(pad_rows(att["g"], a.gate_dim) if a.gate == "head" else pad_heads(att["g"], a.heads, a.width))
+        if a.bias:
+            bias = torch.cat([pad_heads(att[n + ".b"].float(), heads, a.width)
+                              for n, heads in (("q", a.heads), ("k", a.kv_heads), ("v", a.kv_heads))])
+        kw["v_mix"] = att["vmix"].float().reshape(1).contiguous() if a.v_mix else None
         outs.append(pad_heads(att["o"], a.heads, a.width, dim=1))
         if a.qk_norm:
             full = a.qk_norm == "full"
@@ -252,26 +366,34 @@ def listed_mixer(spec: LayerSpec, att: Dict[str, torch.Tensor], ret: Dict[str, t
         for n, width in (("q", r.k_width), ("k", r.k_width), ("v", r.v_width), ("g", r.v_width)):
             ins.append(pad_heads(ret[n], r.heads, width))
         outs.append(pad_heads(ret["o"], r.heads, r.v_width, dim=1))
-    kw["wqkv"] = LinearWeight([dense_qtensor(torch.cat(ins, dim=0).contiguous())])
-    kw["wo"] = LinearWeight([dense_qtensor(torch.cat(outs, dim=1).contiguous())])
+    if d is not None:
+        rows, kw["delta"] = delta_weights(d, rec, rec["q"].dtype)
+        ins += rows
+        outs.append(pad_heads(rec["o"], d.heads, d.v_width, dim=1))
+    w_in = torch.cat(ins, dim=0).contiguous()
+    kw["wqkv"] = LinearWeight([dense_qtensor(w_in)], None if bias is None else pad_rows(bias, w_in.shape[0]).contiguous())
+    if isinstance(spec.mixer, ParallelSpec) and spec.mixer.norms:
+        kw["wo"], kw["wo_right"] = (LinearWeight([dense_qtensor(o.contiguous())]) for o in outs)
+    else:
+        kw["wo"] = LinearWeight([dense_qtensor(torch.cat(outs, dim=1).contiguous())])
     return kw
 
 
-def gated_pair(gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor, size: int, rows: int = 0,
+def gated_pair(gate: Optional[torch.Tensor], up: torch.Tensor, down: torch.Tensor, size: int, rows: int = 0,
                cols: int = 0) -> Tuple[QTensor, QTensor]:
-    """([gate | up], down) with ``size`` feed-forward columns, the input padded to ``cols`` values and the output to
-    ``rows``."""
+    """([gate | up], down), or (up, down) without a gate, with ``size`` feed-forward columns, the input padded to ``cols``
+    values and the output to ``rows``."""
     def grow(t, n, k):
         return torch.nn.functional.pad(t, (0, max(k - t.shape[1], 0), 0, max(n - t.shape[0], 0)))
 
-    gu = torch.cat([grow(gate, size, cols), grow(up, size, cols)], dim=0).contiguous()
+    gu = torch.cat([grow(t, size, cols) for t in (gate, up) if t is not None], dim=0).contiguous()
     return dense_qtensor(gu), dense_qtensor(grow(down, rows, size).contiguous())
 
 
 def listed_experts(spec: MoESpec, triples, hidden: int) -> ExpertWeights:
-    """The experts' (gate, up, down), stacked; inner sizes are multiples of the grouped product's k-block."""
-    h64 = (hidden + 63) // 64 * 64
-    pairs = [gated_pair(g, u, d, spec.expert.pad_size, h64, h64) for g, u, d in triples]
+    """The experts' (gate or None, up, down), stacked; inner sizes are multiples of the grouped product's k-block."""
+    h64 = pad_to(hidden, 64)
+    pairs = [gated_pair(g, u, d, pad_to(spec.expert.size, 64), h64, h64) for g, u, d in triples]
     ex = ExpertWeights([p[0] for p in pairs], [p[1] for p in pairs])
     for name in ("gate_up", "down"):
         lst = getattr(ex, name)
@@ -317,6 +439,35 @@ def _load_listed(src: LayeredWeightSource, cfg: ModelConfig, i: int) -> LayerWei
     return lw
 
 
+def _load_joint(src: LayeredWeightSource, cfg: ModelConfig, i: int) -> LayerWeights:
+    """A layer with one norm that both branches read."""
+    spec, p = cfg.layer_specs[i], f"l{i}"
+    a, d, f = spec.attention, spec.delta, spec.ffn
+    both = isinstance(spec.mixer, ParallelSpec)
+
+    def mixer(prefix: str, matrices, vectors) -> Dict[str, torch.Tensor]:
+        out = {n: src.dense(f"{p}.mix.{prefix}{n}") for n in matrices}
+        out.update({n: src.vector(f"{p}.mix.{prefix}{n}") for n in vectors})
+        return out
+
+    att, rec = {}, {}
+    if a is not None:
+        att = mixer("left." if both else "", ["q", "k", "v", "o"] + (["g"] if a.gate else []),
+                    (["q.b", "k.b", "v.b"] if a.bias else []) + (["q.norm", "k.norm"] if a.qk_norm else [])
+                    + (["vmix"] if a.v_mix else []))
+    if d is not None:
+        rec = mixer("right." if both else "", ["q", "k", "v", "o", "b", "q.conv", "k.conv", "v.conv"]
+                    + (["a1", "a2"] if d.decay_rank else ["a"]) + (["g1", "g2"] if d.gate_rank else ["g"]), ["A_log", "dt_bias", "norm"])
+    lw = LayerWeights(attn_norm=src.vector(f"{p}.norm1"), ffn_norm=None, **listed_mixer(spec, att, rec))
+    if both:
+        lw.out_norms = (src.vector(f"{p}.mix.left.out"), src.vector(f"{p}.mix.right.out"))
+    if f is not None:
+        lw.router, lw.router_bias = src.matrix(f"{p}.mlp.router"), src.vector(f"{p}.mlp.correction")
+        lw.experts = listed_experts(f, [(None, src.dense(f"{p}.mlp.e{e}.up"), src.dense(f"{p}.mlp.e{e}.down"))
+                                        for e in range(f.n_experts)], cfg.hidden_size)
+    return lw
+
+
 def _load_layer(src: LayeredWeightSource, spec: LayerSpec, i: int, tp_rank: int, tp_size: int) -> LayerWeights:
     p, m = f"l{i}", spec.mixer
     h0, h1 = shard_range(m.heads, tp_rank, tp_size)
@@ -342,12 +493,12 @@ def load_layered_weights(ck: LayeredCheckpoint, cfg: ModelConfig, device="cpu", 
     replicated (every rank caches the whole latent row)."""
     src = LayeredWeightSource(ck, device, act_dtype)
     n = cfg.n_layers
-    sandwich = cfg.norm_placement == "sandwich"
-    if sandwich and tp_size > 1:
+    whole = {"sandwich": _load_listed, "parallel": _load_joint}.get(cfg.norm_placement)
+    if whole is not None and tp_size > 1:
         raise ValueError("a norm over all heads and per-sequence states are not sharded: run this model with tp_size = 1")
 
     def load(i: int) -> LayerWeights:
-        return _load_listed(src, cfg, i) if sandwich else _load_layer(src, cfg.layer_specs[i], i, tp_rank, tp_size)
+        return whole(src, cfg, i) if whole is not None else _load_layer(src, cfg.layer_specs[i], i, tp_rank, tp_size)
 
     source = [i if l.weights_of is None else l.weights_of for i, l in enumerate(cfg.layer_specs)]
     if 0 < resident_layers < n:
@@ -356,8 +507,9 @@ def load_layered_weights(ck: LayeredCheckpoint, cfg: ModelConfig, device="cpu", 
         own = {i: load(i) for i in sorted(set(source))}
         layers = [own[i] for i in source]
     v0, v1 = shard_range(cfg.vocab_size, tp_rank, tp_size) if cfg.vocab_size % tp_size == 0 else (0, cfg.vocab_size)
-    mw = ModelWeights(cfg, src.matrix("embed"), layers, src.vector("final.norm"), LinearWeight([src.matrix("head", rows=(v0, v1))]),
-                      [], tp_rank, tp_size, 0, 1, 0, v0)
+    embed = src.matrix("embed")
+    head = embed if cfg.tie_embeddings else src.matrix("head", rows=(v0, v1))
+    mw = ModelWeights(cfg, embed, layers, src.vector("final.norm"), LinearWeight([head]), [], tp_rank, tp_size, 0, 1, 0, v0)
     if cfg.norm_kind == "layer":
         mw.out_norm_bias = src.vector("final.norm.b")
     if cfg.embed_norm:

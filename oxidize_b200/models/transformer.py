@@ -187,12 +187,13 @@ class Transformer:
                     max_pos=min(max_context, 1 << 20))
             return ropes[key]
 
-        # (attention's, retention's) rotation of every layer
-        self.layer_ropes = [tuple(None if p is None else rope(p.rotary) for p in (l.attention, l.retention)) for l in cfg.layer_specs]
+        # (attention's, recurrence's) rotation of every layer
+        self.layer_ropes = [tuple(None if p is None or p.rotary is None else rope(p.rotary) for p in (l.attention, l.recurrent))
+                            for l in cfg.layer_specs]
         owners = [i for i, l in enumerate(cfg.layer_specs) if l.owns_rows]
         self.kv_index = [-1 if l.attention is None else owners.index(i if l.attention.kv_from is None else l.attention.kv_from)
                          for i, l in enumerate(cfg.layer_specs)]
-        stateful = [i for i, l in enumerate(cfg.layer_specs) if l.retention is not None]
+        stateful = [i for i, l in enumerate(cfg.layer_specs) if l.recurrent is not None]
         self.state_index = {i: n for n, i in enumerate(stateful)}
         self.n_kv_layers, self.n_kv_local, self.kv_head_dim = len(owners), 1, cfg.head_dim
 
@@ -309,7 +310,7 @@ class Transformer:
             kv.conv = KVCache(KVCacheSpec(self.n_conv_layers, 1, self.cfg.hidden_size // 2, page_size, plain), num_blocks,
                               self.device)
         if self.cfg.state_shapes:
-            kv.states = StateStore(self.cfg.state_shapes, state_slots, self.device)
+            kv.states = StateStore(self.cfg.state_shapes, state_slots, self.device, self.cfg.state_windows)
         return kv
 
     def _ssm_slot(self, kv, first_block: int, position: int) -> int:
@@ -510,6 +511,25 @@ class Transformer:
                 self._layer_done(li, x, capture)
         return (x if y is None else ops.branch_norm(x, y, post, None, eps, self.act_dtype)[0]), None
 
+    def _layers_parallel(self, h: torch.Tensor, meta: BatchMeta, kv, lo: int, hi: int, capture: Optional[dict]):
+        """Layers with one norm that both branches read, x <- x + mixer(norm(x)) + ffn(norm(x)), the stream ``x`` in float32.
+        One kernel adds both branches (each mixer's output through a norm of its own where the layer has two, the routed
+        experts' rows by their weights) and norms the sum for the next layer."""
+        cfg = self.cfg
+        eps = cfg.rms_eps
+        x, mix, ffn = h.float(), None, None
+        carry: dict = {}  # what later layers read of earlier ones
+        want = set(capture.get("layers", ())) if capture is not None else set()
+        for li in range(lo, hi):
+            lw, spec = self.w.layers[li], cfg.layer_specs[self.w.first_layer + li]
+            x, xa = ops.joint_norm(x, mix, ffn, lw.attn_norm, eps, self.act_dtype)
+            mix = self._listed_mixer(li, lw, spec, xa, meta, kv, carry)
+            ffn = None if spec.ffn is None else self._listed_ffn(lw, spec.ffn, xa, combine=False)
+            if self.w.first_layer + li in want or _profiler.TRACE_FWD:
+                x, mix, ffn = ops.joint_norm(x, mix, ffn, None, eps, self.act_dtype)[0], None, None
+                self._layer_done(li, x, capture)
+        return (x if mix is None else ops.joint_norm(x, mix, ffn, None, eps, self.act_dtype)[0]), None
+
     def _layer_done(self, li: int, x: torch.Tensor, capture: Optional[dict]) -> None:
         gl = self.w.first_layer + li
         if capture is not None and gl in capture.get("layers", ()):
@@ -517,18 +537,23 @@ class Transformer:
         if _profiler.TRACE_FWD:
             _profiler.trace_hidden(gl, x, None)
 
-    def _listed_mixer(self, li: int, lw: LayerWeights, spec, xa: torch.Tensor, meta: BatchMeta, kv) -> torch.Tensor:
-        """The mixer branch of a listed layer: from its normed input to its output projection."""
+    def _listed_mixer(self, li: int, lw: LayerWeights, spec, xa: torch.Tensor, meta: BatchMeta, kv, carry: Optional[dict] = None):
+        """The mixer branch of a listed layer: from its normed input to its output projection; with a norm on each side's
+        output, both projected outputs as ``ops.NormedPair``.  ``carry``: what this step's earlier layers left for it."""
         eps = self.cfg.rms_eps
         if lw.mla is not None:
             o = ops.latent_mixer(xa, lw.mla, spec.mixer, self.layer_ropes[li][0], meta, kv, self.kv_index[li], eps)
         else:
-            o = ops.listed_mixer(xa, lw, spec, self.layer_ropes[li], meta, kv, self.kv_index[li], self.state_index.get(li, -1), eps)
+            o = ops.listed_mixer(xa, lw, spec, self.layer_ropes[li], meta, kv, self.kv_index[li], self.state_index.get(li, -1), eps, carry)
+        if lw.out_norms is not None:
+            return ops.NormedPair(self.comm.linear_allreduce(o[0], lw.wo), self.comm.linear_allreduce(o[1], lw.wo_right), *lw.out_norms,
+                                  *spec.branch_scales)
         return self.comm.linear_allreduce(o, lw.wo)
 
-    def _listed_ffn(self, lw: LayerWeights, f, xa: torch.Tensor) -> torch.Tensor:
+    def _listed_ffn(self, lw: LayerWeights, f, xa: torch.Tensor, combine: bool = True):
+        """``combine`` False: routed experts may come as ``ops.RoutedRows``, their weighted sum left to the next kernel."""
         if isinstance(f, MoESpec):
-            return ops.moe_ffn(xa, lw, f)
+            return ops.moe_ffn(xa, lw, f, combine)
         if f.gated:
             return ops.gated_ffn(xa, lw.w_gate_up, lw.w_down)
         return self.comm.linear_allreduce(ops.linear_act(xa, lw.w_up, f.act), lw.w_down)
@@ -670,7 +695,8 @@ class Transformer:
         cfg = self.cfg
         lo, hi = layers if layers is not None else (0, len(self.w.layers))
         if cfg.is_layered:
-            layers_fn = self._layers_sandwich if cfg.norm_placement == "sandwich" else self._layers_norm_after
+            layers_fn = {"sandwich": self._layers_sandwich, "parallel": self._layers_parallel}.get(cfg.norm_placement,
+                                                                                                  self._layers_norm_after)
             return layers_fn(h, meta, kv, lo, hi, capture)
         acc, cur = None, 0  # per-token sum-of-squares accumulators of the residual stream while it is in folded form
         for li in range(lo, hi):
@@ -729,7 +755,9 @@ class Transformer:
             self.last_features = torch.cat([h if idx is None else h.index_select(0, idx) for h in hs], dim=-1)
 
     def embed(self, token_ids: torch.Tensor) -> torch.Tensor:
-        return ops.embed(token_ids, self.w.embed, self.act_dtype, self.cfg.embedding_scale)
+        # (a scaled row enters a float32 stream without being rounded first)
+        wide = self.cfg.is_layered and self.cfg.embedding_scale != 1.0
+        return ops.embed(token_ids, self.w.embed, torch.float32 if wide else self.act_dtype, self.cfg.embedding_scale)
 
     # ------------------------------------------------------------------ pipeline stages
     def _stage_input(self, meta: BatchMeta):

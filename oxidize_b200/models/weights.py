@@ -215,6 +215,18 @@ class GDNWeights:
 
 
 @dataclass
+class DeltaWeights:
+    """What acts behind the projections of a gated-delta-rule mixer (heads padded to their kernel widths)."""
+
+    conv: torch.Tensor  # [taps, q | k | v channels] float32, the last row on the current token
+    a_log: torch.Tensor  # [heads] float32
+    dt_bias: torch.Tensor  # [heads] or, with a decay per channel, [heads * k_width] float32
+    norm: torch.Tensor  # [v_width] float32
+    decay_up: Optional[torch.Tensor] = None  # [heads * k_width, decay_dim]: second half of a low-rank decay projection
+    gate_up: Optional[torch.Tensor] = None  # [heads * v_width, gate_dim]: the same of a low-rank gate projection
+
+
+@dataclass
 class LayerWeights:
     attn_norm: torch.Tensor
     wqkv: Optional[LinearWeight]  # None in a latent-attention layer (``mla`` holds its projections) or a convolution layer
@@ -226,6 +238,12 @@ class LayerWeights:
     # listed layers: per-head logits of the attention's softmax denominator.  ``wqkv`` then holds every projection of the
     # layer's input (attention q | k | v, retention q | k | v | gate) and ``wo`` the output projections side by side
     sink: Optional[torch.Tensor] = None
+    v_mix: Optional[torch.Tensor] = None  # [1] float32: the share of the first value-mixing layer's values
+    delta: Optional[DeltaWeights] = None
+    # two mixers whose projected outputs pass norms of their own: the right one's output projection (``wo`` is the left
+    # one's) and both norms
+    wo_right: Optional[LinearWeight] = None
+    out_norms: Optional[Tuple[torch.Tensor, torch.Tensor]] = None
     # short-convolution mixer (LFM2) instead of attention: in_proj [3 hidden, hidden] (rows: B, C, x), depthwise kernel
     # [hidden, l_cache] (oldest tap first), out_proj [hidden, hidden]
     conv_in: Optional[QTensor] = None
@@ -337,7 +355,7 @@ class ModelWeights:
     def nbytes(self) -> int:
         n = self.embed.nbytes() + self.lm_head.nbytes()
         for l in (self.layers.resident() if isinstance(self.layers, StreamedLayers) else self.layers):
-            for lw in (l.wqkv, l.wo, l.w_gate_up, l.w_up, l.w_down, l.shared_gate_up, l.shared_down):
+            for lw in (l.wqkv, l.wo, l.wo_right, l.w_gate_up, l.w_up, l.w_down, l.shared_gate_up, l.shared_down):
                 if lw is not None:
                     n += lw.nbytes()
             if l.experts is not None:

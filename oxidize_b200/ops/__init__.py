@@ -7,6 +7,7 @@ on a GPU machine the call raises.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -31,6 +32,27 @@ def _cuda_listed():
     from . import cuda_listed as _c
 
     return _c
+
+
+@dataclass
+class NormedPair:
+    """Projected outputs of two mixers that pass RMS norms of their own: left_scale * norm(left) + right_scale * norm(right)."""
+
+    left: torch.Tensor
+    right: torch.Tensor
+    left_norm: torch.Tensor
+    right_norm: torch.Tensor
+    left_scale: float
+    right_scale: float
+
+
+@dataclass
+class RoutedRows:
+    """Routed experts ahead of their weighted sum: token t's is sum_j weights[t, j] * rows[index[t, j]]."""
+
+    rows: torch.Tensor  # [T * k, hidden or more]
+    index: torch.Tensor  # [T, k] int32
+    weights: torch.Tensor  # [T, k] float32
 
 
 @instrument("linear")
@@ -97,24 +119,52 @@ def branch_norm(res, y, w_post, w_next, eps, act_dtype=torch.float32):
     return ref.branch_norm(res, y, w_post, w_next, eps, act_dtype)
 
 
+@instrument("joint_norm")
+def joint_norm(res, mix, ffn, w_next, eps, act_dtype=torch.float32):
+    """Both branches of a layer join the stream: x = res + mix + ffn (float32) and the next layer's input rmsnorm(x) * w_next
+    in ``act_dtype`` (None without ``w_next``).  ``mix``: None, a tensor or a ``NormedPair``; ``ffn``: None, a tensor or
+    ``RoutedRows``."""
+    if res.is_cuda:
+        return _cuda_listed().joint_norm(res, mix, ffn, w_next, eps, act_dtype)
+    return ref.joint_norm(res, mix, ffn, w_next, eps, act_dtype)
+
+
+def first_values(z, a, lw, carry):
+    """(values of the model's first value-mixing layer [T, kv_heads, width], this layer's share of them) for a layer that mixes
+    them into its own; (None, None) elsewhere.  The first such layer leaves its own in ``carry``."""
+    if not a.v_mix:
+        return None, None
+    v = z[:, (a.heads + a.kv_heads) * a.width : a.qkv_dim].unflatten(1, (a.kv_heads, a.width))
+    if carry is None:
+        raise ValueError("a layer that mixes values needs the step's earlier layers")
+    first = carry.setdefault("values", v)
+    return (None, None) if first is v else (first, lw.v_mix)
+
+
 @instrument("listed_mixer")
-def listed_mixer(x, lw, spec, ropes, meta, kv, kv_layer, state_layer, eps):
-    """Attention and / or retention of one listed layer on its normed input, up to (not including) the output projection:
-    [T, spec.out_dim], attention heads first.  ``ropes``: rotations of the two; in a layer with both, each side's output
-    carries its scale."""
+def listed_mixer(x, lw, spec, ropes, meta, kv, kv_layer, state_layer, eps, carry=None):
+    """Attention and / or a recurrence of one listed layer on its normed input, up to (not including) the output projection:
+    [T, spec.out_dim], attention heads first, or the two sides apart where each has an output projection of its own.
+    ``ropes``: rotations of the two; in a layer with one projection over both, each side's output carries its scale.
+    ``carry``: what this step's earlier layers left for later ones."""
     if x.is_cuda:
-        return _cuda_listed().listed_mixer(x, lw, spec, ropes, meta, kv, kv_layer, state_layer, eps)
+        return _cuda_listed().listed_mixer(x, lw, spec, ropes, meta, kv, kv_layer, state_layer, eps, carry)
     z = linear(x, lw.wqkv)
-    a, r, outs = spec.attention, spec.retention, []
-    sl, sr = spec.branch_scales
+    a, r, d, outs = spec.attention, spec.retention, spec.delta, []
+    sl, sr = spec.branch_scales if lw.out_norms is None else (1.0, 1.0)
     if a is not None:
-        q = ref.head_prep(z[:, : a.proj_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps)
+        q = ref.head_prep(z[:, : a.qkv_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps, *first_values(z, a, lw, carry))
         o = ref.paged_attention(q, kv, kv_layer, meta, a.scale, a.window, sink=lw.sink)
+        if a.gate:
+            o = ref.head_gate(o, z[:, a.qkv_dim : a.proj_dim], a)
         outs.append(o.reshape(x.shape[0], -1) * sl)
+    zr = z[:, 0 if a is None else a.proj_dim :]
     if r is not None:
-        zr = z[:, 0 if a is None else a.proj_dim :]
         outs.append((ref.retention(zr, r, ropes[1], meta, kv.states.data[state_layer], eps) * sr).to(x.dtype))
-    return torch.cat(outs, dim=-1)
+    if d is not None:
+        o = ref.delta_rule(zr, lw.delta, d, meta, kv.states.data[state_layer], kv.states.windows[state_layer], eps)
+        outs.append((o * sr).to(x.dtype))
+    return tuple(outs) if lw.out_norms is not None else torch.cat(outs, dim=-1)
 
 
 @instrument("gated_ffn")
@@ -126,18 +176,20 @@ def gated_ffn(x, gate_up, down):
 
 
 @instrument("moe_ffn")
-def moe_ffn(x, lw, spec):
-    """Routed experts (``spec``: ``models.config.MoESpec``) with float32 router logits, plus the shared expert."""
+def moe_ffn(x, lw, spec, combine=True):
+    """Routed experts (``spec``: ``models.config.MoESpec``) with float32 router logits, plus the shared expert.  ``combine``
+    False: the result may be ``RoutedRows`` (``joint_norm`` takes either)."""
     if x.is_cuda:
-        return _cuda_listed().moe_ffn(x, lw, spec)
-    ids, wts = ref.moe_route(linear(x.float(), lw.router), spec)
+        return _cuda_listed().moe_ffn(x, lw, spec, combine)
+    ids, wts = ref.moe_route(linear(x.float(), lw.router), spec, lw.router_bias if spec.correction else None)
+    one = gated_ffn if spec.expert.gated else lambda h, up, down: linear(ref.activation(linear(h, up), spec.expert.act), down)
     ex, H = lw.experts, x.shape[1]
     xp = torch.nn.functional.pad(x, (0, ex.gate_up[0].shape[1] - H))
     out = torch.zeros(x.shape[0], ex.down[0].shape[0], dtype=torch.float32)
     for e in range(spec.n_experts):
         rows, slot = (ids == e).nonzero(as_tuple=True)
         if rows.numel():
-            y = gated_ffn(xp[rows], ex.gate_up[e], ex.down[e]).float()
+            y = one(xp[rows], ex.gate_up[e], ex.down[e]).float()
             out.index_add_(0, rows, y * wts[rows, slot][:, None])
     out = out[:, :H]
     if lw.shared_gate_up is not None:

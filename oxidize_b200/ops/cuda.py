@@ -115,7 +115,7 @@ def _declare(L) -> None:
     L.oxb_gemm_plan.argtypes = [i32, i32, i32, i32, ctypes.POINTER(i32), ctypes.POINTER(sz), ctypes.POINTER(i32)]
     L.oxb_gemm_bf16.argtypes = [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, sz, vp, i32, vp]
     L.oxb_dequant_rows.argtypes = [vp, i32, sz, i32, i32, vp, i32, vp]
-    L.oxb_embed.argtypes = [vp, vp, i32, sz, i32, i32, f32, vp, i32, vp]
+    L.oxb_embed.argtypes = [vp, vp, i32, sz, i32, i32, f32, vp, i32, i32, vp]
     L.oxb_add_rmsnorm.argtypes = [vp, vp, vp, vp, vp, i32, i32, f32, vp]
     L.oxb_silu_mul.argtypes = [vp, vp, i32, i32, vp]
     L.oxb_gelu_mul.argtypes = [vp, vp, i32, i32, vp]
@@ -390,13 +390,11 @@ def linear_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, sumsq_in: Option
 def embed(tokens: torch.Tensor, table, dtype: torch.dtype, scale: float = 1.0) -> torch.Tensor:
     T = tokens.shape[0]
     V, H = table.shape
-    if dtype == torch.float32 and table.qtype == "F32":  # float32 compute: the kernel's output is bf16
-        return table.data.index_select(0, tokens.long()) * scale
-    out = torch.empty(T, H, dtype=torch.bfloat16, device=tokens.device)
+    out = torch.empty(T, H, dtype=torch.float32 if dtype == torch.float32 else torch.bfloat16, device=tokens.device)
     row_bytes = table.data.stride(0) * table.data.element_size()
     _check(lib().oxb_embed(tokens.data_ptr(), table.data.data_ptr(), QTYPE_CODE[table.qtype], row_bytes, H, V, scale,
-                           out.data_ptr(), T, _stream()), "oxb_embed")
-    return out if dtype == torch.bfloat16 else out.to(dtype)
+                           out.data_ptr(), 1 if out.dtype == torch.float32 else 0, T, _stream()), "oxb_embed")
+    return out.to(dtype)
 
 
 def add_rmsnorm(x: torch.Tensor, residual: Optional[torch.Tensor], w: torch.Tensor, eps: float):

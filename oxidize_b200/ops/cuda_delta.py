@@ -1,0 +1,51 @@
+"""Bindings of the gated-delta-rule kernels (``csrc/oxb_delta.cu``), in bfloat16 and float32.  CUDA tensors only; see
+:func:`oxidize_b200.ops.ref.delta_rule` for the operator's meaning."""
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from . import cuda_latent as latent
+from .cuda import _check, _p, _stream
+
+_declared = False
+_ALL = 1 << 30
+
+
+def lib():
+    global _declared
+    L = latent.lib()
+    if not _declared:
+        vp, i32, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
+        L.oxb_delta.argtypes = ([vp] + [i32] * 5 + [vp] * 4 + [i32, vp, vp, vp, i32, vp, i32, vp, vp, vp, i32, vp, i32, f32]
+                                + [i32] * 6 + [f32, f32, i32, i32, i32, vp])
+        L.oxb_delta_window.argtypes = [vp, i32, i32, vp, vp, vp, i32, vp] + [i32] * 6 + [vp]
+        _declared = True
+    return L
+
+
+def delta_rule(z: torch.Tensor, w, spec, meta, state: torch.Tensor, window: torch.Tensor, eps: float, out: torch.Tensor,
+               out_scale: float = 1.0) -> None:
+    """z [T, q | k | v | gate | decay | beta] to the normed, gated heads ``out`` [T, heads * v_width] (either may be a column
+    slice); ``state`` [slots, H, K, V] and ``window`` [slots, conv, channels] are updated."""
+    L = lib()
+    H, K, V = spec.state_shape
+    G, B, C = spec.kv_heads, meta.seq_lens.shape[0], spec.channels
+    if meta.state_slots is None:
+        raise ValueError("a layer with a recurrent state needs the sequences' state slots")
+    most = max(1, meta.max_query_len)
+    dt = latent.DT[z.dtype]
+
+    def step(lo: int, hi: int) -> None:
+        _check(L.oxb_delta(z.data_ptr(), z.stride(0), dt, C, C + spec.gate_dim, C + spec.gate_dim + spec.decay_dim,
+                           meta.query_start.data_ptr(), meta.seq_lens.data_ptr(), meta.state_slots.data_ptr(), w.conv.data_ptr(), spec.conv,
+                           w.a_log.data_ptr(), w.dt_bias.data_ptr(), _p(w.decay_up), spec.decay_dim, _p(w.gate_up), spec.gate_dim,
+                           w.norm.data_ptr(), state.data_ptr(), window.data_ptr(), state.shape[0], out.data_ptr(), out.stride(0), out_scale,
+                           B, H, G, K, V, spec.v_dim, spec.dim ** -0.5, eps, lo, hi, 1 if most == 1 else 0, _stream()), "oxb_delta")
+
+    step(1, _ALL)
+    if most > 1:
+        _check(L.oxb_delta_window(z.data_ptr(), z.stride(0), dt, meta.query_start.data_ptr(), meta.seq_lens.data_ptr(),
+                                  meta.state_slots.data_ptr(), spec.conv, window.data_ptr(), state.shape[0], B, H, G, K, V, _stream()),
+               "oxb_delta_window")

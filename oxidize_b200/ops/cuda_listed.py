@@ -24,7 +24,10 @@ def lib():
     if not _declared:
         vp, i32, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
         L.oxb_branch_norm.argtypes = [vp] * 6 + [i32] * 3 + [f32, vp]
-        L.oxb_head_prep.argtypes = [vp, i32, i32, vp, vp, vp] + [i32] * 3 + [vp, vp, i32, f32] + [i32] * 5 + [vp, vp, i32, i32, vp]
+        L.oxb_head_prep.argtypes = ([vp, i32, i32, vp, vp, vp] + [i32] * 3 + [vp, vp, i32, f32] + [i32] * 5 + [vp, vp, i32, i32]
+                                    + [f32, f32, vp, i32, i32, i32, vp, vp])
+        L.oxb_joint_norm.argtypes = [vp] * 5 + [f32, f32, vp, i32, vp, vp, i32, vp, vp, vp] + [i32] * 3 + [f32, vp]
+        L.oxb_head_gate.argtypes = [vp, i32, vp] + [i32] * 6 + [vp]
         L.oxb_gqa_attention_simt.argtypes = [vp, vp, i32, f32, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp]
         L.oxb_kv_gather.argtypes = [vp] * 4 + [i32] * 7 + [vp, vp]
         L.oxb_gqa_prefill.argtypes = [vp, vp, vp, i32, f32] + [vp] * 5 + [i32] * 7 + [f32, i32, vp]
@@ -34,7 +37,7 @@ def lib():
         L.oxb_silu_mul_f32.argtypes = [vp, vp, vp, i32, i32, vp]
         L.oxb_moe_combine_f32.argtypes = [vp, i32, vp, vp, i32, vp, vp, i32, i32, vp]
         L.oxb_router_logits.argtypes = [vp, vp, i32, vp] + [i32] * 3 + [vp]
-        L.oxb_gemm_f32_rows.argtypes = [vp] * 5 + [i32] * 6 + [vp]
+        L.oxb_gemm_f32_rows.argtypes = [vp] * 5 + [i32] * 7 + [vp]
         _declared = True
     return L
 
@@ -52,18 +55,49 @@ def branch_norm(res: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[t
     return x, a
 
 
+def joint_norm(res: torch.Tensor, mix, ffn, w_next: Optional[torch.Tensor], eps: float, act_dtype: torch.dtype):
+    from . import NormedPair, RoutedRows
+
+    T, H = res.shape
+
+    def rows(t):
+        return t if t is None or (t.dtype == act_dtype and t.is_contiguous()) else t.to(act_dtype).contiguous()
+
+    pair = mix if isinstance(mix, NormedPair) else None
+    y0, y1 = (rows(pair.left), rows(pair.right)) if pair else (rows(mix), None)
+    routed = ffn if isinstance(ffn, RoutedRows) else None
+    f = rows(routed.rows if routed else ffn)
+    x = res if mix is None and ffn is None else torch.empty_like(res)
+    a = None if w_next is None else torch.empty(T, H, dtype=act_dtype, device=res.device)
+    _check(lib().oxb_joint_norm(res.data_ptr(), _p(y0), _p(y1), _p(pair.left_norm) if pair else None, _p(pair.right_norm) if pair else None,
+                                pair.left_scale if pair else 1.0, pair.right_scale if pair else 1.0, _p(f), 0 if f is None else f.stride(0),
+                                _p(routed.index) if routed else None, _p(routed.weights) if routed else None,
+                                routed.index.shape[1] if routed else 0, _p(w_next), None if x is res else x.data_ptr(), _p(a),
+                                DT[act_dtype], T, H, eps, _stream()), "oxb_joint_norm")
+    return x, a
+
+
 # --------------------------------------------------------------------------- attention
-def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int, eps: float) -> torch.Tensor:
-    """q | k | v projections [T, ...] to rotated queries [T, heads, width]; keys and values go into the cache pages."""
+def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int, eps: float, v_first: Optional[torch.Tensor] = None,
+              v_mix: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """q | k | v projections [T, ...] to (rotated, scaled) queries [T, heads, width]; keys and (mixed) values go into the cache
+    pages."""
     T = z.shape[0]
-    tab = opcuda.rope_table(rope, rope.max_pos)
+    tab = meta.positions if rope is None else opcuda.rope_table(rope, rope.max_pos)  # (nothing of it is read without a rotation)
+    max_pos, rot, pairing = (1, 0, 0) if rope is None else (tab.shape[0], tab.shape[1], 0 if rope.pairing == "split_half" else 1)
+    first = (None, 0, 0) if v_first is None else (v_first.data_ptr(), v_first.stride(0), v_first.shape[2])
     q = torch.empty(T, spec.heads, spec.width, dtype=z.dtype, device=z.device)
     _check(lib().oxb_head_prep(z.data_ptr(), z.stride(0), DT[z.dtype], meta.positions.data_ptr(), meta.slot_mapping.data_ptr(),
-                               tab.data_ptr(), tab.shape[0], tab.shape[1], 0 if rope.pairing == "split_half" else 1, _p(q_norm),
-                               _p(k_norm), 1 if spec.qk_norm == "full" else 0, eps, T, spec.heads, spec.kv_heads, spec.dim,
-                               spec.width, q.data_ptr(), kv.data[layer].data_ptr(), kv.page_size, kv.num_blocks, _stream()),
-           "oxb_head_prep")
+                               tab.data_ptr(), max_pos, rot, pairing, _p(q_norm), _p(k_norm), 1 if spec.qk_norm == "full" else 0, eps, T, spec.heads, spec.kv_heads, spec.dim,
+                               spec.width, q.data_ptr(), kv.data[layer].data_ptr(), kv.page_size, kv.num_blocks, spec.temp_coef, spec.temp_every,
+                               *first, spec.v_dim, _p(v_mix), _stream()), "oxb_head_prep")
     return q
+
+
+def head_gate(o: torch.Tensor, gate: torch.Tensor, spec) -> None:
+    """``o`` [T, heads * width] (may be a column slice) times the sigmoid of its gates, in place."""
+    _check(lib().oxb_head_gate(o.data_ptr(), o.stride(0), gate.data_ptr(), gate.stride(0), 1 if spec.gate == "value" else 0, DT[o.dtype],
+                               o.shape[0], spec.heads, spec.width, _stream()), "oxb_head_gate")
 
 
 def attention_simt(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> None:
@@ -164,26 +198,35 @@ def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, decay: tor
     run(cut, _ALL, form, n_seg, ws)
 
 
-def listed_mixer(x: torch.Tensor, lw, spec, ropes, meta, kv, kv_layer: int, state_layer: int, eps: float) -> torch.Tensor:
-    from . import linear
+def listed_mixer(x: torch.Tensor, lw, spec, ropes, meta, kv, kv_layer: int, state_layer: int, eps: float, carry=None):
+    from . import first_values, linear
 
     z = linear(x, lw.wqkv)
-    a, r = spec.attention, spec.retention
-    sl, sr = spec.branch_scales
-    out = torch.empty(x.shape[0], spec.out_dim, dtype=x.dtype, device=x.device)
+    a, r, d = spec.attention, spec.retention, spec.delta
+    apart = lw.out_norms is not None  # each side has an output projection (and a scale) of its own
+    sl, sr = (1.0, 1.0) if apart else spec.branch_scales
+    T = x.shape[0]
+    outs = [torch.empty(T, n, dtype=x.dtype, device=x.device) for n in ((a.out_dim, spec.recurrent.out_dim) if apart else (spec.out_dim,))]
     na = no = 0
     if a is not None:
         if kv.data[kv_layer].dtype != x.dtype:
             raise ValueError(f"cache rows of listed layers are kept in the compute type on the GPU ({x.dtype}), not {kv.dtype_name}")
         na, no = a.proj_dim, a.out_dim
-        q = head_prep(z[:, :na], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps)
-        attention(q, kv, kv_layer, meta, a, lw.sink, out[:, :no], sl)
+        q = head_prep(z[:, : a.qkv_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps, *first_values(z, a, lw, carry))
+        attention(q, kv, kv_layer, meta, a, lw.sink, outs[0][:, :no], sl)
+        if a.gate:
+            head_gate(outs[0][:, :no], z[:, a.qkv_dim : na], a)
+    out = outs[-1][:, 0 if apart else no :]
+    if d is not None:
+        from . import cuda_delta
+
+        cuda_delta.delta_rule(z[:, na:], lw.delta, d, meta, kv.states.data[state_layer], kv.states.windows[state_layer], eps, out, sr)
     if r is not None:
         decay = getattr(lw, "_decay", None)
         if decay is None:
             decay = lw._decay = torch.tensor(r.decay, dtype=torch.float32, device=x.device)
-        retention(z[:, na:], r, ropes[1], meta, kv.states.data[state_layer], decay, eps, out[:, no:], sr)
-    return out
+        retention(z[:, na:], r, ropes[1], meta, kv.states.data[state_layer], decay, eps, out, sr)
+    return tuple(outs) if apart else outs[0]
 
 
 # --------------------------------------------------------------------------- feed-forward blocks
@@ -217,34 +260,42 @@ def router_logits(x: torch.Tensor, w) -> torch.Tensor:
     return out
 
 
-def _gemm_rows(x, w, offsets, perm, groups: int, rows: int, max_rows: int) -> torch.Tensor:
+def _gemm_rows(x, w, offsets, perm, groups: int, rows: int, max_rows: int, act: int = 0) -> torch.Tensor:
     N, K = w.shape[0] // groups, w.shape[1]
     y = torch.empty(rows, N, dtype=torch.float32, device=x.device)
     _check(lib().oxb_gemm_f32_rows(x.data_ptr(), w.data.data_ptr(), y.data_ptr(), offsets.data_ptr(), _p(perm), groups, max_rows, N, K,
-                                   x.stride(0), N, _stream()), "oxb_gemm_f32_rows")
+                                   x.stride(0), N, act, _stream()), "oxb_gemm_f32_rows")
     return y
 
 
-def moe_ffn(x: torch.Tensor, lw, spec) -> torch.Tensor:
-    from . import cuda_moe
+def moe_ffn(x: torch.Tensor, lw, spec, combine: bool = True):
+    from . import RoutedRows, cuda_moe
 
     T, H = x.shape
     ex = lw.experts
+    bias = lw.router_bias if spec.correction else None
+    relu2 = not spec.expert.gated
+    if relu2 and spec.expert.act != "relu2":
+        raise ValueError(f"ungated experts have the relu2 activation, not {spec.expert.act!r}")
     logits = router_logits(x, lw.router)
     shared = gated_ffn(x, lw.shared_gate_up, lw.shared_down) if lw.shared_gate_up is not None else None
     pad = ex.gate_up_stack.shape[1] - H
     xp = torch.nn.functional.pad(x, (0, pad)) if pad else x.contiguous()
     if x.dtype == torch.bfloat16:
         sp = torch.nn.functional.pad(shared, (0, pad)) if pad and shared is not None else shared
-        out = cuda_moe.moe_layer(xp, logits, spec, None, ex, sp)[0]
+        if not combine and shared is None and T * spec.n_experts_used <= cuda_moe.MAX_DISPATCH_ENTRIES:
+            return RoutedRows(*cuda_moe.moe_layer(xp, logits, spec, bias, ex, relu2=relu2, combine=False))
+        out = cuda_moe.moe_layer(xp, logits, spec, bias, ex, sp, relu2=relu2)[0]
         return out[:, :H].contiguous() if pad else out
     E, k = spec.n_experts, spec.n_experts_used
     if E > 256 or T * k > cuda_moe.MAX_DISPATCH_ENTRIES:
         raise ValueError("float32 expert dispatch covers up to 256 experts and 2^17 token x expert pairs in a step")
-    ids, wts = cuda_moe.moe_route(logits, spec)
+    ids, wts = cuda_moe.moe_route(logits, spec, bias)
     offsets, perm, inv = cuda_moe.moe_dispatch(ids, 0, E)
-    h = _gemm_rows(xp, ex.gate_up_stack, offsets, perm, E, T * k, T)
-    y = _gemm_rows(silu_mul_f32(h, offsets[E:]), ex.down_stack, offsets, None, E, T * k, T)
+    h = _gemm_rows(xp, ex.gate_up_stack, offsets, perm, E, T * k, T, latent.ACTS["relu2"] if relu2 else 0)
+    y = _gemm_rows(h if relu2 else silu_mul_f32(h, offsets[E:]), ex.down_stack, offsets, None, E, T * k, T)
+    if not combine and shared is None:
+        return RoutedRows(y, inv, wts)
     out = torch.empty(T, H, dtype=torch.float32, device=x.device)
     _check(lib().oxb_moe_combine_f32(y.data_ptr(), y.stride(0), inv.data_ptr(), wts.data_ptr(), k, _p(shared), out.data_ptr(), T, H,
                                      _stream()), "oxb_moe_combine_f32")

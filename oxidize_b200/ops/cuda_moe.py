@@ -24,6 +24,7 @@ import torch
 from . import cuda as C
 
 GROUPED_MAX_TOKENS = 256
+EPI_RELU2 = 5
 
 
 def _declare(L):
@@ -38,7 +39,7 @@ def _declare(L):
     L.oxb_moe_permute.argtypes = [vp, i32, i32, i32, i32, vp, vp, vp, vp]
     L.oxb_moe_gather.argtypes = [vp, i32, vp, vp, i32, vp, vp]
     L.oxb_silu_mul_rows.argtypes = [vp, vp, vp, i32, i32, vp]
-    L.oxb_gemm_grouped_rows.argtypes = [vp, i32, vp, i32, sz, vp, vp, i32, i32, i32, i32, i32, vp]
+    L.oxb_gemm_grouped_rows.argtypes = [vp, i32, vp, i32, sz, vp, vp, i32, i32, i32, i32, i32, i32, vp]
     u64p = ctypes.POINTER(ctypes.c_uint64)
     L.oxb_moe_combine_gathered.argtypes = [vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, u64p, u64p, vp, i32, i32, i32,
                                            ctypes.c_ulonglong, vp]
@@ -105,8 +106,9 @@ def moe_combine(y: torch.Tensor, scale: torch.Tensor, shared: Optional[torch.Ten
     return out
 
 
-def gemm_grouped_rows(xg: torch.Tensor, w, offsets: torch.Tensor, groups: int, max_rows: int) -> torch.Tensor:
-    """y[r] = xg[r] @ W_g^T for every gathered row r of group g (rows [offsets[g], offsets[g+1])); [rows_cap, N] bf16."""
+def gemm_grouped_rows(xg: torch.Tensor, w, offsets: torch.Tensor, groups: int, max_rows: int, epi: int = 0) -> torch.Tensor:
+    """y[r] = xg[r] @ W_g^T for every gathered row r of group g (rows [offsets[g], offsets[g+1])); [rows_cap, N] bf16.
+    ``epi``: epilogue of the product (0 none, ``EPI_RELU2``)."""
     L = C.lib()
     _declare(L)
     N = w.shape[0] // groups
@@ -114,7 +116,7 @@ def gemm_grouped_rows(xg: torch.Tensor, w, offsets: torch.Tensor, groups: int, m
     y = torch.empty(xg.shape[0], N, dtype=torch.bfloat16, device=xg.device)
     row_bytes = w.data.stride(0) * w.data.element_size()
     C._check(L.oxb_gemm_grouped_rows(xg.data_ptr(), xg.shape[0], w.data.data_ptr(), C.QTYPE_CODE[w.qtype], row_bytes,
-                                     y.data_ptr(), offsets.data_ptr(), groups, max_rows, N, K, N, C._stream()),
+                                     y.data_ptr(), offsets.data_ptr(), groups, max_rows, N, K, N, epi, C._stream()),
              "oxb_gemm_grouped_rows")
     return y
 
@@ -163,9 +165,11 @@ MAX_DISPATCH_ENTRIES = 1 << 17  # token x top-k entries one permute launch (a si
 
 
 def moe_layer(x: torch.Tensor, router_logits: torch.Tensor, cfg, router_bias, experts,
-              shared: Optional[torch.Tensor] = None, comm=None, gathered: bool = True):
+              shared: Optional[torch.Tensor] = None, comm=None, gathered: bool = True, relu2: bool = False, combine: bool = True):
     """Whole routed-expert block for the experts held locally (+ optional shared-expert output).
-    Returns (out, reduced): ``reduced`` says that the expert-parallel all-reduce already happened (fused combine)."""
+    Returns (out, reduced): ``reduced`` says that the expert-parallel all-reduce already happened (fused combine).
+    ``relu2``: ungated experts, the square of relu being the epilogue of their up projection.  Without ``combine`` the result
+    is (rows, row of every token and choice, weights), their sum left to the caller."""
     T = x.shape[0]
     E = len(experts.gate_up)
     k = cfg.n_experts_used
@@ -180,13 +184,21 @@ def moe_layer(x: torch.Tensor, router_logits: torch.Tensor, cfg, router_bias, ex
         xg = torch.empty(T * k, x.shape[1], dtype=torch.bfloat16, device=x.device)
         C._check(L.oxb_moe_gather(x.data_ptr(), x.shape[1], perm.data_ptr(), n_rows.data_ptr(), T * k, xg.data_ptr(),
                                   C._stream()), "oxb_moe_gather")
-        h = gemm_grouped_rows(xg, experts.gate_up_stack, offsets, E, T)  # [T*k, 2F]
-        F = h.shape[1] // 2
-        act = torch.empty(T * k, F, dtype=torch.bfloat16, device=x.device)
-        C._check(L.oxb_silu_mul_rows(h.data_ptr(), act.data_ptr(), n_rows.data_ptr(), T * k, F, C._stream()),
-                 "oxb_silu_mul_rows")
+        if relu2:
+            act = gemm_grouped_rows(xg, experts.gate_up_stack, offsets, E, T, EPI_RELU2)  # [T*k, F]
+        else:
+            h = gemm_grouped_rows(xg, experts.gate_up_stack, offsets, E, T)  # [T*k, 2F]
+            F = h.shape[1] // 2
+            act = torch.empty(T * k, F, dtype=torch.bfloat16, device=x.device)
+            C._check(L.oxb_silu_mul_rows(h.data_ptr(), act.data_ptr(), n_rows.data_ptr(), T * k, F, C._stream()),
+                     "oxb_silu_mul_rows")
         y = gemm_grouped_rows(act, experts.down_stack, offsets, E, T)  # [T*k, H]
+        if not combine:
+            return y, inv, wts
         return moe_combine_gathered(y, inv, wts, shared, T, comm)
+    if relu2 or not combine:
+        raise ValueError(f"{cfg.n_experts} experts ({k} per token) over {T} tokens: the grouped kernels take up to 256 experts, "
+                         f"16 per token and {MAX_DISPATCH_ENTRIES} token x expert pairs")
     # the dense form runs one token tile per expert: 256 tokens with bf16 experts, 128 with packed ones
     if stacked and T <= (GROUPED_MAX_TOKENS if experts.gate_up_stack.qtype == "BF16" else GROUPED_MAX_TOKENS // 2):
         scale = torch.empty(E, max(T, 1), dtype=torch.float32, device=x.device)

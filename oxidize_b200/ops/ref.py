@@ -97,6 +97,21 @@ def branch_norm(res: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[t
     return x, None if w_next is None else rmsnorm(x, w_next, eps).to(act_dtype)
 
 
+def joint_norm(res: torch.Tensor, mix, ffn, w_next: Optional[torch.Tensor], eps: float, act_dtype: torch.dtype = torch.float32):
+    """Both branches of a layer join the stream: x = res + mix + ffn in float32 and the next layer's input rmsnorm(x) * w_next
+    in ``act_dtype``; (x, None) without ``w_next``.  ``mix`` may be a pair of outputs with norms and scales of their own."""
+    x = res.float()
+    if mix is not None:
+        y = mix
+        if not isinstance(mix, torch.Tensor):
+            y = (mix.left_scale * rmsnorm(mix.left.float(), mix.left_norm, eps)
+                 + mix.right_scale * rmsnorm(mix.right.float(), mix.right_norm, eps))
+        x = x + y.float()
+    if ffn is not None:
+        x = x + ffn.float()
+    return x, None if w_next is None else rmsnorm(x, w_next, eps).to(act_dtype)
+
+
 def activation(x: torch.Tensor, act: str) -> torch.Tensor:
     """Elementwise activation of a feed-forward block without a gate: ``relu2`` is the square of relu."""
     if act == "relu2":
@@ -357,9 +372,14 @@ def padded_norm(x: torch.Tensor, w: torch.Tensor, n: int, eps: float) -> torch.T
     return x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / n + eps) * w
 
 
-def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int, eps: float) -> torch.Tensor:
-    """From a layer's q | k | v projections (heads of ``spec.width`` values): norms, rotation, this step's cache rows; the
-    queries [T, heads, width]."""
+def query_temperature(positions: torch.Tensor, coef: float, every: float) -> torch.Tensor:
+    return 1.0 + coef * torch.log(torch.floor((positions.float() + 1.0) / every) + 1.0)
+
+
+def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int, eps: float, v_first: Optional[torch.Tensor] = None,
+              v_mix: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """From a layer's q | k | v projections (heads of ``spec.width`` values): norms, rotation, query temperature, values mixed
+    with ``v_first`` [T, kv_heads, v_dim or more], this step's cache rows; the queries [T, heads, width]."""
     T, H, G, W = z.shape[0], spec.heads, spec.kv_heads, spec.width
     q, k, v = z[:, : H * W].float(), z[:, H * W : (H + G) * W].float(), z[:, (H + G) * W : (H + 2 * G) * W]
     if spec.qk_norm == "full":
@@ -367,10 +387,25 @@ def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int,
     q, k = q.reshape(T, H, W), k.reshape(T, G, W)
     if spec.qk_norm == "head":
         q, k = padded_norm(q, q_norm, spec.dim, eps), padded_norm(k, k_norm, spec.dim, eps)
-    q = apply_rope(q, meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
-    k = apply_rope(k, meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
-    kv_write(kv, layer, k, v.reshape(T, G, W), meta.slot_mapping)
+    if rope is not None:
+        q = apply_rope(q, meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
+        k = apply_rope(k, meta.positions, rope.inv_freq, rope.pairing, rope.mscale)
+    if spec.temp_coef != 0.0:
+        q = q * query_temperature(meta.positions, spec.temp_coef, spec.temp_every)[:, None, None]
+    v = v.reshape(T, G, W)
+    if v_first is not None:
+        v = v.float().clone()
+        v[..., : spec.v_dim] = (1.0 - v_mix) * v[..., : spec.v_dim] + v_mix * v_first[..., : spec.v_dim].float()
+    kv_write(kv, layer, k, v, meta.slot_mapping)
     return q.to(z.dtype)
+
+
+def head_gate(o: torch.Tensor, gate: torch.Tensor, spec) -> torch.Tensor:
+    """Heads' outputs [T, heads, width] times the sigmoid of their gates (one per head, or per value)."""
+    T = o.shape[0]
+    g = torch.sigmoid(gate.float())
+    g = g[:, : spec.heads, None] if spec.gate == "head" else g.reshape(T, spec.heads, spec.width)
+    return (o.float() * g).to(o.dtype)
 
 
 def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, eps: float) -> torch.Tensor:
@@ -396,6 +431,45 @@ def retention(z: torch.Tensor, spec, rope, meta, state: torch.Tensor, eps: float
         state[slots[b]] = S
     y = padded_norm(o, 1.0, spec.v_dim, eps) * torch.nn.functional.silu(g)
     return y.reshape(T, H * V)
+
+
+def delta_rule(z: torch.Tensor, w, spec, meta, state: torch.Tensor, window: torch.Tensor, eps: float) -> torch.Tensor:
+    """Gated delta rule of one layer, token by token: z [T, q | k | v | gate | decay | beta] (``spec``:
+    ``models.config.DeltaSpec``), state [slots, heads, k_width, v_width] and the ring of convolution inputs ``window`` [slots,
+    conv, channels] (both updated); a sequence whose rows start at position 0 starts from nothing.  [T, heads * v_width]."""
+    T, H, G, K, V, n = z.shape[0], spec.heads, spec.kv_heads, spec.k_width, spec.v_width, spec.conv
+    F = torch.nn.functional
+    C = spec.channels
+    zf = z.float()
+    u, gate, decay = zf[:, :C], zf[:, C : C + spec.gate_dim], zf[:, C + spec.gate_dim : C + spec.gate_dim + spec.decay_dim]
+    beta = torch.sigmoid(zf[:, C + spec.gate_dim + spec.decay_dim :][:, :H])
+    gate = torch.sigmoid(gate @ w.gate_up.float().t()) if spec.gate_rank else F.silu(gate)
+    a = (decay @ w.decay_up.float().t()) if spec.decay_rank else decay[:, :H]
+    g = torch.exp(-torch.exp(w.a_log)[None, :, None] * F.softplus(a + w.dt_bias).reshape(T, H, -1))
+    o = torch.zeros(T, H, V, dtype=torch.float32, device=z.device)
+    qs, lens, slots = meta.query_start.tolist(), meta.seq_lens.tolist(), meta.state_slots.tolist()
+    unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
+    for b in range(len(lens)):
+        t0, t1 = qs[b], qs[b + 1]
+        m = t1 - t0
+        if slots[b] < 0 or m == 0:
+            continue
+        pos0, ring = lens[b] - m, window[slots[b]]
+        past = torch.stack([ring[p % n] if p >= 0 else torch.zeros_like(ring[0]) for p in range(pos0 - n + 1, pos0)] or [ring[0]])
+        rows = torch.cat([past[: n - 1], u[t0:t1]])
+        y = F.silu(sum(w.conv[j] * rows[j : j + m] for j in range(n)))
+        for p in range(max(pos0, pos0 + m - n), pos0 + m):
+            ring[p % n] = u[t0 + p - pos0]
+        q = unit(y[:, : G * K].reshape(m, G, K)).repeat_interleave(H // G, dim=1) * spec.dim ** -0.5
+        k = unit(y[:, G * K : 2 * G * K].reshape(m, G, K)).repeat_interleave(H // G, dim=1)
+        v = y[:, 2 * G * K :].reshape(m, H, V)
+        S = torch.zeros_like(state[slots[b]]) if pos0 == 0 else state[slots[b]]
+        for t in range(m):
+            S = g[t0 + t][:, :, None] * S
+            S = S + k[t][:, :, None] * (beta[t0 + t][:, None] * (v[t] - (S * k[t][:, :, None]).sum(1)))[:, None, :]
+            o[t0 + t] = (S * q[t][:, :, None]).sum(1)
+        state[slots[b]] = S
+    return padded_norm(o, w.norm, spec.v_dim, eps).reshape(T, H * V) * gate
 
 
 # --------------------------------------------------------------------------- MoE routing

@@ -246,7 +246,7 @@ def prefill_token_budget(cfg: ModelConfig, tp: int = 1, sm_count: int = 148, lo:
         if isinstance(m, LatentAttentionSpec):
             shapes = [(m.heads * m.qk_dim // tp + m.kv_rank + m.rope_dim, h), (h, m.heads * m.v_dim // tp)]
         else:
-            shapes = [(sum(p.proj_dim for p in (l.attention, l.retention) if p is not None) // tp, h), (h, l.out_dim // tp)]
+            shapes = [(l.in_dim // tp, h), (h, l.out_dim // tp)]
         shapes += [(f // tp, h), (h, f // tp)] if f >= tp else []
     best, best_eff = lo, -1.0
     t = (lo + token_tile - 1) // token_tile * token_tile
