@@ -40,6 +40,7 @@ struct AttnArgs {
   const float* sink;  // [nq] logits that join the softmax denominator only, or null
   int ld_out;         // values between the output rows of neighbouring tokens
   float out_scale;    // factor on the outputs
+  HeadGate gate;
   float* ws_o;   // [B*nkv*max_mtiles*n_cta_splits, 16, hd]
   float* ws_ml;  // [.., 16, 2]
   int* counters; // [B*nkv*max_mtiles] zero-initialised tickets (CTA splits only)
@@ -146,6 +147,18 @@ __device__ __forceinline__ void decode_page(uint8_t* stage, uint8_t* dec, int kv
   }
 }
 
+// Factor of an output row by its head's gate, and of two neighbouring values by theirs (1 where there is none).
+__device__ __forceinline__ float attn_row_gate(const AttnArgs& a, int t, int head) {
+  if (a.gate.rows == nullptr || a.gate.per_value) return 1.f;
+  return head_gate_of(__bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.gate.rows)[(size_t)t * a.gate.ld + head]));
+}
+__device__ __forceinline__ float2 attn_value_gate(const AttnArgs& a, int t, int col) {
+  if (a.gate.rows == nullptr || !a.gate.per_value) return make_float2(1.f, 1.f);
+  const float2 z = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(reinterpret_cast<const __nv_bfloat16*>(a.gate.rows) +
+                                                                    (size_t)t * a.gate.ld + col));
+  return make_float2(head_gate_of(z.x), head_gate_of(z.y));
+}
+
 // Merge the CTA-split partials of one (sequence, kv head, row tile): 128 threads = 16 rows x 8
 // column segments.  Partials were written by other CTAs, so they are read through L2 (__ldcg).
 template <int HD>
@@ -177,10 +190,13 @@ __device__ __forceinline__ void attn_merge_rows(const AttnArgs& a, int G, int b,
       acc[4 * d + 3] += w * v.w;
     }
   }
-  const float inv = L > 0.f ? a.out_scale / L : 0.f;
+  const float inv = (L > 0.f ? a.out_scale / L : 0.f) * attn_row_gate(a, q0 + r / G, kvh * G + r % G);
   __nv_bfloat16* dst = a.out + (size_t)(q0 + r / G) * a.ld_out + (kvh * G + r % G) * HD + seg;
 #pragma unroll
-  for (int d = 0; d < HD / 8; d += 2) *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(acc[d] * inv, acc[d + 1] * inv);
+  for (int d = 0; d < HD / 8; d += 2) {
+    const float2 f = attn_value_gate(a, q0 + r / G, (kvh * G + r % G) * HD + seg + d);
+    *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(acc[d] * inv * f.x, acc[d + 1] * inv * f.y);
+  }
 }
 
 template <int HD>
@@ -432,7 +448,7 @@ paged_attention_kernel(const AttnArgs a, int G /*q heads per kv head*/) {
     }
     if (a.n_cta_splits == 1) {
       if (valid) {
-        const float inv = L > 0.f ? a.out_scale / L : 0.f;
+        const float inv = (L > 0.f ? a.out_scale / L : 0.f) * attn_row_gate(a, q0 + r / G, kvh * G + r % G);
         __nv_bfloat16* dst = a.out + (size_t)(q0 + r / G) * a.ld_out + (kvh * G + r % G) * HD + seg;
         for (int d = 0; d < HD / 8; d += 2) {
           float v0 = 0.f, v1 = 0.f;
@@ -441,7 +457,8 @@ paged_attention_kernel(const AttnArgs a, int G /*q heads per kv head*/) {
             v0 += wgt[w] * mo[((size_t)w * 16 + row) * HD + seg + d];
             v1 += wgt[w] * mo[((size_t)w * 16 + row) * HD + seg + d + 1];
           }
-          *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(v0 * inv, v1 * inv);
+          const float2 f = attn_value_gate(a, q0 + r / G, (kvh * G + r % G) * HD + seg + d);
+          *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(v0 * inv * f.x, v1 * inv * f.y);
         }
       }
     } else {

@@ -78,6 +78,13 @@ __device__ __forceinline__ float2 unpack_bf16x2(uint32_t u) {
   return __bfloat1622float2(v);
 }
 
+// Gates on attention outputs, out *= sigmoid(gate): one per head (rows [T, heads]), or one per value (rows [T, heads * width]).
+struct HeadGate {
+  const void* rows;  // in the activation type, or null
+  int ld, per_value;
+};
+__device__ __forceinline__ float head_gate_of(float z) { return 1.f / (1.f + expf(-z)); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

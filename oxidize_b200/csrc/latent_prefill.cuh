@@ -92,6 +92,7 @@ struct LatentPrefillArgs {
   int H, window, group;     // group: query heads per key head
   int ld_out;
   float out_scale;
+  HeadGate gate;
   int nope16, rot16, full_ld;  // k-steps of 16 values of the two key parts; values per head of a query row
   int nope_ld, v_off, v_ld, v; // expanded row: head h's key at h * nope_ld, its value at v_off + h * v_ld
   float scale_log2;
@@ -330,13 +331,36 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     __syncwarp();
     tc_fence_after();
     if (sink > -INFINITY) l += exp2f(sink - m);  // the sink's share of the denominator, once
-    const float inv = l > 0.f ? a.out_scale / l : 0.f;
+    float inv = l > 0.f ? a.out_scale / l : 0.f;
+    const __nv_bfloat16* gates = reinterpret_cast<const __nv_bfloat16*>(a.gate.rows);  // this row's
+    if (gates != nullptr) {
+      gates += (size_t)(q0 + min(r, qlen - 1)) * a.gate.ld;
+      if (!a.gate.per_value) {
+        inv *= head_gate_of(__bfloat162float(gates[h]));
+        gates = nullptr;
+      } else {
+        gates += h * a.v;
+      }
+    }
     __nv_bfloat16* o_row = a.out + (size_t)(q0 + r) * a.ld_out + h * a.v;
     for (int c = 0; c < v16; ++c) {
       uint32_t o[16];
       tmem_ld16(o_col + 16 * c, o);
       tmem_ld_wait();
       if (r < qlen) {
+        if (gates != nullptr) {  // (v a multiple of 16)
+#pragma unroll
+          for (int j = 0; j < 16; j += 8) {
+            const uint4 u = *reinterpret_cast<const uint4*>(gates + 16 * c + j);
+            const uint32_t us[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float2 z = unpack_bf16x2(us[e]);
+              o[j + 2 * e] = __float_as_uint(__uint_as_float(o[j + 2 * e]) * head_gate_of(z.x));
+              o[j + 2 * e + 1] = __float_as_uint(__uint_as_float(o[j + 2 * e + 1]) * head_gate_of(z.y));
+            }
+          }
+        }
         if ((a.v | a.ld_out) % 8 == 0) {
 #pragma unroll
           for (int j = 0; j < 16; j += 8) {

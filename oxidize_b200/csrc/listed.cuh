@@ -187,26 +187,6 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
   }
 }
 
-// Heads' outputs times the sigmoid of their gates, in place: one gate per head (per_value 0: gate [T, H]) or per value.
-template <typename T>
-__global__ void __launch_bounds__(256) head_gate_kernel(T* __restrict__ o, int ld, const T* __restrict__ gate, int ld_gate,
-                                                        int per_value, int rows, int H, int W) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int n = H * W >> 2;  // groups of four values
-  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < (size_t)rows * n; i += (size_t)gridDim.x * blockDim.x) {
-    const size_t t = i / n;
-    const int c = (int)(i % n) * 4;
-    float v[4], g[4];
-    head_load<4>(o + t * ld + c, v);
-    if (per_value) head_load<4>(gate + t * ld_gate + c, g);
-    else g[0] = g[1] = g[2] = g[3] = lat_f32(gate[t * ld_gate + c / W]);
-#pragma unroll
-    for (int j = 0; j < 4; ++j) v[j] /= 1.f + expf(-g[j]);
-    head_store<4>(o + t * ld + c, v);
-  }
-}
-
 struct GqaSimtArgs {
   const void* q;            // [T, H, width]
   void* out;                // [T, H * width], rows ld_out apart
@@ -217,6 +197,7 @@ struct GqaSimtArgs {
   const float* sink;        // [H] or null
   int B, max_blocks, T, H, G, width, page, num_blocks, window, ld_out;
   float scale, out_scale;
+  HeadGate gate;
 };
 
 // The plain attention step (any type, width and page): one warp per (token, head), keys one after the other; NC * 32 >= width.
@@ -272,12 +253,15 @@ __global__ void __launch_bounds__(128) gqa_attention_simt_kernel(const GqaSimtAr
       acc[i] = acc[i] * c + (d < a.width ? p * lat_f32(vr[d]) : 0.f);
     }
   }
-  const float inv = l > 0.f ? a.out_scale / l : 0.f;
+  float inv = l > 0.f ? a.out_scale / l : 0.f;
+  const T* gates = a.gate.rows == nullptr ? nullptr : reinterpret_cast<const T*>(a.gate.rows) + (size_t)t * a.gate.ld;
+  if (gates != nullptr && !a.gate.per_value) inv *= head_gate_of(lat_f32(gates[h]));
   T* o = reinterpret_cast<T*>(a.out) + (size_t)t * a.ld_out + (size_t)h * a.width;
 #pragma unroll
   for (int i = 0; i < NC; ++i) {
     const int d = lane + 32 * i;
-    if (d < a.width) o[d] = lat_from<T>(acc[i] * inv);
+    if (d < a.width)
+      o[d] = lat_from<T>(acc[i] * inv * (gates != nullptr && a.gate.per_value ? head_gate_of(lat_f32(gates[h * a.width + d])) : 1.f));
   }
 }
 

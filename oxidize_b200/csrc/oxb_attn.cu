@@ -39,9 +39,10 @@ OXB_API int oxb_paged_attention(const void* q, void* out, const void* kv_data, c
                                 int max_blocks, int nq, int nkv, int hd, int kv_mode, int max_query_len,
                                 int n_cta_splits, int window, float scale, float softcap, const float* sink, int ld_out,
                                 float out_scale, float* ws_o, float* ws_ml, int* counters, int num_blocks,
-                                cudaStream_t stream) {
+                                const void* gate, int ld_gate, int gate_per_value, cudaStream_t stream) {
   if (B <= 0) return 0;
-  if (nq % nkv != 0) return (int)cudaErrorInvalidValue;
+  if (nq % nkv != 0 || (gate != nullptr && gate_per_value && (ld_gate % 2 != 0 || (reinterpret_cast<uintptr_t>(gate) & 3) != 0)))
+    return (int)cudaErrorInvalidValue;
   const int G = nq / nkv;
   AttnArgs a;
   a.q = reinterpret_cast<const __nv_bfloat16*>(q);
@@ -64,6 +65,7 @@ OXB_API int oxb_paged_attention(const void* q, void* out, const void* kv_data, c
   a.sink = sink;
   a.ld_out = ld_out;
   a.out_scale = out_scale;
+  a.gate = HeadGate{gate, ld_gate, gate_per_value};
   a.ws_o = ws_o;
   a.ws_ml = ws_ml;
   a.counters = counters;

@@ -1,6 +1,7 @@
-// liboxb, entry points of the gated delta rule (delta.cuh).
+// liboxb, entry points of the gated delta rule (delta.cuh, delta_chunk.cuh).
 #include "common.cuh"
 #include "delta.cuh"
+#include "delta_chunk.cuh"
 using namespace oxb;
 
 template <typename T, int NK, int THREADS>
@@ -26,15 +27,56 @@ static int delta_step_launch(const DeltaArgs& a, int B, cudaStream_t stream) {
   return (int)cudaErrorInvalidValue;
 }
 
+template <int KT, bool CH>
+static int delta_chunk_go(const DeltaChunkArgs& x, int B, int longest, int nv, cudaStream_t stream) {
+  constexpr int K = KT * 16;
+  const int V = x.a.V, chunks = (longest + DC - 1) / DC;
+  const int most[4] = {delta_prep_smem(K, 128).total, delta_state_smem(K, 32), delta_state_smem(K, 16), delta_output_smem(K, 128)};
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
+  if (!configured[dev]) {
+    constexpr cudaFuncAttribute attr = cudaFuncAttributeMaxDynamicSharedMemorySize;
+    cudaError_t e = cudaFuncSetAttribute(delta_prepare_kernel<KT, CH>, attr, most[0]);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_state_kernel<KT, 32>, attr, most[1]);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_state_kernel<KT, 16>, attr, most[2]);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_output_kernel<KT>, attr, most[3]);
+    if (e != cudaSuccess) return (int)e;
+    configured[dev] = true;
+  }
+  cudaError_t e = oxb_launch(delta_prepare_kernel<KT, CH>, dim3(chunks, x.a.H, B), dim3(DP_THREADS), (size_t)delta_prep_smem(K, V).total,
+                             stream, x);
+  if (e == cudaSuccess) {
+    const dim3 grid(V / nv, x.a.H, B);
+    e = nv == 32 ? oxb_launch(delta_state_kernel<KT, 32>, grid, dim3(DS_THREADS), (size_t)most[1], stream, x)
+                 : oxb_launch(delta_state_kernel<KT, 16>, grid, dim3(DS_THREADS), (size_t)most[2], stream, x);
+  }
+  if (e == cudaSuccess)
+    e = oxb_launch(delta_output_kernel<KT>, dim3(chunks, x.a.H, B), dim3(DO_THREADS), (size_t)delta_output_smem(K, V), stream, x);
+  if (e != cudaSuccess) return (int)e;
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+// Bytes of scratch per (chunk of 64 tokens, head) of heads that the chunk kernels cover, 0: not covered
+OXB_API int oxb_delta_chunk_bytes(int K, int V) {
+  const bool ok = (K == 32 || K == 64 || K == 96 || K == 128) && V > 0 && V % 16 == 0 && V <= 128;
+  return ok ? delta_plan(K, V).bytes : 0;
+}
+
 // Gated delta rule of a step: z [T, ld] holds q | k (G heads of K values) | v (H heads of V values) and, at the given columns,
 // gate, decay and beta; the state [num_slots, H, K, V] float32 is read and updated, the ring of convolution inputs [num_slots,
 // taps, channels] read.  Only sequences that feed min_rows .. max_rows rows take part.  write_window (single-row steps): the
-// ring is updated too; elsewhere oxb_delta_window does that afterwards.
+// ring is updated too; elsewhere oxb_delta_window does that afterwards.  chunk_values 0: delta_step_kernel; else (bf16) the chunk
+// kernels with that many values of the state per CTA (16 or 32), portions of up to `longest` rows and scratch ws of
+// (T / 64 + B) * H * oxb_delta_chunk_bytes(K, V) bytes.
 OXB_API int oxb_delta(const void* z, int ld, int dtype, int gate_off, int decay_off, int beta_off, const int* query_start,
                       const int* seq_lens, const int* slots, const float* conv, int taps, const float* a_log, const float* dt_bias,
                       const void* decay_up, int decay_rank, const void* gate_up, int gate_rank, const float* norm, float* state,
                       float* window, int num_slots, void* out, int ld_out, float out_scale, int B, int H, int G, int K, int V,
-                      int v_dim, float q_scale, float eps, int min_rows, int max_rows, int write_window, cudaStream_t stream) {
+                      int v_dim, float q_scale, float eps, int min_rows, int max_rows, int write_window, int chunk_values,
+                      int longest, void* ws, cudaStream_t stream) {
   if (B <= 0 || H <= 0) return 0;
   if (G <= 0 || H % G != 0 || V % 4 != 0 || V <= 0 || K <= 0 || taps <= 0 || B > 65535 || slots == nullptr ||
       (decay_up != nullptr && (decay_rank % 8 != 0 || decay_off % 8 != 0)) || (gate_up != nullptr && (gate_rank % 8 != 0 || gate_off % 8 != 0)) ||
@@ -43,7 +85,22 @@ OXB_API int oxb_delta(const void* z, int ld, int dtype, int gate_off, int decay_
   const DeltaArgs a{z, ld, gate_off, decay_off, beta_off, query_start, seq_lens, slots, conv, taps, a_log, dt_bias, decay_up, decay_rank,
                     gate_up, gate_rank, norm, state, window, num_slots, out, ld_out, out_scale, H, G, K, V, v_dim, q_scale, eps,
                     min_rows, max_rows, write_window};
-  return dtype == 0 ? delta_step_launch<float>(a, B, stream) : delta_step_launch<__nv_bfloat16>(a, B, stream);
+  if (chunk_values == 0) return dtype == 0 ? delta_step_launch<float>(a, B, stream) : delta_step_launch<__nv_bfloat16>(a, B, stream);
+  if (dtype != 2 || ws == nullptr || write_window || oxb_delta_chunk_bytes(K, V) == 0 || (chunk_values != 16 && chunk_values != 32) ||
+      V % chunk_values != 0 || longest <= 0 || H > 65535 || ld_out % 2 != 0 || (reinterpret_cast<uintptr_t>(out) & 3) != 0 ||
+      (decay_up != nullptr && decay_rank % 16 != 0) || (gate_up != nullptr && gate_rank % 16 != 0) || gate_off % 2 != 0)
+    return (int)cudaErrorInvalidValue;
+  const DeltaChunkArgs x{a, reinterpret_cast<uint8_t*>(ws)};
+  switch (K * 2 + (decay_up != nullptr)) {
+    case 64: return delta_chunk_go<2, false>(x, B, longest, chunk_values, stream);
+    case 65: return delta_chunk_go<2, true>(x, B, longest, chunk_values, stream);
+    case 128: return delta_chunk_go<4, false>(x, B, longest, chunk_values, stream);
+    case 129: return delta_chunk_go<4, true>(x, B, longest, chunk_values, stream);
+    case 192: return delta_chunk_go<6, false>(x, B, longest, chunk_values, stream);
+    case 193: return delta_chunk_go<6, true>(x, B, longest, chunk_values, stream);
+    case 256: return delta_chunk_go<8, false>(x, B, longest, chunk_values, stream);
+    default: return delta_chunk_go<8, true>(x, B, longest, chunk_values, stream);
+  }
 }
 
 OXB_API int oxb_delta_window(const void* z, int ld, int dtype, const int* query_start, const int* seq_lens, const int* slots, int taps,

@@ -223,6 +223,7 @@ OXB_API int oxb_latent_prefill(const void* q, const void* kv, const void* rot_ro
   a.group = 1;
   a.ld_out = H * v;
   a.out_scale = 1.f;
+  a.gate = HeadGate{nullptr, 0, 0};
   a.nope16 = (nope + 15) / 16;
   a.rot16 = (rot + 15) / 16;
   a.full_ld = 16 * (a.nope16 + a.rot16);
@@ -250,10 +251,13 @@ OXB_API int oxb_kv_gather(const void* cache, const int* block_tables, const int*
 // ld_out apart; width a multiple of 16.
 OXB_API int oxb_gqa_prefill(const void* q, const void* kv, void* out, int ld_out, float out_scale, const int* query_start,
                             const int* seq_lens, const int* span_lo, const int* span_off, const float* sink, int B, int T, int H,
-                            int G, int rows, int width, int window, float scale, int max_query_len, cudaStream_t stream) {
+                            int G, int rows, int width, int window, float scale, int max_query_len, const void* gate, int ld_gate,
+                            int gate_per_value, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || max_query_len <= 0 || rows <= 0) return 0;
   const LatentPrefillPlan pl = latent_prefill_plan(width, 0, width);
-  if (pl.smem == 0 || width % 16 != 0 || G <= 0 || H % G != 0 || H > 65535 || B > 65535) return (int)cudaErrorInvalidValue;
+  if (pl.smem == 0 || width % 16 != 0 || G <= 0 || H % G != 0 || H > 65535 || B > 65535 ||
+      (gate != nullptr && gate_per_value && (ld_gate % 8 != 0 || (reinterpret_cast<uintptr_t>(gate) & 15) != 0)))
+    return (int)cudaErrorInvalidValue;
   LatentPrefillArgs a;
   a.query_start = query_start;
   a.seq_lens = seq_lens;
@@ -266,6 +270,7 @@ OXB_API int oxb_gqa_prefill(const void* q, const void* kv, void* out, int ld_out
   a.group = H / G;
   a.ld_out = ld_out;
   a.out_scale = out_scale;
+  a.gate = HeadGate{gate, ld_gate, gate_per_value};
   a.nope16 = width / 16;
   a.rot16 = 0;
   a.full_ld = width;

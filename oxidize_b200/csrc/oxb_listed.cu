@@ -24,23 +24,6 @@ OXB_API int oxb_joint_norm(const float* res, const void* y0, const void* y1, con
   return dtype == 0 ? joint_norm_launch<float>(a, T, stream) : joint_norm_launch<__nv_bfloat16>(a, T, stream);
 }
 
-// o [T, ld] (H heads of W values, W a multiple of 4) times the sigmoid of its gates, in place
-OXB_API int oxb_head_gate(void* o, int ld, const void* gate, int ld_gate, int per_value, int dtype, int T, int H, int W,
-                          cudaStream_t stream) {
-  if (T <= 0) return 0;
-  if (W % 4 != 0 || ld % 4 != 0 || (per_value && ld_gate % 4 != 0)) return (int)cudaErrorInvalidValue;
-  const size_t blocks = ((size_t)T * H * W / 4 + 255) / 256;
-  const dim3 grid((unsigned)(blocks < 8192 ? blocks : 8192));
-  if (dtype == 0)
-    oxb_launch(head_gate_kernel<float>, grid, dim3(256), 0, stream, reinterpret_cast<float*>(o), ld, reinterpret_cast<const float*>(gate),
-               ld_gate, per_value, T, H, W);
-  else
-    oxb_launch(head_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, reinterpret_cast<__nv_bfloat16*>(o), ld,
-               reinterpret_cast<const __nv_bfloat16*>(gate), ld_gate, per_value, T, H, W);
-  OXB_CHECK_LAUNCH();
-  return 0;
-}
-
 template <typename T>
 static int head_prep_launch(HeadPrepArgs a, int rows, cudaStream_t stream) {
   // few tokens: their heads are spread over CTAs, a head per warp
@@ -88,11 +71,11 @@ static int gqa_simt_launch(const GqaSimtArgs& a, cudaStream_t stream) {
 OXB_API int oxb_gqa_attention_simt(const void* q, void* out, int ld_out, float out_scale, const void* cache, int dtype,
                                    const int* block_tables, const int* seq_lens, const int* query_start, const float* sink, int B,
                                    int max_blocks, int T, int H, int G, int width, int page, int num_blocks, int window, float scale,
-                                   cudaStream_t stream) {
+                                   const void* gate, int ld_gate, int gate_per_value, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
   if (G <= 0 || H % G != 0 || page <= 0) return (int)cudaErrorInvalidValue;
   const GqaSimtArgs a{q, out, cache, block_tables, seq_lens, query_start, sink, B, max_blocks, T, H, G, width, page, num_blocks,
-                      window, ld_out, scale, out_scale};
+                      window, ld_out, scale, out_scale, HeadGate{gate, ld_gate, gate_per_value}};
   return dtype == 0 ? gqa_simt_launch<float>(a, stream) : gqa_simt_launch<__nv_bfloat16>(a, stream);
 }
 

@@ -123,7 +123,7 @@ def _declare(L) -> None:
                                       i32, i32, vp]
     L.oxb_argmax.argtypes = [vp, i32, i32, i32, i32, vp, vp, i32, vp]
     L.oxb_paged_attention.argtypes = [vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, f32,
-                                      vp, i32, f32, vp, vp, vp, i32, vp]
+                                      vp, i32, f32, vp, vp, vp, i32, vp, i32, i32, vp]
     L.oxb_sample.argtypes = [vp, i32, i32, i32, vp, vp, vp, vp, vp, i32, vp, vp]
     L.oxb_gemm_quant.argtypes =[vp, vp, i32, sz, vp, i32, vp, vp, i32, i32, i32, i32, i32, i32, vp, sz, vp, i32, vp]
     u64p, ull = ctypes.POINTER(ctypes.c_uint64), ctypes.c_ulonglong
@@ -509,8 +509,10 @@ def attn_splits(B: int, nkv: int, mtiles: int, max_seq_len: int, sms: int) -> in
 
 
 def paged_attention(q, kv, layer, meta, scale, sliding_window=0, splits: Optional[int] = None, softcap: float = 0.0,
-                    sink: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, out_scale: float = 1.0):
-    """``sink`` [nq]: logits of the softmax denominator; ``out`` [T, nq * hd] may be a column slice of a wider buffer."""
+                    sink: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, out_scale: float = 1.0,
+                    gate: Optional[torch.Tensor] = None, gate_per_value: bool = False):
+    """``sink`` [nq]: logits of the softmax denominator; ``out`` [T, nq * hd] may be a column slice of a wider buffer; ``gate``
+    [T, nq] or, ``gate_per_value``, [T, nq * hd]: the outputs are multiplied by its sigmoid."""
     T, nq, hd = q.shape
     nkv = kv.spec.heads(layer)
     B = meta.seq_lens.shape[0]
@@ -534,7 +536,8 @@ def paged_attention(q, kv, layer, meta, scale, sliding_window=0, splits: Optiona
                                      meta.block_tables.data_ptr(), meta.seq_lens.data_ptr(), meta.query_start.data_ptr(),
                                      B, meta.block_tables.stride(0), nq, nkv, hd, KV_MODE[kv.dtype_name],
                                      max(1, meta.max_query_len), splits, sliding_window, scale, float(softcap), _p(sink),
-                                     out.stride(0), out_scale, _p(ws_o), _p(ws_ml), _p(cnt), kv.num_blocks, _stream()),
+                                     out.stride(0), out_scale, _p(ws_o), _p(ws_ml), _p(cnt), kv.num_blocks, _p(gate),
+                                     0 if gate is None else gate.stride(0), int(gate_per_value), _stream()),
            "oxb_paged_attention")
     return out
 

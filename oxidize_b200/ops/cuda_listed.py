@@ -27,10 +27,9 @@ def lib():
         L.oxb_head_prep.argtypes = ([vp, i32, i32, vp, vp, vp] + [i32] * 3 + [vp, vp, i32, f32] + [i32] * 5 + [vp, vp, i32, i32]
                                     + [f32, f32, vp, i32, i32, i32, vp, vp])
         L.oxb_joint_norm.argtypes = [vp] * 5 + [f32, f32, vp, i32, vp, vp, i32, vp, vp, vp] + [i32] * 3 + [f32, vp]
-        L.oxb_head_gate.argtypes = [vp, i32, vp] + [i32] * 6 + [vp]
-        L.oxb_gqa_attention_simt.argtypes = [vp, vp, i32, f32, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp]
+        L.oxb_gqa_attention_simt.argtypes = [vp, vp, i32, f32, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp, i32, i32, vp]
         L.oxb_kv_gather.argtypes = [vp] * 4 + [i32] * 7 + [vp, vp]
-        L.oxb_gqa_prefill.argtypes = [vp, vp, vp, i32, f32] + [vp] * 5 + [i32] * 7 + [f32, i32, vp]
+        L.oxb_gqa_prefill.argtypes = [vp, vp, vp, i32, f32] + [vp] * 5 + [i32] * 7 + [f32, i32, vp, i32, i32, vp]
         L.oxb_retention_chunk_supported.argtypes = L.oxb_retention_mma_supported.argtypes = [i32, i32]
         L.oxb_retention.argtypes = ([vp, i32, i32] + [vp] * 4 + [i32] * 3 + [vp, vp, i32, vp, i32, f32] + [i32] * 5 + [f32, f32]
                                     + [i32] * 4 + [vp, vp])
@@ -94,22 +93,20 @@ def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int,
     return q
 
 
-def head_gate(o: torch.Tensor, gate: torch.Tensor, spec) -> None:
-    """``o`` [T, heads * width] (may be a column slice) times the sigmoid of its gates, in place."""
-    _check(lib().oxb_head_gate(o.data_ptr(), o.stride(0), gate.data_ptr(), gate.stride(0), 1 if spec.gate == "value" else 0, DT[o.dtype],
-                               o.shape[0], spec.heads, spec.width, _stream()), "oxb_head_gate")
+def _gate(gate: Optional[torch.Tensor], spec):
+    return (None, 0, 0) if gate is None else (gate.data_ptr(), gate.stride(0), int(spec.gate == "value"))
 
 
-def attention_simt(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> None:
+def attention_simt(q, kv, layer: int, meta, spec, sink, out, out_scale: float, gate=None) -> None:
     T, H, W = q.shape
     B = meta.seq_lens.shape[0]
     _check(lib().oxb_gqa_attention_simt(q.data_ptr(), out.data_ptr(), out.stride(0), out_scale, kv.data[layer].data_ptr(), DT[q.dtype],
                                         meta.block_tables.data_ptr(), meta.seq_lens.data_ptr(), meta.query_start.data_ptr(), _p(sink),
                                         B, meta.block_tables.stride(0), T, H, spec.kv_heads, W, kv.page_size, kv.num_blocks,
-                                        spec.window, spec.scale, _stream()), "oxb_gqa_attention_simt")
+                                        spec.window, spec.scale, *_gate(gate, spec), _stream()), "oxb_gqa_attention_simt")
 
 
-def attention_prefill(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> None:
+def attention_prefill(q, kv, layer: int, meta, spec, sink, out, out_scale: float, gate=None) -> None:
     """Long portions: the visible rows are gathered from their pages, then flash attention on tcgen05."""
     T, H, W = q.shape
     B, G = meta.seq_lens.shape[0], spec.kv_heads
@@ -120,18 +117,24 @@ def attention_prefill(q, kv, layer: int, meta, spec, sink, out, out_scale: float
            "oxb_kv_gather")
     _check(lib().oxb_gqa_prefill(q.data_ptr(), dense.data_ptr(), out.data_ptr(), out.stride(0), out_scale, meta.query_start.data_ptr(),
                                  meta.seq_lens.data_ptr(), lo.data_ptr(), off.data_ptr(), _p(sink), B, T, H, G, rows, W, spec.window,
-                                 spec.scale, max(n for n, _ in meta.host_lens), _stream()), "oxb_gqa_prefill")
+                                 spec.scale, max(n for n, _ in meta.host_lens), *_gate(gate, spec), _stream()), "oxb_gqa_prefill")
 
 
-def attention(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> None:
-    """Attention of a step's queries over the cache into ``out`` [T, heads * width] (may be a column slice)."""
+def attention(q, kv, layer: int, meta, spec, sink, out, out_scale: float, gate: Optional[torch.Tensor] = None) -> None:
+    """Attention of a step's queries over the cache into ``out`` [T, heads * width] (may be a column slice), times the sigmoid of
+    ``gate`` ([T, heads or more], or [T, heads * width] with a gate per value)."""
     if q.dtype != torch.bfloat16 or kv.page_size != 16 or spec.width not in HEAD_WIDTHS:
-        attention_simt(q, kv, layer, meta, spec, sink, out, out_scale)
+        attention_simt(q, kv, layer, meta, spec, sink, out, out_scale, gate)
         return
+
+    def paged(qs, sub, o, gs) -> None:
+        opcuda.paged_attention(qs, kv, layer, sub, spec.scale, spec.window, sink=sink, out=o, out_scale=out_scale, gate=gs,
+                               gate_per_value=spec.gate == "value")
+
     if (not meta.host_lens or max(n for n, _ in meta.host_lens) < latent.EXPAND_ROWS
             or not lib().oxb_latent_prefill_supported(spec.width, 0, spec.width)
             or latent._spans(meta, spec.window)[2] > latent.MAX_SPAN):
-        opcuda.paged_attention(q, kv, layer, meta, spec.scale, spec.window, sink=sink, out=out, out_scale=out_scale)
+        paged(q, meta, out, gate)
         return
     starts = [0]
     for n, _ in meta.host_lens:
@@ -140,10 +143,11 @@ def attention(q, kv, layer: int, meta, spec, sink, out, out_scale: float) -> Non
     for b0, b1, big in runs:
         t0, t1 = starts[b0], starts[b1]
         sub = meta if len(runs) == 1 else latent._sub_batch(meta, b0, b1, t0, t1)
+        gs = None if gate is None else gate[t0:t1]
         if big:
-            attention_prefill(q[t0:t1], kv, layer, sub, spec, sink, out[t0:t1], out_scale)
+            attention_prefill(q[t0:t1], kv, layer, sub, spec, sink, out[t0:t1], out_scale, gs)
         else:
-            opcuda.paged_attention(q[t0:t1], kv, layer, sub, spec.scale, spec.window, sink=sink, out=out[t0:t1], out_scale=out_scale)
+            paged(q[t0:t1], sub, out[t0:t1], gs)
 
 
 # --------------------------------------------------------------------------- retention
@@ -213,9 +217,7 @@ def listed_mixer(x: torch.Tensor, lw, spec, ropes, meta, kv, kv_layer: int, stat
             raise ValueError(f"cache rows of listed layers are kept in the compute type on the GPU ({x.dtype}), not {kv.dtype_name}")
         na, no = a.proj_dim, a.out_dim
         q = head_prep(z[:, : a.qkv_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps, *first_values(z, a, lw, carry))
-        attention(q, kv, kv_layer, meta, a, lw.sink, outs[0][:, :no], sl)
-        if a.gate:
-            head_gate(outs[0][:, :no], z[:, a.qkv_dim : na], a)
+        attention(q, kv, kv_layer, meta, a, lw.sink, outs[0][:, :no], sl, z[:, a.qkv_dim : na] if a.gate else None)
     out = outs[-1][:, 0 if apart else no :]
     if d is not None:
         from . import cuda_delta

@@ -369,10 +369,10 @@ def synth_layered_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: i
         if spec.weights_of is not None:
             layers.append(layers[spec.weights_of])
             continue
-        if cfg.norm_placement == "sandwich":
+        if cfg.norm_placement in ("sandwich", "parallel"):
             if tp_size > 1:
                 raise ValueError("layers with per-sequence states and norms over all heads are not sharded")
-            layers.append(_synth_listed(spec, h, mat, ones))
+            layers.append((_synth_listed if cfg.norm_placement == "sandwich" else _synth_joint)(spec, h, mat, ones))
             continue
         m, f = spec.mixer, spec.ffn
         H, own = m.heads // tp_size, m.kv_from is None
@@ -387,8 +387,9 @@ def synth_layered_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: i
             lw.w_down = LinearWeight([dense_qtensor(mat(h, f.size // tp_size))])
         layers.append(lw)
     v = cfg.vocab_size // tp_size
-    mw = ModelWeights(cfg, dense_qtensor(mat(cfg.vocab_size, h, own=False)), layers, ones(h), LinearWeight([dense_qtensor(mat(v, h))]),
-                      [], tp_rank, tp_size, 0, 1, 0, v * tp_rank)
+    embed = dense_qtensor(mat(cfg.vocab_size, h, own=False))
+    head = embed if cfg.tie_embeddings else dense_qtensor(mat(v, h))
+    mw = ModelWeights(cfg, embed, layers, ones(h), LinearWeight([head]), [], tp_rank, tp_size, 0, 1, 0, v * tp_rank)
     mw.out_norm_bias = zeros(h)
     if cfg.embed_norm:
         mw.embed_norm, mw.embed_norm_bias = ones(h), zeros(h)
@@ -423,6 +424,37 @@ def _synth_listed(spec, h: int, mat, ones) -> LayerWeights:
             lw.shared_gate_up, lw.shared_down = pair(f.shared)
     else:
         lw.w_gate_up, lw.w_down = pair(f)
+    return lw
+
+
+def _synth_joint(spec, h: int, mat, ones) -> LayerWeights:
+    """One layer with one norm that both branches read."""
+    from ..models.config import ParallelSpec
+    from ..models.layered import dense_qtensor, listed_experts, listed_mixer
+
+    a, d, f = spec.attention, spec.delta, spec.ffn
+    att, rec = {}, {}
+    if a is not None:
+        att = {"q": mat(a.heads * a.dim, h), "k": mat(a.kv_heads * a.dim, h), "v": mat(a.kv_heads * a.v_dim, h),
+               "o": mat(h, a.heads * a.v_dim), "g": mat(a.heads * (a.v_dim if a.gate == "value" else 1), h), "vmix": 0.5 * ones(1),
+               "q.norm": ones(a.dim), "k.norm": ones(a.dim)}
+        att.update({n + ".b": 0.1 * ones(att[n].shape[0]) for n in "qkv"})
+    if d is not None:
+        rows = {"q": d.kv_heads * d.dim, "k": d.kv_heads * d.dim, "v": d.heads * d.v_dim, "b": d.heads}
+        rows.update({"a1": d.decay_rank} if d.decay_rank else {"a": d.heads})
+        rows.update({"g1": d.gate_rank} if d.gate_rank else {"g": d.heads * d.v_dim})
+        rec = {n: mat(r, h) for n, r in rows.items()}
+        rec.update({n + ".conv": mat(rows[n], d.conv) * 25.0 for n in "qkv"})
+        rec.update({"o": mat(h, d.heads * d.v_dim), "A_log": -1.0 * ones(d.heads), "norm": ones(d.v_dim),
+                    "dt_bias": -2.0 * ones(d.heads * (d.dim if d.decay_rank else 1))})
+        rec.update({"a2": mat(d.heads * d.dim, d.decay_rank)} if d.decay_rank else {})
+        rec.update({"g2": mat(d.heads * d.v_dim, d.gate_rank)} if d.gate_rank else {})
+    lw = LayerWeights(attn_norm=ones(h), ffn_norm=None, **listed_mixer(spec, att, rec))
+    if isinstance(spec.mixer, ParallelSpec):
+        lw.out_norms = (ones(h), ones(h))
+    if f is not None:
+        lw.router, lw.router_bias = dense_qtensor(mat(f.n_experts, h)), 0.0 * ones(f.n_experts)
+        lw.experts = listed_experts(f, ((None, mat(f.expert.size, h), mat(h, f.expert.size)) for _ in range(f.n_experts)), h)
     return lw
 
 
