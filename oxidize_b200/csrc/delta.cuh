@@ -43,6 +43,8 @@ struct DeltaArgs {
 
 __device__ __forceinline__ float delta_silu(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float delta_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
+// (for activations and output gates of the 16-bit path)
+__device__ __forceinline__ float delta_sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 __device__ __forceinline__ float delta_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
 // Dot product of n values (n % 8 == 0, both rows aligned to 8 values).

@@ -9,46 +9,51 @@
 // delta_state_kernel, chunk after chunk, the values of a head dealt out to CTAs: U = U0 - W S, then S'.
 // delta_output_kernel, all chunks at once: O, its norm and gate.
 //
-// Exponents are never positive: a block of L and P that lies off the diagonal takes G relative to the last token ahead of its
-// rows (rows exp(G_t - G_ref), columns exp(G_ref - G_s)); blocks of 16 on the diagonal multiply a column by one token's decay
-// at a time.  G is kept as running sums within blocks of 16 and the blocks' totals, so that what lies between two tokens is
-// never the small difference of two large sums; a token's logarithm ends at -50.  Every float32 factor enters the bf16 products as a high and a low half, and hi hi + hi lo + lo hi is summed in
-// float32 (see retention.cuh).
+// A portion is worked off in rounds of as many chunks as fill the GPU once, so that what the kernels hand on stays in the L2.
+//
+// G is kept in binary logarithms, as running sums within blocks of 16 tokens and the blocks' totals, so that what lies between
+// two tokens is never the small difference of two large sums; a token's logarithm ends at -72.  In L and P a block off the
+// diagonal takes its rows relative to the start of their block and its columns relative to that point, so that no exponent is
+// positive; a block on the diagonal takes both relative to its start unless a channel loses more than 2^-60 in it, in which
+// case its columns are multiplied by one token's decay at a time.  Every float32 factor enters the bf16 products as a high and
+// a low half, and hi hi + hi lo + lo hi is summed in float32 (see retention.cuh).
 #pragma once
+#include <type_traits>
+
 #include "delta.cuh"
 #include "retention.cuh"
 
 namespace oxb {
 
-constexpr int DC = 64;              // tokens per chunk
-constexpr int DC_LD = DC + 4;       // floats of a row of L and of the inverse
+constexpr int DC = 64;                // tokens per chunk
+constexpr int DC_LD = DC + 4;         // floats of a row of L and of the inverse
 constexpr int DC_PROW = DC * 2 + 16;  // bytes of a row of 64 halves in shared memory
 
 // Scratch of one (chunk, head), in bytes.
 struct DeltaPlan {
-  int w, kb, qt, p, u0, u, s, gend, bytes;  // offsets; pairs of halves lie behind each other (hi, lo)
+  int w, kb, u0, gend, qt, p, u, s, bytes;  // offsets; pairs of halves lie behind each other (hi, lo)
 };
 __host__ __device__ inline DeltaPlan delta_plan(int K, int V) {
   DeltaPlan p;
   p.w = 0;
   p.kb = p.w + 2 * DC * K * 2;
-  p.qt = p.kb + 2 * DC * K * 2;
+  p.u0 = p.kb + 2 * DC * K * 2;
+  p.gend = p.u0 + DC * V * 4;
+  p.qt = p.gend + K * 4;
   p.p = p.qt + 2 * DC * K * 2;
-  p.u0 = p.p + 2 * DC * DC * 2;
-  p.u = p.u0 + DC * V * 4;
+  p.u = p.p + 2 * DC * DC * 2;
   p.s = p.u + 2 * DC * V * 2;
-  p.gend = p.s + 2 * K * V * 2;
-  p.bytes = p.gend + K * 4;
+  p.bytes = p.s + 2 * K * V * 2;
   return p;
 }
 
 struct DeltaChunkArgs {
   DeltaArgs a;
-  uint8_t* ws;  // (T / 64 + B) * H blocks of delta_plan(K, V).bytes
+  uint8_t* ws;        // B * round * H blocks of delta_plan(K, V).bytes
+  int chunk0, round;  // chunks [chunk0, chunk0 + round) of every portion
 };
-// (sequence b's first block: its chunks never need more than the rows ahead of it and one each)
-__device__ __forceinline__ uint8_t* delta_block(const DeltaChunkArgs& x, int bytes, int q0, int b, int chunk, int h) {
-  return x.ws + ((size_t)(q0 / DC + b + chunk) * x.a.H + h) * bytes;
+__device__ __forceinline__ uint8_t* delta_block(const DeltaChunkArgs& x, int bytes, int b, int chunk, int h) {
+  return x.ws + ((size_t)(b * x.round + chunk - x.chunk0) * x.a.H + h) * bytes;
 }
 
 __device__ __forceinline__ void delta_split8(const float* v, void* hi_at, void* lo_at) {
@@ -62,115 +67,110 @@ __device__ __forceinline__ void delta_load8(const float* p, float* v) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
   v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
 }
+__device__ __forceinline__ void delta_load4(const __nv_bfloat16* p, float* v) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y);
+  v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
+}
 
 // ----------------------------------------------------------------------------- chunks by themselves
-constexpr int DP_THREADS = 512, DP_TAPS = 4;
-constexpr float DP_FLOOR = -50.f;  // exp of it is far below the rounding of anything it is added to
+constexpr int DP_THREADS = 512, DP_WARPS = DP_THREADS / 32, DP_TAPS = 4, DP_RAW = DC + DP_TAPS - 1;
+constexpr float DP_FLOOR = -72.f;  // 2^ of it is far below the rounding of anything it is added to
+constexpr float DP_RANGE = -60.f;  // what a block on the diagonal may lose
 
 struct DeltaPrepSmem {
-  int k, q, g, stage, l, misc, total;  // byte offsets
-  int rows_q, cols, t, tp, kt, v;      // offsets of what shares the staging area
+  int k, q, g, kt, tp, l, t, misc, total;  // byte offsets
 };
 __host__ __device__ inline DeltaPrepSmem delta_prep_smem(int K, int V) {
   DeltaPrepSmem s;
-  const int f32 = DC * (K + 4) * 4, half = DC * (K * 2 + 16), vhalf = DC * (V * 2 + 16);
+  const int f32 = DC * (K + 8) * 4, vhalves = 2 * DC * (V * 2 + 16), rawv = DP_RAW * V * 2, tp = 2 * DC * DC_PROW;
   s.k = 0;
   s.q = s.k + f32;
-  s.g = s.q + f32;
-  s.stage = s.g + f32;
-  // first: rows of k (hi, lo) | rows of q | columns; then: inverse (float32) | inverse * beta (hi, lo) | exp(G) k | v
-  s.rows_q = 2 * half;
-  s.cols = 4 * half;
-  s.t = 0;
-  s.tp = DC * DC_LD * 4;
-  s.kt = s.tp + 2 * DC * DC_PROW;
-  s.v = s.kt + 2 * half;
-  const int a = 6 * half, b = s.v + 2 * vhalf;
-  s.l = s.stage + (a > b ? a : b);
-  s.misc = s.l + DC * DC_LD * 4;
-  s.total = s.misc + (DC + 4 * K) * 4;  // beta | totals of blocks
+  s.g = s.q + f32;                               // decays; later v as halves
+  s.kt = s.g + (f32 > vhalves ? f32 : vhalves);  // raw rows of q and k; later exp(G) k as halves
+  s.tp = s.kt + f32;                             // raw rows of v; later the inverse times beta as halves
+  s.l = s.tp + ((tp > rawv ? tp : rawv) + 15) / 16 * 16;
+  s.t = s.l + DC * DC_LD * 4;
+  s.misc = s.t + DC * DC_LD * 4;
+  s.total = s.misc + (DC + 4 * K + 8) * 4;       // beta | totals of blocks | flags of blocks
   return s;
 }
 
-// Eight channels of the convolution and silu for tokens [j0, j0 + 8) of a portion (rows at or past n: zero); put(token, values).
+// Four channels (this lane's) of the convolution and silu for tokens [t0, t0 + 4) of the chunk, out of raw rows in shared memory
+// (`raw`: this lane's channels three tokens ahead of the chunk, rows `row` values apart), or, for longer convolutions, out of
+// global memory; rows at or past n: zero.
 template <typename F>
-__device__ __forceinline__ void delta_conv8(const DeltaArgs& a, const __nv_bfloat16* z, const float* ring, int C, int pos0, int j0, int n,
-                                            int ch, F put) {
+__device__ __forceinline__ void delta_conv4(const DeltaArgs& a, const __nv_bfloat16* raw, int row, const __nv_bfloat16* z, const float* ring,
+                                            int C, int pos0, int c0, int t0, int n, int ch, F put) {
   if (a.taps <= DP_TAPS) {
-    float w[DP_TAPS][8], x[DP_TAPS][8];
+    float w[DP_TAPS][4], x[DP_TAPS][4];
 #pragma unroll
     for (int i = 0; i < DP_TAPS; ++i) {  // (shorter convolutions: zeros on the oldest rows)
       const int tap = i - (DP_TAPS - a.taps);
-      if (tap >= 0) delta_load8(a.conv + (size_t)tap * C + ch, w[i]);
-      else
-#pragma unroll
-        for (int e = 0; e < 8; ++e) w[i][e] = 0.f;
+      const float4 v = tap >= 0 ? *reinterpret_cast<const float4*>(a.conv + (size_t)tap * C + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
+      w[i][0] = v.x, w[i][1] = v.y, w[i][2] = v.z, w[i][3] = v.w;
     }
-    auto fetch = [&](int j, float* v) {
-      const int p = pos0 + j;
-      if (j >= 0 && j < n) head_load8(z + (size_t)j * a.ld + ch, v);
-      else if (j < 0 && p >= 0 && j >= 1 - a.taps) delta_load8(ring + (size_t)(p % a.taps) * C + ch, v);
-      else
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[e] = 0.f;
-    };
+    for (int i = 0; i < DP_TAPS - 1; ++i) delta_load4(raw + (t0 + i) * row, x[i]);
 #pragma unroll
-    for (int i = 0; i < DP_TAPS - 1; ++i) fetch(j0 - (DP_TAPS - 1) + i, x[i]);
+    for (int t = 0; t < 4; ++t) {
+      delta_load4(raw + (t0 + t + DP_TAPS - 1) * row, x[(t + DP_TAPS - 1) % DP_TAPS]);
+      float y[4];
 #pragma unroll
-    for (int t = 0; t < 8; ++t) {
-      fetch(j0 + t, x[(t + DP_TAPS - 1) % DP_TAPS]);
-      float y[8];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) {
+      for (int e = 0; e < 4; ++e) {
         float s = 0.f;
 #pragma unroll
         for (int i = 0; i < DP_TAPS; ++i) s = fmaf(w[i][e], x[(t + i) % DP_TAPS][e], s);
-        y[e] = j0 + t < n ? delta_silu(s) : 0.f;
+        y[e] = t0 + t < n ? s * delta_sigmoid_fast(s) : 0.f;
       }
-      put(t, y);
+      put(t0 + t, y);
     }
   } else {
-    for (int t = 0; t < 8; ++t) {
-      float y[8];
-      for (int e = 0; e < 8; ++e) y[e] = j0 + t < n ? delta_conv(a, z, ring, C, pos0, j0 + t, ch + e) : 0.f;
+    for (int t = t0; t < t0 + 4; ++t) {
+      float y[4];
+      for (int e = 0; e < 4; ++e) y[e] = t < n ? delta_conv(a, z, ring, C, pos0, c0 + t, ch + e) : 0.f;
       put(t, y);
     }
   }
 }
 
-// A 16 x 16 tile (two accumulators of 8 columns) of rows . columns^T over K values, both as halves.
-template <int KT>
-__device__ __forceinline__ void delta_tile(uint32_t rows_hi, uint32_t rows_lo, uint32_t cols_hi, uint32_t cols_lo, int row_bytes, int lane,
-                                           float (&acc)[2][4]) {
-  const int mi = lane >> 3, r8 = lane & 7;
-  const uint32_t ao = ((mi & 1) * 8 + r8) * row_bytes + (mi >> 1) * 16, bo = ((mi >> 1) * 8 + r8) * row_bytes + (mi & 1) * 16;
+// Products of a low-rank projection: 16 rows (this lane's two: r0, r1) by nt <= NT tiles of 8 columns (`up`: this lane's row of
+// the first).  Which values of a k-step a lane holds is free, as long as both operands agree: four neighbouring ones.
+template <int NT, int STEPS>
+__device__ __forceinline__ void delta_low_rank_steps(const __nv_bfloat16* r0, const __nv_bfloat16* r1, const __nv_bfloat16* up, int rank,
+                                                     int nt, float (&acc)[NT][4]) {
+  uint2 x0[STEPS], x1[STEPS], w[STEPS][NT];
 #pragma unroll
-  for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  for (int j = 0; j < STEPS; ++j) {
+    x0[j] = *reinterpret_cast<const uint2*>(r0 + 16 * j);
+    x1[j] = *reinterpret_cast<const uint2*>(r1 + 16 * j);
 #pragma unroll
-  for (int ks = 0; ks < KT; ++ks) {
-    uint32_t ah[4], al[4], bh[4], bl[4];
-    ldmatrix_x4(rows_hi + ao + ks * 32, ah[0], ah[1], ah[2], ah[3]);
-    ldmatrix_x4(rows_lo + ao + ks * 32, al[0], al[1], al[2], al[3]);
-    ldmatrix_x4(cols_hi + bo + ks * 32, bh[0], bh[1], bh[2], bh[3]);
-    ldmatrix_x4(cols_lo + bo + ks * 32, bl[0], bl[1], bl[2], bl[3]);
+    for (int i = 0; i < NT; ++i) w[j][i] = i < nt ? *reinterpret_cast<const uint2*>(up + (size_t)i * 8 * rank + 16 * j) : make_uint2(0, 0);
+  }
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      mma_bf16_16816(acc[i], ah, bh[2 * i], bh[2 * i + 1]);
-      mma_bf16_16816(acc[i], ah, bl[2 * i], bl[2 * i + 1]);
-      mma_bf16_16816(acc[i], al, bh[2 * i], bh[2 * i + 1]);
-    }
+  for (int j = 0; j < STEPS; ++j) {
+    const uint32_t av[4] = {x0[j].x, x1[j].x, x0[j].y, x1[j].y};
+#pragma unroll
+    for (int i = 0; i < NT; ++i) mma_bf16_16816(acc[i], av, w[j][i].x, w[j][i].y);
   }
 }
+template <int NT>
+__device__ __forceinline__ void delta_low_rank(const __nv_bfloat16* r0, const __nv_bfloat16* r1, const __nv_bfloat16* up, int rank, int nt,
+                                               float (&acc)[NT][4]) {
+  int ks = 0;
+  for (; ks + 64 <= rank; ks += 64) delta_low_rank_steps<NT, 4>(r0 + ks, r1 + ks, up + ks, rank, nt, acc);
+  for (; ks < rank; ks += 16) delta_low_rank_steps<NT, 1>(r0 + ks, r1 + ks, up + ks, rank, nt, acc);
+}
 
-// grid (chunks of the longest portion, H, B); CH: a decay per key channel.
+// grid (chunks of the round, H, B); CH: a decay per key channel.
 template <int KT, bool CH>
 __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const DeltaChunkArgs x) {
-  constexpr int K = KT * 16, KF = K + 4, K8 = K / 8, CPL = K / 32;
-  constexpr int RB = K * 2 + 16;  // bytes of a row of halves
+  constexpr int K = KT * 16, KF = K + 8, K8 = K / 8, CPL = K / 32;
+  constexpr int RB = K * 2 + 16, HALF = DC * RB;  // bytes of a row of halves, of 64 rows
   extern __shared__ __align__(16) uint8_t dp_smem[];
   pdl_launch_dependents();
   const DeltaArgs& a = x.a;
-  const int b = blockIdx.z, h = blockIdx.y, chunk = blockIdx.x;
+  const int b = blockIdx.z, h = blockIdx.y, chunk = x.chunk0 + blockIdx.x;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int q0 = a.query_start[b], n_all = a.query_start[b + 1] - q0, slot = a.slots[b], c0 = chunk * DC;
   if (n_all < a.min_rows || n_all > a.max_rows || c0 >= n_all || (unsigned)slot >= (unsigned)a.num_slots) {
@@ -181,51 +181,59 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
   const int pos0 = a.seq_lens[b] - n_all;
   const DeltaPlan pl = delta_plan(K, V);
   const DeltaPrepSmem sm = delta_prep_smem(K, V);
-  uint8_t* block = delta_block(x, pl.bytes, q0, b, chunk, h);
+  uint8_t* block = delta_block(x, pl.bytes, b, chunk, h);
   float *sK = reinterpret_cast<float*>(dp_smem + sm.k), *sQ = reinterpret_cast<float*>(dp_smem + sm.q);
   float* sG = reinterpret_cast<float*>(dp_smem + sm.g);  // [64][KF], or [64] with one decay per head: sums within blocks of 16
-  uint8_t* stage = dp_smem + sm.stage;
-  float *sL = reinterpret_cast<float*>(dp_smem + sm.l), *beta = reinterpret_cast<float*>(dp_smem + sm.misc), *total = beta + DC;  // [4][K], or [4]
-  const int half = DC * RB, RV = V * 2 + 16;
+  float *sL = reinterpret_cast<float*>(dp_smem + sm.l), *sT = reinterpret_cast<float*>(dp_smem + sm.t);
+  float *beta = reinterpret_cast<float*>(dp_smem + sm.misc), *total = beta + DC;  // total: [4][K], or [4]
+  int* wild = reinterpret_cast<int*>(total + 4 * K);                              // [4] blocks whose decays leave the range
+  __nv_bfloat16 *raw_qk = reinterpret_cast<__nv_bfloat16*>(dp_smem + sm.kt), *raw_v = reinterpret_cast<__nv_bfloat16*>(dp_smem + sm.tp);
+  const int RV = V * 2 + 16, VHALF = DC * RV;
   const float* ring = a.window + (size_t)slot * a.taps * C;
   const __nv_bfloat16* z = reinterpret_cast<const __nv_bfloat16*>(a.z) + (size_t)q0 * a.ld;
+  if (tid < 4) wild[tid] = 0;
   pdl_wait();
-  // ---- convolutions of q and k, decays, step sizes
-  for (int i = tid; i < 2 * K8 * 8; i += DP_THREADS) {
-    const int c = i % (2 * K8), j0 = i / (2 * K8) * 8;
-    float* dst = (c < K8 ? sQ + c * 8 : sK + (c - K8) * 8) + j0 * KF;
-    delta_conv8(a, z, ring, C, pos0, c0 + j0, n_all, c < K8 ? kvh * K + c * 8 : (a.G + kvh) * K + (c - K8) * 8,
-                [&](int t, const float* y) {
-                  *reinterpret_cast<float4*>(dst + t * KF) = make_float4(y[0], y[1], y[2], y[3]);
-                  *reinterpret_cast<float4*>(dst + t * KF + 4) = make_float4(y[4], y[5], y[6], y[7]);
-                });
+  // ---- raw rows of q | k and of v, from three tokens ahead of the chunk on
+  if (a.taps <= DP_TAPS) {
+    const int pieces = 2 * K8 + V8;
+    for (int i = tid; i < DP_RAW * pieces; i += DP_THREADS) {
+      const int r = i / pieces, p = i % pieces, j = c0 - (DP_TAPS - 1) + r;
+      const int ch = p < K8 ? kvh * K + p * 8 : (p < 2 * K8 ? (a.G + kvh) * K + (p - K8) * 8 : 2 * a.G * K + h * V + (p - 2 * K8) * 8);
+      __nv_bfloat16* dst = p < 2 * K8 ? raw_qk + (r * 2 * K8 + p) * 8 : raw_v + (r * V8 + p - 2 * K8) * 8;
+      if (j >= 0 && j < n_all) {
+        cp_async16(dst, z + (size_t)j * a.ld + ch);
+      } else if (j < 0 && pos0 + j >= 0 && j > -a.taps) {  // (an earlier step's projections: 16-bit values)
+        float v[8];
+        delta_load8(ring + (size_t)((pos0 + j) % a.taps) * C + ch, v);
+        *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+      } else {
+        *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+      }
+    }
   }
+  cp_async_commit();
+  // ---- decays and step sizes
   if (tid < DC) beta[tid] = tid < n ? delta_sigmoid(lat_f32(z[(size_t)(c0 + tid) * a.ld + a.beta_off + h])) : 0.f;
-  const float rate = expf(a.a_log[h]);
-  if (CH) {  // z . decay_up^T for 16 tokens x K / 4 channels per warp
-    const int mt = warp & 3, nt0 = (warp >> 2) * (K / 32);
+  const float rate = expf(a.a_log[h]) * 1.4426950408889634f;
+  if (CH) {  // 16 tokens x K / 4 channels per warp
+    const int mt = warp & 3, d0 = (warp >> 2) * (K / 4);
     float acc[K / 32][4];
 #pragma unroll
     for (int i = 0; i < K / 32; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-    const __nv_bfloat16* r0 = z + (size_t)(c0 + min(mt * 16 + g, n - 1)) * a.ld + a.decay_off + 4 * t4;
-    const __nv_bfloat16* r1 = z + (size_t)(c0 + min(mt * 16 + g + 8, n - 1)) * a.ld + a.decay_off + 4 * t4;
-    const __nv_bfloat16* up = reinterpret_cast<const __nv_bfloat16*>(a.decay_up) + (size_t)(h * K + nt0 * 8 + g) * a.decay_rank + 4 * t4;
-    for (int ks = 0; ks < a.decay_rank; ks += 16) {  // (which values of a k-step a lane holds is free, as long as both operands agree)
-      const uint2 x0 = *reinterpret_cast<const uint2*>(r0 + ks), x1 = *reinterpret_cast<const uint2*>(r1 + ks);
-      const uint32_t av[4] = {x0.x, x1.x, x0.y, x1.y};
+    const __nv_bfloat16* rows = z + (size_t)c0 * a.ld + a.decay_off + 4 * t4;
+    delta_low_rank<K / 32>(rows + (size_t)min(mt * 16 + g, n - 1) * a.ld, rows + (size_t)min(mt * 16 + g + 8, n - 1) * a.ld,
+                           reinterpret_cast<const __nv_bfloat16*>(a.decay_up) + (size_t)(h * K + d0 + g) * a.decay_rank + 4 * t4, a.decay_rank,
+                           K / 32, acc);
 #pragma unroll
-      for (int i = 0; i < K / 32; ++i) {
-        const uint2 w = *reinterpret_cast<const uint2*>(up + (size_t)i * 8 * a.decay_rank + ks);
-        mma_bf16_16816(acc[i], av, w.x, w.y);
+    for (int i = 0; i < K / 32; ++i) {
+      const float2 dt = *reinterpret_cast<const float2*>(a.dt_bias + h * K + d0 + i * 8 + 2 * t4);
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        const int t = mt * 16 + g + 8 * (e >> 1);
+        const float v0 = fmaxf(-rate * delta_softplus(acc[i][e] + dt.x), DP_FLOOR), v1 = fmaxf(-rate * delta_softplus(acc[i][e + 1] + dt.y), DP_FLOOR);
+        *reinterpret_cast<float2*>(sG + t * KF + d0 + i * 8 + 2 * t4) = t < n ? make_float2(v0, v1) : make_float2(0.f, 0.f);
       }
     }
-#pragma unroll
-    for (int i = 0; i < K / 32; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = mt * 16 + g + 8 * (e >> 1), d = (nt0 + i) * 8 + 2 * t4 + (e & 1);
-        sG[t * KF + d] = t < n ? fmaxf(-rate * delta_softplus(acc[i][e] + a.dt_bias[h * K + d]), DP_FLOOR) : 0.f;
-      }
   } else if (warp == 0) {
     float v[2];
 #pragma unroll
@@ -245,26 +253,22 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
     sG[2 * lane + 1] = s;
     if ((lane & 7) == 7) total[lane >> 3] = s;
   }
+  cp_async_wait<0>();
   __syncthreads();
-  // ---- unit vectors; running sums of the decays
-  for (int t = warp; t < DC; t += DP_THREADS / 32) {
-    float qv[CPL], kv[CPL], qq = 0.f, kk = 0.f;
-#pragma unroll
-    for (int i = 0; i < CPL; ++i) {
-      qv[i] = sQ[t * KF + lane + 32 * i];
-      kv[i] = sK[t * KF + lane + 32 * i];
-      qq += qv[i] * qv[i];
-      kk += kv[i] * kv[i];
-    }
-    const float iq = rsqrtf(warp_sum(qq) + 1e-6f) * a.q_scale, ik = rsqrtf(warp_sum(kk) + 1e-6f);
-#pragma unroll
-    for (int i = 0; i < CPL; ++i) {
-      sQ[t * KF + lane + 32 * i] = qv[i] * iq;
-      sK[t * KF + lane + 32 * i] = kv[i] * ik;
-    }
+  // ---- q and k: convolution, silu, unit vectors; a warp has four tokens, a lane four channels
+#pragma unroll 1
+  for (int side = 0; side < 2; ++side) {
+    const int d = lane * 4, dc = min(d, K - 4);
+    float* dst = (side ? sK : sQ) + d;
+    delta_conv4(a, raw_qk + side * K + dc, 2 * K, z, ring, C, pos0, c0, warp * 4, n, (side ? a.G + kvh : kvh) * K + dc,
+                [&](int t, const float* y) {
+                  const float ss = d < K ? (y[0] * y[0] + y[1] * y[1]) + (y[2] * y[2] + y[3] * y[3]) : 0.f;
+                  const float f = rsqrtf(warp_sum(ss) + 1e-6f) * (side ? 1.f : a.q_scale);
+                  if (d < K) *reinterpret_cast<float4*>(dst + t * KF) = make_float4(y[0] * f, y[1] * f, y[2] * f, y[3] * f);
+                });
   }
-  if (CH) {
-    const int d = tid % K, blk = tid / K;  // (512 threads: four blocks of up to 128 channels)
+  if (CH) {  // running sums (512 threads: four blocks of up to 128 channels)
+    const int d = tid % K, blk = tid / K;
     if (blk < 4) {
       float v[16];
 #pragma unroll
@@ -274,112 +278,147 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
 #pragma unroll
       for (int i = 1; i < 16; ++i) sG[(blk * 16 + i) * KF + d] = v[i];
       total[blk * K + d] = v[15];
+      if (v[15] < DP_RANGE) wild[blk] = 1;
     }
   }
   __syncthreads();
-  auto add_totals8 = [&](int from, int to, int p, float* v) {  // totals of blocks [from, to)
-    for (int i = from; i < to; ++i) {
-#pragma unroll
-      for (int e = 0; e < 8; ++e) v[e] += total[CH ? i * K + p * 8 + e : i];
+  // logarithm of the decay from the chunk's start through token t, and behind token t through the end of block `block1` - 1, channels d
+  // and d + 1
+  auto since2 = [&](int t, int d) {
+    float2 v;
+    if (CH) v = *reinterpret_cast<const float2*>(sG + t * KF + d);
+    else v.x = v.y = sG[t];
+    for (int i = 0; i < t >> 4; ++i) {
+      v.x += total[CH ? i * K + d : i];
+      v.y += total[CH ? i * K + d + 1 : i];
     }
+    return v;
   };
-  auto since8 = [&](int block0, int t, int p, float* v) {  // decay from the start of block `block0` through token t, eight channels
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = sG[CH ? t * KF + p * 8 + e : t];
-    add_totals8(block0, t >> 4, p, v);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = expf(v[e]);
-  };
-  auto until8 = [&](int t, int block1, int p, float* v) {  // decay behind token t through the end of block `block1` - 1
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = total[CH ? (t >> 4) * K + p * 8 + e : t >> 4] - sG[CH ? t * KF + p * 8 + e : t];
-    add_totals8((t >> 4) + 1, block1, p, v);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = expf(v[e]);
-  };
-  auto between = [&](int s, int t) {  // decay behind token s through token t >= s (one decay per head)
-    if (s >> 4 == t >> 4) return expf(sG[t] - sG[s]);
-    float v = sG[t] + (total[s >> 4] - sG[s]);
-    for (int i = (s >> 4) + 1; i < t >> 4; ++i) v += total[i];
-    return expf(v);
-  };
-  // ---- rows and columns of L and P as halves
-  // with a decay per channel, rows 0-31 of the staging area: tokens 32-63 and 0-31 around token 31; rows 32-47: 16-31 and 0-15
-  // around 15; rows 48-63: 48-63 and 32-47 around 47
-  for (int i = tid; i < DC * K8; i += DP_THREADS) {
-    const int r = i / K8, p = i % K8;
-    const uint32_t o = r * RB + p * 16;
-    const int row = CH ? (r < 32 ? 32 + r : (r < 48 ? r - 16 : r)) : r, col = r < 32 ? r : (r < 48 ? r - 32 : r - 16);
-    float kv[8], qv[8];
-    delta_load8(sK + row * KF + p * 8, kv);
-    delta_load8(sQ + row * KF + p * 8, qv);
+  auto until2 = [&](int t, int block1, int d) {
+    float2 v, w;
+    const int blk = t >> 4;
     if (CH) {
-      const int ref = r < 32 ? 2 : (r < 48 ? 1 : 3);  // the block that starts behind token 31, 15, 47
-      float f[8];
-      since8(ref, row, p, f);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        kv[e] *= f[e];
-        qv[e] *= f[e];
-      }
-      delta_split8(kv, stage + o, stage + half + o);
-      delta_split8(qv, stage + sm.rows_q + o, stage + sm.rows_q + half + o);
-      delta_load8(sK + col * KF + p * 8, kv);
-      until8(col, ref, p, f);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) kv[e] *= f[e];
-      delta_split8(kv, stage + sm.cols + o, stage + sm.cols + half + o);
+      v = *reinterpret_cast<const float2*>(total + blk * K + d);
+      w = *reinterpret_cast<const float2*>(sG + t * KF + d);
     } else {
-      delta_split8(kv, stage + o, stage + half + o);
-      delta_split8(qv, stage + sm.rows_q + o, stage + sm.rows_q + half + o);
+      v.x = v.y = total[blk];
+      w.x = w.y = sG[t];
     }
-  }
+    v.x -= w.x;
+    v.y -= w.y;
+    for (int i = blk + 1; i < block1; ++i) {
+      v.x += total[CH ? i * K + d : i];
+      v.y += total[CH ? i * K + d + 1 : i];
+    }
+    return v;
+  };
   __nv_bfloat16 *p_hi = reinterpret_cast<__nv_bfloat16*>(block + pl.p), *p_lo = p_hi + DC * DC;
-  __syncthreads();
-  {
-    const uint32_t st = smem_u32(stage);
-    const int tasks = CH ? 12 : 20;
-    for (int u = warp; u < tasks; u += DP_THREADS / 32) {
-      const bool is_q = u >= tasks / 2;
-      const int v = is_q ? u - tasks / 2 : u;
-      int mt, np, rr, cr;  // 16-token blocks of the rows and columns, and where they stand
-      if (CH) {
-        mt = v < 4 ? 2 + (v >> 1) : (v == 4 ? 1 : 3);
-        np = v < 4 ? (v & 1) : (v == 4 ? 0 : 2);
-        rr = v < 4 ? (v >> 1) * 16 : (v == 4 ? 32 : 48);
-        cr = v < 4 ? (v & 1) * 16 : (v == 4 ? 32 : 48);
-      } else {
-        mt = v < 1 ? 0 : (v < 3 ? 1 : (v < 6 ? 2 : 3));
-        np = v - mt * (mt + 1) / 2;
-        rr = mt * 16;
-        cr = np * 16;
+  if (warp < 10) {
+    // ---- L and P, blocks of 16 x 16, operands from the float32 rows
+    const int mt = warp < 1 ? 0 : (warp < 3 ? 1 : (warp < 6 ? 2 : 3)), np = warp - mt * (mt + 1) / 2;
+    const bool diag = mt == np;
+    if (!(CH && diag && wild[mt])) {
+      float accK[2][4], accQ[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) accK[i][0] = accK[i][1] = accK[i][2] = accK[i][3] = accQ[i][0] = accQ[i][1] = accQ[i][2] = accQ[i][3] = 0.f;
+#pragma unroll 2
+      for (int ks = 0; ks < KT; ++ks) {
+        uint32_t kh[4], kl[4], qh[4], ql[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {  // (row g + 8 (j & 1), values 2 t4 + 8 (j >> 1))
+          const int t = mt * 16 + g + 8 * (j & 1), d = ks * 16 + 2 * t4 + 8 * (j >> 1);
+          float2 kv = *reinterpret_cast<const float2*>(sK + t * KF + d), qv = *reinterpret_cast<const float2*>(sQ + t * KF + d);
+          if (CH) {
+            const float2 l = *reinterpret_cast<const float2*>(sG + t * KF + d);
+            const float fx = exp2f(l.x), fy = exp2f(l.y);
+            kv = make_float2(kv.x * fx, kv.y * fy);
+            qv = make_float2(qv.x * fx, qv.y * fy);
+          }
+          split_bf16x2(kv.x, kv.y, kh[j], kl[j]);
+          split_bf16x2(qv.x, qv.y, qh[j], ql[j]);
+        }
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          uint32_t bh[2], bl[2];
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {  // (column g of tile i, values 2 t4 + 8 j)
+            const int s = np * 16 + 8 * i + g, d = ks * 16 + 2 * t4 + 8 * j;
+            float2 kv = *reinterpret_cast<const float2*>(sK + s * KF + d);
+            if (CH) {
+              float2 l;
+              if (diag) {
+                l = *reinterpret_cast<const float2*>(sG + s * KF + d);
+                l = make_float2(-l.x, -l.y);
+              } else {
+                l = until2(s, mt, d);
+              }
+              kv = make_float2(kv.x * exp2f(l.x), kv.y * exp2f(l.y));
+            }
+            split_bf16x2(kv.x, kv.y, bh[j], bl[j]);
+          }
+          mma_bf16_16816(accK[i], kh, bh[0], bh[1]);
+          mma_bf16_16816(accQ[i], qh, bh[0], bh[1]);
+          mma_bf16_16816(accK[i], kh, bl[0], bl[1]);
+          mma_bf16_16816(accQ[i], qh, bl[0], bl[1]);
+          mma_bf16_16816(accK[i], kl, bh[0], bh[1]);
+          mma_bf16_16816(accQ[i], ql, bh[0], bh[1]);
+        }
       }
-      const uint32_t rows = st + (is_q ? sm.rows_q : 0) + rr * RB, cols = st + (CH ? sm.cols : 0) + cr * RB;
-      float acc[2][4];
-      delta_tile<KT>(rows, rows + half, cols, cols + half, RB, lane, acc);
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int e = 0; e < 4; e += 2) {
           const int t = mt * 16 + g + 8 * (e >> 1), s = np * 16 + 8 * i + 2 * t4;
-          float v0 = acc[i][e], v1 = acc[i][e + 1];
+          float f0 = 1.f, f1 = 1.f;
           if (!CH) {
-            v0 = s <= t ? v0 * between(s, t) : 0.f;
-            v1 = s + 1 <= t ? v1 * between(s + 1, t) : 0.f;
+            if (diag) {
+              f0 = exp2f(fminf(sG[t] - sG[s], 0.f));  // (positive only where the triangle is cut off)
+              f1 = exp2f(fminf(sG[t] - sG[s + 1], 0.f));
+            } else {
+              f0 = exp2f(sG[t] + until2(s, mt, 0).x);
+              f1 = exp2f(sG[t] + until2(s + 1, mt, 0).x);
+            }
           }
-          if (is_q) {
-            uint32_t hi, lo;
-            split_bf16x2(v0, v1, hi, lo);
-            *reinterpret_cast<uint32_t*>(p_hi + t * DC + s) = hi;
-            *reinterpret_cast<uint32_t*>(p_lo + t * DC + s) = lo;
-          } else {
-            sL[t * DC_LD + s] = v0 * beta[t];
-            sL[t * DC_LD + s + 1] = v1 * beta[t];
-          }
+          const bool on0 = !diag || s <= t, on1 = !diag || s + 1 <= t;
+          uint32_t hi, lo;
+          split_bf16x2(on0 ? accQ[i][e] * f0 : 0.f, on1 ? accQ[i][e + 1] * f1 : 0.f, hi, lo);
+          *reinterpret_cast<uint32_t*>(p_hi + t * DC + s) = hi;
+          *reinterpret_cast<uint32_t*>(p_lo + t * DC + s) = lo;
+          *reinterpret_cast<float2*>(sL + t * DC_LD + s) = make_float2(on0 ? accK[i][e] * f0 * beta[t] : 0.f, on1 ? accK[i][e + 1] * f1 * beta[t] : 0.f);
         }
     }
+  } else {
+    // ---- meanwhile: exp(G) k for this kernel, exp(G) q and exp(G_end - G) k for the others
+    for (int i = tid - 320; i < DC * K8; i += DP_THREADS - 320) {
+      const int t = i / K8, p = i % K8;
+      float kv[8], qv[8], f[8], r[8], y[8];
+      delta_load8(sK + t * KF + p * 8, kv);
+      delta_load8(sQ + t * KF + p * 8, qv);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        const float2 u = since2(t, p * 8 + e), w = until2(t, DC / 16, p * 8 + e);
+        f[e] = exp2f(u.x), f[e + 1] = exp2f(u.y), r[e] = exp2f(w.x), r[e + 1] = exp2f(w.y);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = kv[e] * f[e];
+      uint8_t* at = dp_smem + sm.kt + t * RB + p * 16;
+      delta_split8(y, at, at + HALF);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = qv[e] * f[e];
+      at = block + pl.qt + (t * K + p * 8) * 2;
+      delta_split8(y, at, at + DC * K * 2);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) y[e] = kv[e] * r[e];
+      at = block + pl.kb + (t * K + p * 8) * 2;
+      delta_split8(y, at, at + DC * K * 2);
+    }
+    for (int d = tid - 320; d < K; d += DP_THREADS - 320) {
+      float s = 0.f;
+      for (int i = 0; i < DC / 16; ++i) s += total[CH ? i * K + d : i];
+      reinterpret_cast<float*>(block + pl.gend)[d] = exp2f(s);
+    }
   }
-  if (CH) {  // blocks of 16 on the diagonal: a warp has four columns of one block, a lane CPL channels
+  if (CH && wild[warp >> 2]) {  // a block on the diagonal column by column: a warp has four columns, a lane CPL channels
     const int t0 = (warp >> 2) * 16, s0 = t0 + (warp & 3) * 4;
     float w[4][CPL];
 #pragma unroll
@@ -395,7 +434,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
         for (int i = 0; i < CPL; ++i) {
           const int d = lane + 32 * i;
           const float kt = sK[t * KF + d], qt = sQ[t * KF + d];
-          const float f = t > s0 ? expf(sG[t * KF + d] - sG[(t - 1) * KF + d]) : 0.f;
+          const float f = t > s0 ? exp2f(sG[t * KF + d] - sG[(t - 1) * KF + d]) : 0.f;
 #pragma unroll
           for (int s = 0; s < 4; ++s) {
             w[s][i] = t == s0 + s ? kt : w[s][i] * f;  // (zero ahead of its own token)
@@ -431,192 +470,188 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
   }
   __syncthreads();
   // ---- the inverse of I + L: blocks of 16 on the diagonal by substitution, the others from them
-  float* sT = reinterpret_cast<float*>(stage + sm.t);
-  if (tid < DC) {
+  if (warp < 2) {
     const int t0 = tid & ~15, c = tid & 15;
     float v[16];
 #pragma unroll
     for (int r = 0; r < 16; ++r) {
-      float s = 0.f;
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int i = 0; i < 16; ++i)
-        if (i < r) s = fmaf(sL[(t0 + r) * DC_LD + t0 + i], v[i], s);
-      v[r] = r < c ? 0.f : (r == c ? 1.f : -s);
+        if (i < r) s[i & 3] = fmaf(sL[(t0 + r) * DC_LD + t0 + i], v[i], s[i & 3]);
+      v[r] = r < c ? 0.f : (r == c ? 1.f : -((s[0] + s[1]) + (s[2] + s[3])));
       sT[(t0 + r) * DC_LD + t0 + c] = v[r];
     }
-  } else if (tid >= 128) {  // (meanwhile) v into its halves, and exp(G) k
-    for (int i = tid - 128; i < V8 * 8; i += DP_THREADS - 128) {
-      const int c = i % V8, j0 = i / V8 * 8;
-      delta_conv8(a, z, ring, C, pos0, c0 + j0, n_all, 2 * a.G * K + h * V + c * 8, [&](int t, const float* y) {
-        uint8_t* at = stage + sm.v + (j0 + t) * RV + c * 16;
-        delta_split8(y, at, at + DC * RV);
+  } else {  // (meanwhile) v: convolution and silu, as halves where the decays were
+    const int d = lane * 4, dc = min(d, V - 4);
+    for (int r = warp - 2; r < DC / 4; r += DP_WARPS - 2)
+      delta_conv4(a, raw_v + dc, V, z, ring, C, pos0, c0, r * 4, n, 2 * a.G * K + h * V + dc, [&](int t, const float* y) {
+        if (d >= V) return;
+        uint32_t h0, l0, h1, l1;
+        split_bf16x2(y[0], y[1], h0, l0);
+        split_bf16x2(y[2], y[3], h1, l1);
+        uint8_t* at = dp_smem + sm.g + t * RV + d * 2;
+        *reinterpret_cast<uint2*>(at) = make_uint2(h0, h1);
+        *reinterpret_cast<uint2*>(at + VHALF) = make_uint2(l0, l1);
       });
-    }
-    for (int i = tid - 128; i < DC * K8; i += DP_THREADS - 128) {
-      const int t = i / K8, p = i % K8;
-      float kv[8], f[8];
-      delta_load8(sK + t * KF + p * 8, kv);
-      since8(0, t, p, f);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) kv[e] *= f[e];
-      uint8_t* at = stage + sm.kt + t * RB + p * 16;
-      delta_split8(kv, at, at + half);
-    }
   }
   __syncthreads();
+#pragma unroll
   for (int dist = 1; dist < 4; ++dist) {
     // block (i, i - dist): first sum_k L_ik T_kj into the (unused) mirror block above the diagonal, then - T_ii times that
     for (int u = tid; u < (4 - dist) * 256; u += DP_THREADS) {
       const int j = u >> 8, i = j + dist, r = u >> 4 & 15, c = u & 15;
-      float s = 0.f;
-      for (int m = j * 16; m < i * 16; ++m) s = fmaf(sL[(i * 16 + r) * DC_LD + m], sT[m * DC_LD + j * 16 + c], s);
-      sL[(j * 16 + r) * DC_LD + i * 16 + c] = s;
+      const float *lr = sL + (i * 16 + r) * DC_LD + j * 16, *tc = sT + j * 16 * DC_LD + j * 16 + c;
+      float s[2] = {0.f, 0.f};
+#pragma unroll
+      for (int m = 0; m < 16 * dist; m += 4) {
+        const float4 y = *reinterpret_cast<const float4*>(lr + m);
+        s[0] = fmaf(y.x, tc[m * DC_LD], s[0]);
+        s[1] = fmaf(y.y, tc[(m + 1) * DC_LD], s[1]);
+        s[0] = fmaf(y.z, tc[(m + 2) * DC_LD], s[0]);
+        s[1] = fmaf(y.w, tc[(m + 3) * DC_LD], s[1]);
+      }
+      sL[(j * 16 + r) * DC_LD + i * 16 + c] = s[0] + s[1];
     }
     __syncthreads();
     for (int u = tid; u < (4 - dist) * 256; u += DP_THREADS) {
       const int j = u >> 8, i = j + dist, r = u >> 4 & 15, c = u & 15;
-      float s = 0.f;
+      const float *tr = sT + (i * 16 + r) * DC_LD + i * 16, *mc = sL + j * 16 * DC_LD + i * 16 + c;
+      float s[2] = {0.f, 0.f};
 #pragma unroll
-      for (int m = 0; m < 16; ++m) s = fmaf(sT[(i * 16 + r) * DC_LD + i * 16 + m], sL[(j * 16 + m) * DC_LD + i * 16 + c], s);
-      sT[(i * 16 + r) * DC_LD + j * 16 + c] = -s;
+      for (int m = 0; m < 16; m += 4) {
+        const float4 y = *reinterpret_cast<const float4*>(tr + m);
+        s[0] = fmaf(y.x, mc[m * DC_LD], s[0]);
+        s[1] = fmaf(y.y, mc[(m + 1) * DC_LD], s[1]);
+        s[0] = fmaf(y.z, mc[(m + 2) * DC_LD], s[0]);
+        s[1] = fmaf(y.w, mc[(m + 3) * DC_LD], s[1]);
+      }
+      sT[(i * 16 + r) * DC_LD + j * 16 + c] = -(s[0] + s[1]);
     }
     __syncthreads();
   }
-  for (int i = tid; i < DC * DC / 8; i += DP_THREADS) {  // times beta, as halves
-    const int t = i / 8, p = i % 8;
-    if (p * 8 > (t | 15)) continue;
-    float v[8];
-    delta_load8(sT + t * DC_LD + p * 8, v);
+  {  // times beta, as halves: 64 rows of eight pieces
+    const int t = tid >> 3, p = tid & 7;
+    if (p * 8 <= (t | 15)) {
+      float v[8];
+      delta_load8(sT + t * DC_LD + p * 8, v);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] *= beta[p * 8 + e];
-    uint8_t* at = stage + sm.tp + t * DC_PROW + p * 16;
-    delta_split8(v, at, at + DC * DC_PROW);
-  }
-  // ---- exp(G) q and exp(G_end - G) k for the other kernels
-  for (int i = tid; i < DC * K8; i += DP_THREADS) {
-    const int t = i / K8, p = i % K8;
-    float v[8], f[8];
-    since8(0, t, p, f);
-    delta_load8(sQ + t * KF + p * 8, v);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] *= f[e];
-    uint8_t* at = block + pl.qt + (t * K + p * 8) * 2;
-    delta_split8(v, at, at + DC * K * 2);
-    delta_load8(sK + t * KF + p * 8, v);
-    until8(t, DC / 16, p, f);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] *= f[e];
-    at = block + pl.kb + (t * K + p * 8) * 2;
-    delta_split8(v, at, at + DC * K * 2);
-  }
-  if (tid < K) {
-    float s = 0.f;
-    for (int i = 0; i < DC / 16; ++i) s += total[CH ? i * K + tid : i];
-    reinterpret_cast<float*>(block + pl.gend)[tid] = expf(s);
+      for (int e = 0; e < 8; ++e) v[e] *= beta[p * 8 + e];
+      uint8_t* at = dp_smem + sm.tp + t * DC_PROW + p * 16;
+      delta_split8(v, at, at + DC * DC_PROW);
+    }
   }
   __syncthreads();
-  // ---- W = T exp(G) k and U0 = T v (T: the inverse times beta), 16 x 16 tiles
+  // ---- W = T exp(G) k and U0 = T v (T: the inverse times beta), all 64 tokens of 16 columns per warp
   {
     const int mi = lane >> 3, r8 = lane & 7, nk = K / 16, nv = V / 16;
-    const uint32_t tp = smem_u32(stage + sm.tp), kt = smem_u32(stage + sm.kt), vt = smem_u32(stage + sm.v);
-    for (int u = warp; u < 4 * (nk + nv); u += DP_THREADS / 32) {
-      const int mt = 3 - (u & 3), nt = u >> 2;
-      const bool is_w = nt < nk;
-      const int rb = is_w ? RB : RV, col = is_w ? nt : nt - nk;
-      const uint32_t A = tp + (mt * 16 + (mi & 1) * 8 + r8) * DC_PROW + (mi >> 1) * 16;
-      const uint32_t Bm = (is_w ? kt : vt) + ((mi & 1) * 8 + r8) * rb + (mi >> 1) * 16 + col * 32;
-      float acc[2][4];
+    const uint32_t A = smem_u32(dp_smem + sm.tp) + ((mi & 1) * 8 + r8) * DC_PROW + (mi >> 1) * 16;
+    for (int u = warp; u < nk + nv; u += DP_WARPS) {
+      const bool is_w = u < nk;
+      const int rb = is_w ? RB : RV, col = is_w ? u : u - nk;
+      const uint32_t Bm = smem_u32(dp_smem + (is_w ? sm.kt : sm.g)) + ((mi & 1) * 8 + r8) * rb + (mi >> 1) * 16 + col * 32;
+      float acc[4][2][4];
 #pragma unroll
-      for (int i = 0; i < 2; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-      for (int ks = 0; ks <= mt; ++ks) {
-        uint32_t ah[4], al[4], bh[4], bl[4];
-        ldmatrix_x4(A + ks * 32, ah[0], ah[1], ah[2], ah[3]);
-        ldmatrix_x4(A + DC * DC_PROW + ks * 32, al[0], al[1], al[2], al[3]);
+      for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) acc[mt][i][0] = acc[mt][i][1] = acc[mt][i][2] = acc[mt][i][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        uint32_t bh[4], bl[4];
         ldmatrix_x4_trans(Bm + ks * 16 * rb, bh[0], bh[1], bh[2], bh[3]);
         ldmatrix_x4_trans(Bm + DC * rb + ks * 16 * rb, bl[0], bl[1], bl[2], bl[3]);
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          mma_bf16_16816(acc[i], ah, bh[2 * i], bh[2 * i + 1]);
-          mma_bf16_16816(acc[i], ah, bl[2 * i], bl[2 * i + 1]);
-          mma_bf16_16816(acc[i], al, bh[2 * i], bh[2 * i + 1]);
+        for (int mt = ks; mt < 4; ++mt) {
+          uint32_t ah[4], al[4];
+          ldmatrix_x4(A + mt * 16 * DC_PROW + ks * 32, ah[0], ah[1], ah[2], ah[3]);
+          ldmatrix_x4(A + (DC + mt * 16) * DC_PROW + ks * 32, al[0], al[1], al[2], al[3]);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            mma_bf16_16816(acc[mt][i], ah, bh[2 * i], bh[2 * i + 1]);
+            mma_bf16_16816(acc[mt][i], ah, bl[2 * i], bl[2 * i + 1]);
+            mma_bf16_16816(acc[mt][i], al, bh[2 * i], bh[2 * i + 1]);
+          }
         }
       }
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
+      for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-        for (int e = 0; e < 4; e += 2) {
-          const int t = mt * 16 + g + 8 * (e >> 1), c = col * 16 + 8 * i + 2 * t4;
-          if (is_w) {
-            uint32_t hi, lo;
-            split_bf16x2(acc[i][e], acc[i][e + 1], hi, lo);
-            uint8_t* at = block + pl.w + (t * K + c) * 2;
-            *reinterpret_cast<uint32_t*>(at) = hi;
-            *reinterpret_cast<uint32_t*>(at + DC * K * 2) = lo;
-          } else {
-            *reinterpret_cast<float2*>(block + pl.u0 + (t * V + c) * 4) = make_float2(acc[i][e], acc[i][e + 1]);
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            const int t = mt * 16 + g + 8 * (e >> 1), c = col * 16 + 8 * i + 2 * t4;
+            if (is_w) {
+              uint32_t hi, lo;
+              split_bf16x2(acc[mt][i][e], acc[mt][i][e + 1], hi, lo);
+              uint8_t* at = block + pl.w + (t * K + c) * 2;
+              *reinterpret_cast<uint32_t*>(at) = hi;
+              *reinterpret_cast<uint32_t*>(at + DC * K * 2) = lo;
+            } else {
+              *reinterpret_cast<float2*>(block + pl.u0 + (t * V + c) * 4) = make_float2(acc[mt][i][e], acc[mt][i][e + 1]);
+            }
           }
-        }
     }
   }
 }
 
 // ----------------------------------------------------------------------------- the state, chunk after chunk
-constexpr int DS_THREADS = 256;
+constexpr int DS_THREADS = 512;
+__host__ __device__ inline int delta_state_stage(int K, int NV) { return 4 * DC * (K * 2 + 16) + DC * (NV * 4 + 16) + K * 4; }
 __host__ __device__ inline int delta_state_smem(int K, int NV) {
-  return 2 * 4 * DC * (K * 2 + 16) + 2 * K * (NV * 2 + 16) + 2 * DC * (NV * 2 + 16);
+  return 2 * delta_state_stage(K, NV) + 2 * K * (NV * 2 + 16) + 2 * DC * (NV * 2 + 16);
 }
 
-// grid (V / NV, H, B): a CTA has NV values of one head's state, warp w its rows 16 w .. 16 w + 15 in accumulator registers.
+// grid (V / NV, H, B): a CTA has NV values of one head's state; warp w has rows 16 (w % KT) .. and values 16 (w / KT) .. of it in
+// accumulator registers, and a tile of U of 16 tokens x 8 values.
 template <int KT, int NV>
 __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaChunkArgs x) {
-  constexpr int K = KT * 16, RB = K * 2 + 16, RN = NV * 2 + 16, NT = NV / 8, K8 = K / 8;
-  constexpr int UT = NV / 16;  // tiles of 8 values that a warp has of U: 16 tokens x NV / 2 values
+  constexpr int K = KT * 16, RB = K * 2 + 16, RN = NV * 2 + 16, RU = NV * 4 + 16, K8 = K / 8, NV4 = NV / 4;
   extern __shared__ __align__(16) uint8_t dt_smem[];
   pdl_launch_dependents();
   const DeltaArgs& a = x.a;
   const int v0 = blockIdx.x * NV, h = blockIdx.y, b = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3, mi = lane >> 3, r8 = lane & 7;
   const int q0 = a.query_start[b], n = a.query_start[b + 1] - q0, slot = a.slots[b];
-  if (n < a.min_rows || n > a.max_rows || n <= 0 || (unsigned)slot >= (unsigned)a.num_slots) {
-    pdl_wait();
-    return;
-  }
-  const int V = a.V, chunks = (n + DC - 1) / DC;
+  const int V = a.V, chunk1 = min((n + DC - 1) / DC, x.chunk0 + x.round);
+  pdl_wait();
+  if (n < a.min_rows || n > a.max_rows || x.chunk0 >= chunk1 || (unsigned)slot >= (unsigned)a.num_slots) return;
   const DeltaPlan pl = delta_plan(K, V);
-  uint8_t* ops = dt_smem;               // [2][W hi, lo, Kb hi, lo][64][RB]
-  uint8_t* sS = ops + 8 * DC * RB;      // [hi, lo][K][RN]
-  uint8_t* sU = sS + 2 * K * RN;        // [hi, lo][64][RN]
-  const bool rows = warp < KT;          // this warp has rows of the state
-  float S[NT][4];
-  float* st = a.state + ((size_t)slot * a.H + h) * K * V + (size_t)(warp * 16 + g) * V + v0 + 2 * t4;
-  const bool resumed = a.seq_lens[b] > n;
+  const int stage_bytes = delta_state_stage(K, NV);
+  uint8_t* sS = dt_smem + 2 * stage_bytes;  // [hi, lo][K][RN]
+  uint8_t* sU = sS + 2 * K * RN;            // [hi, lo][64][RN]
+  auto fetch = [&](int c) {                 // W hi, lo, Kb hi, lo [64][RB] | U0 [64][RU] | gend [K]
+    const uint8_t* block = delta_block(x, pl.bytes, b, c, h);
+    uint8_t* dst = dt_smem + (c & 1) * stage_bytes;
+    for (int i = tid; i < 4 * DC * K8; i += DS_THREADS) cp_async16(dst + i / K8 * RB + i % K8 * 16, block + (size_t)i * 16);
+    dst += 4 * DC * RB;
+    for (int i = tid; i < DC * NV4; i += DS_THREADS)
+      cp_async16(dst + i / NV4 * RU + i % NV4 * 16, block + pl.u0 + ((size_t)(i / NV4) * V + v0) * 4 + i % NV4 * 16);
+    for (int i = tid; i < K / 4; i += DS_THREADS) cp_async16(dst + DC * RU + i * 16, block + pl.gend + i * 16);
+    cp_async_commit();
+  };
+  fetch(x.chunk0);
+  const int srow = warp % KT, scol = warp / KT;
+  const bool owner = scol < NV / 16;  // this warp has a part of the state
+  const bool resumed = a.seq_lens[b] > n || x.chunk0 > 0;
+  float S[2][4];
+  float* st = a.state + ((size_t)slot * a.H + h) * K * V + (size_t)(srow * 16 + g) * V + v0 + scol * 16 + 2 * t4;
 #pragma unroll
-  for (int i = 0; i < NT; ++i)
+  for (int i = 0; i < 2; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; e += 2) {  // (written by an earlier step: no need to wait for this step's kernels)
-      const float2 y = (rows && resumed) ? *reinterpret_cast<const float2*>(st + (size_t)(e >> 1) * 8 * V + 8 * i) : make_float2(0.f, 0.f);
+    for (int e = 0; e < 4; e += 2) {
+      const float2 y = (owner && resumed) ? __ldcg(reinterpret_cast<const float2*>(st + (size_t)(e >> 1) * 8 * V + 8 * i)) : make_float2(0.f, 0.f);
       S[i][e] = y.x;
       S[i][e + 1] = y.y;
     }
-  pdl_wait();
-  auto fetch = [&](int c) {
-    const uint8_t* block = delta_block(x, pl.bytes, q0, b, c, h);
-    uint8_t* dst = ops + (c & 1) * 4 * DC * RB;
-    for (int i = tid; i < 4 * DC * K8; i += DS_THREADS) {  // (W and Kb lie behind each other: 256 rows of halves)
-      const int r = i / K8, p = i % K8;
-      cp_async16(dst + r * RB + p * 16, block + (size_t)i * 16);
-    }
-    cp_async_commit();
-  };
-  auto put_state = [&](uint8_t* block) {  // halves of this warp's rows: for the next products, and for the outputs
-    if (!rows) return;
+  auto put_state = [&](uint8_t* block) {  // halves: for the next products, and for the outputs
+    if (!owner) return;
 #pragma unroll
-    for (int i = 0; i < NT; ++i)
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
       for (int e = 0; e < 4; e += 2) {
         uint32_t hi, lo;
         split_bf16x2(S[i][e], S[i][e + 1], hi, lo);
-        const int k = warp * 16 + g + 8 * (e >> 1), c = 8 * i + 2 * t4;
+        const int k = srow * 16 + g + 8 * (e >> 1), c = scol * 16 + 8 * i + 2 * t4;
         *reinterpret_cast<uint32_t*>(sS + k * RN + c * 2) = hi;
         *reinterpret_cast<uint32_t*>(sS + K * RN + k * RN + c * 2) = lo;
         uint8_t* at = block + pl.s + ((size_t)k * V + v0 + c) * 2;
@@ -624,108 +659,89 @@ __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaC
         *reinterpret_cast<uint32_t*>(at + (size_t)K * V * 2) = lo;
       }
   };
-  const uint32_t ops_u = smem_u32(ops), s_u = smem_u32(sS), u_u = smem_u32(sU);
-  const int mt = warp & 3, un = (warp >> 2) * (NV / 2);  // this warp's tile of U
+  const uint32_t base = smem_u32(dt_smem), s_u = smem_u32(sS), u_u = smem_u32(sU);
+  const int mt = warp & 3, un = (warp >> 2) * 8;  // this warp's tile of U
+  const bool has_u = un < NV;
   const uint32_t wa = (mt * 16 + (mi & 1) * 8 + r8) * RB + (mi >> 1) * 16;
-  const uint32_t sb = ((mi & 1) * 8 + r8) * RN + (NV == 32 ? un * 2 + (mi >> 1) * 16 : (mi >> 1) * 16);
-  const uint32_t ka = ((mi >> 1) * 8 + r8) * RB + warp * 32 + (mi & 1) * 16;  // transposed: 16 keys x 16 tokens
-  const uint32_t ub = ((mi & 1) * 8 + r8) * RN + (mi >> 1) * 16;
-  fetch(0);
-  for (int c = 0; c < chunks; ++c) {
-    uint8_t* block = delta_block(x, pl.bytes, q0, b, c, h);
+  const uint32_t sb = lane * RN + un * 2;                                      // transposed: 32 keys x 8 values
+  const uint32_t ka = ((mi >> 1) * 8 + r8) * RB + srow * 32 + (mi & 1) * 16;   // transposed: 16 keys x 16 tokens
+  const uint32_t ub = ((mi & 1) * 8 + r8) * RN + scol * 32 + (mi >> 1) * 16;
+  for (int c = x.chunk0; c < chunk1; ++c) {
+    uint8_t* block = delta_block(x, pl.bytes, b, c, h);
     put_state(block);
-    float u0[UT][4];
-    const float* up = reinterpret_cast<const float*>(block + pl.u0) + (size_t)(mt * 16 + g) * V + v0 + un + 2 * t4;
+    cp_async_wait<0>();
+    __syncthreads();  // this chunk's operands and the state are in shared memory; the other buffer has been read
+    if (c + 1 < chunk1) fetch(c + 1);
+    const uint32_t W = base + (c & 1) * stage_bytes, Kb = W + 2 * DC * RB;
+    const uint8_t* extra = dt_smem + (c & 1) * stage_bytes + 4 * DC * RB;
+    if (has_u) {
+      float acc[3][4];
 #pragma unroll
-    for (int i = 0; i < UT; ++i)
+      for (int j = 0; j < 3; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < KT; ks += 2) {
+        uint32_t bh[4], bl[4];
+        ldmatrix_x4_trans(s_u + sb + ks * 16 * RN, bh[0], bh[1], bh[2], bh[3]);
+        ldmatrix_x4_trans(s_u + K * RN + sb + ks * 16 * RN, bl[0], bl[1], bl[2], bl[3]);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          uint32_t ah[4], al[4];
+          ldmatrix_x4(W + wa + (ks + j) * 32, ah[0], ah[1], ah[2], ah[3]);
+          ldmatrix_x4(W + DC * RB + wa + (ks + j) * 32, al[0], al[1], al[2], al[3]);
+          mma_bf16_16816(acc[0], ah, bh[2 * j], bh[2 * j + 1]);
+          mma_bf16_16816(acc[1], ah, bl[2 * j], bl[2 * j + 1]);
+          mma_bf16_16816(acc[2], al, bh[2 * j], bh[2 * j + 1]);
+        }
+      }
 #pragma unroll
       for (int e = 0; e < 4; e += 2) {
-        const float2 y = *reinterpret_cast<const float2*>(up + (size_t)(e >> 1) * 8 * V + 8 * i);
-        u0[i][e] = y.x;
-        u0[i][e + 1] = y.y;
-      }
-    float ge[2] = {0.f, 0.f};
-    if (rows) {
-      const float* gp = reinterpret_cast<const float*>(block + pl.gend) + warp * 16 + g;
-      ge[0] = gp[0];
-      ge[1] = gp[8];
-    }
-    if (c + 1 < chunks) {
-      fetch(c + 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();  // this chunk's operands and the state are in shared memory
-    const uint32_t W = ops_u + (c & 1) * 4 * DC * RB, Kb = W + 2 * DC * RB;
-    float acc[UT][3][4];
-#pragma unroll
-    for (int i = 0; i < UT; ++i)
-#pragma unroll
-      for (int j = 0; j < 3; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
-#pragma unroll
-    for (int ks = 0; ks < KT; ++ks) {
-      uint32_t ah[4], al[4], bh[4], bl[4];
-      ldmatrix_x4(W + wa + ks * 32, ah[0], ah[1], ah[2], ah[3]);
-      ldmatrix_x4(W + DC * RB + wa + ks * 32, al[0], al[1], al[2], al[3]);
-      ldmatrix_x4_trans(s_u + sb + ks * 16 * RN, bh[0], bh[1], bh[2], bh[3]);
-      ldmatrix_x4_trans(s_u + K * RN + sb + ks * 16 * RN, bl[0], bl[1], bl[2], bl[3]);
-#pragma unroll
-      for (int i = 0; i < UT; ++i) {
-        const bool second = NV == 32 ? i == 1 : un > 0;
-        const uint32_t b0 = second ? bh[2] : bh[0], b1 = second ? bh[3] : bh[1], l0 = second ? bl[2] : bl[0], l1 = second ? bl[3] : bl[1];
-        mma_bf16_16816(acc[i][0], ah, b0, b1);
-        mma_bf16_16816(acc[i][1], ah, l0, l1);
-        mma_bf16_16816(acc[i][2], al, b0, b1);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < UT; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; e += 2) {
+        const int t = mt * 16 + g + 8 * (e >> 1), cc = un + 2 * t4;
+        const float2 u0 = *reinterpret_cast<const float2*>(extra + t * RU + cc * 4);
         uint32_t hi, lo;
-        split_bf16x2(u0[i][e] - (acc[i][0][e] + (acc[i][1][e] + acc[i][2][e])),
-                     u0[i][e + 1] - (acc[i][0][e + 1] + (acc[i][1][e + 1] + acc[i][2][e + 1])), hi, lo);
-        const int t = mt * 16 + g + 8 * (e >> 1), cc = un + 8 * i + 2 * t4;
+        split_bf16x2(u0.x - (acc[0][e] + (acc[1][e] + acc[2][e])), u0.y - (acc[0][e + 1] + (acc[1][e + 1] + acc[2][e + 1])), hi, lo);
         *reinterpret_cast<uint32_t*>(sU + t * RN + cc * 2) = hi;
         *reinterpret_cast<uint32_t*>(sU + DC * RN + t * RN + cc * 2) = lo;
         uint8_t* at = block + pl.u + ((size_t)t * V + v0 + cc) * 2;
         *reinterpret_cast<uint32_t*>(at) = hi;
         *reinterpret_cast<uint32_t*>(at + (size_t)DC * V * 2) = lo;
       }
+    }
     __syncthreads();  // U is complete; the state's halves have been read
-    if (rows) {
+    if (owner) {
+      const float* ge = reinterpret_cast<const float*>(extra + DC * RU) + srow * 16 + g;
+      float acc[2][2][4];  // (the low halves' products in accumulators of their own)
 #pragma unroll
-      for (int i = 0; i < NT; ++i) {
+      for (int i = 0; i < 2; ++i) {
         S[i][0] *= ge[0];
         S[i][1] *= ge[0];
-        S[i][2] *= ge[1];
-        S[i][3] *= ge[1];
+        S[i][2] *= ge[8];
+        S[i][3] *= ge[8];
+#pragma unroll
+        for (int j = 0; j < 2; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
       }
 #pragma unroll
       for (int ks = 0; ks < DC / 16; ++ks) {
-        uint32_t ah[4], al[4];
+        uint32_t ah[4], al[4], bh[4], bl[4];
         ldmatrix_x4_trans(Kb + ka + ks * 16 * RB, ah[0], ah[1], ah[2], ah[3]);
         ldmatrix_x4_trans(Kb + DC * RB + ka + ks * 16 * RB, al[0], al[1], al[2], al[3]);
+        ldmatrix_x4_trans(u_u + ub + ks * 16 * RN, bh[0], bh[1], bh[2], bh[3]);
+        ldmatrix_x4_trans(u_u + DC * RN + ub + ks * 16 * RN, bl[0], bl[1], bl[2], bl[3]);
 #pragma unroll
-        for (int i = 0; i < NT; i += 2) {
-          uint32_t bh[4], bl[4];
-          ldmatrix_x4_trans(u_u + ub + ks * 16 * RN + i * 16, bh[0], bh[1], bh[2], bh[3]);
-          ldmatrix_x4_trans(u_u + DC * RN + ub + ks * 16 * RN + i * 16, bl[0], bl[1], bl[2], bl[3]);
-#pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            mma_bf16_16816(S[i + j], ah, bh[2 * j], bh[2 * j + 1]);
-            mma_bf16_16816(S[i + j], ah, bl[2 * j], bl[2 * j + 1]);
-            mma_bf16_16816(S[i + j], al, bh[2 * j], bh[2 * j + 1]);
-          }
+        for (int i = 0; i < 2; ++i) {
+          mma_bf16_16816(S[i], ah, bh[2 * i], bh[2 * i + 1]);
+          mma_bf16_16816(acc[i][0], ah, bl[2 * i], bl[2 * i + 1]);
+          mma_bf16_16816(acc[i][1], al, bh[2 * i], bh[2 * i + 1]);
         }
       }
-    }
-    __syncthreads();  // this chunk's operands have been read: their buffer takes the chunk after next
-  }
-  if (rows) {
 #pragma unroll
-    for (int i = 0; i < NT; ++i)
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[i][e] += acc[i][0][e] + acc[i][1][e];
+    }
+  }
+  if (owner) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
 #pragma unroll
       for (int e = 0; e < 4; e += 2) *reinterpret_cast<float2*>(st + (size_t)(e >> 1) * 8 * V + 8 * i) = make_float2(S[i][e], S[i][e + 1]);
   }
@@ -737,14 +753,14 @@ __host__ __device__ inline int delta_output_smem(int K, int V) {
   return 2 * DC * (K * 2 + 16) + 2 * K * (V * 2 + 16) + 2 * DC * DC_PROW + 2 * DC * (V * 2 + 16) + 4 * DC * 4;
 }
 
-// grid (chunks of the longest portion, H, B); warp w: tokens 16 (w % 4) .., values 32 (w / 4) ..
+// grid (chunks of the round, H, B); warp w: tokens 16 (w % 4) .., values 32 (w / 4) ..
 template <int KT>
 __global__ void __launch_bounds__(DO_THREADS, 1) delta_output_kernel(const DeltaChunkArgs x) {
   constexpr int K = KT * 16, RB = K * 2 + 16, K8 = K / 8;
   extern __shared__ __align__(16) uint8_t do_smem[];
   pdl_launch_dependents();
   const DeltaArgs& a = x.a;
-  const int b = blockIdx.z, h = blockIdx.y, chunk = blockIdx.x, c0 = chunk * DC;
+  const int b = blockIdx.z, h = blockIdx.y, chunk = x.chunk0 + blockIdx.x, c0 = chunk * DC;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3, mi = lane >> 3, r8 = lane & 7;
   const int q0 = a.query_start[b], n_all = a.query_start[b + 1] - q0, slot = a.slots[b];
   const int V = a.V, V8 = V / 8, RV = V * 2 + 16;
@@ -758,7 +774,7 @@ __global__ void __launch_bounds__(DO_THREADS, 1) delta_output_kernel(const Delta
     return;
   }
   const DeltaPlan pl = delta_plan(K, V);
-  const uint8_t* block = delta_block(x, pl.bytes, q0, b, chunk, h);
+  const uint8_t* block = delta_block(x, pl.bytes, b, chunk, h);
   uint8_t* sq = do_smem;                   // [hi, lo][64][RB]
   uint8_t* ss = sq + 2 * DC * RB;          // [hi, lo][K][RV]
   uint8_t* sp = ss + 2 * K * RV;           // [hi, lo][64][DC_PROW]
@@ -778,18 +794,8 @@ __global__ void __launch_bounds__(DO_THREADS, 1) delta_output_kernel(const Delta
   for (int i = 0; i < 4; ++i) gate[i][0] = gate[i][1] = gate[i][2] = gate[i][3] = 0.f;
   const int ta = min(mt * 16 + g, n - 1), tb = min(mt * 16 + g + 8, n - 1);
   if (a.gate_up != nullptr) {
-    const __nv_bfloat16 *r0 = z + (size_t)ta * a.ld + a.gate_off + 4 * t4, *r1 = z + (size_t)tb * a.ld + a.gate_off + 4 * t4;
     const __nv_bfloat16* up = reinterpret_cast<const __nv_bfloat16*>(a.gate_up) + (size_t)(h * V + vn + g) * a.gate_rank + 4 * t4;
-    for (int ks = 0; ks < a.gate_rank; ks += 16) {
-      const uint2 x0 = *reinterpret_cast<const uint2*>(r0 + ks), x1 = *reinterpret_cast<const uint2*>(r1 + ks);
-      const uint32_t av[4] = {x0.x, x1.x, x0.y, x1.y};
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        if (i >= nt) continue;  // (the same for the whole warp)
-        const uint2 w = *reinterpret_cast<const uint2*>(up + (size_t)i * 8 * a.gate_rank + ks);
-        mma_bf16_16816(gate[i], av, w.x, w.y);
-      }
-    }
+    if (nt > 0) delta_low_rank<4>(z + (size_t)ta * a.ld + a.gate_off + 4 * t4, z + (size_t)tb * a.ld + a.gate_off + 4 * t4, up, a.gate_rank, nt, gate);
   } else {
 #pragma unroll
     for (int i = 0; i < 4; ++i)
@@ -803,7 +809,7 @@ __global__ void __launch_bounds__(DO_THREADS, 1) delta_output_kernel(const Delta
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) gate[i][e] = (a.gate_up != nullptr ? 1.f : gate[i][e]) / (1.f + expf(-gate[i][e]));
+    for (int e = 0; e < 4; ++e) gate[i][e] = (a.gate_up != nullptr ? 1.f : gate[i][e]) * delta_sigmoid_fast(gate[i][e]);
   float O[4][4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) O[i][0] = O[i][1] = O[i][2] = O[i][3] = 0.f;

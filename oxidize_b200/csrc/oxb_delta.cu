@@ -28,7 +28,7 @@ static int delta_step_launch(const DeltaArgs& a, int B, cudaStream_t stream) {
 }
 
 template <int KT, bool CH>
-static int delta_chunk_go(const DeltaChunkArgs& x, int B, int longest, int nv, cudaStream_t stream) {
+static int delta_chunk_go(DeltaChunkArgs x, int B, int longest, int nv, cudaStream_t stream) {
   constexpr int K = KT * 16;
   const int V = x.a.V, chunks = (longest + DC - 1) / DC;
   const int most[4] = {delta_prep_smem(K, 128).total, delta_state_smem(K, 32), delta_state_smem(K, 16), delta_output_smem(K, 128)};
@@ -45,17 +45,17 @@ static int delta_chunk_go(const DeltaChunkArgs& x, int B, int longest, int nv, c
     if (e != cudaSuccess) return (int)e;
     configured[dev] = true;
   }
-  cudaError_t e = oxb_launch(delta_prepare_kernel<KT, CH>, dim3(chunks, x.a.H, B), dim3(DP_THREADS), (size_t)delta_prep_smem(K, V).total,
-                             stream, x);
-  if (e == cudaSuccess) {
-    const dim3 grid(V / nv, x.a.H, B);
-    e = nv == 32 ? oxb_launch(delta_state_kernel<KT, 32>, grid, dim3(DS_THREADS), (size_t)most[1], stream, x)
-                 : oxb_launch(delta_state_kernel<KT, 16>, grid, dim3(DS_THREADS), (size_t)most[2], stream, x);
+  for (x.chunk0 = 0; x.chunk0 < chunks; x.chunk0 += x.round) {
+    const dim3 units(chunks - x.chunk0 < x.round ? chunks - x.chunk0 : x.round, x.a.H, B), slices(V / nv, x.a.H, B);
+    cudaError_t e = oxb_launch(delta_prepare_kernel<KT, CH>, units, dim3(DP_THREADS), (size_t)delta_prep_smem(K, V).total, stream, x);
+    if (e == cudaSuccess)
+      e = nv == 32 ? oxb_launch(delta_state_kernel<KT, 32>, slices, dim3(DS_THREADS), (size_t)most[1], stream, x)
+                   : oxb_launch(delta_state_kernel<KT, 16>, slices, dim3(DS_THREADS), (size_t)most[2], stream, x);
+    if (e == cudaSuccess)
+      e = oxb_launch(delta_output_kernel<KT>, units, dim3(DO_THREADS), (size_t)delta_output_smem(K, V), stream, x);
+    if (e != cudaSuccess) return (int)e;
+    OXB_CHECK_LAUNCH();
   }
-  if (e == cudaSuccess)
-    e = oxb_launch(delta_output_kernel<KT>, dim3(chunks, x.a.H, B), dim3(DO_THREADS), (size_t)delta_output_smem(K, V), stream, x);
-  if (e != cudaSuccess) return (int)e;
-  OXB_CHECK_LAUNCH();
   return 0;
 }
 
@@ -69,14 +69,14 @@ OXB_API int oxb_delta_chunk_bytes(int K, int V) {
 // gate, decay and beta; the state [num_slots, H, K, V] float32 is read and updated, the ring of convolution inputs [num_slots,
 // taps, channels] read.  Only sequences that feed min_rows .. max_rows rows take part.  write_window (single-row steps): the
 // ring is updated too; elsewhere oxb_delta_window does that afterwards.  chunk_values 0: delta_step_kernel; else (bf16) the chunk
-// kernels with that many values of the state per CTA (16 or 32), portions of up to `longest` rows and scratch ws of
-// (T / 64 + B) * H * oxb_delta_chunk_bytes(K, V) bytes.
+// kernels with that many values of the state per CTA (16 or 32), portions of up to `longest` rows, in rounds of `round`
+// chunks with scratch ws of B * round * H * oxb_delta_chunk_bytes(K, V) bytes.
 OXB_API int oxb_delta(const void* z, int ld, int dtype, int gate_off, int decay_off, int beta_off, const int* query_start,
                       const int* seq_lens, const int* slots, const float* conv, int taps, const float* a_log, const float* dt_bias,
                       const void* decay_up, int decay_rank, const void* gate_up, int gate_rank, const float* norm, float* state,
                       float* window, int num_slots, void* out, int ld_out, float out_scale, int B, int H, int G, int K, int V,
                       int v_dim, float q_scale, float eps, int min_rows, int max_rows, int write_window, int chunk_values,
-                      int longest, void* ws, cudaStream_t stream) {
+                      int longest, int round, void* ws, cudaStream_t stream) {
   if (B <= 0 || H <= 0) return 0;
   if (G <= 0 || H % G != 0 || V % 4 != 0 || V <= 0 || K <= 0 || taps <= 0 || B > 65535 || slots == nullptr ||
       (decay_up != nullptr && (decay_rank % 8 != 0 || decay_off % 8 != 0)) || (gate_up != nullptr && (gate_rank % 8 != 0 || gate_off % 8 != 0)) ||
@@ -87,10 +87,10 @@ OXB_API int oxb_delta(const void* z, int ld, int dtype, int gate_off, int decay_
                     min_rows, max_rows, write_window};
   if (chunk_values == 0) return dtype == 0 ? delta_step_launch<float>(a, B, stream) : delta_step_launch<__nv_bfloat16>(a, B, stream);
   if (dtype != 2 || ws == nullptr || write_window || oxb_delta_chunk_bytes(K, V) == 0 || (chunk_values != 16 && chunk_values != 32) ||
-      V % chunk_values != 0 || longest <= 0 || H > 65535 || ld_out % 2 != 0 || (reinterpret_cast<uintptr_t>(out) & 3) != 0 ||
+      V % chunk_values != 0 || longest <= 0 || round <= 0 || H > 65535 || ld_out % 2 != 0 || (reinterpret_cast<uintptr_t>(out) & 3) != 0 ||
       (decay_up != nullptr && decay_rank % 16 != 0) || (gate_up != nullptr && gate_rank % 16 != 0) || gate_off % 2 != 0)
     return (int)cudaErrorInvalidValue;
-  const DeltaChunkArgs x{a, reinterpret_cast<uint8_t*>(ws)};
+  const DeltaChunkArgs x{a, reinterpret_cast<uint8_t*>(ws), 0, round};
   switch (K * 2 + (decay_up != nullptr)) {
     case 64: return delta_chunk_go<2, false>(x, B, longest, chunk_values, stream);
     case 65: return delta_chunk_go<2, true>(x, B, longest, chunk_values, stream);

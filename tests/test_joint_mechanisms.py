@@ -339,16 +339,17 @@ def test_delta_rule_batches_and_reused_slots(device, dtype):
 
 
 @gpu
-@pytest.mark.parametrize("values", [16, 32])
+@pytest.mark.parametrize("values,rounds", [(16, 1), (32, 2), (32, 100)])
 @pytest.mark.parametrize("shape", [s for s in SHAPES if s[3] <= 128 and s[2] <= 128], ids=str)
-def test_chunks_agree_with_steps(shape, values):
-    """The tensor-core kernels against the token-by-token one on the same 16-bit rows, and twice the same."""
+def test_chunks_agree_with_steps(shape, values, rounds):
+    """The tensor-core kernels, in rounds of any number of chunks, against the token-by-token one on the same 16-bit rows, and
+    twice the same."""
     spec, t = delta_case(*shape, seed=3)
     if spec.v_width % values:
         pytest.skip("not a multiple")
     z = draw(spec, 333, torch.Generator().manual_seed(9), torch.bfloat16)
     for cuts in ([333], [64, 128, 141], [9, 55, 269]):
-        runs = [DeltaRun(spec, t, "cuda", torch.bfloat16, chunk_rows=r, values=values) for r in (2, 2, 1 << 20)]
+        runs = [DeltaRun(spec, t, "cuda", torch.bfloat16, chunk_rows=r, values=values, rounds=rounds) for r in (2, 2, 1 << 20)]
         outs = [r.feed(z, cuts) for r in runs]
         assert torch.equal(outs[0], outs[1]) and torch.equal(runs[0].state(), runs[1].state())
         assert rel(runs[0].state(), runs[2].state()) < 4e-5 and worst_row(outs[0], outs[2].cpu()) < 1e-2
