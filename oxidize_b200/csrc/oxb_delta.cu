@@ -27,6 +27,33 @@ static int delta_step_launch(const DeltaArgs& a, int B, cudaStream_t stream) {
   return (int)cudaErrorInvalidValue;
 }
 
+template <int NK, int CH>
+static int delta_decode_go(const DeltaArgs& a, int B, const float* low, cudaStream_t stream) {
+  const int R = 512 / (a.V / 4);
+  oxb_launch(delta_decode_kernel<NK, CH>, dim3(a.H, B), dim3(512), (size_t)(3 * a.K + 2 * a.V + 2 * R * a.V) * sizeof(float), stream, a, low);
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
+// Steps of one row per sequence; `low`: B x (H K (+) H V) floats of scratch with low-rank projections, -1: not covered
+static int delta_decode_launch(const DeltaArgs& a, int B, float* low, cudaStream_t stream) {
+  const int n = (a.decay_up != nullptr ? a.H * a.K : 0) + (a.gate_up != nullptr ? a.H * a.V : 0);
+  if (a.taps > 4 || a.V > 256 || a.K > 256 || (n > 0 && low == nullptr) || (a.decay_up != nullptr && (a.K % 32 != 0 || a.decay_rank % 16 != 0)) ||
+      (a.gate_up != nullptr && a.gate_rank % 16 != 0))
+    return -1;
+  if (n > 0) {
+    oxb_launch(delta_low_rank_kernel, dim3((n + 255) / 256, (B + 15) / 16), dim3(256), 0, stream, a, low, B);
+    OXB_CHECK_LAUNCH();
+  }
+  const int R = 512 / (a.V / 4), nk = (a.K + R - 1) / R;
+  const bool one = 2 * a.K + a.V <= 512;
+  if (nk <= 2) return one ? delta_decode_go<2, 1>(a, B, low, stream) : delta_decode_go<2, 2>(a, B, low, stream);
+  if (nk <= 4) return one ? delta_decode_go<4, 1>(a, B, low, stream) : delta_decode_go<4, 2>(a, B, low, stream);
+  if (nk <= 8) return one ? delta_decode_go<8, 1>(a, B, low, stream) : delta_decode_go<8, 2>(a, B, low, stream);
+  if (nk <= 16) return delta_decode_go<16, 2>(a, B, low, stream);
+  return delta_decode_go<32, 2>(a, B, low, stream);
+}
+
 template <int KT, bool CH>
 static int delta_chunk_go(DeltaChunkArgs x, int B, int longest, int nv, cudaStream_t stream) {
   constexpr int K = KT * 16;
@@ -68,7 +95,8 @@ OXB_API int oxb_delta_chunk_bytes(int K, int V) {
 // Gated delta rule of a step: z [T, ld] holds q | k (G heads of K values) | v (H heads of V values) and, at the given columns,
 // gate, decay and beta; the state [num_slots, H, K, V] float32 is read and updated, the ring of convolution inputs [num_slots,
 // taps, channels] read.  Only sequences that feed min_rows .. max_rows rows take part.  write_window (single-row steps): the
-// ring is updated too; elsewhere oxb_delta_window does that afterwards.  chunk_values 0: delta_step_kernel; else (bf16) the chunk
+// ring is updated too; elsewhere oxb_delta_window does that afterwards; in bf16 these steps take delta_decode_kernel, with scratch
+// ws of B * H * (K + V) floats where a projection has a low rank.  chunk_values 0: delta_step_kernel; else (bf16) the chunk
 // kernels with that many values of the state per CTA (16 or 32), portions of up to `longest` rows, in rounds of `round`
 // chunks with scratch ws of B * round * H * oxb_delta_chunk_bytes(K, V) bytes.
 OXB_API int oxb_delta(const void* z, int ld, int dtype, int gate_off, int decay_off, int beta_off, const int* query_start,
@@ -85,6 +113,10 @@ OXB_API int oxb_delta(const void* z, int ld, int dtype, int gate_off, int decay_
   const DeltaArgs a{z, ld, gate_off, decay_off, beta_off, query_start, seq_lens, slots, conv, taps, a_log, dt_bias, decay_up, decay_rank,
                     gate_up, gate_rank, norm, state, window, num_slots, out, ld_out, out_scale, H, G, K, V, v_dim, q_scale, eps,
                     min_rows, max_rows, write_window};
+  if (chunk_values == 0 && write_window && dtype == 2) {
+    const int e = delta_decode_launch(a, B, reinterpret_cast<float*>(ws), stream);
+    if (e != -1) return e;
+  }
   if (chunk_values == 0) return dtype == 0 ? delta_step_launch<float>(a, B, stream) : delta_step_launch<__nv_bfloat16>(a, B, stream);
   if (dtype != 2 || ws == nullptr || write_window || oxb_delta_chunk_bytes(K, V) == 0 || (chunk_values != 16 && chunk_values != 32) ||
       V % chunk_values != 0 || longest <= 0 || round <= 0 || H > 65535 || ld_out % 2 != 0 || (reinterpret_cast<uintptr_t>(out) & 3) != 0 ||

@@ -63,7 +63,10 @@ def delta_rule(z: torch.Tensor, w, spec, meta, state: torch.Tensor, window: torc
     cut = CHUNK_ROWS if chunk_rows is None else chunk_rows
     size = L.oxb_delta_chunk_bytes(K, V) if z.dtype == torch.bfloat16 and most >= cut else 0
     if size == 0:
-        run(1, _ALL)
+        low = None
+        if most == 1 and z.dtype == torch.bfloat16 and z.shape[0] == B and (w.decay_up is not None or w.gate_up is not None):
+            low = torch.empty(B * H * (K + V), dtype=torch.float32, device=z.device)
+        run(1, _ALL, ws=low)
     else:
         lens = [n for n, _ in meta.host_lens] if meta.host_lens else [1, most] * B
         if min(lens) < cut:
