@@ -9,7 +9,7 @@
 // delta_state_kernel, chunk after chunk, the values of a head dealt out to CTAs: U = U0 - W S, then S'.
 // delta_output_kernel, all chunks at once: O, its norm and gate.
 //
-// A portion is worked off in rounds of as many chunks as fill the GPU once, so that what the kernels hand on stays in the L2.
+// A portion is worked off in rounds of as many chunks as the scratch holds.
 //
 // G is kept in binary logarithms, as running sums within blocks of 16 tokens and the blocks' totals, so that what lies between
 // two tokens is never the small difference of two large sums; a token's logarithm ends at -72.  In L and P a block off the
@@ -73,6 +73,13 @@ __device__ __forceinline__ void delta_load4(const __nv_bfloat16* p, float* v) {
   v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
 }
 
+// 2^x, 0 where that is no normal number
+__device__ __forceinline__ float delta_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // ----------------------------------------------------------------------------- chunks by themselves
 constexpr int DP_THREADS = 512, DP_WARPS = DP_THREADS / 32, DP_TAPS = 4, DP_RAW = DC + DP_TAPS - 1;
 constexpr float DP_FLOOR = -72.f;  // 2^ of it is far below the rounding of anything it is added to
@@ -96,41 +103,38 @@ __host__ __device__ inline DeltaPrepSmem delta_prep_smem(int K, int V) {
   return s;
 }
 
-// Four channels (this lane's) of the convolution and silu for tokens [t0, t0 + 4) of the chunk, out of raw rows in shared memory
-// (`raw`: this lane's channels three tokens ahead of the chunk, rows `row` values apart), or, for longer convolutions, out of
-// global memory; rows at or past n: zero.
-template <typename F>
-__device__ __forceinline__ void delta_conv4(const DeltaArgs& a, const __nv_bfloat16* raw, int row, const __nv_bfloat16* z, const float* ring,
-                                            int C, int pos0, int c0, int t0, int n, int ch, F put) {
+// (The kernels of this file run most of their code once per warp, and instructions that are run once come no faster than they are
+// fetched: loops stay rolled wherever registers allow it.)
+
+// Taps of this lane's four channels, zeros on the oldest rows of shorter convolutions.
+__device__ __forceinline__ void delta_taps4(const DeltaArgs& a, int C, int ch, float4 (&w)[DP_TAPS]) {
+#pragma unroll
+  for (int i = 0; i < DP_TAPS; ++i) {
+    const int tap = i - (DP_TAPS - a.taps);
+    w[i] = (tap >= 0 && a.taps <= DP_TAPS) ? *reinterpret_cast<const float4*>(a.conv + (size_t)tap * C + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+}
+// Those channels of token t of the chunk after convolution and silu, out of raw rows in shared memory (`raw`: three tokens ahead
+// of the chunk, rows `row` values apart; zeros past the portion), or, for longer convolutions, out of global memory.
+__device__ __forceinline__ void delta_conv4(const DeltaArgs& a, const float4 (&w)[DP_TAPS], const __nv_bfloat16* raw, int row,
+                                            const __nv_bfloat16* z, const float* ring, int C, int pos0, int c0, int t, int n, int ch,
+                                            float* y) {
   if (a.taps <= DP_TAPS) {
-    float w[DP_TAPS][4], x[DP_TAPS][4];
+    y[0] = y[1] = y[2] = y[3] = 0.f;
 #pragma unroll
-    for (int i = 0; i < DP_TAPS; ++i) {  // (shorter convolutions: zeros on the oldest rows)
-      const int tap = i - (DP_TAPS - a.taps);
-      const float4 v = tap >= 0 ? *reinterpret_cast<const float4*>(a.conv + (size_t)tap * C + ch) : make_float4(0.f, 0.f, 0.f, 0.f);
-      w[i][0] = v.x, w[i][1] = v.y, w[i][2] = v.z, w[i][3] = v.w;
+    for (int i = 0; i < DP_TAPS; ++i) {
+      float x[4];
+      delta_load4(raw + (t + i) * row, x);
+      y[0] = fmaf(w[i].x, x[0], y[0]);
+      y[1] = fmaf(w[i].y, x[1], y[1]);
+      y[2] = fmaf(w[i].z, x[2], y[2]);
+      y[3] = fmaf(w[i].w, x[3], y[3]);
     }
 #pragma unroll
-    for (int i = 0; i < DP_TAPS - 1; ++i) delta_load4(raw + (t0 + i) * row, x[i]);
-#pragma unroll
-    for (int t = 0; t < 4; ++t) {
-      delta_load4(raw + (t0 + t + DP_TAPS - 1) * row, x[(t + DP_TAPS - 1) % DP_TAPS]);
-      float y[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        float s = 0.f;
-#pragma unroll
-        for (int i = 0; i < DP_TAPS; ++i) s = fmaf(w[i][e], x[(t + i) % DP_TAPS][e], s);
-        y[e] = t0 + t < n ? s * delta_sigmoid_fast(s) : 0.f;
-      }
-      put(t0 + t, y);
-    }
+    for (int e = 0; e < 4; ++e) y[e] *= delta_sigmoid_fast(y[e]);
   } else {
-    for (int t = t0; t < t0 + 4; ++t) {
-      float y[4];
-      for (int e = 0; e < 4; ++e) y[e] = t < n ? delta_conv(a, z, ring, C, pos0, c0 + t, ch + e) : 0.f;
-      put(t, y);
-    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[e] = t < n ? delta_conv(a, z, ring, C, pos0, c0 + t, ch + e) : 0.f;
   }
 }
 
@@ -195,19 +199,26 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
   pdl_wait();
   // ---- raw rows of q | k and of v, from three tokens ahead of the chunk on
   if (a.taps <= DP_TAPS) {
-    const int pieces = 2 * K8 + V8;
-    for (int i = tid; i < DP_RAW * pieces; i += DP_THREADS) {
-      const int r = i / pieces, p = i % pieces, j = c0 - (DP_TAPS - 1) + r;
-      const int ch = p < K8 ? kvh * K + p * 8 : (p < 2 * K8 ? (a.G + kvh) * K + (p - K8) * 8 : 2 * a.G * K + h * V + (p - 2 * K8) * 8);
-      __nv_bfloat16* dst = p < 2 * K8 ? raw_qk + (r * 2 * K8 + p) * 8 : raw_v + (r * V8 + p - 2 * K8) * 8;
-      if (j >= 0 && j < n_all) {
-        cp_async16(dst, z + (size_t)j * a.ld + ch);
-      } else if (j < 0 && pos0 + j >= 0 && j > -a.taps) {  // (an earlier step's projections: 16-bit values)
-        float v[8];
-        delta_load8(ring + (size_t)((pos0 + j) % a.taps) * C + ch, v);
-        *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
-      } else {
-        *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+    const __nv_bfloat16 *zq = z + kvh * K, *zv = z + 2 * a.G * K + h * V;
+#pragma unroll 1
+    for (int r = warp; r < DP_RAW; r += DP_WARPS) {
+      const int j = c0 - (DP_TAPS - 1) + r;
+      const bool now = j >= 0 && j < n_all, past = j < 0 && pos0 + j >= 0 && j > -a.taps;
+      const float* old = ring + (past ? (size_t)((pos0 + j) % a.taps) * C : 0);
+#pragma unroll 1
+      for (int p = lane; p < 2 * K8 + V8; p += 32) {
+        const bool is_v = p >= 2 * K8;
+        const int off = is_v ? (p - 2 * K8) * 8 : (p < K8 ? p * 8 : a.G * K + (p - K8) * 8);
+        __nv_bfloat16* dst = is_v ? raw_v + r * V + off : raw_qk + (r * 2 * K8 + p) * 8;
+        if (now) {
+          cp_async16(dst, (is_v ? zv : zq) + (size_t)j * a.ld + off);
+        } else if (past) {  // (an earlier step's projections: 16-bit values)
+          float v[8];
+          delta_load8(old + (is_v ? 2 * a.G * K + h * V : kvh * K) + off, v);
+          *reinterpret_cast<uint4*>(dst) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+        } else {
+          *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        }
       }
     }
   }
@@ -225,15 +236,10 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
                            reinterpret_cast<const __nv_bfloat16*>(a.decay_up) + (size_t)(h * K + d0 + g) * a.decay_rank + 4 * t4, a.decay_rank,
                            K / 32, acc);
 #pragma unroll
-    for (int i = 0; i < K / 32; ++i) {
-      const float2 dt = *reinterpret_cast<const float2*>(a.dt_bias + h * K + d0 + i * 8 + 2 * t4);
+    for (int i = 0; i < K / 32; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int t = mt * 16 + g + 8 * (e >> 1);
-        const float v0 = fmaxf(-rate * delta_softplus(acc[i][e] + dt.x), DP_FLOOR), v1 = fmaxf(-rate * delta_softplus(acc[i][e + 1] + dt.y), DP_FLOOR);
-        *reinterpret_cast<float2*>(sG + t * KF + d0 + i * 8 + 2 * t4) = t < n ? make_float2(v0, v1) : make_float2(0.f, 0.f);
-      }
-    }
+      for (int e = 0; e < 4; e += 2)
+        *reinterpret_cast<float2*>(sG + (mt * 16 + g + 8 * (e >> 1)) * KF + d0 + i * 8 + 2 * t4) = make_float2(acc[i][e], acc[i][e + 1]);
   } else if (warp == 0) {
     float v[2];
 #pragma unroll
@@ -258,27 +264,32 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
   // ---- q and k: convolution, silu, unit vectors; a warp has four tokens, a lane four channels
 #pragma unroll 1
   for (int side = 0; side < 2; ++side) {
-    const int d = lane * 4, dc = min(d, K - 4);
+    const int d = lane * 4, dc = min(d, K - 4), ch = (side ? a.G + kvh : kvh) * K + dc;
     float* dst = (side ? sK : sQ) + d;
-    delta_conv4(a, raw_qk + side * K + dc, 2 * K, z, ring, C, pos0, c0, warp * 4, n, (side ? a.G + kvh : kvh) * K + dc,
-                [&](int t, const float* y) {
-                  const float ss = d < K ? (y[0] * y[0] + y[1] * y[1]) + (y[2] * y[2] + y[3] * y[3]) : 0.f;
-                  const float f = rsqrtf(warp_sum(ss) + 1e-6f) * (side ? 1.f : a.q_scale);
-                  if (d < K) *reinterpret_cast<float4*>(dst + t * KF) = make_float4(y[0] * f, y[1] * f, y[2] * f, y[3] * f);
-                });
+    float4 w[DP_TAPS];
+    delta_taps4(a, C, ch, w);
+#pragma unroll 2
+    for (int t = warp * 4; t < warp * 4 + 4; ++t) {
+      float y[4];
+      delta_conv4(a, w, raw_qk + side * K + dc, 2 * K, z, ring, C, pos0, c0, t, n, ch, y);
+      const float ss = d < K ? (y[0] * y[0] + y[1] * y[1]) + (y[2] * y[2] + y[3] * y[3]) : 0.f;
+      const float f = t < n ? rsqrtf(warp_sum(ss) + 1e-6f) * (side ? 1.f : a.q_scale) : 0.f;
+      if (d < K) *reinterpret_cast<float4*>(dst + t * KF) = make_float4(y[0] * f, y[1] * f, y[2] * f, y[3] * f);
+    }
   }
   if (CH) {  // running sums (512 threads: four blocks of up to 128 channels)
     const int d = tid % K, blk = tid / K;
     if (blk < 4) {
-      float v[16];
-#pragma unroll
-      for (int i = 0; i < 16; ++i) v[i] = sG[(blk * 16 + i) * KF + d];
-#pragma unroll
-      for (int i = 1; i < 16; ++i) v[i] += v[i - 1];
-#pragma unroll
-      for (int i = 1; i < 16; ++i) sG[(blk * 16 + i) * KF + d] = v[i];
-      total[blk * K + d] = v[15];
-      if (v[15] < DP_RANGE) wild[blk] = 1;
+      const float dt = a.dt_bias[h * K + d];
+      float sum = 0.f;
+#pragma unroll 2
+      for (int t = blk * 16; t < blk * 16 + 16; ++t) {
+        const float v = fmaxf(-rate * delta_softplus(sG[t * KF + d] + dt), DP_FLOOR);
+        sum += t < n ? v : 0.f;
+        sG[t * KF + d] = sum;
+      }
+      total[blk * K + d] = sum;
+      if (sum < DP_RANGE) wild[blk] = 1;
     }
   }
   __syncthreads();
@@ -321,7 +332,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
       float accK[2][4], accQ[2][4];
 #pragma unroll
       for (int i = 0; i < 2; ++i) accK[i][0] = accK[i][1] = accK[i][2] = accK[i][3] = accQ[i][0] = accQ[i][1] = accQ[i][2] = accQ[i][3] = 0.f;
-#pragma unroll 2
+#pragma unroll 1
       for (int ks = 0; ks < KT; ++ks) {
         uint32_t kh[4], kl[4], qh[4], ql[4];
 #pragma unroll
@@ -330,7 +341,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
           float2 kv = *reinterpret_cast<const float2*>(sK + t * KF + d), qv = *reinterpret_cast<const float2*>(sQ + t * KF + d);
           if (CH) {
             const float2 l = *reinterpret_cast<const float2*>(sG + t * KF + d);
-            const float fx = exp2f(l.x), fy = exp2f(l.y);
+            const float fx = delta_exp2(l.x), fy = delta_exp2(l.y);
             kv = make_float2(kv.x * fx, kv.y * fy);
             qv = make_float2(qv.x * fx, qv.y * fy);
           }
@@ -352,7 +363,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
               } else {
                 l = until2(s, mt, d);
               }
-              kv = make_float2(kv.x * exp2f(l.x), kv.y * exp2f(l.y));
+              kv = make_float2(kv.x * delta_exp2(l.x), kv.y * delta_exp2(l.y));
             }
             split_bf16x2(kv.x, kv.y, bh[j], bl[j]);
           }
@@ -372,11 +383,11 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
           float f0 = 1.f, f1 = 1.f;
           if (!CH) {
             if (diag) {
-              f0 = exp2f(fminf(sG[t] - sG[s], 0.f));  // (positive only where the triangle is cut off)
-              f1 = exp2f(fminf(sG[t] - sG[s + 1], 0.f));
+              f0 = delta_exp2(fminf(sG[t] - sG[s], 0.f));  // (positive only where the triangle is cut off)
+              f1 = delta_exp2(fminf(sG[t] - sG[s + 1], 0.f));
             } else {
-              f0 = exp2f(sG[t] + until2(s, mt, 0).x);
-              f1 = exp2f(sG[t] + until2(s + 1, mt, 0).x);
+              f0 = delta_exp2(sG[t] + until2(s, mt, 0).x);
+              f1 = delta_exp2(sG[t] + until2(s + 1, mt, 0).x);
             }
           }
           const bool on0 = !diag || s <= t, on1 = !diag || s + 1 <= t;
@@ -389,6 +400,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
     }
   } else {
     // ---- meanwhile: exp(G) k for this kernel, exp(G) q and exp(G_end - G) k for the others
+#pragma unroll 1
     for (int i = tid - 320; i < DC * K8; i += DP_THREADS - 320) {
       const int t = i / K8, p = i % K8;
       float kv[8], qv[8], f[8], r[8], y[8];
@@ -397,7 +409,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
 #pragma unroll
       for (int e = 0; e < 8; e += 2) {
         const float2 u = since2(t, p * 8 + e), w = until2(t, DC / 16, p * 8 + e);
-        f[e] = exp2f(u.x), f[e + 1] = exp2f(u.y), r[e] = exp2f(w.x), r[e + 1] = exp2f(w.y);
+        f[e] = delta_exp2(u.x), f[e + 1] = delta_exp2(u.y), r[e] = delta_exp2(w.x), r[e + 1] = delta_exp2(w.y);
       }
 #pragma unroll
       for (int e = 0; e < 8; ++e) y[e] = kv[e] * f[e];
@@ -415,7 +427,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
     for (int d = tid - 320; d < K; d += DP_THREADS - 320) {
       float s = 0.f;
       for (int i = 0; i < DC / 16; ++i) s += total[CH ? i * K + d : i];
-      reinterpret_cast<float*>(block + pl.gend)[d] = exp2f(s);
+      reinterpret_cast<float*>(block + pl.gend)[d] = delta_exp2(s);
     }
   }
   if (CH && wild[warp >> 2]) {  // a block on the diagonal column by column: a warp has four columns, a lane CPL channels
@@ -425,6 +437,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
     for (int s = 0; s < 4; ++s)
 #pragma unroll
       for (int i = 0; i < CPL; ++i) w[s][i] = 0.f;
+#pragma unroll 1
     for (int t = t0; t < t0 + 16; ++t) {
       float sum[8];  // k . w, q . w of the four columns
 #pragma unroll
@@ -434,7 +447,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
         for (int i = 0; i < CPL; ++i) {
           const int d = lane + 32 * i;
           const float kt = sK[t * KF + d], qt = sQ[t * KF + d];
-          const float f = t > s0 ? exp2f(sG[t * KF + d] - sG[(t - 1) * KF + d]) : 0.f;
+          const float f = t > s0 ? delta_exp2(sG[t * KF + d] - sG[(t - 1) * KF + d]) : 0.f;
 #pragma unroll
           for (int s = 0; s < 4; ++s) {
             w[s][i] = t == s0 + s ? kt : w[s][i] * f;  // (zero ahead of its own token)
@@ -472,63 +485,65 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
   // ---- the inverse of I + L: blocks of 16 on the diagonal by substitution, the others from them
   if (warp < 2) {
     const int t0 = tid & ~15, c = tid & 15;
-    float v[16];
+    float *col = sT + t0 * DC_LD + t0 + c, *rows = sL + t0 * DC_LD + t0;
 #pragma unroll
-    for (int r = 0; r < 16; ++r) {
-      float s[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int r = 0; r < 16; ++r) col[r * DC_LD] = r == c ? 1.f : 0.f;
+#pragma unroll 1
+    for (int r = 1; r < 16; ++r) {  // (rows at and past r are zero, but for the one on the diagonal)
+      float s[4];
 #pragma unroll
-      for (int i = 0; i < 16; ++i)
-        if (i < r) s[i & 3] = fmaf(sL[(t0 + r) * DC_LD + t0 + i], v[i], s[i & 3]);
-      v[r] = r < c ? 0.f : (r == c ? 1.f : -((s[0] + s[1]) + (s[2] + s[3])));
-      sT[(t0 + r) * DC_LD + t0 + c] = v[r];
+      for (int i = 0; i < 16; i += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(rows + r * DC_LD + i);
+        s[i >> 2] = (l.x * col[i * DC_LD] + l.y * col[(i + 1) * DC_LD]) + (l.z * col[(i + 2) * DC_LD] + l.w * col[(i + 3) * DC_LD]);
+      }
+      if (r > c) col[r * DC_LD] = -((s[0] + s[1]) + (s[2] + s[3]));
     }
   } else {  // (meanwhile) v: convolution and silu, as halves where the decays were
-    const int d = lane * 4, dc = min(d, V - 4);
-    for (int r = warp - 2; r < DC / 4; r += DP_WARPS - 2)
-      delta_conv4(a, raw_v + dc, V, z, ring, C, pos0, c0, r * 4, n, 2 * a.G * K + h * V + dc, [&](int t, const float* y) {
-        if (d >= V) return;
-        uint32_t h0, l0, h1, l1;
-        split_bf16x2(y[0], y[1], h0, l0);
-        split_bf16x2(y[2], y[3], h1, l1);
-        uint8_t* at = dp_smem + sm.g + t * RV + d * 2;
-        *reinterpret_cast<uint2*>(at) = make_uint2(h0, h1);
-        *reinterpret_cast<uint2*>(at + VHALF) = make_uint2(l0, l1);
-      });
+    const int d = lane * 4, dc = min(d, V - 4), ch = 2 * a.G * K + h * V + dc;
+    float4 w[DP_TAPS];
+    delta_taps4(a, C, ch, w);
+#pragma unroll 1
+    for (int t = warp - 2; t < DC; t += DP_WARPS - 2) {
+      float y[4];
+      delta_conv4(a, w, raw_v + dc, V, z, ring, C, pos0, c0, t, n, ch, y);
+      if (d >= V) continue;
+      uint32_t h0, l0, h1, l1;
+      split_bf16x2(t < n ? y[0] : 0.f, t < n ? y[1] : 0.f, h0, l0);
+      split_bf16x2(t < n ? y[2] : 0.f, t < n ? y[3] : 0.f, h1, l1);
+      uint8_t* at = dp_smem + sm.g + t * RV + d * 2;
+      *reinterpret_cast<uint2*>(at) = make_uint2(h0, h1);
+      *reinterpret_cast<uint2*>(at + VHALF) = make_uint2(l0, l1);
+    }
   }
   __syncthreads();
-#pragma unroll
+#pragma unroll 1
   for (int dist = 1; dist < 4; ++dist) {
     // block (i, i - dist): first sum_k L_ik T_kj into the (unused) mirror block above the diagonal, then - T_ii times that
-    for (int u = tid; u < (4 - dist) * 256; u += DP_THREADS) {
-      const int j = u >> 8, i = j + dist, r = u >> 4 & 15, c = u & 15;
-      const float *lr = sL + (i * 16 + r) * DC_LD + j * 16, *tc = sT + j * 16 * DC_LD + j * 16 + c;
-      float s[2] = {0.f, 0.f};
+#pragma unroll 1
+    for (int step = 0; step < 2; ++step) {
+#pragma unroll 1
+      for (int u = tid; u < (4 - dist) * 256; u += DP_THREADS) {
+        const int j = u >> 8, i = j + dist, r = u >> 4 & 15, c = u & 15;
+        const float* x = step ? sT + (i * 16 + r) * DC_LD + i * 16 : sL + (i * 16 + r) * DC_LD + j * 16;
+        const float* y = step ? sL + j * 16 * DC_LD + i * 16 + c : sT + j * 16 * DC_LD + j * 16 + c;
+        float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 1
+        for (int m = 0; m < (step ? 1 : dist); ++m, x += 16, y += 16 * DC_LD) {
 #pragma unroll
-      for (int m = 0; m < 16 * dist; m += 4) {
-        const float4 y = *reinterpret_cast<const float4*>(lr + m);
-        s[0] = fmaf(y.x, tc[m * DC_LD], s[0]);
-        s[1] = fmaf(y.y, tc[(m + 1) * DC_LD], s[1]);
-        s[0] = fmaf(y.z, tc[(m + 2) * DC_LD], s[0]);
-        s[1] = fmaf(y.w, tc[(m + 3) * DC_LD], s[1]);
+          for (int k = 0; k < 16; k += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(x + k);
+            s[0] = fmaf(v.x, y[k * DC_LD], s[0]);
+            s[1] = fmaf(v.y, y[(k + 1) * DC_LD], s[1]);
+            s[2] = fmaf(v.z, y[(k + 2) * DC_LD], s[2]);
+            s[3] = fmaf(v.w, y[(k + 3) * DC_LD], s[3]);
+          }
+        }
+        const float sum = (s[0] + s[1]) + (s[2] + s[3]);
+        if (step) sT[(i * 16 + r) * DC_LD + j * 16 + c] = -sum;
+        else sL[(j * 16 + r) * DC_LD + i * 16 + c] = sum;
       }
-      sL[(j * 16 + r) * DC_LD + i * 16 + c] = s[0] + s[1];
+      __syncthreads();
     }
-    __syncthreads();
-    for (int u = tid; u < (4 - dist) * 256; u += DP_THREADS) {
-      const int j = u >> 8, i = j + dist, r = u >> 4 & 15, c = u & 15;
-      const float *tr = sT + (i * 16 + r) * DC_LD + i * 16, *mc = sL + j * 16 * DC_LD + i * 16 + c;
-      float s[2] = {0.f, 0.f};
-#pragma unroll
-      for (int m = 0; m < 16; m += 4) {
-        const float4 y = *reinterpret_cast<const float4*>(tr + m);
-        s[0] = fmaf(y.x, mc[m * DC_LD], s[0]);
-        s[1] = fmaf(y.y, mc[(m + 1) * DC_LD], s[1]);
-        s[0] = fmaf(y.z, mc[(m + 2) * DC_LD], s[0]);
-        s[1] = fmaf(y.w, mc[(m + 3) * DC_LD], s[1]);
-      }
-      sT[(i * 16 + r) * DC_LD + j * 16 + c] = -(s[0] + s[1]);
-    }
-    __syncthreads();
   }
   {  // times beta, as halves: 64 rows of eight pieces
     const int t = tid >> 3, p = tid & 7;
@@ -555,13 +570,14 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
       for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
         for (int i = 0; i < 2; ++i) acc[mt][i][0] = acc[mt][i][1] = acc[mt][i][2] = acc[mt][i][3] = 0.f;
-#pragma unroll
+#pragma unroll 1
       for (int ks = 0; ks < 4; ++ks) {
         uint32_t bh[4], bl[4];
         ldmatrix_x4_trans(Bm + ks * 16 * rb, bh[0], bh[1], bh[2], bh[3]);
         ldmatrix_x4_trans(Bm + DC * rb + ks * 16 * rb, bl[0], bl[1], bl[2], bl[3]);
 #pragma unroll
-        for (int mt = ks; mt < 4; ++mt) {
+        for (int mt = 0; mt < 4; ++mt) {
+          if (mt < ks) continue;  // (the same for all)
           uint32_t ah[4], al[4];
           ldmatrix_x4(A + mt * 16 * DC_PROW + ks * 32, ah[0], ah[1], ah[2], ah[3]);
           ldmatrix_x4(A + (DC + mt * 16) * DC_PROW + ks * 32, al[0], al[1], al[2], al[3]);

@@ -13,6 +13,7 @@ from .cuda import _check, _p, _stream
 
 _declared = False
 _ALL = 1 << 30
+SCRATCH_BYTES = 512 << 20  # of the chunk kernels
 CHUNK, CHUNK_ROWS = 64, 9  # tokens per chunk; sequences that feed at least CHUNK_ROWS rows in a step go through chunks
 
 
@@ -29,14 +30,16 @@ def lib():
     return L
 
 
-def chunk_values(V: int) -> int:
-    """Values of a head's state per CTA of the kernel that goes from chunk to chunk."""
-    return 32 if V % 32 == 0 else 16
+def chunk_values(V: int, heads: int, sms: int) -> int:
+    """Values of a head's state per CTA of the kernel that goes from chunk to chunk: the fewer, the shorter each of its steps,
+    as long as all CTAs run at once."""
+    return 32 if V % 32 == 0 and heads * (V // 16) > sms else 16
 
 
-def round_chunks(heads: int, sms: int) -> int:
-    """Chunks of a round: as many as give every SM one (chunk, head)."""
-    return max(1, sms // max(1, heads))
+def round_chunks(chunks: int, bytes_per_chunk: int) -> int:
+    """Chunks of a round: as many as the scratch limit lets through, in rounds of equal length."""
+    rounds = -(-chunks * bytes_per_chunk // SCRATCH_BYTES)
+    return max(1, -(-chunks // rounds))
 
 
 def delta_rule(z: torch.Tensor, w, spec, meta, state: torch.Tensor, window: torch.Tensor, eps: float, out: torch.Tensor,
@@ -72,9 +75,9 @@ def delta_rule(z: torch.Tensor, w, spec, meta, state: torch.Tensor, window: torc
         if min(lens) < cut:
             run(1, cut - 1)
         long, sms = H * sum(n >= cut for n in lens), opcuda.sm_count(z.device)
-        rnd = min((most + CHUNK - 1) // CHUNK, round_chunks(long, sms) if rounds is None else rounds)
+        rnd = round_chunks((most + CHUNK - 1) // CHUNK, B * H * size) if rounds is None else rounds
         ws = torch.empty(B * rnd * H * size, dtype=torch.uint8, device=z.device)
-        run(cut, _ALL, chunk_values(V) if values is None else values, rnd, ws)
+        run(cut, _ALL, chunk_values(V, long, sms) if values is None else values, rnd, ws)
     if most > 1:
         _check(L.oxb_delta_window(z.data_ptr(), z.stride(0), dt, meta.query_start.data_ptr(), meta.seq_lens.data_ptr(),
                                   meta.state_slots.data_ptr(), spec.conv, window.data_ptr(), state.shape[0], B, H, G, K, V, _stream()),
