@@ -167,6 +167,12 @@ __device__ __forceinline__ void tma_prefetch_l2_2d(const CUtensorMap* d, int c0,
                : "memory");
 }
 // 2-D tiled load into this CTA's own shared memory (every CTA fetches its own tiles)
+// `bytes` (a multiple of 16) of this GPU's own memory; both addresses on 16-byte boundaries
+__device__ __forceinline__ void bulk_load(void* smem_dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(smem_dst)), "l"(src),
+               "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
+}
 __device__ __forceinline__ void tma_load_2d(void* smem_dst, const CUtensorMap* d, uint64_t* bar, int c0, int c1) {
   asm volatile(
       "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"

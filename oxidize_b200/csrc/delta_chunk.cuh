@@ -29,21 +29,24 @@ constexpr int DC = 64;                // tokens per chunk
 constexpr int DC_LD = DC + 4;         // floats of a row of L and of the inverse
 constexpr int DC_PROW = DC * 2 + 16;  // bytes of a row of 64 halves in shared memory
 
-// Scratch of one (chunk, head), in bytes.
+// Scratch of one (chunk, head), in bytes: arrays as they stand in shared memory (rows padded by 16 bytes), one bulk copy each.
+// Pairs of halves lie behind each other (hi, lo).
 struct DeltaPlan {
-  int w, kb, u0, gend, qt, p, u, s, bytes;  // offsets; pairs of halves lie behind each other (hi, lo)
+  int w, kb, u0, gend, qt, s, p, u, bytes;  // offsets
 };
+constexpr int DC_USLICE = DC * (16 * 4 + 16);  // bytes of 16 values of U0, [64][16 + padding]
 __host__ __device__ inline DeltaPlan delta_plan(int K, int V) {
+  const int rk = 2 * DC * (K * 2 + 16), rv = V * 2 + 16;
   DeltaPlan p;
   p.w = 0;
-  p.kb = p.w + 2 * DC * K * 2;
-  p.u0 = p.kb + 2 * DC * K * 2;
-  p.gend = p.u0 + DC * V * 4;
+  p.kb = p.w + rk;
+  p.u0 = p.kb + rk;
+  p.gend = p.u0 + V / 16 * DC_USLICE;
   p.qt = p.gend + K * 4;
-  p.p = p.qt + 2 * DC * K * 2;
-  p.u = p.p + 2 * DC * DC * 2;
-  p.s = p.u + 2 * DC * V * 2;
-  p.bytes = p.s + 2 * K * V * 2;
+  p.s = p.qt + rk;
+  p.p = p.s + 2 * K * rv;
+  p.u = p.p + 2 * DC * DC_PROW;
+  p.bytes = p.u + 2 * DC * rv;
   return p;
 }
 
@@ -323,7 +326,8 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
     }
     return v;
   };
-  __nv_bfloat16 *p_hi = reinterpret_cast<__nv_bfloat16*>(block + pl.p), *p_lo = p_hi + DC * DC;
+  constexpr int PR = DC_PROW / 2;
+  __nv_bfloat16 *p_hi = reinterpret_cast<__nv_bfloat16*>(block + pl.p), *p_lo = p_hi + DC * PR;
   if (warp < 10) {
     // ---- L and P, blocks of 16 x 16, operands from the float32 rows
     const int mt = warp < 1 ? 0 : (warp < 3 ? 1 : (warp < 6 ? 2 : 3)), np = warp - mt * (mt + 1) / 2;
@@ -393,8 +397,8 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
           const bool on0 = !diag || s <= t, on1 = !diag || s + 1 <= t;
           uint32_t hi, lo;
           split_bf16x2(on0 ? accQ[i][e] * f0 : 0.f, on1 ? accQ[i][e + 1] * f1 : 0.f, hi, lo);
-          *reinterpret_cast<uint32_t*>(p_hi + t * DC + s) = hi;
-          *reinterpret_cast<uint32_t*>(p_lo + t * DC + s) = lo;
+          *reinterpret_cast<uint32_t*>(p_hi + t * PR + s) = hi;
+          *reinterpret_cast<uint32_t*>(p_lo + t * PR + s) = lo;
           *reinterpret_cast<float2*>(sL + t * DC_LD + s) = make_float2(on0 ? accK[i][e] * f0 * beta[t] : 0.f, on1 ? accK[i][e + 1] * f1 * beta[t] : 0.f);
         }
     }
@@ -417,12 +421,12 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
       delta_split8(y, at, at + HALF);
 #pragma unroll
       for (int e = 0; e < 8; ++e) y[e] = qv[e] * f[e];
-      at = block + pl.qt + (t * K + p * 8) * 2;
-      delta_split8(y, at, at + DC * K * 2);
+      at = block + pl.qt + t * RB + p * 16;
+      delta_split8(y, at, at + HALF);
 #pragma unroll
       for (int e = 0; e < 8; ++e) y[e] = kv[e] * r[e];
-      at = block + pl.kb + (t * K + p * 8) * 2;
-      delta_split8(y, at, at + DC * K * 2);
+      at = block + pl.kb + t * RB + p * 16;
+      delta_split8(y, at, at + HALF);
     }
     for (int d = tid - 320; d < K; d += DP_THREADS - 320) {
       float s = 0.f;
@@ -475,8 +479,8 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
         } else {
           const float v = s <= t ? sum[0] : 0.f;
           const __nv_bfloat16 hi = __float2bfloat16(v);
-          p_hi[t * DC + s] = hi;
-          p_lo[t * DC + s] = __float2bfloat16(v - __bfloat162float(hi));
+          p_hi[t * PR + s] = hi;
+          p_lo[t * PR + s] = __float2bfloat16(v - __bfloat162float(hi));
         }
       }
     }
@@ -599,11 +603,11 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
             if (is_w) {
               uint32_t hi, lo;
               split_bf16x2(acc[mt][i][e], acc[mt][i][e + 1], hi, lo);
-              uint8_t* at = block + pl.w + (t * K + c) * 2;
+              uint8_t* at = block + pl.w + t * RB + c * 2;
               *reinterpret_cast<uint32_t*>(at) = hi;
-              *reinterpret_cast<uint32_t*>(at + DC * K * 2) = lo;
+              *reinterpret_cast<uint32_t*>(at + HALF) = lo;
             } else {
-              *reinterpret_cast<float2*>(block + pl.u0 + (t * V + c) * 4) = make_float2(acc[mt][i][e], acc[mt][i][e + 1]);
+              *reinterpret_cast<float2*>(block + pl.u0 + col * DC_USLICE + t * 80 + (8 * i + 2 * t4) * 4) = make_float2(acc[mt][i][e], acc[mt][i][e + 1]);
             }
           }
     }
@@ -612,7 +616,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
 
 // ----------------------------------------------------------------------------- the state, chunk after chunk
 constexpr int DS_THREADS = 512;
-__host__ __device__ inline int delta_state_stage(int K, int NV) { return 4 * DC * (K * 2 + 16) + DC * (NV * 4 + 16) + K * 4; }
+__host__ __device__ inline int delta_state_stage(int K, int NV) { return 4 * DC * (K * 2 + 16) + NV / 16 * DC_USLICE + K * 4; }
 __host__ __device__ inline int delta_state_smem(int K, int NV) {
   return 2 * delta_state_stage(K, NV) + 2 * K * (NV * 2 + 16) + 2 * DC * (NV * 2 + 16);
 }
@@ -621,8 +625,10 @@ __host__ __device__ inline int delta_state_smem(int K, int NV) {
 // accumulator registers, and a tile of U of 16 tokens x 8 values.
 template <int KT, int NV>
 __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaChunkArgs x) {
-  constexpr int K = KT * 16, RB = K * 2 + 16, RN = NV * 2 + 16, RU = NV * 4 + 16, K8 = K / 8, NV4 = NV / 4;
+  constexpr int K = KT * 16, RB = K * 2 + 16, RN = NV * 2 + 16, US = NV / 16 * DC_USLICE;
   extern __shared__ __align__(16) uint8_t dt_smem[];
+  __shared__ uint64_t full[2];
+  __shared__ volatile int abort_flag;
   pdl_launch_dependents();
   const DeltaArgs& a = x.a;
   const int v0 = blockIdx.x * NV, h = blockIdx.y, b = blockIdx.z;
@@ -635,17 +641,23 @@ __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaC
   const int stage_bytes = delta_state_stage(K, NV);
   uint8_t* sS = dt_smem + 2 * stage_bytes;  // [hi, lo][K][RN]
   uint8_t* sU = sS + 2 * K * RN;            // [hi, lo][64][RN]
-  auto fetch = [&](int c) {                 // W hi, lo, Kb hi, lo [64][RB] | U0 [64][RU] | gend [K]
+  const int RV = V * 2 + 16;
+  if (tid == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    abort_flag = 0;
+    mbar_fence_init();
+  }
+  auto fetch = [&](int c) {  // one thread: W, Kb [hi, lo][64][RB] | U0, slices of 16 values | gend [K]
     const uint8_t* block = delta_block(x, pl.bytes, b, c, h);
-    uint8_t* dst = dt_smem + (c & 1) * stage_bytes;
-    for (int i = tid; i < 4 * DC * K8; i += DS_THREADS) cp_async16(dst + i / K8 * RB + i % K8 * 16, block + (size_t)i * 16);
-    dst += 4 * DC * RB;
-    for (int i = tid; i < DC * NV4; i += DS_THREADS)
-      cp_async16(dst + i / NV4 * RU + i % NV4 * 16, block + pl.u0 + ((size_t)(i / NV4) * V + v0) * 4 + i % NV4 * 16);
-    for (int i = tid; i < K / 4; i += DS_THREADS) cp_async16(dst + DC * RU + i * 16, block + pl.gend + i * 16);
-    cp_async_commit();
+    const int i = (c - x.chunk0) & 1;
+    uint8_t* dst = dt_smem + i * stage_bytes;
+    mbar_expect_tx(&full[i], stage_bytes);
+    bulk_load(dst, block, 4 * DC * RB, &full[i]);
+    bulk_load(dst + 4 * DC * RB, block + pl.u0 + v0 / 16 * DC_USLICE, US, &full[i]);
+    bulk_load(dst + 4 * DC * RB + US, block + pl.gend, K * 4, &full[i]);
   };
-  fetch(x.chunk0);
+  if (tid == 0) fetch(x.chunk0);
   const int srow = warp % KT, scol = warp / KT;
   const bool owner = scol < NV / 16;  // this warp has a part of the state
   const bool resumed = a.seq_lens[b] > n || x.chunk0 > 0;
@@ -670,9 +682,9 @@ __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaC
         const int k = srow * 16 + g + 8 * (e >> 1), c = scol * 16 + 8 * i + 2 * t4;
         *reinterpret_cast<uint32_t*>(sS + k * RN + c * 2) = hi;
         *reinterpret_cast<uint32_t*>(sS + K * RN + k * RN + c * 2) = lo;
-        uint8_t* at = block + pl.s + ((size_t)k * V + v0 + c) * 2;
+        uint8_t* at = block + pl.s + k * RV + (v0 + c) * 2;
         *reinterpret_cast<uint32_t*>(at) = hi;
-        *reinterpret_cast<uint32_t*>(at + (size_t)K * V * 2) = lo;
+        *reinterpret_cast<uint32_t*>(at + K * RV) = lo;
       }
   };
   const uint32_t base = smem_u32(dt_smem), s_u = smem_u32(sS), u_u = smem_u32(sU);
@@ -685,11 +697,13 @@ __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaC
   for (int c = x.chunk0; c < chunk1; ++c) {
     uint8_t* block = delta_block(x, pl.bytes, b, c, h);
     put_state(block);
-    cp_async_wait<0>();
-    __syncthreads();  // this chunk's operands and the state are in shared memory; the other buffer has been read
-    if (c + 1 < chunk1) fetch(c + 1);
-    const uint32_t W = base + (c & 1) * stage_bytes, Kb = W + 2 * DC * RB;
-    const uint8_t* extra = dt_smem + (c & 1) * stage_bytes + 4 * DC * RB;
+    __syncthreads();  // the state is in shared memory; the other buffer has been read
+    if (tid == 0 && c + 1 < chunk1) fetch(c + 1);
+    const int step = c - x.chunk0, stage = (step & 1) * stage_bytes;
+    mbar_wait_bounded(&full[step & 1], step >> 1 & 1, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+    __syncwarp();
+    const uint32_t W = base + stage, Kb = W + 2 * DC * RB;
+    const uint8_t* extra = dt_smem + stage + 4 * DC * RB;
     if (has_u) {
       float acc[3][4];
 #pragma unroll
@@ -712,19 +726,19 @@ __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaC
 #pragma unroll
       for (int e = 0; e < 4; e += 2) {
         const int t = mt * 16 + g + 8 * (e >> 1), cc = un + 2 * t4;
-        const float2 u0 = *reinterpret_cast<const float2*>(extra + t * RU + cc * 4);
+        const float2 u0 = *reinterpret_cast<const float2*>(extra + (cc >> 4) * DC_USLICE + t * 80 + (cc & 15) * 4);
         uint32_t hi, lo;
         split_bf16x2(u0.x - (acc[0][e] + (acc[1][e] + acc[2][e])), u0.y - (acc[0][e + 1] + (acc[1][e + 1] + acc[2][e + 1])), hi, lo);
         *reinterpret_cast<uint32_t*>(sU + t * RN + cc * 2) = hi;
         *reinterpret_cast<uint32_t*>(sU + DC * RN + t * RN + cc * 2) = lo;
-        uint8_t* at = block + pl.u + ((size_t)t * V + v0 + cc) * 2;
+        uint8_t* at = block + pl.u + t * RV + (v0 + cc) * 2;
         *reinterpret_cast<uint32_t*>(at) = hi;
-        *reinterpret_cast<uint32_t*>(at + (size_t)DC * V * 2) = lo;
+        *reinterpret_cast<uint32_t*>(at + DC * RV) = lo;
       }
     }
     __syncthreads();  // U is complete; the state's halves have been read
     if (owner) {
-      const float* ge = reinterpret_cast<const float*>(extra + DC * RU) + srow * 16 + g;
+      const float* ge = reinterpret_cast<const float*>(extra + US) + srow * 16 + g;
       float acc[2][2][4];  // (the low halves' products in accumulators of their own)
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
@@ -761,6 +775,10 @@ __global__ void __launch_bounds__(DS_THREADS, 1) delta_state_kernel(const DeltaC
 #pragma unroll
       for (int e = 0; e < 4; e += 2) *reinterpret_cast<float2*>(st + (size_t)(e >> 1) * 8 * V + 8 * i) = make_float2(S[i][e], S[i][e + 1]);
   }
+  if (abort_flag) {
+    // a wait gave up: give copies that may still be in flight time to land before the CTA exits
+    for (int i = 0; i < 64; ++i) __nanosleep(2000);
+  }
 }
 
 // ----------------------------------------------------------------------------- outputs
@@ -772,14 +790,16 @@ __host__ __device__ inline int delta_output_smem(int K, int V) {
 // grid (chunks of the round, H, B); warp w: tokens 16 (w % 4) .., values 32 (w / 4) ..
 template <int KT>
 __global__ void __launch_bounds__(DO_THREADS, 1) delta_output_kernel(const DeltaChunkArgs x) {
-  constexpr int K = KT * 16, RB = K * 2 + 16, K8 = K / 8;
+  constexpr int K = KT * 16, RB = K * 2 + 16;
   extern __shared__ __align__(16) uint8_t do_smem[];
+  __shared__ uint64_t full[2];
+  __shared__ volatile int abort_flag;
   pdl_launch_dependents();
   const DeltaArgs& a = x.a;
   const int b = blockIdx.z, h = blockIdx.y, chunk = x.chunk0 + blockIdx.x, c0 = chunk * DC;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3, mi = lane >> 3, r8 = lane & 7;
   const int q0 = a.query_start[b], n_all = a.query_start[b + 1] - q0, slot = a.slots[b];
-  const int V = a.V, V8 = V / 8, RV = V * 2 + 16;
+  const int V = a.V, RV = V * 2 + 16;
   pdl_wait();
   if (n_all < a.min_rows || n_all > a.max_rows || c0 >= n_all) return;
   const int n = min(DC, n_all - c0);
@@ -796,12 +816,18 @@ __global__ void __launch_bounds__(DO_THREADS, 1) delta_output_kernel(const Delta
   uint8_t* sp = ss + 2 * K * RV;           // [hi, lo][64][DC_PROW]
   uint8_t* su = sp + 2 * DC * DC_PROW;     // [hi, lo][64][RV]
   float* red = reinterpret_cast<float*>(su + 2 * DC * RV);  // [4][64]
-  for (int i = tid; i < 2 * DC * K8; i += DO_THREADS) cp_async16(sq + i / K8 * RB + i % K8 * 16, block + pl.qt + (size_t)i * 16);
-  for (int i = tid; i < 2 * K * V8; i += DO_THREADS) cp_async16(ss + i / V8 * RV + i % V8 * 16, block + pl.s + (size_t)i * 16);
-  cp_async_commit();
-  for (int i = tid; i < 2 * DC * 8; i += DO_THREADS) cp_async16(sp + i / 8 * DC_PROW + i % 8 * 16, block + pl.p + (size_t)i * 16);
-  for (int i = tid; i < 2 * DC * V8; i += DO_THREADS) cp_async16(su + i / V8 * RV + i % V8 * 16, block + pl.u + (size_t)i * 16);
-  cp_async_commit();
+  if (tid == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    abort_flag = 0;
+    mbar_fence_init();
+    const uint32_t first = 2 * DC * RB + 2 * K * RV, second = 2 * DC * DC_PROW + 2 * DC * RV;
+    mbar_expect_tx(&full[0], first);
+    bulk_load(do_smem, block + pl.qt, first, &full[0]);  // (q and the state lie behind each other, P and U as well)
+    mbar_expect_tx(&full[1], second);
+    bulk_load(sp, block + pl.p, second, &full[1]);
+  }
+  __syncthreads();
   const int mt = warp & 3, vn = (warp >> 2) * 32, nt = min(4, max(0, (V - vn) / 8));  // 8-value tiles of this warp (even)
   const __nv_bfloat16* z = reinterpret_cast<const __nv_bfloat16*>(a.z) + (size_t)(q0 + c0) * a.ld;
   // ---- gates, in the layout of the outputs
@@ -852,11 +878,11 @@ __global__ void __launch_bounds__(DO_THREADS, 1) delta_output_kernel(const Delta
       }
     }
   };
-  cp_async_wait<1>();
-  __syncthreads();
+  mbar_wait_bounded(&full[0], 0, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+  __syncwarp();
   product(smem_u32(sq), RB, DC * RB, smem_u32(ss), K * RV, KT);
-  cp_async_wait<0>();
-  __syncthreads();
+  mbar_wait_bounded(&full[1], 0, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+  __syncwarp();
   product(smem_u32(sp), DC_PROW, DC * DC_PROW, smem_u32(su), DC * RV, mt + 1);
   // ---- norm over the head's values: this warp's, then across the four warps of the same tokens
 #pragma unroll
