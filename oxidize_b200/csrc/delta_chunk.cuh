@@ -296,18 +296,7 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
     }
   }
   __syncthreads();
-  // logarithm of the decay from the chunk's start through token t, and behind token t through the end of block `block1` - 1, channels d
-  // and d + 1
-  auto since2 = [&](int t, int d) {
-    float2 v;
-    if (CH) v = *reinterpret_cast<const float2*>(sG + t * KF + d);
-    else v.x = v.y = sG[t];
-    for (int i = 0; i < t >> 4; ++i) {
-      v.x += total[CH ? i * K + d : i];
-      v.y += total[CH ? i * K + d + 1 : i];
-    }
-    return v;
-  };
+  // logarithm of the decay behind token t through the end of block `block1` - 1, channels d and d + 1
   auto until2 = [&](int t, int block1, int d) {
     float2 v, w;
     const int blk = t >> 4;
@@ -407,13 +396,42 @@ __global__ void __launch_bounds__(DP_THREADS, 1) delta_prepare_kernel(const Delt
 #pragma unroll 1
     for (int i = tid - 320; i < DC * K8; i += DP_THREADS - 320) {
       const int t = i / K8, p = i % K8;
-      float kv[8], qv[8], f[8], r[8], y[8];
+      float kv[8], qv[8], f[8], r[8], y[8], l[8];
       delta_load8(sK + t * KF + p * 8, kv);
       delta_load8(sQ + t * KF + p * 8, qv);
+      const int blk = t >> 4;
+      if (CH) {
+        delta_load8(sG + t * KF + p * 8, l);
 #pragma unroll
-      for (int e = 0; e < 8; e += 2) {
-        const float2 u = since2(t, p * 8 + e), w = until2(t, DC / 16, p * 8 + e);
-        f[e] = delta_exp2(u.x), f[e + 1] = delta_exp2(u.y), r[e] = delta_exp2(w.x), r[e + 1] = delta_exp2(w.y);
+        for (int e = 0; e < 8; ++e) {
+          f[e] = l[e];
+          r[e] = -l[e];
+        }
+#pragma unroll
+        for (int i = 0; i < DC / 16; ++i) {
+          delta_load8(total + i * K + p * 8, l);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            if (i < blk) f[e] += l[e];
+            else r[e] += l[e];
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          f[e] = delta_exp2(f[e]);
+          r[e] = delta_exp2(r[e]);
+        }
+      } else {
+        float u = sG[t], w = -u;
+#pragma unroll
+        for (int i = 0; i < DC / 16; ++i) {
+          if (i < blk) u += total[i];
+          else w += total[i];
+        }
+        u = delta_exp2(u);
+        w = delta_exp2(w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = u, r[e] = w;
       }
 #pragma unroll
       for (int e = 0; e < 8; ++e) y[e] = kv[e] * f[e];
