@@ -272,9 +272,9 @@ static __global__ void __launch_bounds__(256) delta_low_rank_kernel(const DeltaA
 
 // Steps of one row per sequence (decoding), taps <= 4 and 2 K + V <= CH * 512, 2 V <= 512: everything that does not come out of this step's
 // projections (state, ring, weights) is loaded ahead of the dependency, and what does in one go.  `low`: what
-// delta_low_rank_kernel left, or null without low-rank projections.  grid (H, B), threads as in
+// delta_low_rank_kernel left, or null without low-rank projections.  EXACT: the threads have all of the state's rows.  grid (H, B), threads as in
 // delta_step_kernel; dynamic shared memory: 3 K + 2 V + 2 R V floats.
-template <int NK, int CH>
+template <int NK, int CH, bool EXACT>
 __global__ void __launch_bounds__(512, NK <= 8 ? 2 : 1) delta_decode_kernel(const DeltaArgs a, const float* __restrict__ low) {
   constexpr int THREADS = 512, TAPS = 4;
   extern __shared__ __align__(16) float ds_smem[];
@@ -286,8 +286,8 @@ __global__ void __launch_bounds__(512, NK <= 8 ? 2 : 1) delta_decode_kernel(cons
     pdl_wait();
     return;
   }
-  const int K = a.K, V = a.V, cols = V >> 2, R = THREADS / cols, r = tid / cols, c = tid % cols;
-  const bool on = r < R;
+  const int V = a.V, cols = V >> 2, R = THREADS / cols, K = EXACT ? NK * R : a.K, r = tid / cols, c = tid % cols;
+  const bool on = EXACT || r < R;
   __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (size_t)q0 * a.ld_out + (size_t)h * V;
   if ((unsigned)slot >= (unsigned)a.num_slots) {
     if (slot >= 0 && tid == 0) oxb_report(OXB_BAD_SLOT, slot);
@@ -296,14 +296,15 @@ __global__ void __launch_bounds__(512, NK <= 8 ? 2 : 1) delta_decode_kernel(cons
     return;
   }
   float *sq = ds_smem, *sk = sq + K, *sg = sk + K, *sv = sg + K, *su = sv + V, *pa = su + V, *po = pa + R * V;
-  float4* S = reinterpret_cast<float4*>(a.state + ((size_t)slot * a.H + h) * K * V);
+  float4* S = reinterpret_cast<float4*>(a.state + ((size_t)slot * a.H + h) * K * V) + tid;  // (row r, column c: thread order)
+  const int step = R * cols;
   const int pos = a.seq_lens[b] - 1, C = 2 * a.G * K + a.H * V, tasks = 2 * K + V, taps = a.taps;
   float* ring = a.window + (size_t)slot * taps * C;
   float4 s[NK];
 #pragma unroll
   for (int i = 0; i < NK; ++i) {  // (written by an earlier step: no need to wait for this step's kernels)
     const int k = i * R + r;
-    s[i] = (on && k < K && pos > 0) ? S[(size_t)k * cols + c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    s[i] = (on && (EXACT || k < K) && pos > 0) ? S[i * step] : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   // this thread's channels: what the earlier rows of the ring give to the convolution, and the current row's weight
   float past[CH], w_now[CH];
@@ -361,7 +362,7 @@ __global__ void __launch_bounds__(512, NK <= 8 ? 2 : 1) delta_decode_kernel(cons
 #pragma unroll
     for (int i = 0; i < NK; ++i) {
       const int k = i * R + r;
-      if (k < K) {
+      if (EXACT || k < K) {
         const float g = sg[low_d ? k : 0], kv = sk[k] * ik, qv = sq[k] * iq;
         s[i] = make_float4(g * s[i].x, g * s[i].y, g * s[i].z, g * s[i].w);
         p.x = fmaf(kv, s[i].x, p.x);
@@ -393,9 +394,9 @@ __global__ void __launch_bounds__(512, NK <= 8 ? 2 : 1) delta_decode_kernel(cons
 #pragma unroll
     for (int i = 0; i < NK; ++i) {
       const int k = i * R + r;
-      if (k < K) {
+      if (EXACT || k < K) {
         const float kv = sk[k] * ik;
-        S[(size_t)k * cols + c] = make_float4(fmaf(kv, u.x, s[i].x), fmaf(kv, u.y, s[i].y), fmaf(kv, u.z, s[i].z), fmaf(kv, u.w, s[i].w));
+        S[i * step] = make_float4(fmaf(kv, u.x, s[i].x), fmaf(kv, u.y, s[i].y), fmaf(kv, u.z, s[i].z), fmaf(kv, u.w, s[i].w));
       }
     }
   }

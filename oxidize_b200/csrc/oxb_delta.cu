@@ -30,7 +30,9 @@ static int delta_step_launch(const DeltaArgs& a, int B, cudaStream_t stream) {
 template <int NK, int CH>
 static int delta_decode_go(const DeltaArgs& a, int B, const float* low, cudaStream_t stream) {
   const int R = 512 / (a.V / 4);
-  oxb_launch(delta_decode_kernel<NK, CH>, dim3(a.H, B), dim3(512), (size_t)(3 * a.K + 2 * a.V + 2 * R * a.V) * sizeof(float), stream, a, low);
+  const size_t smem = (size_t)(3 * a.K + 2 * a.V + 2 * R * a.V) * sizeof(float);
+  if (512 % (a.V / 4) == 0 && a.K == NK * R) oxb_launch(delta_decode_kernel<NK, CH, true>, dim3(a.H, B), dim3(512), smem, stream, a, low);
+  else oxb_launch(delta_decode_kernel<NK, CH, false>, dim3(a.H, B), dim3(512), smem, stream, a, low);
   OXB_CHECK_LAUNCH();
   return 0;
 }
