@@ -29,14 +29,14 @@ def pavatar(width: int, heads: int):
     from oxidize_b200.models.layered import layered_config
 
     half = heads // 2
-    moe = MoESpec(EXPERTS, TOP, FeedForwardSpec(expert_size(width), "relu2"), expert_weights_scale=1.5, correction=True)
+    moe = MoESpec(EXPERTS, TOP, FeedForwardSpec(expert_size(width), "relu2"), expert_weights_scale=2.0, correction=True)
     att = AttentionSpec(heads, max(1, heads // 4), DIM, DIM, DIM ** -0.5, None, bias=True, temp_coef=0.1, temp_every=8192.0, v_mix=True,
                         gate="head")
     par = ParallelSpec(AttentionSpec(half, max(1, half // 4), DIM, DIM, DIM ** -0.5, RotarySpec(DIM, 1e6), qk_norm="head", gate="value"),
                        DeltaSpec(half, half, DIM, DIM, 4, RANK, RANK), 0.5, 0.5, norms=True)
     kinds = [DeltaSpec(heads, half, DIM, DIM, 4), att, par, att]
     cfg = layered_config("pavatar", VOCAB, width, [LayerSpec(kinds[i % 4], moe) for i in range(LAYERS)], 1e-5, "rms", norm_placement="parallel")
-    cfg.embedding_scale, cfg.final_softcap, cfg.tie_embeddings = 16.0, 30.0, True
+    cfg.embedding_scale, cfg.final_softcap, cfg.tie_embeddings = 8.0, 50.0, True
     return cfg
 
 

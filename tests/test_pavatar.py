@@ -37,9 +37,9 @@ CONFIGS = {
         (plain.attn(5, 1, 33, 5, (0.3, 2.5)), None)], eps=1e-3, embed_scale=1.0, softcap=5.0),
     # wide heads
     "wide": plain.config(128, 90, [
-        (plain.parallel(plain.rotated(8, 2, 96, 128, rot(64, 3e4), 0.1), plain.dlt(2, 2, 128, 128, 4)), plain.moe(8, 2, 64, 1.5)),
-        (plain.attn(4, 2, 128, 96, (0.1, 64), True, 0.08), plain.moe(8, 2, 64, 1.5)),
-        (plain.dlt(4, 1, 96, 112, 4), plain.moe(8, 2, 64, 1.5)),
+        (plain.parallel(plain.rotated(8, 2, 96, 128, rot(64, 3e4), 0.1), plain.dlt(2, 2, 128, 128, 4)), plain.moe(8, 2, 64, 1.3)),
+        (plain.attn(4, 2, 128, 96, (0.1, 64), True, 0.08), plain.moe(8, 2, 64, 1.3)),
+        (plain.dlt(4, 1, 96, 112, 4), plain.moe(8, 2, 64, 1.3)),
         (plain.attn(4, 2, 128, 96, (0.1, 64), True, 0.08), None)], embed_scale=11.3),
 }
 
