@@ -284,6 +284,5 @@ def test_trace_program(model_dirs, tmp_path, dtype):
     assert [l for l in r.stdout.splitlines() if l.startswith("done")] == [f"done {i}" for i in range(4)]
     assert sorted(os.listdir(tmp_path)) == ["0.f32", "1.f32", "3.f32"]
     lg = {"a": oracle("wide", a)[1], "b": oracle("wide", b)[1]}
-    for s, rows in want.items():
-        got = torch.from_numpy(np.fromfile(tmp_path / f"{s}.f32", dtype="<f4").reshape(len(rows), -1))
-        check(got, np.stack([lg[i][p] for i, p in rows]), dtype, f"step {s}")
+    got = [torch.from_numpy(np.fromfile(tmp_path / f"{s}.f32", dtype="<f4").reshape(len(rows), -1)) for s, rows in want.items()]
+    check(torch.cat(got), np.stack([lg[i][p] for rows in want.values() for i, p in rows]), dtype)
