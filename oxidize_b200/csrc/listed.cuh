@@ -27,6 +27,10 @@ struct HeadPrepArgs {
   const void* v_first;  // values that are mixed into this layer's, rows ld_first apart, heads first_width apart; or null
   int ld_first, first_width, v_dim;
   const float* v_mix;   // [1]: their share
+  int unit;             // 1: queries and keys over their root mean square per head, without a weight
+  // 1: there are no values; the cache has one row per key head, [blocks, G, page, width + tail], the key as projected and behind
+  // it the float that turns it into the normed key
+  int shared, tail;
 };
 
 constexpr int HEAD_PREP_WARPS = 8;
@@ -109,10 +113,10 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int W = a.width, d0 = lane * VPL;
   const T* z = reinterpret_cast<const T*>(a.z) + (size_t)t * a.ld;
-  const bool norm = a.q_norm != nullptr, on = d0 < W;
-  const int h0 = blockIdx.y * a.per_cta, h1 = min(h0 + a.per_cta, a.H + 2 * a.G);
+  const bool norm = a.unit || a.q_norm != nullptr, on = d0 < W;
+  const int h0 = blockIdx.y * a.per_cta, h1 = min(h0 + a.per_cta, a.H + (a.shared ? 1 : 2) * a.G);
   float inv_q = 0.f, inv_k = 0.f;
-  if (norm && a.full && h0 < a.H + a.G) {
+  if (norm && !a.unit && a.full && h0 < a.H + a.G) {
     float sq = 0.f, sk = 0.f;
     const int f0 = h0 < a.H ? 0 : a.H, f1 = h1 > a.H ? a.H + a.G : a.H;
 #pragma unroll 4
@@ -144,19 +148,26 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
 #pragma unroll
     for (int j = 0; j < VPL; ++j) v[j] = 0.f;
     if (on) head_load<VPL>(z + (size_t)h * W + d0, v);
+    float inv = is_q ? inv_q : inv_k;
     if (!is_v) {
       if (norm) {
-        float inv = is_q ? inv_q : inv_k;
-        if (!a.full) {
+        if (a.unit || !a.full) {
           float s = 0.f;
 #pragma unroll
           for (int j = 0; j < VPL; ++j) s += v[j] * v[j];
           inv = rsqrtf(warp_sum(s) / (float)a.dim + a.eps);
         }
-        const float* w = (is_q ? a.q_norm : a.k_norm) + (a.full ? (size_t)(is_q ? h : h - a.H) * W : 0);
-        if (on) {
+        if (a.unit) {
+          if (!a.shared || is_q) {
 #pragma unroll
-          for (int j = 0; j < VPL; ++j) v[j] *= inv * w[d0 + j];
+            for (int j = 0; j < VPL; ++j) v[j] *= inv;
+          }
+        } else {
+          const float* w = (is_q ? a.q_norm : a.k_norm) + (a.full ? (size_t)(is_q ? h : h - a.H) * W : 0);
+          if (on) {
+#pragma unroll
+            for (int j = 0; j < VPL; ++j) v[j] *= inv * w[d0 + j];
+          }
         }
       }
       if (on && d0 < a.rot) head_store<VPL>(row + d0, v);
@@ -179,6 +190,9 @@ __global__ void __launch_bounds__(HEAD_PREP_WARPS * 32) head_prep_kernel(const H
     T* dst;
     if (is_q) {
       dst = reinterpret_cast<T*>(a.q) + ((size_t)t * a.H + h) * W;
+    } else if (a.shared) {
+      dst = reinterpret_cast<T*>(a.cache) + (((size_t)blk * a.G + h - a.H) * a.page + off) * (W + a.tail);
+      if (lane == 0) *reinterpret_cast<float*>(dst + W) = inv;
     } else {
       const int g = is_v ? h - a.H - a.G : h - a.H;
       dst = reinterpret_cast<T*>(a.cache) + ((((size_t)blk * a.G + g) * 2 + is_v) * a.page + off) * W;

@@ -24,10 +24,20 @@ OXB_API int oxb_joint_norm(const float* res, const void* y0, const void* y1, con
   return dtype == 0 ? joint_norm_launch<float>(a, T, stream) : joint_norm_launch<__nv_bfloat16>(a, T, stream);
 }
 
+OXB_API int oxb_add_normed(const float* res, const void* y, int ldy, const int* index, const float* weights, int k, const float* w,
+                           int groups, float eps, const float* first, float* results, int n, const float* depth, float* x_out,
+                           void* a_out, int dtype, int T, int H, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (groups <= 0 || H <= 0 || (depth != nullptr && (first == nullptr || results == nullptr || n < 0 || y == nullptr)))
+    return (int)cudaErrorInvalidValue;
+  const AddNormedArgs a{res, y, index, weights, k, ldy, w, groups, eps, first, results, (size_t)T * H, n, depth, x_out, a_out, H};
+  return dtype == 0 ? add_normed_launch<float>(a, T, stream) : add_normed_launch<__nv_bfloat16>(a, T, stream);
+}
+
 template <typename T>
 static int head_prep_launch(HeadPrepArgs a, int rows, cudaStream_t stream) {
   // few tokens: their heads are spread over CTAs, a head per warp
-  const int heads = a.H + 2 * a.G, groups = (heads + HEAD_PREP_WARPS - 1) / HEAD_PREP_WARPS;
+  const int heads = a.H + (a.shared ? 1 : 2) * a.G, groups = (heads + HEAD_PREP_WARPS - 1) / HEAD_PREP_WARPS;
   const int split = rows * groups <= 4 * oxb_sm_count() ? groups : 1;
   a.per_cta = (heads + split - 1) / split;
   const dim3 grid(rows, split), block(HEAD_PREP_WARPS * 32);
@@ -46,13 +56,14 @@ static int head_prep_launch(HeadPrepArgs a, int rows, cudaStream_t stream) {
 OXB_API int oxb_head_prep(const void* z, int ld, int dtype, const int* positions, const int* slots, const float* cos_sin, int max_pos,
                           int rot, int pairing, const float* q_norm, const float* k_norm, int full, float eps, int T, int H, int G,
                           int dim, int width, void* q, void* cache, int page, int num_blocks, float temp_coef, float temp_every,
-                          const void* v_first, int ld_first, int first_width, int v_dim, const float* v_mix, cudaStream_t stream) {
+                          const void* v_first, int ld_first, int first_width, int v_dim, const float* v_mix, int unit, int shared,
+                          int tail, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (rot < 0 || rot % 2 != 0 || rot > width || width % 32 != 0 || page <= 0 || H <= 0 || G <= 0 || (temp_coef != 0.f && !(temp_every > 0.f)) ||
+  if (rot < 0 || rot % 2 != 0 || rot > width || width % 32 != 0 || page <= 0 || H <= 0 || G <= 0 || (temp_coef != 0.f && !(temp_every > 0.f)) || (shared && (!unit || tail * (dtype == 0 ? 4 : 2) < 4)) ||
       (v_first != nullptr && (v_mix == nullptr || v_dim > first_width)))
     return (int)cudaErrorInvalidValue;
   const HeadPrepArgs a{z, ld, positions, slots, cos_sin, max_pos, rot, pairing, q_norm, k_norm, full, eps, H, G, dim, width,
-                       q, cache, page, num_blocks, 0, temp_coef, temp_every, v_first, ld_first, first_width, v_dim, v_mix};
+                       q, cache, page, num_blocks, 0, temp_coef, temp_every, v_first, ld_first, first_width, v_dim, v_mix, unit, shared, tail};
   return dtype == 0 ? head_prep_launch<float>(a, T, stream) : head_prep_launch<__nv_bfloat16>(a, T, stream);
 }
 

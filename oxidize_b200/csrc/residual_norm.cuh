@@ -383,6 +383,184 @@ int joint_norm_launch(const JointNormArgs& a, int T, cudaStream_t stream) {
   return 0;
 }
 
+// A branch's output joins the stream through an RMS norm in groups, x = res + norm(y) w, every one of `groups` consecutive parts
+// over its own root mean square; y may be the weighted sum of routed rows, sum_j weights[t, j] y[index[t, j]].  With `depth`, x
+// becomes the n-th of the kept results and what goes on is depth[0] first + sum_(j < n) depth[j + 1] results[j] + depth[n + 1] x.
+// Without a branch (y null): a = norm(res) w.
+struct AddNormedArgs {
+  const float* res;     // [T, H]
+  const void* y;        // [T, H] in the activation type, or rows ldy apart with index; or null
+  const int* index;     // [T, k] or null; < 0: none
+  const float* weights; // [T, k]
+  int k, ldy;
+  const float* w;       // [H]
+  int groups;
+  float eps;
+  const float* first;   // [T, H]
+  float* results;       // [n + 1, T, H]
+  size_t step;          // T * H
+  int n;
+  const float* depth;   // [n + 2] or null
+  float* x_out;         // [T, H] or null
+  void* a_out;          // [T, H] in the activation type, or null
+  int H;
+};
+
+// One CTA per row; every thread owns CH groups of four neighbouring values (H <= 4 * CH * threads); a part is a multiple of 128
+// values, so that a warp's values lie in one part.
+template <typename A, int CH>
+__global__ void __launch_bounds__(1024) add_normed_kernel(const AddNormedArgs a) {
+  __shared__ float part[128];  // sums of 128 values each
+  const int H4 = a.H >> 2, t = blockIdx.x, lane = threadIdx.x & 31;
+  const size_t base = (size_t)t * a.H;
+  float4 y[CH], w[CH];
+  pdl_launch_dependents();
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {  // weights are static: fetched ahead of the dependency
+    const int i = threadIdx.x + c * blockDim.x;
+    w[c] = y[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < H4) w[c] = rn_load4(a.w + 4 * i);
+  }
+  pdl_wait();
+  float4 v[CH];
+  const A* yp = reinterpret_cast<const A*>(a.y);
+  const int k = a.index != nullptr ? a.k : 1;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    v[c] = i < H4 ? rn_load4(a.res + base + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (yp == nullptr) y[c] = v[c];
+  }
+  for (int j = 0; j < k && yp != nullptr; ++j) {
+    const int r = a.index != nullptr ? a.index[(size_t)t * k + j] : t;
+    if (r < 0) continue;
+    const float g = a.index != nullptr ? a.weights[(size_t)t * k + j] : 1.f;
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int i = threadIdx.x + c * blockDim.x;
+      if (i < H4) {
+        const float4 f = rn_load4(yp + (size_t)r * a.ldy + 4 * i);
+        y[c] = make_float4(fmaf(g, f.x, y[c].x), fmaf(g, f.y, y[c].y), fmaf(g, f.z, y[c].z), fmaf(g, f.w, y[c].w));
+      }
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    const float ss = warp_sum((y[c].x * y[c].x + y[c].y * y[c].y) + (y[c].z * y[c].z + y[c].w * y[c].w));
+    if (lane == 0 && i < H4) part[i >> 5] = ss;
+  }
+  __syncthreads();
+  const int per = a.H / a.groups;  // values of a part
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    if (i >= H4) continue;
+    const int g0 = 4 * i / per * (per >> 7);
+    float ss = 0.f;
+    for (int j = 0; j < per >> 7; ++j) ss += part[g0 + j];
+    const float inv = rsqrtf(ss / (float)per + a.eps);
+    y[c] = make_float4(y[c].x * inv * w[c].x, y[c].y * inv * w[c].y, y[c].z * inv * w[c].z, y[c].w * inv * w[c].w);
+    if (yp == nullptr) v[c] = y[c];
+    else v[c] = make_float4(v[c].x + y[c].x, v[c].y + y[c].y, v[c].z + y[c].z, v[c].w + y[c].w);
+  }
+  if (a.depth != nullptr) {
+    const float d0 = a.depth[0], dn = a.depth[a.n + 1];
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int i = threadIdx.x + c * blockDim.x;
+      if (i >= H4) continue;
+      const float* row = a.results + base + 4 * i;
+      rn_store4(a.results + a.n * a.step + base + 4 * i, v[c]);
+      const float4 f = rn_load4(a.first + base + 4 * i);
+      float4 s = make_float4(d0 * f.x, d0 * f.y, d0 * f.z, d0 * f.w);
+#pragma unroll 8
+      for (int j = 0; j < a.n; ++j) {
+        const float4 r = rn_load4(row + j * a.step);
+        const float d = a.depth[j + 1];
+        s = make_float4(fmaf(d, r.x, s.x), fmaf(d, r.y, s.y), fmaf(d, r.z, s.z), fmaf(d, r.w, s.w));
+      }
+      v[c] = make_float4(fmaf(dn, v[c].x, s.x), fmaf(dn, v[c].y, s.y), fmaf(dn, v[c].z, s.z), fmaf(dn, v[c].w, s.w));
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = threadIdx.x + c * blockDim.x;
+    if (i >= H4) continue;
+    if (a.x_out != nullptr) rn_store4(a.x_out + base + 4 * i, v[c]);
+    if (a.a_out != nullptr) rn_store4(reinterpret_cast<A*>(a.a_out) + base + 4 * i, v[c]);
+  }
+}
+
+// Any width and part: the row is staged in shared memory (dynamic, H + groups floats).
+template <typename A>
+__global__ void __launch_bounds__(256) add_normed_any_kernel(const AddNormedArgs a) {
+  extern __shared__ float rn_row[];
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, per = a.H / a.groups;
+  const size_t base = (size_t)t * a.H;
+  const A* y = reinterpret_cast<const A*>(a.y);
+  float* inv = rn_row + a.H;
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    float v = 0.f;
+    if (y == nullptr) v = a.res[base + i];
+    else if (a.index == nullptr) v = rn_load(y + (size_t)t * a.ldy + i);
+    else
+      for (int j = 0; j < a.k; ++j) {
+        const int r = a.index[(size_t)t * a.k + j];
+        if (r >= 0) v = fmaf(a.weights[(size_t)t * a.k + j], rn_load(y + (size_t)r * a.ldy + i), v);
+      }
+    rn_row[i] = v;
+  }
+  __syncthreads();
+  if (a.groups >= 8) {
+    for (int g = warp; g < a.groups; g += blockDim.x >> 5) {
+      float ss = 0.f;
+      for (int i = lane; i < per; i += 32) ss += rn_row[g * per + i] * rn_row[g * per + i];
+      ss = warp_sum(ss);
+      if (lane == 0) inv[g] = rsqrtf(ss / (float)per + a.eps);
+    }
+  } else {
+    for (int g = 0; g < a.groups; ++g) {
+      float ss = 0.f;
+      for (int i = threadIdx.x; i < per; i += blockDim.x) ss += rn_row[g * per + i] * rn_row[g * per + i];
+      ss = block_sum(ss, red);
+      if (threadIdx.x == 0) inv[g] = rsqrtf(ss / (float)per + a.eps);
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < a.H; i += blockDim.x) {
+    float v = rn_row[i] * inv[i / per] * a.w[i];
+    if (y != nullptr) v += a.res[base + i];
+    if (a.depth != nullptr) {
+      a.results[a.n * a.step + base + i] = v;
+      float s = a.depth[0] * a.first[base + i];
+      for (int j = 0; j < a.n; ++j) s = fmaf(a.depth[j + 1], a.results[j * a.step + base + i], s);
+      v = fmaf(a.depth[a.n + 1], v, s);
+    }
+    if (a.x_out != nullptr) a.x_out[base + i] = v;
+    if (a.a_out != nullptr) rn_store(reinterpret_cast<A*>(a.a_out) + base + i, v);
+  }
+}
+
+template <typename A>
+int add_normed_launch(const AddNormedArgs& a, int T, cudaStream_t stream) {
+  if (a.H % a.groups == 0 && (a.H / a.groups) % 128 == 0 && a.ldy % 4 == 0 && a.H <= 16384) {
+    const int H4 = a.H / 4, lim = T >= 512 ? 256 : 1024, ch = H4 <= lim ? 1 : (H4 <= 2 * lim ? 2 : 4);
+    const int threads = ((H4 + ch - 1) / ch + 31) / 32 * 32;
+    if (ch == 1) oxb_launch(add_normed_kernel<A, 1>, dim3(T), dim3(threads), 0, stream, a);
+    else if (ch == 2) oxb_launch(add_normed_kernel<A, 2>, dim3(T), dim3(threads), 0, stream, a);
+    else oxb_launch(add_normed_kernel<A, 4>, dim3(T), dim3(threads), 0, stream, a);
+  } else {
+    if (a.H % a.groups != 0 || a.H + a.groups > 12 * 1024) return (int)cudaErrorInvalidValue;  // 48 KB of shared memory
+    oxb_launch(add_normed_any_kernel<A>, dim3(T), dim3(256), (size_t)(a.H + a.groups) * sizeof(float), stream, a);
+  }
+  OXB_CHECK_LAUNCH();
+  return 0;
+}
+
 template <typename A>
 int branch_norm_launch(const BranchNormArgs& a, int T, cudaStream_t stream) {
   if (a.H % 4 == 0 && a.H <= 16384) {

@@ -116,7 +116,8 @@ class LLM:
         self.pool = make_block_pool(nblocks, c.kv_page_size, prefix_cache)
         # a window that applies to every layer lets the scheduler hand pages back as they fall out of it
         self.scheduler = Scheduler(SchedulerConfig(c.max_num_batched_tokens, c.prefill_chunk_size, c.max_num_seqs,
-                                                   c.policy, prefix_cache, c.max_model_len, self.cfg.uniform_window), self.pool,
+                                                   c.policy, prefix_cache, c.max_model_len, self.cfg.uniform_window,
+                                                   self.cfg.kept_first), self.pool,
                                    StateSlots(c.max_num_seqs) if self.kv.states is not None else None)
         self.runner = ModelRunner(self.model, self.kv, max(c.max_num_batched_tokens, c.max_num_seqs), c.max_num_seqs,
                                   c.max_model_len, c.cuda_graphs and not _profiler.PROFILE and not _profiler.TRACE_FWD

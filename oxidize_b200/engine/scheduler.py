@@ -44,6 +44,7 @@ class SchedulerConfig:
     # next query are handed back to the pool while the sequence runs (the reference keeps a ring of `window` rows per layer,
     # oxidize-core/src/compute/kv_cache/cache.rs; with pages the ring becomes "free what fell out of the window")
     attention_window: int = 0
+    kept_first: int = 0  # leading positions that stay visible all the same: their pages are never handed back
 
 
 class Sequence:
@@ -165,7 +166,8 @@ class Scheduler:
 
     def _give_back(self, seq: Sequence) -> None:
         """What a sequence holds in the cache and the state store."""
-        self.pool.release_all(seq.blocks[seq._released:])
+        kept = min(-(-self.config.kept_first // self.pool.page_size), seq._released)
+        self.pool.release_all(seq.blocks[:kept] + seq.blocks[seq._released:])
         seq.blocks, seq._released = [], 0
         if seq.state_slot >= 0:
             self.slots.release(seq.state_slot)
@@ -412,15 +414,18 @@ class Scheduler:
 
     def _release_outside_window(self, seq: Sequence) -> None:
         """Return the pages no later query of ``seq`` can see: the next query sits at position ``num_computed`` and sees
-        keys at positions > num_computed - window, so a page whose last position is <= num_computed - window is dead."""
+        keys at positions > num_computed - window, so a page whose last position is <= num_computed - window is dead (unless it
+        holds one of the first positions that every query sees)."""
         ps = self.pool.page_size
+        kept = -(-self.config.kept_first // ps)
         dead = min(max(0, (seq.num_computed - self.config.attention_window) // ps), len(seq.blocks) - 1)
-        if dead <= seq._released:
+        first = max(seq._released, kept)
+        if dead <= first:
             return
         keep = seq.blocks[dead]
-        for i in range(seq._released, dead):
+        for i in range(first, dead):
             self.pool.release(seq.blocks[i])  # a page published to the prefix cache stays findable there until evicted
-        seq.blocks[:dead] = [keep] * dead  # every dead slot names a page this sequence still owns
+        seq.blocks[kept:dead] = [keep] * (dead - kept)  # every dead slot names a page this sequence still owns
         seq._released = dead
 
     def _trim_blocks(self, seq: Sequence) -> None:

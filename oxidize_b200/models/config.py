@@ -9,6 +9,7 @@ one (``:425-428``), and the architecture string selects routing / norm conventio
 from __future__ import annotations
 
 import dataclasses
+import math
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Tuple, Union
 
@@ -127,8 +128,20 @@ class LatentAttentionSpec:
 HEAD_WIDTHS = (32, 64, 96, 128, 192, 256)
 
 
+ROW_TAIL = 8  # values behind a cached row that serves as key and value
+
+
 def pad_to(n: int, unit: int) -> int:
     return (n + unit - 1) // unit * unit
+
+
+def distance_bucket(n: int, rows: int, far: float) -> int:
+    """Row of a table of ``rows`` biases for a key ``n`` positions back: its own below half of the table, from there on in
+    logarithmic steps that end at ``far``."""
+    half = rows // 2
+    if n < half:
+        return n
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half)))
 
 
 @dataclass
@@ -142,7 +155,13 @@ class AttentionSpec:
     ``v_mix``: the values are mixed, v <- (1 - lambda) v + lambda v_first, with those that the first such layer of the model
     has for the same token (lambda is a weight of the layer; the first layer's values stay as they are).  ``gate``: the
     outputs are multiplied by the sigmoid of a projection of the layer's input, one value per ``head`` or per output
-    ``value``.  ``bias``: the q, k and v projections have one."""
+    ``value``.  ``bias``: the q, k and v projections have one.
+
+    ``keep_first``: a windowed query also sees the first that many positions.  ``softcap`` > 0: scaled scores become
+    softcap * tanh(score / softcap).  ``bias_rows`` > 0: a learned bias per distance bucket and head is added to them
+    (:func:`distance_bucket`, logarithmic up to ``bias_max``).  ``talk``: the scores are then mixed over the heads by a learned
+    matrix.  ``unit_sink``: one is added to the softmax denominator.  ``shared_kv``: there is no value projection; the values are
+    the keys as projected (ahead of their norm)."""
 
     heads: int
     kv_heads: int
@@ -152,14 +171,27 @@ class AttentionSpec:
     rotary: Optional[RotarySpec]
     window: int = 0
     sink: bool = False
-    qk_norm: str = ""  # "" | head | full
+    qk_norm: str = ""  # "" | unit (per head, without a weight) | head | full
     bias: bool = False
     temp_coef: float = 0.0
     temp_every: float = 1.0
     v_mix: bool = False
     gate: str = ""  # "" | head | value
+    keep_first: int = 0
+    softcap: float = 0.0
+    bias_rows: int = 0
+    bias_max: int = 0
+    talk: bool = False
+    unit_sink: bool = False
+    shared_kv: bool = False
 
     kv_from = None  # (every layer of this kind owns cache rows)
+
+    @property
+    def joint_scores(self) -> bool:
+        """The attention step works on the scores of all heads together (``ops.cuda_joint``): one cached row serves as key and
+        value, with one over the key's root mean square behind it."""
+        return self.shared_kv
 
     @property
     def width(self) -> int:
@@ -169,7 +201,8 @@ class AttentionSpec:
 
     @property
     def cache_shape(self) -> Tuple[int, int, int]:
-        return self.kv_heads, 2, self.width
+        # (a shared row ends in 16 bytes or more of which the first four hold the factor that makes it a key)
+        return (self.kv_heads, 1, self.width + ROW_TAIL) if self.shared_kv else (self.kv_heads, 2, self.width)
 
     @property
     def out_dim(self) -> int:
@@ -177,7 +210,7 @@ class AttentionSpec:
 
     @property
     def qkv_dim(self) -> int:
-        return (self.heads + 2 * self.kv_heads) * self.width
+        return (self.heads + (1 if self.shared_kv else 2) * self.kv_heads) * self.width
 
     @property
     def gate_dim(self) -> int:
@@ -286,6 +319,51 @@ class DeltaSpec:
 
 
 @dataclass
+class WkvSpec:
+    """RWKV time mixing: five mixes of a token's input with the one ahead of it feed r, k, v, a silu gate and the decay
+    w = exp(-exp(W_2 tanh(W_1 x) + w_0)), one per head and key channel (``rank``: of those two projections);
+    o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t with a learned bonus u for the current token, S_t = diag(w_t) S_(t-1) + k_t v_t^T.
+    Each head's o is divided by its root mean square and weighted.  Every sequence carries one [dim, dim] float32 state per
+    head and its last input (``hidden`` values)."""
+
+    heads: int
+    dim: int
+    rank: int
+    hidden: int
+
+    rotary = None  # (positions enter through the recurrence alone)
+
+    # head widths in projections, state and outputs (the padding is zero)
+    @property
+    def k_width(self) -> int:
+        return next((w for w in HEAD_WIDTHS if w >= self.dim), pad_to(self.dim, 32))
+
+    v_width = k_width
+
+    @property
+    def state_shape(self) -> Tuple[int, int, int]:
+        return self.heads, self.k_width, self.v_width
+
+    @property
+    def window_shape(self) -> Tuple[int, int]:
+        """The last input of a sequence."""
+        return 1, self.hidden
+
+    @property
+    def out_dim(self) -> int:
+        return self.heads * self.v_width
+
+    @property
+    def decay_dim(self) -> int:
+        return pad_to(self.rank, 16)
+
+    @property
+    def proj_dim(self) -> int:
+        """Columns of the projections of the layer's input: r | k | v | gate."""
+        return 4 * self.out_dim
+
+
+@dataclass
 class ParallelSpec:
     """Attention and a recurrent mixer side by side on the same input: left_scale * left + right_scale * right; with
     ``norms`` each side's projected output first passes an RMS norm of its own."""
@@ -295,6 +373,9 @@ class ParallelSpec:
     left_scale: float = 1.0
     right_scale: float = 1.0
     norms: bool = False
+
+
+RECURRENT = (RetentionSpec, DeltaSpec, WkvSpec)
 
 
 @dataclass
@@ -314,7 +395,8 @@ class FeedForwardSpec:
 @dataclass
 class MoESpec:
     """Routed experts: the ``n_experts_used`` largest scores choose, the chosen scores divided by their sum weigh (with
-    softmax scores: the softmax over the chosen logits); ``correction`` adds a learned offset per expert to the scores that
+    softmax scores: the softmax over the chosen logits), or without ``expert_weights_norm`` the scores as they are;
+    ``correction`` adds a learned offset per expert to the scores that
     choose; ``shared`` runs for every token and is added.  (The routing fields carry the names that the routing operators read
     from ``ModelConfig``.)"""
 
@@ -339,7 +421,7 @@ class MoESpec:
 class LayerSpec:
     """One decoder layer of a model whose layers are listed one by one."""
 
-    mixer: Union[LatentAttentionSpec, AttentionSpec, RetentionSpec, DeltaSpec, ParallelSpec]
+    mixer: Union[LatentAttentionSpec, AttentionSpec, RetentionSpec, DeltaSpec, WkvSpec, ParallelSpec]
     ffn: Union[FeedForwardSpec, MoESpec, None] = None  # None: the layer has no feed-forward block
     weights_of: Optional[int] = None  # an earlier layer whose weights this one uses (with cache rows and state of its own)
 
@@ -347,13 +429,13 @@ class LayerSpec:
     def attention(self) -> Union[LatentAttentionSpec, AttentionSpec, None]:
         """The part of the mixer that attends over cached rows."""
         m = self.mixer
-        return m.left if isinstance(m, ParallelSpec) else None if isinstance(m, (RetentionSpec, DeltaSpec)) else m
+        return m.left if isinstance(m, ParallelSpec) else None if isinstance(m, RECURRENT) else m
 
     @property
-    def recurrent(self) -> Union[RetentionSpec, DeltaSpec, None]:
+    def recurrent(self) -> Union[RetentionSpec, DeltaSpec, WkvSpec, None]:
         """The part of the mixer that carries a recurrent state."""
         m = self.mixer
-        return m.right if isinstance(m, ParallelSpec) else m if isinstance(m, (RetentionSpec, DeltaSpec)) else None
+        return m.right if isinstance(m, ParallelSpec) else m if isinstance(m, RECURRENT) else None
 
     @property
     def retention(self) -> Optional[RetentionSpec]:
@@ -364,6 +446,11 @@ class LayerSpec:
     def delta(self) -> Optional[DeltaSpec]:
         r = self.recurrent
         return r if isinstance(r, DeltaSpec) else None
+
+    @property
+    def wkv(self) -> Optional[WkvSpec]:
+        r = self.recurrent
+        return r if isinstance(r, WkvSpec) else None
 
     @property
     def owns_rows(self) -> bool:
@@ -473,8 +560,12 @@ class ModelConfig:
     residual_alpha: float = 0.0
     # Listed layers only: "after_sum" (the rule above); "sandwich": norms on both sides of the branch,
     # x <- x + norm_b(branch(norm_a(x))); "parallel": one norm that both branches read, x <- x + mixer(h) + ffn(h) with
-    # h = norm(x).  The residual stream is in float32 in all three
+    # h = norm(x); "output": a norm on the branch's output only, x <- x + norm(branch(x)).  The residual stream is in float32
+    # in all of them
     norm_placement: str = "after_sum"
+    norm_groups: int = 1  # an RMS norm divides this many equal consecutive parts of a row by their own root mean squares
+    # what a layer hands on is a learned weighted sum of the embedding and the results of all layers so far
+    depth_average: bool = False
     embed_norm: bool = False  # the embedding passes a norm of its own
 
     @property
@@ -516,6 +607,11 @@ class ModelConfig:
             ws = [l.attention.window for l in self.layer_specs if l.attention is not None]
             return max(ws) if ws and min(ws) > 0 else 0
         return self.sliding_window if (self.sliding_window > 0 and self.sliding_window_pattern == 0) else 0
+
+    @property
+    def kept_first(self) -> int:
+        """Leading positions that windowed layers go on seeing."""
+        return max((getattr(l.attention, "keep_first", 0) for l in self.layer_specs if l.attention is not None), default=0)
 
     @property
     def is_ssm(self) -> bool:
@@ -584,9 +680,11 @@ class ModelConfig:
                 n += a.heads * (h * (a.qk_dim + a.v_dim) + a.kv_rank * (a.nope_dim + a.v_dim))
                 n += 0 if a.kv_from is not None else h * (a.kv_rank + a.rope_dim) + a.kv_rank
             elif a is not None:
-                n += h * (a.heads + a.kv_heads) * (a.dim + a.v_dim)
-                n += {"": 0, "head": 2, "full": a.heads + a.kv_heads}[a.qk_norm] * a.dim
-                n += ((a.heads + a.kv_heads) * a.dim + a.kv_heads * a.v_dim if a.bias else 0) + a.v_mix
+                values = 0 if a.shared_kv else a.kv_heads * a.v_dim
+                n += h * ((a.heads + a.kv_heads) * a.dim + values + a.heads * a.v_dim)
+                n += {"": 0, "unit": 0, "head": 2, "full": a.heads + a.kv_heads}[a.qk_norm] * a.dim
+                n += ((a.heads + a.kv_heads) * a.dim + values if a.bias else 0) + a.v_mix
+                n += a.bias_rows * a.heads + (a.heads ** 2 if a.talk else 0)
                 n += {"": 0, "head": a.heads, "value": a.heads * a.v_dim}[a.gate] * h
             n += a.heads if a is not None and a.sink else 0
             n += h * r.heads * (2 * r.dim + 3 * r.v_dim) if r is not None else 0
@@ -595,7 +693,11 @@ class ModelConfig:
                 n += (2 * qk + v) * (h + d.conv) + h * (v + d.heads) + d.heads + d.v_dim
                 n += d.decay_rank * (h + d.heads * d.dim) + d.heads * d.dim if d.decay_rank else (h + 1) * d.heads
                 n += d.gate_rank * (h + v) if d.gate_rank else h * v
-        return n
+            k = l.wkv
+            if k is not None:
+                c = k.heads * k.dim
+                n += 5 * h + 5 * c * h + k.rank * (h + c) + 3 * c  # mixes; r, k, v, gate, output; decay; w_0, bonus, norm
+        return n + (sum(i + 2 for i in range(len(self.layer_specs))) if self.depth_average else 0)
 
     def to_dict(self) -> Dict[str, Any]:
         return dataclasses.asdict(self)

@@ -16,9 +16,16 @@ Pavatar: one RMS norm that mixer and feed-forward block both read, x <- x + mixe
 a query factor that grows with the position, values mixed with an earlier layer's, a gate per head), the gated delta rule with
 a decay per head, or rotated attention (q / k norms, a gate per output value) beside the gated delta rule with a decay per key
 channel, each side with a norm of its own; routed squared-relu experts with a correction of the choice; a scaled embedding that
-is the output head as well, and soft-capped logits."""
+is the output head as well, and soft-capped logits.
+
+Netovik: RMS norms in groups on the branches' outputs only, x <- x + norm(branch(x)), and after every layer a learned weighted
+sum of the embedding and all results so far; RWKV time mixing, or unrotated attention whose values are its keys (soft-capped
+scores, a bias by distance, scores mixed over the heads, a window with kept first tokens, one in the softmax denominator);
+gated feed-forward blocks, dense or routed with the scores as they are; a scaled embedding that is the output head as well."""
 from __future__ import annotations
 
+import dataclasses
+import functools
 import math
 from typing import Any, Callable, Dict, List, Optional, Tuple
 
@@ -27,9 +34,9 @@ import torch
 
 from ..formats.layered import LayeredCheckpoint
 from .config import (AttentionSpec, DeltaSpec, FeedForwardSpec, LatentAttentionSpec, LayerSpec, ModelConfig, MoESpec,
-                     ParallelSpec, RetentionSpec, RopeScaling, RotarySpec, UnsupportedArchitecture, pad_to)
+                     ParallelSpec, RetentionSpec, RopeScaling, RotarySpec, UnsupportedArchitecture, WkvSpec, distance_bucket, pad_to)
 from .weights import (DeltaWeights, ExpertWeights, LayerWeights, LinearWeight, MLAWeights, ModelWeights, QTensor,
-                      StreamedLayers, shard_range)
+                      StreamedLayers, WkvWeights, shard_range)
 
 
 # --------------------------------------------------------------------------- configuration
@@ -228,6 +235,52 @@ def _pavatar_config(ck: LayeredCheckpoint) -> ModelConfig:
     return cfg
 
 
+def _joint_attention(ck: LayeredCheckpoint, m: Dict[str, Any], prefix: str, layer: int) -> AttentionSpec:
+    """Unrotated attention whose heads' scores are mixed and whose values are the keys as projected."""
+    rows = int(ck.tensors[prefix + "rel"].shape[0])
+    a = _attention(dict(m, rot=None), "unit", False, layer, bias=True, keep_first=int((m.get("mask") or {}).get("keep_first") or 0),
+                   softcap=float(m.get("softcap") or 0.0), bias_rows=rows, bias_max=int(m["bias_max"]), talk=True, unit_sink=True,
+                   shared_kv=True)
+    if a.v_dim != a.dim:
+        raise UnsupportedArchitecture(f"layer {layer}: values of {a.v_dim} that are keys of {a.dim}")
+    if rows < 2 or rows % 2 or a.bias_max <= rows // 2:
+        raise UnsupportedArchitecture(f"layer {layer}: {rows} biases for distances up to {a.bias_max}")
+    return a
+
+
+def _wkv(ck: LayeredCheckpoint, m: Dict[str, Any], prefix: str, hidden: int) -> WkvSpec:
+    return WkvSpec(int(m["heads"]), int(m["dim"]), int(ck.tensors[prefix + "w1"].shape[0]), hidden)
+
+
+def _unnormed_experts(f: Optional[Dict[str, Any]], layer: int):
+    """Gated blocks; routed experts are weighed by their scores as they are."""
+    s = _gated_ffn(f, layer)
+    return dataclasses.replace(s, expert_weights_norm=False) if isinstance(s, MoESpec) else s
+
+
+def _netovik_config(ck: LayeredCheckpoint) -> ModelConfig:
+    c = ck.config
+    width, specs = int(c["width"]), []
+    for i, l in enumerate(c["layers"]):
+        p = f"l{i}.mix."
+        if l.get("type") == "attention":
+            mixer = _joint_attention(ck, l["mixer"], p, i)
+        elif l.get("type") == "wkv":
+            mixer = _wkv(ck, l["mixer"], p, width)
+        else:
+            raise UnsupportedArchitecture(f"layer {i}: mixer type {l.get('type')!r}")
+        specs.append(LayerSpec(mixer, _unnormed_experts(l.get("mlp"), i)))
+    cfg = layered_config("netovik", int(c["vocab"]), width, specs, eps=float(c["norm"]["eps"]), norm_kind="rms",
+                         norm_placement="output", name=str(ck.get("general.name", "")))
+    cfg.norm_groups = int(c["norm"].get("groups") or 1)
+    if cfg.norm_groups < 1 or width % cfg.norm_groups:
+        raise UnsupportedArchitecture(f"a norm over {cfg.norm_groups} parts of {width} values")
+    cfg.depth_average = True
+    cfg.embedding_scale = float((c.get("embedding") or {}).get("scale", 1.0))
+    cfg.tie_embeddings = True
+    return cfg
+
+
 def layered_config(arch: str, vocab: int, width: int, specs: List[LayerSpec], eps: float, norm_kind: str,
                    residual_alpha: float = 1.0, embed_norm: bool = False, name: str = "",
                    norm_placement: str = "after_sum") -> ModelConfig:
@@ -244,7 +297,7 @@ def layered_config(arch: str, vocab: int, width: int, specs: List[LayerSpec], ep
 
 
 READERS: Dict[str, Callable[[LayeredCheckpoint], ModelConfig]] = {"vefilix": _vefilix_config, "sokirax": _sokirax_config,
-                                                                      "pavatar": _pavatar_config}
+                                                                      "pavatar": _pavatar_config, "netovik": _netovik_config}
 
 
 def config_from_layered(ck: LayeredCheckpoint) -> ModelConfig:
@@ -339,6 +392,33 @@ def delta_weights(d: DeltaSpec, t: Dict[str, torch.Tensor], act_dtype: torch.dty
     return ins, w
 
 
+@functools.lru_cache(None)
+def distance_rows(rows: int, far: int) -> Tuple[int, ...]:
+    """Bias rows of the distances 0, 1, ... up to the first that has the last row (as have all beyond it)."""
+    out = [0]
+    while out[-1] < rows - 1:
+        out.append(distance_bucket(len(out), rows, far))
+    return tuple(out)
+
+
+def distance_bias(rel: torch.Tensor, far: int, mix: Optional[torch.Tensor]) -> torch.Tensor:
+    """Bias table [rows, heads] to [heads, distances], what every head's mixed score gets from it."""
+    t = rel.double()[torch.tensor(distance_rows(rel.shape[0], far), device=rel.device)].t()
+    return (t if mix is None else mix.double() @ t).float().contiguous()
+
+
+def wkv_weights(k: WkvSpec, t: Dict[str, torch.Tensor], act_dtype: torch.dtype) -> Dict[str, Any]:
+    """Time-mixing tensors (as stored) in the layout the forward pass uses."""
+    H, W = k.heads, k.k_width
+    pad, ld = lambda n: pad_heads(t[n].float().reshape(-1), H, W).contiguous(), pad_to(k.hidden, 8)
+    w = WkvWeights(mu=torch.stack([t["mu." + n].float().reshape(-1) for n in "rkvgw"]).contiguous(),
+                   proj=torch.stack([pad_cols(pad_heads(t[n], H, W), ld) for n in "rkvg"]).contiguous(),
+                   decay_down=LinearWeight([dense_qtensor(pad_cols(pad_rows(t["w1"], k.decay_dim), ld))]),
+                   decay_up=pad_cols(pad_heads(t["w2"], H, W), k.decay_dim).to(act_dtype), decay_base=pad("w0"), bonus=pad("u"),
+                   norm=pad("norm"))
+    return {"wqkv": None, "wo": LinearWeight([dense_qtensor(pad_heads(t["o"], H, W, dim=1).contiguous())]), "wkv": w}
+
+
 def listed_mixer(spec: LayerSpec, att: Dict[str, torch.Tensor], rec: Dict[str, torch.Tensor]) -> Dict[str, Any]:
     """Attention and / or recurrent tensors (as stored) of one layer in the layout the forward pass uses: one matrix over
     the layer's input, attention q | k | v | gate then retention q | k | v | gate or the delta rule's rows, and one output
@@ -348,20 +428,26 @@ def listed_mixer(spec: LayerSpec, att: Dict[str, torch.Tensor], rec: Dict[str, t
     a, r, d = spec.attention, spec.retention, spec.delta
     ret, bias = rec, None
     if a is not None:
-        for n, heads in (("q", a.heads), ("k", a.kv_heads), ("v", a.kv_heads)):
+        parts = (("q", a.heads), ("k", a.kv_heads)) + (() if a.shared_kv else (("v", a.kv_heads),))
+        for n, heads in parts:
             ins.append(pad_heads(att[n], heads, a.width))
         if a.gate:
             ins.append(pad_rows(att["g"], a.gate_dim) if a.gate == "head" else pad_heads(att["g"], a.heads, a.width))
         if a.bias:
-            bias = torch.cat([pad_heads(att[n + ".b"].float(), heads, a.width)
-                              for n, heads in (("q", a.heads), ("k", a.kv_heads), ("v", a.kv_heads))])
+            bias = torch.cat([pad_heads(att[n + ".b"].float(), heads, a.width) for n, heads in parts])
         kw["v_mix"] = att["vmix"].float().reshape(1).contiguous() if a.v_mix else None
         outs.append(pad_heads(att["o"], a.heads, a.width, dim=1))
-        if a.qk_norm:
+        if a.qk_norm in ("head", "full"):
             full = a.qk_norm == "full"
             kw["q_norm"] = pad_heads(att["q.norm"], a.heads if full else 1, a.width).contiguous()
             kw["k_norm"] = pad_heads(att["k.norm"], a.kv_heads if full else 1, a.width).contiguous()
         kw["sink"] = att["sink"] if a.sink else None
+        if a.unit_sink:
+            kw["sink"] = torch.zeros(a.heads, dtype=torch.float32, device=att["q"].device)
+        if a.talk:
+            kw["score_mix"] = att["talk"].float().reshape(a.heads, a.heads).contiguous()
+        if a.bias_rows:
+            kw["score_bias"] = distance_bias(att["rel"], a.bias_max, kw.get("score_mix"))
     if r is not None:
         for n, width in (("q", r.k_width), ("k", r.k_width), ("v", r.v_width), ("g", r.v_width)):
             ins.append(pad_heads(ret[n], r.heads, width))
@@ -427,15 +513,12 @@ def _load_listed(src: LayeredWeightSource, cfg: ModelConfig, i: int) -> LayerWei
     def triple(prefix: str):
         return tuple(src.dense(f"{p}.mlp.{prefix}{n}") for n in ("gate", "up", "down"))
 
+    gated_block(lw, f, cfg.hidden_size, triple)
     if isinstance(f, MoESpec):
         lw.router = src.matrix(f"{p}.mlp.router")
-        lw.experts = listed_experts(f, [triple(f"e{e}.") for e in range(f.n_experts)], cfg.hidden_size)
         if f.shared is not None:
             gu, down = gated_pair(*triple("shared."), f.shared.pad_size)
             lw.shared_gate_up, lw.shared_down = LinearWeight([gu]), LinearWeight([down])
-    else:
-        gu, down = gated_pair(*triple(""), f.pad_size)
-        lw.w_gate_up, lw.w_down = LinearWeight([gu]), LinearWeight([down])
     return lw
 
 
@@ -468,6 +551,36 @@ def _load_joint(src: LayeredWeightSource, cfg: ModelConfig, i: int) -> LayerWeig
     return lw
 
 
+def gated_block(lw: LayerWeights, f, hidden: int, triple) -> None:
+    """Feed-forward weights of a layer, dense or routed; ``triple(prefix)``: (gate, up, down) as stored."""
+    if isinstance(f, MoESpec):
+        lw.experts = listed_experts(f, [triple(f"e{e}.") for e in range(f.n_experts)], hidden)
+    else:
+        gu, down = gated_pair(*triple(""), f.pad_size)
+        lw.w_gate_up, lw.w_down = LinearWeight([gu]), LinearWeight([down])
+
+
+def _load_output_normed(src: LayeredWeightSource, cfg: ModelConfig, i: int) -> LayerWeights:
+    """A layer with norms on its branches' outputs only."""
+    spec, p = cfg.layer_specs[i], f"l{i}"
+    dense, vectors = lambda *names: {n: src.dense(f"{p}.mix.{n}") for n in names}, lambda *names: {n: src.vector(f"{p}.mix.{n}") for n in names}
+    a = spec.attention
+    if spec.wkv is not None:
+        kw = wkv_weights(spec.wkv, {**dense("r", "k", "v", "g", "w1", "w2", "o"), **vectors(*("mu." + n for n in "rkvgw"), "w0", "u", "norm")},
+                         src.act_dtype)
+    else:
+        att = {**dense("q", "k", "o"), **vectors("q.b", "k.b", "talk"), "rel": src.vector(f"{p}.mix.rel").reshape(a.bias_rows, a.heads)}
+        kw = listed_mixer(spec, att, {})
+    lw = LayerWeights(attn_norm=None, post_attn_norm=src.vector(f"{p}.norm1"), ffn_norm=None, **kw)
+    lw.depth = src.vector(f"{p}.dwa") if cfg.depth_average else None
+    if spec.ffn is not None:
+        lw.post_ffn_norm = src.vector(f"{p}.norm2")
+        if isinstance(spec.ffn, MoESpec):
+            lw.router = src.matrix(f"{p}.mlp.router")
+        gated_block(lw, spec.ffn, cfg.hidden_size, lambda prefix: tuple(src.dense(f"{p}.mlp.{prefix}{n}") for n in ("gate", "up", "down")))
+    return lw
+
+
 def _load_layer(src: LayeredWeightSource, spec: LayerSpec, i: int, tp_rank: int, tp_size: int) -> LayerWeights:
     p, m = f"l{i}", spec.mixer
     h0, h1 = shard_range(m.heads, tp_rank, tp_size)
@@ -493,7 +606,7 @@ def load_layered_weights(ck: LayeredCheckpoint, cfg: ModelConfig, device="cpu", 
     replicated (every rank caches the whole latent row)."""
     src = LayeredWeightSource(ck, device, act_dtype)
     n = cfg.n_layers
-    whole = {"sandwich": _load_listed, "parallel": _load_joint}.get(cfg.norm_placement)
+    whole = {"sandwich": _load_listed, "parallel": _load_joint, "output": _load_output_normed}.get(cfg.norm_placement)
     if whole is not None and tp_size > 1:
         raise ValueError("a norm over all heads and per-sequence states are not sharded: run this model with tp_size = 1")
 

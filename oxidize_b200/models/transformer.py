@@ -530,6 +530,27 @@ class Transformer:
                 self._layer_done(li, x, capture)
         return (x if mix is None else ops.joint_norm(x, mix, ffn, None, eps, self.act_dtype)[0]), None
 
+    def _layers_output_normed(self, h: torch.Tensor, meta: BatchMeta, kv, lo: int, hi: int, capture: Optional[dict]):
+        """Layers with norms on their branches' outputs only, x <- x + norm(branch(x)), the stream ``x`` in float32; what goes on
+        from a layer may be a weighted sum of the embedding and all results so far.  One kernel norms a branch's output (of
+        routed experts: their weighted sum), adds it and averages."""
+        cfg = self.cfg
+        norm = (cfg.norm_groups, cfg.rms_eps)
+        x, a = h.float(), None
+        streams = ops.DepthStreams(x, hi - lo) if cfg.depth_average else None
+        for li in range(lo, hi):
+            lw, spec = self.w.layers[li], cfg.layer_specs[self.w.first_layer + li]
+            if a is None and spec.attention is not None:
+                a = x.to(self.act_dtype)
+            res, y, w = x, self._listed_mixer(li, lw, spec, a, meta, kv, stream=x), lw.post_attn_norm
+            if spec.ffn is not None:
+                res, a = ops.add_normed(res, y, w, *norm, self.act_dtype)
+                y, w = self._listed_ffn(lw, spec.ffn, a, combine=False), lw.post_ffn_norm
+            wants = li + 1 < hi and cfg.layer_specs[self.w.first_layer + li + 1].attention is not None
+            x, a = ops.add_normed(res, y, w, *norm, self.act_dtype if wants else None, streams, lw.depth)
+            self._layer_done(li, x, capture)
+        return x, None
+
     def _layer_done(self, li: int, x: torch.Tensor, capture: Optional[dict]) -> None:
         gl = self.w.first_layer + li
         if capture is not None and gl in capture.get("layers", ()):
@@ -537,11 +558,16 @@ class Transformer:
         if _profiler.TRACE_FWD:
             _profiler.trace_hidden(gl, x, None)
 
-    def _listed_mixer(self, li: int, lw: LayerWeights, spec, xa: torch.Tensor, meta: BatchMeta, kv, carry: Optional[dict] = None):
+    def _listed_mixer(self, li: int, lw: LayerWeights, spec, xa: torch.Tensor, meta: BatchMeta, kv, carry: Optional[dict] = None,
+                      stream: Optional[torch.Tensor] = None):
         """The mixer branch of a listed layer: from its normed input to its output projection; with a norm on each side's
-        output, both projected outputs as ``ops.NormedPair``.  ``carry``: what this step's earlier layers left for it."""
+        output, both projected outputs as ``ops.NormedPair``.  ``carry``: what this step's earlier layers left for it;
+        ``stream``: the same input in float32, for mixers that read it unrounded."""
         eps = self.cfg.rms_eps
-        if lw.mla is not None:
+        if lw.wkv is not None:
+            n = self.state_index[li]
+            o = ops.wkv_mixer(stream, lw.wkv, spec.wkv, meta, kv.states.data[n], kv.states.windows[n], eps, self.act_dtype)
+        elif lw.mla is not None:
             o = ops.latent_mixer(xa, lw.mla, spec.mixer, self.layer_ropes[li][0], meta, kv, self.kv_index[li], eps)
         else:
             o = ops.listed_mixer(xa, lw, spec, self.layer_ropes[li], meta, kv, self.kv_index[li], self.state_index.get(li, -1), eps, carry)
@@ -561,6 +587,8 @@ class Transformer:
     def final_norm(self, h: torch.Tensor, residual: Optional[torch.Tensor]):
         """(normed rows for the output head, the hidden state in front of that norm)."""
         cfg = self.cfg
+        if cfg.norm_groups > 1:
+            return ops.grouped_norm(h, self.w.out_norm, cfg.norm_groups, cfg.rms_eps, self.act_dtype), h
         if cfg.is_layered:
             return ops.residual_norm(h, None, 1.0, self.w.out_norm, self.w.out_norm_bias, cfg.rms_eps, cfg.norm_kind,
                                      self.act_dtype, keep_stream=False)[1], h
@@ -695,8 +723,8 @@ class Transformer:
         cfg = self.cfg
         lo, hi = layers if layers is not None else (0, len(self.w.layers))
         if cfg.is_layered:
-            layers_fn = {"sandwich": self._layers_sandwich, "parallel": self._layers_parallel}.get(cfg.norm_placement,
-                                                                                                  self._layers_norm_after)
+            layers_fn = {"sandwich": self._layers_sandwich, "parallel": self._layers_parallel,
+                         "output": self._layers_output_normed}.get(cfg.norm_placement, self._layers_norm_after)
             return layers_fn(h, meta, kv, lo, hi, capture)
         acc, cur = None, 0  # per-token sum-of-squares accumulators of the residual stream while it is in folded form
         for li in range(lo, hi):

@@ -227,6 +227,19 @@ class DeltaWeights:
 
 
 @dataclass
+class WkvWeights:
+    """Weights of an RWKV time mixer (heads padded to their kernel widths)."""
+
+    mu: torch.Tensor  # [5, hidden] float32: share of the preceding token's input in the mixes for r, k, v, gate and decay
+    proj: torch.Tensor  # [4, heads * width, hidden (padded to eight)]: r, k, v, gate
+    decay_down: LinearWeight  # [decay_dim, hidden (padded to eight)]
+    decay_up: torch.Tensor  # [heads * width, decay_dim]
+    decay_base: torch.Tensor  # [heads * width] float32
+    bonus: torch.Tensor  # [heads * width] float32
+    norm: torch.Tensor  # [heads * width] float32
+
+
+@dataclass
 class LayerWeights:
     attn_norm: torch.Tensor
     wqkv: Optional[LinearWeight]  # None in a latent-attention layer (``mla`` holds its projections) or a convolution layer
@@ -240,6 +253,10 @@ class LayerWeights:
     sink: Optional[torch.Tensor] = None
     v_mix: Optional[torch.Tensor] = None  # [1] float32: the share of the first value-mixing layer's values
     delta: Optional[DeltaWeights] = None
+    wkv: Optional[WkvWeights] = None
+    score_bias: Optional[torch.Tensor] = None  # [heads, distances] float32, of the mixed scores; the last column serves all further ones
+    score_mix: Optional[torch.Tensor] = None  # [heads, heads] float32: scores of all heads to one head's
+    depth: Optional[torch.Tensor] = None  # [layer + 2] float32: weights of the embedding and of all results so far
     # two mixers whose projected outputs pass norms of their own: the right one's output projection (``wo`` is the left
     # one's) and both norms
     wo_right: Optional[LinearWeight] = None

@@ -34,6 +34,27 @@ def _cuda_listed():
     return _c
 
 
+def _cuda_joint():
+    from . import cuda_joint as _c
+
+    return _c
+
+
+def _cuda_wkv():
+    from . import cuda_wkv as _c
+
+    return _c
+
+
+class DepthStreams:
+    """The embedding and the layers' results of a step, kept for the weighted sums that go on from layer to layer."""
+
+    def __init__(self, x: torch.Tensor, layers: int):
+        self.first = x  # [T, hidden] float32
+        self.results = torch.empty(layers, *x.shape, dtype=torch.float32, device=x.device)
+        self.n = 0
+
+
 @dataclass
 class NormedPair:
     """Projected outputs of two mixers that pass RMS norms of their own: left_scale * norm(left) + right_scale * norm(right)."""
@@ -129,6 +150,38 @@ def joint_norm(res, mix, ffn, w_next, eps, act_dtype=torch.float32):
     return ref.joint_norm(res, mix, ffn, w_next, eps, act_dtype)
 
 
+@instrument("add_normed")
+def add_normed(res, y, w, groups, eps, act_dtype=None, streams: Optional[DepthStreams] = None, depth=None):
+    """A branch's output joins the stream through a norm in groups: x = res + norm(y) * w in float32, every one of ``groups``
+    consecutive parts over its own root mean square; ``y``: a tensor or ``RoutedRows``.  With ``streams`` and ``depth`` [n + 2] x
+    becomes the n-th result and what comes back is depth[0] * first + sum_j depth[j + 1] * results[j].  (that, the same in
+    ``act_dtype`` or None without one)."""
+    if res.is_cuda:
+        return _cuda_listed().add_normed(res, y, w, groups, eps, act_dtype, streams, depth)
+    return ref.add_normed(res, y, w, groups, eps, act_dtype, streams, depth)
+
+
+@instrument("grouped_norm")
+def grouped_norm(x, w, groups, eps, act_dtype=torch.float32):
+    """norm(x) * w, every one of ``groups`` consecutive parts over its own root mean square."""
+    if x.is_cuda:
+        return _cuda_listed().grouped_norm(x, w, groups, eps, act_dtype)
+    return ref.grouped_norm(x, w, groups, eps).to(act_dtype)
+
+
+@instrument("wkv_mixer")
+def wkv_mixer(x, w, spec, meta, state, window, eps, act_dtype=torch.float32):
+    """RWKV time mixing of one layer on its float32 input, up to (not including) the output projection: [T, spec.out_dim] in
+    ``act_dtype``; ``state`` [slots, heads, k_width, v_width] and ``window`` [slots, 1, hidden] are updated."""
+    if x.is_cuda:
+        return _cuda_wkv().wkv_mixer(x, w, spec, meta, state, window, eps, act_dtype)
+    mixes = ref.token_shift(x, w.mu, meta, window).to(act_dtype)
+    mixes = torch.nn.functional.pad(mixes, (0, w.proj.shape[2] - spec.hidden))
+    rkvg = torch.stack([(mixes[i].float() @ w.proj[i].float().t()).to(act_dtype) for i in range(4)])
+    low = linear(mixes[4], w.decay_down)
+    return ref.wkv(rkvg, ref.wkv_log_decay(low, w), w, spec, meta, state, eps).to(act_dtype)
+
+
 def first_values(z, a, lw, carry):
     """(values of the model's first value-mixing layer [T, kv_heads, width], this layer's share of them) for a layer that mixes
     them into its own; (None, None) elsewhere.  The first such layer leaves its own in ``carry``."""
@@ -152,7 +205,11 @@ def listed_mixer(x, lw, spec, ropes, meta, kv, kv_layer, state_layer, eps, carry
     z = linear(x, lw.wqkv)
     a, r, d, outs = spec.attention, spec.retention, spec.delta, []
     sl, sr = spec.branch_scales if lw.out_norms is None else (1.0, 1.0)
-    if a is not None:
+    if a is not None and a.joint_scores:
+        q = ref.joint_prep(z[:, : a.qkv_dim], a, meta, kv, kv_layer, eps)
+        o = ref.joint_attention(q, kv, kv_layer, meta, a, lw.score_bias, lw.score_mix, lw.sink, eps)
+        outs.append(o.reshape(x.shape[0], -1) * sl)
+    elif a is not None:
         q = ref.head_prep(z[:, : a.qkv_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps, *first_values(z, a, lw, carry))
         o = ref.paged_attention(q, kv, kv_layer, meta, a.scale, a.window, sink=lw.sink)
         if a.gate:

@@ -8,7 +8,7 @@ from typing import Optional
 
 import torch
 
-from ..models.config import HEAD_WIDTHS
+from ..models.config import HEAD_WIDTHS, ROW_TAIL
 from . import cuda as opcuda
 from . import cuda_latent as latent
 from .cuda import _check, _p, _stream
@@ -25,7 +25,8 @@ def lib():
         vp, i32, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
         L.oxb_branch_norm.argtypes = [vp] * 6 + [i32] * 3 + [f32, vp]
         L.oxb_head_prep.argtypes = ([vp, i32, i32, vp, vp, vp] + [i32] * 3 + [vp, vp, i32, f32] + [i32] * 5 + [vp, vp, i32, i32]
-                                    + [f32, f32, vp, i32, i32, i32, vp, vp])
+                                    + [f32, f32, vp, i32, i32, i32, vp, i32, i32, i32, vp])
+        L.oxb_add_normed.argtypes = [vp, vp, i32, vp, vp, i32, vp, i32, f32, vp, vp, i32, vp, vp, vp, i32, i32, i32, vp]
         L.oxb_joint_norm.argtypes = [vp] * 5 + [f32, f32, vp, i32, vp, vp, i32, vp, vp, vp] + [i32] * 3 + [f32, vp]
         L.oxb_gqa_attention_simt.argtypes = [vp, vp, i32, f32, vp, i32, vp, vp, vp, vp] + [i32] * 9 + [f32, vp, i32, i32, vp]
         L.oxb_kv_gather.argtypes = [vp] * 4 + [i32] * 7 + [vp, vp]
@@ -76,6 +77,39 @@ def joint_norm(res: torch.Tensor, mix, ffn, w_next: Optional[torch.Tensor], eps:
     return x, a
 
 
+def add_normed(res: torch.Tensor, y, w: torch.Tensor, groups: int, eps: float, act_dtype: Optional[torch.dtype], streams=None,
+               depth: Optional[torch.Tensor] = None):
+    from . import RoutedRows
+
+    T, H = res.shape
+    routed = y if isinstance(y, RoutedRows) else None
+    f = routed.rows if routed else y
+    if f.stride(-1) != 1:
+        f = f.contiguous()
+    x = torch.empty_like(res)
+    # (a float32 activation is the stream itself)
+    a = x if act_dtype == torch.float32 else None if act_dtype is None else torch.empty(T, H, dtype=act_dtype, device=res.device)
+    first = results = None
+    n = 0
+    if streams is not None:
+        first, results, n = streams.first, streams.results, streams.n
+        streams.n += 1
+    _check(lib().oxb_add_normed(res.data_ptr(), f.data_ptr(), f.stride(0), _p(routed.index) if routed else None,
+                                _p(routed.weights) if routed else None, routed.index.shape[1] if routed else 0, w.data_ptr(), groups, eps,
+                                _p(first), _p(results), n, _p(depth) if streams is not None else None, x.data_ptr(),
+                                None if a is x else _p(a), DT[f.dtype], T, H, _stream()), "oxb_add_normed")
+    return x, a
+
+
+def grouped_norm(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float, act_dtype: torch.dtype) -> torch.Tensor:
+    T, H = x.shape
+    x = x.contiguous()
+    a = torch.empty(T, H, dtype=act_dtype, device=x.device)
+    _check(lib().oxb_add_normed(x.data_ptr(), None, H, None, None, 0, w.data_ptr(), groups, eps, None, None, 0, None, None, a.data_ptr(),
+                                DT[act_dtype], T, H, _stream()), "oxb_add_normed")
+    return a
+
+
 # --------------------------------------------------------------------------- attention
 def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int, eps: float, v_first: Optional[torch.Tensor] = None,
               v_mix: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -89,7 +123,8 @@ def head_prep(z: torch.Tensor, q_norm, k_norm, spec, rope, meta, kv, layer: int,
     _check(lib().oxb_head_prep(z.data_ptr(), z.stride(0), DT[z.dtype], meta.positions.data_ptr(), meta.slot_mapping.data_ptr(),
                                tab.data_ptr(), max_pos, rot, pairing, _p(q_norm), _p(k_norm), 1 if spec.qk_norm == "full" else 0, eps, T, spec.heads, spec.kv_heads, spec.dim,
                                spec.width, q.data_ptr(), kv.data[layer].data_ptr(), kv.page_size, kv.num_blocks, spec.temp_coef, spec.temp_every,
-                               *first, spec.v_dim, _p(v_mix), _stream()), "oxb_head_prep")
+                               *first, spec.v_dim, _p(v_mix), int(spec.qk_norm == "unit"), int(spec.shared_kv),
+                               ROW_TAIL if spec.shared_kv else 0, _stream()), "oxb_head_prep")
     return q
 
 
@@ -216,8 +251,14 @@ def listed_mixer(x: torch.Tensor, lw, spec, ropes, meta, kv, kv_layer: int, stat
         if kv.data[kv_layer].dtype != x.dtype:
             raise ValueError(f"cache rows of listed layers are kept in the compute type on the GPU ({x.dtype}), not {kv.dtype_name}")
         na, no = a.proj_dim, a.out_dim
-        q = head_prep(z[:, : a.qkv_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps, *first_values(z, a, lw, carry))
-        attention(q, kv, kv_layer, meta, a, lw.sink, outs[0][:, :no], sl, z[:, a.qkv_dim : na] if a.gate else None)
+        prep = () if a.joint_scores else first_values(z, a, lw, carry)
+        q = head_prep(z[:, : a.qkv_dim], lw.q_norm, lw.k_norm, a, ropes[0], meta, kv, kv_layer, eps, *prep)
+        if a.joint_scores:
+            from . import cuda_joint
+
+            cuda_joint.attention(q, kv, kv_layer, meta, a, lw.score_bias, lw.score_mix, lw.sink, outs[0][:, :no], sl)
+        else:
+            attention(q, kv, kv_layer, meta, a, lw.sink, outs[0][:, :no], sl, z[:, a.qkv_dim : na] if a.gate else None)
     out = outs[-1][:, 0 if apart else no :]
     if d is not None:
         from . import cuda_delta

@@ -472,6 +472,116 @@ def delta_rule(z: torch.Tensor, w, spec, meta, state: torch.Tensor, window: torc
     return padded_norm(o, w.norm, spec.v_dim, eps).reshape(T, H * V) * gate
 
 
+def grouped_norm(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    parts = x.float().unflatten(-1, (groups, -1))
+    return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2) * w
+
+
+def add_normed(res: torch.Tensor, y, w: torch.Tensor, groups: int, eps: float, act_dtype, streams=None, depth=None):
+    x = res + grouped_norm(y, w, groups, eps)
+    if streams is not None:
+        streams.results[streams.n] = x
+        streams.n += 1
+        x = depth[0] * streams.first + torch.einsum("l,lth->th", depth[1:], streams.results[: streams.n])
+    return x, None if act_dtype is None else x.to(act_dtype)
+
+
+def token_shift(x: torch.Tensor, mu: torch.Tensor, meta, window: torch.Tensor) -> torch.Tensor:
+    """Mixes of every token's input with the one ahead of it: x [T, hidden] float32, mu [n, hidden] to [n, T, hidden];
+    ``window`` [slots, 1, hidden] holds the last input of earlier steps (updated)."""
+    before = torch.zeros_like(x)
+    qs, lens, slots = meta.query_start.tolist(), meta.seq_lens.tolist(), meta.state_slots.tolist()
+    for b in range(len(lens)):
+        t0, t1 = qs[b], qs[b + 1]
+        if t1 == t0:
+            continue
+        before[t0 + 1 : t1] = x[t0 : t1 - 1]
+        if slots[b] >= 0:
+            if lens[b] > t1 - t0:
+                before[t0] = window[slots[b], 0]
+            window[slots[b], 0] = x[t1 - 1]
+    return x + (before - x) * mu[:, None, :]
+
+
+def wkv_log_decay(low: torch.Tensor, w) -> torch.Tensor:
+    """Logarithms of the decays [T, heads * k_width], never positive, from the first of their two projections."""
+    return -torch.exp(torch.tanh(low.float()) @ w.decay_up.float().t() + w.decay_base)
+
+
+def wkv(rkvg: torch.Tensor, log_decay: torch.Tensor, w, spec, meta, state: torch.Tensor, eps: float) -> torch.Tensor:
+    """RWKV time mixing of one layer, token by token: rkvg [4, T, heads * width], state [slots, heads, k_width, v_width]
+    (updated); a sequence whose rows start at position 0 starts from a zero state.  Returns [T, heads * v_width] float32."""
+    T, H, K = rkvg.shape[1], spec.heads, spec.k_width
+    r, k, v, g = rkvg.float().unflatten(2, (H, K))
+    decay, u = torch.exp(log_decay.float()).unflatten(1, (H, K)), w.bonus.reshape(H, K)
+    o = torch.zeros(T, H, K, dtype=torch.float32, device=r.device)
+    qs, lens, slots = meta.query_start.tolist(), meta.seq_lens.tolist(), meta.state_slots.tolist()
+    for b in range(len(lens)):
+        t0, t1 = qs[b], qs[b + 1]
+        if slots[b] < 0 or t1 == t0:
+            continue
+        S = torch.zeros_like(state[slots[b]]) if lens[b] == t1 - t0 else state[slots[b]]
+        for t in range(t0, t1):
+            o[t] = (S * r[t][:, :, None]).sum(1) + (r[t] * u * k[t]).sum(-1, keepdim=True) * v[t]
+            S = decay[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        state[slots[b]] = S
+    y = padded_norm(o, w.norm.reshape(H, K), spec.dim, eps) * torch.nn.functional.silu(g)
+    return y.reshape(T, H * K)
+
+
+def unit_heads(x: torch.Tensor, n: int, eps: float) -> torch.Tensor:
+    """Zero-padded heads that hold ``n`` values over their root mean squares."""
+    return padded_norm(x.float(), 1.0, n, eps)
+
+
+def joint_prep(z: torch.Tensor, spec, meta, kv, layer: int, eps: float) -> torch.Tensor:
+    """From a layer's q | k projections (heads of ``spec.width`` values): this step's cache rows, keys as projected with one over
+    their root mean square behind them; the queries [T, heads, width] over theirs."""
+    T, H, G, W = z.shape[0], spec.heads, spec.kv_heads, spec.width
+    q, k = z[:, : H * W].reshape(T, H, W), z[:, H * W : (H + G) * W].reshape(T, G, W)
+    row = torch.zeros(T, G, spec.cache_shape[2], dtype=z.dtype, device=z.device)
+    row[..., :W] = k
+    row[..., W] = torch.rsqrt(k.float().pow(2).sum(-1) / spec.dim + eps)
+    kv_write(kv, layer, row, None, meta.slot_mapping)
+    return unit_heads(q, spec.dim, eps).to(z.dtype)
+
+
+def visible(qpos: torch.Tensor, kpos: torch.Tensor, window: int, keep_first: int) -> torch.Tensor:
+    """Which keys a query sees: those up to it that are in its window (0: all) or among the first ``keep_first``."""
+    seen = kpos <= qpos
+    return seen & ((kpos > qpos - window) | (kpos < keep_first)) if window > 0 else seen
+
+
+def joint_attention(q: torch.Tensor, kv, layer: int, meta, spec, bias: Optional[torch.Tensor], mix: Optional[torch.Tensor],
+                    sink: Optional[torch.Tensor], eps: float) -> torch.Tensor:
+    """Attention on the scores of all heads together: soft-capped, mixed over the heads by ``mix``, plus ``bias`` [heads,
+    distances] (of the mixed scores; the last one serves all further distances).  One cached row is key and value."""
+    T, H, W = q.shape
+    out = torch.zeros(T, H, W, dtype=torch.float32, device=q.device)
+    qs, lens = meta.query_start.tolist(), meta.seq_lens.tolist()
+    per = H // spec.kv_heads
+    for b in range(len(lens)):
+        t0, t1 = qs[b], qs[b + 1]
+        n, L = t1 - t0, lens[b]
+        if n == 0:
+            continue
+        nb = (L + kv.page_size - 1) // kv.page_size
+        rows = kv.data[layer][meta.block_tables[b][:nb].long()][:, :, 0].float()  # [pages, heads, page, row]
+        k = rows.transpose(1, 2).reshape(-1, spec.kv_heads, rows.shape[-1])[:L, :, :W].repeat_interleave(per, dim=1)
+        s = torch.einsum("qhd,lhd->hql", q[t0:t1].float(), unit_heads(k, spec.dim, eps)) * spec.scale
+        if spec.softcap > 0:
+            s = torch.tanh(s / spec.softcap) * spec.softcap
+        if mix is not None:
+            s = torch.einsum("hg,gql->hql", mix, s)
+        qpos, kpos = torch.arange(L - n, L, device=q.device)[:, None], torch.arange(L, device=q.device)[None, :]
+        if bias is not None:
+            s = s + bias[:, (qpos - kpos).clamp(0, bias.shape[1] - 1)]
+        s = s.masked_fill(~visible(qpos, kpos, spec.window, spec.keep_first)[None], float("-inf"))
+        p = softmax_sink(s, None if sink is None else sink[:, None, None])
+        out[t0:t1] = torch.einsum("hql,lhd->qhd", p, k)
+    return out.to(q.dtype)
+
+
 # --------------------------------------------------------------------------- MoE routing
 
 
