@@ -109,6 +109,17 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return r;
 }
 
+// The sequence that holds row t.
+__device__ __forceinline__ int sequence_of(const int* query_start, int B, int t) {
+  int b = 0, hi = B - 1;
+  while (b < hi) {
+    const int mid = (b + hi + 1) >> 1;
+    if (query_start[mid] <= t) b = mid;
+    else hi = mid - 1;
+  }
+  return b;
+}
+
 // ----------------------------------------------------------------------------- smem / mbarrier
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {
   return static_cast<uint32_t>(__cvta_generic_to_shared(p));

@@ -25,17 +25,6 @@ struct TokenShiftArgs {
   int B, T, H, n, ld;
 };
 
-// The sequence that holds row t.
-__device__ __forceinline__ int sequence_of(const int* query_start, int B, int t) {
-  int b = 0, hi = B - 1;
-  while (b < hi) {
-    const int mid = (b + hi + 1) >> 1;
-    if (query_start[mid] <= t) b = mid;
-    else hi = mid - 1;
-  }
-  return b;
-}
-
 // out[i] = x + (x_before - x) mu[i].  grid (T, channel blocks); the CTA of a sequence's first row reads what earlier steps left
 // in the window and then leaves the portion's last row there.
 template <typename A, int VEC>

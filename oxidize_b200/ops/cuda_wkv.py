@@ -3,15 +3,18 @@
 from __future__ import annotations
 
 import ctypes
+from typing import Optional
 
 import torch
 
 from ..models.config import pad_to
 from . import cuda_latent as latent
-from .cuda import _check, _stream
+from .cuda import _check, _p, _stream
 
 _declared = False
 _ALL = 1 << 30
+SCRATCH_BYTES = 512 << 20  # of the chunk kernels
+CHUNK, CHUNK_ROWS = 64, 9  # tokens per chunk; sequences that feed at least CHUNK_ROWS rows in a step go through chunks
 
 
 def lib():
@@ -21,7 +24,8 @@ def lib():
         vp, i32, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_float
         L.oxb_token_shift.argtypes = [vp] * 6 + [i32, vp] + [i32] * 6 + [vp]
         L.oxb_wkv_decay.argtypes = [vp] * 4 + [i32] * 4 + [vp]
-        L.oxb_wkv.argtypes = [vp, i32, i32] + [vp] * 7 + [i32, vp] + [i32] * 5 + [f32, i32, i32, vp]
+        L.oxb_wkv.argtypes = [vp, i32, i32] + [vp] * 7 + [i32, vp] + [i32] * 5 + [f32] + [i32] * 4 + [vp, vp]
+        L.oxb_wkv_chunk_bytes.argtypes = [i32]
         _declared = True
     return L
 
@@ -48,17 +52,34 @@ def log_decay(low: torch.Tensor, w) -> torch.Tensor:
     return out
 
 
-def wkv(z: torch.Tensor, decay: torch.Tensor, w, spec, meta, state: torch.Tensor, eps: float, out: torch.Tensor) -> None:
+def round_chunks(chunks: int, bytes_per_chunk: int) -> int:
+    """Chunks of a round: as many as the scratch limit lets through, in rounds of equal length."""
+    rounds = -(-chunks * bytes_per_chunk // SCRATCH_BYTES)
+    return max(1, -(-chunks // rounds))
+
+
+def wkv(z: torch.Tensor, decay: torch.Tensor, w, spec, meta, state: torch.Tensor, eps: float, out: torch.Tensor,
+        chunk_rows: Optional[int] = None, rounds: Optional[int] = None) -> None:
     """z [T, r | k | v | gate] to the normed, gated heads ``out`` [T, heads * width]; ``state`` [slots, H, K, K] is updated."""
     H, K, _ = spec.state_shape
     B = meta.seq_lens.shape[0]
+    most = max(1, meta.max_query_len)
 
-    def run(lo: int, hi: int) -> None:
+    def run(lo: int, hi: int, rnd: int = 0, ws: Optional[torch.Tensor] = None) -> None:
         _check(lib().oxb_wkv(z.data_ptr(), z.stride(0), latent.DT[z.dtype], decay.data_ptr(), meta.query_start.data_ptr(),
                              meta.seq_lens.data_ptr(), meta.state_slots.data_ptr(), w.bonus.data_ptr(), w.norm.data_ptr(), state.data_ptr(),
-                             state.shape[0], out.data_ptr(), out.stride(0), B, H, K, spec.dim, eps, lo, hi, _stream()), "oxb_wkv")
+                             state.shape[0], out.data_ptr(), out.stride(0), B, H, K, spec.dim, eps, lo, hi, most, rnd, _p(ws), _stream()),
+               "oxb_wkv")
 
-    run(1, _ALL)
+    cut = CHUNK_ROWS if chunk_rows is None else chunk_rows
+    size = lib().oxb_wkv_chunk_bytes(K) if z.dtype == torch.bfloat16 and most >= cut else 0
+    if size == 0:
+        run(1, _ALL)
+        return
+    if meta.host_lens is None or min(n for n, _ in meta.host_lens) < cut:
+        run(1, cut - 1)
+    rnd = round_chunks((most + CHUNK - 1) // CHUNK, B * H * size) if rounds is None else rounds
+    run(cut, _ALL, rnd, torch.empty(B * rnd * H * size, dtype=torch.uint8, device=z.device))
 
 
 def wkv_mixer(x: torch.Tensor, w, spec, meta, state: torch.Tensor, window: torch.Tensor, eps: float, act_dtype: torch.dtype) -> torch.Tensor:
