@@ -4,10 +4,11 @@
 // [width + tail] holds the key as projected, which is the value, and behind it the float that turns it into the normed key.
 //
 // joint_attention_simt_kernel: any type, width, page and number of heads that fits shared memory.
+// joint_decode_kernel: one token per cluster, keys dealt out to its CTAs (decoded tokens and short portions).
+// joint_prefill.cuh: long portions.
 #pragma once
 #include "attention.cuh"
 #include "latent.cuh"
-#include "wkv.cuh"
 
 namespace oxb {
 
@@ -26,6 +27,7 @@ struct JointArgs {
   int distances;
   int B, max_blocks, T, H, G, W, tail, page, num_blocks, window, keep_first;
   float scale, cap;         // cap 0: scores as they are
+  int max_rows;             // sequences that feed more rows belong to other kernels
 };
 
 __device__ __forceinline__ float joint_capped(const JointArgs& a, float s) { return a.cap > 0.f ? a.cap * tanhf(s / a.cap) : s; }
@@ -43,6 +45,7 @@ __global__ void __launch_bounds__(256) joint_attention_simt_kernel(const JointAr
   const int b = sequence_of(a.query_start, a.B, t);
   const int pos = a.seq_lens[b] - (a.query_start[b + 1] - t);
   pdl_wait();
+  if (a.query_start[b + 1] - a.query_start[b] > a.max_rows) return;
   for (int i = tid; i < H * W; i += 256) {
     q[i] = lat_f32(reinterpret_cast<const T*>(a.q)[(size_t)t * H * W + i]) * a.scale;
     acc[i] = 0.f;
@@ -115,6 +118,325 @@ __global__ void __launch_bounds__(256) joint_attention_simt_kernel(const JointAr
   }
   T* out = reinterpret_cast<T*>(a.out) + (size_t)t * a.ld_out;
   for (int i = tid; i < H * W; i += 256) out[i] = lat_from<T>(l[i / W] > 0.f ? acc[i] * a.out_scale / l[i / W] : 0.f);
+}
+
+// ----------------------------------------------------------------------------- decoded tokens
+// cap tanh(s / cap) for scores of bfloat16 factors: tanh(x) = 1 - 2 / (1 + exp(2 x)), absolute error about 1e-7
+__device__ __forceinline__ float joint_capped_fast(float s, float cap, float inv_cap2 /* 2 / cap */) {
+  return cap > 0.f ? cap - __fdividef(2.f * cap, 1.f + __expf(s * inv_cap2)) : s;
+}
+
+// A page of one key head: 16 rows of HD values and their tails, as it stands in the cache (rows HD * 2 + 16 bytes apart, which
+// ldmatrix reads without bank conflicts).  One warp.
+template <int HD>
+__device__ __forceinline__ void joint_load_page(uint8_t* stage, const JointArgs& a, int blk, int g, int lane) {
+  constexpr int BYTES = 16 * (HD * 2 + 16);
+  const uint8_t* src = reinterpret_cast<const uint8_t*>(a.cache) + ((size_t)blk * a.G + g) * BYTES;
+#pragma unroll
+  for (int c = lane; c < BYTES / 16; c += 32) cp_async16(stage + c * 16, src + c * 16);
+}
+
+constexpr int JD_WARPS = 8, JD_PAGES = 4, JD_KEYS = 16 * JD_PAGES, JD_SROW = JD_KEYS + 4, JD_PROW = JD_KEYS + 8;
+struct JointDecodeSmem {
+  int s, o, mix, p, stat, total;  // byte offsets; the rings of pages come first
+};
+__host__ __device__ inline JointDecodeSmem joint_decode_smem(int H, int G, int HD) {
+  const int parts = G < JD_WARPS ? JD_WARPS / G : 1, h4 = (H + 3) / 4 * 4;
+  JointDecodeSmem m;
+  m.s = JD_WARPS * 2 * 16 * (HD * 2 + 16);
+  m.o = m.s + H * JD_SROW * 4;
+  m.mix = m.o + parts * H * HD * 4;
+  m.p = m.mix + H * h4 * 4;
+  m.stat = m.p + (H * JD_PROW * 2 + 15) / 16 * 16;
+  m.total = m.stat + 3 * h4 * 4;
+  return m;
+}
+
+// grid (splits, T), the splits of a token one cluster.  A round covers 64 keys: every warp takes the scores of its key heads
+// (where there are fewer than eight, of some of their pages), the CTA mixes them and takes the softmax step, and every warp
+// reads its pages once more (out of the L2) as values.
+template <int HD>
+__global__ void __launch_bounds__(JD_WARPS * 32, HD <= 128 ? 2 : 1) joint_decode_kernel(const JointArgs a) {
+  constexpr int ROWB = HD * 2 + 16, STAGE = 16 * ROWB, KS = HD / 16, NT = HD / 8;
+  extern __shared__ __align__(16) uint8_t jd_smem[];
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3, mi = lane >> 3, lr = lane & 7;
+  const int t = blockIdx.y, split = blockIdx.x, splits = gridDim.x;
+  const int H = a.H, G = a.G, per = H / G, h4 = (H + 3) / 4 * 4, parts = G < JD_WARPS ? JD_WARPS / G : 1, units = G * parts;
+  const int b = sequence_of(a.query_start, a.B, t), rows = a.query_start[b + 1] - a.query_start[b];
+  if (rows > a.max_rows) {  // (the whole cluster leaves)
+    pdl_wait();
+    return;
+  }
+  const int pos = a.seq_lens[b] - (a.query_start[b + 1] - t);
+  const JointDecodeSmem sm = joint_decode_smem(H, G, HD);
+  float *sS = reinterpret_cast<float*>(jd_smem + sm.s), *sO = reinterpret_cast<float*>(jd_smem + sm.o), *sMix = reinterpret_cast<float*>(jd_smem + sm.mix);
+  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(jd_smem + sm.p);
+  float *m_run = reinterpret_cast<float*>(jd_smem + sm.stat), *l_run = m_run + h4, *corr = l_run + h4;
+  uint8_t* ring = jd_smem + warp * 2 * STAGE;
+  for (int i = tid; i < H * h4; i += JD_WARPS * 32) {  // [g][h]
+    const int g = i / h4, h = i % h4;
+    sMix[i] = h < H ? (a.mix != nullptr ? a.mix[h * H + g] : (g == h ? 1.f : 0.f)) : 0.f;
+  }
+  for (int i = tid; i < parts * H * HD; i += JD_WARPS * 32) sO[i] = 0.f;
+  if (tid < h4) {
+    m_run[tid] = -INFINITY;
+    l_run[tid] = 0.f;
+  }
+  // the pages this token sees: those of kept first positions ahead of the window's, then the window's
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0, page_lo = lo >> 4;
+  const int kept = min((a.keep_first + 15) >> 4, page_lo), n_pages = pos < 0 ? 0 : kept + (pos >> 4) - page_lo + 1;
+  const int share = (n_pages + splits - 1) / splits, p0 = split * share, p1 = min(n_pages, p0 + share);
+  const int* bt = a.block_tables + (size_t)b * a.max_blocks;
+  auto page_of = [&](int i) { return i < kept ? i : page_lo + i - kept; };
+  const float inv_cap2 = a.cap > 0.f ? 2.f / a.cap : 0.f;
+  int slot = 0;
+  auto load = [&](int r0, int u, int p) {
+    int blk = bt[page_of(r0 + p)];
+    if ((unsigned)blk >= (unsigned)a.num_blocks) {
+      if (lane == 0) oxb_report(OXB_BAD_BLOCK_ID, blk);
+      blk = 0;
+    }
+    joint_load_page<HD>(ring + slot * STAGE, a, blk, u / parts, lane);
+  };
+  auto first_unit = [&](int npg, int& u, int& p) {  // (a warp without pages in this round: u = units)
+    u = warp;
+    p = u < units ? u % parts : 0;
+    if (u < units && p >= npg) u = units;
+  };
+  auto next_unit = [&](int npg, int& u, int& p) {
+    p += parts;
+    if (p >= npg) {
+      u += JD_WARPS;
+      p = u < units ? u % parts : 0;
+    }
+    if (u < units && p >= npg) u = units;
+  };
+  __syncthreads();
+  pdl_wait();
+  if (p0 < p1) {
+    int u, p;
+    first_unit(min(JD_PAGES, p1 - p0), u, p);
+    if (u < units) load(p0, u, p);
+  }
+  cp_async_commit();
+  for (int r0 = p0; r0 < p1; r0 += JD_PAGES) {
+    const int npg = min(JD_PAGES, p1 - r0);
+    // ---- scores
+    {
+      int u, p, held = -1;
+      uint32_t qf[KS][4];
+      first_unit(npg, u, p);
+      while (u < units) {
+        int nu = u, np = p;
+        next_unit(npg, nu, np);
+        slot ^= 1;
+        if (nu < units) load(r0, nu, np);
+        slot ^= 1;
+        cp_async_commit();
+        const int g = u / parts;
+        if (g != held) {
+          held = g;
+          const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.q) + ((size_t)t * H + g * per) * HD + 2 * t4;
+#pragma unroll
+          for (int ks = 0; ks < KS; ++ks)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+              const bool on = g8 + 8 * i < per;
+              const __nv_bfloat16* qp = q + (size_t)(on ? g8 + 8 * i : 0) * HD + ks * 16;
+              qf[ks][i] = on ? *reinterpret_cast<const uint32_t*>(qp) : 0u;
+              qf[ks][i + 2] = on ? *reinterpret_cast<const uint32_t*>(qp + 8) : 0u;
+            }
+        }
+        cp_async_wait<1>();
+        __syncwarp();
+        const uint8_t* st = ring + slot * STAGE;
+        const uint32_t addr = smem_u32(st) + ((mi >> 1) * 8 + lr) * ROWB + (mi & 1) * 16;
+        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4(addr + ks * 32, b0, b1, b2, b3);
+          mma_bf16_16816(s[0], qf[ks], b0, b1);
+          mma_bf16_16816(s[1], qf[ks], b2, b3);
+        }
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          const int key = nt * 8 + 2 * t4;
+          const float f0 = *reinterpret_cast<const float*>(st + key * ROWB + HD * 2) * a.scale;
+          const float f1 = *reinterpret_cast<const float*>(st + (key + 1) * ROWB + HD * 2) * a.scale;
+#pragma unroll
+          for (int i = 0; i < 2; ++i)
+            if (g8 + 8 * i < per)
+              *reinterpret_cast<float2*>(sS + (g * per + g8 + 8 * i) * JD_SROW + p * 16 + key) =
+                  make_float2(joint_capped_fast(s[nt][2 * i] * f0, a.cap, inv_cap2), joint_capped_fast(s[nt][2 * i + 1] * f1, a.cap, inv_cap2));
+        }
+        __syncwarp();
+        slot ^= 1;
+        u = nu;
+        p = np;
+      }
+      first_unit(npg, u, p);  // the first page of the values is on its way during the mixing
+      if (u < units) load(r0, u, p);
+      cp_async_commit();
+    }
+    __syncthreads();
+    // ---- mixing and softmax: a warp has four heads and all keys, a lane keys `lane` and `lane` + 32
+    for (int h0 = 4 * warp; h0 < H; h0 += 4 * JD_WARPS) {
+      float v[2][4];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.f;
+#pragma unroll 4
+      for (int g = 0; g < H; ++g) {
+        const float4 w = *reinterpret_cast<const float4*>(sMix + g * h4 + h0);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const float x = sS[g * JD_SROW + lane + 32 * j];
+          v[j][0] = fmaf(w.x, x, v[j][0]);
+          v[j][1] = fmaf(w.y, x, v[j][1]);
+          v[j][2] = fmaf(w.z, x, v[j][2]);
+          v[j][3] = fmaf(w.w, x, v[j][3]);
+        }
+      }
+      bool ok[2];
+      int dist[2];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int pg = (lane >> 4) + 2 * j, key = page_of(r0 + min(pg, npg - 1)) * 16 + (lane & 15);
+        ok[j] = pg < npg && key <= pos && (a.window <= 0 || key > pos - a.window || key < a.keep_first);
+        dist[j] = min(max(pos - key, 0), a.distances - 1);
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int h = h0 + i;
+        if (h >= H) break;
+        float x[2];
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const float bias = a.bias != nullptr ? a.bias[(size_t)h * a.distances + dist[j]] : 0.f;
+          x[j] = ok[j] ? (v[j][i] + bias) * 1.4426950408889634f : -INFINITY;
+        }
+        const float old = m_run[h], top = fmaxf(old, warp_max(fmaxf(x[0], x[1]))), base = top == -INFINITY ? 0.f : top;
+        const float y0 = exp2f(x[0] - base), y1 = exp2f(x[1] - base), sum = warp_sum(y0 + y1), c = exp2f(old - base);
+        sP[h * JD_PROW + lane] = __float2bfloat16(y0);
+        sP[h * JD_PROW + lane + 32] = __float2bfloat16(y1);
+        __syncwarp();
+        if (lane == 0) {
+          m_run[h] = top;
+          l_run[h] = l_run[h] * c + sum;
+          corr[h] = c;
+        }
+      }
+    }
+    __syncthreads();
+    // ---- values
+    {
+      int u, p;
+      float o[NT][4];
+      bool fresh = true;
+      auto flush = [&](int unit, bool any) {  // O <- corr O + o
+        const int g = unit / parts;
+        float* dst = sO + ((size_t)(unit % parts) * H + g * per) * HD + 2 * t4;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int r = g8 + 8 * i;
+          if (r >= per) continue;
+          const float c = corr[g * per + r];
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt) {
+            float2* at = reinterpret_cast<float2*>(dst + r * HD + nt * 8);
+            const float2 x = *at;
+            *at = make_float2(fmaf(c, x.x, any ? o[nt][2 * i] : 0.f), fmaf(c, x.y, any ? o[nt][2 * i + 1] : 0.f));
+          }
+        }
+      };
+      first_unit(npg, u, p);
+      if (u >= units && warp < units) flush(warp, false);  // (no page of its own in this round)
+      while (u < units) {
+        int nu = u, np = p;
+        next_unit(npg, nu, np);
+        slot ^= 1;
+        if (nu < units) load(r0, nu, np);
+        slot ^= 1;
+        cp_async_commit();
+        if (fresh) {
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
+        }
+        const int g = u / parts;
+        uint32_t pf[4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const bool on = g8 + 8 * i < per;
+          const __nv_bfloat16* src = sP + (g * per + (on ? g8 + 8 * i : 0)) * JD_PROW + p * 16 + 2 * t4;
+          pf[i] = on ? *reinterpret_cast<const uint32_t*>(src) : 0u;
+          pf[i + 2] = on ? *reinterpret_cast<const uint32_t*>(src + 8) : 0u;
+        }
+        cp_async_wait<1>();
+        __syncwarp();
+        const uint32_t addr = smem_u32(ring + slot * STAGE) + ((mi & 1) * 8 + lr) * ROWB + (mi >> 1) * 16;
+#pragma unroll
+        for (int nt = 0; nt < NT; nt += 2) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4_trans(addr + nt * 16, b0, b1, b2, b3);
+          mma_bf16_16816(o[nt], pf, b0, b1);
+          mma_bf16_16816(o[nt + 1], pf, b2, b3);
+        }
+        __syncwarp();
+        slot ^= 1;
+        fresh = nu != u;
+        if (fresh) flush(u, true);
+        u = nu;
+        p = np;
+      }
+      if (r0 + JD_PAGES < p1) {
+        first_unit(min(JD_PAGES, p1 - r0 - JD_PAGES), u, p);
+        if (u < units) load(r0 + JD_PAGES, u, p);
+      }
+      cp_async_commit();
+    }
+    // (the next round's scores overwrite sS, which nobody reads any more; its mixing starts behind a barrier)
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  if (parts > 1) {
+    for (int i = tid; i < H * HD; i += JD_WARPS * 32) {
+      float s = sO[i];
+      for (int k = 1; k < parts; ++k) s += sO[(size_t)k * H * HD + i];
+      sO[i] = s;
+    }
+    __syncthreads();
+  }
+  if (splits > 1) cluster_sync_all();
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (size_t)t * a.ld_out;
+  for (int i = split * JD_WARPS * 32 + tid; i < H * HD / 4; i += splits * JD_WARPS * 32) {
+    const int h = 4 * i / HD;
+    const float sink = a.sink != nullptr ? a.sink[h] * 1.4426950408889634f : -INFINITY;
+    float4 v;
+    float L, M = sink;
+    if (splits == 1) {
+      M = fmaxf(M, m_run[h]);
+      const float w = m_run[h] == -INFINITY ? 0.f : exp2f(m_run[h] - M);
+      v = *reinterpret_cast<const float4*>(sO + 4 * i);
+      v = make_float4(w * v.x, w * v.y, w * v.z, w * v.w);
+      L = w * l_run[h];
+    } else {
+      const uint32_t m_at = smem_u32(m_run + h), l_at = smem_u32(l_run + h), o_at = smem_u32(sO + 4 * i);
+      for (int r = 0; r < splits; ++r) M = fmaxf(M, dsmem_ld_f32(dsmem_map(m_at, r)));
+      v = make_float4(0.f, 0.f, 0.f, 0.f);
+      L = 0.f;
+      for (int r = 0; r < splits; ++r) {
+        const float m = dsmem_ld_f32(dsmem_map(m_at, r)), w = m == -INFINITY ? 0.f : exp2f(m - M);
+        const float4 x = dsmem_ld_f32x4(dsmem_map(o_at, r));
+        L = fmaf(w, dsmem_ld_f32(dsmem_map(l_at, r)), L);
+        v = make_float4(fmaf(w, x.x, v.x), fmaf(w, x.y, v.y), fmaf(w, x.z, v.z), fmaf(w, x.w, v.w));
+      }
+    }
+    if (sink != -INFINITY) L += exp2f(sink - M);
+    const float inv = L > 0.f ? a.out_scale / L : 0.f;
+    *reinterpret_cast<uint2*>(out + 4 * i) = make_uint2(pack_bf16x2(v.x * inv, v.y * inv), pack_bf16x2(v.z * inv, v.w * inv));
+  }
+  if (splits > 1) cluster_sync_all();  // every peer has finished reading this CTA's partial
 }
 
 }  // namespace oxb
