@@ -65,8 +65,8 @@ def parse_args():
     ap.add_argument("--draft-tokens", type=int, default=4)
     ap.add_argument("--layered", default=None, metavar="WIDTHxHEADS",
                     help="instead of the headline workload: a model that lists its layers beside the closest uniform "
-                         "models of that size (see bench/layered_bench.py, sokirax_bench.py, pavatar_bench.py), e.g. 4096x32")
-    ap.add_argument("--design", default="vefilix", choices=["vefilix", "sokirax", "pavatar"], help="the design that --layered measures")
+                         "models of that size (see bench/layered_bench.py, sokirax_bench.py, pavatar_bench.py, netovik_bench.py), e.g. 4096x32")
+    ap.add_argument("--design", default="vefilix", choices=["vefilix", "sokirax", "pavatar", "netovik"], help="the design that --layered measures")
     return ap.parse_args()
 
 

@@ -220,6 +220,10 @@ def kernel_numbers(width: int, heads: int, window: int, dev, steps: int) -> list
 def main(args) -> int:
     if args.gpus != 1:
         raise SystemExit("--layered runs on one GPU")
+    if args.design == "netovik":
+        import netovik_bench
+
+        return netovik_bench.main(args)
     if args.design == "pavatar":
         import pavatar_bench
 

@@ -554,7 +554,7 @@ def _load_joint(src: LayeredWeightSource, cfg: ModelConfig, i: int) -> LayerWeig
 def gated_block(lw: LayerWeights, f, hidden: int, triple) -> None:
     """Feed-forward weights of a layer, dense or routed; ``triple(prefix)``: (gate, up, down) as stored."""
     if isinstance(f, MoESpec):
-        lw.experts = listed_experts(f, [triple(f"e{e}.") for e in range(f.n_experts)], hidden)
+        lw.experts = listed_experts(f, (triple(f"e{e}.") for e in range(f.n_experts)), hidden)
     else:
         gu, down = gated_pair(*triple(""), f.pad_size)
         lw.w_gate_up, lw.w_down = LinearWeight([gu]), LinearWeight([down])

@@ -369,10 +369,14 @@ def synth_layered_weights(cfg: ModelConfig, device, quant: str = "BF16", seed: i
         if spec.weights_of is not None:
             layers.append(layers[spec.weights_of])
             continue
-        if cfg.norm_placement in ("sandwich", "parallel"):
+        whole = {"sandwich": _synth_listed, "parallel": _synth_joint, "output": _synth_output_normed}.get(cfg.norm_placement)
+        if whole is not None:
             if tp_size > 1:
                 raise ValueError("layers with per-sequence states and norms over all heads are not sharded")
-            layers.append((_synth_listed if cfg.norm_placement == "sandwich" else _synth_joint)(spec, h, mat, ones))
+            layers.append(whole(spec, h, mat, ones))
+            if cfg.depth_average:  # (mostly the layer's own result)
+                n = len(layers) + 1
+                layers[-1].depth = torch.cat([0.1 / n * ones(n - 1), ones(1)])
             continue
         m, f = spec.mixer, spec.ffn
         H, own = m.heads // tp_size, m.kv_from is None
@@ -455,6 +459,34 @@ def _synth_joint(spec, h: int, mat, ones) -> LayerWeights:
     if f is not None:
         lw.router, lw.router_bias = dense_qtensor(mat(f.n_experts, h)), 0.0 * ones(f.n_experts)
         lw.experts = listed_experts(f, ((None, mat(f.expert.size, h), mat(h, f.expert.size)) for _ in range(f.n_experts)), h)
+    return lw
+
+
+def _synth_output_normed(spec, h: int, mat, ones) -> LayerWeights:
+    """One layer with norms on its branches' outputs only."""
+    from ..models.config import MoESpec
+    from ..models.layered import dense_qtensor, gated_block, listed_mixer, wkv_weights
+
+    a, k, f = spec.attention, spec.wkv, spec.ffn
+    if k is not None:
+        c = k.heads * k.dim
+        t = {n: mat(c, h) for n in "rkvg"}
+        t.update({"w1": mat(k.rank, h), "w2": mat(c, k.rank), "o": mat(h, c), "w0": -3.0 * ones(c), "u": 0.5 * ones(c), "norm": ones(c)})
+        t.update({"mu." + n: 0.5 * ones(h) for n in "rkvgw"})
+        kw = wkv_weights(k, t, t["r"].dtype)
+    else:
+        att = {"q": mat(a.heads * a.dim, h), "k": mat(a.kv_heads * a.dim, h), "o": mat(h, a.heads * a.dim),
+               "rel": mat(a.bias_rows, a.heads).float(), "talk": torch.diag(ones(a.heads)) + mat(a.heads, a.heads).float()}
+        att.update({n + ".b": 0.1 * ones(att[n].shape[0]) for n in "qk"})
+        kw = listed_mixer(spec, att, {})
+    lw = LayerWeights(attn_norm=None, post_attn_norm=ones(h), ffn_norm=None, **kw)
+    if f is None:
+        return lw
+    lw.post_ffn_norm = ones(h)
+    one = f.expert if isinstance(f, MoESpec) else f
+    if isinstance(f, MoESpec):
+        lw.router = dense_qtensor(mat(f.n_experts, h))
+    gated_block(lw, f, h, lambda prefix: (mat(one.size, h), mat(one.size, h), mat(h, one.size)))
     return lw
 
 
