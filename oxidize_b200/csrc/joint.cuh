@@ -121,9 +121,23 @@ __global__ void __launch_bounds__(256) joint_attention_simt_kernel(const JointAr
 }
 
 // ----------------------------------------------------------------------------- decoded tokens
-// cap tanh(s / cap) for scores of bfloat16 factors: tanh(x) = 1 - 2 / (1 + exp(2 x)), absolute error about 1e-7
-__device__ __forceinline__ float joint_capped_fast(float s, float cap, float inv_cap2 /* 2 / cap */) {
-  return cap > 0.f ? cap - __fdividef(2.f * cap, 1.f + __expf(s * inv_cap2)) : s;
+__device__ __forceinline__ float joint_exp2(float x) {  // 0 where that is no normal number
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// cap tanh(f s / cap) for scores of bfloat16 factors, tanh(x) = 1 - 2 / (1 + exp(2 x)): `f` carries the factor 2 log2(e) / cap
+// (joint_factor), absolute error about 1e-7 cap.
+struct JointCap {
+  float cap, factor;
+};
+__device__ __forceinline__ JointCap joint_cap(const JointArgs& a) {
+  return JointCap{a.cap, a.cap > 0.f ? a.scale * 2.f * 1.4426950408889634f / a.cap : a.scale};
+}
+__device__ __forceinline__ float joint_capped_fast(float s, float f, const JointCap& c) {
+  if (c.cap <= 0.f) return s * f;
+  return fmaf(-2.f * c.cap, __fdividef(1.f, 1.f + joint_exp2(s * f)), c.cap);
 }
 
 // A page of one key head: 16 rows of HD values and their tails, as it stands in the cache (rows HD * 2 + 16 bytes apart, which
@@ -138,12 +152,16 @@ __device__ __forceinline__ void joint_load_page(uint8_t* stage, const JointArgs&
 
 constexpr int JD_WARPS = 8, JD_PAGES = 4, JD_KEYS = 16 * JD_PAGES, JD_SROW = JD_KEYS + 4, JD_PROW = JD_KEYS + 8;
 struct JointDecodeSmem {
-  int s, o, mix, p, stat, total;  // byte offsets; the rings of pages come first
+  int s, o, mix, p, stat, total;  // byte offsets; the warps' pages come first
 };
+// Whether a warp's pages of a round stay in shared memory, and how many warps share a key head.
+__host__ __device__ inline bool joint_decode_resident(int G, int HD) { return G <= JD_WARPS && HD <= 128; }
+__host__ __device__ inline int joint_decode_parts(int G, bool res) { return res && G < JD_WARPS ? JD_WARPS / G : 1; }
 __host__ __device__ inline JointDecodeSmem joint_decode_smem(int H, int G, int HD) {
-  const int parts = G < JD_WARPS ? JD_WARPS / G : 1, h4 = (H + 3) / 4 * 4;
+  const bool res = joint_decode_resident(G, HD);
+  const int parts = joint_decode_parts(G, res), h4 = (H + 3) / 4 * 4;
   JointDecodeSmem m;
-  m.s = JD_WARPS * 2 * 16 * (HD * 2 + 16);
+  m.s = JD_WARPS * (res ? JD_PAGES : 2) * 16 * (HD * 2 + 16);
   m.o = m.s + H * JD_SROW * 4;
   m.mix = m.o + parts * H * HD * 4;
   m.p = m.mix + H * h4 * 4;
@@ -154,15 +172,16 @@ __host__ __device__ inline JointDecodeSmem joint_decode_smem(int H, int G, int H
 
 // grid (splits, T), the splits of a token one cluster.  A round covers 64 keys: every warp takes the scores of its key heads
 // (where there are fewer than eight, of some of their pages), the CTA mixes them and takes the softmax step, and every warp
-// reads its pages once more (out of the L2) as values.
-template <int HD>
-__global__ void __launch_bounds__(JD_WARPS * 32, HD <= 128 ? 2 : 1) joint_decode_kernel(const JointArgs a) {
-  constexpr int ROWB = HD * 2 + 16, STAGE = 16 * ROWB, KS = HD / 16, NT = HD / 8;
+// weighs its pages as values.  RES (up to eight key heads of up to 128 values): a warp's pages of a round stay in shared memory in between, and those
+// of the next round take their places one by one; else they pass through two places and are read a second time, out of the L2.
+template <int HD, bool RES>
+__global__ void __launch_bounds__(JD_WARPS * 32, (HD <= 128 && !RES) ? 2 : 1) joint_decode_kernel(const JointArgs a) {
+  constexpr int ROWB = HD * 2 + 16, STAGE = 16 * ROWB, KS = HD / 16, NT = HD / 8, STAGES = RES ? JD_PAGES : 2;
   extern __shared__ __align__(16) uint8_t jd_smem[];
   pdl_launch_dependents();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3, mi = lane >> 3, lr = lane & 7;
   const int t = blockIdx.y, split = blockIdx.x, splits = gridDim.x;
-  const int H = a.H, G = a.G, per = H / G, h4 = (H + 3) / 4 * 4, parts = G < JD_WARPS ? JD_WARPS / G : 1, units = G * parts;
+  const int H = a.H, G = a.G, per = H / G, h4 = (H + 3) / 4 * 4, parts = joint_decode_parts(G, RES), units = G * parts;
   const int b = sequence_of(a.query_start, a.B, t), rows = a.query_start[b + 1] - a.query_start[b];
   if (rows > a.max_rows) {  // (the whole cluster leaves)
     pdl_wait();
@@ -173,10 +192,10 @@ __global__ void __launch_bounds__(JD_WARPS * 32, HD <= 128 ? 2 : 1) joint_decode
   float *sS = reinterpret_cast<float*>(jd_smem + sm.s), *sO = reinterpret_cast<float*>(jd_smem + sm.o), *sMix = reinterpret_cast<float*>(jd_smem + sm.mix);
   __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(jd_smem + sm.p);
   float *m_run = reinterpret_cast<float*>(jd_smem + sm.stat), *l_run = m_run + h4, *corr = l_run + h4;
-  uint8_t* ring = jd_smem + warp * 2 * STAGE;
-  for (int i = tid; i < H * h4; i += JD_WARPS * 32) {  // [g][h]
+  uint8_t* ring = jd_smem + warp * STAGES * STAGE;
+  for (int i = tid; i < H * h4; i += JD_WARPS * 32) {  // [g][h], in binary logarithms
     const int g = i / h4, h = i % h4;
-    sMix[i] = h < H ? (a.mix != nullptr ? a.mix[h * H + g] : (g == h ? 1.f : 0.f)) : 0.f;
+    sMix[i] = h < H ? (a.mix != nullptr ? a.mix[h * H + g] : (g == h ? 1.f : 0.f)) * 1.4426950408889634f : 0.f;
   }
   for (int i = tid; i < parts * H * HD; i += JD_WARPS * 32) sO[i] = 0.f;
   if (tid < h4) {
@@ -189,104 +208,110 @@ __global__ void __launch_bounds__(JD_WARPS * 32, HD <= 128 ? 2 : 1) joint_decode
   const int share = (n_pages + splits - 1) / splits, p0 = split * share, p1 = min(n_pages, p0 + share);
   const int* bt = a.block_tables + (size_t)b * a.max_blocks;
   auto page_of = [&](int i) { return i < kept ? i : page_lo + i - kept; };
-  const float inv_cap2 = a.cap > 0.f ? 2.f / a.cap : 0.f;
-  int slot = 0;
-  auto load = [&](int r0, int u, int p) {
-    int blk = bt[page_of(r0 + p)];
+  const JointCap cap = joint_cap(a);
+  auto load = [&](int page, int u, int slot) {
+    int blk = bt[page_of(page)];
     if ((unsigned)blk >= (unsigned)a.num_blocks) {
       if (lane == 0) oxb_report(OXB_BAD_BLOCK_ID, blk);
       blk = 0;
     }
     joint_load_page<HD>(ring + slot * STAGE, a, blk, u / parts, lane);
   };
-  auto first_unit = [&](int npg, int& u, int& p) {  // (a warp without pages in this round: u = units)
-    u = warp;
-    p = u < units ? u % parts : 0;
-    if (u < units && p >= npg) u = units;
-  };
-  auto next_unit = [&](int npg, int& u, int& p) {
-    p += parts;
-    if (p >= npg) {
-      u += JD_WARPS;
-      p = u < units ? u % parts : 0;
-    }
-    if (u < units && p >= npg) u = units;
-  };
-  __syncthreads();
-  pdl_wait();
-  if (p0 < p1) {
-    int u, p;
-    first_unit(min(JD_PAGES, p1 - p0), u, p);
-    if (u < units) load(p0, u, p);
-  }
-  cp_async_commit();
-  for (int r0 = p0; r0 < p1; r0 += JD_PAGES) {
-    const int npg = min(JD_PAGES, p1 - r0);
-    // ---- scores
-    {
-      int u, p, held = -1;
-      uint32_t qf[KS][4];
-      first_unit(npg, u, p);
-      while (u < units) {
-        int nu = u, np = p;
-        next_unit(npg, nu, np);
-        slot ^= 1;
-        if (nu < units) load(r0, nu, np);
-        slot ^= 1;
-        cp_async_commit();
-        const int g = u / parts;
-        if (g != held) {
-          held = g;
-          const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.q) + ((size_t)t * H + g * per) * HD + 2 * t4;
+  uint32_t qf[KS][4];
+  auto load_q = [&](int g) {
+    const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.q) + ((size_t)t * H + g * per) * HD + 2 * t4;
 #pragma unroll
-          for (int ks = 0; ks < KS; ++ks)
+    for (int ks = 0; ks < KS; ++ks)
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
-              const bool on = g8 + 8 * i < per;
-              const __nv_bfloat16* qp = q + (size_t)(on ? g8 + 8 * i : 0) * HD + ks * 16;
-              qf[ks][i] = on ? *reinterpret_cast<const uint32_t*>(qp) : 0u;
-              qf[ks][i + 2] = on ? *reinterpret_cast<const uint32_t*>(qp + 8) : 0u;
-            }
-        }
-        cp_async_wait<1>();
-        __syncwarp();
-        const uint8_t* st = ring + slot * STAGE;
-        const uint32_t addr = smem_u32(st) + ((mi >> 1) * 8 + lr) * ROWB + (mi & 1) * 16;
-        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-#pragma unroll
-        for (int ks = 0; ks < KS; ++ks) {
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(addr + ks * 32, b0, b1, b2, b3);
-          mma_bf16_16816(s[0], qf[ks], b0, b1);
-          mma_bf16_16816(s[1], qf[ks], b2, b3);
-        }
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          const int key = nt * 8 + 2 * t4;
-          const float f0 = *reinterpret_cast<const float*>(st + key * ROWB + HD * 2) * a.scale;
-          const float f1 = *reinterpret_cast<const float*>(st + (key + 1) * ROWB + HD * 2) * a.scale;
-#pragma unroll
-          for (int i = 0; i < 2; ++i)
-            if (g8 + 8 * i < per)
-              *reinterpret_cast<float2*>(sS + (g * per + g8 + 8 * i) * JD_SROW + p * 16 + key) =
-                  make_float2(joint_capped_fast(s[nt][2 * i] * f0, a.cap, inv_cap2), joint_capped_fast(s[nt][2 * i + 1] * f1, a.cap, inv_cap2));
-        }
-        __syncwarp();
-        slot ^= 1;
-        u = nu;
-        p = np;
+      for (int i = 0; i < 2; ++i) {
+        const bool on = g8 + 8 * i < per;
+        const __nv_bfloat16* qp = q + (size_t)(on ? g8 + 8 * i : 0) * HD + ks * 16;
+        qf[ks][i] = on ? *reinterpret_cast<const uint32_t*>(qp) : 0u;
+        qf[ks][i + 2] = on ? *reinterpret_cast<const uint32_t*>(qp + 8) : 0u;
       }
-      first_unit(npg, u, p);  // the first page of the values is on its way during the mixing
-      if (u < units) load(r0, u, p);
-      cp_async_commit();
+  };
+  auto scores = [&](int g, int p, int slot) {
+    const uint8_t* st = ring + slot * STAGE;
+    const uint32_t addr = smem_u32(st) + ((mi >> 1) * 8 + lr) * ROWB + (mi & 1) * 16;
+    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) {
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4(addr + ks * 32, b0, b1, b2, b3);
+      mma_bf16_16816(s[0], qf[ks], b0, b1);
+      mma_bf16_16816(s[1], qf[ks], b2, b3);
     }
-    __syncthreads();
-    // ---- mixing and softmax: a warp has four heads and all keys, a lane keys `lane` and `lane` + 32
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      const int key = nt * 8 + 2 * t4;
+      const float f0 = *reinterpret_cast<const float*>(st + key * ROWB + HD * 2) * cap.factor;
+      const float f1 = *reinterpret_cast<const float*>(st + (key + 1) * ROWB + HD * 2) * cap.factor;
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        if (g8 + 8 * i < per)
+          *reinterpret_cast<float2*>(sS + (g * per + g8 + 8 * i) * JD_SROW + p * 16 + key) =
+              make_float2(joint_capped_fast(s[nt][2 * i], f0, cap), joint_capped_fast(s[nt][2 * i + 1], f1, cap));
+    }
+  };
+  float o[NT][4];
+  auto clear = [&]() {
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
+  };
+  auto values = [&](int g, int p, int slot) {
+    uint32_t pf[4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const bool on = g8 + 8 * i < per;
+      const __nv_bfloat16* src = sP + (g * per + (on ? g8 + 8 * i : 0)) * JD_PROW + p * 16 + 2 * t4;
+      pf[i] = on ? *reinterpret_cast<const uint32_t*>(src) : 0u;
+      pf[i + 2] = on ? *reinterpret_cast<const uint32_t*>(src + 8) : 0u;
+    }
+    const uint32_t addr = smem_u32(ring + slot * STAGE) + ((mi & 1) * 8 + lr) * ROWB + (mi >> 1) * 16;
+#pragma unroll
+    for (int nt = 0; nt < NT; nt += 2) {
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4_trans(addr + nt * 16, b0, b1, b2, b3);
+      mma_bf16_16816(o[nt], pf, b0, b1);
+      mma_bf16_16816(o[nt + 1], pf, b2, b3);
+    }
+  };
+  // O <- corr O + o; RES: a warp has one unit, whose O stays in o
+  auto flush = [&](int unit) {
+    const int g = unit / parts;
+    float* dst = sO + ((size_t)(unit % parts) * H + g * per) * HD + 2 * t4;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int r = g8 + 8 * i;
+      if (r >= per) continue;
+      const float c = RES ? 0.f : corr[g * per + r];
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        float2* at = reinterpret_cast<float2*>(dst + r * HD + nt * 8);
+        const float2 x = RES ? make_float2(0.f, 0.f) : *at;
+        *at = make_float2(fmaf(c, x.x, o[nt][2 * i]), fmaf(c, x.y, o[nt][2 * i + 1]));
+      }
+    }
+  };
+  // ---- mixing and softmax of a round: a warp has four heads and all keys, a lane keys `lane` and `lane` + 32
+  auto mix_round = [&](int r0, int npg) {
+    bool ok[2];
+    int dist[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int pg = (lane >> 4) + 2 * j, key = page_of(r0 + min(pg, npg - 1)) * 16 + (lane & 15);
+      ok[j] = pg < npg && key <= pos && (a.window <= 0 || key > pos - a.window || key < a.keep_first);
+      dist[j] = min(max(pos - key, 0), a.distances - 1);
+    }
     for (int h0 = 4 * warp; h0 < H; h0 += 4 * JD_WARPS) {
       float v[2][4];
 #pragma unroll
-      for (int j = 0; j < 2; ++j) v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.f;
-#pragma unroll 4
+      for (int i = 0; i < 4; ++i) {
+        const float* bias = a.bias + (size_t)min(h0 + i, H - 1) * a.distances;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) v[j][i] = a.bias != nullptr ? bias[dist[j]] * 1.4426950408889634f : 0.f;
+      }
+#pragma unroll 8
       for (int g = 0; g < H; ++g) {
         const float4 w = *reinterpret_cast<const float4*>(sMix + g * h4 + h0);
 #pragma unroll
@@ -298,104 +323,154 @@ __global__ void __launch_bounds__(JD_WARPS * 32, HD <= 128 ? 2 : 1) joint_decode
           v[j][3] = fmaf(w.w, x, v[j][3]);
         }
       }
-      bool ok[2];
-      int dist[2];
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int pg = (lane >> 4) + 2 * j, key = page_of(r0 + min(pg, npg - 1)) * 16 + (lane & 15);
-        ok[j] = pg < npg && key <= pos && (a.window <= 0 || key > pos - a.window || key < a.keep_first);
-        dist[j] = min(max(pos - key, 0), a.distances - 1);
-      }
+      float old[4], top[4], sum[4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int h = h0 + i;
-        if (h >= H) break;
-        float x[2];
+        v[0][i] = ok[0] ? v[0][i] : -INFINITY;
+        v[1][i] = ok[1] ? v[1][i] : -INFINITY;
+        old[i] = m_run[h0 + i];  // (rows up to h4 exist)
+        top[i] = fmaxf(v[0][i], v[1][i]);
+      }
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          const float bias = a.bias != nullptr ? a.bias[(size_t)h * a.distances + dist[j]] : 0.f;
-          x[j] = ok[j] ? (v[j][i] + bias) * 1.4426950408889634f : -INFINITY;
-        }
-        const float old = m_run[h], top = fmaxf(old, warp_max(fmaxf(x[0], x[1]))), base = top == -INFINITY ? 0.f : top;
-        const float y0 = exp2f(x[0] - base), y1 = exp2f(x[1] - base), sum = warp_sum(y0 + y1), c = exp2f(old - base);
-        sP[h * JD_PROW + lane] = __float2bfloat16(y0);
-        sP[h * JD_PROW + lane + 32] = __float2bfloat16(y1);
-        __syncwarp();
+      for (int d = 16; d > 0; d >>= 1)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) top[i] = fmaxf(top[i], __shfl_xor_sync(0xffffffffu, top[i], d));
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        top[i] = fmaxf(top[i], old[i]);
+        const float base = top[i] == -INFINITY ? 0.f : top[i];
+        v[0][i] = joint_exp2(v[0][i] - base);
+        v[1][i] = joint_exp2(v[1][i] - base);
+        old[i] = joint_exp2(old[i] - base);
+        sum[i] = v[0][i] + v[1][i];
+      }
+#pragma unroll
+      for (int d = 16; d > 0; d >>= 1)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], d);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (h0 + i >= H) continue;
+        sP[(h0 + i) * JD_PROW + lane] = __float2bfloat16(v[0][i]);
+        sP[(h0 + i) * JD_PROW + lane + 32] = __float2bfloat16(v[1][i]);
         if (lane == 0) {
-          m_run[h] = top;
-          l_run[h] = l_run[h] * c + sum;
-          corr[h] = c;
+          m_run[h0 + i] = top[i];
+          l_run[h0 + i] = l_run[h0 + i] * old[i] + sum[i];
+          corr[h0 + i] = old[i];
         }
       }
+      __syncwarp();
     }
-    __syncthreads();
-    // ---- values
-    {
-      int u, p;
-      float o[NT][4];
-      bool fresh = true;
-      auto flush = [&](int unit, bool any) {  // O <- corr O + o
-        const int g = unit / parts;
-        float* dst = sO + ((size_t)(unit % parts) * H + g * per) * HD + 2 * t4;
+  };
+  __syncthreads();
+  pdl_wait();
+  if constexpr (RES) {
+    const int u = warp, g = u / parts, part = u % parts;
+    const bool works = u < units;
+    clear();
+    // page k of a round (k-th of this warp's) lies in place k
+    auto mine = [&](int k, int r0) { return works && k * parts + part < min(JD_PAGES, p1 - r0); };
+#pragma unroll
+    for (int k = 0; k < JD_PAGES; ++k) {
+      if (p0 < p1 && mine(k, p0)) load(p0 + k * parts + part, u, k);
+      cp_async_commit();
+    }
+    if (works) load_q(g);
+    for (int r0 = p0; r0 < p1; r0 += JD_PAGES) {
+      const int npg = min(JD_PAGES, p1 - r0);
+      cp_async_wait<3>();
+      __syncwarp();
+      if (mine(0, r0)) scores(g, part, 0);
+      cp_async_wait<2>();
+      __syncwarp();
+      if (mine(1, r0)) scores(g, parts + part, 1);
+      cp_async_wait<1>();
+      __syncwarp();
+      if (mine(2, r0)) scores(g, 2 * parts + part, 2);
+      cp_async_wait<0>();
+      __syncwarp();
+      if (mine(3, r0)) scores(g, 3 * parts + part, 3);
+      __syncthreads();
+      mix_round(r0, npg);
+      __syncthreads();
+      if (works) {
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-          const int r = g8 + 8 * i;
-          if (r >= per) continue;
-          const float c = corr[g * per + r];
+          if (g8 + 8 * i >= per) continue;
+          const float c = corr[g * per + g8 + 8 * i];
 #pragma unroll
           for (int nt = 0; nt < NT; ++nt) {
-            float2* at = reinterpret_cast<float2*>(dst + r * HD + nt * 8);
-            const float2 x = *at;
-            *at = make_float2(fmaf(c, x.x, any ? o[nt][2 * i] : 0.f), fmaf(c, x.y, any ? o[nt][2 * i + 1] : 0.f));
+            o[nt][2 * i] *= c;
+            o[nt][2 * i + 1] *= c;
           }
         }
-      };
-      first_unit(npg, u, p);
-      if (u >= units && warp < units) flush(warp, false);  // (no page of its own in this round)
+      }
+#pragma unroll
+      for (int k = 0; k < JD_PAGES; ++k) {
+        if (mine(k, r0)) values(g, k * parts + part, k);
+        __syncwarp();
+        if (r0 + JD_PAGES < p1 && mine(k, r0 + JD_PAGES)) load(r0 + JD_PAGES + k * parts + part, u, k);
+        cp_async_commit();
+      }
+    }
+    if (works) flush(u);
+  } else {
+    int slot = 0;
+    auto first_unit = [&](int& u, int& p) {
+      u = warp;
+      p = 0;
+    };
+    auto next_unit = [&](int npg, int& u, int& p) {
+      if (++p >= npg) {
+        u += JD_WARPS;
+        p = 0;
+      }
+    };
+    if (p0 < p1 && warp < units) load(p0, warp, 0);
+    cp_async_commit();
+    for (int r0 = p0; r0 < p1; r0 += JD_PAGES) {
+      const int npg = min(JD_PAGES, p1 - r0);
+      int u, p, held = -1;
+      first_unit(u, p);
       while (u < units) {
         int nu = u, np = p;
         next_unit(npg, nu, np);
-        slot ^= 1;
-        if (nu < units) load(r0, nu, np);
-        slot ^= 1;
+        if (nu < units) load(r0 + np, nu, slot ^ 1);
         cp_async_commit();
-        if (fresh) {
-#pragma unroll
-          for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
-        }
-        const int g = u / parts;
-        uint32_t pf[4];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const bool on = g8 + 8 * i < per;
-          const __nv_bfloat16* src = sP + (g * per + (on ? g8 + 8 * i : 0)) * JD_PROW + p * 16 + 2 * t4;
-          pf[i] = on ? *reinterpret_cast<const uint32_t*>(src) : 0u;
-          pf[i + 2] = on ? *reinterpret_cast<const uint32_t*>(src + 8) : 0u;
-        }
+        if (u != held) load_q(held = u);
         cp_async_wait<1>();
         __syncwarp();
-        const uint32_t addr = smem_u32(ring + slot * STAGE) + ((mi & 1) * 8 + lr) * ROWB + (mi >> 1) * 16;
-#pragma unroll
-        for (int nt = 0; nt < NT; nt += 2) {
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(addr + nt * 16, b0, b1, b2, b3);
-          mma_bf16_16816(o[nt], pf, b0, b1);
-          mma_bf16_16816(o[nt + 1], pf, b2, b3);
-        }
+        scores(u, p, slot);
         __syncwarp();
         slot ^= 1;
-        fresh = nu != u;
-        if (fresh) flush(u, true);
         u = nu;
         p = np;
       }
-      if (r0 + JD_PAGES < p1) {
-        first_unit(min(JD_PAGES, p1 - r0 - JD_PAGES), u, p);
-        if (u < units) load(r0 + JD_PAGES, u, p);
-      }
+      if (warp < units) load(r0, warp, slot);  // the first page of the values is on its way during the mixing
       cp_async_commit();
+      __syncthreads();
+      mix_round(r0, npg);
+      __syncthreads();
+      first_unit(u, p);
+      while (u < units) {
+        int nu = u, np = p;
+        next_unit(npg, nu, np);
+        if (nu < units) load(r0 + np, nu, slot ^ 1);
+        cp_async_commit();
+        if (p == 0) clear();
+        cp_async_wait<1>();
+        __syncwarp();
+        values(u, p, slot);
+        __syncwarp();
+        slot ^= 1;
+        if (nu != u) flush(u);
+        u = nu;
+        p = np;
+      }
+      if (r0 + JD_PAGES < p1 && warp < units) load(r0 + JD_PAGES, warp, slot);
+      cp_async_commit();
+      // (the next round's scores overwrite sS, which nobody reads any more; its mixing starts behind a barrier)
     }
-    // (the next round's scores overwrite sS, which nobody reads any more; its mixing starts behind a barrier)
   }
   cp_async_wait<0>();
   __syncthreads();
@@ -422,9 +497,11 @@ __global__ void __launch_bounds__(JD_WARPS * 32, HD <= 128 ? 2 : 1) joint_decode
       L = w * l_run[h];
     } else {
       const uint32_t m_at = smem_u32(m_run + h), l_at = smem_u32(l_run + h), o_at = smem_u32(sO + 4 * i);
+#pragma unroll 4
       for (int r = 0; r < splits; ++r) M = fmaxf(M, dsmem_ld_f32(dsmem_map(m_at, r)));
       v = make_float4(0.f, 0.f, 0.f, 0.f);
       L = 0.f;
+#pragma unroll 4
       for (int r = 0; r < splits; ++r) {
         const float m = dsmem_ld_f32(dsmem_map(m_at, r)), w = m == -INFINITY ? 0.f : exp2f(m - M);
         const float4 x = dsmem_ld_f32x4(dsmem_map(o_at, r));

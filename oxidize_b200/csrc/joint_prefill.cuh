@@ -24,8 +24,8 @@ struct JointPrefillArgs {
   const int* block_seq;  // [blocks] sequence of every block of 16 tokens
   const int* block_row;  // [blocks] its first row
   const int* wide;       // [wide blocks, 2]: first block of 16, number of them (up to 8, of one sequence)
-  uint4* weights;        // [blocks, H, 16, tiles, 4]
-  float2* stats;         // [blocks, H, 16, tiles]: m, sum
+  uint4* weights;        // [blocks, tiles, H, 16, 4]
+  float2* stats;         // [blocks, tiles, H, 16]: m, sum
   int tiles;             // most tiles of a block
   int block0;            // the first block of this launch: scratch is numbered from there
 };
@@ -63,11 +63,11 @@ __global__ void __launch_bounds__(JP_WARPS * 32, 1) joint_scores_kernel(const Jo
   const JointSpan sp = joint_span(a, b, row0);
   uint8_t* ring = jp_smem + warp * 2 * STAGE;
   float* sS = reinterpret_cast<float*>(jp_smem + JP_WARPS * 2 * STAGE);  // [HP][16][40]
-  uint8_t* sMix = reinterpret_cast<uint8_t*>(sS + HP * JP_HEAD);          // [2 (hi, lo)][HP] rows of HP halves
+  uint8_t* sMix = reinterpret_cast<uint8_t*>(sS + HP * JP_HEAD);          // [2 (hi, lo)][HP] rows of HP halves, in binary logarithms
   for (int i = tid; i < HP * JP_HEAD; i += JP_WARPS * 32) sS[i] = 0.f;    // (heads that do not exist count for nothing)
   for (int i = tid; i < HP * HP; i += JP_WARPS * 32) {
     const int h = i / HP, g = i % HP;
-    const float w = (h < H && g < H) ? (a.mix != nullptr ? a.mix[h * H + g] : (g == h ? 1.f : 0.f)) : 0.f;
+    const float w = (h < H && g < H) ? (a.mix != nullptr ? a.mix[h * H + g] : (g == h ? 1.f : 0.f)) * 1.4426950408889634f : 0.f;
     const __nv_bfloat16 hi = __float2bfloat16(w);
     *reinterpret_cast<__nv_bfloat16*>(sMix + h * MIXB + g * 2) = hi;
     *reinterpret_cast<__nv_bfloat16*>(sMix + (HP + h) * MIXB + g * 2) = __float2bfloat16(w - __bfloat162float(hi));
@@ -101,7 +101,7 @@ __global__ void __launch_bounds__(JP_WARPS * 32, 1) joint_scores_kernel(const Jo
     }
     joint_load_page<HD>(ring + slot * STAGE, a, id, head / per, lane);
   };
-  const float inv_cap2 = a.cap > 0.f ? 2.f / a.cap : 0.f;
+  const JointCap cap = joint_cap(a);
   const int items = works ? n_tiles * ITEMS : 0;
   if (items > 0) load(0, 0);
   cp_async_commit();
@@ -113,8 +113,11 @@ __global__ void __launch_bounds__(JP_WARPS * 32, 1) joint_scores_kernel(const Jo
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int h = m * 16 + g8 + 8 * i;
-      far[m][i] = (a.bias != nullptr && h < H) ? a.bias[(size_t)h * a.distances + a.distances - 1] : 0.f;
+      far[m][i] = (a.bias != nullptr && h < H) ? a.bias[(size_t)h * a.distances + a.distances - 1] * 1.4426950408889634f : 0.f;
     }
+  // this lane's pieces of a tile: head 8 (2 m + e) further is 8 * 16 rows further
+  uint4* weights = x.weights + ((size_t)blockIdx.x * x.tiles * H + g8) * (JP_ROWS * 4) + warp * 4 + t4;
+  float2* stats = x.stats + ((size_t)blockIdx.x * x.tiles * H + g8) * JP_ROWS + warp;
   __syncthreads();
   for (int i = 0; i < n_tiles; ++i) {
     const int tile = tile_of(i);
@@ -148,8 +151,8 @@ __global__ void __launch_bounds__(JP_WARPS * 32, 1) joint_scores_kernel(const Jo
 #pragma unroll
           for (int nt = 0; nt < 2; ++nt) {
             const int key = nt * 8 + 2 * t4;
-            const float f0 = *reinterpret_cast<const float*>(st + key * ROWB + HD * 2) * a.scale;
-            const float f1 = *reinterpret_cast<const float*>(st + (key + 1) * ROWB + HD * 2) * a.scale;
+            const float f0 = *reinterpret_cast<const float*>(st + key * ROWB + HD * 2) * cap.factor;
+            const float f1 = *reinterpret_cast<const float*>(st + (key + 1) * ROWB + HD * 2) * cap.factor;
 #pragma unroll
             for (int j = 0; j < NH; ++j) {
               const int h = h0 + (SAME ? j : it % HPW);
@@ -157,7 +160,7 @@ __global__ void __launch_bounds__(JP_WARPS * 32, 1) joint_scores_kernel(const Jo
 #pragma unroll
               for (int e = 0; e < 2; ++e)
                 *reinterpret_cast<float2*>(sS + h * JP_HEAD + (g8 + 8 * e) * JP_QROW + half * 16 + key) =
-                    make_float2(joint_capped_fast(s[j][nt][2 * e] * f0, a.cap, inv_cap2), joint_capped_fast(s[j][nt][2 * e + 1] * f1, a.cap, inv_cap2));
+                    make_float2(joint_capped_fast(s[j][nt][2 * e], f0, cap), joint_capped_fast(s[j][nt][2 * e + 1], f1, cap));
             }
           }
         }
@@ -165,12 +168,16 @@ __global__ void __launch_bounds__(JP_WARPS * 32, 1) joint_scores_kernel(const Jo
       }
     }
     __syncthreads();
+    float acc[HPW][4][4];
+    const int key0 = tile * JP_KEYS;
+    const bool near = a.bias != nullptr && pos - key0 - (JP_KEYS - 1) < a.distances - 1;
     if (warp < sp.rows) {
-      float acc[HPW][4][4];
 #pragma unroll
       for (int m = 0; m < HPW; ++m)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[m][j][e] = near ? 0.f : far[m][e >> 1];
 #pragma unroll
       for (int ks = 0; ks < HPW; ++ks) {
         uint32_t wh[HPW][4], wl[HPW][4];
@@ -186,51 +193,80 @@ __global__ void __launch_bounds__(JP_WARPS * 32, 1) joint_scores_kernel(const Jo
           split_bf16x2(src[8 * j], src[JP_HEAD + 8 * j], bh[0], bl[0]);
           split_bf16x2(src[8 * JP_HEAD + 8 * j], src[9 * JP_HEAD + 8 * j], bh[1], bl[1]);
 #pragma unroll
-          for (int m = 0; m < HPW; ++m) {
-            mma_bf16_16816(acc[m][j], wh[m], bl[0], bl[1]);
-            mma_bf16_16816(acc[m][j], wl[m], bh[0], bh[1]);
-            mma_bf16_16816(acc[m][j], wh[m], bh[0], bh[1]);
-          }
+          for (int m = 0; m < HPW; ++m) mma_bf16_16816(acc[m][j], wh[m], bl[0], bl[1]);
+#pragma unroll
+          for (int m = 0; m < HPW; ++m) mma_bf16_16816(acc[m][j], wl[m], bh[0], bh[1]);
+#pragma unroll
+          for (int m = 0; m < HPW; ++m) mma_bf16_16816(acc[m][j], wh[m], bh[0], bh[1]);
         }
       }
-      const int key0 = tile * JP_KEYS;
-      const bool near = a.bias != nullptr && pos - key0 - (JP_KEYS - 1) < a.distances - 1;
+    }
+    __syncthreads();  // the scores are in registers: the next tile's may follow while this one's weights are made
+    if (warp < sp.rows) {
       const bool whole = key0 + JP_KEYS - 1 <= pos && (a.window <= 0 || key0 > pos - a.window || key0 + JP_KEYS <= a.keep_first);
+      if (near || !whole) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const int key = key0 + 8 * (j >> 1) + 2 * t4 + (j & 1), dist = min(max(pos - key, 0), a.distances - 1);
+          const bool ok = key <= pos && (a.window <= 0 || key > pos - a.window || key < a.keep_first);
+#pragma unroll
+          for (int m = 0; m < HPW; ++m)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              float& v = acc[m][j >> 1][2 * e + (j & 1)];
+              if (near) v = fmaf(a.bias[(size_t)min(m * 16 + g8 + 8 * e, H - 1) * a.distances + dist], 1.4426950408889634f, v);
+              v = ok ? v : -INFINITY;
+            }
+        }
+      }
+      float top[HPW][2], sum[HPW][2];
 #pragma unroll
       for (int m = 0; m < HPW; ++m)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int h = m * 16 + g8 + 8 * e;
-          const float* bias = a.bias + (size_t)min(h, H - 1) * a.distances;
-          float v[8], top = -INFINITY;
+          top[m][e] = -INFINITY;
 #pragma unroll
-          for (int j = 0; j < 8; ++j) {
-            const int key = key0 + 8 * (j >> 1) + 2 * t4 + (j & 1);
-            const float f = near ? bias[min(max(pos - key, 0), a.distances - 1)] : far[m][e];
-            v[j] = (acc[m][j >> 1][2 * e + (j & 1)] + f) * 1.4426950408889634f;
-            if (!whole && !(key <= pos && (a.window <= 0 || key > pos - a.window || key < a.keep_first))) v[j] = -INFINITY;
-            top = fmaxf(top, v[j]);
-          }
-          top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
-          top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
-          const float base = top == -INFINITY ? 0.f : ceilf(top);
-          float sum = 0.f;
-#pragma unroll
-          for (int j = 0; j < 8; ++j) {
-            v[j] = exp2f(v[j] - base);
-            sum += v[j];
-          }
-          sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-          sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-          if (h < H) {
-            const size_t at = (((size_t)blockIdx.x * H + h) * JP_ROWS + warp) * x.tiles + i;
-            x.weights[at * 4 + t4] =
-                make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
-            if (t4 == 0) x.stats[at] = make_float2(top == -INFINITY ? JP_NONE : base, sum);
-          }
+          for (int j = 0; j < 4; ++j) top[m][e] = fmaxf(top[m][e], fmaxf(acc[m][j][2 * e], acc[m][j][2 * e + 1]));
         }
+#pragma unroll
+      for (int d = 1; d < 4; d <<= 1)
+#pragma unroll
+        for (int m = 0; m < HPW; ++m)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) top[m][e] = fmaxf(top[m][e], __shfl_xor_sync(0xffffffffu, top[m][e], d));
+#pragma unroll
+      for (int m = 0; m < HPW; ++m)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float base = top[m][e] == -INFINITY ? 0.f : ceilf(top[m][e]);
+          top[m][e] = top[m][e] == -INFINITY ? JP_NONE : base;
+          float v[8];
+          sum[m][e] = 0.f;
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            v[j] = joint_exp2(acc[m][j >> 1][2 * e + (j & 1)] - base);
+            sum[m][e] += v[j];
+          }
+          if (m * 16 + 8 * e + g8 < H)
+            weights[(m * 16 + 8 * e) * (JP_ROWS * 4)] =
+                make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+        }
+#pragma unroll
+      for (int d = 1; d < 4; d <<= 1)
+#pragma unroll
+        for (int m = 0; m < HPW; ++m)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) sum[m][e] += __shfl_xor_sync(0xffffffffu, sum[m][e], d);
+      if (t4 == 0) {
+#pragma unroll
+        for (int m = 0; m < HPW; ++m)
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+            if (m * 16 + 8 * e + g8 < H) stats[(m * 16 + 8 * e) * JP_ROWS] = make_float2(top[m][e], sum[m][e]);
+      }
     }
-    __syncthreads();
+    weights += H * JP_ROWS * 4;
+    stats += H * JP_ROWS;
   }
 }
 
@@ -277,69 +313,71 @@ __global__ void __launch_bounds__(JV_WARPS * 32, 2) joint_values_kernel(const Jo
     if (i < n_tiles) load(i);
     cp_async_commit();
   }
-  const size_t rows_at = ((size_t)(blk - x.block0) * H + h) * JP_ROWS;
+  // this warp's weights and stats of a tile: 16 rows of 64 bytes, 16 pairs
+  const uint4* weights = x.weights + ((size_t)(blk - x.block0) * x.tiles * H + h) * (JP_ROWS * 4) + t4;
+  const float2* stats = x.stats + ((size_t)(blk - x.block0) * x.tiles * H + h) * JP_ROWS;
   const int own = sp.kept + sp.hi - sp.lo + 1;
-  if (works) {
+  if (works) {  // a lane has row lane % 16 and every other tile
     const float sink = a.sink != nullptr ? a.sink[h] * 1.4426950408889634f : -INFINITY;
-    for (int r = 0; r < sp.rows; ++r) {
-      const float2* st = x.stats + (rows_at + r) * x.tiles;
-      float M = sink == -INFINITY ? JP_NONE : ceilf(sink), L = 0.f;
-      for (int i = lane; i < own; i += 32) M = fmaxf(M, st[i].x);
-      M = warp_max(M);
-      for (int i = lane; i < own; i += 32) L += st[i].y * joint_pow2(st[i].x - M);
-      L = warp_sum(L);
-      if (sink != -INFINITY) L += exp2f(sink - M);
-      if (lane == 0) {
-        sM[r] = M;
-        sM[JP_ROWS + r] = L > 0.f ? a.out_scale / L : 0.f;
-      }
+    const bool on = (lane & 15) < sp.rows;
+    float M = sink == -INFINITY ? JP_NONE : ceilf(sink), L = 0.f;
+    for (int i = lane >> 4; i < own && on; i += 2) {
+      const float2 st = stats[(size_t)i * H * JP_ROWS + (lane & 15)];
+      const float top = fmaxf(M, st.x);
+      L = L * joint_pow2(M - top) + st.y * joint_pow2(st.x - top);
+      M = top;
+    }
+    const float other = __shfl_xor_sync(0xffffffffu, M, 16), top = fmaxf(M, other);
+    L *= joint_pow2(M - top);
+    L += __shfl_xor_sync(0xffffffffu, L, 16);
+    if (sink != -INFINITY) L += exp2f(sink - top);
+    if (lane < JP_ROWS) {
+      sM[lane] = top;
+      sM[JP_ROWS + lane] = L > 0.f ? a.out_scale / L : 0.f;
     }
     __syncwarp();
   }
   float o[NT][4];
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
-  float M[2];
-#pragma unroll
-  for (int e = 0; e < 2; ++e) M[e] = works && g8 + 8 * e < sp.rows ? sM[g8 + 8 * e] : 0.f;
+  const float M[2] = {works ? sM[g8] : 0.f, works ? sM[g8 + 8] : 0.f};
   // this warp's number of a tile, -1: not one of its own
   auto mine = [&](int i) {
     if (!works || i >= n_tiles) return -1;
     const int tile = tile_of(i);
     return tile < sp.kept ? tile : (tile >= sp.lo && tile <= sp.hi ? sp.kept + tile - sp.lo : -1);
   };
-  uint4 w[2];
-  float m[2];
-  auto fetch = [&](int i) {
+  uint4 w[2][2];
+  float m[2][2];
+  auto fetch = [&](int i, uint4 (&fw)[2], float (&fm)[2]) {
     const int k = mine(i);
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const bool on = k >= 0 && g8 + 8 * e < sp.rows;
-      const size_t at = (rows_at + (on ? g8 + 8 * e : 0)) * x.tiles + (on ? k : 0);
-      w[e] = on ? x.weights[at * 4 + t4] : make_uint4(0, 0, 0, 0);
-      m[e] = on ? x.stats[at].x : JP_NONE;
+      const size_t at = on ? (size_t)k * H * JP_ROWS + g8 + 8 * e : 0;
+      fw[e] = on ? weights[at * 4] : make_uint4(0, 0, 0, 0);
+      fm[e] = on ? stats[at].x : JP_NONE;
     }
   };
-  fetch(0);
-  for (int i = 0; i < n_tiles; ++i) {
+  auto step = [&](int i, uint4 (&fw)[2], float (&fm)[2]) {
     uint32_t p[2][4];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const float f = joint_pow2(m[e] - M[e]);
+      const float f = joint_pow2(fm[e] - M[e]);
       const __nv_bfloat162 f2 = __floats2bfloat162_rn(f, f);
-      const uint32_t src[4] = {w[e].x, w[e].y, w[e].z, w[e].w};
+      const uint32_t src[4] = {fw[e].x, fw[e].y, fw[e].z, fw[e].w};
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const __nv_bfloat162 y = __hmul2(*reinterpret_cast<const __nv_bfloat162*>(&src[j]), f2);
         p[e][j] = *reinterpret_cast<const uint32_t*>(&y);
       }
     }
-    fetch(i + 1);
+    fetch(i + 2, fw, fm);
     cp_async_wait<JV_STAGES - 2>();
     __syncthreads();
     if (i + JV_STAGES - 1 < n_tiles) load(i + JV_STAGES - 1);
     cp_async_commit();
-    if (mine(i) < 0) continue;
+    if (mine(i) < 0) return;
     const uint32_t addr = smem_u32(jv_smem + (i % JV_STAGES) * STAGE) + ((mi & 1) * 8 + lr) * ROWB + (mi >> 1) * 16;
 #pragma unroll
     for (int ks = 0; ks < 2; ++ks) {
@@ -352,6 +390,12 @@ __global__ void __launch_bounds__(JV_WARPS * 32, 2) joint_values_kernel(const Jo
         mma_bf16_16816(o[nt + 1], av, b2, b3);
       }
     }
+  };
+  fetch(0, w[0], m[0]);
+  fetch(1, w[1], m[1]);
+  for (int i = 0; i < n_tiles; i += 2) {
+    step(i, w[0], m[0]);
+    if (i + 1 < n_tiles) step(i + 1, w[1], m[1]);
   }
   if (!works) return;
 #pragma unroll

@@ -41,18 +41,18 @@ OXB_API int oxb_joint_simt(const void* q, void* out, int ld_out, float out_scale
 // ----------------------------------------------------------------------------- decoded tokens
 constexpr int JD_MAX_SPLITS = 16;  // clusters of more than 8 CTAs where the device takes them
 
-// Largest cluster of joint_decode_kernel<HD> with this much shared memory; sets the kernel up once per device.
-template <int HD>
+// Largest cluster of joint_decode_kernel; sets the kernel up once per device.
+template <int HD, bool RES>
 static int joint_decode_setup(int smem) {
   static int most[64] = {0};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return 0;
   if (most[dev] == 0) {
-    cudaError_t e = cudaFuncSetAttribute(joint_decode_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(joint_decode_kernel<HD, RES>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
     if (e != cudaSuccess) return 0;
     most[dev] = 8;
-    if (cudaFuncSetAttribute(joint_decode_kernel<HD>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
+    if (cudaFuncSetAttribute(joint_decode_kernel<HD, RES>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess) {
       cudaLaunchConfig_t cfg = {};
       cfg.gridDim = dim3(JD_MAX_SPLITS, 1, 1);
       cfg.blockDim = dim3(JD_WARPS * 32);
@@ -65,24 +65,32 @@ static int joint_decode_setup(int smem) {
       cfg.attrs = &at;
       cfg.numAttrs = 1;
       int n = 0;
-      if (cudaOccupancyMaxActiveClusters(&n, joint_decode_kernel<HD>, &cfg) == cudaSuccess && n > 0) most[dev] = JD_MAX_SPLITS;
+      if (cudaOccupancyMaxActiveClusters(&n, joint_decode_kernel<HD, RES>, &cfg) == cudaSuccess && n > 0) most[dev] = JD_MAX_SPLITS;
     }
     cudaGetLastError();
   }
   return smem > 227 * 1024 ? 0 : most[dev];
 }
 
-template <int HD>
-static int joint_decode_go(const JointArgs& a, int splits, cudaStream_t stream) {
-  const int smem = joint_decode_smem(a.H, a.G, HD).total, most = joint_decode_setup<HD>(smem);
+template <int HD, bool RES>
+static int joint_decode_launch(const JointArgs& a, int splits, cudaStream_t stream) {
+  const int smem = joint_decode_smem(a.H, a.G, HD).total, most = joint_decode_setup<HD, RES>(smem);
   if (most == 0) return (int)cudaErrorInvalidValue;
   if (splits > most) splits = most;
   const dim3 grid(splits, a.T), block(JD_WARPS * 32);
-  const cudaError_t e = splits > 1 ? oxb_launch_cluster(joint_decode_kernel<HD>, grid, block, dim3(splits, 1, 1), (size_t)smem, stream, a)
-                                   : oxb_launch(joint_decode_kernel<HD>, grid, block, (size_t)smem, stream, a);
+  const cudaError_t e = splits > 1 ? oxb_launch_cluster(joint_decode_kernel<HD, RES>, grid, block, dim3(splits, 1, 1), (size_t)smem, stream, a)
+                                   : oxb_launch(joint_decode_kernel<HD, RES>, grid, block, (size_t)smem, stream, a);
   if (e != cudaSuccess) return (int)e;
   OXB_CHECK_LAUNCH();
   return 0;
+}
+
+template <int HD>
+static int joint_decode_go(const JointArgs& a, int splits, cudaStream_t stream) {
+  if constexpr (HD <= 128) {
+    if (joint_decode_resident(a.G, HD)) return joint_decode_launch<HD, true>(a, splits, stream);
+  }
+  return joint_decode_launch<HD, false>(a, splits, stream);
 }
 
 // 1 when joint_decode_kernel covers these heads (bf16, pages of 16 tokens)

@@ -49,9 +49,9 @@ def attention_simt(q, kv, layer: int, meta, spec, bias, mix, sink, out, out_scal
                                 max_rows, _stream()), "oxb_joint_simt")
 
 
-def decode_splits(tokens: int, span: int, sms: int) -> int:
-    """CTAs that share a token's keys: two per SM in all, two pages or more each."""
-    return max(1, min(2 * sms // max(1, tokens), (span // 16 + 1) // 2, 16 if tokens <= 2 else 8))
+def decode_splits(tokens: int, span: int, sms: int, per_sm: int) -> int:
+    """CTAs that share a token's keys: ``per_sm`` per SM in all, two pages or more each."""
+    return max(1, min(per_sm * sms // max(1, tokens), (span // 16 + 1) // 2, 16 if tokens <= 2 else 8))
 
 
 def attention_decode(q, kv, layer: int, meta, spec, bias, mix, sink, out, out_scale: float, max_rows: int = _ALL,
@@ -60,7 +60,7 @@ def attention_decode(q, kv, layer: int, meta, spec, bias, mix, sink, out, out_sc
         span = meta.max_seq_len or kv.page_size
         if spec.window > 0:
             span = min(span, spec.window + spec.keep_first)
-        splits = decode_splits(q.shape[0], span, opcuda.sm_count(q.device))
+        splits = decode_splits(q.shape[0], span, opcuda.sm_count(q.device), 1 if spec.kv_heads <= 8 else 2)
     _check(lib().oxb_joint_decode(*_head(q, kv, layer, out, out_scale), *_tail(q, kv, meta, spec, bias, mix, sink), max_rows, splits,
                                   _stream()), "oxb_joint_decode")
 
