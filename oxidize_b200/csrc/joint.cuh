@@ -127,6 +127,12 @@ __device__ __forceinline__ float joint_exp2(float x) {  // 0 where that is no no
   return y;
 }
 
+__device__ __forceinline__ float joint_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // cap tanh(f s / cap) for scores of bfloat16 factors, tanh(x) = 1 - 2 / (1 + exp(2 x)): `f` carries the factor 2 log2(e) / cap
 // (joint_factor), absolute error about 1e-7 cap.
 struct JointCap {
@@ -135,9 +141,9 @@ struct JointCap {
 __device__ __forceinline__ JointCap joint_cap(const JointArgs& a) {
   return JointCap{a.cap, a.cap > 0.f ? a.scale * 2.f * 1.4426950408889634f / a.cap : a.scale};
 }
+__device__ __forceinline__ float joint_capped_of(float x, const JointCap& c) { return fmaf(-2.f * c.cap, joint_rcp(1.f + joint_exp2(x)), c.cap); }
 __device__ __forceinline__ float joint_capped_fast(float s, float f, const JointCap& c) {
-  if (c.cap <= 0.f) return s * f;
-  return fmaf(-2.f * c.cap, __fdividef(1.f, 1.f + joint_exp2(s * f)), c.cap);
+  return c.cap > 0.f ? joint_capped_of(s * f, c) : s * f;
 }
 
 // A page of one key head: 16 rows of HD values and their tails, as it stands in the cache (rows HD * 2 + 16 bytes apart, which

@@ -476,7 +476,7 @@ def _synth_output_normed(spec, h: int, mat, ones) -> LayerWeights:
         kw = wkv_weights(k, t, t["r"].dtype)
     else:
         att = {"q": mat(a.heads * a.dim, h), "k": mat(a.kv_heads * a.dim, h), "o": mat(h, a.heads * a.dim),
-               "rel": mat(a.bias_rows, a.heads).float(), "talk": torch.diag(ones(a.heads)) + mat(a.heads, a.heads).float()}
+               "rel": mat(a.bias_rows, a.heads).float(), "talk": (torch.diag(ones(a.heads)) + mat(a.heads, a.heads).float()).bfloat16()}
         att.update({n + ".b": 0.1 * ones(att[n].shape[0]) for n in "qk"})
         kw = listed_mixer(spec, att, {})
     lw = LayerWeights(attn_norm=None, post_attn_norm=ones(h), ffn_norm=None, **kw)
