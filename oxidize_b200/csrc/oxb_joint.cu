@@ -121,31 +121,38 @@ OXB_API int oxb_joint_decode(const void* q, void* out, int ld_out, float out_sca
 }
 
 // ----------------------------------------------------------------------------- long portions
-template <int HD, int HPW, bool SAME>
-static int joint_prefill_go(const JointPrefillArgs& x, int blocks, int wide_blocks, cudaStream_t stream) {
-  const int scores = joint_scores_smem(HD, HPW), values = joint_values_smem(HD);
+template <int HD, bool SAME>
+static int joint_prefill_go(const JointPrefillArgs& x, int wide_blocks, cudaStream_t stream) {
+  constexpr int scores = joint_scores_smem<HD, SAME>();
+  const int values = joint_values_smem(HD), quads = (x.a.H + 3) / 4;
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
   if (!configured[dev]) {
     constexpr cudaFuncAttribute attr = cudaFuncAttributeMaxDynamicSharedMemorySize;
-    cudaError_t e = cudaFuncSetAttribute(joint_scores_kernel<HD, HPW, SAME>, attr, scores);
+    cudaError_t e = cudaFuncSetAttribute(joint_scores_kernel<HD, SAME>, attr, scores);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(joint_values_kernel<HD>, attr, values);
     if (e != cudaSuccess) return (int)e;
     configured[dev] = true;
   }
-  cudaError_t e = oxb_launch(joint_scores_kernel<HD, HPW, SAME>, dim3(blocks), dim3(JP_WARPS * 32), (size_t)scores, stream, x);
+  // the tiles of 64 tokens are dealt out to as many CTAs as run at once
+  int parts = 2 * oxb_sm_count() / (2 * wide_blocks * quads);
+  if (parts > x.tiles / 4) parts = x.tiles / 4;
+  if (parts < 1) parts = 1;
+  const dim3 mix((unsigned)x.blocks * 2, (x.tiles + JM_TILES - 1) / JM_TILES);
+  cudaError_t e = oxb_launch(joint_scores_kernel<HD, SAME>, dim3(2 * wide_blocks, quads, parts), dim3(JC_WARPS * 32), (size_t)scores, stream, x);
+  if (e == cudaSuccess)
+    e = x.a.H <= 16 ? oxb_launch(joint_mix_kernel<1>, mix, dim3(JM_WARPS * 32), 0, stream, x)
+                    : oxb_launch(joint_mix_kernel<2>, mix, dim3(JM_WARPS * 32), 0, stream, x);
   if (e == cudaSuccess) e = oxb_launch(joint_values_kernel<HD>, dim3(wide_blocks, x.a.H), dim3(JV_WARPS * 32), (size_t)values, stream, x);
   if (e != cudaSuccess) return (int)e;
   OXB_CHECK_LAUNCH();
   return 0;
 }
 template <int HD>
-static int joint_prefill_heads(const JointPrefillArgs& x, int blocks, int wide_blocks, cudaStream_t stream) {
-  if (x.a.H <= 16) return joint_prefill_go<HD, 1, true>(x, blocks, wide_blocks, stream);
-  if (x.a.H / x.a.G % 2 == 0) return joint_prefill_go<HD, 2, true>(x, blocks, wide_blocks, stream);
-  return joint_prefill_go<HD, 2, false>(x, blocks, wide_blocks, stream);
+static int joint_prefill_heads(const JointPrefillArgs& x, int wide_blocks, cudaStream_t stream) {
+  return x.a.H / x.a.G % 4 == 0 ? joint_prefill_go<HD, true>(x, wide_blocks, stream) : joint_prefill_go<HD, false>(x, wide_blocks, stream);
 }
 
 // 1 when the kernels for long portions cover these heads (bf16, pages of 16 tokens)
@@ -154,26 +161,29 @@ OXB_API int oxb_joint_prefill_supported(int H, int G, int W) {
 }
 
 // The same in bf16 on pages of 16 tokens for the given blocks of 16 tokens (block0 .. block0 + blocks, of long portions), which
-// wide [wide_blocks, 2] groups by up to eight of one sequence; scratch weights blocks * H * 16 * tiles * 64 bytes and stats
-// blocks * H * 16 * tiles * 8 bytes, tiles: the most tiles of 32 keys that a block sees.
+// wide [wide_blocks, 2] groups by up to eight of one sequence; scratch scores blocks * (H / 4 rounded up) *
+// tiles * 8192 bytes, weights blocks * H * 16 * tiles * 64 bytes and stats blocks * H * 16 * tiles * 8 bytes, tiles: the most tiles
+// of 32 keys that a block sees.
 OXB_API int oxb_joint_prefill(const void* q, void* out, int ld_out, float out_scale, const void* cache, const int* block_tables,
                               const int* seq_lens, const int* query_start, const float* sink, const float* mix, const float* bias,
                               int distances, int B, int max_blocks, int T, int H, int G, int W, int tail, int page, int num_blocks,
                               int window, int keep_first, float scale, float cap, const int* block_seq, const int* block_row,
-                              const int* wide, int block0, int blocks, int wide_blocks, void* weights, void* stats, int tiles,
-                              cudaStream_t stream) {
+                              const int* wide, int block0, int blocks, int wide_blocks, void* scores, void* weights, void* stats,
+                              int tiles, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || blocks <= 0 || wide_blocks <= 0) return 0;
   const JointArgs a{q, out, ld_out, out_scale, cache, block_tables, seq_lens, query_start, sink, mix, bias, distances,
                     B, max_blocks, T, H, G, W, tail, page, num_blocks, window, keep_first, scale, cap, 0};
   if (joint_check(a) || !oxb_joint_prefill_supported(H, G, W) || page != 16 || tail != 8 || tiles <= 0 || ld_out % 2 != 0 ||
       (reinterpret_cast<uintptr_t>(out) & 3) != 0 ||
-      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(weights) | reinterpret_cast<uintptr_t>(stats)) & 15) != 0)
+      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(scores) | reinterpret_cast<uintptr_t>(weights) |
+        reinterpret_cast<uintptr_t>(stats)) & 15) != 0)
     return (int)cudaErrorInvalidValue;
-  const JointPrefillArgs x{a, block_seq, block_row, wide, reinterpret_cast<uint4*>(weights), reinterpret_cast<float2*>(stats), tiles, block0};
+  const JointPrefillArgs x{a, block_seq, block_row, wide, reinterpret_cast<uint4*>(scores), reinterpret_cast<uint4*>(weights),
+                           reinterpret_cast<float2*>(stats), tiles, block0, blocks};
   switch (W) {
-    case 32: return joint_prefill_heads<32>(x, blocks, wide_blocks, stream);
-    case 64: return joint_prefill_heads<64>(x, blocks, wide_blocks, stream);
-    case 96: return joint_prefill_heads<96>(x, blocks, wide_blocks, stream);
-    default: return joint_prefill_heads<128>(x, blocks, wide_blocks, stream);
+    case 32: return joint_prefill_heads<32>(x, wide_blocks, stream);
+    case 64: return joint_prefill_heads<64>(x, wide_blocks, stream);
+    case 96: return joint_prefill_heads<96>(x, wide_blocks, stream);
+    default: return joint_prefill_heads<128>(x, wide_blocks, stream);
   }
 }

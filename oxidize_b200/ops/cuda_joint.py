@@ -27,7 +27,7 @@ def lib():
         head, tail = [vp, vp, i32, f32, vp], [vp] * 6 + [i32] * 12 + [f32, f32]
         L.oxb_joint_simt.argtypes = head + [i32] + tail + [i32, vp]
         L.oxb_joint_decode.argtypes = head + tail + [i32, i32, vp]
-        L.oxb_joint_prefill.argtypes = head + tail + [vp, vp, vp, i32, i32, i32, vp, vp, i32, vp]
+        L.oxb_joint_prefill.argtypes = head + tail + [vp, vp, vp, i32, i32, i32, vp, vp, vp, i32, vp]
         L.oxb_joint_decode_supported.argtypes = L.oxb_joint_prefill_supported.argtypes = [i32] * 3
         _declared = True
     return L
@@ -105,17 +105,17 @@ def attention_prefill(q, kv, layer: int, meta, spec, bias, mix, sink, out, out_s
     seq, row, wide_dev, wide = _blocks(meta, long_rows)
     H = q.shape[1]
     tiles = most_tiles(meta.host_lens, spec.window, spec.keep_first, long_rows)
-    per_block = H * BLOCK * tiles
-    groups = max(1, scratch // (WIDE * per_block * 72))
-    n = min(groups * WIDE, len(seq)) * per_block
-    weights = torch.empty(n * 64, dtype=torch.uint8, device=q.device)
-    stats = torch.empty(n, 2, dtype=torch.float32, device=q.device)
+    quads = -(-H // 4)
+    groups = max(1, scratch // (WIDE * tiles * (quads * 8192 + H * BLOCK * 72)))
+    n = min(groups * WIDE, len(seq)) * tiles
+    new = lambda size: torch.empty(n * size, dtype=torch.uint8, device=q.device)
+    scores, weights, stats = new(quads * 8192), new(H * BLOCK * 64), new(H * BLOCK * 8)
     for w0 in range(0, len(wide), groups):
         part = wide[w0 : w0 + groups]
         b0, b1 = part[0][0], part[-1][0] + part[-1][1]
         _check(lib().oxb_joint_prefill(*_head(q, kv, layer, out, out_scale), *_tail(q, kv, meta, spec, bias, mix, sink), seq.data_ptr(),
-                                       row.data_ptr(), wide_dev[2 * w0 :].data_ptr(), b0, b1 - b0, len(part), weights.data_ptr(),
-                                       stats.data_ptr(), tiles, _stream()), "oxb_joint_prefill")
+                                       row.data_ptr(), wide_dev[2 * w0 :].data_ptr(), b0, b1 - b0, len(part), scores.data_ptr(),
+                                       weights.data_ptr(), stats.data_ptr(), tiles, _stream()), "oxb_joint_prefill")
 
 
 def attention(q, kv, layer: int, meta, spec, bias: Optional[torch.Tensor], mix: Optional[torch.Tensor], sink: Optional[torch.Tensor],
