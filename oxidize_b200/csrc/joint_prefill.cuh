@@ -403,11 +403,18 @@ __global__ void __launch_bounds__(JV_WARPS * 32, 2) joint_values_kernel(const Jo
     const float sink = a.sink != nullptr ? a.sink[h] * 1.4426950408889634f : -INFINITY;
     const bool on = (lane & 15) < sp.rows;
     float M = sink == -INFINITY ? JP_NONE : ceilf(sink), L = 0.f;
-    for (int i = lane >> 4; i < own && on; i += 2) {
-      const float2 st = stats[(size_t)i * H * JP_ROWS + (lane & 15)];
-      const float top = fmaxf(M, st.x);
-      L = L * joint_pow2(M - top) + st.y * joint_pow2(st.x - top);
+    for (int i0 = lane >> 4; i0 < own && on; i0 += 16) {
+      float2 st[8];
+      float top = M;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        st[j] = i0 + 2 * j < own ? stats[(size_t)(i0 + 2 * j) * H * JP_ROWS + (lane & 15)] : make_float2(JP_NONE, 0.f);
+        top = fmaxf(top, st[j].x);
+      }
+      L *= joint_pow2(M - top);
       M = top;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) L = fmaf(st[j].y, joint_pow2(st[j].x - top), L);
     }
     const float other = __shfl_xor_sync(0xffffffffu, M, 16), top = fmaxf(M, other);
     L *= joint_pow2(M - top);

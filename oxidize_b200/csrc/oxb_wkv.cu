@@ -73,7 +73,7 @@ static int wkv_step_launch(const WkvArgs& a, int B, cudaStream_t stream) {
 
 template <int KT>
 static int wkv_chunk_go(WkvChunkArgs x, int B, int longest, cudaStream_t stream) {
-  constexpr int K = KT * 16, MT = (K / 16 + 3) / 4;
+  constexpr int K = KT * 16, MT = (K / 16 + WST_WARPS - 1) / WST_WARPS;
   const int chunks = (longest + WC - 1) / WC, state = wkv_state_smem(K), output = wkv_output_smem(K).total;
   static bool configured[64] = {false};
   int dev = 0;

@@ -31,22 +31,24 @@ struct WkvChunkArgs {
   int chunk0, round;  // chunks [chunk0, chunk0 + round) of every portion
 };
 
-constexpr int WST_THREADS = 128;
-__host__ __device__ inline int wkv_state_smem(int K) { return 2 * WC * (K * 2 + 16) + 2 * WC * (WC_CH * 2 + 16) + 8 * WC_CH * 4; }
+constexpr int WST_WARPS = 8, WST_THREADS = WST_WARPS * 32, WST_ROWS = WC / WST_WARPS;  // tokens per warp
+__host__ __device__ inline int wkv_state_smem(int K) {
+  return 2 * WC * (K * 2 + 16) + 2 * WC * (WC_CH * 2 + 16) + 2 * (WST_WARPS + 1) * WC_CH * 4;
+}
 
-// This thread's 16 tokens from t0 on of channel `col`: logarithms and keys, zeros past the portion.
+// This thread's tokens from t0 on of channel `col`: logarithms and keys, zeros past the portion.
 __device__ __forceinline__ void wkv_fetch(const WkvArgs& a, const __nv_bfloat16* z, const float* decay, int t0, int n, int col, float* l,
                                           __nv_bfloat16* k) {
   const size_t hk = (size_t)a.H * a.K;
 #pragma unroll
-  for (int i = 0; i < 16; ++i) {
+  for (int i = 0; i < WST_ROWS; ++i) {
     const bool have = t0 + i < n;
     l[i] = have ? decay[(size_t)(t0 + i) * hk + col] : 0.f;
     k[i] = have ? z[(size_t)(t0 + i) * a.ld + hk + col] : __float2bfloat16(0.f);
   }
 }
 
-// grid (K / 32, H, B).  Every warp owns 16 MT values of a head (MT * 64 = V rounded up).
+// grid (K / 32, H, B).  Every warp owns 16 MT values of a head (MT * 128 = V rounded up).
 template <int MT>
 __global__ void __launch_bounds__(WST_THREADS) wkv_state_kernel(const WkvChunkArgs x) {
   extern __shared__ __align__(16) uint8_t wst_smem[];
@@ -62,7 +64,7 @@ __global__ void __launch_bounds__(WST_THREADS) wkv_state_kernel(const WkvChunkAr
   const int RV = V * 2 + 16, RK = WC_CH * 2 + 16, vtiles = V / 16;
   uint8_t* sv = wst_smem;                   // [2][64] rows of V halves
   uint8_t* skh = sv + 2 * WC * RV;          // [2 (hi, lo)][64] rows of 32 halves
-  float* total = reinterpret_cast<float*>(skh + 2 * WC * RK);  // [2][4][32] logarithms of the blocks' decays
+  float* total = reinterpret_cast<float*>(skh + 2 * WC * RK);  // [2][8 + 1][32] logarithms of what the warps' tokens decay by, and the chunk's decay
   float* S0 = a.state + ((size_t)slot * a.H + h) * K * V;
   const bool fresh = a.seq_lens[b] == n_all && x.chunk0 == 0;
   const size_t hk = (size_t)a.H * K;
@@ -89,13 +91,14 @@ __global__ void __launch_bounds__(WST_THREADS) wkv_state_kernel(const WkvChunkAr
       else *reinterpret_cast<uint4*>(dst + r * RV + p * 16) = make_uint4(0, 0, 0, 0);
     }
   };
-  float l[16];
-  __nv_bfloat16 k[16];
-  wkv_fetch(a, z, decay, c0 + warp * 16, n_all, col, l, k);
+  float l2[2][WST_ROWS];  // two chunks' inputs on their way
+  __nv_bfloat16 k2[2][WST_ROWS];
+  wkv_fetch(a, z, decay, c0 + warp * WST_ROWS, n_all, col, l2[0], k2[0]);
+  wkv_fetch(a, z, decay, c0 + WC + warp * WST_ROWS, n_all, col, l2[1], k2[1]);
   load_v(0);
   cp_async_commit();
   uint4* ws = x.ws + ((size_t)b * x.round * a.H + h) * (K * V / 4);
-  for (int c = 0; c < chunks; ++c) {
+  auto chunk = [&](int c, float (&l)[WST_ROWS], __nv_bfloat16 (&k)[WST_ROWS]) {
     // ---- the state in front of the chunk, as operand registers: (channels 16 j .., values 8 n ..) of this lane
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
@@ -112,46 +115,40 @@ __global__ void __launch_bounds__(WST_THREADS) wkv_state_kernel(const WkvChunkAr
         }
     }
     ws += (size_t)a.H * (K * V / 4);
-    // ---- running sums of this thread's 16 tokens; the keys relative to the end of the chunk
+    // ---- running sums of this thread's tokens; the keys relative to the end of the chunk
     float sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < WST_ROWS; ++i) {
       sum += fmaxf(l[i] * 1.4426950408889634f, DP_FLOOR);
       l[i] = sum;
     }
-    float* tot = total + (c & 1) * 4 * WC_CH;
+    float* tot = total + (c & 1) * (WST_WARPS + 1) * WC_CH;
     tot[warp * WC_CH + lane] = sum;
     __syncthreads();  // (also: every warp is done with the previous chunk's operands)
     float rest = sum;
-    for (int i = warp + 1; i < 4; ++i) rest += tot[i * WC_CH + lane];
+    for (int i = warp + 1; i < WST_WARPS; ++i) rest += tot[i * WC_CH + lane];
+    if (warp == 0) tot[WST_WARPS * WC_CH + lane] = delta_exp2(rest);
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
+    for (int i = 0; i < WST_ROWS; ++i) {
       const float y = __bfloat162float(k[i]) * delta_exp2(rest - l[i]);
       const __nv_bfloat16 hi = __float2bfloat16(y);
-      uint8_t* at = skh + (warp * 16 + i) * RK + lane * 2;
+      uint8_t* at = skh + (warp * WST_ROWS + i) * RK + lane * 2;
       *reinterpret_cast<__nv_bfloat16*>(at) = hi;
       *reinterpret_cast<__nv_bfloat16*>(at + WC * RK) = __float2bfloat16(y - __bfloat162float(hi));
     }
     cp_async_wait<0>();
     __syncthreads();
-    if (c + 1 < chunks) {  // the next chunk's inputs are on their way during the products
-      wkv_fetch(a, z, decay, c0 + (c + 1) * WC + warp * 16, n_all, col, l, k);
-      load_v(c + 1);
-    }
+    if (c + 2 < chunks) wkv_fetch(a, z, decay, c0 + (c + 2) * WC + warp * WST_ROWS, n_all, col, l, k);
+    if (c + 1 < chunks) load_v(c + 1);
     cp_async_commit();
     // ---- S' = exp(G_end) S + V^T k
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      float d[2];
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int o = 8 * i + 2 * t4 + e;
-        d[e] = delta_exp2((tot[o] + tot[WC_CH + o]) + (tot[2 * WC_CH + o] + tot[3 * WC_CH + o]));
-      }
+      const float2 d = *reinterpret_cast<const float2*>(tot + WST_WARPS * WC_CH + 8 * i + 2 * t4);
 #pragma unroll
       for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[m][i][e] *= d[e & 1];
+        for (int e = 0; e < 4; ++e) s[m][i][e] *= e & 1 ? d.y : d.x;
     }
     const uint32_t v_base = smem_u32(sv + (c & 1) * WC * RV), k_base = smem_u32(skh);
     const int mi = lane >> 3, r = lane & 7;
@@ -177,6 +174,10 @@ __global__ void __launch_bounds__(WST_THREADS) wkv_state_kernel(const WkvChunkAr
         }
       }
     }
+  };
+  for (int c = 0; c < chunks; c += 2) {
+    chunk(c, l2[0], k2[0]);
+    if (c + 1 < chunks) chunk(c + 1, l2[1], k2[1]);
   }
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -403,9 +404,16 @@ __global__ void __launch_bounds__(WO_THREADS, 2) wkv_output_kernel(const WkvChun
     }
     delta_split8(v, at_hi, at_lo);
   }
+  const int nt0 = warp * NT;  // (warps past the last value have nothing to multiply)
+  constexpr int AHEAD = KT < 4 ? KT : 4;  // k-steps of the state on their way
+  const uint4* ws = x.ws + (((size_t)b * x.round + blockIdx.x) * a.H + h) * (K * V / 4) + lane;
+  uint4 s[AHEAD][NT];
+#pragma unroll
+  for (int ks = 0; ks < AHEAD; ++ks)
+#pragma unroll
+    for (int i = 0; i < NT; ++i) s[ks][i] = ws[((size_t)ks * (V / 8) + min(nt0 + i, V / 8 - 1)) * 32];
   cp_async_wait<0>();
   __syncthreads();
-  const int nt0 = warp * NT;  // (warps past the last value have nothing to multiply)
   float o[4][NT][4];
 #pragma unroll
   for (int m = 0; m < 4; ++m)
@@ -434,13 +442,9 @@ __global__ void __launch_bounds__(WO_THREADS, 2) wkv_output_kernel(const WkvChun
         }
       }
     }
-    const uint4* ws = x.ws + (((size_t)b * x.round + blockIdx.x) * a.H + h) * (K * V / 4) + lane;
     const uint32_t r_at = smem_u32(sRR) + ((mi & 1) * 8 + lr) * RB + (mi >> 1) * 16;
-#pragma unroll 2
-    for (int ks = 0; ks < KT; ++ks) {
-      uint4 s[NT];
 #pragma unroll
-      for (int i = 0; i < NT; ++i) s[i] = ws[((size_t)ks * (V / 8) + min(nt0 + i, V / 8 - 1)) * 32];
+    for (int ks = 0; ks < KT; ++ks) {
 #pragma unroll
       for (int m = 0; m < 4; ++m) {
         uint32_t ah[4], al[4];
@@ -448,10 +452,15 @@ __global__ void __launch_bounds__(WO_THREADS, 2) wkv_output_kernel(const WkvChun
         ldmatrix_x4(r_at + HALF + m * 16 * RB + ks * 32, al[0], al[1], al[2], al[3]);
 #pragma unroll
         for (int i = 0; i < NT; ++i) {
-          mma_bf16_16816(o[m][i], ah, s[i].z, s[i].w);
-          mma_bf16_16816(o[m][i], al, s[i].x, s[i].y);
-          mma_bf16_16816(o[m][i], ah, s[i].x, s[i].y);
+          const uint4 v = s[ks % AHEAD][i];
+          mma_bf16_16816(o[m][i], ah, v.z, v.w);
+          mma_bf16_16816(o[m][i], al, v.x, v.y);
+          mma_bf16_16816(o[m][i], ah, v.x, v.y);
         }
+      }
+      if (ks + AHEAD < KT) {
+#pragma unroll
+        for (int i = 0; i < NT; ++i) s[ks % AHEAD][i] = ws[((size_t)(ks + AHEAD) * (V / 8) + min(nt0 + i, V / 8 - 1)) * 32];
       }
     }
   }
@@ -468,6 +477,16 @@ __global__ void __launch_bounds__(WO_THREADS, 2) wkv_output_kernel(const WkvChun
       ss += __shfl_xor_sync(0xffffffffu, ss, 2);
       if (t4 == 0) sums[warp * WC + m * 16 + g + 8 * (e >> 1)] = ss;
     }
+  uint32_t gates[4][2][NT];
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+#pragma unroll
+    for (int e = 0; e < 2; ++e)
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const int t = m * 16 + g + 8 * e;
+        gates[m][e][i] = t < n && nt0 + i < V / 8 ? *reinterpret_cast<const uint32_t*>(z + (size_t)t * a.ld + 3 * hk + (nt0 + i) * 8 + 2 * t4) : 0u;
+      }
   __syncthreads();
 #pragma unroll
   for (int m = 0; m < 4; ++m)
@@ -483,7 +502,7 @@ __global__ void __launch_bounds__(WO_THREADS, 2) wkv_output_kernel(const WkvChun
       for (int i = 0; i < NT; ++i) {
         const int c = (nt0 + i) * 8 + 2 * t4;
         if (nt0 + i >= V / 8) continue;
-        const float2 gate = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(z + (size_t)t * a.ld + 3 * hk + c));
+        const float2 gate = unpack_bf16x2(gates[m][e >> 1][i]);
         const float2 w = *reinterpret_cast<const float2*>(a.norm + (size_t)h * V + c);
         *reinterpret_cast<uint32_t*>(out + (size_t)t * a.ld_out + c) =
             pack_bf16x2(o[m][i][e] * inv * w.x * gate.x * delta_sigmoid_fast(gate.x), o[m][i][e + 1] * inv * w.y * gate.y * delta_sigmoid_fast(gate.y));
