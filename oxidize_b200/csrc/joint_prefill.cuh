@@ -1,24 +1,30 @@
 // Attention on the scores of all heads together (joint.cuh) for long portions, in three kernels.
 //
-// joint_scores_kernel: capped scores of four heads for 64 tokens per CTA, left as the operand registers that the mixing wants: a
-// high and a low half each, the four heads of a (token, key) in 16 bytes.
+// joint_scores_kernel: scores of four heads for 128 tokens per CTA, products on tcgen05 with the keys as rows: a thread has a key, a
+// warp a tile.  What it caps goes out as the operand registers that the mixing wants: a high and a low half each, the four heads of
+// a (token, key) in 16 bytes.
 // joint_mix_kernel: a warp mixes one token's scores with 32 keys at a time over all heads (hi hi + hi lo + lo hi, float32 sums)
 // and leaves exp2(score - m) in bfloat16, its sum and m, the largest score rounded up to a whole power of two.
-// joint_values_kernel: weights times values, a head and 128 tokens per CTA.  Between tiles with different m the weights are
-// multiplied by powers of two, which rounds nothing.
+// joint_values_kernel: weights times values, a head and 128 tokens per CTA, on tcgen05 with the weights as the operand in tensor
+// memory.  Between tiles with different m they are multiplied by powers of two, which rounds nothing.
 //
-// Weights lie as the last kernel's operand registers want them: of the 32 keys of a tile a lane has 2 t4, 2 t4 + 1 and those
-// 8, 16 and 24 further, 16 bytes in all.
+// Keys and values are the same rows, which come by TMA out of the cache pages: four tiles of 32 keys per place of the scores' ring,
+// two per place of the values'.  Of the 32 keys of a tile a lane of the mixing has 2 t4, 2 t4 + 1 and those 8, 16 and 24 further,
+// 16 bytes of weights in all.
 #pragma once
 #include "joint.cuh"
+#include "latent_mma.cuh"
+#include "latent_prefill.cuh"
 #include "retention.cuh"
 
 namespace oxb {
 
-constexpr int JP_ROWS = 16, JP_KEYS = 32;   // tokens of a block, keys of a tile
-constexpr int JC_WARPS = 8, JC_BLOCKS = 4;  // joint_scores_kernel: a warp has a block and a page of the tile
-constexpr int JM_WARPS = 8, JM_TILES = 8;   // joint_mix_kernel: tiles per warp
-constexpr int JV_WARPS = 8, JV_STAGES = 6;
+constexpr int JP_ROWS = 16, JP_KEYS = 32;  // tokens of a block, keys of a tile
+constexpr int JP_M = 128;                  // tokens of a CTA
+constexpr int JC_PLACE = 128, JC_CHUNK = JC_PLACE * 128, JC_PLACES = 2;  // joint_scores_kernel: keys of a place, bytes of 64 columns
+constexpr int JC_WARPS = 16, JC_THREADS = JC_WARPS * 32 + 64;
+constexpr int JM_WARPS = 8, JM_TILES = 8;  // joint_mix_kernel: tiles per warp
+constexpr int JV_PLACE = 64, JV_CHUNK = JV_PLACE * 128, JV_PLACES = 4, JV_THREADS = 128 + 64;
 constexpr float JP_NONE = -1e30f;  // m of a tile without a visible key
 
 struct JointPrefillArgs {
@@ -64,138 +70,203 @@ struct JointOwn {
   __device__ __forceinline__ int number(int i) const { return i < head ? i : head + i - lo; }  // among the block's own
 };
 
-template <int HD, bool SAME>
-__host__ __device__ constexpr int joint_scores_stages() { return SAME ? 4 : 2; }
-template <int HD, bool SAME>
-__host__ __device__ constexpr int joint_scores_smem() {
-  return 4 * JC_BLOCKS * JP_ROWS * (HD * 2 + 16) + joint_scores_stages<HD, SAME>() * (SAME ? 1 : 4) * JP_KEYS * (HD * 2 + 16) + 2 * 8 * 4;
+// The pages of tiles i .. i + n/2, by number; -1 past the end, where a place keeps what is there.
+struct JointLoader {
+  const JointArgs& a;
+  const JointTiles& all;
+  const int* bt;
+  __device__ __forceinline__ int pages(int i, int most) const {
+    int n = 0;
+    for (int p = 0; p < most; ++p) n += page(i, p) >= 0;
+    return n;
+  }
+  __device__ __forceinline__ int page(int i, int p) const {
+    const int t = i + (p >> 1), n = 2 * all.tile(t) + (p & 1);
+    return t < all.n && n <= all.last_page ? n : -1;
+  }
+  __device__ __forceinline__ int row(int page, int g) const {  // of the cache, in rows of 16 per key head
+    int id = bt[page];
+    if ((unsigned)id >= (unsigned)a.num_blocks) {
+      oxb_report(OXB_BAD_BLOCK_ID, id);
+      id = 0;
+    }
+    return (id * a.G + g) * 16;
+  }
+};
+
+// ----------------------------------------------------------------------------- scores
+__host__ __device__ inline int joint_scores_smem(int W) {  // queries of four heads, keys, factors of the keys (rows of 16 bytes)
+  return (4 * JP_M + JC_PLACES * JC_PLACE) * ((W + 63) / 64) * 128 + JC_PLACES * JC_PLACE * 16 + 1024;
 }
 
-// grid (wide blocks x 2, quads of heads, parts of the tiles).  SAME: the four heads share a key head.
-template <int HD, bool SAME>
-__global__ void __launch_bounds__(JC_WARPS * 32, SAME ? 2 : 1) joint_scores_kernel(const JointPrefillArgs x) {
-  constexpr int ROWB = HD * 2 + 16, PAGE = 16 * ROWB, KS = HD / 16, NK = SAME ? 1 : 4, STAGES = joint_scores_stages<HD, SAME>();
-  constexpr int QROWS = JC_BLOCKS * JP_ROWS, STAGE = 2 * NK * PAGE;
-  extern __shared__ __align__(16) uint8_t jc_smem[];
-  __shared__ int gave_up;
-  pdl_launch_dependents();
+// grid (wide blocks, quads of heads, parts of the tiles).  Sixteen warps cap, one loads, one multiplies.  Tensor memory: tokens
+// 64 s .. 64 s + 63 of head h at 256 s + 64 h.
+static __global__ void __launch_bounds__(JC_THREADS, 1)
+joint_scores_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmT,
+                    const JointPrefillArgs x, const int same) {
+  extern __shared__ uint8_t jc_raw[];
+  __shared__ uint64_t q_full, k_full[JC_PLACES], k_empty[JC_PLACES], t_empty[JC_PLACES], s_full[2], s_empty[2];
+  __shared__ uint32_t tmem_slot;
+  __shared__ volatile int abort_flag;
   const JointArgs& a = x.a;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3, mi = lane >> 3, lr = lane & 7;
-  const int H = a.H, per = H / a.G, quad = blockIdx.y, quads = gridDim.y;
-  const int blk0 = x.wide[2 * (blockIdx.x >> 1)] + (blockIdx.x & 1) * JC_BLOCKS;
-  const int n_blk = min(JC_BLOCKS, x.wide[2 * (blockIdx.x >> 1)] + x.wide[2 * (blockIdx.x >> 1) + 1] - blk0);
-  if (n_blk <= 0) {
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0), lane = threadIdx.x & 31;
+  const int H = a.H, per = H / a.G, quad = blockIdx.y, quads = gridDim.y, chunks = (a.W + 63) / 64;
+  const int blk0 = x.wide[2 * blockIdx.x], n_blk = x.wide[2 * blockIdx.x + 1], b = x.block_seq[blk0], row0 = x.block_row[blk0];
+  const JointTiles all(joint_span(a, b, row0), joint_span(a, b, x.block_row[blk0 + n_blk - 1]));
+  const int places = (all.n + 3) / 4, share = (places + gridDim.z - 1) / gridDim.z;
+  const int u0 = blockIdx.z * share, u1 = min(places, u0 + share);
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(jc_raw) + 1023) & ~uintptr_t(1023));
+  if (u0 >= u1) {
     pdl_wait();
     return;
   }
-  const int b = x.block_seq[blk0], row0 = x.block_row[blk0], qg = warp % JC_BLOCKS, half = warp / JC_BLOCKS;
-  const JointSpan last = joint_span(a, b, x.block_row[blk0 + n_blk - 1]);
-  const JointTiles all(joint_span(a, b, row0), last);
-  const JointOwn own(all, joint_span(a, b, x.block_row[min(blk0 + qg, blk0 + n_blk - 1)]), qg < n_blk);
-  const int share = (all.n + gridDim.z - 1) / gridDim.z, i0 = blockIdx.z * share, i1 = min(all.n, i0 + share);
-  uint8_t *sQ = jc_smem, *ring = sQ + 4 * QROWS * ROWB;  // [4 heads][64] rows; [stages][2 pages][NK]
-  uint64_t *full = reinterpret_cast<uint64_t*>(ring + STAGES * STAGE), *empty = full + STAGES;
-  const int* bt = a.block_tables + (size_t)b * a.max_blocks;
-  const int rows = last.pos0 + last.rows - joint_span(a, b, row0).pos0;
-  if (tid == 0) {
-    gave_up = 0;
-    for (int i = 0; i < STAGES; ++i) {
-      mbar_init(full + i, 1);
-      mbar_init(empty + i, JC_WARPS);
+  if (threadIdx.x == 0) {
+    mbar_init(&q_full, 1);
+    for (int i = 0; i < JC_PLACES; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&k_empty[i], 1);
+      mbar_init(&t_empty[i], JC_WARPS);
     }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&s_full[i], 1);
+      mbar_init(&s_empty[i], JC_WARPS);
+    }
+    abort_flag = 0;
     mbar_fence_init();
   }
-  auto load = [&](int i) {  // by one thread
-    const int k = (i - i0) % STAGES, page = 2 * all.tile(i), pages = page + 1 <= all.last_page ? 2 : 1;
-    mbar_expect_tx(full + k, pages * NK * PAGE);
-    for (int p = 0; p < pages; ++p) {
-      int id = bt[page + p];
-      if ((unsigned)id >= (unsigned)a.num_blocks) {
-        oxb_report(OXB_BAD_BLOCK_ID, id);
-        id = 0;
-      }
-      for (int c = 0; c < NK; ++c)
-        bulk_load(ring + k * STAGE + (p * NK + c) * PAGE,
-                  reinterpret_cast<const uint8_t*>(a.cache) + ((size_t)id * a.G + min(quad * 4 + c, H - 1) / per) * PAGE, PAGE, full + k);
-    }
-  };
-  pdl_wait();
-  if (tid == 0)
-    for (int i = i0; i < i0 + STAGES && i < i1; ++i) load(i);
-  for (int i = tid; i < 4 * QROWS * (HD / 8); i += JC_WARPS * 32) {
-    const int c = i % (HD / 8), r = i / (HD / 8) % QROWS, h = i / (HD / 8) / QROWS;
-    uint8_t* dst = sQ + (h * QROWS + r) * ROWB + c * 16;
-    if (r < rows && quad * 4 + h < H)
-      cp_async16(dst, reinterpret_cast<const __nv_bfloat16*>(a.q) + ((size_t)(row0 + r) * H + quad * 4 + h) * HD + c * 8);
-    else
-      *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);  // (a head past the last has scores of zero)
+  if (warp == JC_WARPS + 1) {
+    tmem_alloc(&tmem_slot, 512);
+    tmem_relinquish();
   }
-  cp_async_commit();
-  cp_async_wait<0>();
+  tc_fence_before();
   __syncthreads();
-  const JointCap cap = joint_cap(a);
-  const uint32_t q_at = smem_u32(sQ) + (qg * JP_ROWS + (mi & 1) * 8 + lr) * ROWB + (mi >> 1) * 16;
-  uint4* dst = x.scores + ((size_t)(blk0 + qg - x.block0) * x.tiles * quads + quad) * (JP_ROWS * JP_KEYS) + g8 * JP_KEYS + half * 16 + 2 * t4;
-  for (int i = i0; i < i1; ++i) {
-    const int k = (i - i0) % STAGES, turn = (i - i0) / STAGES;
-    const int done = i - 1;  // the next tile of its place, once every warp is done with it
-    if (tid == 0 && done >= i0 && done + STAGES < i1) {
-      mbar_wait_bounded(empty + (done - i0) % STAGES, ((done - i0) / STAGES) & 1, &gave_up, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
-      load(done + STAGES);
+  tc_fence_after();
+  pdl_launch_dependents();  // (only now: a CTA of the next kernel must not take the tensor memory that this one still waits for)
+  const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_slot, 0);
+  pdl_wait();
+
+  // item j: place u0 + j / nk, key head j % nk of the quad; it lies in place j % JC_PLACES of the ring
+  const int nk = same ? 1 : 4, items = (u1 - u0) * nk, halves = (n_blk + 3) / 4;
+  uint8_t *sK = smem + 4 * chunks * JP_M * 128, *sT = sK + JC_PLACES * chunks * JC_CHUNK;
+  if (warp == JC_WARPS) {
+    const JointLoader ld{a, all, a.block_tables + (size_t)b * a.max_blocks};
+    const bool leader = elect_one();
+    if (leader) {
+      mbar_expect_tx(&q_full, 4 * chunks * JP_M * 128);
+      for (int h = 0; h < 4; ++h)
+        for (int c = 0; c < chunks; ++c) tma_load_2d(smem + (h * chunks + c) * JP_M * 128, &tmQ, &q_full, (quad * 4 + h) * a.W + c * 64, row0);
     }
-    mbar_wait_bounded(full + k, turn & 1, &gave_up, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
-    if (own.has(i) && 2 * all.tile(i) + half <= all.last_page) {
-      const uint8_t* st = ring + k * STAGE + half * NK * PAGE;
-      const uint32_t k_at = smem_u32(st) + ((mi >> 1) * 8 + lr) * ROWB + (mi & 1) * 16;
-      float s[4][2][4];
-#pragma unroll
-      for (int h = 0; h < 4; ++h)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[h][0][e] = s[h][1][e] = 0.f;
-#pragma unroll
-      for (int ks = 0; ks < KS; ++ks) {
-        uint32_t kb[4];
-        if (SAME) ldmatrix_x4(k_at + ks * 32, kb[0], kb[1], kb[2], kb[3]);
-#pragma unroll
-        for (int h = 0; h < 4; ++h) {
-          uint32_t qa[4];
-          ldmatrix_x4(q_at + h * QROWS * ROWB + ks * 32, qa[0], qa[1], qa[2], qa[3]);
-          if (!SAME) ldmatrix_x4(k_at + h * PAGE + ks * 32, kb[0], kb[1], kb[2], kb[3]);
-          mma_bf16_16816(s[h][0], qa, kb[0], kb[1]);
-          mma_bf16_16816(s[h][1], qa, kb[2], kb[3]);
+    bool ok = true;
+    for (int j = 0; j < items && ok; ++j) {
+      const int s = j % JC_PLACES, turn = j / JC_PLACES, i = 4 * (u0 + j / nk), g = min(quad * 4 + j % nk, H - 1) / per;
+      if (turn > 0)
+        ok = mbar_wait_bounded(&k_empty[s], (turn - 1) & 1, &abort_flag, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x) &&
+             mbar_wait_bounded(&t_empty[s], (turn - 1) & 1, &abort_flag, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      if (leader) {
+        mbar_expect_tx(&k_full[s], ld.pages(i, 8) * (chunks * 2048 + 256));
+        for (int p = 0; p < 8; ++p) {
+          const int page = ld.page(i, p);
+          if (page < 0) continue;
+          const int row = ld.row(page, g);
+          for (int c = 0; c < chunks; ++c) tma_load_2d(sK + (s * chunks + c) * JC_CHUNK + p * 2048, &tmK, &k_full[s], c * 64, row);
+          tma_load_2d(sT + (s * JC_PLACE + p * 16) * 16, &tmT, &k_full[s], a.W / 2, row);  // (coordinates in words)
         }
       }
-      const float* inv = reinterpret_cast<const float*>(st + 2 * t4 * ROWB + HD * 2);
-#pragma unroll
-      for (int h = 0; h < 4; ++h)
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) s[h][nt][e] *= inv[((SAME ? 0 : h) * PAGE + (nt * 8 + (e & 1)) * ROWB) / 4] * cap.factor;
-      if (cap.cap > 0.f) {
-#pragma unroll
-        for (int h = 0; h < 4; ++h)
-#pragma unroll
-          for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) s[h][nt][e] = joint_capped_of(s[h][nt][e], cap);
+      __syncwarp();
+    }
+  } else if (warp == JC_WARPS + 1) {
+    const bool leader = elect_one();
+    constexpr uint32_t idesc = umma_idesc_bf16(JC_PLACE, 64);
+    const uint32_t qa = smem_u32(smem), ka = smem_u32(sK);
+    bool ok = __all_sync(0xffffffffu, mbar_wait_bounded(&q_full, 0, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x));
+    for (int j = 0; j < items && ok; ++j) {
+      const int s = j % JC_PLACES, t = j / nk, heads = same ? 4 : 1, h0 = same ? 0 : j % nk;
+      ok = mbar_wait_bounded(&k_full[s], (j / JC_PLACES) & 1, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+      for (int half = 0; half < halves; ++half) {
+        if (j % nk == 0 && t > 0) ok = mbar_wait_bounded(&s_empty[half], (t - 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x) && ok;
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        tc_fence_after();
+        for (int h = h0; h < h0 + heads; ++h)
+          for (int c = 0; c < chunks; ++c) {
+            const uint32_t qd = umma_desc_lo(qa + (h * chunks + c) * JP_M * 128 + half * 8192), kd = umma_desc_lo(ka + (s * chunks + c) * JC_CHUNK);
+            const int left = min(4, a.W / 16 - 4 * c);
+            for (int k = 0; k < left; ++k)
+              umma_bf16_if<UMMA_DESC_HI_SW128, UMMA_DESC_HI_SW128, idesc>(leader, tmem + 256 * half + 64 * h, kd + 2 * k, qd + 2 * k, k > 0 || c > 0);
+          }
+        if (j % nk == nk - 1) umma_commit_if(leader, &s_full[half]);
       }
-      uint4* to = dst + (size_t)own.number(i) * quads * (JP_ROWS * JP_KEYS);
-#pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {  // row g8 + 8 (e >> 1), key 2 t4 + (e & 1) of tile nt
-          uint4 o;
-          split_bf16x2(s[0][nt][e], s[1][nt][e], o.x, o.z);
-          split_bf16x2(s[2][nt][e], s[3][nt][e], o.y, o.w);
-          to[(e >> 1) * 8 * JP_KEYS + nt * 8 + (e & 1)] = o;
-        }
+      if (ok) umma_commit_if(leader, &k_empty[s]);
     }
     __syncwarp();
-    if (lane == 0) mbar_arrive(empty + k);
+  } else {
+    // ---------------- thread = key, warp = a tile of the place and a block of the half
+    const int quarter = warp & 3, group = warp >> 2;
+    const uint32_t lanes = (uint32_t)(quarter * 32) << 16;
+    const JointCap cap = joint_cap(a);
+    for (int u = u0; u < u1; ++u) {
+      const int t = u - u0, i = 4 * u + quarter;
+      float f[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {  // what the keys' rows are divided by
+        if (c < nk) {
+          const int j = t * nk + c, s = j % JC_PLACES;
+          mbar_wait_bounded(&k_full[s], (j / JC_PLACES) & 1, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
+          __syncwarp();
+          f[c] = *reinterpret_cast<const float*>(sT + (s * JC_PLACE + quarter * 32 + lane) * 16) * cap.factor;
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&t_empty[s]);
+        } else {
+          f[c] = f[0];
+        }
+      }
+      for (int half = 0; half < halves; ++half) {
+        mbar_wait_bounded(&s_full[half], t & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+        __syncwarp();
+        tc_fence_after();
+        const int bi = 4 * half + group;
+        if (bi < n_blk) {
+          const JointOwn own(all, joint_span(a, b, x.block_row[blk0 + bi]), true);
+          if (i < all.n && own.has(i)) {
+            float s[4][16];
+#pragma unroll
+            for (int h = 0; h < 4; ++h) tmem_ld16(tmem + lanes + 256 * half + 64 * h + 16 * group, reinterpret_cast<uint32_t*>(s[h]));
+            tmem_ld_wait();
+            uint4* to = x.scores + (((size_t)(blk0 + bi - x.block0) * x.tiles + own.number(i)) * quads + quad) * (JP_ROWS * JP_KEYS) + lane;
+#pragma unroll
+            for (int k = 0; k < 16; ++k) {
+              float v[4];
+#pragma unroll
+              for (int h = 0; h < 4; ++h) v[h] = s[h][k] * f[h];
+              if (cap.cap > 0.f) {
+#pragma unroll
+                for (int h = 0; h < 4; ++h) v[h] = joint_capped_of(v[h], cap);
+              }
+              uint4 o;
+              split_bf16x2(v[0], v[1], o.x, o.z);
+              split_bf16x2(v[2], v[3], o.y, o.w);
+              to[k * JP_KEYS] = o;
+            }
+          }
+        }
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&s_empty[half]);
+      }
+    }
   }
+  if (abort_flag) {
+    // a wait gave up: give copies that may still be in flight time to land before the CTA exits
+    for (int i = 0; i < 64; ++i) __nanosleep(2000);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == JC_WARPS + 1) tmem_dealloc(tmem, 512);
 }
 
+// ----------------------------------------------------------------------------- mixing
 // grid (blocks x 2, parts of JM_TILES tiles): a warp has a token.  HPW = heads / 16 rounded up.
 template <int HPW>
 __global__ void __launch_bounds__(JM_WARPS * 32, 2) joint_mix_kernel(const JointPrefillArgs x) {
@@ -340,75 +411,111 @@ __global__ void __launch_bounds__(JM_WARPS * 32, 2) joint_mix_kernel(const Joint
   }
 }
 
-__host__ __device__ inline int joint_values_smem(int HD) {
-  return JV_STAGES * JP_KEYS * (HD * 2 + 16) + JV_WARPS * JP_ROWS * 2 * 4 + 2 * JV_STAGES * 8;
-}
+// ----------------------------------------------------------------------------- values
+__host__ __device__ inline int joint_values_smem(int W) { return JV_PLACES * ((W + 63) / 64) * JV_CHUNK + 1024; }
 
 __device__ __forceinline__ float joint_pow2(float e) {  // of a whole number up to 0
   return e < -126.f ? 0.f : __int_as_float(((int)e + 127) << 23);
 }
 
-// grid (wide blocks, H).  A warp has 16 tokens.
-template <int HD>
-__global__ void __launch_bounds__(JV_WARPS * 32, 2) joint_values_kernel(const JointPrefillArgs x) {
-  constexpr int ROWB = HD * 2 + 16, NT = HD / 8, STAGE = JP_KEYS * ROWB;
-  extern __shared__ __align__(16) uint8_t jv_smem[];
-  pdl_launch_dependents();
+// grid (wide blocks, H).  Four warps bring the weights to tensor memory (thread = token), one loads values, one multiplies.  Tensor
+// memory: O at 0, the weights of place u at 128 + 32 (u % 2).
+static __global__ void __launch_bounds__(JV_THREADS, 2)
+joint_values_kernel(const __grid_constant__ CUtensorMap tmV, const JointPrefillArgs x) {
+  extern __shared__ uint8_t jv_raw[];
+  __shared__ uint64_t v_full[JV_PLACES], v_empty[JV_PLACES], p_full[2], pv_done[2];
+  __shared__ uint32_t tmem_slot;
+  __shared__ volatile int abort_flag;
   const JointArgs& a = x.a;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3, mi = lane >> 3, lr = lane & 7;
-  const int H = a.H, h = blockIdx.y, g = h / (H / a.G), blk0 = x.wide[2 * blockIdx.x], n_blk = x.wide[2 * blockIdx.x + 1];
-  const int b = x.block_seq[blk0], last = blk0 + n_blk - 1, blk = min(blk0 + warp, last), row0 = x.block_row[blk];
-  const bool works = warp < n_blk;
-  const JointSpan first = joint_span(a, b, x.block_row[blk0]), end = joint_span(a, b, x.block_row[last]), sp = joint_span(a, b, row0);
-  float* sM = reinterpret_cast<float*>(jv_smem + JV_STAGES * STAGE) + warp * JP_ROWS * 2;  // [16] m of the row, [16] 1 / sum
-  const int* bt = a.block_tables + (size_t)b * a.max_blocks;
-  const JointTiles all(first, end);
-  const JointOwn owned(all, sp, works);
-  const int n_tiles = all.n;
-  uint64_t *full = reinterpret_cast<uint64_t*>(jv_smem + JV_STAGES * STAGE + JV_WARPS * JP_ROWS * 2 * 4), *empty = full + JV_STAGES;
-  __shared__ int gave_up;
-  // tile i of all, both pages, by one thread; places of pages past the portion keep what they hold (zeros, or another tile)
-  auto load = [&](int i) {
-    uint8_t* st = jv_smem + (i % JV_STAGES) * STAGE;
-    const int page = 2 * all.tile(i), pages = page + 1 <= all.last_page ? 2 : 1;
-    mbar_expect_tx(full + i % JV_STAGES, pages * (STAGE / 2));
-    for (int k = 0; k < pages; ++k) {
-      int id = bt[page + k];
-      if ((unsigned)id >= (unsigned)a.num_blocks) {
-        oxb_report(OXB_BAD_BLOCK_ID, id);
-        id = 0;
-      }
-      bulk_load(st + k * (STAGE / 2), reinterpret_cast<const uint8_t*>(a.cache) + ((size_t)id * a.G + g) * (STAGE / 2), STAGE / 2, full + i % JV_STAGES);
-    }
-  };
-  for (int i = tid; i < JV_STAGES * STAGE / 16; i += JV_WARPS * 32) reinterpret_cast<uint4*>(jv_smem)[i] = make_uint4(0, 0, 0, 0);
+  const int warp = __shfl_sync(0xffffffffu, threadIdx.x >> 5, 0);
+  const int H = a.H, h = blockIdx.y, blk0 = x.wide[2 * blockIdx.x], n_blk = x.wide[2 * blockIdx.x + 1], b = x.block_seq[blk0];
+  const JointTiles all(joint_span(a, b, x.block_row[blk0]), joint_span(a, b, x.block_row[blk0 + n_blk - 1]));
+  const int places = (all.n + 1) / 2, chunks = (a.W + 63) / 64;
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(jv_raw) + 1023) & ~uintptr_t(1023));
+  // (places whose pages end early: their rows are multiplied by weights of zero)
+  for (int i = threadIdx.x; i < JV_PLACES * chunks * JV_CHUNK / 16; i += JV_THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-  if (tid == 0) {
-    gave_up = 0;
-    for (int i = 0; i < JV_STAGES; ++i) {
-      mbar_init(full + i, 1);
-      mbar_init(empty + i, JV_WARPS);
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < JV_PLACES; ++i) {
+      mbar_init(&v_full[i], 1);
+      mbar_init(&v_empty[i], 1);
     }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&p_full[i], 128);
+      mbar_init(&pv_done[i], 1);
+    }
+    abort_flag = 0;
     mbar_fence_init();
   }
+  if (warp == 5) {
+    tmem_alloc(&tmem_slot, 256);
+    tmem_relinquish();
+  }
+  tc_fence_before();
   __syncthreads();
+  tc_fence_after();
+  pdl_launch_dependents();  // (only now: a CTA of the next kernel must not take the tensor memory that this one still waits for)
+  const uint32_t tmem = __shfl_sync(0xffffffffu, tmem_slot, 0);
   pdl_wait();
-  if (tid == 0)
-    for (int i = 0; i < JV_STAGES && i < n_tiles; ++i) load(i);
-  // this warp's weights and stats of a tile: 16 rows of 64 bytes, 16 pairs
-  const uint4* weights = x.weights + ((size_t)(blk - x.block0) * x.tiles * H + h) * (JP_ROWS * 4) + t4;
-  const float2* stats = x.stats + ((size_t)(blk - x.block0) * x.tiles * H + h) * JP_ROWS;
-  const int own = sp.kept + sp.hi - sp.lo + 1;
-  if (works) {  // a lane has row lane % 16 and every other tile
+
+  if (warp == 4) {
+    const JointLoader ld{a, all, a.block_tables + (size_t)b * a.max_blocks};
+    const bool leader = elect_one();
+    const int g = h / (H / a.G);
+    bool ok = true;
+    for (int u = 0; u < places && ok; ++u) {
+      const int s = u % JV_PLACES, turn = u / JV_PLACES;
+      if (turn > 0) ok = mbar_wait_bounded(&v_empty[s], (turn - 1) & 1, &abort_flag, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      if (leader) {
+        mbar_expect_tx(&v_full[s], ld.pages(2 * u, 4) * chunks * 2048);
+        for (int p = 0; p < 4; ++p) {
+          const int page = ld.page(2 * u, p);
+          if (page < 0) continue;
+          const int row = ld.row(page, g);
+          for (int c = 0; c < chunks; ++c) tma_load_2d(smem + (s * chunks + c) * JV_CHUNK + p * 2048, &tmV, &v_full[s], c * 64, row);
+        }
+      }
+      __syncwarp();
+    }
+  } else if (warp == 5) {
+    const bool leader = elect_one();
+    const uint32_t idesc = umma_idesc_bf16(JP_M, a.W) | UMMA_B_MN_MAJOR, va = smem_u32(smem);
+    bool ok = true;
+    for (int u = 0; u < places && ok; ++u) {
+      const int s = u % JV_PLACES;
+      ok = mbar_wait_bounded(&v_full[s], (u / JV_PLACES) & 1, &abort_flag, OXB_TIMEOUT_TMA_FULL, blockIdx.x) &&
+           mbar_wait_bounded(&p_full[u & 1], (u >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      tc_fence_after();
+      const uint32_t vd = umma_desc_lo(va + s * chunks * JV_CHUNK, JV_CHUNK);
+#pragma unroll
+      for (int k = 0; k < JV_PLACE / 16; ++k)  // 16 keys: 8 columns of weights, 2 KB of the values
+        umma_bf16_ts_if(leader, tmem, tmem + 128 + 32 * (u & 1) + 8 * k, vd + k * (2048 >> 4), UMMA_DESC_HI_SW128, idesc, u > 0 || k > 0);
+      umma_commit_if(leader, &pv_done[u & 1]);
+      umma_commit_if(leader, &v_empty[s]);
+    }
+    __syncwarp();
+  } else {
+    const int r = threadIdx.x, bi = min(r / JP_ROWS, n_blk - 1), rb = r - bi * JP_ROWS, row0 = x.block_row[blk0 + bi];
+    const uint32_t lanes = (uint32_t)(warp * 32) << 16;
+    const JointSpan sp = joint_span(a, b, row0);
+    const bool on = rb < sp.rows;
+    const JointOwn own(all, sp, on);
+    const size_t at = (size_t)(blk0 + bi - x.block0) * x.tiles * H + h, step = (size_t)H;
+    const uint4* wp = x.weights + at * 64 + (on ? rb : 0) * 4;
+    const float2* mp = x.stats + at * JP_ROWS + (on ? rb : 0);
     const float sink = a.sink != nullptr ? a.sink[h] * 1.4426950408889634f : -INFINITY;
-    const bool on = (lane & 15) < sp.rows;
     float M = sink == -INFINITY ? JP_NONE : ceilf(sink), L = 0.f;
-    for (int i0 = lane >> 4; i0 < own && on; i0 += 16) {
+    const int n_own = on ? sp.kept + sp.hi - sp.lo + 1 : 0;
+    for (int i = 0; i < n_own; i += 8) {
       float2 st[8];
       float top = M;
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        st[j] = i0 + 2 * j < own ? stats[(size_t)(i0 + 2 * j) * H * JP_ROWS + (lane & 15)] : make_float2(JP_NONE, 0.f);
+        st[j] = i + j < n_own ? mp[(size_t)(i + j) * step * JP_ROWS] : make_float2(JP_NONE, 0.f);
         top = fmaxf(top, st[j].x);
       }
       L *= joint_pow2(M - top);
@@ -416,93 +523,81 @@ __global__ void __launch_bounds__(JV_WARPS * 32, 2) joint_values_kernel(const Jo
 #pragma unroll
       for (int j = 0; j < 8; ++j) L = fmaf(st[j].y, joint_pow2(st[j].x - top), L);
     }
-    const float other = __shfl_xor_sync(0xffffffffu, M, 16), top = fmaxf(M, other);
-    L *= joint_pow2(M - top);
-    L += __shfl_xor_sync(0xffffffffu, L, 16);
-    if (sink != -INFINITY) L += exp2f(sink - top);
-    if (lane < JP_ROWS) {
-      sM[lane] = top;
-      sM[JP_ROWS + lane] = L > 0.f ? a.out_scale / L : 0.f;
-    }
-    __syncwarp();
-  }
-  float o[NT][4];
+    if (sink != -INFINITY) L += exp2f(sink - M);
+    struct Fetched {
+      uint4 w[2][4];
+      float m[2];
+    };
+    auto fetch = [&](int u) {  // of the place's two tiles, what is this token's
+      Fetched f;
 #pragma unroll
-  for (int nt = 0; nt < NT; ++nt) o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f;
-  const float M[2] = {works ? sM[g8] : 0.f, works ? sM[g8 + 8] : 0.f};
-  const bool on[2] = {works && g8 < sp.rows, works && g8 + 8 < sp.rows};
-  const uint4* wp = weights + g8 * 4;
-  const float2* mp = stats + g8;
-  const size_t step = (size_t)H * JP_ROWS;
-  uint4 w[2][2];
-  float m[2][2];
-  auto fetch = [&](int i, uint4 (&fw)[2], float (&fm)[2]) {  // of this warp's next tile, if i is one
-    const bool my = owned.has(i);
+      for (int e = 0; e < 2; ++e) {
+        const bool my = own.has(2 * u + e);
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      fw[e] = on[e] && my ? wp[8 * e * 4] : make_uint4(0, 0, 0, 0);
-      fm[e] = on[e] && my ? mp[8 * e].x : JP_NONE;
-    }
-    if (my) {
-      wp += step * 4;
-      mp += step;
-    }
-  };
-  auto multiply = [&](int i, uint4 (&fw)[2], float (&fm)[2]) {
-    const bool my = owned.has(i);
-    uint32_t p[2][4];
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const float f = joint_pow2(fm[e] - M[e]);
-      const __nv_bfloat162 f2 = __floats2bfloat162_rn(f, f);
-      const uint32_t src[4] = {fw[e].x, fw[e].y, fw[e].z, fw[e].w};
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const __nv_bfloat162 y = __hmul2(*reinterpret_cast<const __nv_bfloat162*>(&src[j]), f2);
-        p[e][j] = *reinterpret_cast<const uint32_t*>(&y);
-      }
-    }
-    fetch(i + 2, fw, fm);
-    // (every warp waits, whether the tile is its own or not: none may be a whole turn of the places ahead)
-    mbar_wait_bounded(full + i % JV_STAGES, (i / JV_STAGES) & 1, &gave_up, OXB_TIMEOUT_TMA_FULL, blockIdx.x);
-    if (my) {
-      const uint32_t addr = smem_u32(jv_smem + (i % JV_STAGES) * STAGE) + ((mi & 1) * 8 + lr) * ROWB + (mi >> 1) * 16;
-#pragma unroll
-      for (int ks = 0; ks < 2; ++ks) {
-        const uint32_t av[4] = {p[0][2 * ks], p[1][2 * ks], p[0][2 * ks + 1], p[1][2 * ks + 1]};
-#pragma unroll
-        for (int nt = 0; nt < NT; nt += 2) {
-          uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(addr + ks * 16 * ROWB + nt * 16, b0, b1, b2, b3);
-          mma_bf16_16816(o[nt], av, b0, b1);
-          mma_bf16_16816(o[nt + 1], av, b2, b3);
+        for (int g = 0; g < 4; ++g) f.w[e][g] = my ? wp[g] : make_uint4(0, 0, 0, 0);
+        f.m[e] = my ? mp->x : JP_NONE;
+        if (my) {
+          wp += step * 64;
+          mp += step * JP_ROWS;
         }
       }
+      return f;
+    };
+    Fetched next = fetch(0), after = fetch(1);  // (two places ahead; none is own.has() past the last)
+    for (int u = 0; u < places; ++u) {
+      const Fetched now = next;
+      next = after;
+      after = fetch(u + 2);
+      uint32_t pk[32];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float f = joint_pow2(now.m[e] - M);
+        const __nv_bfloat162 f2 = __floats2bfloat162_rn(f, f);
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          const uint32_t src[4] = {now.w[e][g].x, now.w[e][g].y, now.w[e][g].z, now.w[e][g].w};
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const __nv_bfloat162 y = __hmul2(*reinterpret_cast<const __nv_bfloat162*>(&src[j]), f2);
+            pk[16 * e + 4 * j + g] = *reinterpret_cast<const uint32_t*>(&y);
+          }
+        }
+      }
+      // (no early exit on a failed wait: every thread arrives at every barrier, later waits return at once)
+      if (u > 1) mbar_wait_bounded(&pv_done[u & 1], ((u >> 1) - 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
+      __syncwarp();
+      tc_fence_after();
+      tmem_st16(tmem + lanes + 128 + 32 * (u & 1), pk);
+      tmem_st16(tmem + lanes + 128 + 32 * (u & 1) + 16, pk + 16);
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(&p_full[u & 1]);
     }
+    mbar_wait_bounded(&pv_done[(places - 1) & 1], ((places - 1) >> 1) & 1, &abort_flag, OXB_TIMEOUT_ACCUM, blockIdx.x);
     __syncwarp();
-    if (lane == 0) mbar_arrive(empty + i % JV_STAGES);
-    const int done = i - 2;  // the next tile of its place, once every warp is done with it
-    if (tid == 0 && done >= 0 && done + JV_STAGES < n_tiles) {
-      mbar_wait_bounded(empty + done % JV_STAGES, (done / JV_STAGES) & 1, &gave_up, OXB_TIMEOUT_TMA_EMPTY, blockIdx.x);
-      load(done + JV_STAGES);
+    tc_fence_after();
+    const float inv = L > 0.f ? a.out_scale / L : 0.f;
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (size_t)(row0 + (on ? rb : 0)) * a.ld_out + (size_t)h * a.W;
+    for (int c = 0; c < a.W / 16; ++c) {
+      uint32_t o[16];
+      tmem_ld16(tmem + lanes + 16 * c, o);
+      tmem_ld_wait();
+      if (on) {
+        uint32_t p[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) p[j] = pack_bf16x2(__uint_as_float(o[2 * j]) * inv, __uint_as_float(o[2 * j + 1]) * inv);
+        *reinterpret_cast<uint4*>(out + 16 * c) = make_uint4(p[0], p[1], p[2], p[3]);
+        *reinterpret_cast<uint4*>(out + 16 * c + 8) = make_uint4(p[4], p[5], p[6], p[7]);
+      }
     }
-  };
-  fetch(0, w[0], m[0]);
-  fetch(1, w[1], m[1]);
-  for (int i = 0; i < n_tiles; i += 2) {
-    multiply(i, w[0], m[0]);
-    if (i + 1 < n_tiles) multiply(i + 1, w[1], m[1]);
   }
-  if (!works) return;
-#pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int r = g8 + 8 * e;
-    if (r >= sp.rows) continue;
-    const float inv = sM[JP_ROWS + r];
-    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (size_t)(row0 + r) * a.ld_out + (size_t)h * HD + 2 * t4;
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt) *reinterpret_cast<uint32_t*>(out + nt * 8) = pack_bf16x2(o[nt][2 * e] * inv, o[nt][2 * e + 1] * inv);
+  if (abort_flag) {
+    // a wait gave up: give copies that may still be in flight time to land before the CTA exits
+    for (int i = 0; i < 64; ++i) __nanosleep(2000);
   }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 5) tmem_dealloc(tmem, 256);
 }
 
 }  // namespace oxb

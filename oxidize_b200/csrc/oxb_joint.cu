@@ -121,43 +121,46 @@ OXB_API int oxb_joint_decode(const void* q, void* out, int ld_out, float out_sca
 }
 
 // ----------------------------------------------------------------------------- long portions
-template <int HD, bool SAME>
 static int joint_prefill_go(const JointPrefillArgs& x, int wide_blocks, cudaStream_t stream) {
-  constexpr int scores = joint_scores_smem<HD, SAME>();
-  const int values = joint_values_smem(HD), quads = (x.a.H + 3) / 4;
+  const JointArgs& a = x.a;
+  const int quads = (a.H + 3) / 4, same = a.H / a.G % 4 == 0;
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < 0 || dev >= 64) return (int)cudaErrorInvalidDevice;
   if (!configured[dev]) {
     constexpr cudaFuncAttribute attr = cudaFuncAttributeMaxDynamicSharedMemorySize;
-    cudaError_t e = cudaFuncSetAttribute(joint_scores_kernel<HD, SAME>, attr, scores);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(joint_values_kernel<HD>, attr, values);
+    cudaError_t e = cudaFuncSetAttribute(joint_scores_kernel, attr, joint_scores_smem(128));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(joint_values_kernel, attr, joint_values_smem(128));
     if (e != cudaSuccess) return (int)e;
     configured[dev] = true;
   }
-  // the tiles of 64 tokens are dealt out to as many CTAs as run at once
-  int parts = 2 * oxb_sm_count() / (2 * wide_blocks * quads);
-  if (parts > x.tiles / 4) parts = x.tiles / 4;
+  CUtensorMap tq, tk, tt;
+  const uint64_t rows = (uint64_t)a.num_blocks * a.G * 16, pitch = (uint64_t)(a.W + a.tail) * 2;
+  int e = oxb_make_tmap_2d(&tq, a.q, a.T, (uint64_t)a.H * a.W, (uint64_t)a.H * a.W * 2, JP_M, 64, 2);
+  if (e == 0) e = oxb_make_tmap_2d(&tk, a.cache, rows, a.W + a.tail, pitch, 16, 64, 2);
+  if (e == 0) e = oxb_make_tmap_bytes(&tt, a.cache, rows, pitch, 16, 16);
+  if (e) return e;
+  // the tiles of 128 tokens are dealt out to as many CTAs as run at once
+  int parts = oxb_sm_count() / (wide_blocks * quads);
+  if (parts > x.tiles / 16) parts = x.tiles / 16;
   if (parts < 1) parts = 1;
   const dim3 mix((unsigned)x.blocks * 2, (x.tiles + JM_TILES - 1) / JM_TILES);
-  cudaError_t e = oxb_launch(joint_scores_kernel<HD, SAME>, dim3(2 * wide_blocks, quads, parts), dim3(JC_WARPS * 32), (size_t)scores, stream, x);
-  if (e == cudaSuccess)
-    e = x.a.H <= 16 ? oxb_launch(joint_mix_kernel<1>, mix, dim3(JM_WARPS * 32), 0, stream, x)
-                    : oxb_launch(joint_mix_kernel<2>, mix, dim3(JM_WARPS * 32), 0, stream, x);
-  if (e == cudaSuccess) e = oxb_launch(joint_values_kernel<HD>, dim3(wide_blocks, x.a.H), dim3(JV_WARPS * 32), (size_t)values, stream, x);
-  if (e != cudaSuccess) return (int)e;
+  cudaError_t le = oxb_launch(joint_scores_kernel, dim3(wide_blocks, quads, parts), dim3(JC_THREADS), (size_t)joint_scores_smem(a.W),
+                              stream, tq, tk, tt, x, same);
+  if (le == cudaSuccess)
+    le = a.H <= 16 ? oxb_launch(joint_mix_kernel<1>, mix, dim3(JM_WARPS * 32), 0, stream, x)
+                   : oxb_launch(joint_mix_kernel<2>, mix, dim3(JM_WARPS * 32), 0, stream, x);
+  if (le == cudaSuccess)
+    le = oxb_launch(joint_values_kernel, dim3(wide_blocks, a.H), dim3(JV_THREADS), (size_t)joint_values_smem(a.W), stream, tk, x);
+  if (le != cudaSuccess) return (int)le;
   OXB_CHECK_LAUNCH();
   return 0;
-}
-template <int HD>
-static int joint_prefill_heads(const JointPrefillArgs& x, int wide_blocks, cudaStream_t stream) {
-  return x.a.H / x.a.G % 4 == 0 ? joint_prefill_go<HD, true>(x, wide_blocks, stream) : joint_prefill_go<HD, false>(x, wide_blocks, stream);
 }
 
 // 1 when the kernels for long portions cover these heads (bf16, pages of 16 tokens)
 OXB_API int oxb_joint_prefill_supported(int H, int G, int W) {
-  return (W == 32 || W == 64 || W == 96 || W == 128) && G > 0 && H % G == 0 && H <= 32;
+  return W >= 16 && W <= 128 && W % 16 == 0 && G > 0 && H % G == 0 && H <= 32;
 }
 
 // The same in bf16 on pages of 16 tokens for the given blocks of 16 tokens (block0 .. block0 + blocks, of long portions), which
@@ -173,17 +176,12 @@ OXB_API int oxb_joint_prefill(const void* q, void* out, int ld_out, float out_sc
   if (T <= 0 || B <= 0 || blocks <= 0 || wide_blocks <= 0) return 0;
   const JointArgs a{q, out, ld_out, out_scale, cache, block_tables, seq_lens, query_start, sink, mix, bias, distances,
                     B, max_blocks, T, H, G, W, tail, page, num_blocks, window, keep_first, scale, cap, 0};
-  if (joint_check(a) || !oxb_joint_prefill_supported(H, G, W) || page != 16 || tail != 8 || tiles <= 0 || ld_out % 2 != 0 ||
-      (reinterpret_cast<uintptr_t>(out) & 3) != 0 ||
+  if (joint_check(a) || !oxb_joint_prefill_supported(H, G, W) || page != 16 || tail != 8 || tiles <= 0 || ld_out % 8 != 0 ||
+      (reinterpret_cast<uintptr_t>(out) & 15) != 0 ||
       ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(scores) | reinterpret_cast<uintptr_t>(weights) |
         reinterpret_cast<uintptr_t>(stats)) & 15) != 0)
     return (int)cudaErrorInvalidValue;
   const JointPrefillArgs x{a, block_seq, block_row, wide, reinterpret_cast<uint4*>(scores), reinterpret_cast<uint4*>(weights),
                            reinterpret_cast<float2*>(stats), tiles, block0, blocks};
-  switch (W) {
-    case 32: return joint_prefill_heads<32>(x, wide_blocks, stream);
-    case 64: return joint_prefill_heads<64>(x, wide_blocks, stream);
-    case 96: return joint_prefill_heads<96>(x, wide_blocks, stream);
-    default: return joint_prefill_heads<128>(x, wide_blocks, stream);
-  }
+  return joint_prefill_go(x, wide_blocks, stream);
 }
