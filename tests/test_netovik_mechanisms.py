@@ -547,7 +547,7 @@ def test_key_splits_of_a_decoded_token(H, G, d, splits):
 
 
 @gpu
-@pytest.mark.parametrize("H,G,d,window,keep", [(32, 8, 128, 200, 4), (32, 32, 64, 0, 0), (6, 6, 48, 128, 40), (17, 17, 32, 90, 7)])
+@pytest.mark.parametrize("H,G,d,window,keep", [(32, 8, 128, 200, 4), (32, 32, 64, 0, 0), (6, 6, 80, 128, 40), (17, 17, 32, 90, 7), (9, 3, 16, 50, 1)])
 def test_long_portions_in_several_launches(H, G, d, window, keep):
     """Scratch for few blocks at a time, portions of two sequences behind what earlier steps left, against the plain kernel."""
     spec = joint_spec(H, G, d, window, keep, rows=32, far=128)
